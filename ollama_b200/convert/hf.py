@@ -25,6 +25,7 @@ from ..gguf import quants
 from ..gguf.types import GGMLType
 from ..gguf.writer import WriteTensor, write_gguf
 from .safetensors import ModelDir
+from .stack import is_stack_config, stack_kv, stack_tensors
 
 
 class ConvertError(ValueError):
@@ -528,24 +529,39 @@ def _order(name: str) -> tuple:
     return (1, int(m.group(1)), m.group(2)) if m else (0, 0, name)
 
 
+def checkpoint_parts(path: str, cfg: dict[str, Any], outtype: str = "auto",
+                     progress: Callable[[str], None] | None = None) -> tuple[dict[str, Any], list[WriteTensor]]:
+    """Metadata and tensors of the checkpoint directory ``path`` with configuration ``cfg``, in GGUF terms."""
+    name = os.path.basename(os.path.normpath(path))
+    stack = is_stack_config(cfg)
+    archs = cfg.get("architectures") or []
+    if not stack and (not archs or archs[0] not in ARCHS):
+        raise ConvertError(f"unsupported architecture {cfg.get('architecture') or (archs[0] if archs else '(none)')}")
+    src = ModelDir(path)
+    try:
+        if stack:
+            kv = stack_kv(cfg, name)
+            if any(os.path.exists(os.path.join(path, n)) for n in ("tokenizer.json", "tokenizer.model")):
+                kv.update(tokenizer_kv(path, cfg["vocab"]))
+            tensors = list(stack_tensors(src, cfg, outtype, progress))
+        else:
+            arch = ARCHS[archs[0]]
+            kv = _kv(cfg, arch, name)
+            kv.update(tokenizer_kv(path, kv.get(f"{arch}.vocab_size", 0)))
+            tensors = list(convert_tensors(src, cfg, arch, outtype, progress))
+        types = {t.dtype for t in tensors if len(t.shape) >= 2}
+        kv["general.file_type"] = 32 if GGMLType.BF16 in types else 1 if GGMLType.F16 in types else 0
+    finally:
+        src.close()
+    return kv, tensors
+
+
 def convert_hf(path: str, out_path: str, outtype: str = "auto", progress: Callable[[str], None] | None = None) -> dict[str, Any]:
     """Convert the checkpoint directory ``path`` into the GGUF file ``out_path``; returns the metadata written."""
     with open(os.path.join(path, "config.json"), encoding="utf-8") as f:
         cfg = json.load(f)
-    archs = cfg.get("architectures") or []
-    if not archs or archs[0] not in ARCHS:
-        raise ConvertError(f"unsupported architecture {archs[0] if archs else '(none)'}")
-    arch = ARCHS[archs[0]]
-    src = ModelDir(path)
-    try:
-        kv = _kv(cfg, arch, os.path.basename(os.path.normpath(path)))
-        kv.update(tokenizer_kv(path, kv.get(f"{arch}.vocab_size", 0)))
-        tensors = list(convert_tensors(src, cfg, arch, outtype, progress))
-        types = {t.dtype for t in tensors if len(t.shape) >= 2}
-        kv["general.file_type"] = 32 if GGMLType.BF16 in types else 1 if GGMLType.F16 in types else 0
-        write_gguf(out_path, kv, tensors)
-    finally:
-        src.close()
+    kv, tensors = checkpoint_parts(path, cfg, outtype, progress)
+    write_gguf(out_path, kv, tensors)
     return kv
 
 

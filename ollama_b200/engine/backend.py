@@ -7,6 +7,7 @@ portable implementation (reference graph, any torch device); the sm_100a engine 
 """
 from __future__ import annotations
 
+import os
 from typing import Protocol, Sequence
 
 import torch
@@ -114,6 +115,10 @@ class TorchBackend:
 
 
 def open_model(path: str) -> GGUFFile:
+    """A GGUF file, or a checkpoint directory (config.json + safetensors) read through the converter."""
+    if os.path.isdir(path):
+        from ..convert.folder import open_folder
+        return normalise(open_folder(path))
     return normalise(open_gguf(path))
 
 
@@ -122,9 +127,17 @@ def make_backend(g: GGUFFile, device: str = "auto", adapters: Sequence[str] = ()
     ``adapters``: LoRA adapter files merged into the weights at load time."""
     if device == "auto":
         device = "cuda" if torch.cuda.is_available() else "cpu"
+    cfg = config_from_gguf(g)
+    if cfg.stack is not None:
+        from .stack import StackBackend
+        if not device.startswith("cuda"):
+            raise NotImplementedError(f"{cfg.arch} runs on the sm_100a engine only")
+        if adapters:
+            raise NotImplementedError(f"{cfg.arch} takes no adapters")
+        return StackBackend(g, device=device, cfg=cfg, **kw)
     if device.startswith("cuda"):
         from .b200 import B200Backend, supports
-        if supports(config_from_gguf(g)):
+        if supports(cfg):
             if adapters:
                 from ..models.lora import LoraTensors
                 src = LoraTensors(g, adapters)

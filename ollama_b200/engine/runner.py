@@ -43,6 +43,7 @@ class RunnerOptions:
     adapter_paths: tuple = ()         # LoRA adapter files merged into the weights at load time (Modelfile ADAPTER)
     draft_path: str = ""              # a smaller model of the same vocabulary that drafts tokens (Modelfile DRAFT)
     draft_num_predict: int = 4        # tokens drafted per verification pass (api/types.go:1119)
+    dtype: str = "bfloat16"           # compute type of models that also run in 32 bits ("float32")
     shift_mode: str = "rotate"        # context shift: "rotate" re-rotates the cached keys in place, "recompute" evaluates the kept tokens again
 
 

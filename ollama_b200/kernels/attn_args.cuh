@@ -15,6 +15,10 @@ struct AttnDecodeArgs {
     float2* part_ml;         // scratch [nb][H][splits] (max, sum)
     const __half* k_scale;   // q8_0 cache (k_cache / v_cache hold int8): [slots][Hkv][n_ctx][HD/32] scales, or null for f16
     const __half* v_scale;
+    // paged cache (page_table set; tensor-core kernel only): caches are [page][Hkv][64][HD], n_ctx and the scales are not used
+    const int* page_table;   // [slots][max_pages]
+    int max_pages;
+    int chunk;               // > 0: position p sees the keys from floor(p / chunk) * chunk on
 };
 
 // Optional second argument of the tensor-core kernel: with `qkv` set the kernel takes the query rows straight from the
@@ -26,6 +30,48 @@ struct AttnRopeArgs {
     const float* inv_freq;   // [n_rot / 2]
     float mscale;
     int n_rot, neox;
+    // paged form: heads of dim / vdim columns inside rows of pitch ldq (the cache rows are padded to HD), RMS norms over the whole
+    // q and k projections (or null), rotation in the half-split order with frequencies in double
+    const float* q_norm;     // [H * dim]
+    const float* k_norm;     // [Hkv * dim]
+    float eps;
+    int ldq, dim, vdim;
+    const double* freqs;     // [n_rot / 2]
+};
+
+// Rows of a step over a paged cache: see attn_paged.cu.
+struct PagedAppendArgs {
+    const float* qkv;        // [rows][ldq]: q heads | k heads | v heads
+    int ldq, n_heads, n_kv_heads, dim, vdim;
+    const float* q_norm;     // [H * dim], or null with k_norm
+    const float* k_norm;     // [Hkv * dim]
+    float eps;
+    const double* freqs;     // [n_rot / 2]
+    int n_rot;
+    const int* positions;    // [rows]
+    const int* slots;        // [rows]
+    const int* page_table;   // [slots][max_pages]
+    int max_pages;
+    float* q_out;            // [rows][H][dq]
+    int dq;
+    void* k_cache;           // [pages][Hkv][64][dk]
+    void* v_cache;           // [pages][Hkv][64][dv]
+    int dk, dv, cache32;     // cache32: fp32 caches, else f16
+};
+
+struct PagedAttnArgs {
+    const float* q;          // [rows][H][dq]
+    int dq, n_heads, n_kv_heads, dim, vdim;
+    const void* k_cache;
+    const void* v_cache;
+    int dk, dv, cache32;
+    const int* positions;
+    const int* slots;
+    const int* page_table;
+    int max_pages, chunk;
+    float scale, softcap;
+    void* out;               // [rows][ldo], head h at column h * vdim
+    int ldo, out16;
 };
 
 // Tensor-core variant (attn_decode_mma.cu): same partial outputs, so the same combine kernel follows.

@@ -10,7 +10,10 @@
 // every tile and keeps its own running soft-max statistics and output accumulator, the four warps are merged
 // through shared memory at the end.  The scalar kernel stays the choice for short contexts and for head
 // sizes without an instantiation here.
+// The paged form (PAGED) reads its tiles through a page table (a tile of 64 positions is a page), starts at the query's chunk
+// instead of a sliding window, and normalises q and k over their whole projections before the rotation.
 #include "attn_args.cuh"
+#include "rows.cuh"
 
 namespace {
 
@@ -35,7 +38,7 @@ __device__ __forceinline__ uint32_t pack_half2(float a, float b) {
     return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-template <int D, int NS>
+template <int D, int NS, bool PAGED>
 __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_constant__ AttnDecodeArgs a, const __grid_constant__ AttnRopeArgs r) {
     constexpr int LD = D + PAD;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -54,11 +57,12 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
     pdl_wait();
     const int qpos = a.positions[b], slot = a.slots[b];
     const int kv_len = qpos + 1;
-    const int start = (a.window > 0 && kv_len > a.window) ? kv_len - a.window : 0;
-    const int span = kv_len - start;
+    const int start = a.chunk > 0 ? qpos - qpos % a.chunk : (a.window > 0 && kv_len > a.window) ? kv_len - a.window : 0;
+    const int base = PAGED ? start & ~(BN - 1) : start;         // paged: tiles begin at page borders
+    const int span = kv_len - base;
     int chunk = (span + a.n_splits - 1) / a.n_splits;
     chunk = ((chunk + BN - 1) / BN) * BN;
-    const int p0 = start + split * chunk, p1 = min(p0 + chunk, kv_len);
+    const int p0 = base + split * chunk, p1 = min(p0 + chunk, kv_len);
     const int n_tiles = p1 > p0 ? (p1 - p0 + BN - 1) / BN : 0;
     const size_t row0 = ((size_t)slot * a.n_kv_heads + kvh) * a.n_ctx;      // first cache row of this (slot, kv head)
 
@@ -66,6 +70,16 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         const int n0 = p0 + tile * BN;
         __half* dk = sK + stage * BN * LD;
         __half* dv = sV + stage * BN * LD;
+        if (PAGED) {
+            const size_t r0 = paged_row(a.page_table + (size_t)slot * a.max_pages, n0, a.n_kv_heads, kvh);
+            for (int c = tid; c < BN * (D / 8); c += 128) {
+                const int r = c / (D / 8), col = (c % (D / 8)) * 8;
+                cp_async16(dk + r * LD + col, a.k_cache + (r0 + r) * D + col);
+                cp_async16(dv + r * LD + col, a.v_cache + (r0 + r) * D + col);
+            }
+            asm volatile("cp.async.commit_group;" ::: "memory");
+            return;
+        }
         if (a.k_scale) {      // q8_0 cache: plain loads, expanded to f16 on the way into shared memory
             const int8_t* kq = reinterpret_cast<const int8_t*>(a.k_cache) + row0 * D;
             const int8_t* vq = reinterpret_cast<const int8_t*>(a.v_cache) + row0 * D;
@@ -125,8 +139,43 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         // the raw rows (query heads of this group, the key and the value) are staged in the last K stage, which stays unused
         // until the tile loop requests tile NS - 1; cos / sin of the position are computed once per CTA meanwhile
         float* raw = reinterpret_cast<float*>(sK + (NS - 1) * BN * LD);       // [group + 2][D]
-        const float* tok = r.qkv + (size_t)b * (a.n_heads + 2 * a.n_kv_heads) * D;
         const int nrows = group + (owner ? 2 : 0);
+        if (PAGED) {
+            const float* tok = r.qkv + (size_t)b * r.ldq;
+            const int nq = a.n_heads * r.dim, nk = a.n_kv_heads * r.dim;
+            float iq = 1.f, ik = 1.f;
+            if (r.q_norm) {
+                float s0 = 0.f, s1 = 0.f;
+                for (int i = tid; i < nq; i += 128) s0 += tok[i] * tok[i];
+                if (owner)
+                    for (int i = tid; i < nk; i += 128) s1 += tok[nq + i] * tok[nq + i];
+                s0 = warp_sum(s0);
+                s1 = warp_sum(s1);
+                if (lane == 0) {
+                    s_m[warp][0] = s0;
+                    s_l[warp][0] = s1;
+                }
+                __syncthreads();
+                iq = 1.f / sqrtf((s_m[0][0] + s_m[1][0] + s_m[2][0] + s_m[3][0]) / (float)nq + r.eps);
+                ik = 1.f / sqrtf((s_l[0][0] + s_l[1][0] + s_l[2][0] + s_l[3][0]) / (float)nk + r.eps);
+            }
+            for (int c = tid; c < nrows * D; c += 128) {
+                const int rr = c / D, col = c % D;
+                float v = 0.f;
+                if (rr <= group) {
+                    if (col < r.dim) {
+                        const int i = rr < group ? (head0 + rr) * r.dim + col : kvh * r.dim + col;
+                        v = tok[rr < group ? i : nq + i];
+                        if (r.q_norm) v *= rr < group ? iq * r.q_norm[i] : ik * r.k_norm[i];
+                    }
+                } else if (col < r.vdim) {
+                    v = tok[nq + nk + kvh * r.vdim + col];
+                }
+                raw[c] = v;
+            }
+            for (int p = tid; p < (r.n_rot >> 1); p += 128) sincosf(rot_angle(qpos, r.freqs[p]), &s_sn[p], &s_cs[p]);
+        } else {
+        const float* tok = r.qkv + (size_t)b * (a.n_heads + 2 * a.n_kv_heads) * D;
         for (int c = tid; c < nrows * (D / 4); c += 128) {
             const int rr = c / (D / 4), col = (c % (D / 4)) * 4;
             const float* src = rr < group ? tok + (size_t)(head0 + rr) * D
@@ -139,12 +188,14 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
             s_sn[p] = sn * r.mscale;
             s_cs[p] = cs * r.mscale;
         }
+        }
         __syncthreads();
         if (owner) {      // append the new key / value rows to the cache and keep them for the last tile
             const float* krow = raw + group * D;
             const float* vrow = raw + (group + 1) * D;
-            __half* kc = const_cast<__half*>(a.k_cache) + (row0 + qpos) * D;
-            __half* vc = const_cast<__half*>(a.v_cache) + (row0 + qpos) * D;
+            const size_t own = PAGED ? paged_row(a.page_table + (size_t)slot * a.max_pages, qpos, a.n_kv_heads, kvh) : row0 + qpos;
+            __half* kc = const_cast<__half*>(a.k_cache) + own * D;
+            __half* vc = const_cast<__half*>(a.v_cache) + own * D;
             for (int i = tid; i < D; i += 128) {
                 const __half kh = __float2half_rn(rotated(krow, i)), vh = __float2half_rn(vrow[i]);
                 s_newk[i] = kh;
@@ -215,7 +266,10 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
 #pragma unroll
         for (int j = 0; j < 2; j++) {
 #pragma unroll
-            for (int e = 0; e < 2; e++) ok[j][e] = n0 + 8 * j + 2 * tq + e < p1;
+            for (int e = 0; e < 2; e++) {
+                const int kp = n0 + 8 * j + 2 * tq + e;
+                ok[j][e] = kp < p1 && (!PAGED || kp >= start);
+            }
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 float v = s[j][e] * a.scale;
@@ -302,11 +356,11 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
     }
 }
 
-template <int D, int NS>
+template <int D, int NS, bool PAGED>
 int launch(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int pdl, cudaStream_t st) {
     constexpr int SMEM = (ROWS + 2 * NS * BN) * (D + PAD) * 2;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(attn_decode_mma_kernel<D, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    if (once.first()) cudaFuncSetAttribute(attn_decode_mma_kernel<D, NS, PAGED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(a.n_splits, a.n_kv_heads, nb);
     cfg.blockDim = dim3(128);
@@ -320,7 +374,7 @@ int launch(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int pdl, cuda
     AttnDecodeArgs copy = a;
     AttnRopeArgs rcopy = r;
     void* args[] = {&copy, &rcopy};
-    return (int)cudaLaunchKernelExC(&cfg, (const void*)attn_decode_mma_kernel<D, NS>, args);
+    return (int)cudaLaunchKernelExC(&cfg, (const void*)attn_decode_mma_kernel<D, NS, PAGED>, args);
 }
 
 int g_stages = 0;      // 0: by the size of the launch; 2, 3 or 4: forced (tests)
@@ -344,18 +398,17 @@ int stages_for(const AttnDecodeArgs& a, int nb) {
 
 template <int D>
 int launch_d(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int pdl, cudaStream_t st) {
-    switch (stages_for(a, nb)) {
-        case 4: return launch<D, 4>(a, r, nb, pdl, st);
-        case 3: return launch<D, 3>(a, r, nb, pdl, st);
-        default: return launch<D, 2>(a, r, nb, pdl, st);
-    }
+    const int ns = stages_for(a, nb);
+    if (a.page_table) return ns == 4 ? launch<D, 4, true>(a, r, nb, pdl, st) : ns == 3 ? launch<D, 3, true>(a, r, nb, pdl, st) : launch<D, 2, true>(a, r, nb, pdl, st);
+    return ns == 4 ? launch<D, 4, false>(a, r, nb, pdl, st) : ns == 3 ? launch<D, 3, false>(a, r, nb, pdl, st) : launch<D, 2, false>(a, r, nb, pdl, st);
 }
 
 }  // namespace
 
 int attn_decode_mma_rope_launch(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int hd, int pdl, cudaStream_t st) {
     if (a.n_kv_heads < 1 || a.n_heads % a.n_kv_heads || a.n_heads / a.n_kv_heads > ROWS) return (int)cudaErrorNotSupported;
-    if (r.qkv && (a.k_scale || a.v_scale || r.n_rot > 256 || r.n_rot > hd || (r.n_rot & 1) || !r.inv_freq)) return (int)cudaErrorNotSupported;
+    if (r.qkv && (a.k_scale || a.v_scale || r.n_rot > 256 || r.n_rot > hd || (r.n_rot & 1) || (a.page_table ? r.n_rot && !r.freqs : !r.inv_freq))) return (int)cudaErrorNotSupported;
+    if (a.page_table && (!r.qkv || !r.neox || r.dim < 1 || r.dim > hd || r.vdim < 1 || r.vdim > hd || r.n_rot > r.dim || a.max_pages < 1)) return (int)cudaErrorInvalidValue;
     if (hd == 128) return launch_d<128>(a, r, nb, pdl, st);
     if (hd == 64) return launch_d<64>(a, r, nb, pdl, st);
     return (int)cudaErrorNotSupported;

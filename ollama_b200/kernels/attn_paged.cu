@@ -1,0 +1,230 @@
+// Attention over a paged cache: preparation of a batch of rows, an attention kernel for any head size and for 32-bit models, and
+// the entry points of the tensor-core kernels' paged forms (attn_decode_mma.cu, attn_prefill_tc.cu).
+//
+// Cache layout per layer run: K [page][kv head][64 positions][dk], V [page][kv head][64 positions][dv]; page_table[slot][i]
+// is the page that holds positions 64 i .. 64 i + 63 of the slot.  dk and dv are the padded row lengths (pad columns are zero).
+//
+// Chunked masks: with chunk > 0 the query at position p sees the keys floor(p / chunk) * chunk .. p.
+#include "attn_args.cuh"
+#include "rows.cuh"
+
+namespace {
+
+// ---------------------------------------------------------------------------------------------------------------------
+// RMS norm of q and k over their whole projections, rotary embedding, q to padded fp32 rows, k and v into the cache.
+// One CTA per row.
+// ---------------------------------------------------------------------------------------------------------------------
+template <typename CT>
+__global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant__ PagedAppendArgs a) {
+    extern __shared__ float sm[];
+    __shared__ float red[2][8];
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nq = a.n_heads * a.dim, nk = a.n_kv_heads * a.dim, half = a.n_rot >> 1;
+    float* sq = sm;                // [nq + nk]
+    float* cs = sm + nq + nk;      // [half], then sines
+    float* sn = cs + half;
+    pdl_launch();
+    pdl_wait();
+    const int pos = a.positions[t], slot = a.slots[t];
+    const float* row = a.qkv + (size_t)t * a.ldq;
+    float s0 = 0.f, s1 = 0.f;
+    for (int i = tid; i < nq + nk; i += 256) {
+        const float v = row[i];
+        sq[i] = v;
+        if (i < nq) s0 += v * v;
+        else s1 += v * v;
+    }
+    for (int p = tid; p < half; p += 256) {
+        float s, c;
+        sincosf(rot_angle(pos, a.freqs[p]), &s, &c);
+        cs[p] = c;
+        sn[p] = s;
+    }
+    s0 = warp_sum(s0);
+    s1 = warp_sum(s1);
+    if (lane == 0) {
+        red[0][warp] = s0;
+        red[1][warp] = s1;
+    }
+    __syncthreads();
+    float iq = 1.f, ik = 1.f;
+    if (a.q_norm) {
+        s0 = s1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            s0 += red[0][i];
+            s1 += red[1][i];
+        }
+        iq = 1.f / sqrtf(s0 / (float)nq + a.eps);
+        ik = 1.f / sqrtf(s1 / (float)nk + a.eps);
+    }
+    auto normed = [&](int i) -> float {
+        const float v = sq[i];
+        if (!a.q_norm) return v;
+        return i < nq ? v * iq * a.q_norm[i] : v * ik * a.k_norm[i - nq];
+    };
+    auto rotated = [&](int base, int d) -> float {
+        const float x = normed(base + d);
+        if (d >= a.n_rot) return x;
+        const bool first = d < half;
+        const int p = first ? d : d - half;
+        const float y = normed(base + (first ? d + half : p));
+        return first ? x * cs[p] - y * sn[p] : x * cs[p] + y * sn[p];
+    };
+    float* qo = a.q_out + (size_t)t * a.n_heads * a.dq;
+    for (int i = tid; i < a.n_heads * a.dq; i += 256) {
+        const int h = i / a.dq, d = i - h * a.dq;
+        qo[i] = d < a.dim ? rotated(h * a.dim, d) : 0.f;
+    }
+    const int* table = a.page_table + (size_t)slot * a.max_pages;
+    CT* kc = (CT*)a.k_cache;
+    CT* vc = (CT*)a.v_cache;
+    for (int i = tid; i < a.n_kv_heads * a.dk; i += 256) {
+        const int g = i / a.dk, d = i - g * a.dk;
+        kc[paged_row(table, pos, a.n_kv_heads, g) * a.dk + d] = from_f<CT>(d < a.dim ? rotated(nq + g * a.dim, d) : 0.f);
+    }
+    for (int i = tid; i < a.n_kv_heads * a.dv; i += 256) {
+        const int g = i / a.dv, d = i - g * a.dv;
+        vc[paged_row(table, pos, a.n_kv_heads, g) * a.dv + d] = from_f<CT>(d < a.vdim ? row[nq + nk + g * a.vdim + d] : 0.f);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// Any head size, fp16 or fp32 cache.  One CTA per (row, head), keys in tiles of 128: a thread scores one key, the
+// softmax statistics are merged across the CTA, then the threads own value columns.  The kernel of 32-bit models, and of
+// head sizes the tensor-core kernels do not take.
+// ---------------------------------------------------------------------------------------------------------------------
+constexpr int VCOLS = 4;      // value columns per thread: value heads up to 512
+
+template <typename CT, typename OT>
+__global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__ PagedAttnArgs a) {
+    extern __shared__ float sq[];      // [dim]
+    __shared__ float sp[128];
+    __shared__ float red[2][4];
+    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    pdl_launch();
+    pdl_wait();
+    const int pos = a.positions[t], slot = a.slots[t], g = h / (a.n_heads / a.n_kv_heads);
+    const int* table = a.page_table + (size_t)slot * a.max_pages;
+    const float* q = a.q + ((size_t)t * a.n_heads + h) * a.dq;
+    for (int i = tid; i < a.dim; i += 128) sq[i] = q[i];
+    __syncthreads();
+    const int lo = a.chunk > 0 ? pos - pos % a.chunk : 0;
+    float acc[VCOLS] = {}, m = -INFINITY, l = 0.f;
+    for (int k0 = lo; k0 <= pos; k0 += 128) {
+        const int kp = k0 + tid;
+        float s = -INFINITY;
+        if (kp <= pos) {
+            const CT* kr = (const CT*)a.k_cache + paged_row(table, kp, a.n_kv_heads, g) * a.dk;
+            float d = 0.f;
+            for (int i = 0; i < a.dim; i++) d = fmaf(sq[i], to_f(kr[i]), d);
+            s = d * a.scale;
+            if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+        }
+        float mx = warp_max(s);
+        if (lane == 0) red[0][warp] = mx;
+        __syncthreads();
+        mx = fmaxf(fmaxf(red[0][0], red[0][1]), fmaxf(red[0][2], red[0][3]));
+        const float mn = fmaxf(m, mx);
+        const float corr = expf(m - mn);      // the first tile always holds a visible key, so mn is finite
+        const float p = expf(s - mn);
+        sp[tid] = p;
+        const float ps = warp_sum(p);
+        if (lane == 0) red[1][warp] = ps;
+        __syncthreads();
+        l = l * corr + red[1][0] + red[1][1] + red[1][2] + red[1][3];
+        m = mn;
+        const int n = min(128, pos - k0 + 1);
+#pragma unroll
+        for (int j = 0; j < VCOLS; j++) acc[j] *= corr;
+        for (int i = 0; i < n; i++) {
+            const CT* vr = (const CT*)a.v_cache + paged_row(table, k0 + i, a.n_kv_heads, g) * a.dv;
+            const float w = sp[i];
+#pragma unroll
+            for (int j = 0; j < VCOLS; j++) {
+                const int d = tid + 128 * j;
+                if (d < a.vdim) acc[j] = fmaf(w, to_f(vr[d]), acc[j]);
+            }
+        }
+        __syncthreads();
+    }
+    OT* o = (OT*)a.out + (size_t)t * a.ldo + h * a.vdim;
+#pragma unroll
+    for (int j = 0; j < VCOLS; j++) {
+        const int d = tid + 128 * j;
+        if (d < a.vdim) o[d] = from_f<OT>(acc[j] / l);
+    }
+}
+
+// Merge of the decode kernel's splits into rows of pitch ldo, heads of vdim columns (the partials' rows are padded to hd).
+struct PagedCombineArgs {
+    const float* part_acc;
+    const float2* part_ml;
+    int n_heads, n_splits, hd, vdim;
+    void* out;
+    int ldo, out16;
+};
+
+__global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constant__ PagedCombineArgs a) {
+    const int h = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
+    pdl_launch();
+    pdl_wait();
+    if (d >= a.vdim) return;
+    const size_t p0 = ((size_t)b * a.n_heads + h) * a.n_splits;
+    float mn = -1e30f;
+    for (int s = 0; s < a.n_splits; s++) mn = fmaxf(mn, a.part_ml[p0 + s].x);
+    float o = 0.f, l = 0.f;
+    for (int s = 0; s < a.n_splits; s++) {
+        const float2 ml = a.part_ml[p0 + s];
+        const float c = __expf(ml.x - mn);
+        o += a.part_acc[(p0 + s) * a.hd + d] * c;
+        l += ml.y * c;
+    }
+    const float v = l > 0.f ? o / l : 0.f;
+    const size_t oi = (size_t)b * a.ldo + (size_t)h * a.vdim + d;
+    if (a.out16) ((__nv_bfloat16*)a.out)[oi] = __float2bfloat16_rn(v);
+    else ((float*)a.out)[oi] = v;
+}
+
+bool bad_shape(int H, int G, int dim, int vdim) { return H < 1 || G < 1 || H % G || dim < 1 || vdim < 1; }
+
+}  // namespace
+
+// Returns a cudaError_t value (as do the entry points below).
+B2_API int b2_paged_append(const PagedAppendArgs* a, int rows, int pdl, cudaStream_t st) {
+    if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dq < a->dim || a->dk < a->dim || a->dv < a->vdim || a->n_rot < 0 || a->n_rot > a->dim ||
+        (a->n_rot & 1) || (a->n_rot && !a->freqs) || (!a->q_norm != !a->k_norm))
+        return (int)cudaErrorInvalidValue;
+    const size_t smem = ((size_t)(a->n_heads + a->n_kv_heads) * a->dim + a->n_rot) * 4;
+    if (smem > 200 * 1024) return (int)cudaErrorNotSupported;
+    static PerDeviceOnce once;
+    if (once.first()) {
+        cudaFuncSetAttribute(paged_append_kernel<__half>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(paged_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    }
+    PagedAppendArgs c = *a;
+    void* args[] = {&c};
+    return launch_rows(a->cache32 ? (const void*)paged_append_kernel<float> : (const void*)paged_append_kernel<__half>, dim3(rows), dim3(256), smem, args, st, pdl);
+}
+
+B2_API int b2_paged_attn(const PagedAttnArgs* a, int rows, int pdl, cudaStream_t st) {
+    if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dim > 8192 || a->n_heads > 65535) return (int)cudaErrorInvalidValue;
+    if (a->vdim > 128 * VCOLS) return (int)cudaErrorNotSupported;
+    PagedAttnArgs c = *a;
+    void* args[] = {&c};
+    const void* fn = a->cache32 ? (a->out16 ? (const void*)paged_attn_kernel<float, __nv_bfloat16> : (const void*)paged_attn_kernel<float, float>)
+                                : (a->out16 ? (const void*)paged_attn_kernel<__half, __nv_bfloat16> : (const void*)paged_attn_kernel<__half, float>);
+    return launch_rows(fn, dim3(rows, a->n_heads), dim3(128), (size_t)a->dim * 4, args, st, pdl);
+}
+
+// Decode step over a paged f16 cache: norm and rotation of the new query and key, cache append and split-K attention in one launch,
+// then the merge of the splits.  cudaErrorNotSupported (nothing launched): the caller runs b2_paged_append + b2_paged_attn.
+B2_API int b2_attn_decode_paged(const AttnDecodeArgs* a, const AttnRopeArgs* r, int nb, int hd, void* out, int ldo, int out16, int pdl, cudaStream_t st) {
+    if (!r || !r->qkv || !a->page_table || bad_shape(a->n_heads, a->n_kv_heads, r->dim, r->vdim) || r->dim > hd || r->vdim > hd || nb < 1 || a->n_splits < 1)
+        return (int)cudaErrorInvalidValue;
+    const cudaError_t e = (cudaError_t)attn_decode_mma_rope_launch(*a, *r, nb, hd, pdl, st);
+    if (e != cudaSuccess) return (int)e;
+    PagedCombineArgs c{a->part_acc, a->part_ml, a->n_heads, a->n_splits, hd, r->vdim, out, ldo, out16};
+    void* args[] = {&c};
+    return launch_rows((const void*)paged_combine_kernel, dim3(a->n_heads, nb), dim3(128), 0, args, st, pdl);
+}

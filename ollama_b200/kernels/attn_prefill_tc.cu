@@ -36,6 +36,15 @@ struct AttnPrefillArgs {      // the same block as in attn_prefill.cu
     const __half* v_scale;
 };
 
+// Paged form of the pipelined kernel: the query tiles of a step (portions of several sequences) come as a list, K / V tiles are
+// read through a page table (two 64-position pages per tile; caches [page][Hkv][64][D], pad columns zero), the mask may be chunked
+// (position p sees the keys from floor(p / chunk) * chunk on), and heads of vdim <= D columns go to output rows of pitch ldo.
+struct AttnPagedArgs {
+    const int4* tiles;       // [tiles] (first row, rows <= 128, slot, position of the first row)
+    const int* page_table;   // [slots][max_pages]
+    int max_pages, chunk, vdim, ldo;
+};
+
 __device__ int g_attn_tc_status = 0;
 
 namespace {
@@ -106,6 +115,8 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// tanh through one exponential and one division; absolute error about 2^-22
+__device__ __forceinline__ float tanh_ex2(float x) { return 1.f - __fdividef(2.f, ex2(x * 2.885390081777926815f) + 1.f); }
 __device__ __forceinline__ uint32_t pack_h2(float a, float b) {
     const __half2 h = __floats2half2_rn(a, b);
     return *reinterpret_cast<const uint32_t*>(&h);
@@ -114,13 +125,13 @@ __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
 }
 
-// 2-D f16 tensor [rows][d] (d contiguous), box = 64 x 128 rows, 128-byte swizzle, out-of-range rows read as zero.
-bool make_kv_map(CUtensorMap* map, const void* base, size_t rows, int d) {
+// 2-D f16 tensor [rows][d] (d contiguous), box = 64 x box_rows, 128-byte swizzle, out-of-range rows read as zero.
+bool make_kv_map(CUtensorMap* map, const void* base, size_t rows, int d, int box_rows) {
     EncodeTiledFn fn = encode_fn();
     if (!fn) return false;
     cuuint64_t dims[2] = {(cuuint64_t)d, (cuuint64_t)rows};
     cuuint64_t strides[1] = {(cuuint64_t)d * 2};
-    cuuint32_t box[2] = {64u, (cuuint32_t)BKV};
+    cuuint32_t box[2] = {64u, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
     return fn(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
@@ -408,25 +419,25 @@ __global__ void __launch_bounds__(THREADS, 1) attn_prefill_tc_kernel(const __gri
 struct MapKey {
     const void* base;
     size_t rows;
-    int d;
+    int d, box_rows;
 };
 struct MapEntry {
     MapKey key;
     CUtensorMap map;
 };
-bool cached_kv_map(CUtensorMap* out, const void* base, size_t rows, int d) {
+bool cached_kv_map(CUtensorMap* out, const void* base, size_t rows, int d, int box_rows = BKV) {
     constexpr int CAP = 512;                      // K and V of up to 256 layers; beyond that the oldest entries are replaced
     static thread_local MapEntry* table = nullptr;
     static thread_local int used = 0, next = 0;
     if (!table) table = new MapEntry[CAP];
     for (int i = 0; i < used; i++)
-        if (table[i].key.base == base && table[i].key.rows == rows && table[i].key.d == d) {
+        if (table[i].key.base == base && table[i].key.rows == rows && table[i].key.d == d && table[i].key.box_rows == box_rows) {
             *out = table[i].map;
             return true;
         }
-    if (!make_kv_map(out, base, rows, d)) return false;
+    if (!make_kv_map(out, base, rows, d, box_rows)) return false;
     const int at = used < CAP ? used++ : (next++ % CAP);
-    table[at] = MapEntry{{base, rows, d}, *out};
+    table[at] = MapEntry{{base, rows, d, box_rows}, *out};
     return true;
 }
 
@@ -449,9 +460,9 @@ struct Lay2 {
     static constexpr int TOTAL = OFF_BAR + 256 + 2 * 2 * 128 * 4 + 1024;
 };
 
-template <int D>
+template <int D, bool PAGED>
 __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
-                                                                       const __grid_constant__ AttnPrefillArgs a) {
+                                                                       const __grid_constant__ AttnPrefillArgs a, const __grid_constant__ AttnPagedArgs pg) {
     using L = Lay2<D>;
     constexpr int ATOMS = L::ATOMS;
     constexpr int OH = D / 2;
@@ -474,10 +485,13 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int mt = gridDim.x - 1 - blockIdx.x;
-    const int m0 = mt * BQ, h = blockIdx.y, hkv = h / (a.H / a.Hkv);
-    const int q_lo = a.pos0 + m0, q_hi = a.pos0 + min(m0 + BQ, a.T) - 1;
-    const int k_end = a.causal ? min(a.kv_len, q_hi + 1) : a.kv_len;
-    const int k_begin = (a.window > 0 ? max(0, q_lo - a.window + 1) : 0) & ~(BKV - 1);
+    const int4 tile = PAGED ? pg.tiles[mt] : make_int4(mt * BQ, min(BQ, a.T - mt * BQ), a.slot, a.pos0 + mt * BQ);
+    const int m0 = tile.x, rows = tile.y, h = blockIdx.y, hkv = h / (a.H / a.Hkv);
+    const int q_lo = tile.w, q_hi = q_lo + rows - 1;
+    const int kv_len = PAGED ? q_hi + 1 : a.kv_len;
+    const int k_end = a.causal ? min(kv_len, q_hi + 1) : kv_len;
+    const int chunk = PAGED ? pg.chunk : 0;
+    const int k_begin = (chunk > 0 ? q_lo - q_lo % chunk : a.window > 0 ? max(0, q_lo - a.window + 1) : 0) & ~(BKV - 1);
     const int n_tiles = k_end > k_begin ? (k_end - k_begin + BKV - 1) / BKV : 0;
 
     if (threadIdx.x == 0) {
@@ -500,7 +514,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     }
     if (warp < SOFTMAX_WARPS) {
         const int r = 32 * (warp & 3) + lane, c = warp >> 2;
-        const bool live = m0 + r < a.T;
+        const bool live = r < rows;
         const float* qp = a.q + ((size_t)(m0 + r) * a.H + h) * D + OH * c;
 #pragma unroll
         for (int j = 0; j < OH / 8; j++) {
@@ -520,7 +534,8 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
-    const int row0 = (a.slot * a.Hkv + hkv) * a.n_ctx + k_begin;
+    const int row0 = PAGED ? 0 : (a.slot * a.Hkv + hkv) * a.n_ctx + k_begin;
+    const int* table = PAGED ? pg.page_table + (size_t)tile.z * pg.max_pages : nullptr;
 
     if (warp == 8 || warp == 10) {
         if (lane == 0) {                 // one thread streams the K tiles, another the V tiles: each waits only for its own buffers
@@ -534,7 +549,16 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                 if (t >= 2 && !mbar_wait(&empty[b], ((t >> 1) - 1) & 1)) { atomicExch(failed, 1); break; }
                 mbar_expect_tx(&full[b], L::KV_BYTES);
 #pragma unroll
-                for (int at = 0; at < ATOMS; at++) tma_load_2d(base + b * L::KV_BYTES + at * ATOM_BYTES, map, 64 * at, row0 + t * BKV, &full[b]);
+                for (int at = 0; at < ATOMS; at++) {
+                    uint8_t* dst = base + b * L::KV_BYTES + at * ATOM_BYTES;
+                    if (PAGED) {          // a tile may reach past the sequence's last page: any page will do there, its keys are masked
+                        const int p0 = (k_begin + t * BKV) >> 6, last = (kv_len - 1) >> 6;
+                        tma_load_2d(dst, map, 64 * at, (table[min(p0, last)] * a.Hkv + hkv) * 64, &full[b]);
+                        tma_load_2d(dst + ATOM_BYTES / 2, map, 64 * at, (table[min(p0 + 1, last)] * a.Hkv + hkv) * 64, &full[b]);
+                    } else {
+                        tma_load_2d(dst, map, 64 * at, row0 + t * BKV, &full[b]);
+                    }
+                }
             }
         }
     } else if (warp == 9) {
@@ -574,7 +598,8 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     } else {
         const int q = warp & 3, c = warp >> 2;
         const int r = 32 * q + lane;
-        const int qp = a.pos0 + m0 + r;
+        const int qp = q_lo + r;
+        const int chunk_lo = chunk > 0 ? qp - qp % chunk : 0, chunk_hi = chunk > 0 ? q_hi - q_hi % chunk : 0;      // this row's first key; the last row's
         const float LOG2E = 1.4426950408889634f;
         const float sl2 = a.scale * LOG2E;
         const uint32_t lane_base = (uint32_t)(32 * q) << 16;
@@ -604,14 +629,14 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             uint32_t v[2][32];
             tmem_ld32(tmem + lane_base + (uint32_t)(128 * b + 64 * c), v[0]);
             tmem_ld32(tmem + lane_base + (uint32_t)(128 * b + 64 * c + 32), v[1]);
-            const bool masked = (a.causal && n0 + BKV - 1 > q_lo) || n0 + BKV > a.kv_len || a.window > 0;
+            const bool masked = (a.causal && n0 + BKV - 1 > q_lo) || n0 + BKV > kv_len || a.window > 0 || n0 < chunk_hi;
             float mx = -INFINITY;
             if (a.softcap > 0.f) {
                 const float cap2 = a.softcap * LOG2E, inv_cap = a.scale / a.softcap;
 #pragma unroll
                 for (int i = 0; i < 2; i++)
 #pragma unroll
-                    for (int j = 0; j < 32; j++) v[i][j] = __float_as_uint(cap2 * tanhf(__uint_as_float(v[i][j]) * inv_cap));
+                    for (int j = 0; j < 32; j++) v[i][j] = __float_as_uint(cap2 * tanh_ex2(__uint_as_float(v[i][j]) * inv_cap));
             } else {
 #pragma unroll
                 for (int i = 0; i < 2; i++)
@@ -620,7 +645,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             }
             if (masked) {
                 const int kp0 = n0 + 64 * c;
-                const int hi = min(a.causal ? qp : a.kv_len - 1, a.kv_len - 1), lo = a.window > 0 ? qp - a.window + 1 : 0;
+                const int hi = min(a.causal ? qp : kv_len - 1, kv_len - 1), lo = PAGED ? chunk_lo : a.window > 0 ? qp - a.window + 1 : 0;
 #pragma unroll
                 for (int i = 0; i < 2; i++)
 #pragma unroll
@@ -679,7 +704,27 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                 l = l * oc + ex2(sk - m_new);
             }
             const float inv = l > 0.f ? oc / l : 0.f;
-            if (m0 + r < a.T) {
+            if (PAGED && r < rows) {
+                __nv_bfloat16* op = a.out + (size_t)(m0 + r) * pg.ldo + (size_t)h * pg.vdim + OH * c;
+                const bool whole = (pg.vdim & 7) == 0 && (pg.ldo & 7) == 0;
+#pragma unroll
+                for (int j = 0; j < OH; j += 8) {
+                    if (OH * c + j >= pg.vdim) continue;
+                    if (whole) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const __nv_bfloat162 bb = __floats2bfloat162_rn(o[j + 2 * e] * inv, o[j + 2 * e + 1] * inv);
+                            w[e] = *reinterpret_cast<const uint32_t*>(&bb);
+                        }
+                        *(uint4*)(op + j) = make_uint4(w[0], w[1], w[2], w[3]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; e++)
+                            if (OH * c + j + e < pg.vdim) op[j + e] = __float2bfloat16_rn(o[j + e] * inv);
+                    }
+                }
+            } else if (!PAGED && r < rows) {
                 __nv_bfloat16* op = a.out + (size_t)(m0 + r) * a.H * D + (size_t)h * D + OH * c;
 #pragma unroll
                 for (int j = 0; j < OH; j += 8) {
@@ -724,13 +769,41 @@ int launch2(const AttnPrefillArgs& a, int n_slots, cudaStream_t st) {
     const size_t rows = (size_t)n_slots * a.Hkv * a.n_ctx;
     if (!cached_kv_map(&mk, a.k_cache, rows, D) || !cached_kv_map(&mv, a.v_cache, rows, D)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D>::TOTAL);
+    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D>::TOTAL);
     dim3 grid((a.T + BQ - 1) / BQ, a.H);
-    attn_prefill_tc2_kernel<D><<<grid, THREADS2, Lay2<D>::TOTAL, st>>>(mk, mv, a);
+    attn_prefill_tc2_kernel<D, false><<<grid, THREADS2, Lay2<D>::TOTAL, st>>>(mk, mv, a, AttnPagedArgs{});
+    return (int)cudaGetLastError();
+}
+
+template <int D>
+int launch_paged(const AttnPrefillArgs& a, const AttnPagedArgs& pg, int n_tiles, int n_pages, cudaStream_t st) {
+    CUtensorMap mk, mv;
+    const size_t rows = (size_t)n_pages * a.Hkv * 64;
+    if (!cached_kv_map(&mk, a.k_cache, rows, D, 64) || !cached_kv_map(&mv, a.v_cache, rows, D, 64)) return (int)cudaErrorNotSupported;
+    static PerDeviceOnce once;
+    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D>::TOTAL);
+    attn_prefill_tc2_kernel<D, true><<<dim3(n_tiles, a.H), THREADS2, Lay2<D>::TOTAL, st>>>(mk, mv, a, pg);
     return (int)cudaGetLastError();
 }
 
 }  // namespace
+
+// Attention of a step's query tiles over a paged f16 cache (rows padded to head_dim 64 or 128; anything else: cudaErrorNotSupported,
+// nothing launched).  a: q [rows][H][head_dim], caches, out, H, Hkv, scale, softcap; the other fields are not used.
+B2_API int b2_attn_prefill_paged(const AttnPrefillArgs* a, const AttnPagedArgs* pg, int head_dim, int n_tiles, int n_pages, cudaStream_t st) {
+    if (!a || !pg || !pg->tiles || !pg->page_table || n_tiles < 1 || n_pages < 1 || pg->max_pages < 1 || a->H < 1 || a->H > 65535 || a->Hkv < 1 || a->H % a->Hkv ||
+        pg->vdim < 1 || pg->vdim > head_dim || pg->ldo < a->H * pg->vdim)
+        return (int)cudaErrorInvalidValue;
+    if (((uintptr_t)a->k_cache & 15) || ((uintptr_t)a->v_cache & 15) || ((uintptr_t)a->q & 15) || ((uintptr_t)a->out & 15)) return (int)cudaErrorNotSupported;
+    if ((size_t)n_pages * a->Hkv * 64 >= ((size_t)1 << 31)) return (int)cudaErrorNotSupported;
+    AttnPrefillArgs c = *a;
+    c.causal = 1;
+    c.window = 0;
+    c.sinks = nullptr;
+    if (head_dim == 128) return launch_paged<128>(c, *pg, n_tiles, n_pages, st);
+    if (head_dim == 64) return launch_paged<64>(c, *pg, n_tiles, n_pages, st);
+    return (int)cudaErrorNotSupported;
+}
 
 // Prefill attention on tcgen05: f16 caches, head size 64 or 128 (anything else: cudaErrorNotSupported, nothing launched; the
 // caller then runs b2_attn_prefill).  `n_slots`: slots of the cache tensors (the extent of the TMA maps).  Returns a cudaError_t value.

@@ -35,9 +35,26 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
+# sources of a part of the library, for a first start that should compile what one kind of model needs and no more
+GROUPS = {"stack": ("attn_decode_mma.cu", "attn_paged.cu", "attn_prefill_tc.cu", "elementwise.cu", "gemm_f32.cu", "gemm_tc.cu", "gemv_rows.cu",
+                    "norm_rows.cu", "sample.cu", "ssm.cu")}
+
+
+def build_group(group: str, verbose: bool = False, force: bool = False) -> str:
+    """Compile the sources of ``group`` and link them into a library of their own; their objects are the ones a later full build uses."""
+    lib = os.path.join(HERE, f"libb200{group}.so")
+    _compile(sorted(GROUPS[group]), lib, verbose, force)
+    return lib
+
+
 def build(verbose: bool = False, force: bool = False) -> str:
+    _compile(sorted(f for f in os.listdir(HERE) if f.endswith(".cu")), LIB, verbose, force)
+    build_host(verbose, force)
+    return LIB
+
+
+def _compile(srcs: list[str], lib: str, verbose: bool, force: bool) -> None:
     nvcc = _nvcc()
-    srcs = sorted(f for f in os.listdir(HERE) if f.endswith(".cu"))
     hdrs = [os.path.join(HERE, f) for f in os.listdir(HERE) if f.endswith((".cuh", ".h"))]
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
@@ -61,13 +78,12 @@ def build(verbose: bool = False, force: bool = False) -> str:
                 if rc:
                     raise RuntimeError(f"nvcc failed on {name}")
     objs = [os.path.join(objdir, s[:-3] + ".o") for s in srcs]
-    if force or _stale(LIB, objs):
-        cmd = [nvcc, "-shared", "-o", LIB, *objs, "-lcuda"]
-        r = subprocess.run(cmd, capture_output=True, text=True)
+    if force or _stale(lib, objs):
+        part = f"{lib}.{os.getpid()}"          # linked beside it and renamed: another process never loads half a library
+        r = subprocess.run([nvcc, "-shared", "-o", part, *objs, "-lcuda"], capture_output=True, text=True)
         if r.returncode:
             raise RuntimeError("link failed:\n" + r.stdout + r.stderr)
-    build_host(verbose, force)
-    return LIB
+        os.replace(part, lib)
 
 
 def build_host(verbose: bool = False, force: bool = False) -> str | None:

@@ -83,6 +83,15 @@ __device__ __forceinline__ float e8m0_to_float(uint32_t e) {
     return e == 0 ? __uint_as_float(0x00400000u) : __uint_as_float(e << 23);
 }
 
+// Activation of an ungated FFN in a matrix product's epilogue: 0 none, 1 square of relu.
+__device__ __forceinline__ float out_act(float v, int act) {
+    if (act == 1) {
+        const float r = fmaxf(v, 0.f);
+        return r * r;
+    }
+    return v;
+}
+
 // Gated FFN activation: 0 = SiLU(g) * u, 1 = tanh-GELU(g) * u, 2 = clamped SwiGLU with alpha and limit (gpt-oss).
 __device__ __forceinline__ float glu_act(float g, float u, int act, float alpha, float limit) {
     if (act == 0) return g / (1.f + __expf(-g)) * u;

@@ -46,6 +46,8 @@ struct GemmParams {
     // gated activation in the epilogue: columns 2i / 2i + 1 are gate / up of output i; out is bf16 [m][ldo] with n / 2 columns
     int glu;                // 0: off, 1 + act otherwise (0 silu, 1 gelu_tanh, 2 clamped swiglu)
     float glu_alpha, glu_limit;
+    int act;                // ungated activation of the result (out_act), before it is stored or accumulated
+    int lda;                // row pitch of a, 0: k
 };
 
 template <int BN>
@@ -206,6 +208,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                     if (row >= p.m || col >= p.n) continue;
                     float4 r = *(const float4*)(st + lr * L::EPI_LD + cq);
                     r.x += bias.x; r.y += bias.y; r.z += bias.z; r.w += bias.w;
+                    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
                     if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
                         const float h0 = glu_act(r.x, r.y, p.glu - 1, p.glu_alpha, p.glu_limit), h1 = glu_act(r.z, r.w, p.glu - 1, p.glu_alpha, p.glu_limit);
                         *(uint32_t*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + (col >> 1)) = pack2_bf16(h0, h1);
@@ -256,7 +259,7 @@ int sm_count() {
 template <int BN>
 int launch(const void* a, const void* b, const GemmParams& p, cudaStream_t st, int b_rows = 0) {
     CUtensorMap ma, mb;
-    if (!make_map(&ma, a, p.m, p.k, BM) || !make_map(&mb, b, b_rows ? b_rows : p.n, p.k, BN)) return (int)cudaErrorNotSupported;
+    if (!make_map(&ma, a, p.m, p.k, BM, p.lda) || !make_map(&mb, b, b_rows ? b_rows : p.n, p.k, BN)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
     if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
     const int total = ((p.m + BM - 1) / BM) * ((p.n + BN - 1) / BN);
@@ -270,7 +273,7 @@ int dispatch(const void* a, const void* b, const GemmParams& p, cudaStream_t st,
     const long tiles_m = (p.m + BM - 1) / BM;
     // a handful of rows (a decode step of several sequences): the product streams b once, so the narrowest tile that spreads
     // b over the most SMs wins
-    if (p.m <= 32 && !p.out_bf16 && !p.glu && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
+    if (p.m <= 32 && (!p.out_bf16 || p.act || p.lda) && !p.glu && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
         return launch<64>(a, b, p, st, b_rows);
     if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256>(a, b, p, st, b_rows);
     // one round either way: the widest tile that still gives every SM at most one tile
@@ -298,6 +301,15 @@ B2_API int b2_gemm_bf16(const void* a, const void* b, int m, int n, int k, float
 B2_API int b2_gemm_bf16_out16(const void* a, const void* b, int m, int n, int k, void* out, int ldo, const float* bias, cudaStream_t st) {
     if (bad_operands(a, b, m, n, k, ldo) || (n & 7) || (ldo & 7) || ((uintptr_t)out & 15)) return (int)cudaErrorInvalidValue;
     GemmParams p{m, n, k, out, ldo, bias, 0, 1, {}, 0, nullptr, 0, 0.f, 0.f};
+    return dispatch(a, b, p, st);
+}
+
+// The same product for operands and results inside wider buffers: a has row pitch lda (k % 8 == 0, lda % 8 == 0), the result goes
+// to rows of pitch ldo as bf16 (n % 4 == 0, out 8-byte aligned) or fp32, after the ungated activation `act` (0 none, 1 square of relu).
+B2_API int b2_gemm_bf16_act(const void* a, int lda, const void* b, int m, int n, int k, void* out, int ldo, int out16, int act, int accumulate, cudaStream_t st) {
+    if (bad_operands(a, b, m, n, k, ldo) || lda < k || (lda & 7) || act < 0 || act > 1 || (out16 && accumulate) || ((uintptr_t)out & (out16 ? 7 : 15)))
+        return (int)cudaErrorInvalidValue;
+    GemmParams p{m, n, k, out, ldo, nullptr, accumulate, out16, {}, 0, nullptr, 0, 0.f, 0.f, act, lda};
     return dispatch(a, b, p, st);
 }
 

@@ -1,0 +1,47 @@
+// Element access shared by the kernels that exist in a 16-bit and a 32-bit form.
+#pragma once
+#include "common.cuh"
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f(__half v) { return __half2float(v); }
+
+template <typename T>
+__device__ __forceinline__ T from_f(float v);
+template <>
+__device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+template <>
+__device__ __forceinline__ __half from_f<__half>(float v) { return __float2half_rn(v); }
+
+__device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
+__device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+
+// Rotation angle of `pos` at frequency `f`, reduced to one turn: the product is formed in double, so that the angle keeps its
+// 24 bits at any position.
+__device__ __forceinline__ float rot_angle(int pos, double f) {
+    constexpr double TURN = 6.283185307179586476925;
+    const double a = (double)pos * f;
+    return (float)(a - TURN * rint(a / TURN));
+}
+
+// Cache position -> row of a paged cache [page][kv head][64 positions][row length].
+constexpr int PAGE_SHIFT = 6, PAGE = 1 << PAGE_SHIFT;
+__device__ __forceinline__ size_t paged_row(const int* table, int pos, int n_kv_heads, int kvh) {
+    return ((size_t)table[pos >> PAGE_SHIFT] * n_kv_heads + kvh) * PAGE + (pos & (PAGE - 1));
+}
+
+static inline int launch_rows(const void* fn, dim3 grid, dim3 block, size_t smem, void** args, cudaStream_t st, int pdl) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[0].val.programmaticStreamSerializationAllowed = pdl ? 1 : 0;
+    cfg.attrs = at;
+    cfg.numAttrs = 1;
+    return (int)cudaLaunchKernelExC(&cfg, fn, args);
+}

@@ -1,0 +1,326 @@
+// Selective state-space mixer (a diagonal recurrence per channel and state dimension with input-dependent step size):
+//
+//   u = silu(conv(x)),  dt = softplus(W_dt d + b),  S[c][n] <- exp(dt_c A[c][n]) S[c][n] + dt_c u_c B[n],
+//   y_c = (sum_n S[c][n] C[n] + D_c u_c) * silu(z_c)
+//
+// Four kernels: the causal depthwise convolution of a batch of prompt rows, the scan over prompt rows, and a decode step that
+// does projection of the step size, convolution, recurrence and gate of one token per sequence in one launch.  Recurrence,
+// step sizes and decays are fp32.  A slot's state is [channel][state] fp32 plus the convolution's last taps - 1 inputs; a sequence at
+// position 0 takes both as zeros, whatever an earlier owner of the slot left there.
+//
+// A is passed as log2(e) * A, so that exp(dt A) = exp2(dt A2); 32-bit models pass A itself and advance S by S * expm1(dt A), which keeps the
+// distance of a slow decay from 1 to full precision (an error of an exponential near 1 adds up over the steps that a state remembers).
+#include "rows.cuh"
+
+__device__ __forceinline__ float ex2_f(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+template <bool EXACT>
+__device__ __forceinline__ float decayed(float s, float x) { return EXACT ? fmaf(s, expm1f(x), s) : s * ex2_f(x); }
+
+// rows: token rows of one step.  seg [n_seg][4] = first row, rows, slot, position of the first row.
+struct SsmConvArgs {
+    const void* xz;          // [rows][ldx], x in the first `inner` columns
+    int ldx, inner, taps;    // inner: padded to a multiple of 8
+    const float* w;          // [taps][inner]
+    const float* b;          // [inner]
+    const float* state;      // [slots][taps - 1][inner], oldest first
+    const int* slots;        // [rows]
+    const int* positions;    // [rows]
+    const int* offs;         // [rows] index of the row within its sequence's portion
+    void* u;                 // [rows][ldu]
+    int ldu;
+};
+
+constexpr int CONV_ROWS = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ SsmConvArgs a, int rows) {
+    const int c = 4 * (blockIdx.x * 128 + threadIdx.x);
+    pdl_launch();
+    pdl_wait();
+    if (c >= a.inner) return;
+    const T* xz = (const T*)a.xz;
+    const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
+    const float4 bias = *(const float4*)(a.b + c);
+    for (int r = r0; r < r1; r++) {
+        const int off = a.offs[r];
+        float acc[4] = {bias.x, bias.y, bias.z, bias.w};
+        for (int j = 0; j < a.taps; j++) {
+            const int back = a.taps - 1 - j;
+            const float4 w = *(const float4*)(a.w + (size_t)j * a.inner + c);
+            float v[4];
+            if (back <= off) {
+                const T* p = xz + (size_t)(r - back) * a.ldx + c;
+#pragma unroll
+                for (int i = 0; i < 4; i++) v[i] = to_f(p[i]);
+            } else if (a.positions[r] - back >= 0) {      // before this portion: input `back - off` places before its first row
+                const float4 s = *(const float4*)(a.state + ((size_t)a.slots[r] * (a.taps - 1) + (a.taps - 1) - (back - off)) * a.inner + c);
+                v[0] = s.x; v[1] = s.y; v[2] = s.z; v[3] = s.w;
+            } else {
+                continue;
+            }
+            acc[0] += w.x * v[0]; acc[1] += w.y * v[1]; acc[2] += w.z * v[2]; acc[3] += w.w * v[3];
+        }
+        T* o = (T*)a.u + (size_t)r * a.ldu + c;
+#pragma unroll
+        for (int i = 0; i < 4; i++) o[i] = from_f<T>(silu_f(acc[i]));
+    }
+}
+
+B2_API int b2_ssm_conv(const SsmConvArgs* a, int rows, int f32, int pdl, cudaStream_t st) {
+    if (rows < 1 || a->inner < 8 || (a->inner & 7) || a->taps < 1 || a->ldx < a->inner || a->ldu < a->inner || (rows + CONV_ROWS - 1) / CONV_ROWS > 65535)
+        return (int)cudaErrorInvalidValue;
+    SsmConvArgs c = *a;
+    void* args[] = {&c, &rows};
+    const dim3 grid((a->inner + 511) / 512, (rows + CONV_ROWS - 1) / CONV_ROWS);
+    return launch_rows(f32 ? (const void*)ssm_conv_kernel<float> : (const void*)ssm_conv_kernel<__nv_bfloat16>, grid, dim3(128), 0, args, st, pdl);
+}
+
+struct SsmScanArgs {
+    const void* xz;          // [rows][ldx]: x columns 0 .. inner - 1 (for the convolution state), z from column off_z
+    int ldx, off_z;
+    const void* u;           // [rows][ldu]
+    int ldu;
+    const float* dt;         // [rows][lddt] step sizes before bias and softplus
+    int lddt;
+    const float* bc;         // [rows][ldbc]: B at column off_b, C at column off_b + n_state
+    int ldbc, off_b;
+    const float* dt_bias;    // [inner]
+    const float* a2;         // [inner][n_state] log2(e) * A (fp32 form: A)
+    const float* d;          // [inner]
+    int inner, n_state, taps;
+    float* state;            // [slots][inner][n_state]
+    float* conv_state;       // [slots][taps - 1][inner]
+    const int4* seg;         // [n_seg] (first row, rows, slot, position of the first row)
+    void* out;               // [rows][ldo]
+    int ldo;
+};
+
+// LPC lanes share a channel and hold SPL state dimensions each.  Time runs in tiles of TT rows whose inputs are fetched into
+// registers while the previous tile is worked on.
+template <typename T, int LPC, int SPL>
+__global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ SsmScanArgs a) {
+    constexpr int CH = 128 / LPC, NP = LPC * SPL, TT = NP <= 32 ? 32 : 16;
+    constexpr int PER = TT * CH / 128, PERN = (TT * NP + 127) / 128;
+    __shared__ float2 s_dt[TT][CH];          // (dt, dt * u)
+    __shared__ float s_y[TT][CH];            // in: D u, out: y
+    __shared__ __align__(16) float s_b[TT][NP], s_c[TT][NP];
+    const int tid = threadIdx.x, ch = tid / LPC, l = tid % LPC;
+    const int c0 = blockIdx.x * CH, c = c0 + ch;
+    pdl_launch();
+    pdl_wait();
+    const int4 sg = a.seg[blockIdx.y];
+    const int row0 = sg.x, rows = sg.y, slot = sg.z, pos0 = sg.w;
+    const bool live = c < a.inner;
+    float A[SPL], S[SPL];
+#pragma unroll
+    for (int i = 0; i < SPL; i++) {
+        const int n = l * SPL + i;
+        const bool ok = live && n < a.n_state;
+        A[i] = ok ? a.a2[(size_t)c * a.n_state + n] : 0.f;
+        S[i] = ok && pos0 > 0 ? a.state[((size_t)slot * a.inner + c) * a.n_state + n] : 0.f;
+    }
+    const T* xz = (const T*)a.xz;
+    const T* u = (const T*)a.u;
+    T* out = (T*)a.out;
+    const int lc = tid % CH, lt = tid / CH;      // element (lt + LPC * i, lc) of a tile is this thread's to move
+    const bool lok = c0 + lc < a.inner;
+    const float bias = lok ? a.dt_bias[c0 + lc] : 0.f, dd = lok ? a.d[c0 + lc] : 0.f;
+    float rdt[PER], ru[PER], rz[PER], rb[PERN], rc[PERN];
+    auto fetch = [&](int t0) {
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const int t = t0 + lt + LPC * i;
+            const bool ok = lok && t < rows;
+            const size_t r = (size_t)(row0 + t);
+            rdt[i] = ok ? a.dt[r * a.lddt + c0 + lc] : 0.f;
+            ru[i] = ok ? to_f(u[r * a.ldu + c0 + lc]) : 0.f;
+            rz[i] = ok ? to_f(xz[r * a.ldx + a.off_z + c0 + lc]) : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < PERN; i++) {
+            const int e = tid + 128 * i, t = e / NP, n = e % NP;
+            const bool ok = t < TT && t0 + t < rows && n < a.n_state;
+            const float* p = a.bc + (size_t)(row0 + t0 + t) * a.ldbc + a.off_b + n;
+            rb[i] = ok ? p[0] : 0.f;
+            rc[i] = ok ? p[a.n_state] : 0.f;
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < rows; t0 += TT) {
+        float z[PER];
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const float dt = softplus_f(rdt[i] + bias);
+            s_dt[lt + LPC * i][lc] = make_float2(dt, dt * ru[i]);
+            s_y[lt + LPC * i][lc] = dd * ru[i];
+            z[i] = rz[i];
+        }
+#pragma unroll
+        for (int i = 0; i < PERN; i++) {
+            const int e = tid + 128 * i;
+            if (e < TT * NP) {
+                (&s_b[0][0])[e] = rb[i];
+                (&s_c[0][0])[e] = rc[i];
+            }
+        }
+        __syncthreads();
+        if (t0 + TT < rows) fetch(t0 + TT);
+        const int nt = min(TT, rows - t0);
+#pragma unroll 4
+        for (int t = 0; t < nt; t++) {
+            const float2 dv = s_dt[t][ch];
+            float y = 0.f;
+#pragma unroll
+            for (int i = 0; i < SPL; i++) {
+                S[i] = decayed<sizeof(T) == 4>(S[i], dv.x * A[i]) + dv.y * s_b[t][l * SPL + i];
+                y += S[i] * s_c[t][l * SPL + i];
+            }
+#pragma unroll
+            for (int o = LPC / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+            if (l == 0) s_y[t][ch] += y;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const int t = t0 + lt + LPC * i;
+            if (lok && t < rows) out[(size_t)(row0 + t) * a.ldo + c0 + lc] = from_f<T>(s_y[lt + LPC * i][lc] * silu_f(z[i]));
+        }
+        __syncthreads();
+    }
+    if (!live) return;
+#pragma unroll
+    for (int i = 0; i < SPL; i++) {
+        const int n = l * SPL + i;
+        if (n < a.n_state) a.state[((size_t)slot * a.inner + c) * a.n_state + n] = S[i];
+    }
+    if (l == 0) {
+        float* cs = a.conv_state + (size_t)slot * (a.taps - 1) * a.inner + c;
+        for (int i = 0; i < a.taps - 1; i++) {
+            const int src = rows - (a.taps - 1) + i;      // ascending: an entry is read before it is overwritten
+            cs[(size_t)i * a.inner] = src >= 0 ? to_f(xz[(size_t)(row0 + src) * a.ldx + c]) : pos0 > 0 ? cs[(size_t)(i + rows) * a.inner] : 0.f;
+        }
+    }
+}
+
+template <typename T>
+static const void* pick_scan(int n, int& ch) {
+    if (n <= 16) { ch = 32; return (const void*)ssm_scan_kernel<T, 4, 4>; }
+    if (n <= 32) { ch = 32; return (const void*)ssm_scan_kernel<T, 4, 8>; }
+    if (n <= 64) { ch = 16; return (const void*)ssm_scan_kernel<T, 8, 8>; }
+    if (n <= 128) { ch = 8; return (const void*)ssm_scan_kernel<T, 16, 8>; }
+    if (n <= 256) { ch = 8; return (const void*)ssm_scan_kernel<T, 16, 16>; }
+    return nullptr;
+}
+
+// At most 256 state dimensions.  The outputs' padding columns are not written.  Returns a cudaError_t value.
+B2_API int b2_ssm_scan(const SsmScanArgs* a, int n_seg, int f32, int pdl, cudaStream_t st) {
+    if (n_seg < 1 || n_seg > 65535 || a->inner < 8 || (a->inner & 7) || a->n_state < 1 || a->taps < 1) return (int)cudaErrorInvalidValue;
+    int ch = 0;
+    const void* fn = f32 ? pick_scan<float>(a->n_state, ch) : pick_scan<__nv_bfloat16>(a->n_state, ch);
+    if (!fn) return (int)cudaErrorNotSupported;
+    SsmScanArgs c = *a;
+    void* args[] = {&c};
+    return launch_rows(fn, dim3((a->inner + ch - 1) / ch, n_seg), dim3(128), 0, args, st, pdl);
+}
+
+struct SsmStepArgs {
+    const void* xz;          // [nb][ldx]
+    int ldx, off_z, xz16;    // xz16: bf16, else fp32
+    const float* conv_w;     // [taps][inner]
+    const float* conv_b;
+    float* conv_state;       // [slots][taps - 1][inner]
+    int taps, inner, n_state;
+    const float* p;          // [nb][ldp]: low-rank step-size input at column 0, B at column off_b, C at off_b + n_state
+    int ldp, off_b;
+    const void* w_dt;        // [inner][rank] bf16 or fp32 (rank padded to a multiple of 8, pad columns zero)
+    int rank, w32;
+    const float* dt;         // [nb][lddt] projected step sizes, or null: projected here from p and w_dt
+    int lddt;
+    const float* dt_bias;
+    const float* a2;
+    const float* d;
+    float* state;            // [slots][inner][n_state]
+    const int* slots;
+    const int* positions;
+    void* out;               // [nb][ldo]
+    int ldo, out16;
+    int exact;               // a2 holds A: see above
+};
+
+// eight lanes per channel, four channels per warp, 32 channels per CTA; grid (channel blocks, sequences)
+__global__ void __launch_bounds__(256) ssm_step_kernel(const __grid_constant__ SsmStepArgs a) {
+    const int lane = threadIdx.x & 31, l = lane & 7, b = blockIdx.y;
+    const int c_raw = blockIdx.x * 32 + (threadIdx.x >> 3);
+    const bool live = c_raw < a.inner;
+    const int c = live ? c_raw : a.inner - 1;
+    const float bias = a.dt_bias[c], dd = a.d[c];
+    pdl_launch();
+    pdl_wait();
+    const int slot = a.slots[b];
+    const bool fresh = a.positions[b] == 0;
+    float dt = 0.f;
+    if (a.dt) {
+        dt = a.dt[(size_t)b * a.lddt + c];
+    } else {
+        const float* p = a.p + (size_t)b * a.ldp;
+        if (a.w32) {
+            const float* w = (const float*)a.w_dt + (size_t)c * a.rank;
+            for (int i = 4 * l; i < a.rank; i += 32) {
+                const float4 wv = *(const float4*)(w + i), pv = *(const float4*)(p + i);
+                dt += wv.x * pv.x + wv.y * pv.y + wv.z * pv.z + wv.w * pv.w;
+            }
+        } else {
+            const __nv_bfloat16* w = (const __nv_bfloat16*)a.w_dt + (size_t)c * a.rank;
+#pragma unroll 4
+            for (int i = 8 * l; i < a.rank; i += 64) {
+                const uint4 q = ldg16(w + i);
+                const float4 p0 = *(const float4*)(p + i), p1 = *(const float4*)(p + i + 4);
+                dt += __uint_as_float(q.x << 16) * p0.x + __uint_as_float(q.x & 0xffff0000u) * p0.y + __uint_as_float(q.y << 16) * p0.z +
+                      __uint_as_float(q.y & 0xffff0000u) * p0.w + __uint_as_float(q.z << 16) * p1.x + __uint_as_float(q.z & 0xffff0000u) * p1.y +
+                      __uint_as_float(q.w << 16) * p1.z + __uint_as_float(q.w & 0xffff0000u) * p1.w;
+            }
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) dt += __shfl_xor_sync(0xffffffffu, dt, o);
+    }
+    dt = softplus_f(dt + bias);
+    const size_t xi = (size_t)b * a.ldx;
+    auto in = [&](int col) -> float { return a.xz16 ? to_f(((const __nv_bfloat16*)a.xz)[xi + col]) : ((const float*)a.xz)[xi + col]; };
+    const float x = in(c), z = in(a.off_z + c);
+    float* cs = a.conv_state + (size_t)slot * (a.taps - 1) * a.inner + c;
+    float u = a.conv_b[c] + a.conv_w[(size_t)(a.taps - 1) * a.inner + c] * x;
+    if (!fresh)
+        for (int j = 0; j < a.taps - 1; j++) u += cs[(size_t)j * a.inner] * a.conv_w[(size_t)j * a.inner + c];
+    u = silu_f(u);
+    const float* B = a.p + (size_t)b * a.ldp + a.off_b;
+    const float* C = B + a.n_state;
+    float* S = a.state + ((size_t)slot * a.inner + c) * a.n_state;
+    const float* A = a.a2 + (size_t)c * a.n_state;
+    float y = 0.f;
+    for (int n = l; n < a.n_state; n += 8) {
+        const float old = fresh ? 0.f : S[n];
+        const float s = (a.exact ? decayed<true>(old, dt * A[n]) : decayed<false>(old, dt * A[n])) + dt * u * B[n];
+        y += s * C[n];
+        if (live) S[n] = s;
+    }
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);      // also: every lane has read the convolution state by now
+    if (!live || l != 0) return;
+    for (int j = 0; j < a.taps - 1; j++) cs[(size_t)j * a.inner] = j + 1 < a.taps - 1 ? (fresh ? 0.f : cs[(size_t)(j + 1) * a.inner]) : x;
+    const float v = (y + dd * u) * silu_f(z);
+    if (a.out16) ((__nv_bfloat16*)a.out)[(size_t)b * a.ldo + c] = __float2bfloat16_rn(v);
+    else ((float*)a.out)[(size_t)b * a.ldo + c] = v;
+}
+
+B2_API int b2_ssm_step(const SsmStepArgs* a, int nb, int pdl, cudaStream_t st) {
+    if (nb < 1 || nb > 65535 || a->inner < 8 || (a->inner & 7) || a->n_state < 1 || a->taps < 1 || (!a->dt && (!a->w_dt || (a->rank & 7) || (a->ldp & 3))))
+        return (int)cudaErrorInvalidValue;
+    SsmStepArgs c = *a;
+    void* args[] = {&c};
+    return launch_rows((const void*)ssm_step_kernel, dim3((a->inner + 31) / 32, nb), dim3(256), 0, args, st, pdl);
+}

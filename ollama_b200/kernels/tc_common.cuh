@@ -94,12 +94,12 @@ inline EncodeTiledFn encode_fn() {
     return fn;
 }
 
-// 2-D bf16 tensor [rows][k] (k contiguous), box = 64 x box_rows, 128-byte swizzle, out-of-range reads give zero.
-inline bool make_map(CUtensorMap* map, const void* base, int rows, int k, int box_rows) {
+// 2-D bf16 tensor [rows][k] (k contiguous, rows `pitch` elements apart, 0: k), box = 64 x box_rows, 128-byte swizzle, out-of-range reads give zero.
+inline bool make_map(CUtensorMap* map, const void* base, int rows, int k, int box_rows, int pitch = 0) {
     EncodeTiledFn fn = encode_fn();
     if (!fn) return false;
     cuuint64_t dims[2] = {(cuuint64_t)k, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {(cuuint64_t)k * 2};
+    cuuint64_t strides[1] = {(cuuint64_t)(pitch ? pitch : k) * 2};
     cuuint32_t box[2] = {(cuuint32_t)BK, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
     return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,

@@ -14,8 +14,10 @@ from typing import Any
 
 import numpy as np
 
+from .stack import STACK_ARCHS, AttentionMixer, Stack, parse_stack
+
 SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "qwen3", "qwen3moe", "gemma", "gemma2", "gemma3", "gpt-oss", "phi3",
-                   "bert", "nomic-bert")
+                   "bert", "nomic-bert", *STACK_ARCHS.values())
 
 
 @dataclass
@@ -70,6 +72,13 @@ class ModelConfig:
     # pooling (embedding models)
     pooling: str = "none"          # none | mean | cls | last
     causal: bool = True
+    # layers that differ from each other (models/stack.py); the fields above then hold the largest sizes
+    stack: Stack | None = None
+
+    @property
+    def recurrent(self) -> bool:
+        """Part of a sequence's memory is a state that only moves forward: no position can be dropped, rolled back or re-used."""
+        return self.stack is not None and self.stack.recurrent
 
     @property
     def is_moe(self) -> bool:
@@ -96,6 +105,9 @@ class ModelConfig:
         return self.rope_base
 
     def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
+        if self.stack is not None:
+            ms = [self.stack.layers[r.layer].mixer for r in self.stack.runs()]
+            return sum(m.kv_heads * (m.dim + m.vdim) for m in ms if isinstance(m, AttentionMixer)) * elem_bytes
         return self.n_layers * (self.n_kv_heads * (self.head_dim + self.v_head_dim)) * elem_bytes
 
 
@@ -196,6 +208,14 @@ def config_from_gguf(g) -> ModelConfig:
             c.sliding_window = 128
         # alternating window / full layers, even layers use the window (fs/ggml/ggml.go:877-886)
         c.swa_layers = [i % 2 == 0 for i in range(c.n_layers)]
+    elif arch in STACK_ARCHS.values():
+        st = c.stack = parse_stack(g.string("stack"))
+        c.n_layers, c.d_model, c.vocab_size, c.norm_eps = len(st.layers), st.width, st.vocab, st.eps
+        c.embed_scale, c.final_softcap = st.embed_scale, st.logit_softcap
+        c.rope_style, c.act = "neox", "relu2"
+        c.ctx_train = u("context_length", 0)             # 0: no trained length to stay below
+        att = [L.mixer for L in st.layers if isinstance(L.mixer, AttentionMixer)]
+        c.n_heads, c.n_kv_heads = max((m.heads for m in att), default=0), max((m.kv_heads for m in att), default=0)
     elif arch in ("bert", "nomic-bert"):
         c.causal = False
         c.pooling = {0: "none", 1: "mean", 2: "cls", 3: "last"}.get(u("pooling_type", 1), "mean")

@@ -27,14 +27,52 @@ class CudaKernelError(RuntimeError):
     pass
 
 
+class _Library:
+    """The kernel library, or while that has not been built a part of it (:func:`need`): an entry point that the part does not have
+    builds and loads the whole."""
+
+    def __init__(self):
+        self._cdll = None
+
+    def load(self, path: str) -> None:
+        self._cdll = C.CDLL(path)
+        self.__dict__.update({"_path": path})
+
+    def __getattr__(self, name: str):
+        if name.startswith("__"):
+            raise AttributeError(name)
+        try:
+            f = getattr(self._cdll, name)
+        except AttributeError:
+            if self._path == _LIB_PATH:
+                raise
+            from ..kernels.build import build
+            self.load(build())
+            f = getattr(self._cdll, name)
+        self.__dict__[name] = f
+        return f
+
+
 def lib():
     global _lib
     if _lib is None:
         if not os.path.exists(_LIB_PATH):
             from ..kernels.build import build
             build()
-        _lib = C.CDLL(_LIB_PATH)
+        _lib = _Library()
+        _lib.load(_LIB_PATH)
     return _lib
+
+
+def need(group: str) -> None:
+    """Make the kernels of ``group`` available: the whole library when it is there, else only that group is compiled."""
+    global _lib
+    if _lib is None and not os.path.exists(_LIB_PATH):
+        from ..kernels.build import build_group
+        _lib = _Library()
+        _lib.load(build_group(group))
+    else:
+        lib()
 
 
 def available() -> bool:
@@ -120,11 +158,12 @@ class AttnDecodeArgs(C.Structure):
     _fields_ = [("q", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("positions", C.c_void_p),
                 ("slots", C.c_void_p), ("n_heads", C.c_int), ("n_kv_heads", C.c_int), ("n_ctx", C.c_int), ("n_splits", C.c_int),
                 ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int), ("part_acc", C.c_void_p), ("part_ml", C.c_void_p),
-                ("k_scale", C.c_void_p), ("v_scale", C.c_void_p)]
+                ("k_scale", C.c_void_p), ("v_scale", C.c_void_p), ("page_table", C.c_void_p), ("max_pages", C.c_int), ("chunk", C.c_int)]
 
 
 class AttnRopeArgs(C.Structure):
-    _fields_ = [("qkv", C.c_void_p), ("inv_freq", C.c_void_p), ("mscale", C.c_float), ("n_rot", C.c_int), ("neox", C.c_int)]
+    _fields_ = [("qkv", C.c_void_p), ("inv_freq", C.c_void_p), ("mscale", C.c_float), ("n_rot", C.c_int), ("neox", C.c_int),
+                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float), ("ldq", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("freqs", C.c_void_p)]
 
 
 class AttnCombineArgs(C.Structure):

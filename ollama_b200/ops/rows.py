@@ -1,0 +1,157 @@
+"""Bindings of the row kernels behind stack models: norms, fused decode products, 32-bit products, paged attention and the selective
+state-space mixer (kernels/norm_rows.cu, gemv_rows.cu, gemm_f32.cu, attn_paged.cu, ssm.cu)."""
+from __future__ import annotations
+
+import ctypes as C
+
+import torch
+
+from .cuda import AttnDecodeArgs, AttnPrefillArgs, AttnRopeArgs, _check, lib, ptr, stream
+
+P, I, F = C.c_void_p, C.c_int, C.c_float
+ACT = {"": 0, "relu2": 1}
+SRC_ROWS, SRC_NORM, SRC_JOINED, SRC_CONV = range(4)
+GEMV_MAX_ROWS = 4
+
+
+def _st(name: str, fields: list) -> type:
+    return type(name, (C.Structure,), {"_fields_": fields})
+
+
+NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), ("eps", F), ("w1", P), ("w2", P), ("o1", P), ("o2", P), ("f32", I)])
+JoinRowsArgs = _st("JoinRowsArgs", [("a", P), ("b", P), ("lda", I), ("n_a", I), ("ldb", I), ("n_b", I), ("out", P), ("ldo", I), ("off_b", I), ("f32", I)])
+RowSeg = _st("RowSeg", [("w", P), ("g", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I)])
+GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
+                                    ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_w", P), ("conv_b", P), ("conv_state", P), ("slots", P),
+                                    ("positions", P), ("taps", I)])
+PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
+                                          ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
+                                          ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I)])
+PagedAttnArgs = _st("PagedAttnArgs", [("q", P), ("dq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("k_cache", P), ("v_cache", P),
+                                      ("dk", I), ("dv", I), ("cache32", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
+                                      ("chunk", I), ("scale", F), ("softcap", F), ("out", P), ("ldo", I), ("out16", I)])
+AttnPagedArgs = _st("AttnPagedArgs", [("tiles", P), ("page_table", P), ("max_pages", I), ("chunk", I), ("vdim", I), ("ldo", I)])
+SsmConvArgs = _st("SsmConvArgs", [("xz", P), ("ldx", I), ("inner", I), ("taps", I), ("w", P), ("b", P), ("state", P), ("slots", P), ("positions", P),
+                                  ("offs", P), ("u", P), ("ldu", I)])
+SsmScanArgs = _st("SsmScanArgs", [("xz", P), ("ldx", I), ("off_z", I), ("u", P), ("ldu", I), ("dt", P), ("lddt", I), ("bc", P), ("ldbc", I), ("off_b", I),
+                                  ("dt_bias", P), ("a2", P), ("d", P), ("inner", I), ("n_state", I), ("taps", I), ("state", P), ("conv_state", P), ("seg", P),
+                                  ("out", P), ("ldo", I)])
+SsmStepArgs = _st("SsmStepArgs", [("xz", P), ("ldx", I), ("off_z", I), ("xz16", I), ("conv_w", P), ("conv_b", P), ("conv_state", P), ("taps", I),
+                                  ("inner", I), ("n_state", I), ("p", P), ("ldp", I), ("off_b", I), ("w_dt", P), ("rank", I), ("w32", I), ("dt", P),
+                                  ("lddt", I), ("dt_bias", P), ("a2", P), ("d", P), ("state", P), ("slots", P), ("positions", P), ("out", P), ("ldo", I),
+                                  ("out16", I), ("exact", I)])
+
+
+def _is32(t: torch.Tensor) -> int:
+    return int(t.dtype == torch.float32)
+
+
+def _call(name: str, args, *more) -> None:
+    _check(getattr(lib(), name)(C.byref(args), *more, stream()), name)
+
+
+def norm_rows(x: torch.Tensor, k: int, eps: float, w1: torch.Tensor, o1: torch.Tensor, w2: torch.Tensor | None = None, o2: torch.Tensor | None = None,
+              pdl: bool = False) -> None:
+    """o1 = rmsnorm(x) * w1 and, in the same pass, o2 = rmsnorm(x) * w2, for the first ``k`` columns; pad columns of the results are zeroed."""
+    a = NormRowsArgs(ptr(x), x.stride(0), k, o1.stride(0), eps, ptr(w1), ptr(w2), ptr(o1), ptr(o2), _is32(o1))
+    _call("b2_norm_rows", a, x.shape[0], int(pdl))
+
+
+def join_rows(a: torch.Tensor, n_a: int, out: torch.Tensor, b: torch.Tensor | None = None, n_b: int = 0, off_b: int = 0, pdl: bool = False) -> None:
+    """Columns 0 .. n_a - 1 of ``a`` and, from column ``off_b`` on, ``n_b`` columns of ``b``; zeros elsewhere; in the result's element type."""
+    args = JoinRowsArgs(ptr(a), ptr(b), a.stride(0), n_a, b.stride(0) if b is not None else 0, n_b, ptr(out), out.stride(0), off_b, _is32(out))
+    _call("b2_join_rows", args, a.shape[0], int(pdl))
+
+
+def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = None, act: str = "", accumulate: bool = False) -> RowSeg:
+    """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``."""
+    return RowSeg(ptr(w), ptr(g), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate))
+
+
+def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,
+         k1: int = 0, conv=None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None, pdl: bool = False) -> None:
+    """``conv`` = (weights [taps, k], bias [k], state [slots, taps - 1, k])."""
+    a = GemvRowsArgs()
+    for i, s in enumerate(segs):
+        a.seg[i] = s
+    a.nseg, a.nb, a.k, a.src, a.f32, a.x, a.ldx, a.eps, a.kn = len(segs), nb, k, src, int(f32), ptr(x), x.stride(0), eps, kn
+    if x2 is not None:
+        a.x2, a.ldx2, a.k1 = ptr(x2), x2.stride(0), k1
+    if conv is not None:
+        a.conv_w, a.conv_b, a.conv_state, a.taps = ptr(conv[0]), ptr(conv[1]), ptr(conv[2]), conv[0].shape[0]
+        a.slots, a.positions = ptr(slots), ptr(positions)
+    _call("b2_gemv_rows", a, int(pdl))
+
+
+def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", accumulate: bool = False, k: int | None = None) -> None:
+    """out (+)= act(a[:, :k] @ w[:, :k]^T); bf16 operands on tcgen05 (result bf16 or fp32), fp32 operands in full 32 bits.  ``a`` and ``out`` may be
+    column windows of wider buffers."""
+    m, n, k = a.shape[0], w.shape[0], w.shape[1] if k is None else k
+    if a.dtype != w.dtype or out.shape[0] != m or out.shape[1] != n or a.shape[1] < k or a.stride(1) != 1 or out.stride(1) != 1:
+        raise ValueError(f"gemm: {tuple(a.shape)} {a.dtype} x {tuple(w.shape)} {w.dtype} -> {tuple(out.shape)}")
+    if a.dtype == torch.float32:
+        f = lib().b2_gemm_f32
+        f.argtypes = [P, I, P, I, I, I, I, P, I, I, I, P]
+        _check(f(ptr(a), a.stride(0), ptr(w), w.stride(0), m, n, k, ptr(out), out.stride(0), ACT[act], int(accumulate), stream()), "gemm_f32")
+        return
+    f = lib().b2_gemm_bf16_act
+    f.argtypes = [P, I, P, I, I, I, P, I, I, I, I, P]
+    _check(f(ptr(a), a.stride(0), ptr(w), m, n, k, ptr(out), out.stride(0), 1 - _is32(out), ACT[act], int(accumulate), stream()), "gemm_bf16_act")
+
+
+def paged_append(qkv, *, heads, kv_heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, positions, slots, table, q_out, k_cache, v_cache, pdl=False) -> None:
+    """Norm over the whole q / k projections, rotation, q to padded fp32 rows [rows, H, dq], k and v into the paged caches."""
+    a = PagedAppendArgs(ptr(qkv), qkv.stride(0), heads, kv_heads, dim, vdim, ptr(q_norm), ptr(k_norm), eps, ptr(freqs), n_rot, ptr(positions), ptr(slots),
+                        ptr(table), table.shape[1], ptr(q_out), q_out.shape[2], ptr(k_cache), ptr(v_cache), k_cache.shape[3], v_cache.shape[3], _is32(k_cache))
+    _call("b2_paged_append", a, qkv.shape[0], int(pdl))
+
+
+def paged_attn(q, k_cache, v_cache, positions, slots, table, out, *, dim, vdim, scale, softcap=0.0, chunk=0, pdl=False) -> None:
+    """Attention of any head size over a paged cache: q [rows, H, dq] fp32 -> out[row, h * vdim ...]."""
+    a = PagedAttnArgs(ptr(q), q.shape[2], q.shape[1], k_cache.shape[1], dim, vdim, ptr(k_cache), ptr(v_cache), k_cache.shape[3], v_cache.shape[3], _is32(k_cache),
+                      ptr(positions), ptr(slots), ptr(table), table.shape[1], chunk, scale, softcap, ptr(out), out.stride(0), 1 - _is32(out))
+    _call("b2_paged_attn", a, q.shape[0], int(pdl))
+
+
+def attn_prefill_paged(q, k_cache, v_cache, tiles, table, out, *, vdim, scale, softcap=0.0, chunk=0) -> None:
+    """tcgen05 attention of query tiles ([n, 4] int32: first row, rows, slot, position) over a paged f16 cache of row length 64 or 128."""
+    a = AttnPrefillArgs(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), None, q.shape[0], q.shape[1], k_cache.shape[1], 0, 0, 0, 0, 1, 0, scale, softcap, None, None)
+    pg = AttnPagedArgs(ptr(tiles), ptr(table), table.shape[1], chunk, vdim, out.stride(0))
+    _check(lib().b2_attn_prefill_paged(C.byref(a), C.byref(pg), q.shape[2], tiles.shape[0], k_cache.shape[0], stream()), "attn_prefill_paged")
+
+
+def attn_decode_paged(qkv, k_cache, v_cache, positions, slots, table, out, nb, *, heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, scale, softcap,
+                      chunk, n_splits, n_ctx, part_acc, part_ml, pdl=False) -> bool:
+    """Decode attention on raw projections: norms, rotation, cache append, split-K attention, merge.  False: shape not taken, nothing launched."""
+    hd = k_cache.shape[3]
+    a = AttnDecodeArgs(None, ptr(k_cache), ptr(v_cache), ptr(positions), ptr(slots), heads, k_cache.shape[1], n_ctx, n_splits, scale, softcap, 0,
+                       ptr(part_acc), ptr(part_ml), None, None, ptr(table), table.shape[1], chunk)
+    r = AttnRopeArgs(ptr(qkv), None, 1.0, n_rot, 1, ptr(q_norm), ptr(k_norm), eps, qkv.stride(0), dim, vdim, ptr(freqs))
+    f = lib().b2_attn_decode_paged
+    f.argtypes = [P, P, I, I, P, I, I, I, P]
+    rc = f(C.addressof(a), C.addressof(r), nb, hd, ptr(out), out.stride(0), 1 - _is32(out), int(pdl), stream())
+    if rc == 801:
+        return False
+    _check(rc, "attn_decode_paged")
+    return True
+
+
+def ssm_conv(xz, inner, w, b, state, slots, positions, offs, u, pdl=False) -> None:
+    a = SsmConvArgs(ptr(xz), xz.stride(0), inner, w.shape[0], ptr(w), ptr(b), ptr(state), ptr(slots), ptr(positions), ptr(offs), ptr(u), u.stride(0))
+    _call("b2_ssm_conv", a, xz.shape[0], _is32(xz), int(pdl))
+
+
+def ssm_scan(xz, off_z, u, dt, bc, off_b, dt_bias, a2, d, taps, state, conv_state, segs, out, pdl=False) -> None:
+    """``segs`` [n, 4] int32: first row, rows, slot, position of the first row."""
+    a = SsmScanArgs(ptr(xz), xz.stride(0), off_z, ptr(u), u.stride(0), ptr(dt), dt.stride(0), ptr(bc), bc.stride(0), off_b, ptr(dt_bias), ptr(a2), ptr(d),
+                    a2.shape[0], a2.shape[1], taps, ptr(state), ptr(conv_state), ptr(segs), ptr(out), out.stride(0))
+    _call("b2_ssm_scan", a, segs.shape[0], _is32(u), int(pdl))
+
+
+def ssm_step(xz, off_z, conv, p, off_b, w_dt, dt, dt_bias, a2, d, state, slots, positions, out, nb, exact=False, pdl=False) -> None:
+    """One token per sequence.  ``dt``: projected step sizes, or None: projected inside from the first columns of ``p``.
+    ``exact``: ``a2`` holds A instead of log2(e) A (32-bit models)."""
+    a = SsmStepArgs(ptr(xz), xz.stride(0), off_z, 1 - _is32(xz), ptr(conv[0]), ptr(conv[1]), ptr(conv[2]), conv[0].shape[0], a2.shape[0], a2.shape[1],
+                    ptr(p), p.stride(0), off_b, ptr(w_dt), w_dt.shape[1], _is32(w_dt), ptr(dt), dt.stride(0) if dt is not None else 0, ptr(dt_bias), ptr(a2),
+                    ptr(d), ptr(state), ptr(slots), ptr(positions), ptr(out), out.stride(0), 1 - _is32(out), int(exact))
+    _call("b2_ssm_step", a, nb, int(pdl))

@@ -71,7 +71,7 @@ def target_tensor_type(name: str, shape: tuple[int, ...], cur: GGMLType, ft: Fil
     """Per-tensor encoding inside a file of type ``ft`` (same rule the synthetic generator uses)."""
     from ..models.synth import use_more_bits
     if len(shape) == 1 or "ffn_gate_inp" in name or "_norm." in name or name.startswith(("v.", "mm.", "a.")) or "rope_freqs" in name \
-            or "attn_sinks" in name or name.endswith(".bias"):
+            or "attn_sinks" in name or name.endswith((".bias", "ssm_a", "ssm_d", "ssm_conv1d.weight")):
         return cur if cur in (GGMLType.F32, GGMLType.F16, GGMLType.BF16) else GGMLType.F32
     if ft in (FileType.F32, FileType.F16, FileType.BF16):
         return {FileType.F32: GGMLType.F32, FileType.F16: GGMLType.F16, FileType.BF16: GGMLType.BF16}[ft]
@@ -163,7 +163,7 @@ def create_model(req: dict[str, Any]) -> Iterator[dict[str, Any]]:
             out = os.path.join(tmp, "model.gguf")
             try:
                 convert_hf(tmp, out)
-            except (ConvertError, KeyError, OSError) as e:
+            except (ConvertError, ValueError, KeyError, OSError) as e:
                 raise CreateError(f"conversion failed: {e}") from None
             layer = M.new_layer(out, M.MT_MODEL)
         layers.append(layer)

@@ -67,14 +67,6 @@ class PagedCache:
             self.table_np[slot] = 0
             self._dirty = True
 
-    def trim(self, slot: int, n_tokens: int) -> None:
-        """Give back the pages behind the first ``n_tokens`` positions."""
-        own, keep = self.owned[slot], -(-n_tokens // PAGE)
-        while len(own) > keep:
-            self.free.append(own.pop())
-            self.table_np[slot, len(own)] = 0
-            self._dirty = True
-
     def sync(self) -> int:
         """Bring the device's page table up to date; returns the bytes copied."""
         if not self._dirty:
@@ -85,7 +77,6 @@ class PagedCache:
 
     def copy(self, src: int, dst: int, n_tokens: int) -> None:
         """Positions 0 .. n_tokens - 1 and the state of slot ``src`` become those of slot ``dst``."""
-        self.trim(dst, n_tokens)
         self.reserve(dst, n_tokens)
         n = -(-n_tokens // PAGE)
         if n:

@@ -44,6 +44,7 @@ class RunnerOptions:
     draft_path: str = ""              # a smaller model of the same vocabulary that drafts tokens (Modelfile DRAFT)
     draft_num_predict: int = 4        # tokens drafted per verification pass (api/types.go:1119)
     dtype: str = "bfloat16"           # compute type of models that also run in 32 bits ("float32")
+    kv_pool_tokens: int = 0           # paged caches: positions all slots hold together (0: every slot can fill its context)
     shift_mode: str = "rotate"        # context shift: "rotate" re-rotates the cached keys in place, "recompute" evaluates the kept tokens again
 
 
@@ -168,7 +169,8 @@ class Runner:
         self.n_ctx = n_ctx
         self.n_slots = max(1, int(self.opts.num_parallel))
         with self._on(self._cuda_device):
-            self.backend.alloc(self.n_slots, self.n_ctx)
+            paged = int(self.opts.kv_pool_tokens) > 0 and hasattr(self.backend, "admit")
+            self.backend.alloc(self.n_slots, self.n_ctx, **({"pool_tokens": int(self.opts.kv_pool_tokens)} if paged else {}))
             self.draft = None
             if self.opts.draft_path and int(self.opts.draft_num_predict) > 0 and getattr(self.backend, "supports_verify", False):
                 self._load_draft()
@@ -199,7 +201,7 @@ class Runner:
         dev = str(getattr(self.backend, "device", self.opts.device))
         draft = make_backend(g, dev if dev.startswith("cuda") else "cpu", opts=self.opts) if dev.startswith("cuda") \
             else make_backend(g, "cpu")
-        if draft.cfg.vocab_size != self.cfg.vocab_size:
+        if draft.cfg.vocab_size != self.cfg.vocab_size or draft.cfg.recurrent:      # a recurrent draft cannot take rejected tokens back
             draft.close()
             return
         draft.alloc(self.n_slots, self.n_ctx)
@@ -373,6 +375,8 @@ class Runner:
             from ..models.config import config_from_gguf
             from ..parallel.tp_engine import shard_plan
             cfg = config_from_gguf(self.gguf)
+            if cfg.stack is not None:
+                return []
             shard_plan(cfg, tp, {n: t.dtype for n, t in self.gguf.tensors.items()})
             if cfg.sandwich_norm or cfg.d_model > 8192:
                 return []
@@ -462,7 +466,14 @@ class Runner:
             reuse = max(0, min(best_lcp, len(seq.prompt) - 1))   # always evaluate at least one token
             if seq.req.embedding or not self.cfg.causal:
                 reuse = 0
-            elif seq.req.cache_prompt and hasattr(self.backend, "copy_rows"):
+            if self.cfg.recurrent and reuse != len(self.slot_tokens[best]):
+                reuse = 0            # a state stands behind the last token the slot has seen: all of it is a prefix, or none
+            if hasattr(self.backend, "admit") and not self._reserve(seq, best, free):
+                self.pending.insert(0, seq)      # the page pool is busy: wait for a sequence to end
+                return
+            if seq.state == "done":
+                continue
+            if seq.req.cache_prompt and not seq.req.embedding and self.cfg.causal and hasattr(self.backend, "copy_rows"):
                 # a longer prefix of this prompt may sit in another slot, busy or not: its cache rows are copied over
                 # (x/mlxrunner/prefix_cache.go:86-140 keeps such prefixes in a trie of snapshots; here the slots are the store)
                 donor, donor_lcp = -1, reuse + self.PREFIX_COPY_MIN - 1
@@ -472,7 +483,7 @@ class Runner:
                     other = self.slot_seq[i]
                     valid = self.slot_tokens[i] if other is None else self.slot_tokens[i][:other.n_past]
                     lcp = min(_common_prefix(valid, seq.prompt), len(seq.prompt) - 1)
-                    if lcp > donor_lcp:
+                    if lcp > donor_lcp and not (self.cfg.recurrent and lcp != len(valid)):
                         donor, donor_lcp = i, lcp
                 if donor >= 0:
                     self.backend.copy_rows(donor, best, donor_lcp)
@@ -499,6 +510,20 @@ class Runner:
                 continue
             seq.limit = r.num_predict if r.num_predict >= 0 else 10 * self.n_ctx
 
+    def _reserve(self, seq: _Seq, slot: int, free: list[int]) -> bool:
+        """Room in a paged cache for all the tokens the sequence may come to hold; slots without a sequence give up their cached
+        prefixes for it, the longest unused first.  False: not now, running sequences hold the pages."""
+        n = min(self.n_ctx, len(seq.prompt) + (seq.req.num_predict if seq.req.num_predict >= 0 else self.n_ctx))
+        idle = sorted((i for i in free if i != slot), key=lambda i: self.slot_used_at[i])
+        ok, dropped = self.backend.admit(slot, n, idle)
+        for i in dropped:
+            self.slot_tokens[i] = []
+        if not ok and not any(self.slot_seq):
+            seq.slot = -1
+            self._fail(seq, RunnerError(f"the cache pool is too small for a sequence of {n} tokens"))
+            return True
+        return ok
+
     def _step(self) -> None:
         active = [s for s in self.slot_seq if s is not None]
         for s in active:
@@ -507,6 +532,11 @@ class Runner:
         # one prefill pass per iteration keeps decode latency of the other slots bounded; the pass takes rows of every
         # sequence that is waiting for its prompt, up to num_batch rows in all, when the backend can run them as one matrix
         waiting = [s for s in active if s.state == "prefill"]
+        running = [s for s in active if s.state == "decode"]
+        if waiting and running and hasattr(self.backend, "step") and not any(s.req.embedding or s.image_rows or s.pixels for s in waiting):
+            with self._range("mixed_step"):       # portions of prompts beside single tokens: one batch
+                self._mixed(waiting, running)
+            return
         if len(waiting) > 1 and hasattr(self.backend, "prefill_many") and not any(s.req.embedding or s.image_rows or s.pixels for s in waiting):
             with self._range("prefill_batch"):
                 self._prefill_batch(waiting)
@@ -571,30 +601,62 @@ class Runner:
         came first reaches its first token first and short prompts ride along in what a longer one leaves over (the order in which
         the reference's runner packs the prompts of its slots into a batch)."""
         t0 = time.perf_counter()
-        budget = max(1, self.opts.num_batch)
-        left = {id(s): len(s.prompt) - s.n_past for s in seqs}
-        take = {id(s): 0 for s in seqs}
-        for s in seqs:
-            if budget == 0:
-                break
-            take[id(s)] = min(left[id(s)], budget)
-            budget -= take[id(s)]
-        part = [s for s in seqs if take[id(s)] > 0]
-        segs = [(s.slot, s.prompt[s.n_past:s.n_past + take[id(s)]], s.n_past) for s in part]
-        last = [take[id(s)] == left[id(s)] for s in part]
+        part, segs, last = self._portions(seqs, max(1, self.opts.num_batch))
         outs = self.backend.prefill_many(segs, last)
         if not any(last):
             _sync(None)
         self.stats["prefill_batches"] = self.stats.get("prefill_batches", 0) + 1
         for s, (_, chunk, _), done, logits in zip(part, segs, last, outs):
-            s.n_past += len(chunk)
-            s.n_prompt_eval += len(chunk)
-            self.slot_tokens[s.slot].extend(chunk)
-            if done:
-                s.state = "decode"
-                self._sample_accept(s, logits)   # reads the logits: the pass has finished on the device
-                s.t_first = time.perf_counter() - s.t_submit
-            s.t_prefill += time.perf_counter() - t0
+            self._advance_prompt(s, chunk, logits if done else None, t0)
+
+    @staticmethod
+    def _portions(seqs: list[_Seq], budget: int) -> tuple[list[_Seq], list[tuple], list[bool]]:
+        """Fill ``budget`` rows with prompt tokens in arrival order: (sequences, their portions, whether a portion ends its prompt)."""
+        part, segs, last = [], [], []
+        for s in seqs:
+            n = min(len(s.prompt) - s.n_past, budget)
+            if n > 0:
+                part.append(s)
+                segs.append((s.slot, s.prompt[s.n_past:s.n_past + n], s.n_past))
+                last.append(s.n_past + n == len(s.prompt))
+                budget -= n
+        return part, segs, last
+
+    def _advance_prompt(self, s: _Seq, chunk: list[int], logits, t0: float) -> None:
+        """A portion of the sequence's prompt has been evaluated; ``logits``: behind its last token when that ended the prompt."""
+        s.n_past += len(chunk)
+        s.n_prompt_eval += len(chunk)
+        self.slot_tokens[s.slot].extend(chunk)
+        if logits is not None:
+            s.state = "decode"
+            self._sample_accept(s, logits)   # reads the logits: the pass has finished on the device
+            s.t_first = time.perf_counter() - s.t_submit
+        s.t_prefill += time.perf_counter() - t0
+
+    def _mixed(self, waiting: list[_Seq], running: list[_Seq]) -> None:
+        """One step of the backend over the next token of every running sequence and prompt portions of the waiting ones."""
+        t0 = time.perf_counter()
+        ready = [s for s in running if s.n_past + 1 <= self.n_ctx or self._shift(s)]
+        part, segs, last = self._portions(waiting, max(1, self.opts.num_batch - len(ready)))
+        rows = self.backend.step([(s.slot, [s.next_token], s.n_past) for s in ready] + segs,
+                                 [[0]] * len(ready) + [[len(seg[1]) - 1] if end else [] for seg, end in zip(segs, last)])
+        if rows is None:
+            _sync(None)
+        st = self.stats
+        st["mixed_steps"] = st.get("mixed_steps", 0) + 1
+        st["decode_steps"] += 1
+        st["decode_step_sequences"] += len(ready)
+        dt = time.perf_counter() - t0
+        for i, s in enumerate(ready):
+            self.slot_tokens[s.slot].append(s.next_token)
+            s.n_past += 1
+            s.t_decode += dt
+            s.n_decoded += 1
+            self._sample_accept(s, rows[i])
+        at = len(ready)
+        for s, (_, chunk, _), end in zip(part, segs, last):
+            self._advance_prompt(s, chunk, rows[at] if end else None, t0)
+            at += end
 
     def _decode(self, seqs: list[_Seq]) -> None:
         with self._range("decode_step"):
@@ -722,13 +784,12 @@ class Runner:
         toks = self.slot_tokens[s.slot]
         discard = max(1, (len(toks) - keep) // 2)
         new = toks[:keep] + toks[keep + discard:]
-        if hasattr(self.backend, "shift") and self.opts.shift_mode != "recompute":
+        if hasattr(self.backend, "shift") and getattr(self.backend, "supports_shift", True) and self.opts.shift_mode != "recompute":
             # the cache rows of the dropped tokens are removed and the keys behind them re-rotated to their new positions
             self.backend.shift(s.slot, keep, discard, len(toks))
         else:
-            self.slot_tokens[s.slot] = new[:keep]
-            tail = new[keep:]
-            pos = keep
+            pos = 0 if self.cfg.recurrent else keep      # a recurrent state has to see the kept tokens again as well
+            tail = new[pos:]
             while tail:
                 chunk, tail = tail[: self.opts.num_batch], tail[self.opts.num_batch:]
                 self.backend.prefill(s.slot, chunk, pos, need_logits=False)

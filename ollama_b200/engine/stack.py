@@ -29,7 +29,7 @@ from ..models.weights import QWeight, load_tensor
 from ..ops import cuda as K
 from ..ops import reference as R
 from ..ops import rows as O
-from .cache import PagedCache
+from .cache import CacheFull, PagedCache
 from .steps import StepEngine
 
 MAX_DECODE_ROWS = 32
@@ -230,6 +230,21 @@ class StackBackend(StepEngine):
     def close(self) -> None:
         self._graphs.clear()
         self.mem, self.cache, self.buf = [], None, None
+
+    def admit(self, slot: int, n_tokens: int, idle: Sequence[int]) -> tuple[bool, list[int]]:
+        """Reserve pages for ``n_tokens`` positions of ``slot``, giving up what the ``idle`` slots still hold, in their order, as far as
+        needed.  Returns whether that sufficed and the slots that were emptied."""
+        dropped: list[int] = []
+        for s in [None, *idle]:
+            if s is not None:
+                self.cache.release(s)
+                dropped.append(s)
+            try:
+                self.cache.reserve(slot, n_tokens)
+                return True, dropped
+            except CacheFull:
+                continue
+        return False, dropped
 
     def free_slot(self, slot: int) -> None:
         """The sequence in ``slot`` has ended: its pages go back to the pool."""

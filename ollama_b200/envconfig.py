@@ -275,6 +275,12 @@ def pp_degree() -> int:
     return _uint("B200_PP", 0)
 
 
+def compute_dtype() -> str:
+    """B200_DTYPE: bfloat16 or float32, for models that also run in 32 bits."""
+    v = var("B200_DTYPE") or "bfloat16"
+    return v if v in ("bfloat16", "float32") else "bfloat16"
+
+
 def replicas() -> int:
     """B200_REPLICAS: whole copies of a model on different GPUs, requests spread over them; 0 or 1 = one runner."""
     return _uint("B200_REPLICAS", 0)
@@ -335,6 +341,7 @@ def as_map() -> dict[str, tuple[object, str]]:
         "B200_TC_DECODE_MIN": (var("B200_TC_DECODE_MIN") or "4", "Decode steps of at least this many sequences multiply 16-bit matrices on the tcgen05 GEMM (0 = never)"),
         "B200_MOE_STREAM_Q": (var("B200_MOE_STREAM_Q") or "1", "MoE prefill streams MXFP4 experts as they are when no 16-bit copy is resident (0 = expand per chunk)"),
         "B200_SK": (var("B200_SK") or "1", "Streaming decode GEMV for Q4_K / Q6_K / Q8_0 layers (0 = plane kernels)"),
+        "B200_DTYPE": (compute_dtype(), "Compute type of models that also run in 32 bits: bfloat16 or float32"),
         "B200_NVTX": (_bool("B200_NVTX"), "NVTX ranges around prefill chunks and decode steps"),
         "B200_NO_NATIVE": (_bool("B200_NO_NATIVE"), "Do not load the C++ host helpers (codecs, BPE merges)"),
         "B200_COMM": (comm_mode(), "Collective implementation: p2p (fused kernels) or nccl"),

@@ -106,8 +106,7 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
         if self.stack is not None:
-            ms = [self.stack.layers[r.layer].mixer for r in self.stack.runs()]
-            return sum(m.kv_heads * (m.dim + m.vdim) for m in ms if isinstance(m, AttentionMixer)) * elem_bytes
+            return self.stack.kv_bytes_per_token(elem_bytes)
         return self.n_layers * (self.n_kv_heads * (self.head_dim + self.v_head_dim)) * elem_bytes
 
 

@@ -95,6 +95,16 @@ class Stack:
         return ([LayerRun(i, False) for i in range(lo)] + [LayerRun(i, i == lo) for _ in range(times) for i in range(lo, hi)]
                 + [LayerRun(i, False) for i in range(hi, len(self.layers))])
 
+    def kv_bytes_per_token(self, elem_bytes: int = 2) -> int:
+        """Cache bytes of one position over all layer runs."""
+        ms = [self.layers[r.layer].mixer for r in self.runs()]
+        return sum(m.kv_heads * (m.dim + m.vdim) for m in ms if isinstance(m, AttentionMixer)) * elem_bytes
+
+    def state_bytes(self) -> int:
+        """Recurrent state of one sequence over all layer runs (fp32)."""
+        ms = [self.layers[r.layer].mixer for r in self.runs()]
+        return sum(4 * m.inner * (m.state + m.conv - 1) for m in ms if isinstance(m, MambaMixer))
+
     @property
     def recurrent(self) -> bool:
         return any(isinstance(L.mixer, MambaMixer) for L in self.layers)

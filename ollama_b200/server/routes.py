@@ -338,7 +338,7 @@ class Server:
             return JSONResponse({"model": name, "created_at": _now(), "_debug_info": {"rendered_template": text}})
         tokens: Any = text
         if req.get("context"):
-            tokens = [int(t) for t in req["context"]] + runner.tokenize(text, add_special=False)
+            tokens = [int(t) for t in req["context"]] + (runner.tokenize(text, add_special=False) if text else [])
         creq = CompletionRequest(prompt=tokens, sampling=self._sampling(opts, bool(req.get("logprobs")), top_lp), num_predict=opts["num_predict"],
                                  num_keep=opts["num_keep"], stop=list(opts.get("stop") or []), grammar=grammar,
                                  grammar_after="" if req.get("raw") else self._grammar_gate(rend, grammar, think, text),

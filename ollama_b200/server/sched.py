@@ -124,6 +124,10 @@ def predict_memory(model: Any, num_ctx: int, num_parallel: int, free: int | None
     size = int(getattr(model, "size", 0) or 0)
     kv = getattr(model, "kv", lambda: {})() or {}
     arch = kv.get("general.architecture", "")
+    if isinstance(kv.get(f"{arch}.stack"), str):     # layers of different kinds: their own count of cache and state
+        from ..models.stack import parse_stack
+        st = parse_stack(kv[f"{arch}.stack"])
+        return size + num_parallel * (st.kv_bytes_per_token() * num_ctx + st.state_bytes())
     layers = _first_int(kv.get(f"{arch}.block_count"))
     heads = _first_int(kv.get(f"{arch}.attention.head_count"), 1) or 1
     kvh = _first_int(kv.get(f"{arch}.attention.head_count_kv"), heads) or heads
@@ -486,7 +490,7 @@ def _default_runner_on(model: Any, opts: dict[str, Any], num_parallel: int, gpus
     if len(gpus) == 1 and device in ("auto", "cuda"):
         device = f"cuda:{gpus[0].index}"            # the GPU the placement chose, not whichever is current
     ro = RunnerOptions(num_ctx=int(opts.get("num_ctx") or 4096), num_batch=int(opts.get("num_batch") or 512), num_parallel=num_parallel,
-                       kv_cache_type=envconfig.kv_cache_type() or "f16", device=device, tp=max(1, len(gpus)),
+                       kv_cache_type=envconfig.kv_cache_type() or "f16", dtype=envconfig.compute_dtype(), device=device, tp=max(1, len(gpus)),
                        gpu_ids=tuple(g.index for g in gpus),
                        adapter_paths=tuple(getattr(model, "adapter_paths", None) or ()),
                        draft_path=(getattr(model, "draft_paths", None) or [""])[0],

@@ -65,7 +65,9 @@ def join_rows(a: torch.Tensor, n_a: int, out: torch.Tensor, b: torch.Tensor | No
 
 def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = None, act: str = "", accumulate: bool = False) -> RowSeg:
     """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``."""
-    return RowSeg(ptr(w), ptr(g), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate))
+    s = RowSeg(ptr(w), ptr(g), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate))
+    s.keep = (w, g, out)             # the structure holds addresses only
+    return s
 
 
 def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,

@@ -1,6 +1,9 @@
 """Plain, slow implementation of the Vazatar design, written from its equations: whole sequences, no cache, no batching, one
 function per mechanism.  The tests compare the framework with it; nothing here is shared with the product path.
 
+``product`` is how every matrix product is formed; :func:`rounded` rounds its input to bf16 first, which shows what that precision alone does
+to the logits of a model.
+
 A model is a pair ``(config, weights)``: the dictionary of ``config.json`` and a dictionary of tensors by name.
 """
 import math
@@ -8,6 +11,14 @@ import math
 import torch
 
 F64 = torch.float64
+
+
+def exact(x, w):
+    return x @ w.t()
+
+
+def rounded(x, w):
+    return x.to(torch.bfloat16).to(x.dtype) @ w.t()
 
 
 def rms(x, eps):
@@ -75,20 +86,20 @@ def attend(q, k, v, scale, cap=0.0, size=0):
     return out
 
 
-def attention_mixer(h, w, m, eps):
+def attention_mixer(h, w, m, eps, product=exact):
     """``w(name)`` gives a tensor of the layer's mixer."""
     T = h.shape[0]
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q = norm_plain(h @ w("q").t(), w("q.norm"), eps).view(T, H, d)
-    k = norm_plain(h @ w("k").t(), w("k.norm"), eps).view(T, G, d)
-    v = (h @ w("v").t()).view(T, G, dv)
+    q = norm_plain(product(h, w("q")), w("q.norm"), eps).view(T, H, d)
+    k = norm_plain(product(h, w("k")), w("k.norm"), eps).view(T, G, d)
+    v = product(h, w("v")).view(T, G, dv)
     rot = m.get("rot")
     if rot:
         f = rotary_freqs(rot["base"], rot["dims"], rot.get("scaling"))
         pos = torch.arange(T)
         q, k = rotate(q, pos, f), rotate(k, pos, f)
     o = attend(q, k, v, m["scale"], m.get("softcap") or 0.0, (m.get("mask") or {}).get("size", 0))
-    return o.reshape(T, H * dv) @ w("o").t()
+    return product(o.reshape(T, H * dv), w("o"))
 
 
 def causal_conv(x, taps, bias):
@@ -120,23 +131,23 @@ def selective_scan(x, dt, A, B, C, D):
     return y
 
 
-def mamba_mixer(h, w, m):
+def mamba_mixer(h, w, m, product=exact):
     inner, n, r = m["inner"], m["state"], m["dt_rank"]
-    xz = h @ w("in").t()
+    xz = product(h, w("in"))
     x, z = xz[:, :inner], xz[:, inner:]
     x = silu(causal_conv(x, w("conv"), w("conv.b")))
-    p = x @ w("x").t()
-    dt = softplus(p[:, :r] @ w("dt").t() + w("dt.b"))
+    p = product(x, w("x"))
+    dt = softplus(product(p[:, :r], w("dt")) + w("dt.b"))
     y = selective_scan(x, dt, -torch.exp(w("A_log")), p[:, r:r + n], p[:, r + n:], w("D"))
-    return (y * silu(z)) @ w("o").t()
+    return product(y * silu(z), w("o"))
 
 
 def relu2(x):
     return torch.clamp(x, min=0.0) ** 2
 
 
-def dense_ff(h, up, down):
-    return relu2(h @ up.t()) @ down.t()
+def dense_ff(h, up, down, product=exact):
+    return product(relu2(product(h, up)), down)
 
 
 def schedule(cfg):
@@ -151,7 +162,7 @@ def schedule(cfg):
 
 
 @torch.no_grad()
-def forward(cfg, weights, tokens, dtype=F64, residuals=None):
+def forward(cfg, weights, tokens, dtype=F64, residuals=None, product=exact):
     """Logits [T, vocab] of a whole sequence; ``residuals``: a list that receives the residual stream after every layer run."""
     W = {k: v.to(dtype) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
@@ -159,16 +170,16 @@ def forward(cfg, weights, tokens, dtype=F64, residuals=None):
     for i, first in schedule(cfg):
         L = cfg["layers"][i]
         if first:
-            x = torch.cat([x, x0], -1) @ W["loop.in"].t()
+            x = product(torch.cat([x, x0], -1), W["loop.in"])
         h = norm_one_plus(x, W[f"l{i}.norm1"], eps)
 
         def w(name, i=i):
             return W[f"l{i}.mix.{name}"]
 
-        y = attention_mixer(h, w, L["mixer"], eps) if L["type"] == "attention" else mamba_mixer(h, w, L["mixer"])
+        y = attention_mixer(h, w, L["mixer"], eps, product) if L["type"] == "attention" else mamba_mixer(h, w, L["mixer"], product)
         if L.get("mlp"):
-            y = y + dense_ff(norm_one_plus(x, W[f"l{i}.norm2"], eps), W[f"l{i}.mlp.up"], W[f"l{i}.mlp.down"])
+            y = y + dense_ff(norm_one_plus(x, W[f"l{i}.norm2"], eps), W[f"l{i}.mlp.up"], W[f"l{i}.mlp.down"], product)
         x = x + y
         if residuals is not None:
             residuals.append(x)
-    return softcap(norm_one_plus(x, W["final.norm"], eps) @ W["head"].t(), cfg.get("logit_softcap") or 0.0)
+    return softcap(product(norm_one_plus(x, W["final.norm"], eps), W["head"]), cfg.get("logit_softcap") or 0.0)

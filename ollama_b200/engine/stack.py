@@ -285,7 +285,12 @@ class StackBackend(StepEngine):
             segs = [O.seg(L.w_in, n_in, h_in, L.norm1)]
             if L.ffp:
                 segs.append(O.seg(L.up, L.ffp, cat[:, L.mixp:], L.norm2, act))
-            O.gemv(segs, wp, x, nb, self.f32, O.SRC_NORM, eps, self.stack.width, pdl=pdl)
+            if isinstance(L.mixer, MambaMixer):      # the convolution follows in the product's epilogue
+                u = B.get("u", L.inner, f32, nb)
+                O.gemv(segs, wp, x, nb, self.f32, O.SRC_NORM, eps, self.stack.width, conv=(L.conv_w, L.conv_b, self.mem[i][1]), conv_out=u, slots=m.slots,
+                       positions=m.positions, pdl=pdl)
+            else:
+                O.gemv(segs, wp, x, nb, self.f32, O.SRC_NORM, eps, self.stack.width, pdl=pdl)
         else:
             h1, h2 = B.get("h1", wp, AT, nb), B.get("h2", wp, AT, nb) if L.ffp else None
             O.norm_rows(x, self.stack.width, eps, L.norm1, h1, L.norm2, h2, pdl=pdl)
@@ -328,8 +333,9 @@ class StackBackend(StepEngine):
         p = B.get("p", L.np, f32, nb)
         conv = (L.conv_w, L.conv_b, conv_state)
         if small:
-            O.gemv([O.seg(L.w_x, L.np, p)], L.inner, xz, nb, self.f32, O.SRC_CONV, conv=conv, slots=m.slots, positions=m.positions, pdl=pdl)
-            O.ssm_step(xz, L.inner, conv, p, L.r8, L.w_dt, None, L.dt_bias, L.a2, L.d, state, m.slots, m.positions, out, nb, self.f32, pdl=pdl)
+            u = B.get("u", L.inner, f32, nb)
+            O.gemv([O.seg(L.w_x, L.np, p)], L.inner, u, nb, self.f32, pdl=pdl)
+            O.ssm_step(xz, L.inner, conv, p, L.r8, L.w_dt, None, L.dt_bias, L.a2, L.d, state, m.slots, m.positions, out, nb, self.f32, u, pdl=pdl)
             self._n += 2
             return
         u, dl, dt = B.get("u", L.inner, xz.dtype, nb), B.get("dl", L.r8, xz.dtype, nb), B.get("dt", L.inner, f32, nb)

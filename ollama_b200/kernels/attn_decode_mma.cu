@@ -143,12 +143,26 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         if (PAGED) {
             const float* tok = r.qkv + (size_t)b * r.ldq;
             const int nq = a.n_heads * r.dim, nk = a.n_kv_heads * r.dim;
+            for (int p = tid; p < (r.n_rot >> 1); p += 128) sincosf(rot_angle(qpos, r.freqs[p]), &s_sn[p], &s_cs[p]);
             float iq = 1.f, ik = 1.f;
             if (r.q_norm) {
                 float s0 = 0.f, s1 = 0.f;
-                for (int i = tid; i < nq; i += 128) s0 += tok[i] * tok[i];
-                if (owner)
-                    for (int i = tid; i < nk; i += 128) s1 += tok[nq + i] * tok[nq + i];
+                const int total = owner ? nq + nk : nq;
+                if (((nq | nk | r.ldq) & 3) == 0) {
+#pragma unroll 8
+                    for (int i = 4 * tid; i < total; i += 512) {
+                        const float4 v = __ldcg(reinterpret_cast<const float4*>(tok + i));
+                        const float d = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                        if (i < nq) s0 += d;
+                        else s1 += d;
+                    }
+                } else {
+                    for (int i = tid; i < total; i += 128) {
+                        const float d = tok[i] * tok[i];
+                        if (i < nq) s0 += d;
+                        else s1 += d;
+                    }
+                }
                 s0 = warp_sum(s0);
                 s1 = warp_sum(s1);
                 if (lane == 0) {
@@ -159,6 +173,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
                 iq = 1.f / sqrtf((s_m[0][0] + s_m[1][0] + s_m[2][0] + s_m[3][0]) / (float)nq + r.eps);
                 ik = 1.f / sqrtf((s_l[0][0] + s_l[1][0] + s_l[2][0] + s_l[3][0]) / (float)nk + r.eps);
             }
+#pragma unroll 4
             for (int c = tid; c < nrows * D; c += 128) {
                 const int rr = c / D, col = c % D;
                 float v = 0.f;
@@ -173,7 +188,6 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
                 }
                 raw[c] = v;
             }
-            for (int p = tid; p < (r.n_rot >> 1); p += 128) sincosf(rot_angle(qpos, r.freqs[p]), &s_sn[p], &s_cs[p]);
         } else {
         const float* tok = r.qkv + (size_t)b * (a.n_heads + 2 * a.n_kv_heads) * D;
         for (int c = tid; c < nrows * (D / 4); c += 128) {

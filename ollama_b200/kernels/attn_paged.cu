@@ -16,7 +16,7 @@ namespace {
 // ---------------------------------------------------------------------------------------------------------------------
 template <typename CT>
 __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant__ PagedAppendArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     __shared__ float red[2][8];
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int nq = a.n_heads * a.dim, nk = a.n_kv_heads * a.dim, half = a.n_rot >> 1;
@@ -28,18 +28,23 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
     const int pos = a.positions[t], slot = a.slots[t];
     const float* row = a.qkv + (size_t)t * a.ldq;
     float s0 = 0.f, s1 = 0.f;
-    for (int i = tid; i < nq + nk; i += 256) {
-        const float v = row[i];
-        sq[i] = v;
-        if (i < nq) s0 += v * v;
-        else s1 += v * v;
+    if (((nq | nk | a.ldq) & 3) == 0) {
+        for (int i = 4 * tid; i < nq + nk; i += 1024) {
+            const float4 v = *(const float4*)(row + i);
+            *(float4*)(sq + i) = v;
+            const float d = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+            if (i < nq) s0 += d;
+            else s1 += d;
+        }
+    } else {
+        for (int i = tid; i < nq + nk; i += 256) {
+            const float v = row[i];
+            sq[i] = v;
+            if (i < nq) s0 += v * v;
+            else s1 += v * v;
+        }
     }
-    for (int p = tid; p < half; p += 256) {
-        float s, c;
-        sincosf(rot_angle(pos, a.freqs[p]), &s, &c);
-        cs[p] = c;
-        sn[p] = s;
-    }
+    for (int p = tid; p < half; p += 256) sincosf(rot_angle(pos, a.freqs[p]), &sn[p], &cs[p]);
     s0 = warp_sum(s0);
     s1 = warp_sum(s1);
     if (lane == 0) {
@@ -47,7 +52,6 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
         red[1][warp] = s1;
     }
     __syncthreads();
-    float iq = 1.f, ik = 1.f;
     if (a.q_norm) {
         s0 = s1 = 0.f;
 #pragma unroll
@@ -55,37 +59,33 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
             s0 += red[0][i];
             s1 += red[1][i];
         }
-        iq = 1.f / sqrtf(s0 / (float)nq + a.eps);
-        ik = 1.f / sqrtf(s1 / (float)nk + a.eps);
+        const float iq = 1.f / sqrtf(s0 / (float)nq + a.eps), ik = 1.f / sqrtf(s1 / (float)nk + a.eps);
+        for (int i = tid; i < nq; i += 256) sq[i] *= iq * __ldg(a.q_norm + i);
+        for (int i = tid; i < nk; i += 256) sq[nq + i] *= ik * __ldg(a.k_norm + i);
+        __syncthreads();
     }
-    auto normed = [&](int i) -> float {
-        const float v = sq[i];
-        if (!a.q_norm) return v;
-        return i < nq ? v * iq * a.q_norm[i] : v * ik * a.k_norm[i - nq];
-    };
-    auto rotated = [&](int base, int d) -> float {
-        const float x = normed(base + d);
+    auto rotated = [&](const float* head, int d) -> float {
+        const float x = head[d];
         if (d >= a.n_rot) return x;
-        const bool first = d < half;
-        const int p = first ? d : d - half;
-        const float y = normed(base + (first ? d + half : p));
-        return first ? x * cs[p] - y * sn[p] : x * cs[p] + y * sn[p];
+        return d < half ? x * cs[d] - head[d + half] * sn[d] : x * cs[d - half] + head[d - half] * sn[d - half];
     };
-    float* qo = a.q_out + (size_t)t * a.n_heads * a.dq;
-    for (int i = tid; i < a.n_heads * a.dq; i += 256) {
-        const int h = i / a.dq, d = i - h * a.dq;
-        qo[i] = d < a.dim ? rotated(h * a.dim, d) : 0.f;
-    }
     const int* table = a.page_table + (size_t)slot * a.max_pages;
-    CT* kc = (CT*)a.k_cache;
-    CT* vc = (CT*)a.v_cache;
-    for (int i = tid; i < a.n_kv_heads * a.dk; i += 256) {
-        const int g = i / a.dk, d = i - g * a.dk;
-        kc[paged_row(table, pos, a.n_kv_heads, g) * a.dk + d] = from_f<CT>(d < a.dim ? rotated(nq + g * a.dim, d) : 0.f);
-    }
-    for (int i = tid; i < a.n_kv_heads * a.dv; i += 256) {
-        const int g = i / a.dv, d = i - g * a.dv;
-        vc[paged_row(table, pos, a.n_kv_heads, g) * a.dv + d] = from_f<CT>(d < a.vdim ? row[nq + nk + g * a.vdim + d] : 0.f);
+    for (int h = warp; h < a.n_heads + 2 * a.n_kv_heads; h += 8) {          // a warp per head
+        if (h < a.n_heads) {
+            const float* head = sq + h * a.dim;
+            float* q = a.q_out + ((size_t)t * a.n_heads + h) * a.dq;
+            for (int d = lane; d < a.dq; d += 32) q[d] = d < a.dim ? rotated(head, d) : 0.f;
+        } else if (h < a.n_heads + a.n_kv_heads) {
+            const int g = h - a.n_heads;
+            const float* head = sq + nq + g * a.dim;
+            CT* k = (CT*)a.k_cache + paged_row(table, pos, a.n_kv_heads, g) * a.dk;
+            for (int d = lane; d < a.dk; d += 32) k[d] = from_f<CT>(d < a.dim ? rotated(head, d) : 0.f);
+        } else {
+            const int g = h - a.n_heads - a.n_kv_heads;
+            const float* head = row + nq + nk + g * a.vdim;
+            CT* v = (CT*)a.v_cache + paged_row(table, pos, a.n_kv_heads, g) * a.dv;
+            for (int d = lane; d < a.dv; d += 32) v[d] = from_f<CT>(d < a.vdim ? head[d] : 0.f);
+        }
     }
 }
 

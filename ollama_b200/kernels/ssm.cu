@@ -35,49 +35,95 @@ struct SsmConvArgs {
     int ldu;
 };
 
-constexpr int CONV_ROWS = 8;
-
+// Input of the convolution `back` places before row r (zeros before the sequence's start), four channels from c on.
 template <typename T>
-__global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ SsmConvArgs a, int rows) {
+__device__ __forceinline__ void conv_input(const SsmConvArgs& a, int r, int back, int c, float (&v)[4]) {
+    const int off = a.offs[r];
+    if (back <= off) {
+        const T* p = (const T*)a.xz + (size_t)(r - back) * a.ldx + c;
+        if (sizeof(T) == 2) {
+            const uint2 q = *(const uint2*)p;
+            v[0] = __uint_as_float(q.x << 16); v[1] = __uint_as_float(q.x & 0xffff0000u);
+            v[2] = __uint_as_float(q.y << 16); v[3] = __uint_as_float(q.y & 0xffff0000u);
+        } else {
+            *(float4*)v = *(const float4*)p;
+        }
+    } else if (a.positions[r] - back >= 0) {      // before this portion: `back - off` places before its first row
+        *(float4*)v = *(const float4*)(a.state + ((size_t)a.slots[r] * (a.taps - 1) + (a.taps - 1) - (back - off)) * a.inner + c);
+    } else {
+        v[0] = v[1] = v[2] = v[3] = 0.f;
+    }
+}
+
+// A thread carries four channels down PR rows and keeps the last inputs in registers (TAPS > 0), or reads every tap (TAPS = 0: any number).
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ SsmConvArgs a, int rows, int per) {
     const int c = 4 * (blockIdx.x * 128 + threadIdx.x);
     pdl_launch();
-    pdl_wait();
     if (c >= a.inner) return;
-    const T* xz = (const T*)a.xz;
-    const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
     const float4 bias = *(const float4*)(a.b + c);
-    for (int r = r0; r < r1; r++) {
-        const int off = a.offs[r];
-        float acc[4] = {bias.x, bias.y, bias.z, bias.w};
-        for (int j = 0; j < a.taps; j++) {
-            const int back = a.taps - 1 - j;
-            const float4 w = *(const float4*)(a.w + (size_t)j * a.inner + c);
-            float v[4];
-            if (back <= off) {
-                const T* p = xz + (size_t)(r - back) * a.ldx + c;
+    constexpr int W = TAPS > 0 ? TAPS : 1;
+    float w[W][4], win[W][4];
+    if (TAPS > 0) {
 #pragma unroll
-                for (int i = 0; i < 4; i++) v[i] = to_f(p[i]);
-            } else if (a.positions[r] - back >= 0) {      // before this portion: input `back - off` places before its first row
-                const float4 s = *(const float4*)(a.state + ((size_t)a.slots[r] * (a.taps - 1) + (a.taps - 1) - (back - off)) * a.inner + c);
-                v[0] = s.x; v[1] = s.y; v[2] = s.z; v[3] = s.w;
-            } else {
-                continue;
+        for (int j = 0; j < W; j++) *(float4*)w[j] = *(const float4*)(a.w + (size_t)j * a.inner + c);
+    }
+    pdl_wait();
+    const int r0 = blockIdx.y * per, r1 = min(r0 + per, rows);
+    for (int r = r0; r < r1; r++) {
+        float acc[4] = {bias.x, bias.y, bias.z, bias.w};
+        if (TAPS > 0) {
+            if (r == r0 || a.offs[r] == 0) {
+#pragma unroll
+                for (int j = 0; j < W - 1; j++) conv_input<T>(a, r, W - 1 - j, c, win[j]);
             }
-            acc[0] += w.x * v[0]; acc[1] += w.y * v[1]; acc[2] += w.z * v[2]; acc[3] += w.w * v[3];
+            conv_input<T>(a, r, 0, c, win[W - 1]);
+#pragma unroll
+            for (int j = 0; j < W; j++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) acc[i] += w[j][i] * win[j][i];
+#pragma unroll
+            for (int j = 0; j < W - 1; j++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) win[j][i] = win[j + 1][i];
+        } else {
+            for (int j = 0; j < a.taps; j++) {
+                float v[4];
+                conv_input<T>(a, r, a.taps - 1 - j, c, v);
+                const float4 wj = *(const float4*)(a.w + (size_t)j * a.inner + c);
+                acc[0] += wj.x * v[0]; acc[1] += wj.y * v[1]; acc[2] += wj.z * v[2]; acc[3] += wj.w * v[3];
+            }
         }
         T* o = (T*)a.u + (size_t)r * a.ldu + c;
 #pragma unroll
-        for (int i = 0; i < 4; i++) o[i] = from_f<T>(silu_f(acc[i]));
+        for (int i = 0; i < 4; i++) acc[i] = silu_f(acc[i]);
+        if (sizeof(T) == 2) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1]), hi = __floats2bfloat162_rn(acc[2], acc[3]);
+            *(uint2*)o = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            *(float4*)o = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        }
+    }
+}
+
+template <typename T>
+static const void* pick_conv(int taps) {
+    switch (taps) {
+        case 2: return (const void*)ssm_conv_kernel<T, 2>;
+        case 3: return (const void*)ssm_conv_kernel<T, 3>;
+        case 4: return (const void*)ssm_conv_kernel<T, 4>;
+        default: return (const void*)ssm_conv_kernel<T, 0>;
     }
 }
 
 B2_API int b2_ssm_conv(const SsmConvArgs* a, int rows, int f32, int pdl, cudaStream_t st) {
-    if (rows < 1 || a->inner < 8 || (a->inner & 7) || a->taps < 1 || a->ldx < a->inner || a->ldu < a->inner || (rows + CONV_ROWS - 1) / CONV_ROWS > 65535)
+    if (rows < 1 || a->inner < 8 || (a->inner & 7) || a->taps < 1 || a->ldx < a->inner || (a->ldx & 3) || a->ldu < a->inner || (a->ldu & 3) || rows > 65535 * 16)
         return (int)cudaErrorInvalidValue;
     SsmConvArgs c = *a;
-    void* args[] = {&c, &rows};
-    const dim3 grid((a->inner + 511) / 512, (rows + CONV_ROWS - 1) / CONV_ROWS);
-    return launch_rows(f32 ? (const void*)ssm_conv_kernel<float> : (const void*)ssm_conv_kernel<__nv_bfloat16>, grid, dim3(128), 0, args, st, pdl);
+    int per = rows >= 512 ? 16 : rows >= 64 ? 4 : 1;
+    void* args[] = {&c, &rows, &per};
+    const dim3 grid((a->inner + 511) / 512, (rows + per - 1) / per);
+    return launch_rows(f32 ? pick_conv<float>(a->taps) : pick_conv<__nv_bfloat16>(a->taps), grid, dim3(128), 0, args, st, pdl);
 }
 
 struct SsmScanArgs {
@@ -101,13 +147,14 @@ struct SsmScanArgs {
 };
 
 // LPC lanes share a channel and hold SPL state dimensions each.  Time runs in tiles of TT rows whose inputs are fetched into
-// registers while the previous tile is worked on.
+// registers while the previous tile is worked on; eight rows are advanced before their partial sums over the state are reduced, so that
+// the exponentials and loads of a row do not wait for another row's shuffles.
 template <typename T, int LPC, int SPL>
 __global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ SsmScanArgs a) {
-    constexpr int CH = 128 / LPC, NP = LPC * SPL, TT = NP <= 32 ? 32 : 16;
+    constexpr int CH = 128 / LPC, NP = LPC * SPL, TT = NP <= 128 ? 32 : 16, U = 8;
     constexpr int PER = TT * CH / 128, PERN = (TT * NP + 127) / 128;
     __shared__ float2 s_dt[TT][CH];          // (dt, dt * u)
-    __shared__ float s_y[TT][CH];            // in: D u, out: y
+    __shared__ float s_y[TT][CH];
     __shared__ __align__(16) float s_b[TT][NP], s_c[TT][NP];
     const int tid = threadIdx.x, ch = tid / LPC, l = tid % LPC;
     const int c0 = blockIdx.x * CH, c = c0 + ch;
@@ -152,12 +199,12 @@ __global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ S
     };
     fetch(0);
     for (int t0 = 0; t0 < rows; t0 += TT) {
-        float z[PER];
+        float z[PER], du[PER];
 #pragma unroll
-        for (int i = 0; i < PER; i++) {
-            const float dt = softplus_f(rdt[i] + bias);
+        for (int i = 0; i < PER; i++) {          // rows past the end take no step
+            const float dt = t0 + lt + LPC * i < rows ? softplus_f(rdt[i] + bias) : 0.f;
             s_dt[lt + LPC * i][lc] = make_float2(dt, dt * ru[i]);
-            s_y[lt + LPC * i][lc] = dd * ru[i];
+            du[i] = dd * ru[i];
             z[i] = rz[i];
         }
 #pragma unroll
@@ -170,27 +217,46 @@ __global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ S
         }
         __syncthreads();
         if (t0 + TT < rows) fetch(t0 + TT);
-        const int nt = min(TT, rows - t0);
-#pragma unroll 4
-        for (int t = 0; t < nt; t++) {
-            const float2 dv = s_dt[t][ch];
-            float y = 0.f;
+#pragma unroll 1
+        for (int t = 0; t < TT && t0 + t < rows; t += U) {
+            float y[U];
 #pragma unroll
-            for (int i = 0; i < SPL; i++) {
-                S[i] = decayed<sizeof(T) == 4>(S[i], dv.x * A[i]) + dv.y * s_b[t][l * SPL + i];
-                y += S[i] * s_c[t][l * SPL + i];
+            for (int k = 0; k < U; k++) {
+                const float2 dv = s_dt[t + k][ch];
+                y[k] = 0.f;
+#pragma unroll
+                for (int i = 0; i < SPL; i++) {
+                    S[i] = decayed<sizeof(T) == 4>(S[i], dv.x * A[i]) + dv.y * s_b[t + k][l * SPL + i];
+                    y[k] += S[i] * s_c[t + k][l * SPL + i];
+                }
             }
+            // sum over the channel's lanes, halving the rows a lane is responsible for at each exchange
+            int cnt = U, mine = 0;
 #pragma unroll
-            for (int o = LPC / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (l == 0) s_y[t][ch] += y;
+            for (int o = LPC / 2; o > 0; o >>= 1) {
+                if (cnt > 1) {
+                    cnt >>= 1;
+                    const bool up = (l & o) != 0;
+#pragma unroll
+                    for (int k = 0; k < U / 2; k++) {
+                        if (k < cnt) {
+                            const float send = up ? y[k] : y[k + cnt], keep = up ? y[k + cnt] : y[k];
+                            y[k] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
+                    }
+                    if (up) mine += cnt;
+                } else {
+                    y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
+                }
+            }
+            s_y[t + mine][ch] = y[0];
         }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < PER; i++) {
             const int t = t0 + lt + LPC * i;
-            if (lok && t < rows) out[(size_t)(row0 + t) * a.ldo + c0 + lc] = from_f<T>(s_y[lt + LPC * i][lc] * silu_f(z[i]));
+            if (lok && t < rows) out[(size_t)(row0 + t) * a.ldo + c0 + lc] = from_f<T>((s_y[lt + LPC * i][lc] + du[i]) * silu_f(z[i]));
         }
-        __syncthreads();
     }
     if (!live) return;
 #pragma unroll
@@ -209,10 +275,10 @@ __global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ S
 
 template <typename T>
 static const void* pick_scan(int n, int& ch) {
-    if (n <= 16) { ch = 32; return (const void*)ssm_scan_kernel<T, 4, 4>; }
-    if (n <= 32) { ch = 32; return (const void*)ssm_scan_kernel<T, 4, 8>; }
-    if (n <= 64) { ch = 16; return (const void*)ssm_scan_kernel<T, 8, 8>; }
-    if (n <= 128) { ch = 8; return (const void*)ssm_scan_kernel<T, 16, 8>; }
+    if (n <= 16) { ch = 16; return (const void*)ssm_scan_kernel<T, 8, 2>; }
+    if (n <= 32) { ch = 16; return (const void*)ssm_scan_kernel<T, 8, 4>; }
+    if (n <= 64) { ch = 8; return (const void*)ssm_scan_kernel<T, 16, 4>; }
+    if (n <= 128) { ch = 4; return (const void*)ssm_scan_kernel<T, 32, 4>; }
     if (n <= 256) { ch = 8; return (const void*)ssm_scan_kernel<T, 16, 16>; }
     return nullptr;
 }
@@ -250,6 +316,8 @@ struct SsmStepArgs {
     void* out;               // [nb][ldo]
     int ldo, out16;
     int exact;               // a2 holds A: see above
+    const float* u;          // [nb][ldu] convolved and activated inputs, or null: formed here
+    int ldu;
 };
 
 // eight lanes per channel, four channels per warp, 32 channels per CTA; grid (channel blocks, sequences)
@@ -293,10 +361,15 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const __grid_constant__ S
     auto in = [&](int col) -> float { return a.xz16 ? to_f(((const __nv_bfloat16*)a.xz)[xi + col]) : ((const float*)a.xz)[xi + col]; };
     const float x = in(c), z = in(a.off_z + c);
     float* cs = a.conv_state + (size_t)slot * (a.taps - 1) * a.inner + c;
-    float u = a.conv_b[c] + a.conv_w[(size_t)(a.taps - 1) * a.inner + c] * x;
-    if (!fresh)
-        for (int j = 0; j < a.taps - 1; j++) u += cs[(size_t)j * a.inner] * a.conv_w[(size_t)j * a.inner + c];
-    u = silu_f(u);
+    float u;
+    if (a.u) {
+        u = a.u[(size_t)b * a.ldu + c];
+    } else {
+        u = a.conv_b[c] + a.conv_w[(size_t)(a.taps - 1) * a.inner + c] * x;
+        if (!fresh)
+            for (int j = 0; j < a.taps - 1; j++) u += cs[(size_t)j * a.inner] * a.conv_w[(size_t)j * a.inner + c];
+        u = silu_f(u);
+    }
     const float* B = a.p + (size_t)b * a.ldp + a.off_b;
     const float* C = B + a.n_state;
     float* S = a.state + ((size_t)slot * a.inner + c) * a.n_state;

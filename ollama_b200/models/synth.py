@@ -51,6 +51,9 @@ SPECS: dict[str, ArchSpec] = {
                              extra_kv={"rope.scaling.type": "yarn", "rope.scaling.factor": 32.0,
                                        "rope.scaling.original_context_length": 4096,
                                        "rope.scaling.yarn_beta_fast": 32.0, "rope.scaling.yarn_beta_slow": 1.0}),
+    # dense models of the size of the stack models below, layer run by layer run (a gated FFN has three matrices for their two)
+    "dense-1b": ArchSpec("llama", 20, 2048, 16, 4, 128, 5504, 32768, 500000.0),
+    "dense-8b": ArchSpec("llama", 32, 4096, 32, 8, 128, 11008, 128256, 500000.0),
     # small stand-ins of every family for tests
     "tiny-tp": ArchSpec("llama", 2, 1024, 16, 8, 64, 4096, 4096, 500000.0, 1e-5, 4096),      # divides 2, 4 and 8 ways
     "tiny-qwen3": ArchSpec("qwen3", 2, 256, 4, 2, 64, 768, 4096, 1e6, 1e-6, 4096),
@@ -271,3 +274,72 @@ def synthetic_header(spec_name: str, file_type: str | int = "Q4_K_M", with_token
     tensors = {n: TensorInfo(n, tuple(reversed(shape)), tensor_type(n, shape, ft, max(layer, 0), spec.n_layers, spec), 0, 0)
                for n, shape, layer in tensor_table(spec)}
     return GGUFFile("", 3, "<", kv, {}, tensors, 0, 32)
+
+
+# ---------------------------------------------------------------------------------------------------
+# stack models (models/stack.py)
+# ---------------------------------------------------------------------------------------------------
+def stack_config(width: int, heads: int, kv_heads: int, dim: int, ff: int, inner: int, state: int, dt_rank: int, vocab: int, layers: str,
+                 loop: tuple[int, int, int] | None, chunk: int) -> dict:
+    """``config.json`` of a Vazatar model; ``layers``: one letter per layer, A (attention) or M (Mamba)."""
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": chunk}, "scale": dim ** -0.5, "softcap": 50.0,
+                                          "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    mam = {"type": "mamba1", "mixer": {"inner": inner, "state": state, "dt_rank": dt_rank, "conv": 4}}
+    return {"architecture": "Vazatar", "embedding": {"scale": math.sqrt(width)}, "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]} if loop else None,
+            "layers": [{**(att if c == "A" else mam), "mlp": {"kind": "dense", "ff": ff}} for c in layers]}
+
+
+STACK_SPECS: dict[str, dict] = {
+    "tiny-vazatar": stack_config(256, 4, 2, 64, 512, 512, 16, 16, 4096, "AMA", (0, 2, 2), 128),
+    "vazatar-1b": stack_config(2048, 16, 4, 128, 8192, 4096, 16, 128, 32768, "AAMA" * 4, (0, 4, 2), 2048),
+    "vazatar-8b": stack_config(4096, 32, 8, 128, 16384, 8192, 16, 256, 128256, "AAMA" * 7, (0, 4, 2), 8192),
+}
+
+
+class SyntheticStackTensors:
+    """Mapping-like source of random :class:`QWeight` tensors of a stack model, under their GGUF names."""
+
+    def __init__(self, cfg: dict, seed: int = 0, device="cpu"):
+        from ..convert.stack import map_stack_name
+        self.seed, self.device, w = seed, device, cfg["width"]
+        names: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], w), "head": (cfg["vocab"], w), "final.norm": (w,)}
+        if cfg.get("loop"):
+            names["loop.in"] = (w, 2 * w)
+        for i, L in enumerate(cfg["layers"]):
+            m, p = L["mixer"], f"l{i}."
+            names[p + "norm1"] = (w,)
+            if L["type"] == "attention":
+                nq, nk, nv, no = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
+                names.update({p + "mix.q": (nq, w), p + "mix.k": (nk, w), p + "mix.v": (nv, w), p + "mix.q.norm": (nq,), p + "mix.k.norm": (nk,), p + "mix.o": (w, no)})
+            else:
+                c, n, r = m["inner"], m["state"], m["dt_rank"]
+                names.update({p + "mix.in": (2 * c, w), p + "mix.conv": (c, m["conv"]), p + "mix.conv.b": (c,), p + "mix.x": (r + 2 * n, c), p + "mix.dt": (c, r),
+                              p + "mix.dt.b": (c,), p + "mix.A_log": (c, n), p + "mix.D": (c,), p + "mix.o": (w, c)})
+            if L.get("mlp"):
+                names.update({p + "norm2": (w,), p + "mlp.up": (L["mlp"]["ff"], w), p + "mlp.down": (w, L["mlp"]["ff"])})
+        self.table = {map_stack_name(n, cfg): s for n, s in names.items()}
+
+    def __contains__(self, name: str) -> bool:
+        return name in self.table
+
+    def keys(self):
+        return self.table.keys()
+
+    def __getitem__(self, name: str):
+        from .weights import QWeight
+        s = self.table[name]
+        x = random_tensor(name, s, self.seed, self.device)
+        if name.endswith("ssm_a"):
+            x = -(1.0 + torch.arange(s[1], device=x.device, dtype=torch.float32)).expand(s).contiguous()
+        f32 = len(s) < 2 or name.endswith(("ssm_a", "ssm_conv1d.weight"))
+        raw = (x if f32 else x.to(torch.bfloat16)).contiguous().view(-1).view(torch.uint8)
+        return QWeight(name, GGMLType.F32 if f32 else GGMLType.BF16, tuple(s), raw)
+
+
+def stack_model_config(cfg: dict):
+    """:class:`ModelConfig` of a stack configuration, as a file with that metadata would give it."""
+    from ..convert.stack import stack_kv
+    from ..gguf.reader import GGUFFile
+    from .config import config_from_gguf
+    return config_from_gguf(GGUFFile("", 3, "<", stack_kv(cfg, ""), {}, {}, 0, 32))

@@ -10,7 +10,7 @@ from .cuda import AttnDecodeArgs, AttnPrefillArgs, AttnRopeArgs, _check, lib, pt
 
 P, I, F = C.c_void_p, C.c_int, C.c_float
 ACT = {"": 0, "relu2": 1}
-SRC_ROWS, SRC_NORM, SRC_JOINED, SRC_CONV = range(4)
+SRC_ROWS, SRC_NORM, SRC_JOINED = range(3)
 GEMV_MAX_ROWS = 4
 
 
@@ -22,8 +22,8 @@ NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), 
 JoinRowsArgs = _st("JoinRowsArgs", [("a", P), ("b", P), ("lda", I), ("n_a", I), ("ldb", I), ("n_b", I), ("out", P), ("ldo", I), ("off_b", I), ("f32", I)])
 RowSeg = _st("RowSeg", [("w", P), ("g", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
-                                    ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_w", P), ("conv_b", P), ("conv_state", P), ("slots", P),
-                                    ("positions", P), ("taps", I)])
+                                    ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
+                                    ("conv_b", P), ("conv_state", P), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P)])
 PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
                                           ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
                                           ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I)])
@@ -39,7 +39,7 @@ SsmScanArgs = _st("SsmScanArgs", [("xz", P), ("ldx", I), ("off_z", I), ("u", P),
 SsmStepArgs = _st("SsmStepArgs", [("xz", P), ("ldx", I), ("off_z", I), ("xz16", I), ("conv_w", P), ("conv_b", P), ("conv_state", P), ("taps", I),
                                   ("inner", I), ("n_state", I), ("p", P), ("ldp", I), ("off_b", I), ("w_dt", P), ("rank", I), ("w32", I), ("dt", P),
                                   ("lddt", I), ("dt_bias", P), ("a2", P), ("d", P), ("state", P), ("slots", P), ("positions", P), ("out", P), ("ldo", I),
-                                  ("out16", I), ("exact", I)])
+                                  ("out16", I), ("exact", I), ("u", P), ("ldu", I)])
 
 
 def _is32(t: torch.Tensor) -> int:
@@ -71,16 +71,19 @@ def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = Non
 
 
 def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,
-         k1: int = 0, conv=None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None, pdl: bool = False) -> None:
-    """``conv`` = (weights [taps, k], bias [k], state [slots, taps - 1, k])."""
+         k1: int = 0, conv=None, conv_out: torch.Tensor | None = None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None,
+         pdl: bool = False) -> None:
+    """Products of up to four matrices with up to four source rows.  ``conv`` = (weights [taps, n], bias [n], state [slots, taps - 1, n]): the first n
+    results of the first matrix also run through that convolution and SiLU, into ``conv_out``."""
     a = GemvRowsArgs()
     for i, s in enumerate(segs):
         a.seg[i] = s
-    a.nseg, a.nb, a.k, a.src, a.f32, a.x, a.ldx, a.eps, a.kn = len(segs), nb, k, src, int(f32), ptr(x), x.stride(0), eps, kn
+    a.nseg, a.nb, a.k, a.src, a.f32, a.x, a.ldx, a.eps, a.kn, a.conv_seg = len(segs), nb, k, src, int(f32), ptr(x), x.stride(0), eps, kn, -1
     if x2 is not None:
         a.x2, a.ldx2, a.k1 = ptr(x2), x2.stride(0), k1
     if conv is not None:
-        a.conv_w, a.conv_b, a.conv_state, a.taps = ptr(conv[0]), ptr(conv[1]), ptr(conv[2]), conv[0].shape[0]
+        a.conv_seg, a.conv_n, a.taps = 0, conv[0].shape[1], conv[0].shape[0]
+        a.conv_w, a.conv_b, a.conv_state, a.conv_out, a.ldu = ptr(conv[0]), ptr(conv[1]), ptr(conv[2]), ptr(conv_out), conv_out.stride(0)
         a.slots, a.positions = ptr(slots), ptr(positions)
     _call("b2_gemv_rows", a, int(pdl))
 
@@ -150,10 +153,10 @@ def ssm_scan(xz, off_z, u, dt, bc, off_b, dt_bias, a2, d, taps, state, conv_stat
     _call("b2_ssm_scan", a, segs.shape[0], _is32(u), int(pdl))
 
 
-def ssm_step(xz, off_z, conv, p, off_b, w_dt, dt, dt_bias, a2, d, state, slots, positions, out, nb, exact=False, pdl=False) -> None:
+def ssm_step(xz, off_z, conv, p, off_b, w_dt, dt, dt_bias, a2, d, state, slots, positions, out, nb, exact=False, u=None, pdl=False) -> None:
     """One token per sequence.  ``dt``: projected step sizes, or None: projected inside from the first columns of ``p``.
-    ``exact``: ``a2`` holds A instead of log2(e) A (32-bit models)."""
+    ``exact``: ``a2`` holds A instead of log2(e) A (32-bit models).  ``u``: convolved inputs, or None: formed inside."""
     a = SsmStepArgs(ptr(xz), xz.stride(0), off_z, 1 - _is32(xz), ptr(conv[0]), ptr(conv[1]), ptr(conv[2]), conv[0].shape[0], a2.shape[0], a2.shape[1],
                     ptr(p), p.stride(0), off_b, ptr(w_dt), w_dt.shape[1], _is32(w_dt), ptr(dt), dt.stride(0) if dt is not None else 0, ptr(dt_bias), ptr(a2),
-                    ptr(d), ptr(state), ptr(slots), ptr(positions), ptr(out), out.stride(0), 1 - _is32(out), int(exact))
+                    ptr(d), ptr(state), ptr(slots), ptr(positions), ptr(out), out.stride(0), 1 - _is32(out), int(exact), ptr(u), u.stride(0) if u is not None else 0)
     _call("b2_ssm_step", a, nb, int(pdl))

@@ -325,15 +325,23 @@ def test_state_space_portions_and_steps(dtype, inner, n, r, taps):
         close(torch.cat([s.step(1, t, given) for t in range(0, 30)]), want[:30], tol)
 
 
-def test_convolution_inside_the_decode_product():
+@pytest.mark.parametrize("given", [False, True])
+def test_convolution_in_the_decode_product(given):
+    """Rows 12, 2 and 0 of three sequences as outputs of a product (with an identity matrix): its epilogue convolves them with the slots' last
+    inputs, and the step takes the result."""
     from ollama_b200.ops import rows as R
     s = Ssm(56, 10, 5, 4, 20, torch.bfloat16, seed=2)
-    s.expected()
-    w = rnd(26, 56, seed=3).to(torch.bfloat16)
+    want = s.expected()
     s.portions(0, 0, 12)
     s.portions(1, 0, 2)
-    x = torch.stack([s.xz[12], s.xz[2], s.xz[0]]).float().cuda()
-    p = torch.zeros(3, 32, device="cuda")
-    R.gemv([R.seg(w.cuda(), 26, p)], 56, x, 3, False, R.SRC_CONV, conv=(s.conv_w.cuda(), s.conv_b.cuda(), s.conv_state),
-           slots=torch.tensor([0, 1, 2], dtype=torch.int32).cuda(), positions=torch.tensor([12, 2, 0], dtype=torch.int32).cuda())
-    close(p[:, :26], s.u[[12, 2, 0]] @ w.double().t(), 1e-5)
+    at = [12, 2, 0]
+    x = s.xz[at].float().cuda()
+    eye = torch.eye(112, dtype=torch.bfloat16, device="cuda")
+    slots, pos = torch.tensor([0, 1, 2], dtype=torch.int32).cuda(), torch.tensor(at, dtype=torch.int32).cuda()
+    xz, u, out = torch.zeros(3, 112, device="cuda"), torch.full((3, 64), 9.0, device="cuda"), torch.zeros(3, 56, device="cuda")
+    conv = (s.conv_w.cuda(), s.conv_b.cuda(), s.conv_state)
+    R.gemv([R.seg(eye, 112, xz)], 112, x, 3, False, conv=conv, conv_out=u, slots=slots, positions=pos)
+    assert torch.equal(xz, x) and (u[:, 56:] == 9).all()
+    close(u[:, :56], s.u[at], 1e-5)
+    R.ssm_step(xz, 56, conv, s.p[at].cuda(), s.r8, s.wp.cuda(), None, s.bias.cuda(), s.a2, s.d.cuda(), s.state, slots, pos, out, 3, u=u if given else None)
+    close(out, want[at], 1e-2)

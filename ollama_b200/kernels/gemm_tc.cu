@@ -48,6 +48,12 @@ struct GemmParams {
     float glu_alpha, glu_limit;
     int act;                // ungated activation of the result (out_act), before it is stored or accumulated
     int lda;                // row pitch of a, 0: k
+    // split-K (splits > 1): part s of a tile covers its own range of k blocks and stores plain fp32 sums at part + s * part_stride
+    // ([m][part_ld]); a second kernel adds the parts in order and applies the epilogue
+    int splits;
+    float* part;
+    long long part_stride;
+    int part_ld;
 };
 
 template <int BN>
@@ -76,7 +82,7 @@ __device__ __forceinline__ uint32_t pack2_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-template <int BN>
+template <int BN, bool SPLIT>
 __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                                                               const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -92,8 +98,10 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
     __shared__ int s_failed;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int tiles_m = (p.m + BM - 1) / BM, tiles_n = (p.n + BN - 1) / BN, total = tiles_m * tiles_n;
-    const int k_blocks = (p.k + BK - 1) / BK;
+    const int tiles_m = (p.m + BM - 1) / BM, tiles_n = (p.n + BN - 1) / BN, n_tiles = tiles_m * tiles_n;
+    const int splits = SPLIT ? p.splits : 1, total = n_tiles * splits;
+    const int k_all = (p.k + BK - 1) / BK;
+    auto k_first = [&](int t) { return (int)((long long)k_all * (t / n_tiles) / splits); };      // k blocks of work item t: [k_first(t), k_first(t + n_tiles))
 
     if (threadIdx.x == 0) {
         s_failed = 0;
@@ -122,10 +130,11 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
             bool ok = true;
             for (int t = blockIdx.x; t < total && ok; t += gridDim.x) {
                 int mt, nt;
-                tile_coords(t, tiles_m, tiles_n, mt, nt);
+                tile_coords(SPLIT ? t % n_tiles : t, tiles_m, tiles_n, mt, nt);
                 const int e = p.tile_expert ? p.tile_expert[mt] : 0;
                 if (e < 0) continue;               // every role skips the same tiles
-                for (int kb = 0; kb < k_blocks; kb++, it++) {
+                const int kb1 = SPLIT ? k_first(t + n_tiles) : k_all;
+                for (int kb = SPLIT ? k_first(t) : 0; kb < kb1; kb++, it++) {
                     const int s = it % STAGES;
                     if (it >= STAGES && !mbar_wait(&empty[s], ((it / STAGES) - 1) & 1)) { ok = false; break; }
                     uint8_t* a_dst = tiles + s * L::STAGE_BYTES;
@@ -144,7 +153,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
             for (int t = blockIdx.x; t < total && ok; t += gridDim.x) {
                 if (p.tile_expert) {
                     int mt, nt;
-                    tile_coords(t, tiles_m, tiles_n, mt, nt);
+                    tile_coords(SPLIT ? t % n_tiles : t, tiles_m, tiles_n, mt, nt);
                     if (p.tile_expert[mt] < 0) continue;
                 }
                 const int buf = i & 1, use = i >> 1;
@@ -152,7 +161,8 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                 if (use >= 1 && !mbar_wait(&acc_empty[buf], (use - 1) & 1)) { ok = false; break; }
                 tc_fence_after();
                 const uint32_t acc = tmem_base + (uint32_t)(buf * L::ACC_STRIDE);
-                for (int kb = 0; kb < k_blocks; kb++, it++) {
+                const int kb0 = SPLIT ? k_first(t) : 0, kb1 = SPLIT ? k_first(t + n_tiles) : k_all;
+                for (int kb = kb0; kb < kb1; kb++, it++) {
                     const int s = it % STAGES;
                     if (!mbar_wait(&full[s], (it / STAGES) & 1)) { ok = false; break; }
                     tc_fence_after();
@@ -161,7 +171,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
 #pragma unroll
                     for (int k = 0; k < BK / UMMA_K; k++) {
                         // advancing 16 elements along K inside the swizzle span = 32 bytes = 2 descriptor units
-                        umma_bf16(acc, adesc + 2 * k, bdesc + 2 * k, idesc, (kb | k) != 0);
+                        umma_bf16(acc, adesc + 2 * k, bdesc + 2 * k, idesc, kb != kb0 || k != 0);
                     }
                     umma_commit(&empty[s]);        // frees the stage once these MMAs have read it
                 }
@@ -176,7 +186,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
         bool ok = true;
         for (int t = blockIdx.x; t < total && ok; t += gridDim.x) {
             int mt, nt;
-            tile_coords(t, tiles_m, tiles_n, mt, nt);
+            tile_coords(SPLIT ? t % n_tiles : t, tiles_m, tiles_n, mt, nt);
             const int e = p.tile_expert ? p.tile_expert[mt] : 0;
             if (e < 0) continue;
             const int buf = i & 1, use = i >> 1;
@@ -207,6 +217,10 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                     const int row = mt * BM + q * 32 + lr;
                     if (row >= p.m || col >= p.n) continue;
                     float4 r = *(const float4*)(st + lr * L::EPI_LD + cq);
+                    if (SPLIT) {
+                        *(float4*)(p.part + (t / n_tiles) * p.part_stride + (size_t)row * p.part_ld + col) = r;
+                        continue;
+                    }
                     r.x += bias.x; r.y += bias.y; r.z += bias.z; r.w += bias.w;
                     if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
                     if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
@@ -256,15 +270,15 @@ int sm_count() {
     return n;
 }
 
-template <int BN>
+template <int BN, bool SPLIT = false>
 int launch(const void* a, const void* b, const GemmParams& p, cudaStream_t st, int b_rows = 0) {
     CUtensorMap ma, mb;
     if (!make_map(&ma, a, p.m, p.k, BM, p.lda) || !make_map(&mb, b, b_rows ? b_rows : p.n, p.k, BN)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
-    const int total = ((p.m + BM - 1) / BM) * ((p.n + BN - 1) / BN);
+    if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
+    const int total = ((p.m + BM - 1) / BM) * ((p.n + BN - 1) / BN) * (SPLIT ? p.splits : 1);
     const int grid = total < sm_count() ? total : sm_count();
-    gemm_bf16_tc_kernel<BN><<<grid, 192, Cfg<BN>::TOTAL, st>>>(ma, mb, p);
+    gemm_bf16_tc_kernel<BN, SPLIT><<<grid, 192, Cfg<BN>::TOTAL, st>>>(ma, mb, p);
     return (int)cudaGetLastError();
 }
 
@@ -274,12 +288,45 @@ int dispatch(const void* a, const void* b, const GemmParams& p, cudaStream_t st,
     // a handful of rows (a decode step of several sequences): the product streams b once, so the narrowest tile that spreads
     // b over the most SMs wins
     if (p.m <= 32 && (!p.out_bf16 || p.act || p.lda) && !p.glu && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
-        return launch<64>(a, b, p, st, b_rows);
+        return p.splits > 1 ? launch<64, true>(a, b, p, st, b_rows) : launch<64>(a, b, p, st, b_rows);
+    if (p.splits > 1) return p.n >= 128 ? launch<128, true>(a, b, p, st, b_rows) : launch<64, true>(a, b, p, st, b_rows);
     if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256>(a, b, p, st, b_rows);
     // one round either way: the widest tile that still gives every SM at most one tile
     if (p.n >= 192 && tiles_m * ((p.n + 191) / 192) <= sm_count() && tiles_m * ((p.n + 127) / 128) > sm_count()) return launch<192>(a, b, p, st, b_rows);
     if (p.n >= 128) return launch<128>(a, b, p, st, b_rows);
     return launch<64>(a, b, p, st, b_rows);
+}
+
+// Parts of a split product, added in order; activation, accumulation and output type of the whole.
+__global__ void __launch_bounds__(256) gemm_parts_kernel(const __grid_constant__ GemmParams p) {
+    const int row = blockIdx.y, col = 4 * (blockIdx.x * 256 + threadIdx.x);
+    if (col >= p.n) return;
+    float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < p.splits; s++) {
+        const float4 v = *(const float4*)(p.part + s * p.part_stride + (size_t)row * p.part_ld + col);
+        r.x += v.x; r.y += v.y; r.z += v.z; r.w += v.w;
+    }
+    r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act);
+    if (p.out_bf16) {
+        *(uint2*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
+        return;
+    }
+    float* o = (float*)p.out + (size_t)row * p.ldo + col;
+    if (p.accumulate) {
+        const float4 old = *(const float4*)o;
+        r.x += old.x; r.y += old.y; r.z += old.z; r.w += old.w;
+    }
+    *(float4*)o = r;
+}
+
+// How many parts to cut the row length into: a product whose tiles leave most SMs idle, as far as each part keeps some length.
+int split_count(int m, int n, int k) {
+    const int bn = m <= 32 && n >= 64 && (n + 127) / 128 < sm_count() ? 64 : n >= 128 ? 128 : 64;      // dispatch()'s tile at such sizes
+    const long tiles = (long)((m + BM - 1) / BM) * ((n + bn - 1) / bn);
+    if (tiles * 2 > sm_count() || k < 1024) return 1;
+    long s = sm_count() / tiles;
+    if (s > k / 512) s = k / 512;
+    return (int)(s > 16 ? 16 : s);
 }
 
 bool bad_operands(const void* a, const void* b, int m, int n, int k, int ldo) {
@@ -306,11 +353,30 @@ B2_API int b2_gemm_bf16_out16(const void* a, const void* b, int m, int n, int k,
 
 // The same product for operands and results inside wider buffers: a has row pitch lda (k % 8 == 0, lda % 8 == 0), the result goes
 // to rows of pitch ldo as bf16 (n % 4 == 0, out 8-byte aligned) or fp32, after the ungated activation `act` (0 none, 1 square of relu).
-B2_API int b2_gemm_bf16_act(const void* a, int lda, const void* b, int m, int n, int k, void* out, int ldo, int out16, int act, int accumulate, cudaStream_t st) {
-    if (bad_operands(a, b, m, n, k, ldo) || lda < k || (lda & 7) || act < 0 || act > 1 || (out16 && accumulate) || ((uintptr_t)out & (out16 ? 7 : 15)))
+// With scratch (`ws_floats` floats, b2_gemm_bf16_act_scratch) products of few tiles are split along k.
+B2_API int b2_gemm_bf16_act(const void* a, int lda, const void* b, int m, int n, int k, void* out, int ldo, int out16, int act, int accumulate, float* ws,
+                            long long ws_floats, cudaStream_t st) {
+    if (bad_operands(a, b, m, n, k, ldo) || lda < k || (lda & 7) || act < 0 || act > 1 || (out16 && accumulate) || ((uintptr_t)out & (out16 ? 7 : 15)) || ((uintptr_t)ws & 15))
         return (int)cudaErrorInvalidValue;
     GemmParams p{m, n, k, out, ldo, nullptr, accumulate, out16, {}, 0, nullptr, 0, 0.f, 0.f, act, lda};
+    const int splits = ws ? split_count(m, n, k) : 1;
+    if (splits > 1 && (long long)splits * m * n <= ws_floats && m <= 65535) {
+        p.splits = splits;
+        p.part = ws;
+        p.part_ld = n;
+        p.part_stride = (long long)m * n;
+        const int rc = dispatch(a, b, p, st);
+        if (rc) return rc;
+        gemm_parts_kernel<<<dim3((n + 1023) / 1024, m), 256, 0, st>>>(p);
+        return (int)cudaGetLastError();
+    }
     return dispatch(a, b, p, st);
+}
+
+// Floats of scratch with which b2_gemm_bf16_act would split a product of this size (0: it would not).
+B2_API long long b2_gemm_bf16_act_scratch(int m, int n, int k) {
+    const int s = split_count(m, n, k);
+    return s > 1 ? (long long)s * m * n : 0;
 }
 
 // Row-parallel GEMM of a tensor-parallel group: row r of the partial result is stored, as bf16, into cm->dst[r / rows_per_rank]

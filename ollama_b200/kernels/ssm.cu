@@ -35,6 +35,20 @@ struct SsmConvArgs {
     int ldu;
 };
 
+// Gates of the 16-bit form: the exponential, quotient and logarithm of the special-function unit; log(1 + e) of a small e by its series,
+// whose next term is below 2e-7 of the result.
+__device__ __forceinline__ float silu_fast(float v) { return __fdividef(v, 1.f + ex2_f(-1.442695041f * v)); }
+__device__ __forceinline__ float softplus_fast(float v) {
+    const float e = ex2_f(1.442695041f * fminf(v, 20.f));
+    const float small = e * (1.f - e * (0.5f - e * (1.f / 3.f - e * (0.25f - e * 0.2f))));
+    const float r = e < 0.06f ? small : __logf(1.f + e);
+    return v > 20.f ? v : r;
+}
+template <typename T>
+__device__ __forceinline__ float silu_of(float v) { return sizeof(T) == 4 ? silu_f(v) : silu_fast(v); }
+template <typename T>
+__device__ __forceinline__ float softplus_of(float v) { return sizeof(T) == 4 ? softplus_f(v) : softplus_fast(v); }
+
 // Input of the convolution `back` places before row r (zeros before the sequence's start), four channels from c on.
 template <typename T>
 __device__ __forceinline__ void conv_input(const SsmConvArgs& a, int r, int back, int c, float (&v)[4]) {
@@ -70,38 +84,65 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ S
     }
     pdl_wait();
     const int r0 = blockIdx.y * per, r1 = min(r0 + per, rows);
-    for (int r = r0; r < r1; r++) {
-        float acc[4] = {bias.x, bias.y, bias.z, bias.w};
-        if (TAPS > 0) {
-            if (r == r0 || a.offs[r] == 0) {
+    auto finish = [&](int r, float (&acc)[4]) {
+        T* o = (T*)a.u + (size_t)r * a.ldu + c;
 #pragma unroll
-                for (int j = 0; j < W - 1; j++) conv_input<T>(a, r, W - 1 - j, c, win[j]);
-            }
-            conv_input<T>(a, r, 0, c, win[W - 1]);
-#pragma unroll
-            for (int j = 0; j < W; j++)
-#pragma unroll
-                for (int i = 0; i < 4; i++) acc[i] += w[j][i] * win[j][i];
-#pragma unroll
-            for (int j = 0; j < W - 1; j++)
-#pragma unroll
-                for (int i = 0; i < 4; i++) win[j][i] = win[j + 1][i];
+        for (int i = 0; i < 4; i++) acc[i] = silu_of<T>(acc[i]);
+        if (sizeof(T) == 2) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1]), hi = __floats2bfloat162_rn(acc[2], acc[3]);
+            *(uint2*)o = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
         } else {
+            *(float4*)o = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        }
+    };
+    if (TAPS == 0) {
+        for (int r = r0; r < r1; r++) {
+            float acc[4] = {bias.x, bias.y, bias.z, bias.w};
             for (int j = 0; j < a.taps; j++) {
                 float v[4];
                 conv_input<T>(a, r, a.taps - 1 - j, c, v);
                 const float4 wj = *(const float4*)(a.w + (size_t)j * a.inner + c);
                 acc[0] += wj.x * v[0]; acc[1] += wj.y * v[1]; acc[2] += wj.z * v[2]; acc[3] += wj.w * v[3];
             }
+            finish(r, acc);
         }
-        T* o = (T*)a.u + (size_t)r * a.ldu + c;
+        return;
+    }
+    // four rows at a time, their inputs requested together
+    for (int q0 = r0; q0 < r1; q0 += 4) {
+        float in[4][4];
+        int off[4];
 #pragma unroll
-        for (int i = 0; i < 4; i++) acc[i] = silu_f(acc[i]);
-        if (sizeof(T) == 2) {
-            const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1]), hi = __floats2bfloat162_rn(acc[2], acc[3]);
-            *(uint2*)o = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
-        } else {
-            *(float4*)o = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        for (int q = 0; q < 4; q++) {
+            const int r = min(q0 + q, r1 - 1);
+            off[q] = a.offs[r];
+            const T* p = (const T*)a.xz + (size_t)r * a.ldx + c;
+            if (sizeof(T) == 2) {
+                const uint2 v = *(const uint2*)p;
+                in[q][0] = __uint_as_float(v.x << 16); in[q][1] = __uint_as_float(v.x & 0xffff0000u);
+                in[q][2] = __uint_as_float(v.y << 16); in[q][3] = __uint_as_float(v.y & 0xffff0000u);
+            } else {
+                *(float4*)in[q] = *(const float4*)p;
+            }
+        }
+#pragma unroll
+        for (int q = 0; q < 4; q++) {
+            const int r = q0 + q;
+            if (r >= r1) break;
+            if (r == r0 || off[q] == 0) {
+#pragma unroll
+                for (int j = 0; j < W - 1; j++) conv_input<T>(a, r, W - 1 - j, c, win[j]);
+            }
+            float acc[4] = {bias.x, bias.y, bias.z, bias.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                win[W - 1][i] = in[q][i];
+#pragma unroll
+                for (int j = 0; j < W; j++) acc[i] += w[j][i] * win[j][i];
+#pragma unroll
+                for (int j = 0; j < W - 1; j++) win[j][i] = win[j + 1][i];
+            }
+            finish(r, acc);
         }
     }
 }
@@ -120,7 +161,7 @@ B2_API int b2_ssm_conv(const SsmConvArgs* a, int rows, int f32, int pdl, cudaStr
     if (rows < 1 || a->inner < 8 || (a->inner & 7) || a->taps < 1 || a->ldx < a->inner || (a->ldx & 3) || a->ldu < a->inner || (a->ldu & 3) || rows > 65535 * 16)
         return (int)cudaErrorInvalidValue;
     SsmConvArgs c = *a;
-    int per = rows >= 512 ? 16 : rows >= 64 ? 4 : 1;
+    int per = rows >= 1024 ? 16 : rows >= 64 ? 4 : 1;
     void* args[] = {&c, &rows, &per};
     const dim3 grid((a->inner + 511) / 512, (rows + per - 1) / per);
     return launch_rows(f32 ? pick_conv<float>(a->taps) : pick_conv<__nv_bfloat16>(a->taps), grid, dim3(128), 0, args, st, pdl);
@@ -172,37 +213,49 @@ __global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ S
         S[i] = ok && pos0 > 0 ? a.state[((size_t)slot * a.inner + c) * a.n_state + n] : 0.f;
     }
     const T* xz = (const T*)a.xz;
-    const T* u = (const T*)a.u;
-    T* out = (T*)a.out;
     const int lc = tid % CH, lt = tid / CH;      // element (lt + LPC * i, lc) of a tile is this thread's to move
     const bool lok = c0 + lc < a.inner;
-    const float bias = lok ? a.dt_bias[c0 + lc] : 0.f, dd = lok ? a.d[c0 + lc] : 0.f;
+    const int col = lok ? c0 + lc : 0;
+    const float bias = a.dt_bias[col], dd = a.d[col];
+    const T* pu = (const T*)a.u + (size_t)(row0 + lt) * a.ldu + col;
+    const T* pz = xz + (size_t)(row0 + lt) * a.ldx + a.off_z + col;
+    const float* pdt = a.dt + (size_t)(row0 + lt) * a.lddt + col;
+    T* po = (T*)a.out + (size_t)(row0 + lt) * a.ldo + col;
+    const float* pb[PERN];
+    bool bok[PERN];
+#pragma unroll
+    for (int i = 0; i < PERN; i++) {
+        const int e = tid + 128 * i, t = e / NP, n = e % NP;
+        bok[i] = t < TT && n < a.n_state;
+        pb[i] = a.bc + (size_t)(row0 + (bok[i] ? t : 0)) * a.ldbc + a.off_b + (bok[i] ? n : 0);
+    }
     float rdt[PER], ru[PER], rz[PER], rb[PERN], rc[PERN];
-    auto fetch = [&](int t0) {
+    auto fetch = [&](int t0) {                   // rows t0 .. t0 + TT - 1, where the pointers stand; they move on to the next tile
+        const bool full = t0 + TT <= rows;
 #pragma unroll
         for (int i = 0; i < PER; i++) {
-            const int t = t0 + lt + LPC * i;
-            const bool ok = lok && t < rows;
-            const size_t r = (size_t)(row0 + t);
-            rdt[i] = ok ? a.dt[r * a.lddt + c0 + lc] : 0.f;
-            ru[i] = ok ? to_f(u[r * a.ldu + c0 + lc]) : 0.f;
-            rz[i] = ok ? to_f(xz[r * a.ldx + a.off_z + c0 + lc]) : 0.f;
+            const bool ok = full || t0 + lt + LPC * i < rows;
+            rdt[i] = ok ? pdt[i * LPC * a.lddt] : 0.f;
+            ru[i] = ok ? to_f(pu[i * LPC * a.ldu]) : 0.f;
+            rz[i] = ok ? to_f(pz[i * LPC * a.ldx]) : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < PERN; i++) {
-            const int e = tid + 128 * i, t = e / NP, n = e % NP;
-            const bool ok = t < TT && t0 + t < rows && n < a.n_state;
-            const float* p = a.bc + (size_t)(row0 + t0 + t) * a.ldbc + a.off_b + n;
-            rb[i] = ok ? p[0] : 0.f;
-            rc[i] = ok ? p[a.n_state] : 0.f;
+            const bool ok = bok[i] && (full || t0 + (tid + 128 * i) / NP < rows);
+            rb[i] = ok ? pb[i][0] : 0.f;
+            rc[i] = ok ? pb[i][a.n_state] : 0.f;
+            pb[i] += (size_t)TT * a.ldbc;
         }
+        pdt += (size_t)TT * a.lddt;
+        pu += (size_t)TT * a.ldu;
+        pz += (size_t)TT * a.ldx;
     };
     fetch(0);
     for (int t0 = 0; t0 < rows; t0 += TT) {
         float z[PER], du[PER];
 #pragma unroll
         for (int i = 0; i < PER; i++) {          // rows past the end take no step
-            const float dt = t0 + lt + LPC * i < rows ? softplus_f(rdt[i] + bias) : 0.f;
+            const float dt = t0 + lt + LPC * i < rows ? softplus_of<T>(rdt[i] + bias) : 0.f;
             s_dt[lt + LPC * i][lc] = make_float2(dt, dt * ru[i]);
             du[i] = dd * ru[i];
             z[i] = rz[i];
@@ -254,9 +307,9 @@ __global__ void __launch_bounds__(128) ssm_scan_kernel(const __grid_constant__ S
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < PER; i++) {
-            const int t = t0 + lt + LPC * i;
-            if (lok && t < rows) out[(size_t)(row0 + t) * a.ldo + c0 + lc] = from_f<T>((s_y[lt + LPC * i][lc] + du[i]) * silu_f(z[i]));
+            if (lok && t0 + lt + LPC * i < rows) po[i * LPC * a.ldo] = from_f<T>((s_y[lt + LPC * i][lc] + du[i]) * silu_of<T>(z[i]));
         }
+        po += (size_t)TT * a.ldo;
     }
     if (!live) return;
 #pragma unroll
@@ -331,6 +384,22 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const __grid_constant__ S
     pdl_wait();
     const int slot = a.slots[b];
     const bool fresh = a.positions[b] == 0;
+    // the first 32 state dimensions are requested at once, ahead of the step size; more than 32 are worked off behind them
+    constexpr int PRE = 4;
+    const float* B = a.p + (size_t)b * a.ldp + a.off_b;
+    const float* C = B + a.n_state;
+    float* S = a.state + ((size_t)slot * a.inner + c) * a.n_state;
+    const float* A = a.a2 + (size_t)c * a.n_state;
+    float pS[PRE], pA[PRE], pB[PRE], pC[PRE];
+#pragma unroll
+    for (int i = 0; i < PRE; i++) {
+        const int n = l + 8 * i;
+        const bool ok = n < a.n_state;
+        pS[i] = ok && !fresh ? S[n] : 0.f;
+        pA[i] = ok ? A[n] : 0.f;
+        pB[i] = ok ? B[n] : 0.f;
+        pC[i] = ok ? C[n] : 0.f;
+    }
     float dt = 0.f;
     if (a.dt) {
         dt = a.dt[(size_t)b * a.lddt + c];
@@ -370,14 +439,19 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const __grid_constant__ S
             for (int j = 0; j < a.taps - 1; j++) u += cs[(size_t)j * a.inner] * a.conv_w[(size_t)j * a.inner + c];
         u = silu_f(u);
     }
-    const float* B = a.p + (size_t)b * a.ldp + a.off_b;
-    const float* C = B + a.n_state;
-    float* S = a.state + ((size_t)slot * a.inner + c) * a.n_state;
-    const float* A = a.a2 + (size_t)c * a.n_state;
     float y = 0.f;
-    for (int n = l; n < a.n_state; n += 8) {
-        const float old = fresh ? 0.f : S[n];
-        const float s = (a.exact ? decayed<true>(old, dt * A[n]) : decayed<false>(old, dt * A[n])) + dt * u * B[n];
+    auto advance = [&](float old, float An, float Bn) { return (a.exact ? decayed<true>(old, dt * An) : decayed<false>(old, dt * An)) + dt * u * Bn; };
+#pragma unroll
+    for (int i = 0; i < PRE; i++) {
+        const int n = l + 8 * i;
+        if (n < a.n_state) {
+            const float s = advance(pS[i], pA[i], pB[i]);
+            y += s * pC[i];
+            if (live) S[n] = s;
+        }
+    }
+    for (int n = l + 8 * PRE; n < a.n_state; n += 8) {
+        const float s = advance(fresh ? 0.f : S[n], A[n], B[n]);
         y += s * C[n];
         if (live) S[n] = s;
     }

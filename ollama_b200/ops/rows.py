@@ -3,6 +3,7 @@ state-space mixer (kernels/norm_rows.cu, gemv_rows.cu, gemm_f32.cu, attn_paged.c
 from __future__ import annotations
 
 import ctypes as C
+import functools
 
 import torch
 
@@ -99,9 +100,18 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", acc
         f.argtypes = [P, I, P, I, I, I, I, P, I, I, I, P]
         _check(f(ptr(a), a.stride(0), ptr(w), w.stride(0), m, n, k, ptr(out), out.stride(0), ACT[act], int(accumulate), stream()), "gemm_f32")
         return
+    size = _split_floats(m, n, k)
+    ws = torch.empty(size, device=a.device) if size else None
     f = lib().b2_gemm_bf16_act
-    f.argtypes = [P, I, P, I, I, I, P, I, I, I, I, P]
-    _check(f(ptr(a), a.stride(0), ptr(w), m, n, k, ptr(out), out.stride(0), 1 - _is32(out), ACT[act], int(accumulate), stream()), "gemm_bf16_act")
+    f.argtypes = [P, I, P, I, I, I, P, I, I, I, I, P, C.c_longlong, P]
+    _check(f(ptr(a), a.stride(0), ptr(w), m, n, k, ptr(out), out.stride(0), 1 - _is32(out), ACT[act], int(accumulate), ptr(ws), size, stream()), "gemm_bf16_act")
+
+
+@functools.lru_cache(maxsize=4096)
+def _split_floats(m: int, n: int, k: int) -> int:
+    f = lib().b2_gemm_bf16_act_scratch
+    f.restype, f.argtypes = C.c_longlong, [I, I, I]
+    return int(f(m, n, k))
 
 
 def paged_append(qkv, *, heads, kv_heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, positions, slots, table, q_out, k_cache, v_cache, pdl=False) -> None:

@@ -48,7 +48,7 @@ def test_join_rows():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("m,n,k", [(1, 8, 8), (33, 56, 72), (130, 200, 24), (300, 264, 520)])
+@pytest.mark.parametrize("m,n,k", [(1, 8, 8), (33, 56, 72), (130, 200, 24), (300, 264, 520), (16, 96, 4104), (200, 64, 8192)])
 def test_gemm_windows_activation_and_accumulation(dtype, m, n, k):
     from ollama_b200.ops import rows as R
     a, w = rnd(m, k + 16, seed=1).to(dtype), rnd(n, k, seed=2).to(dtype)

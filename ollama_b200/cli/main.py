@@ -606,6 +606,10 @@ def build_parser() -> argparse.ArgumentParser:
     p.add_argument("--format", default="benchstat", choices=["benchstat", "csv", "json"])
     p.set_defaults(fn=cmd_bench)
     sub.add_parser("gpu-discover", help="Print the devices this process can see as JSON").set_defaults(fn=cmd_gpu_discover)
+    p = sub.add_parser("trace", help="Replay a token trace through a model and write logits (no server)")
+    from ..engine.trace import add_arguments, run as run_trace
+    add_arguments(p)
+    p.set_defaults(fn=run_trace)
     p = sub.add_parser("agent", help="Let a model work through tools (shell, files, skills) in this directory")
     p.add_argument("model")
     p.add_argument("prompt", nargs="*", help="one task; without it an interactive session starts")

@@ -12,7 +12,6 @@ import json
 import os
 import sys
 
-PAGE = 64
 SLOTS = 4
 
 
@@ -48,20 +47,28 @@ def replay(backend, lines, out_dir: str, say=print) -> None:
         say(f"done {st['step']}")
 
 
-def main(argv: list[str] | None = None) -> int:
-    ap = argparse.ArgumentParser(prog="trace_run", description="Replay a token trace through a model and write logits.")
+def add_arguments(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--model", required=True, help="checkpoint directory (config.json, model.safetensors) or GGUF file")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16", help="precision of weights, activations and cache")
     ap.add_argument("--out", required=True, help="directory of the logits")
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold together (the size of the page pool)")
-    args = ap.parse_args(argv)
+
+
+def main(argv: list[str] | None = None) -> int:
+    ap = argparse.ArgumentParser(prog="trace_run", description="Replay a token trace through a model and write logits.")
+    add_arguments(ap)
+    return run(ap.parse_args(argv))
+
+
+def run(args: argparse.Namespace) -> int:
     from .backend import make_backend, open_model
+    from .cache import PAGE
     from .runner import RunnerOptions
     with open_model(args.model) as g:
         backend = make_backend(g, "cuda", opts=RunnerOptions(dtype=args.dtype))
     if not hasattr(backend, "step"):
         raise SystemExit(f"{backend.cfg.arch} models have no mixed step to replay a trace with")
-    pool = -(-args.max_tokens // PAGE) * PAGE
+    pool = -(-args.max_tokens // PAGE) * PAGE        # whole pages
     backend.alloc(SLOTS, pool, pool_tokens=pool)
     replay(backend, sys.stdin, args.out, lambda s: print(s, flush=True))
     backend.close()

@@ -246,6 +246,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
 #pragma unroll
     for (int j = 0; j < D / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m_run[2] = {-1e30f, -1e30f}, l_run[2] = {0.f, 0.f};
+    const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
 
     for (int tile = 0; tile < n_tiles; tile++) {
         const int stage = tile % NS;
@@ -287,7 +288,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 float v = s[j][e] * a.scale;
-                if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
+                if (a.softcap > 0.f) v = a.softcap * tanh_exp(v * inv_cap);
                 s[j][e] = v;
                 if (ok[j][e & 1]) mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }

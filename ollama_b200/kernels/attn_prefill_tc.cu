@@ -115,8 +115,6 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
-// tanh through one exponential and one division; absolute error about 2^-22
-__device__ __forceinline__ float tanh_ex2(float x) { return 1.f - __fdividef(2.f, ex2(x * 2.885390081777926815f) + 1.f); }
 __device__ __forceinline__ uint32_t pack_h2(float a, float b) {
     const __half2 h = __floats2half2_rn(a, b);
     return *reinterpret_cast<const uint32_t*>(&h);
@@ -636,7 +634,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
 #pragma unroll
                 for (int i = 0; i < 2; i++)
 #pragma unroll
-                    for (int j = 0; j < 32; j++) v[i][j] = __float_as_uint(cap2 * tanh_ex2(__uint_as_float(v[i][j]) * inv_cap));
+                    for (int j = 0; j < 32; j++) v[i][j] = __float_as_uint(cap2 * tanh_exp(__uint_as_float(v[i][j]) * inv_cap));
             } else {
 #pragma unroll
                 for (int i = 0; i < 2; i++)

@@ -83,6 +83,9 @@ __device__ __forceinline__ float e8m0_to_float(uint32_t e) {
     return e == 0 ? __uint_as_float(0x00400000u) : __uint_as_float(e << 23);
 }
 
+// tanh through one exponential and one quotient of the special-function unit; absolute error about 2^-22 (soft caps of attention scores).
+__device__ __forceinline__ float tanh_exp(float x) { return 1.f - __fdividef(2.f, __expf(2.f * x) + 1.f); }
+
 // Activation of an ungated FFN in a matrix product's epilogue: 0 none, 1 square of relu.
 __device__ __forceinline__ float out_act(float v, int act) {
     if (act == 1) {

@@ -9,8 +9,8 @@
 // The epilogue applies an ungated activation and stores or accumulates (the residual add).  The first rows of one matrix may also run
 // through a causal depthwise convolution + SiLU with the slot's last inputs (the state is only read here: the kernel that advances the
 // recurrence shifts it).  A warp owns four consecutive rows of a matrix and strides over their 16-byte pieces; short problems split the row
-// length over KS warps of the CTA.  CTAs stay resident and walk over groups of rows, asking L2 for the next group's weights while they
-// work; the first group's are requested before the grid-dependency wait (weights do not depend on the producer kernel).
+// length over KS warps of the CTA.  Weight rows are requested from L2 before the grid-dependency wait (they do not depend on the producer
+// kernel).  One group of rows per warp measured faster than resident CTAs that walk over groups (5.5 against 4.7 TB/s on 184 MB).
 #include "rows.cuh"
 
 struct RowSeg {
@@ -69,40 +69,33 @@ __device__ __forceinline__ void source8(const GemvRowsArgs& a, const float* g, i
 }
 
 template <int NB, int SRC, bool F32, int KS>
-__global__ void __launch_bounds__(256, NB <= 2 ? 3 : 2) gemv_rows_kernel(const __grid_constant__ GemvRowsArgs a, int n_groups) {
+__global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_kernel(const __grid_constant__ GemvRowsArgs a) {
     constexpr int RGS = 8 / KS;
     constexpr int EB = F32 ? 4 : 2;
-    constexpr int U = F32 ? 1 : 2;           // pieces in flight per row
+    constexpr int U = F32 || NB == 2 ? 1 : 2;           // pieces in flight per row
     __shared__ float red[8][R * NB];
     __shared__ float s_ss[8][NB];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int rg = warp / KS, ks = warp % KS;
     const uint8_t* wp[R];
-    // group -> matrix, first row; false past the last group
-    auto locate = [&](int g, int& s, int& row0) -> bool {
-        for (s = 0; s < a.nseg; s++) {
-            const int groups = (a.seg[s].n + R - 1) / R;
-            if (g < groups) {
-                row0 = g * R;
-                return true;
-            }
-            g -= groups;
-        }
-        s = 0;
-        row0 = 0;
-        return false;
-    };
-    auto prefetch = [&](int g) {
-        int s, row0;
-        if (!locate(g, s, row0)) return;
-        const RowSeg& w = a.seg[s];
-        const uint8_t* p = (const uint8_t*)w.w + (size_t)row0 * w.ldw * EB;
-        const int nr = min(R, w.n - row0);
-        for (int off = (ks * 32 + lane) * 128; off < a.k * EB; off += KS * 32 * 128)
-            for (int r = 0; r < nr; r++) asm volatile("prefetch.global.L2 [%0];" ::"l"(p + (size_t)r * w.ldw * EB + off));
-    };
+    int g = blockIdx.x * RGS + rg, s = 0;
+    for (; s < a.nseg; s++) {
+        const int groups = (a.seg[s].n + R - 1) / R;
+        if (g < groups) break;
+        g -= groups;
+    }
+    const bool active = s < a.nseg;
+    const RowSeg& w = a.seg[active ? s : 0];
+    const int row0 = active ? g * R : 0;
+#pragma unroll
+    for (int r = 0; r < R; r++) wp[r] = (const uint8_t*)w.w + (size_t)min(row0 + r, w.n - 1) * w.ldw * EB;
     pdl_launch();
-    prefetch(blockIdx.x * RGS + rg);
+    if (active) {
+        for (int off = (ks * 32 + lane) * 128; off < a.k * EB; off += KS * 32 * 128) {
+#pragma unroll
+            for (int r = 0; r < R; r++) asm volatile("prefetch.global.L2 [%0];" ::"l"(wp[r] + off));
+        }
+    }
     pdl_wait();
     if (SRC == SRC_NORM) {
 #pragma unroll
@@ -116,104 +109,92 @@ __global__ void __launch_bounds__(256, NB <= 2 ? 3 : 2) gemv_rows_kernel(const _
             ss = warp_sum(ss);
             if (lane == 0) s_ss[warp][b] = ss;
         }
-        __syncthreads();
     }
-    for (int g0 = blockIdx.x * RGS; g0 < n_groups; g0 += gridDim.x * RGS) {      // the same trips for every warp of the CTA
-        int s, row0;
-        const bool active = locate(g0 + rg, s, row0);
-        const RowSeg& w = a.seg[s];
-        prefetch(g0 + rg + gridDim.x * RGS);
+    float acc[R][NB];
 #pragma unroll
-        for (int r = 0; r < R; r++) wp[r] = (const uint8_t*)w.w + (size_t)min(row0 + r, w.n - 1) * w.ldw * EB;
-        float acc[R][NB];
+    for (int r = 0; r < R; r++)
 #pragma unroll
-        for (int r = 0; r < R; r++)
+        for (int b = 0; b < NB; b++) acc[r][b] = 0.f;
+    if (active) {
+        const int pieces = a.k >> 3, step = KS * 32;
+        for (int p0 = ks * 32 + lane; p0 < pieces; p0 += U * step) {
+            uint4 wv[U][R], wv2[U][R];
 #pragma unroll
-            for (int b = 0; b < NB; b++) acc[r][b] = 0.f;
-        if (active) {
-            const int pieces = a.k >> 3, step = KS * 32;
-            for (int p0 = ks * 32 + lane; p0 < pieces; p0 += U * step) {
-                uint4 wv[U][R], wv2[U][R];
-#pragma unroll
-                for (int u = 0; u < U; u++) {
-                    const int p = p0 + u * step;
-                    if (p < pieces) {
-#pragma unroll
-                        for (int r = 0; r < R; r++) {
-                            wv[u][r] = ldg16(wp[r] + (size_t)p * 8 * EB);
-                            if (F32) wv2[u][r] = ldg16(wp[r] + (size_t)p * 8 * EB + 16);
-                        }
-                    }
-                }
-#pragma unroll
-                for (int u = 0; u < U; u++) {
-                    const int p = p0 + u * step;
-                    if (p >= pieces) continue;
-                    float x[NB][8];
-                    source8<NB, SRC>(a, w.g, 8 * p, x);
+            for (int u = 0; u < U; u++) {
+                const int p = p0 + u * step;
+                if (p < pieces) {
 #pragma unroll
                     for (int r = 0; r < R; r++) {
-                        float wf[8];
-                        const uint32_t q[4] = {wv[u][r].x, wv[u][r].y, wv[u][r].z, wv[u][r].w};
-                        if (F32) {
-                            const uint32_t q2[4] = {wv2[u][r].x, wv2[u][r].y, wv2[u][r].z, wv2[u][r].w};
+                        wv[u][r] = ldg16(wp[r] + (size_t)p * 8 * EB);
+                        if (F32) wv2[u][r] = ldg16(wp[r] + (size_t)p * 8 * EB + 16);
+                    }
+                }
+            }
 #pragma unroll
-                            for (int i = 0; i < 4; i++) {
-                                wf[i] = __uint_as_float(q[i]);
-                                wf[4 + i] = __uint_as_float(q2[i]);
-                            }
-                        } else {
+            for (int u = 0; u < U; u++) {
+                const int p = p0 + u * step;
+                if (p >= pieces) continue;
+                float x[NB][8];
+                source8<NB, SRC>(a, w.g, 8 * p, x);
 #pragma unroll
-                            for (int i = 0; i < 4; i++) {
-                                wf[2 * i] = __uint_as_float(q[i] << 16);
-                                wf[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
-                            }
+                for (int r = 0; r < R; r++) {
+                    float wf[8];
+                    const uint32_t q[4] = {wv[u][r].x, wv[u][r].y, wv[u][r].z, wv[u][r].w};
+                    if (F32) {
+                        const uint32_t q2[4] = {wv2[u][r].x, wv2[u][r].y, wv2[u][r].z, wv2[u][r].w};
+#pragma unroll
+                        for (int i = 0; i < 4; i++) {
+                            wf[i] = __uint_as_float(q[i]);
+                            wf[4 + i] = __uint_as_float(q2[i]);
                         }
+                    } else {
 #pragma unroll
-                        for (int b = 0; b < NB; b++) {
-                            float t = 0.f;
-#pragma unroll
-                            for (int i = 0; i < 8; i++) t = fmaf(wf[i], x[b][i], t);
-                            acc[r][b] += t;
+                        for (int i = 0; i < 4; i++) {
+                            wf[2 * i] = __uint_as_float(q[i] << 16);
+                            wf[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
                         }
+                    }
+#pragma unroll
+                    for (int b = 0; b < NB; b++) {
+                        float t = 0.f;
+#pragma unroll
+                        for (int i = 0; i < 8; i++) t = fmaf(wf[i], x[b][i], t);
+                        acc[r][b] += t;
                     }
                 }
             }
         }
+    }
 #pragma unroll
-        for (int r = 0; r < R; r++)
+    for (int r = 0; r < R; r++)
 #pragma unroll
-            for (int b = 0; b < NB; b++) {
-                acc[r][b] = warp_sum(acc[r][b]);
-                if (lane == 0) red[warp][r * NB + b] = acc[r][b];
-            }
-        if (KS > 1) __syncthreads();
-        else __syncwarp();
-        const int r = lane / NB, b = lane % NB, row = row0 + r;
-        if (ks == 0 && active && lane < R * NB && row < w.n && b < a.nb) {
-            float v = 0.f;
-#pragma unroll
-            for (int k2 = 0; k2 < KS; k2++) v += red[rg * KS + k2][lane];
-            if (SRC == SRC_NORM) {
-                float ss = 0.f;
-#pragma unroll
-                for (int i = 0; i < 8; i++) ss += s_ss[i][b];
-                v *= 1.f / sqrtf(ss / (float)a.kn + a.eps);
-            }
-            v = out_act(v, w.act);
-            float* o = w.out + (size_t)b * w.ldo + row;
-            *o = w.accumulate ? *o + v : v;
-            if (s == a.conv_seg && row < a.conv_n) {
-                float u = a.conv_b[row] + a.conv_w[(size_t)(a.taps - 1) * a.conv_n + row] * v;
-                if (a.positions[b] > 0) {
-                    const float* st = a.conv_state + (size_t)a.slots[b] * (a.taps - 1) * a.conv_n + row;
-                    for (int j = 0; j < a.taps - 1; j++) u += st[(size_t)j * a.conv_n] * a.conv_w[(size_t)j * a.conv_n + row];
-                }
-                a.conv_out[(size_t)b * a.ldu + row] = silu_f(u);
-            }
+        for (int b = 0; b < NB; b++) {
+            acc[r][b] = warp_sum(acc[r][b]);
+            if (lane == 0) red[warp][r * NB + b] = acc[r][b];
         }
-        if (KS > 1) __syncthreads();
-        else __syncwarp();
+    __syncthreads();
+    const int r = lane / NB, b = lane % NB, row = row0 + r;
+    if (ks == 0 && active && lane < R * NB && row < w.n && b < a.nb) {
+        float v = 0.f;
+#pragma unroll
+        for (int k2 = 0; k2 < KS; k2++) v += red[rg * KS + k2][lane];
+        if (SRC == SRC_NORM) {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; i++) ss += s_ss[i][b];
+            v *= 1.f / sqrtf(ss / (float)a.kn + a.eps);
+        }
+        v = out_act(v, w.act);
+        float* o = w.out + (size_t)b * w.ldo + row;
+        *o = w.accumulate ? *o + v : v;
+        if (s == a.conv_seg && row < a.conv_n) {
+            float u = a.conv_b[row] + a.conv_w[(size_t)(a.taps - 1) * a.conv_n + row] * v;
+            if (a.positions[b] > 0) {
+                const float* st = a.conv_state + (size_t)a.slots[b] * (a.taps - 1) * a.conv_n + row;
+                for (int j = 0; j < a.taps - 1; j++) u += st[(size_t)j * a.conv_n] * a.conv_w[(size_t)j * a.conv_n + row];
+            }
+            a.conv_out[(size_t)b * a.ldu + row] = silu_f(u);
+        }
     }
 }
 
@@ -255,25 +236,13 @@ B2_API int b2_gemv_rows(const GemvRowsArgs* a, int pdl, cudaStream_t st) {
         if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (a->src == SRC_NORM && (!w.g || ((uintptr_t)w.g & 15)))) return (int)cudaErrorInvalidValue;
         groups += (w.n + R - 1) / R;
     }
-    // split the row length over KS warps until the machine has several row groups per resident warp, or a lane has two pieces left
+    // split the row length over KS warps until there are several row groups per resident warp, or a lane has two pieces left
+    const long want = a->nb <= 2 ? 16000 : 8000;
     int ks = 1;
-    while (ks < 8 && groups * ks < 8000 && (a->k >> 3) / (32 * ks * 2) >= 1) ks <<= 1;
+    while (ks < 8 && groups * ks < want && (a->k >> 3) / (32 * ks * 2) >= 1) ks <<= 1;
     const int rgs = 8 / ks;
     GemvRowsArgs copy = *a;
-    int n_groups = (int)groups;
-    void* args[] = {&copy, &n_groups};
+    void* args[] = {&copy};
     const void* fn = a->f32 ? pick_src<true>(a->src, a->nb, ks) : pick_src<false>(a->src, a->nb, ks);
-    static int sms = 0;
-    if (!sms) {
-        int dev = 0;
-        cudaGetDevice(&dev);
-        cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-        if (sms <= 0) sms = 148;
-    }
-    int per_sm = 0;
-    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, fn, 256, 0) != cudaSuccess || per_sm < 1) per_sm = 2;
-    const long ctas = (groups + rgs - 1) / rgs, resident = (long)sms * per_sm;
-    // as many CTAs as share the groups evenly over the trips that the resident ones need
-    const long trips = (ctas + resident - 1) / resident;
-    return launch_rows(fn, dim3((unsigned)((ctas + trips - 1) / trips)), dim3(256), 0, args, st, pdl);
+    return launch_rows(fn, dim3((unsigned)((groups + rgs - 1) / rgs)), dim3(256), 0, args, st, pdl);
 }

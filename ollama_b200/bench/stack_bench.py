@@ -30,7 +30,7 @@ def peaks() -> tuple[float, float]:
 
 
 def load(name: str, dev: str):
-    """(backend, matrix weights read by one pass over the layers and the head, cache bytes per position)."""
+    """(backend, matrix weights read by one pass over the layers and the head)."""
     from ..models import synth
     if name in synth.STACK_SPECS:
         from ..engine.stack import StackBackend
@@ -91,7 +91,7 @@ def measure(name: str, steps: int, warmup: int, dev: str = "cuda:0") -> dict:
     return out
 
 
-def run(model: str, steps: int, warmup: int, sampler=None) -> dict:
+def run(model: str, steps: int, warmup: int) -> dict:
     names = list(PAIRS) if model in ("auto", "all") else [model]
     rows = [measure(m, steps, max(warmup, 3)) for name in names for m in (name, PAIRS[name])]
     return {"metric": "stack_models", "unit": "tok/s", "dtype": "bf16", "data": "synthetic", "config": {"prompt": PROMPT, "context": CONTEXT, "batches": list(BATCHES),

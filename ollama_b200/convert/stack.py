@@ -1,7 +1,7 @@
 """Stack checkpoints (config.json with a ``layers`` list + safetensors, see models/stack.py) -> GGUF metadata and tensors.
 
-Names follow the GGUF conventions for the same mechanisms (``blk.N.attn_q.weight``, ``blk.N.ssm_in.weight``, ...).  Norm weights stored around
-zero are written as 1 + w and the decay matrix as A = -exp(A_log), both in fp32, as the other converters do.
+Names follow the GGUF conventions for the same mechanisms (``blk.N.attn_q.weight``, ``blk.N.ssm_in.weight``, ...).  The norm vectors that
+hold an offset from 1 are written as 1 + w and the decay matrix as A = -exp(A_log), both in fp32, as the other converters do.
 """
 from __future__ import annotations
 

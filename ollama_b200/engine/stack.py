@@ -440,7 +440,7 @@ class StackBackend(StepEngine):
     @torch.no_grad()
     def step(self, segs: Sequence[tuple[int, Sequence[int], int]], want: Sequence[Sequence[int]]) -> torch.Tensor | None:
         """One batch: portions of prompts beside single tokens, ``(slot, tokens, position of the first)`` each; ``want``: per portion the
-        places whose logits are asked for.  Returns them in order as [wanted, vocab], or None when there are none."""
+        indices of the rows to return logits for.  Returns [rows, vocab] in that order, or None without any."""
         if all(len(t) == 1 for _, t, _ in segs) and len(segs) <= self.max_batch:
             rows = [i for i, w in enumerate(want) for _ in w]
             lg = self.decode([s for s, _, _ in segs], [max(int(t[0]), 0) for _, t, _ in segs], [p for _, _, p in segs])

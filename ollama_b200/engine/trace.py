@@ -1,9 +1,8 @@
 """Replay of a token trace: given ids go through a model step by step and logits come out; nothing is sampled.
 
 Steps arrive on standard input, one JSON object a line: ``{"step": n, "entries": [{"id", "tokens", "want"}, ...], "end": [ids]}``.  The entries of a
-step are one batch; each brings the next tokens of its request, ``want`` names the places among them whose logits are written to
-``<out>/<step>.f32`` (little-endian fp32, [wanted, vocab]).  Requests named in ``end`` give their slot and pages back.  ``done <step>`` on
-standard output answers each step.
+step run as one batch; each continues its request, and ``want`` indexes the tokens whose logits go to ``<out>/<step>.f32`` (little-endian
+fp32, a row per index).  Requests named in ``end`` give their slot and pages back.  ``done <step>`` on standard output answers each step.
 """
 from __future__ import annotations
 
@@ -51,7 +50,7 @@ def add_arguments(ap: argparse.ArgumentParser) -> None:
     ap.add_argument("--model", required=True, help="checkpoint directory (config.json, model.safetensors) or GGUF file")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16", help="precision of weights, activations and cache")
     ap.add_argument("--out", required=True, help="directory of the logits")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold together (the size of the page pool)")
+    ap.add_argument("--max-tokens", type=int, required=True, help="size of the page pool: tokens of all open requests together")
 
 
 def main(argv: list[str] | None = None) -> int:

@@ -1,7 +1,8 @@
 """Stack checkpoints (config.json with a ``layers`` list + safetensors, see models/stack.py) -> GGUF metadata and tensors.
 
-Names follow the GGUF conventions for the same mechanisms (``blk.N.attn_q.weight``, ``blk.N.ssm_in.weight``, ...).  The norm vectors that
-hold an offset from 1 are written as 1 + w and the decay matrix as A = -exp(A_log), both in fp32, as the other converters do.
+Names follow the GGUF conventions for the same mechanisms (``blk.N.attn_q.weight``, ``blk.N.ssm_in.weight``, ...).  Norm vectors that
+hold an offset from 1 are written as 1 + w and the decay matrix as A = -exp(A_log), both in fp32; the experts of a layer are stacked into one
+tensor per matrix.  All as the other converters do.
 """
 from __future__ import annotations
 
@@ -14,15 +15,22 @@ import torch
 from ..gguf import quants
 from ..gguf.types import GGMLType
 from ..gguf.writer import WriteTensor
-from ..models.stack import STACK_ARCHS, AttentionMixer, parse_stack
+from ..models.stack import DESIGNS, STACK_ARCHS, AttentionMixer, ExpertMLP, LatentMixer, parse_stack
 
-_TOP = {"embed": "token_embd.weight", "head": "output.weight", "final.norm": "output_norm.weight", "loop.in": "loop_in.weight"}
+_TOP = {"embed": "token_embd.weight", "head": "output.weight", "final.norm": "output_norm.weight", "final.norm.b": "output_norm.bias",
+        "loop.in": "loop_in.weight", "loop.step": "loop_step.weight", "side.embed": "per_layer_token_embd.weight"}
 _LAYER = {
     "norm1": "attn_norm.weight", "norm2": "ffn_norm.weight", "mlp.up": "ffn_up.weight", "mlp.down": "ffn_down.weight",
     "mix.q": "attn_q.weight", "mix.k": "attn_k.weight", "mix.v": "attn_v.weight", "mix.q.norm": "attn_q_norm.weight", "mix.k.norm": "attn_k_norm.weight",
     "mix.in": "ssm_in.weight", "mix.conv": "ssm_conv1d.weight", "mix.conv.b": "ssm_conv1d.bias", "mix.x": "ssm_x.weight", "mix.dt": "ssm_dt.weight",
     "mix.dt.b": "ssm_dt.bias", "mix.A_log": "ssm_a", "mix.D": "ssm_d",
+    "norm1.b": "attn_norm.bias", "norm2.b": "ffn_norm.bias", "mlp.gate": "ffn_gate.weight",
+    "mix.dkv": "attn_kv_a_mqa.weight", "mix.dkv.norm": "attn_kv_a_norm.weight", "mix.uk": "attn_k_b.weight", "mix.uv": "attn_v_b.weight",
+    "mlp.router": "ffn_gate_inp.weight", "mlp.router.b": "ffn_gate_inp.bias",
+    "mlp.shared.gate": "ffn_gate_shexp.weight", "mlp.shared.up": "ffn_up_shexp.weight", "mlp.shared.down": "ffn_down_shexp.weight",
+    "side.gate": "inp_gate.weight", "side.proj": "proj.weight", "side.norm": "post_norm.weight",
 }
+_EXPERT = re.compile(r"l(\d+)\.mlp\.e(\d+)\.(gate|up|down)")
 _ONE_PLUS = ("attn_norm.weight", "ffn_norm.weight", "output_norm.weight")
 _F32 = ("ssm_a", "ssm_d", "ssm_conv1d.weight", "ssm_conv1d.bias", "ssm_dt.bias")
 
@@ -39,9 +47,18 @@ def stack_kv(cfg: dict[str, Any], name: str) -> dict[str, Any]:
         f"{arch}.embedding_length": st.width, f"{arch}.vocab_size": st.vocab, f"{arch}.attention.layer_norm_rms_epsilon": st.eps,
         f"{arch}.stack": json.dumps(cfg, sort_keys=True),
     }
-    ffs = [L.mlp.ff for L in st.layers if L.mlp is not None]
+    moe = [L.mlp for L in st.layers if isinstance(L.mlp, ExpertMLP)]
+    ffs = [L.mlp.ff for L in st.layers if L.mlp is not None and not isinstance(L.mlp, ExpertMLP)]
     if ffs:
         kv[f"{arch}.feed_forward_length"] = max(ffs)
+    if moe:
+        kv.update({f"{arch}.expert_count": max(m.experts for m in moe), f"{arch}.expert_used_count": max(m.top for m in moe),
+                   f"{arch}.expert_feed_forward_length": max(m.expert.ff for m in moe)})
+    lat = [L.mixer for L in st.layers if isinstance(L.mixer, LatentMixer)]
+    if lat:
+        kv.update({f"{arch}.attention.head_count": max(a.heads for a in lat), f"{arch}.attention.head_count_kv": 1,
+                   f"{arch}.attention.key_length": max(a.dim + a.rot_dim for a in lat), f"{arch}.attention.value_length": max(a.vdim for a in lat),
+                   f"{arch}.attention.kv_lora_rank": max(a.kv_rank for a in lat), f"{arch}.rope.dimension_count": max(a.rot_dim for a in lat)})
     att = [L.mixer for L in st.layers if isinstance(L.mixer, AttentionMixer)]
     if att:
         kv.update({f"{arch}.attention.head_count": max(a.heads for a in att), f"{arch}.attention.head_count_kv": max(a.kv_heads for a in att),
@@ -52,6 +69,7 @@ def stack_kv(cfg: dict[str, Any], name: str) -> dict[str, Any]:
 
 
 def map_stack_name(name: str, cfg: dict[str, Any]) -> str | None:
+    """GGUF name of a checkpoint tensor; an expert's matrix gets the name of the stack it is part of."""
     if name in _TOP:
         return _TOP[name]
     m = re.fullmatch(r"l(\d+)\.(.+)", name)
@@ -60,20 +78,21 @@ def map_stack_name(name: str, cfg: dict[str, Any]) -> str | None:
     rest = m.group(2)
     if rest == "mix.o":
         return f"blk.{m.group(1)}.{'ssm_out' if cfg['layers'][int(m.group(1))]['type'] == 'mamba1' else 'attn_output'}.weight"
+    e = _EXPERT.fullmatch(name)
+    if e:
+        router = (cfg["layers"][int(e.group(1))].get("mlp") or {}).get("router") or {}
+        return f"blk.{e.group(1)}.ffn_{e.group(3)}_exps.weight" if int(e.group(2)) < int(router.get("experts") or 0) else None
     return f"blk.{m.group(1)}.{_LAYER[rest]}" if rest in _LAYER else None
 
 
 def stack_tensors(src, cfg: dict[str, Any], outtype: str = "auto", progress: Callable[[str], None] | None = None) -> Iterator[WriteTensor]:
     """``src``: name -> tensor mapping with ``keys()`` and ``tensor(name)`` (convert/safetensors.py ModelDir)."""
     want = {"f32": GGMLType.F32, "f16": GGMLType.F16, "bf16": GGMLType.BF16}.get(outtype)
-    for name in src.keys():
-        out = map_stack_name(name, cfg)
-        if out is None:
-            raise ValueError(f"tensor {name} has no counterpart in a {cfg['architecture']} model")
-        if progress:
-            progress(out)
-        t = src.tensor(name)
-        if out.endswith(_ONE_PLUS):
+    one_plus = DESIGNS[cfg["architecture"]].norm == "rms_one_plus"
+    experts: dict[str, dict[int, str]] = {}          # stacked tensor -> the checkpoint tensors it is made of
+
+    def encode(out: str, t: torch.Tensor) -> WriteTensor:
+        if one_plus and out.endswith(_ONE_PLUS):
             t = t.float() + 1.0
         elif out.endswith("ssm_a"):
             t = -torch.exp(t.double()).float()
@@ -85,4 +104,23 @@ def stack_tensors(src, cfg: dict[str, Any], outtype: str = "auto", progress: Cal
             raw = t.contiguous().view(-1).view(torch.uint8)      # the stored bits as they are
         else:
             raw = quants.quantize(t.float(), dt)
-        yield WriteTensor(out, tuple(reversed(t.shape)), dt, raw.cpu().numpy())
+        return WriteTensor(out, tuple(reversed(t.shape)), dt, raw.cpu().numpy())
+
+    for name in src.keys():
+        out = map_stack_name(name, cfg)
+        if out is None:
+            raise ValueError(f"tensor {name} has no counterpart in a {cfg['architecture']} model")
+        e = _EXPERT.fullmatch(name)
+        if e:
+            experts.setdefault(out, {})[int(e.group(2))] = name
+            continue
+        if progress:
+            progress(out)
+        yield encode(out, src.tensor(name))
+    for out, parts in experts.items():
+        n = int(cfg["layers"][int(out.split(".")[1])]["mlp"]["router"]["experts"])
+        if len(parts) != n:
+            raise ValueError(f"{out}: {len(parts)} of {n} experts")
+        if progress:
+            progress(out)
+        yield encode(out, torch.stack([src.tensor(parts[i]) for i in range(n)]))

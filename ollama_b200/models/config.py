@@ -14,7 +14,7 @@ from typing import Any
 
 import numpy as np
 
-from .stack import STACK_ARCHS, AttentionMixer, Stack, parse_stack
+from .stack import STACK_ARCHS, AttentionMixer, ExpertMLP, LatentMixer, Stack, parse_stack
 
 SUPPORTED_ARCHS = ("llama", "mistral", "qwen2", "qwen3", "qwen3moe", "gemma", "gemma2", "gemma3", "gpt-oss", "phi3",
                    "bert", "nomic-bert", *STACK_ARCHS.values())
@@ -211,10 +211,13 @@ def config_from_gguf(g) -> ModelConfig:
         st = c.stack = parse_stack(g.string("stack"))
         c.n_layers, c.d_model, c.vocab_size, c.norm_eps = len(st.layers), st.width, st.vocab, st.eps
         c.embed_scale, c.final_softcap = st.embed_scale, st.logit_softcap
-        c.rope_style, c.act = "neox", "relu2"
+        c.rope_style, c.act = "norm" if st.design.interleaved else "neox", st.design.ff_act
         c.ctx_train = u("context_length", 0)             # 0: no trained length to stay below
-        att = [L.mixer for L in st.layers if isinstance(L.mixer, AttentionMixer)]
-        c.n_heads, c.n_kv_heads = max((m.heads for m in att), default=0), max((m.kv_heads for m in att), default=0)
+        att = [L.mixer for L in st.layers if isinstance(L.mixer, (AttentionMixer, LatentMixer))]
+        c.n_heads = max((m.heads for m in att), default=0)
+        c.n_kv_heads = max((m.kv_heads if isinstance(m, AttentionMixer) else 1 for m in att), default=0)
+        moe = [L.mlp for L in st.layers if isinstance(L.mlp, ExpertMLP)]
+        c.n_experts, c.n_experts_used = max((m.experts for m in moe), default=0), max((m.top for m in moe), default=0)
     elif arch in ("bert", "nomic-bert"):
         c.causal = False
         c.pooling = {0: "none", 1: "mean", 2: "cls", 3: "last"}.get(u("pooling_type", 1), "mean")

@@ -37,7 +37,7 @@ def load(name: str, dev: str):
         cfg = synth.stack_model_config(synth.STACK_SPECS[name])
         be = StackBackend(None, device=dev, cfg=cfg, tensors=synth.SyntheticStackTensors(synth.STACK_SPECS[name], device=dev))
         n = be.head.numel()
-        for r in be.runs:
+        for r in be.runs if be.stack.design.parallel else ():
             L = be.layers[r.layer]
             n += sum(t.numel() for t in (L.w_in, L.up, L.w_out, getattr(L, "w_x", None), getattr(L, "w_dt", None)) if t is not None)
             n += be.loop_in.numel() if r.joins else 0

@@ -1,0 +1,341 @@
+"""Mixers and feed-forwards of stack models that run one after the other inside a layer (engine/stack.py): latent attention, gated and
+mixture-of-experts feed-forwards, inputs of a layer's own per token.
+
+Each class holds a layer's weights, laid out for the kernels, and adds its result to the residual rows of a :class:`Step`.
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass, field
+
+import torch
+
+from ..models.stack import DenseMLP, Expert, ExpertMLP, LatentMixer
+from ..ops import cuda as K
+from ..ops import latent as A
+from ..ops import rows as O
+
+LONG_PORTION = 64                # prompt portions of this many tokens multiply keys and values out; shorter ones stay in the latent space
+MAX_SPLITS = 128
+
+
+def up(n: int, m: int = 8) -> int:
+    return -(-n // m) * m
+
+
+class WeightSource:
+    """Named tensors of a model as zero-padded matrices and vectors on the device."""
+
+    def __init__(self, get, device, act_dtype, width: int):
+        self._get, self.device, self.act_dtype, self.width, self.wp = get, device, act_dtype, width, up(width)
+
+    def tensor(self, name: str, *shape: int) -> torch.Tensor:
+        t = self._get(name)
+        if tuple(t.shape) != tuple(shape):
+            raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
+        return t
+
+    def vec(self, name: str, n: int) -> torch.Tensor:
+        t = torch.zeros(up(n), device=self.device)
+        v = self._get(name).float()
+        if v.numel() != n:
+            raise ValueError(f"{name}: {v.numel()} values, expected {n}")
+        t[:n] = v.reshape(-1)
+        return t
+
+    def zeros(self, *shape: int) -> torch.Tensor:
+        return torch.zeros(*shape, device=self.device, dtype=self.act_dtype)
+
+    def pack(self, parts, n_rows: int, cols: int) -> torch.Tensor:
+        """[n_rows, cols] in the compute type; ``parts``: (row, column, name, shape)."""
+        w = self.zeros(n_rows, cols)
+        for r0, c0, name, shape in parts:
+            w[r0:r0 + shape[0], c0:c0 + shape[1]] = self.tensor(name, *shape)
+        return w
+
+    def gate_up(self, gate: str, up_name: str, ff: int, lead: tuple[int, ...] = ()) -> torch.Tensor:
+        """[..., 2 * padded ff, wp]: rows 2i and 2i + 1 are gate and up of column i."""
+        w = self.zeros(*lead, 2 * up(ff), self.wp)
+        w[..., 0:2 * ff:2, :self.width] = self.tensor(gate, *lead, ff, self.width)
+        w[..., 1:2 * ff:2, :self.width] = self.tensor(up_name, *lead, ff, self.width)
+        return w
+
+
+@dataclass
+class Norm:
+    """Layer norm."""
+    g: torch.Tensor
+    b: torch.Tensor
+
+
+@dataclass
+class Mat:
+    """Matrix of a product; ``rs`` and ``rc`` fold a layer norm before it in (see kernels/gemv_rows.cu)."""
+    w: torch.Tensor
+    n: int                            # rows that hold something
+    bias: torch.Tensor | None = None
+    rs: torch.Tensor | None = None
+    rc: torch.Tensor | None = None
+
+    def fold(self, norm: Norm) -> "Mat":
+        w = self.w.float()
+        self.rs, self.rc = w @ norm.g, w @ norm.b
+        if self.bias is not None:
+            self.rc += self.bias
+        return self
+
+
+def make_norm(src: WeightSource, name: str) -> Norm:
+    return Norm(src.vec(name + ".weight", src.width), src.vec(name + ".bias", src.width))
+
+
+@dataclass
+class LongPortions:
+    """Rows of a step whose keys and values are multiplied out: query tiles, the sequences' places in the scratch buffer, and the other rows."""
+    tiles: torch.Tensor               # [n, 4]: first row, rows, buffer row of the sequence's position 0, position
+    seqs: torch.Tensor                # [n, 4]: first buffer row, positions, slot, -
+    total: int
+    longest: int
+    rest: torch.Tensor | None         # step rows that stay in the latent space
+
+
+class Step:
+    """The rows of one step on their way through the layers.
+
+    A layer may leave an update of the residual ``pending`` (a normalised branch, the vectors that join a pass of a loop); the next norm
+    applies it in its own pass over the rows.
+    """
+
+    def __init__(self, be, B, m, x: torch.Tensor, x0: torch.Tensor | None, decode: bool):
+        self.be, self.B, self.m, self.x, self.x0, self.decode = be, B, m, x, x0, decode
+        self.nb = x.shape[0]
+        self.small = decode and self.nb <= be.gemv_rows
+        self.folded = self.small and not be.f32        # norms inside the products; 32-bit models form them first
+        self.act = torch.float32 if self.small else be.act_dtype
+        self.pdl = be.pdl and decode
+        self.pending: dict = {}
+
+    def buf(self, name: str, cols: int, dtype=None, zero: bool = False) -> torch.Tensor:
+        return self.B.get(name, cols, dtype or self.act, self.nb, zero)
+
+    def launched(self, n: int = 1) -> None:
+        self.be._n += n
+
+    def flush(self) -> None:
+        if self.pending:
+            O.norm_rows(self.x, self.be.stack.width, self.be.stack.eps, None, None, pdl=self.pdl, **self.pending)
+            self.pending = {}
+            self.launched()
+
+    def product(self, h: torch.Tensor, mat: Mat, out: torch.Tensor, **kw) -> None:
+        """out (+)= f(mat h + bias)."""
+        if self.small:
+            O.gemv([O.seg(mat.w, mat.n, out, rc=mat.bias, **kw)], mat.w.shape[1], h, self.nb, self.be.f32, pdl=self.pdl)
+        else:
+            O.gemm(h, mat.w, out, bias=mat.bias, **kw)
+        self.launched()
+
+    def add(self, h: torch.Tensor, mat: Mat) -> None:
+        """x += residual multiplier * mat h."""
+        self.product(h, mat, self.x, accumulate=True, alpha=self.be.stack.residual_mult)
+
+    def normed(self, norm: Norm, mat: Mat, out: torch.Tensor, keep: bool = False, **kw) -> torch.Tensor | None:
+        """out = f(mat norm(x) + bias); returns the normalised rows where they exist (always with ``keep``)."""
+        be, st = self.be, self.be.stack
+        h = self.buf("h", be.wp) if keep or not self.folded else None
+        if self.folded:
+            self.flush()
+            O.gemv([O.seg(mat.w, mat.n, out, norm.g, rs=mat.rs, rc=mat.rc, **kw)], be.wp, self.x, self.nb, False, O.SRC_NORM, st.eps, st.width, layer=True, h=h,
+                   hb=norm.b, pdl=self.pdl)
+            self.launched()
+            return h
+        O.norm_rows(self.x, st.width, st.eps, norm.g, h, b1=norm.b, pdl=self.pdl, **self.pending)
+        self.pending = {}
+        self.launched()
+        self.product(h, mat, out, **kw)
+        return h
+
+
+class LatentAttention:
+    def __init__(self, src: WeightSource, p: str, m: LatentMixer, norm: Norm, f32: bool):
+        H, w = m.heads, src.width
+        self.m, self.norm, self.f32 = m, norm, f32
+        nq = H * (m.dim + m.rot_dim)
+        n_in = nq + m.kv_rank + m.rot_dim
+        self.w_in = Mat(src.pack([(0, 0, p + "attn_q.weight", (nq, w)), (nq, 0, p + "attn_kv_a_mqa.weight", (m.kv_rank + m.rot_dim, w))], up(n_in), src.wp), n_in)
+        self.w_o = Mat(src.pack([(0, 0, p + "attn_output.weight", (w, H * m.vdim))], src.wp, up(H * m.vdim)), w)
+        self.c_norm = src.vec(p + "attn_kv_a_norm.weight", m.kv_rank)
+        self.cp = up(m.kv_rank, 16)
+        self.row = up(self.cp + m.rot_dim, 32)           # values of a cache row
+        # the tensor-core kernel takes latents of up to 512 values in f16; wider ones and 32-bit models keep an fp32 cache
+        self.cache_type = torch.float32 if f32 or self.cp > 512 or self.row > 640 else torch.float16
+        uk, uv = src.tensor(p + "attn_k_b.weight", H * m.dim, m.kv_rank), src.tensor(p + "attn_v_b.weight", H * m.vdim, m.kv_rank)
+        self.uk, self.uv = src.zeros(H, m.dim, self.cp), src.zeros(H * m.vdim, self.cp)
+        self.uk[..., :m.kv_rank] = uk.view(H, m.dim, m.kv_rank)
+        self.uv[:, :m.kv_rank] = uv
+        self.freqs = torch.tensor(m.rot.freqs() if m.rot else [0.0], dtype=torch.float64, device=src.device)
+        self.interleaved = bool(m.rot and m.rot.interleaved)
+        self.dp, self.rp, self.vp = up(m.dim, 64), up(m.rot_dim, 64), up(m.vdim, 64)
+        self.w_kv = None
+        if self.cache_type == torch.float16 and A.parts_supported(self.dp, self.rp, self.vp):
+            self.w_kv = src.zeros(H * (self.dp + self.vp), self.cp)      # rows: every head's keys, then every head's values
+            self.w_kv[:H * self.dp].view(H, self.dp, self.cp)[:, :m.dim] = self.uk
+            self.w_kv[H * self.dp:].view(H, self.vp, self.cp)[:, :m.vdim] = self.uv.view(H, m.vdim, self.cp)
+        if not f32:
+            self.w_in.fold(norm)
+
+    def make_cache(self, cache) -> tuple[torch.Tensor]:
+        return (cache.add_pages(1, self.row, self.cache_type),)
+
+    def run(self, s: Step, mem: tuple[torch.Tensor]) -> None:
+        m, (cache,), lp = self.m, mem, s.m.long
+        qkv = s.buf("in", self.w_in.w.shape[0], torch.float32)
+        s.normed(self.norm, self.w_in, qkv)
+        out = s.buf("mix", self.w_o.w.shape[1], zero=True)
+        if lp is None or self.w_kv is None or s.decode:
+            self._latent(s, qkv, cache, out, s.nb, None, True)
+        else:
+            A.latent_step(qkv, s.nb, cache=cache, **self._step_args(s))
+            s.launched()
+            self._long(s, qkv, cache, out, lp)
+            if lp.rest is not None:
+                self._latent(s, qkv, cache, out, lp.rest.numel(), lp.rest, False)
+        s.add(out, self.w_o)
+
+    def _step_args(self, s: Step) -> dict:
+        m = self.m
+        return dict(heads=m.heads, dim=m.dim, rot=m.rot_dim, rank=m.kv_rank, norm=self.c_norm, eps=s.be.stack.eps, freqs=self.freqs, interleaved=self.interleaved,
+                    positions=s.m.positions, slots=s.m.slots, table=s.be.cache.table, cp=self.cp, pdl=s.pdl)
+
+    def splits(self, n: int, n_ctx: int, sms: int) -> int:
+        """Parts of the keys for ``n`` queries: about two CTAs per SM, none shorter than two pages."""
+        groups = -(-self.m.heads // (16 if self.m.heads <= 16 else 32))
+        return max(1, min(-(-n_ctx // 128), 2 * sms // (groups * n), MAX_SPLITS))
+
+    def _latent(self, s: Step, qkv, cache, out, n: int, rows, append: bool) -> None:
+        """Attention of ``n`` rows in the latent space."""
+        m, dev, table = self.m, qkv.device, s.be.cache.table
+        q = torch.empty(n, m.heads, self.row, device=dev, dtype=cache.dtype)
+        A.latent_step(qkv, n, cache=cache, rows=rows, append=append, uk=self.uk, q_out=q, **self._step_args(s))
+        at = dict(positions=s.m.positions, slots=s.m.slots, table=table, pdl=s.pdl)
+        splits, ml = self.splits(n, s.be.n_ctx, s.be.sms), None
+        if cache.dtype == torch.float16:
+            acc, ml = torch.empty(n, m.heads, splits, self.cp, device=dev), torch.empty(n, m.heads, splits, 2, device=dev)
+            if not A.attn_latent(q, n, cache, acc, ml, heads=m.heads, cp=self.cp, scale=m.scale, splits=splits, rows=rows, **at):
+                raise ValueError(f"latent attention of {m.heads} heads on rows of {self.row}")
+        else:
+            splits, acc = 1, torch.empty(n, m.heads * self.cp, device=dev)
+            O.paged_attn(q, cache, cache, dim=self.row, vdim=self.cp, scale=m.scale, out=acc, **at)
+        A.latent_merge(acc, ml, n, self.uv, out, heads=m.heads, splits=splits, cp=self.cp, vdim=m.vdim, rows=rows, pdl=s.pdl)
+        s.launched(3)
+
+    def _long(self, s: Step, qkv, cache, out, lp: LongPortions) -> None:
+        """Attention of the query tiles of ``lp`` over keys and values multiplied out of the latents."""
+        m, dev, H = self.m, qkv.device, self.m.heads
+        q = torch.empty(s.nb, H, self.dp + self.rp, device=dev, dtype=torch.float16)
+        A.latent_query(qkv, q, heads=H, dim=m.dim, rot=m.rot_dim, freqs=self.freqs, interleaved=self.interleaved, positions=s.m.positions, dp=self.dp, rp=self.rp)
+        c = torch.empty(lp.total, self.cp, device=dev, dtype=torch.bfloat16)
+        r = torch.empty(lp.total, max(self.rp, 8), device=dev, dtype=torch.float16)
+        A.latent_gather(cache, self.cp, m.rot_dim, lp.seqs, lp.longest, s.be.cache.table, c, r)
+        kv = torch.empty(lp.total, self.w_kv.shape[0], device=dev, dtype=torch.float16)
+        O.gemm(c, self.w_kv, kv)
+        A.attn_prefill_parts(q, kv, r, lp.tiles, out, heads=H, dp=self.dp, vp=self.vp, rp=self.rp, vdim=m.vdim, scale=m.scale)
+        s.launched(4)
+
+
+class GatedFFN:
+    def __init__(self, src: WeightSource, p: str, m: DenseMLP, norm: Norm, f32: bool, names=("ffn_gate", "ffn_up", "ffn_down")):
+        gate, up_name, down = (p + n + ".weight" for n in names)
+        self.norm, self.act, self.ffp = norm, "glu:" + m.act, up(m.ff)
+        self.w_gu = Mat(src.gate_up(gate, up_name, m.ff), 2 * m.ff)
+        self.w_down = Mat(src.pack([(0, 0, down, (src.width, m.ff))], src.wp, self.ffp), src.width)
+        if not f32:
+            self.w_gu.fold(norm)
+
+    def run(self, s: Step) -> None:
+        f = s.buf("ff", self.ffp, zero=True)
+        s.normed(self.norm, self.w_gu, f, act=self.act)
+        s.add(f, self.w_down)
+
+
+@dataclass
+class _Shared:
+    e: Expert
+    gu: Mat = field(default=None)
+    down: Mat = field(default=None)
+
+
+class ExpertFFN:
+    """Mixture of experts; the experts stand stacked in one matrix each for gate / up and down."""
+    ACT = "glu:swiglu_oai"
+
+    def __init__(self, src: WeightSource, p: str, m: ExpertMLP, norm: Norm, f32: bool):
+        w, E = src.width, m.experts
+        self.m, self.norm, self.ffp = m, norm, up(m.expert.ff)
+        self.router = Mat(src.pack([(0, 0, p + "ffn_gate_inp.weight", (E, w))], up(E), src.wp), E, bias=src.vec(p + "ffn_gate_inp.bias", E))
+        self.gu = src.gate_up(p + "ffn_gate_exps.weight", p + "ffn_up_exps.weight", m.expert.ff, (E,))
+        self.down = src.zeros(E, src.wp, self.ffp)
+        self.down[:, :w, :m.expert.ff] = src.tensor(p + "ffn_down_exps.weight", E, w, m.expert.ff)
+        self.shared = None
+        if m.shared is not None:
+            ff = m.shared.ff
+            self.shared = _Shared(m.shared, Mat(src.gate_up(p + "ffn_gate_shexp.weight", p + "ffn_up_shexp.weight", ff), 2 * ff),
+                                  Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff)), w))
+        if not f32:
+            self.router.fold(norm)
+
+    def run(self, s: Step) -> None:
+        m, sh = self.m, self.shared
+        z = s.buf("router", self.router.w.shape[0], torch.float32)
+        h = s.normed(self.norm, self.router, z, keep=True)
+        if s.small:
+            sfp = up(sh.e.ff) if sh else 0
+            a = s.buf("experts", m.top * self.ffp + sfp, zero=True)
+            ids, wts = s.buf("ids", m.top, torch.int32), s.buf("weights", m.top)
+            A.moe_up_rows(z, h, s.nb, self.gu, 2 * m.expert.ff, a, ids, wts, experts=m.experts, top=m.top, ffp=self.ffp, limit=m.expert.limit,
+                          ws=sh.gu.w if sh else None, ns=2 * sh.e.ff if sh else 0, limit_s=sh.e.limit if sh else math.inf, pdl=s.pdl)
+            A.moe_down_rows(a, s.nb, ids, wts, self.down, s.x, top=m.top, n=s.be.stack.width, mult=s.be.stack.residual_mult, ws=sh.down.w if sh else None, pdl=s.pdl)
+            s.launched(2)
+            return
+        ids, wts = A.moe_route(z, m.experts, m.top)
+        row, tile_expert, rows = K.moe_plan(ids, m.experts)
+        xs = K.moe_gather(h, row, m.top, rows)
+        f = torch.empty(rows, self.ffp, device=h.device, dtype=s.act)
+        O.gemm(xs, self.gu.view(-1, self.gu.shape[2]), f, act=self.ACT, limit=m.expert.limit, experts=m.experts, tile_expert=tile_expert)
+        y = torch.empty(rows, s.be.wp, device=h.device)
+        O.gemm(f, self.down.view(-1, self.ffp), y, experts=m.experts, tile_expert=tile_expert)
+        K.moe_scatter_combine(y, row, wts, s.nb, m.top, out=s.x, accumulate=True, mult=s.be.stack.residual_mult)
+        s.launched(6)
+        if sh:
+            f = s.buf("shared", up(sh.e.ff), zero=True)
+            s.product(h, sh.gu, f, act=self.ACT, limit=sh.e.limit)
+            s.add(f, sh.down)
+
+
+class SideInput:
+    """g = gelu(gate x) * e[token]; x += multiplier * rmsnorm(proj g) * w, after a layer's feed-forward."""
+
+    def __init__(self, src: WeightSource, p: str, dim: int, table: torch.Tensor):
+        self.dim, self.dimp, self.e = dim, up(dim), table      # table [vocab, dimp]: this layer's part of every token's row
+        self.gate = Mat(src.pack([(0, 0, p + "inp_gate.weight", (dim, src.width))], self.dimp, src.wp), dim)
+        self.proj = Mat(src.pack([(0, 0, p + "proj.weight", (src.width, dim))], src.wp, self.dimp), src.width)
+        self.w = src.vec(p + "post_norm.weight", src.width)
+
+    def run(self, s: Step, join: dict) -> dict:
+        """``join``: vectors that the next layer run adds first; returned where they are still to be added."""
+        st, mult = s.be.stack, s.be.stack.residual_mult
+        if s.small and A.side_rows(s.x, s.nb, st.width, self.gate.w, self.e, self.dim, s.m.tokens, self.proj.w, self.w, st.eps, mult, pdl=s.pdl, **join):
+            s.launched()
+            return {}
+        act = s.be.act_dtype
+        xb = s.x
+        if act != torch.float32:
+            xb = s.buf("side_x", s.be.wp, act)
+            O.join_rows(s.x, s.be.wp, xb, pdl=s.pdl)
+            s.launched()
+        g, y = s.buf("side_g", self.dimp, act), s.buf("side_y", s.be.wp, torch.float32)
+        O.gemm(xb, self.gate.w, g, act="gelu_tanh", mul=self.e, mul_row=s.m.tokens)
+        O.gemm(g, self.proj.w, y)
+        s.launched(2)
+        s.pending = {"y": y, "wy": self.w, "mult": mult}
+        return join

@@ -6,7 +6,8 @@ matrix products; attention reads each sequence's pages, the state-space scan eac
     norm pair -> [q|k|v] product, feed-forward product with the activation in its epilogue -> attention
               -> one product over [attention output | feed-forward hidden] with the residual add in its epilogue
 
-because W_o a + W_down f is one product over joined columns.  Decode steps of up to four sequences fuse the norms into a
+because W_o a + W_down f is one product over joined columns.  Layers whose mixer and feed-forward follow one another (engine/blocks.py) take
+each norm into the product behind it, or into one pass with what is still to be added to the stream.  Decode steps of up to four sequences fuse the norms into a
 multi-matrix GEMV (kernels/gemv_rows.cu), norm + rotation + cache append into the attention kernel, and the convolution and step-size
 projection into the products around the recurrence: four launches per layer plus the merge of the attention splits.  Larger steps and
 prompts multiply on the tcgen05 GEMM.  ``dtype`` "float32" runs weights, activations, cache and products in 32 bits.
@@ -24,11 +25,12 @@ import torch
 from .. import envconfig
 from ..gguf.reader import GGUFFile
 from ..models.config import ModelConfig, config_from_gguf
-from ..models.stack import AttentionMixer, MambaMixer
+from ..models.stack import AttentionMixer, DenseMLP, ExpertMLP, LatentMixer, LayerRun, MambaMixer
 from ..models.weights import QWeight, load_tensor
 from ..ops import cuda as K
 from ..ops import reference as R
 from ..ops import rows as O
+from .blocks import LONG_PORTION, ExpertFFN, GatedFFN, LatentAttention, LongPortions, Mat, Norm, SideInput, Step, WeightSource, make_norm, up
 from .cache import CacheFull, PagedCache
 from .steps import StepEngine
 
@@ -37,8 +39,7 @@ LOGIT_ROWS = 256                 # rows per pass of the output head
 LOG2E = 1.4426950408889634
 
 
-def _up8(n: int) -> int:
-    return -(-n // 8) * 8
+_up8 = up
 
 
 class _Layer:
@@ -62,8 +63,8 @@ class _Rows:
 class _Meta:
     """Device arrays that describe the rows of a step."""
 
-    def __init__(self, tokens, positions, slots, offs=None, segs=None, tiles=None):
-        self.tokens, self.positions, self.slots, self.offs, self.segs, self.tiles = tokens, positions, slots, offs, segs, tiles
+    def __init__(self, tokens, positions, slots, offs=None, segs=None, tiles=None, long: LongPortions | None = None):
+        self.tokens, self.positions, self.slots, self.offs, self.segs, self.tiles, self.long = tokens, positions, slots, offs, segs, tiles, long
 
 
 class StackBackend(StepEngine):
@@ -89,6 +90,7 @@ class StackBackend(StepEngine):
         self.supports_verify = not self.cfg.recurrent
         self.max_batch = MAX_DECODE_ROWS
         self.gemv_rows = O.GEMV_MAX_ROWS      # steps of more sequences multiply on the tensor-core GEMM
+        self.sms = torch.cuda.get_device_properties(self.device).multi_processor_count
         self.runs = self.stack.runs()
         self._load(g, tensors)
 
@@ -100,29 +102,18 @@ class StackBackend(StepEngine):
         def get(name: str) -> torch.Tensor:
             return (tensors[name] if tensors is not None else load_tensor(g, name)).dequant().to(dev)
 
-        def vec(name: str, n: int) -> torch.Tensor:
-            t = torch.zeros(_up8(n), device=dev)
-            v = get(name).float()
-            if v.numel() != n:
-                raise ValueError(f"{name}: {v.numel()} values, expected {n}")
-            t[:n] = v.reshape(-1)
-            return t
-
-        def pack(parts, n_rows: int, cols: int) -> torch.Tensor:
-            """[n_rows, cols] in the compute type; ``parts``: (row, column, name, shape)."""
-            w = torch.zeros(n_rows, cols, device=dev, dtype=self.act_dtype)
-            for r0, c0, name, shape in parts:
-                t = get(name)
-                if tuple(t.shape) != tuple(shape):
-                    raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
-                w[r0:r0 + shape[0], c0:c0 + shape[1]] = t
-            return w
-
+        src = WeightSource(get, dev, self.act_dtype, width)
+        vec, pack = src.vec, src.pack
         wp = self.wp
         self.embd = K.DevWeight(K.WT_F32 if self.f32 else K.WT_BF16, st.vocab, wp, [pack([(0, 0, "token_embd.weight", (st.vocab, width))], st.vocab, wp)])
         self.head = pack([(0, 0, "output.weight", (st.vocab, width))], _up8(st.vocab), wp)
+        self.loop_in = self.loop_step = self.side_table = None
+        self.layers: list[_Layer] = []
+        if not st.design.parallel:
+            self._load_sequential(src)
+            torch.cuda.synchronize(dev)
+            return
         self.out_norm = vec("output_norm.weight", width)
-        self.loop_in = None
         if st.loop is not None:
             w = get("loop_in.weight")
             if tuple(w.shape) != (width, 2 * width):
@@ -130,7 +121,6 @@ class StackBackend(StepEngine):
             self.loop_in = torch.zeros(wp, 2 * wp, device=dev, dtype=self.act_dtype)
             self.loop_in[:width, :width] = w[:, :width]
             self.loop_in[:width, wp:wp + width] = w[:, width:]
-        self.layers: list[_Layer] = []
         for i, sl in enumerate(st.layers):
             L, p, m = _Layer(), f"blk.{i}.", sl.mixer
             L.mixer, L.mlp = m, sl.mlp
@@ -186,9 +176,52 @@ class StackBackend(StepEngine):
             self.layers.append(L)
         torch.cuda.synchronize(dev)
 
+    def _load_sequential(self, src: WeightSource) -> None:
+        """Layers whose mixer and feed-forward follow one another, each behind a layer norm."""
+        st, f32 = self.stack, self.f32
+        self.out_norm = make_norm(src, "output_norm")
+        self.out_mat = Mat(self.head, st.vocab)
+        if not f32:
+            self.out_mat.fold(self.out_norm)
+        if st.loop is not None:
+            self.loop_step = torch.zeros(st.loop[2], src.wp, device=src.device)
+            self.loop_step[:, :st.width] = src.tensor("loop_step.weight", st.loop[2], st.width).float()
+        if st.side_dim:
+            n, d = len(st.layers), st.side_dim
+            self.side_table = src.zeros(st.vocab, n, _up8(d))
+            self.side_table[..., :d] = src.tensor("per_layer_token_embd.weight", st.vocab, n * d).view(st.vocab, n, d)
+        for i, sl in enumerate(st.layers):
+            L, p = _Layer(), f"blk.{i}."
+            if not isinstance(sl.mixer, LatentMixer):
+                raise NotImplementedError(f"{type(sl.mixer).__name__} in a sequential layer")
+            L.mix = LatentAttention(src, p, sl.mixer, make_norm(src, p + "attn_norm"), f32)
+            L.ff = L.side = None
+            if isinstance(sl.mlp, ExpertMLP):
+                L.ff = ExpertFFN(src, p, sl.mlp, make_norm(src, p + "ffn_norm"), f32)
+            elif isinstance(sl.mlp, DenseMLP):
+                L.ff = GatedFFN(src, p, sl.mlp, make_norm(src, p + "ffn_norm"), f32)
+            if st.side_dim:
+                L.side = SideInput(src, p, st.side_dim, self.side_table[:, i])
+            self.layers.append(L)
+
+    def _weights(self):
+        """Every weight tensor on the device, once."""
+        seen: set[int] = set()
+
+        def walk(o):
+            if isinstance(o, torch.Tensor):
+                if o.data_ptr() not in seen:
+                    seen.add(o.data_ptr())
+                    yield o
+            elif isinstance(o, (list, tuple)):
+                for v in o:
+                    yield from walk(v)
+            elif hasattr(o, "__dict__") and type(o).__module__.startswith(__package__):
+                yield from walk(list(vars(o).values()))
+        yield from walk([self.embd.planes[0], self.head, self.loop_in, self.loop_step, self.side_table, self.out_norm, self.layers])
+
     def weight_bytes(self) -> int:
-        ts = [self.embd.planes[0], self.head, self.loop_in] + [t for L in self.layers for t in vars(L).values() if isinstance(t, torch.Tensor)]
-        return sum(t.numel() * t.element_size() for t in ts if t is not None)
+        return sum(t.numel() * t.element_size() for t in self._weights())
 
     def kv_bytes(self) -> int:
         return self.cache.nbytes() if getattr(self, "cache", None) is not None else 0
@@ -203,7 +236,9 @@ class StackBackend(StepEngine):
         self.mem: list[tuple[torch.Tensor, torch.Tensor]] = []        # per layer run: (keys, values) or (state, convolution inputs)
         for r in self.runs:
             L = self.layers[r.layer]
-            if isinstance(L.mixer, AttentionMixer):
+            if not self.stack.design.parallel:
+                self.mem.append(L.mix.make_cache(self.cache))
+            elif isinstance(L.mixer, AttentionMixer):
                 self.mem.append((self.cache.add_pages(L.mixer.kv_heads, L.dk, kv_dt), self.cache.add_pages(L.mixer.kv_heads, L.dv, kv_dt)))
             else:
                 self.mem.append((self.cache.add_state(L.inner, L.mixer.state), self.cache.add_state(max(L.mixer.conv - 1, 1), L.inner)))
@@ -218,7 +253,7 @@ class StackBackend(StepEngine):
         b.sampled = torch.zeros(MB, device=dev, dtype=i32)
         b.host_in, b.host_out = torch.zeros(3, MB, dtype=i32).pin_memory(), torch.zeros(MB, dtype=i32).pin_memory()
         b.host_np, b.host_out_np = b.host_in.numpy(), b.host_out.numpy()
-        att = [L for L in self.layers if isinstance(L.mixer, AttentionMixer) and L.hd]
+        att = [L for L in self.layers if self.stack.design.parallel and isinstance(L.mixer, AttentionMixer) and L.hd]
         for L in att:       # split-K width of decode attention, by the most keys a query of the layer can see
             L.keys = min(n_ctx, L.mixer.chunk or n_ctx)
             L.n_splits = max(1, min(envconfig.attn_splits(), L.keys // envconfig.attn_split_len()))
@@ -355,19 +390,55 @@ class StackBackend(StepEngine):
         K.embed(self.embd, m.tokens[:nb], self.stack.embed_scale, out=x)
         self._n += 1
         x0 = x
-        if self.loop_in is not None:
+        if self.stack.loop is not None:
             x0 = B.get("x0", self.wp, torch.float32, nb, True)
             x0.copy_(x)
+        if not self.stack.design.parallel:
+            return self._run_sequential(Step(self, B, m, x, x0, decode), tap)
         for i in range(len(self.runs)):
             x = self._layer(i, x, x0, B, m, decode)
             if tap is not None:
                 tap(i, x[:, :self.stack.width])
         return x
 
+    def _join(self, run: LayerRun | None, s: Step) -> dict:
+        """What a layer run adds to the stream before it begins: a pass of the loop starts with a vector of its own and, but for the first, with the
+        embedding output."""
+        if run is None or not run.joins:
+            return {}
+        return {"step": self.loop_step[run.turn], **({"x0": s.x0} if run.turn else {})}
+
+    def _run_sequential(self, s: Step, tap=None) -> torch.Tensor:
+        s.pending = self._join(self.runs[0], s)
+        for i, run in enumerate(self.runs):
+            L, nxt = self.layers[run.layer], self.runs[i + 1] if i + 1 < len(self.runs) else None
+            L.mix.run(s, self.mem[i])
+            if L.ff is not None:
+                L.ff.run(s)
+            join = self._join(nxt, s)
+            if tap is not None:                # the stream of this layer run, before anything is added for the next one
+                if L.side is not None:
+                    L.side.run(s, {})
+                s.flush()
+                tap(i, s.x[:, :self.stack.width])
+            elif L.side is not None:
+                join = L.side.run(s, join)
+            s.pending.update(join)
+        s.flush()
+        return s.x
+
     def _head_rows(self, x: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
         """Logits (before the soft cap) of hidden rows ``x`` into the rows of ``out`` [rows, padded vocabulary]."""
         nb, st = x.shape[0], self.stack
-        if nb <= self.gemv_rows:
+        if isinstance(self.out_norm, Norm):
+            if nb <= self.gemv_rows and not self.f32:
+                m = self.out_mat
+                O.gemv([O.seg(m.w, m.n, out, self.out_norm.g, rs=m.rs, rc=m.rc)], self.wp, x, nb, False, O.SRC_NORM, st.eps, st.width, layer=True, pdl=pdl)
+            else:
+                h = torch.empty(nb, self.wp, device=self.device, dtype=self.act_dtype)
+                O.norm_rows(x, st.width, st.eps, self.out_norm.g, h, b1=self.out_norm.b, pdl=pdl)
+                self._mm(h, self.head, out)
+        elif nb <= self.gemv_rows:
             O.gemv([O.seg(self.head, st.vocab, out, self.out_norm)], self.wp, x, nb, self.f32, O.SRC_NORM, st.eps, st.width, pdl=pdl)
         else:
             h = torch.empty(nb, self.wp, device=self.device, dtype=self.act_dtype)
@@ -406,6 +477,8 @@ class StackBackend(StepEngine):
         self._reserve([s for s, _, _ in segs], [p0 + len(t) for _, t, p0 in segs])
         cols: list[list[int]] = [[], [], [], []]
         seg_rows, tiles, at = [], [], 0
+        latent = any(isinstance(L.mixer, LatentMixer) for L in self.stack.layers)
+        long_tiles, seqs, rest, total = [], [], [], 0
         for slot, toks, p0 in segs:
             n = len(toks)
             cols[0] += [max(int(t), 0) for t in toks]
@@ -414,11 +487,21 @@ class StackBackend(StepEngine):
             cols[3] += range(n)
             seg_rows.append((at, n, slot, p0))
             tiles += [(at + r, min(128, n - r), slot, p0 + r) for r in range(0, n, 128)]
+            if latent and n >= LONG_PORTION:
+                long_tiles += [(at + r, min(128, n - r), total, p0 + r) for r in range(0, n, 128)]
+                seqs.append((total, p0 + n, slot, 0))
+                total += p0 + n
+            else:
+                rest += range(at, at + n)
             at += n
         meta = torch.tensor(cols, dtype=torch.int32).to(dev)
-        geom = torch.tensor(seg_rows + tiles, dtype=torch.int32).to(dev)
+        geom = torch.tensor(seg_rows + tiles + long_tiles + seqs, dtype=torch.int32).to(dev)
         self.h2d_bytes += 4 * (meta.numel() + geom.numel())
-        m = _Meta(meta[0], meta[1], meta[2], meta[3], geom[:len(segs)], geom[len(segs):])
+        long, n1, n2 = None, len(segs) + len(tiles), len(segs) + len(tiles) + len(long_tiles)
+        if seqs:
+            long = LongPortions(geom[n1:n2], geom[n2:], total, max(q[1] for q in seqs), torch.tensor(rest, dtype=torch.int32).to(dev) if rest else None)
+            self.h2d_bytes += 4 * len(rest)
+        m = _Meta(meta[0], meta[1], meta[2], meta[3], geom[:len(segs)], geom[len(segs):n1], long)
         self._n = 0
         out = self._run_rows(_Rows(at, dev), m, at, decode=False, tap=tap)
         self.kernel_launches += self._n
@@ -426,6 +509,8 @@ class StackBackend(StepEngine):
 
     def _final_norm(self, x: torch.Tensor) -> torch.Tensor:
         w = self.stack.width
+        if isinstance(self.out_norm, Norm):
+            return torch.nn.functional.layer_norm(x[:, :w], (w,), self.out_norm.g[:w], self.out_norm.b[:w], self.stack.eps)
         return R.rmsnorm(x[:, :w], self.out_norm[:w], self.stack.eps)
 
     def _logits(self, x: torch.Tensor) -> torch.Tensor:

@@ -94,14 +94,14 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
 // softmax statistics are merged across the CTA, then the threads own value columns.  The kernel of 32-bit models, and of
 // head sizes the tensor-core kernels do not take.
 // ---------------------------------------------------------------------------------------------------------------------
-constexpr int VCOLS = 4;      // value columns per thread: value heads up to 512
+constexpr int VCOLS = 4;      // value columns per thread; wider values take a CTA per 512
 
 template <typename CT, typename OT>
 __global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__ PagedAttnArgs a) {
     extern __shared__ float sq[];      // [dim]
     __shared__ float sp[128];
     __shared__ float red[2][4];
-    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, v0 = blockIdx.z * 128 * VCOLS;
     pdl_launch();
     pdl_wait();
     const int pos = a.positions[t], slot = a.slots[t], g = h / (a.n_heads / a.n_kv_heads);
@@ -142,7 +142,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__
             const float w = sp[i];
 #pragma unroll
             for (int j = 0; j < VCOLS; j++) {
-                const int d = tid + 128 * j;
+                const int d = v0 + tid + 128 * j;
                 if (d < a.vdim) acc[j] = fmaf(w, to_f(vr[d]), acc[j]);
             }
         }
@@ -151,7 +151,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__
     OT* o = (OT*)a.out + (size_t)t * a.ldo + h * a.vdim;
 #pragma unroll
     for (int j = 0; j < VCOLS; j++) {
-        const int d = tid + 128 * j;
+        const int d = v0 + tid + 128 * j;
         if (d < a.vdim) o[d] = from_f<OT>(acc[j] / l);
     }
 }
@@ -209,12 +209,11 @@ B2_API int b2_paged_append(const PagedAppendArgs* a, int rows, int pdl, cudaStre
 
 B2_API int b2_paged_attn(const PagedAttnArgs* a, int rows, int pdl, cudaStream_t st) {
     if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dim > 8192 || a->n_heads > 65535) return (int)cudaErrorInvalidValue;
-    if (a->vdim > 128 * VCOLS) return (int)cudaErrorNotSupported;
     PagedAttnArgs c = *a;
     void* args[] = {&c};
     const void* fn = a->cache32 ? (a->out16 ? (const void*)paged_attn_kernel<float, __nv_bfloat16> : (const void*)paged_attn_kernel<float, float>)
                                 : (a->out16 ? (const void*)paged_attn_kernel<__half, __nv_bfloat16> : (const void*)paged_attn_kernel<__half, float>);
-    return launch_rows(fn, dim3(rows, a->n_heads), dim3(128), (size_t)a->dim * 4, args, st, pdl);
+    return launch_rows(fn, dim3(rows, a->n_heads, (a->vdim + 128 * VCOLS - 1) / (128 * VCOLS)), dim3(128), (size_t)a->dim * 4, args, st, pdl);
 }
 
 // Decode step over a paged f16 cache: norm and rotation of the new query and key, cache append and split-K attention in one launch,

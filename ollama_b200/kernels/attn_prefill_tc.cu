@@ -45,6 +45,19 @@ struct AttnPagedArgs {
     int max_pages, chunk, vdim, ldo;
 };
 
+// Form for keys in two parts (latent attention, latent.cu): rows of one buffer hold every head's own key part and value, rows of another the
+// key part that all heads share; the buffers hold the visible positions of the step's sequences one after the other.
+struct AttnPartsArgs {
+    const __half* q;         // [rows][H][D's own part | shared part], each padded to a multiple of 64
+    const __half* kv;        // [n_rows][H * dp | H * vp]: own key parts, then values
+    const __half* shared;    // [n_rows][rp], or null with rp = 0
+    int n_rows, dp, vp, rp;
+    const int4* tiles;       // [tiles] (first query row, rows <= 128, buffer row of the sequence's position 0, position of the first row)
+    int H, vdim, ldo;
+    float scale;
+    __nv_bfloat16* out;      // [rows][ldo], head h at column h * vdim
+};
+
 __device__ int g_attn_tc_status = 0;
 
 namespace {
@@ -449,21 +462,25 @@ bool cached_kv_map(CUtensorMap* out, const void* base, size_t rows, int d, int b
 constexpr int THREADS2 = (SOFTMAX_WARPS + 3) * 32;
 constexpr int TMEM_COLS2 = 512;
 
-template <int D>
+enum CacheForm : int { FLAT = 0, PAGED_CACHE = 1, PARTS = 2 };
+
+template <int D, int DK>
 struct Lay2 {
-    static constexpr int ATOMS = D / 64;
-    static constexpr int Q_BYTES = ATOMS * ATOM_BYTES;
-    static constexpr int KV_BYTES = ATOMS * ATOM_BYTES;
-    static constexpr int OFF_K = Q_BYTES, OFF_V = OFF_K + 2 * KV_BYTES, OFF_BAR = OFF_V + 2 * KV_BYTES;
+    static constexpr int K_ATOMS = DK / 64, V_ATOMS = D / 64;
+    static constexpr int Q_BYTES = K_ATOMS * ATOM_BYTES;
+    static constexpr int K_BYTES = K_ATOMS * ATOM_BYTES, V_BYTES = V_ATOMS * ATOM_BYTES;
+    static constexpr int OFF_K = Q_BYTES, OFF_V = OFF_K + 2 * K_BYTES, OFF_BAR = OFF_V + 2 * V_BYTES;
     static constexpr int TOTAL = OFF_BAR + 256 + 2 * 2 * 128 * 4 + 1024;
 };
 
-template <int D, bool PAGED>
+// D: value columns, DK: query / key columns (D unless the form is PARTS)
+template <int D, int DK, int FORM>
 __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
-                                                                       const __grid_constant__ AttnPrefillArgs a, const __grid_constant__ AttnPagedArgs pg) {
-    using L = Lay2<D>;
-    constexpr int ATOMS = L::ATOMS;
-    constexpr int OH = D / 2;
+                                                                       const __grid_constant__ AttnPrefillArgs a, const __grid_constant__ AttnPagedArgs pg,
+                                                                       const __grid_constant__ AttnPartsArgs pt) {
+    using L = Lay2<D, DK>;
+    constexpr bool PAGED = FORM != FLAT;       // query tiles come as a list, output rows have a pitch of their own
+    constexpr int OH = D / 2, QH = DK / 2;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* sm = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     uint8_t* sQ = sm;
@@ -483,12 +500,12 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int mt = gridDim.x - 1 - blockIdx.x;
-    const int4 tile = PAGED ? pg.tiles[mt] : make_int4(mt * BQ, min(BQ, a.T - mt * BQ), a.slot, a.pos0 + mt * BQ);
-    const int m0 = tile.x, rows = tile.y, h = blockIdx.y, hkv = h / (a.H / a.Hkv);
+    const int4 tile = FORM == PARTS ? pt.tiles[mt] : PAGED ? pg.tiles[mt] : make_int4(mt * BQ, min(BQ, a.T - mt * BQ), a.slot, a.pos0 + mt * BQ);
+    const int m0 = tile.x, rows = tile.y, h = blockIdx.y, hkv = FORM == PARTS ? h : h / (a.H / a.Hkv);
     const int q_lo = tile.w, q_hi = q_lo + rows - 1;
     const int kv_len = PAGED ? q_hi + 1 : a.kv_len;
     const int k_end = a.causal ? min(kv_len, q_hi + 1) : kv_len;
-    const int chunk = PAGED ? pg.chunk : 0;
+    const int chunk = FORM == PAGED_CACHE ? pg.chunk : 0;
     const int k_begin = (chunk > 0 ? q_lo - q_lo % chunk : a.window > 0 ? max(0, q_lo - a.window + 1) : 0) & ~(BKV - 1);
     const int n_tiles = k_end > k_begin ? (k_end - k_begin + BKV - 1) / BKV : 0;
 
@@ -513,6 +530,14 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     if (warp < SOFTMAX_WARPS) {
         const int r = 32 * (warp & 3) + lane, c = warp >> 2;
         const bool live = r < rows;
+        if (FORM == PARTS) {
+            const __half* qp = pt.q + ((size_t)(m0 + r) * a.H + h) * DK + QH * c;
+#pragma unroll
+            for (int j = 0; j < QH / 8; j++) {
+                const int col = QH * c + 8 * j, atom = col >> 6, chunk = (col & 63) >> 3;
+                *(uint4*)(sQ + atom * ATOM_BYTES + r * 128 + ((chunk ^ (r & 7)) << 4)) = live ? *(const uint4*)(qp + 8 * j) : make_uint4(0, 0, 0, 0);
+            }
+        } else {
         const float* qp = a.q + ((size_t)(m0 + r) * a.H + h) * D + OH * c;
 #pragma unroll
         for (int j = 0; j < OH / 8; j++) {
@@ -526,14 +551,15 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             *(uint4*)(sQ + atom * ATOM_BYTES + r * 128 + ((chunk ^ (r & 7)) << 4)) =
                 make_uint4(pack_h2(v0.x, v0.y), pack_h2(v0.z, v0.w), pack_h2(v1.x, v1.y), pack_h2(v1.z, v1.w));
         }
+        }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
-    const int row0 = PAGED ? 0 : (a.slot * a.Hkv + hkv) * a.n_ctx + k_begin;
-    const int* table = PAGED ? pg.page_table + (size_t)tile.z * pg.max_pages : nullptr;
+    const int row0 = FORM == PARTS ? tile.z + k_begin : PAGED ? 0 : (a.slot * a.Hkv + hkv) * a.n_ctx + k_begin;
+    const int* table = FORM == PAGED_CACHE ? pg.page_table + (size_t)tile.z * pg.max_pages : nullptr;
 
     if (warp == 8 || warp == 10) {
         if (lane == 0) {                 // one thread streams the K tiles, another the V tiles: each waits only for its own buffers
@@ -545,11 +571,18 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             for (int t = 0; t < n_tiles; t++) {
                 const int b = t & 1;
                 if (t >= 2 && !mbar_wait(&empty[b], ((t >> 1) - 1) & 1)) { atomicExch(failed, 1); break; }
-                mbar_expect_tx(&full[b], L::KV_BYTES);
+                const int atoms = is_k ? L::K_ATOMS : L::V_ATOMS;
+                mbar_expect_tx(&full[b], atoms * ATOM_BYTES);
 #pragma unroll
-                for (int at = 0; at < ATOMS; at++) {
-                    uint8_t* dst = base + b * L::KV_BYTES + at * ATOM_BYTES;
-                    if (PAGED) {          // a tile may reach past the sequence's last page: any page will do there, its keys are masked
+                for (int at = 0; at < L::K_ATOMS; at++) {
+                    if (at >= atoms) break;
+                    uint8_t* dst = base + (b * atoms + at) * ATOM_BYTES;
+                    if (FORM == PARTS) {  // rows behind the sequence belong to the next one or read as zero; their keys are masked
+                        const int own = pt.dp >> 6, y = row0 + t * BKV;
+                        if (!is_k) tma_load_2d(dst, &map_k, a.H * pt.dp + h * pt.vp + 64 * at, y, &full[b]);
+                        else if (at < own) tma_load_2d(dst, &map_k, h * pt.dp + 64 * at, y, &full[b]);
+                        else tma_load_2d(dst, &map_v, 64 * (at - own), y, &full[b]);
+                    } else if (PAGED) {   // a tile may reach past the sequence's last page: any page will do there, its keys are masked
                         const int p0 = (k_begin + t * BKV) >> 6, last = (kv_len - 1) >> 6;
                         tma_load_2d(dst, map, 64 * at, (table[min(p0, last)] * a.Hkv + hkv) * 64, &full[b]);
                         tma_load_2d(dst + ATOM_BYTES / 2, map, 64 * at, (table[min(p0 + 1, last)] * a.Hkv + hkv) * 64, &full[b]);
@@ -567,9 +600,9 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                 const int b = t & 1;
                 if (!mbar_wait(&k_full[b], (t >> 1) & 1)) { ok = false; return; }
                 tc_fence_after();
-                const uint8_t* kt = sm + L::OFF_K + b * L::KV_BYTES;
+                const uint8_t* kt = sm + L::OFF_K + b * L::K_BYTES;
 #pragma unroll
-                for (int at = 0; at < ATOMS; at++) {
+                for (int at = 0; at < L::K_ATOMS; at++) {
                     const uint64_t qd = umma_desc(sQ + at * ATOM_BYTES), kd = umma_desc(kt + at * ATOM_BYTES);
 #pragma unroll
                     for (int k = 0; k < 4; k++) umma_f16(tmem + 128 * b, qd + 2 * k, kd + 2 * k, id_s, (at | k) != 0);
@@ -583,7 +616,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                 const int b = t & 1, ph = (t >> 1) & 1;
                 if (!mbar_wait(&p_ready[b], ph) || !mbar_wait(&v_full[b], ph)) { ok = false; break; }
                 tc_fence_after();
-                const uint8_t* vt = sm + L::OFF_V + b * L::KV_BYTES;
+                const uint8_t* vt = sm + L::OFF_V + b * L::V_BYTES;
 #pragma unroll
                 for (int kk = 0; kk < BKV / 16; kk++)      // O_tile(t) = P(t) V(t); P sits in the first 64 columns of its score buffer
                     umma_f16_ts(tmem + 256 + 128 * b, tmem + 128 * b + 8 * kk, umma_desc_mn(vt + kk * 16 * 128, ATOM_BYTES), id_o, kk != 0);
@@ -643,7 +676,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             }
             if (masked) {
                 const int kp0 = n0 + 64 * c;
-                const int hi = min(a.causal ? qp : kv_len - 1, kv_len - 1), lo = PAGED ? chunk_lo : a.window > 0 ? qp - a.window + 1 : 0;
+                const int hi = min(a.causal ? qp : kv_len - 1, kv_len - 1), lo = FORM == PAGED_CACHE ? chunk_lo : a.window > 0 ? qp - a.window + 1 : 0;
 #pragma unroll
                 for (int i = 0; i < 2; i++)
 #pragma unroll
@@ -703,11 +736,12 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             }
             const float inv = l > 0.f ? oc / l : 0.f;
             if (PAGED && r < rows) {
-                __nv_bfloat16* op = a.out + (size_t)(m0 + r) * pg.ldo + (size_t)h * pg.vdim + OH * c;
-                const bool whole = (pg.vdim & 7) == 0 && (pg.ldo & 7) == 0;
+                const int vdim = FORM == PARTS ? pt.vdim : pg.vdim, ldo = FORM == PARTS ? pt.ldo : pg.ldo;
+                __nv_bfloat16* op = a.out + (size_t)(m0 + r) * ldo + (size_t)h * vdim + OH * c;
+                const bool whole = (vdim & 7) == 0 && (ldo & 7) == 0;
 #pragma unroll
                 for (int j = 0; j < OH; j += 8) {
-                    if (OH * c + j >= pg.vdim) continue;
+                    if (OH * c + j >= vdim) continue;
                     if (whole) {
                         uint32_t w[4];
 #pragma unroll
@@ -719,7 +753,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                     } else {
 #pragma unroll
                         for (int e = 0; e < 8; e++)
-                            if (OH * c + j + e < pg.vdim) op[j + e] = __float2bfloat16_rn(o[j + e] * inv);
+                            if (OH * c + j + e < vdim) op[j + e] = __float2bfloat16_rn(o[j + e] * inv);
                     }
                 }
             } else if (!PAGED && r < rows) {
@@ -767,9 +801,9 @@ int launch2(const AttnPrefillArgs& a, int n_slots, cudaStream_t st) {
     const size_t rows = (size_t)n_slots * a.Hkv * a.n_ctx;
     if (!cached_kv_map(&mk, a.k_cache, rows, D) || !cached_kv_map(&mv, a.v_cache, rows, D)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D>::TOTAL);
+    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, D, FLAT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D, D>::TOTAL);
     dim3 grid((a.T + BQ - 1) / BQ, a.H);
-    attn_prefill_tc2_kernel<D, false><<<grid, THREADS2, Lay2<D>::TOTAL, st>>>(mk, mv, a, AttnPagedArgs{});
+    attn_prefill_tc2_kernel<D, D, FLAT><<<grid, THREADS2, Lay2<D, D>::TOTAL, st>>>(mk, mv, a, AttnPagedArgs{}, AttnPartsArgs{});
     return (int)cudaGetLastError();
 }
 
@@ -779,12 +813,44 @@ int launch_paged(const AttnPrefillArgs& a, const AttnPagedArgs& pg, int n_tiles,
     const size_t rows = (size_t)n_pages * a.Hkv * 64;
     if (!cached_kv_map(&mk, a.k_cache, rows, D, 64) || !cached_kv_map(&mv, a.v_cache, rows, D, 64)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D>::TOTAL);
-    attn_prefill_tc2_kernel<D, true><<<dim3(n_tiles, a.H), THREADS2, Lay2<D>::TOTAL, st>>>(mk, mv, a, pg);
+    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, D, PAGED_CACHE>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D, D>::TOTAL);
+    attn_prefill_tc2_kernel<D, D, PAGED_CACHE><<<dim3(n_tiles, a.H), THREADS2, Lay2<D, D>::TOTAL, st>>>(mk, mv, a, pg, AttnPartsArgs{});
+    return (int)cudaGetLastError();
+}
+
+template <int D, int DK>
+int launch_parts(const AttnPartsArgs& p, int n_tiles, cudaStream_t st) {
+    CUtensorMap mk, ms;
+    if (!make_kv_map(&mk, p.kv, p.n_rows, p.H * (p.dp + p.vp), BKV) || !make_kv_map(&ms, p.rp ? p.shared : p.kv, p.n_rows, p.rp ? p.rp : p.H * (p.dp + p.vp), BKV))
+        return (int)cudaErrorNotSupported;
+    static PerDeviceOnce once;
+    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, DK, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D, DK>::TOTAL);
+    AttnPrefillArgs a{};
+    a.H = a.Hkv = p.H;
+    a.causal = 1;
+    a.scale = p.scale;
+    a.out = p.out;
+    attn_prefill_tc2_kernel<D, DK, PARTS><<<dim3(n_tiles, p.H), THREADS2, Lay2<D, DK>::TOTAL, st>>>(mk, ms, a, AttnPagedArgs{}, p);
     return (int)cudaGetLastError();
 }
 
 }  // namespace
+
+// Attention of a step's query tiles over keys in two parts.  dp + rp: 64, 128 or 192 columns, vp: 64 or 128 with vp <= dp + rp; anything else:
+// cudaErrorNotSupported, nothing launched.
+B2_API int b2_attn_prefill_parts(const AttnPartsArgs* p, int n_tiles, cudaStream_t st) {
+    if (!p || !p->tiles || n_tiles < 1 || p->n_rows < 1 || p->H < 1 || p->H > 65535 || p->dp < 64 || (p->dp & 63) || (p->vp & 63) || p->rp < 0 || (p->rp & 63) ||
+        (p->rp && !p->shared) || p->vdim < 1 || p->vdim > p->vp || p->ldo < p->H * p->vdim)
+        return (int)cudaErrorInvalidValue;
+    if (((uintptr_t)p->kv & 15) || ((uintptr_t)p->shared & 15) || ((uintptr_t)p->q & 15) || ((uintptr_t)p->out & 15)) return (int)cudaErrorNotSupported;
+    const int dk = p->dp + p->rp;
+    if (p->vp == 128 && dk == 192) return launch_parts<128, 192>(*p, n_tiles, st);
+    if (p->vp == 128 && dk == 128) return launch_parts<128, 128>(*p, n_tiles, st);
+    if (p->vp == 64 && dk == 192) return launch_parts<64, 192>(*p, n_tiles, st);
+    if (p->vp == 64 && dk == 128) return launch_parts<64, 128>(*p, n_tiles, st);
+    if (p->vp == 64 && dk == 64) return launch_parts<64, 64>(*p, n_tiles, st);
+    return (int)cudaErrorNotSupported;
+}
 
 // Attention of a step's query tiles over a paged f16 cache (rows padded to head_dim 64 or 128; anything else: cudaErrorNotSupported,
 // nothing launched).  a: q [rows][H][head_dim], caches, out, H, Hkv, scale, softcap; the other fields are not used.

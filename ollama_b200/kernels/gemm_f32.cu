@@ -1,26 +1,21 @@
 // 32-bit matrix product of models that run in full precision: D[M, N] (+)= act(A[M, K] . B[N, K]^T), fp32 operands and fp32
-// fused multiply-adds (no reduced-precision matrix mode).  64 x 64 tiles, 4 x 4 outputs per thread, two shared-memory stages.
+// fused multiply-adds (no reduced-precision matrix mode).  64 x 64 tiles, 4 x 4 outputs per thread, two shared-memory stages.  The epilogues
+// are those of the tensor-core product (gemm_tc.cu).
 #include "rows.cuh"
 
 namespace {
 
 constexpr int TM = 64, TN = 64, TK = 16, LD = TM + 4;
 
-struct GemmF32Params {
-    const float* a;
-    const float* b;
-    int m, n, k, lda, ldb;
-    float* out;
-    int ldo, act, accumulate;
-};
-
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ GemmF32Params p) {
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ GemmRowsArgs p) {
     __shared__ __align__(16) float sa[2][TK][LD], sb[2][TK][LD];
     const int tid = threadIdx.x, m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
     const int lr = tid >> 2, lk = (tid & 3) * 4;            // this thread's row and first K element of a stage
     const int tx = tid & 15, ty = tid >> 4;
-    const float* ap = p.a + (size_t)min(m0 + lr, p.m - 1) * p.lda;
-    const float* bp = p.b + (size_t)min(n0 + lr, p.n - 1) * p.ldb;
+    const int e = p.tile_expert ? p.tile_expert[m0 >> 7] : 0;
+    if (e < 0) return;
+    const float* ap = (const float*)p.a + (size_t)min(m0 + lr, p.m - 1) * p.lda;
+    const float* bp = (const float*)p.b + ((size_t)e * p.n + min(n0 + lr, p.n - 1)) * p.ldb;
     auto fetch = [&](const float* row, int k0) {
         const int k = k0 + lk;
         return k < p.k ? *(const float4*)(row + k) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -59,25 +54,44 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
     for (int i = 0; i < 4; i++) {
         const int row = m0 + 4 * ty + i;
         if (row >= p.m) continue;
+        float v[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int col = min(n0 + 4 * tx + j, p.n - 1);
+            v[j] = acc[i][j] + (p.bias ? p.bias[col] : 0.f);
+        }
+        if (p.act >= GLU_BASE) {
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int col = n0 + 4 * tx + j;
+                if (col < p.n) ((float*)p.out)[(size_t)row * p.ldo + (col >> 1)] = glu_act_exact(v[j], v[j + 1], p.act - GLU_BASE, SWIGLU_ALPHA, p.limit);
+            }
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int col = n0 + 4 * tx + j;
             if (col >= p.n) continue;
-            float* o = p.out + (size_t)row * p.ldo + col;
-            const float v = out_act(acc[i][j], p.act);
-            *o = p.accumulate ? *o + v : v;
+            float* o = (float*)p.out + (size_t)row * p.ldo + col;
+            float r = out_act(v[j], p.act);
+            if (p.mul) r *= ((const float*)p.mul)[(size_t)p.mul_row[row] * p.ldm + col];
+            r *= p.alpha;
+            *o = p.accumulate ? *o + r : r;
         }
     }
 }
 
 }  // namespace
 
-// k, lda and ldb multiples of four, bases 16-byte aligned.  act: 0 none, 1 square of relu.  Returns a cudaError_t value.
-B2_API int b2_gemm_f32(const float* a, int lda, const float* b, int ldb, int m, int n, int k, float* out, int ldo, int act, int accumulate, cudaStream_t st) {
-    if (m < 1 || n < 1 || k < 4 || (k & 3) || (lda & 3) || (ldb & 3) || ((uintptr_t)a & 15) || ((uintptr_t)b & 15)) return (int)cudaErrorInvalidValue;
-    GemmF32Params p{a, b, m, n, k, lda, ldb, out, ldo, act, accumulate};
-    const dim3 grid((n + TN - 1) / TN, (m + TM - 1) / TM);
+// k, lda and ldb multiples of four, n even for gated products, bases 16-byte aligned.  Returns a cudaError_t value.
+B2_API int b2_gemm_rows_f32(const GemmRowsArgs* g, cudaStream_t st) {
+    const int glu = g->act >= GLU_BASE ? 1 : 0;
+    if (g->m < 1 || g->n < 1 || g->k < 4 || (g->k & 3) || (g->lda & 3) || (g->ldb & 3) || ((uintptr_t)g->a & 15) || ((uintptr_t)g->b & 15) || g->out_type || g->act < 0 ||
+        (!glu && g->act > 2) || g->act > GLU_BASE + 2 || (glu && ((g->n & 1) || g->accumulate || g->mul)) || (g->mul && !g->mul_row) ||
+        (g->tile_expert && (g->experts < 1 || (g->m & 127))))
+        return (int)cudaErrorInvalidValue;
+    const dim3 grid((g->n + TN - 1) / TN, (g->m + TM - 1) / TM);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-    gemm_f32_kernel<<<grid, 256, 0, st>>>(p);
+    gemm_f32_kernel<<<grid, 256, 0, st>>>(*g);
     return (int)cudaGetLastError();
 }

@@ -23,6 +23,7 @@
 // dequantise + cuBLAS path.
 #include "tc_common.cuh"
 #include "comm.cuh"
+#include "rows.cuh"
 
 __device__ int g_gemm_status = 0;
 
@@ -37,7 +38,7 @@ struct GemmParams {
     int ldo;                // elements
     const float* bias;      // [n] or null
     int accumulate;         // out += result (fp32 output only)
-    int out_bf16;
+    int out_bf16;           // 0 fp32, 1 bf16, 2 f16
     CommSend cm;            // cm.n_dst > 0: row r goes to cm.dst[r / rows_per_rank] at row r % rows_per_rank (bf16)
     int rows_per_rank;
     // grouped (mixture of experts): b holds E stacked [n][k] matrices and bias E x n values; the rows of a are sorted by expert
@@ -47,6 +48,10 @@ struct GemmParams {
     int glu;                // 0: off, 1 + act otherwise (0 silu, 1 gelu_tanh, 2 clamped swiglu)
     float glu_alpha, glu_limit;
     int act;                // ungated activation of the result (out_act), before it is stored or accumulated
+    float alpha;            // factor of the result, 0: none
+    const __nv_bfloat16* mul;      // factor per element: mul[mul_row[row] * ldm + column], or null
+    const int* mul_row;
+    int ldm;
     int lda;                // row pitch of a, 0: k
     // split-K (splits > 1): part s of a tile covers its own range of k blocks and stores plain fp32 sums at part + s * part_stride
     // ([m][part_ld]); a second kernel adds the parts in order and applies the epilogue
@@ -80,6 +85,43 @@ __device__ __forceinline__ void tile_coords(int t, int tiles_m, int tiles_n, int
 __device__ __forceinline__ uint32_t pack2_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+__device__ __forceinline__ uint32_t pack2_f16(float lo, float hi) {
+    const __half2 v = __floats2half2_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+// Four consecutive sums of a row, as the product's caller wants them: activation or gated pairs, factors, type, accumulation.
+__device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, int col) {
+    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
+    if (p.mul) {
+        const uint2 u = *(const uint2*)(p.mul + (size_t)p.mul_row[row] * p.ldm + col);
+        r.x *= __uint_as_float(u.x << 16); r.y *= __uint_as_float(u.x & 0xffff0000u);
+        r.z *= __uint_as_float(u.y << 16); r.w *= __uint_as_float(u.y & 0xffff0000u);
+    }
+    if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
+        const float h0 = glu_act(r.x, r.y, p.glu - 1, p.glu_alpha, p.glu_limit), h1 = glu_act(r.z, r.w, p.glu - 1, p.glu_alpha, p.glu_limit);
+        *(uint32_t*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + (col >> 1)) = pack2_bf16(h0, h1);
+        return;
+    }
+    if (p.alpha != 0.f) { r.x *= p.alpha; r.y *= p.alpha; r.z *= p.alpha; r.w *= p.alpha; }
+    if (p.cm.n_dst > 0) {      // partial rows travel as bf16: half the NVLink bytes of fp32
+        const int owner = row / p.rows_per_rank;
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.cm.dst[owner]) + (size_t)(row - owner * p.rows_per_rank) * p.ldo + col;
+        *(uint2*)dst = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
+    } else if (p.out_bf16 == 1) {
+        *(uint2*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
+    } else if (p.out_bf16) {
+        *(uint2*)((__half*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_f16(r.x, r.y), pack2_f16(r.z, r.w));
+    } else {
+        float* o = (float*)p.out + (size_t)row * p.ldo + col;
+        if (p.accumulate) {
+            const float4 old = *(const float4*)o;
+            r.x += old.x; r.y += old.y; r.z += old.z; r.w += old.w;
+        }
+        *(float4*)o = r;
+    }
 }
 
 template <int BN, bool SPLIT>
@@ -222,24 +264,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                         continue;
                     }
                     r.x += bias.x; r.y += bias.y; r.z += bias.z; r.w += bias.w;
-                    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
-                    if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
-                        const float h0 = glu_act(r.x, r.y, p.glu - 1, p.glu_alpha, p.glu_limit), h1 = glu_act(r.z, r.w, p.glu - 1, p.glu_alpha, p.glu_limit);
-                        *(uint32_t*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + (col >> 1)) = pack2_bf16(h0, h1);
-                    } else if (p.cm.n_dst > 0) {      // partial rows travel as bf16: half the NVLink bytes of fp32
-                        const int owner = row / p.rows_per_rank;
-                        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.cm.dst[owner]) + (size_t)(row - owner * p.rows_per_rank) * p.ldo + col;
-                        *(uint2*)dst = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
-                    } else if (p.out_bf16) {
-                        *(uint2*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
-                    } else {
-                        float* o = (float*)p.out + (size_t)row * p.ldo + col;
-                        if (p.accumulate) {
-                            const float4 old = *(const float4*)o;
-                            r.x += old.x; r.y += old.y; r.z += old.z; r.w += old.w;
-                        }
-                        *(float4*)o = r;
-                    }
+                    store4(p, r, row, col);
                 }
                 __syncwarp();
             }
@@ -287,7 +312,7 @@ int dispatch(const void* a, const void* b, const GemmParams& p, cudaStream_t st,
     const long tiles_m = (p.m + BM - 1) / BM;
     // a handful of rows (a decode step of several sequences): the product streams b once, so the narrowest tile that spreads
     // b over the most SMs wins
-    if (p.m <= 32 && (!p.out_bf16 || p.act || p.lda) && !p.glu && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
+    if (p.m <= 32 && (p.lda || (!p.out_bf16 && !p.glu)) && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
         return p.splits > 1 ? launch<64, true>(a, b, p, st, b_rows) : launch<64>(a, b, p, st, b_rows);
     if (p.splits > 1) return p.n >= 128 ? launch<128, true>(a, b, p, st, b_rows) : launch<64, true>(a, b, p, st, b_rows);
     if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256>(a, b, p, st, b_rows);
@@ -297,7 +322,7 @@ int dispatch(const void* a, const void* b, const GemmParams& p, cudaStream_t st,
     return launch<64>(a, b, p, st, b_rows);
 }
 
-// Parts of a split product, added in order; activation, accumulation and output type of the whole.
+// Parts of a split product, added in order; bias, activation, factors, accumulation and output type of the whole.
 __global__ void __launch_bounds__(256) gemm_parts_kernel(const __grid_constant__ GemmParams p) {
     const int row = blockIdx.y, col = 4 * (blockIdx.x * 256 + threadIdx.x);
     if (col >= p.n) return;
@@ -306,17 +331,11 @@ __global__ void __launch_bounds__(256) gemm_parts_kernel(const __grid_constant__
         const float4 v = *(const float4*)(p.part + s * p.part_stride + (size_t)row * p.part_ld + col);
         r.x += v.x; r.y += v.y; r.z += v.z; r.w += v.w;
     }
-    r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act);
-    if (p.out_bf16) {
-        *(uint2*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
-        return;
+    if (p.bias) {
+        const float4 b = *(const float4*)(p.bias + col);
+        r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
     }
-    float* o = (float*)p.out + (size_t)row * p.ldo + col;
-    if (p.accumulate) {
-        const float4 old = *(const float4*)o;
-        r.x += old.x; r.y += old.y; r.z += old.z; r.w += old.w;
-    }
-    *(float4*)o = r;
+    store4(p, r, row, col);
 }
 
 // How many parts to cut the row length into: a product whose tiles leave most SMs idle, as far as each part keeps some length.
@@ -351,30 +370,35 @@ B2_API int b2_gemm_bf16_out16(const void* a, const void* b, int m, int n, int k,
     return dispatch(a, b, p, st);
 }
 
-// The same product for operands and results inside wider buffers: a has row pitch lda (k % 8 == 0, lda % 8 == 0), the result goes
-// to rows of pitch ldo as bf16 (n % 4 == 0, out 8-byte aligned) or fp32, after the ungated activation `act` (0 none, 1 square of relu).
-// With scratch (`ws_floats` floats, b2_gemm_bf16_act_scratch) products of few tiles are split along k.
-B2_API int b2_gemm_bf16_act(const void* a, int lda, const void* b, int m, int n, int k, void* out, int ldo, int out16, int act, int accumulate, float* ws,
-                            long long ws_floats, cudaStream_t st) {
-    if (bad_operands(a, b, m, n, k, ldo) || lda < k || (lda & 7) || act < 0 || act > 1 || (out16 && accumulate) || ((uintptr_t)out & (out16 ? 7 : 15)) || ((uintptr_t)ws & 15))
+// The product of GemmRowsArgs.  k, lda and ldb multiples of 8 (ldb == k), n and ldo multiples of 4, bases 16-byte aligned (16-bit results: 8-byte;
+// gated: n a multiple of 8, bf16 results).  With scratch (b2_gemm_rows_scratch floats) products of few tiles are split along k.
+B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
+    const int glu = g->act >= GLU_BASE ? 1 + g->act - GLU_BASE : 0, m = g->m, n = g->n, k = g->k;
+    if (bad_operands(g->a, g->b, m, n, k, g->ldo) || g->lda < k || (g->lda & 7) || g->ldb != k || g->act < 0 || (!glu && g->act > 2) || glu > 3 || g->out_type < 0 ||
+        g->out_type > 2 || (g->out_type && g->accumulate) || ((uintptr_t)g->out & (g->out_type ? 7 : 15)) || ((uintptr_t)g->ws & 15) || ((uintptr_t)g->bias & 15))
         return (int)cudaErrorInvalidValue;
-    GemmParams p{m, n, k, out, ldo, nullptr, accumulate, out16, {}, 0, nullptr, 0, 0.f, 0.f, act, lda};
-    const int splits = ws ? split_count(m, n, k) : 1;
-    if (splits > 1 && (long long)splits * m * n <= ws_floats && m <= 65535) {
+    if (glu && (g->out_type != 1 || (n & 7) || g->mul)) return (int)cudaErrorInvalidValue;
+    if (g->mul && (!g->mul_row || (g->ldm & 3) || ((uintptr_t)g->mul & 7))) return (int)cudaErrorInvalidValue;
+    if (g->tile_expert && (g->experts < 1 || (m & 127))) return (int)cudaErrorInvalidValue;
+    GemmParams p{m, n, k, g->out, g->ldo, g->bias, g->accumulate, g->out_type, {}, 0, g->tile_expert, glu, SWIGLU_ALPHA, g->limit, glu ? 0 : g->act, g->alpha == 1.f ? 0.f : g->alpha,
+                 (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, g->lda};
+    if (g->tile_expert) return dispatch(g->a, g->b, p, st, g->experts * n);
+    const int splits = g->ws ? split_count(m, n, k) : 1;
+    if (splits > 1 && (long long)splits * m * n <= g->ws_floats && m <= 65535) {
         p.splits = splits;
-        p.part = ws;
+        p.part = g->ws;
         p.part_ld = n;
         p.part_stride = (long long)m * n;
-        const int rc = dispatch(a, b, p, st);
+        const int rc = dispatch(g->a, g->b, p, st);
         if (rc) return rc;
         gemm_parts_kernel<<<dim3((n + 1023) / 1024, m), 256, 0, st>>>(p);
         return (int)cudaGetLastError();
     }
-    return dispatch(a, b, p, st);
+    return dispatch(g->a, g->b, p, st);
 }
 
-// Floats of scratch with which b2_gemm_bf16_act would split a product of this size (0: it would not).
-B2_API long long b2_gemm_bf16_act_scratch(int m, int n, int k) {
+// Floats of scratch with which b2_gemm_rows would split a product of this size (0: it would not).
+B2_API long long b2_gemm_rows_scratch(int m, int n, int k) {
     const int s = split_count(m, n, k);
     return s > 1 ? (long long)s * m * n : 0;
 }

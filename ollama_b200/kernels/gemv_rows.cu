@@ -4,9 +4,10 @@
 // Up to four matrices share one launch and one source row.  The source is read in one of three ways:
 //   rows     fp32 activations as they are;
 //   norm     RMS-normalised: every segment has a norm weight of its own (branches of a parallel block), the weight is multiplied
-//            into the row while the dot products run and the row's 1 / rms, which every CTA computes, into the results;
+//            into the row while the dot products run and the row's 1 / rms, which every CTA computes, into the results.  A layer norm
+//            also subtracts mean times the matrix row's weighted sum and adds the row's product with the bias, both made at load;
 //   joined   two rows side by side;
-// The epilogue applies an ungated activation and stores or accumulates (the residual add).  The first rows of one matrix may also run
+// The epilogue applies an activation (of single rows, or of gate / up pairs), a factor, and stores or accumulates (the residual add).  The first rows of one matrix may also run
 // through a causal depthwise convolution + SiLU with the slot's last inputs (the state is only read here: the kernel that advances the
 // recurrence shifts it).  A warp owns four consecutive rows of a matrix and strides over their 16-byte pieces; short problems split the row
 // length over KS warps of the CTA.  Weight rows are requested from L2 before the grid-dependency wait (they do not depend on the producer
@@ -16,8 +17,13 @@
 struct RowSeg {
     const void* w;       // [n][ldw]
     const float* g;      // [k] norm weight (norm source)
+    const float* rs;     // [n] sum of w g over the row (layer norm)
+    const float* rc;     // [n] added to the result, or null
     float* out;          // [nb][ldo]
-    int n, ldw, ldo, act, accumulate;
+    int n, ldw, ldo;
+    int act;             // out_act's number, or GLU_BASE + glu_act's: rows 2i / 2i + 1 are gate / up of output i
+    int accumulate;
+    float alpha, limit;  // factor of the result; limit of the clamped gated unit
 };
 
 enum RowSrc : int { SRC_ROWS = 0, SRC_NORM = 1, SRC_JOINED = 2 };
@@ -41,6 +47,11 @@ struct GemvRowsArgs {
     int ldu;
     const int* slots;
     const int* positions;         // 0: the state counts as zeros
+    // norm source: layer norm instead of RMS norm, and the normalised row of matrix 0 as a result of its own (h = null: none)
+    int layer;
+    float* h;                     // [nb][ldh], k columns
+    int ldh;
+    const float* hb;              // [k] layer norm's bias
 };
 
 namespace {
@@ -74,7 +85,7 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
     constexpr int EB = F32 ? 4 : 2;
     constexpr int U = F32 || NB == 2 ? 1 : 2;           // pieces in flight per row
     __shared__ float red[8][R * NB];
-    __shared__ float s_ss[8][NB];
+    __shared__ float s_ss[8][NB], s_sm[8][NB];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int rg = warp / KS, ks = warp % KS;
     const uint8_t* wp[R];
@@ -101,13 +112,18 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
 #pragma unroll
         for (int b = 0; b < NB; b++) {
             const float* x = a.x + (size_t)(b < a.nb ? b : 0) * a.ldx;
-            float ss = 0.f;
+            float ss = 0.f, sm = 0.f;
             for (int i = 4 * threadIdx.x; i < a.k; i += 1024) {      // columns beyond the true length are zero
                 const float4 v = *(const float4*)(x + i);
                 ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                sm += v.x + v.y + v.z + v.w;
             }
             ss = warp_sum(ss);
-            if (lane == 0) s_ss[warp][b] = ss;
+            if (a.layer) sm = warp_sum(sm);
+            if (lane == 0) {
+                s_ss[warp][b] = ss;
+                s_sm[warp][b] = sm;
+            }
         }
     }
     float acc[R][NB];
@@ -173,20 +189,50 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
             if (lane == 0) red[warp][r * NB + b] = acc[r][b];
         }
     __syncthreads();
+    auto row_stats = [&](int b, float& mean, float& inv) {
+        float ss = 0.f, sm = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            ss += s_ss[i][b];
+            sm += s_sm[i][b];
+        }
+        mean = a.layer ? sm / (float)a.kn : 0.f;
+        inv = 1.f / sqrtf(fmaxf(ss / (float)a.kn - mean * mean, 0.f) + a.eps);
+    };
+    if (SRC == SRC_NORM && a.h) {          // a slice of the normalised rows per CTA
+        for (int i = blockIdx.x * 256 + threadIdx.x; i < a.nb * a.k; i += gridDim.x * 256) {
+            const int b = i / a.k, c = i - b * a.k;
+            float mean, inv;
+            row_stats(b, mean, inv);
+            a.h[(size_t)b * a.ldh + c] = (a.x[(size_t)b * a.ldx + c] - mean) * inv * a.seg[0].g[c] + (a.hb ? a.hb[c] : 0.f);
+        }
+    }
     const int r = lane / NB, b = lane % NB, row = row0 + r;
-    if (ks == 0 && active && lane < R * NB && row < w.n && b < a.nb) {
-        float v = 0.f;
+    if (ks != 0 || !active) return;
+    const bool mine = lane < R * NB && row < w.n && b < a.nb;
+    float v = 0.f;
+    if (mine) {
 #pragma unroll
         for (int k2 = 0; k2 < KS; k2++) v += red[rg * KS + k2][lane];
         if (SRC == SRC_NORM) {
-            float ss = 0.f;
-#pragma unroll
-            for (int i = 0; i < 8; i++) ss += s_ss[i][b];
-            v *= 1.f / sqrtf(ss / (float)a.kn + a.eps);
+            float mean, inv;
+            row_stats(b, mean, inv);
+            v = a.layer ? (v - mean * w.rs[row]) * inv : v * inv;
         }
+        if (w.rc) v += w.rc[row];
+    }
+    if (w.act >= GLU_BASE) {
+        const float up = __shfl_down_sync(0xffffffffu, v, NB);
+        if (mine && !(r & 1)) {
+            const float y = F32 ? glu_act_exact(v, up, w.act - GLU_BASE, SWIGLU_ALPHA, w.limit) : glu_act(v, up, w.act - GLU_BASE, SWIGLU_ALPHA, w.limit);
+            w.out[(size_t)b * w.ldo + (row >> 1)] = y;
+        }
+        return;
+    }
+    if (mine) {
         v = out_act(v, w.act);
         float* o = w.out + (size_t)b * w.ldo + row;
-        *o = w.accumulate ? *o + v : v;
+        *o = w.accumulate ? *o + w.alpha * v : w.alpha * v;
         if (s == a.conv_seg && row < a.conv_n) {
             float u = a.conv_b[row] + a.conv_w[(size_t)(a.taps - 1) * a.conv_n + row] * v;
             if (a.positions[b] > 0) {
@@ -230,10 +276,13 @@ B2_API int b2_gemv_rows(const GemvRowsArgs* a, int pdl, cudaStream_t st) {
     if (a->conv_seg >= 0 && (a->conv_seg >= a->nseg || a->conv_n < 1 || a->conv_n > a->seg[a->conv_seg].n || a->taps < 1 || !a->conv_w || !a->conv_b || !a->conv_state ||
                              !a->conv_out || !a->slots || !a->positions))
         return (int)cudaErrorInvalidValue;
+    if (a->h && a->src != SRC_NORM) return (int)cudaErrorInvalidValue;
     long groups = 0;
     for (int s = 0; s < a->nseg; s++) {
         const RowSeg& w = a->seg[s];
-        if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (a->src == SRC_NORM && (!w.g || ((uintptr_t)w.g & 15)))) return (int)cudaErrorInvalidValue;
+        if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (a->src == SRC_NORM && (!w.g || ((uintptr_t)w.g & 15) || (a->layer && !w.rs))) ||
+            w.act < 0 || (w.act > 2 && w.act < GLU_BASE) || w.act > GLU_BASE + 2 || (w.act >= GLU_BASE && (w.n & 1)))
+            return (int)cudaErrorInvalidValue;
         groups += (w.n + R - 1) / R;
     }
     // split the row length over KS warps until there are several row groups per resident warp, or a lane has two pieces left

@@ -1,0 +1,373 @@
+// Latent attention on a paged cache, sm_100a: everything around the scores.
+//
+// A position's cache row is [latent, padded to CP | rotated key part shared by all heads | zeros up to W]; pages of 64 rows as in
+// attn_paged.cu with one key head.  Per head the key is [U_h c | rotated part] and the value V_h c, so a query row may be taken into the
+// latent space instead, q . (U_h c) = (U_h^T q) . c, and the weighted sum of latents out of it, V_h (sum p c): attention then reads each
+// cache row once for all heads ("absorbed" form: decode steps, short portions, 32-bit models).  Long prompt portions multiply U and V
+// out for the visible positions instead, which costs fewer products per score.
+//
+//   latent_step    a row's latent under its RMS norm and rotated key part into the cache; U_h^T q and the rotated query part
+//   latent_merge   the split results of the absorbed form added up and multiplied by V_h
+//   latent_gather  cache rows of whole sequences side by side, for the products of the long form
+//   latent_query   query rows of the long form
+//
+// Rows: `rows` lists the rows of a step that a launch is for (null: all); results are stored in the order of that list, except
+// where noted.
+#include "rows.cuh"
+
+struct LatentStepArgs {
+    const float* qkv;        // [.][ldq]: per head dim unrotated | rot rotated values, then the latent, then the rotated key part
+    int ldq, n_heads, dim, rot, rank;
+    const float* norm;       // [rank] weight of the latent's norm
+    float eps;
+    const double* freqs;     // [rot / 2]
+    int interleaved;         // rotary pairs (2i, 2i + 1) instead of (i, i + rot / 2)
+    const int* rows;
+    const int* positions;    // of the step's rows
+    const int* slots;
+    const int* page_table;   // [slots][max_pages]
+    int max_pages;
+    void* cache;             // [pages][64][w]
+    int cp, w, cache32;      // padded latent, row length; element type f16 or fp32
+    int append;              // write the cache rows
+    const void* uk;          // [heads][dim][cp], bf16 or (w32) fp32; null: no queries
+    int w32;
+    void* q_out;             // [n][heads][w] in the cache's type
+};
+
+struct LatentMergeArgs {
+    const float* acc;        // [n][heads][splits][cp]
+    const float2* ml;        // [n][heads][splits] (max, sum; a sum of 0: nothing there), or null: one split, normalised
+    int n_heads, splits, cp, vdim;
+    const void* uv;          // [heads * vdim][cp]
+    int w32;
+    const int* rows;         // the result of list entry i goes to row rows[i]
+    void* out;               // [.][ldo], head h at column h * vdim
+    int ldo, out16;
+};
+
+struct LatentGatherArgs {
+    const __half* cache;
+    int cp, w, rot;
+    const int4* seqs;        // (first result row, positions, slot, -)
+    const int* page_table;
+    int max_pages;
+    __nv_bfloat16* c;        // [.][cp]
+    __half* r;               // [.][rp] rotated key part, zero-padded
+    int rp;
+};
+
+struct LatentQueryArgs {
+    const float* qkv;
+    int ldq, n_heads, dim, rot;
+    const double* freqs;
+    int interleaved;
+    const int* positions;
+    __half* q;               // [rows][heads][dp + rp]: unrotated part, zeros, rotated part, zeros
+    int dp, rp;
+};
+
+namespace {
+
+// Value i of a rotated part of n values.
+__device__ __forceinline__ float rotated_at(const float* v, int i, int n, int pos, const double* freqs, int interleaved) {
+    const int half = n >> 1;
+    const bool first = interleaved ? !(i & 1) : i < half;
+    const int pair = interleaved ? i >> 1 : (first ? i : i - half);
+    const float other = v[interleaved ? i ^ 1 : (first ? i + half : i - half)];
+    float sn, cs;
+    sincosf(rot_angle(pos, freqs[pair]), &sn, &cs);
+    return first ? v[i] * cs - other * sn : v[i] * cs + other * sn;
+}
+
+// One warp: cache row of step row r.
+template <typename CT>
+__device__ __forceinline__ void append_row(const LatentStepArgs& a, int r, int lane) {
+    const int pos = a.positions[r], slot = a.slots[r];
+    const float* c = a.qkv + (size_t)r * a.ldq + (size_t)a.n_heads * (a.dim + a.rot);
+    float ss = 0.f;
+    for (int i = lane; i < a.rank; i += 32) ss += c[i] * c[i];
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)a.rank + a.eps);
+    CT* o = (CT*)a.cache + paged_row(a.page_table + (size_t)slot * a.max_pages, pos, 1, 0) * a.w;
+    for (int i = lane; i < a.cp; i += 32) o[i] = from_f<CT>(i < a.rank ? c[i] * inv * a.norm[i] : 0.f);
+    for (int i = lane; i < a.w - a.cp; i += 32) o[a.cp + i] = from_f<CT>(i < a.rot ? rotated_at(c + a.rank, i, a.rot, pos, a.freqs, a.interleaved) : 0.f);
+}
+
+template <typename WT>
+__device__ __forceinline__ void load8(const WT* p, float (&f)[8]);
+template <>
+__device__ __forceinline__ void load8<float>(const float* p, float (&f)[8]) {
+    *(float4*)f = __ldg((const float4*)p);
+    *(float4*)(f + 4) = __ldg((const float4*)p + 1);
+}
+template <>
+__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&f)[8]) {
+    const uint4 v = __ldg((const uint4*)p);
+    const uint32_t q[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        f[2 * i] = __uint_as_float(q[i] << 16);
+        f[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
+    }
+}
+
+constexpr int COLS = 128;      // latent columns of a CTA of latent_step
+constexpr int DG = 16;         // groups of d values, one partial sum each
+
+// grid (heads * column parts + 1, row groups of NB): the last CTA of a row group appends, the others form U^T q
+template <typename CT, typename WT, int NB>
+__global__ void __launch_bounds__(256) latent_step_kernel(const __grid_constant__ LatentStepArgs a, int n) {
+    extern __shared__ float sq[];                  // [NB][dim]
+    __shared__ float red[DG][COLS + 4];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, i0 = blockIdx.y * NB;
+    const int parts = (a.cp + COLS - 1) / COLS;
+    const int h = blockIdx.x / parts, part = blockIdx.x % parts;
+    const bool appends = blockIdx.x == gridDim.x - 1;
+    const int cg = tid & 15, dg = tid >> 4, col = part * COLS + 8 * cg;
+    const WT* u = (const WT*)a.uk + ((size_t)h * a.dim) * a.cp + col;
+    pdl_launch();
+    if (!appends && col < a.cp && (cg & 7) == 0)
+        for (int d = dg; d < a.dim; d += DG) asm volatile("prefetch.global.L2 [%0];" ::"l"(u + (size_t)d * a.cp));
+    pdl_wait();
+    if (appends) {
+        if (a.append)
+            for (int b = warp; b < NB && i0 + b < n; b += 8) append_row<CT>(a, a.rows ? a.rows[i0 + b] : i0 + b, lane);
+        return;
+    }
+    const int nb = min(NB, n - i0), dq = a.dim + a.rot;
+    for (int j = tid; j < nb * a.dim; j += 256) {
+        const int b = j / a.dim, d = j - b * a.dim, r = a.rows ? a.rows[i0 + b] : i0 + b;
+        sq[b * a.dim + d] = a.qkv[(size_t)r * a.ldq + (size_t)h * dq + d];
+    }
+    if (part == 0) {                               // the rotated part and the zeros behind it
+        const int m = a.w - a.cp;
+        for (int j = tid; j < nb * m; j += 256) {
+            const int b = j / m, i = j - b * m, r = a.rows ? a.rows[i0 + b] : i0 + b;
+            const float* q = a.qkv + (size_t)r * a.ldq + (size_t)h * dq + a.dim;
+            ((CT*)a.q_out)[((size_t)(i0 + b) * a.n_heads + h) * a.w + a.cp + i] = from_f<CT>(i < a.rot ? rotated_at(q, i, a.rot, a.positions[r], a.freqs, a.interleaved) : 0.f);
+        }
+    }
+    __syncthreads();
+    float acc[NB][8];
+#pragma unroll
+    for (int b = 0; b < NB; b++)
+#pragma unroll
+        for (int e = 0; e < 8; e++) acc[b][e] = 0.f;
+    if (col < a.cp) {
+#pragma unroll 4
+        for (int d = dg; d < a.dim; d += DG) {
+            float w[8];
+            load8<WT>(u + (size_t)d * a.cp, w);
+#pragma unroll
+            for (int b = 0; b < NB; b++) {
+                const float q = b < nb ? sq[b * a.dim + d] : 0.f;
+#pragma unroll
+                for (int e = 0; e < 8; e++) acc[b][e] = fmaf(q, w[e], acc[b][e]);
+            }
+        }
+    }
+#pragma unroll
+    for (int b = 0; b < NB; b++) {
+        if (b >= nb) break;
+        __syncthreads();
+        *(float4*)&red[dg][8 * cg] = make_float4(acc[b][0], acc[b][1], acc[b][2], acc[b][3]);
+        *(float4*)&red[dg][8 * cg + 4] = make_float4(acc[b][4], acc[b][5], acc[b][6], acc[b][7]);
+        __syncthreads();
+        const int c = part * COLS + tid;
+        if (tid < COLS && c < a.cp) {
+            float s = 0.f;
+#pragma unroll
+            for (int g = 0; g < DG; g++) s += red[g][tid];
+            ((CT*)a.q_out)[((size_t)(i0 + b) * a.n_heads + h) * a.w + c] = from_f<CT>(s);
+        }
+    }
+}
+
+template <typename CT>
+__global__ void __launch_bounds__(128) latent_append_kernel(const __grid_constant__ LatentStepArgs a, int n) {
+    const int i = blockIdx.x * 4 + (threadIdx.x >> 5);
+    pdl_launch();
+    pdl_wait();
+    if (i < n) append_row<CT>(a, a.rows ? a.rows[i] : i, threadIdx.x & 31);
+}
+
+constexpr int MAX_SPLITS = 128, VROWS = 32;
+
+// grid (heads, value parts of VROWS, row groups of NB); a warp multiplies four value rows
+template <typename WT, int NB>
+__global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant__ LatentMergeArgs a, int n) {
+    extern __shared__ __align__(16) float so[];    // [NB][cp]
+    __shared__ float sw[NB][MAX_SPLITS];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, i0 = blockIdx.z * NB, nb = min(NB, n - i0);
+    const int v0 = blockIdx.y * VROWS + warp * (VROWS / 8);
+    pdl_launch();
+    for (int j = 0; j < VROWS / 8; j++)
+        if (v0 + j < a.vdim)
+            for (int c = lane * (128 / (int)sizeof(WT)); c < a.cp; c += 32 * (128 / (int)sizeof(WT)))
+                asm volatile("prefetch.global.L2 [%0];" ::"l"((const WT*)a.uv + ((size_t)h * a.vdim + v0 + j) * a.cp + c));
+    pdl_wait();
+    if (a.ml) {
+        if (warp < nb) {
+            const float2* ml = a.ml + ((size_t)(i0 + warp) * a.n_heads + h) * a.splits;
+            float m = -INFINITY, l = 0.f;
+            for (int s = lane; s < a.splits; s += 32)
+                if (ml[s].y > 0.f) m = fmaxf(m, ml[s].x);
+            m = warp_max(m);
+            for (int s = lane; s < a.splits; s += 32) {
+                const float w = ml[s].y > 0.f ? expf(ml[s].x - m) : 0.f;
+                sw[warp][s] = w;
+                l += w * ml[s].y;
+            }
+            l = warp_sum(l);
+            __syncwarp();
+            for (int s = lane; s < a.splits; s += 32) sw[warp][s] /= l;
+        }
+        __syncthreads();
+    }
+    for (int j = tid; j < nb * (a.cp >> 2); j += 256) {
+        const int b = j / (a.cp >> 2), c = 4 * (j - b * (a.cp >> 2));
+        const float* p = a.acc + ((size_t)(i0 + b) * a.n_heads + h) * a.splits * a.cp + c;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (a.ml) {
+            for (int s = 0; s < a.splits; s++) {
+                const float w = sw[b][s];
+                if (w == 0.f) continue;            // splits without keys leave their sums unwritten
+                const float4 v = *(const float4*)(p + (size_t)s * a.cp);
+                o.x += w * v.x; o.y += w * v.y; o.z += w * v.z; o.w += w * v.w;
+            }
+        } else {
+            o = *(const float4*)p;
+        }
+        *(float4*)(so + b * a.cp + c) = o;
+    }
+    __syncthreads();
+    for (int j = 0; j < VROWS / 8; j++) {
+        const int v = v0 + j;
+        if (v >= a.vdim) return;
+        const WT* w = (const WT*)a.uv + ((size_t)h * a.vdim + v) * a.cp;
+        float acc[NB];
+#pragma unroll
+        for (int b = 0; b < NB; b++) acc[b] = 0.f;
+        for (int c = 8 * lane; c < a.cp; c += 256) {
+            float f[8];
+            load8<WT>(w + c, f);
+#pragma unroll
+            for (int b = 0; b < NB; b++) {
+                if (b >= nb) break;
+#pragma unroll
+                for (int e = 0; e < 8; e++) acc[b] = fmaf(f[e], so[b * a.cp + c + e], acc[b]);
+            }
+        }
+#pragma unroll
+        for (int b = 0; b < NB; b++) {
+            if (b >= nb) break;
+            const float s = warp_sum(acc[b]);
+            if (lane == 0) {
+                const size_t o = (size_t)(a.rows ? a.rows[i0 + b] : i0 + b) * a.ldo + (size_t)h * a.vdim + v;
+                if (a.out16) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(s);
+                else ((float*)a.out)[o] = s;
+            }
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256) latent_gather_kernel(const __grid_constant__ LatentGatherArgs a) {
+    const int4 q = a.seqs[blockIdx.y];
+    const int pos = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (pos >= q.y) return;
+    const __half* src = a.cache + paged_row(a.page_table + (size_t)q.z * a.max_pages, pos, 1, 0) * a.w;
+    __nv_bfloat16* c = a.c + (size_t)(q.x + pos) * a.cp;
+    for (int i = 8 * lane; i < a.cp; i += 256) {
+        const uint4 v = *(const uint4*)(src + i);
+        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+        uint32_t o[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const float2 f = __half22float2(*reinterpret_cast<const __half2*>(&w[j]));
+            const __nv_bfloat162 b = __floats2bfloat162_rn(f.x, f.y);
+            o[j] = *reinterpret_cast<const uint32_t*>(&b);
+        }
+        *(uint4*)(c + i) = make_uint4(o[0], o[1], o[2], o[3]);
+    }
+    __half* r = a.r + (size_t)(q.x + pos) * a.rp;
+    for (int i = lane; i < a.rp; i += 32) r[i] = i < a.rot ? src[a.cp + i] : __float2half_rn(0.f);
+}
+
+// one CTA per row
+__global__ void __launch_bounds__(256) latent_query_kernel(const __grid_constant__ LatentQueryArgs a) {
+    extern __shared__ float cs[];                  // [rot / 2] cosines, then sines
+    const int r = blockIdx.x, half = a.rot >> 1, pos = a.positions[r], dk = a.dp + a.rp;
+    for (int i = threadIdx.x; i < half; i += 256) sincosf(rot_angle(pos, a.freqs[i]), &cs[half + i], &cs[i]);
+    __syncthreads();
+    const float* q = a.qkv + (size_t)r * a.ldq;
+    __half* o = a.q + (size_t)r * a.n_heads * dk;
+    for (int j = threadIdx.x; j < a.n_heads * (dk >> 1); j += 256) {      // two neighbouring values
+        const int h = j / (dk >> 1), c = 2 * (j - h * (dk >> 1));
+        const float* qh = q + (size_t)h * (a.dim + a.rot);
+        float v[2];
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int i = c + e - a.dp;
+            if (c + e < a.dim) v[e] = qh[c + e];
+            else if (i < 0 || i >= a.rot) v[e] = 0.f;
+            else {
+                const float* t = qh + a.dim;
+                const bool first = a.interleaved ? !(i & 1) : i < half;
+                const int p = a.interleaved ? i >> 1 : (first ? i : i - half);
+                const float y = t[a.interleaved ? i ^ 1 : (first ? i + half : i - half)];
+                v[e] = first ? t[i] * cs[p] - y * cs[half + p] : t[i] * cs[p] + y * cs[half + p];
+            }
+        }
+        *(__half2*)(o + (size_t)h * dk + c) = __floats2half2_rn(v[0], v[1]);
+    }
+}
+
+template <typename CT, typename WT>
+const void* step_fn(int nb) {
+    return nb == 1 ? (const void*)latent_step_kernel<CT, WT, 1> : (const void*)latent_step_kernel<CT, WT, 4>;
+}
+
+}  // namespace
+
+// Cache rows (append) and absorbed queries (uk set) of n rows.  Returns a cudaError_t value, as do the entry points below.
+B2_API int b2_latent_step(const LatentStepArgs* a, int n, int pdl, cudaStream_t st) {
+    if (n < 1 || a->n_heads < 1 || a->dim < 1 || a->rot < 0 || (a->rot & 1) || a->rank < 1 || a->cp < a->rank || (a->cp & 15) || a->w < a->cp + a->rot || (a->rot && !a->freqs) ||
+        (!a->uk && !a->append) || (a->uk && (!a->q_out || ((uintptr_t)a->uk & 15))) || a->dim > 8192 || a->max_pages < 1)
+        return (int)cudaErrorInvalidValue;
+    LatentStepArgs c = *a;
+    void* args[] = {&c, &n};
+    if (!a->uk)
+        return launch_rows(a->cache32 ? (const void*)latent_append_kernel<float> : (const void*)latent_append_kernel<__half>, dim3((n + 3) / 4), dim3(128), 0, args, st, pdl);
+    const int nb = n == 1 ? 1 : 4, parts = (a->cp + COLS - 1) / COLS;
+    const void* fn = a->cache32 ? (a->w32 ? step_fn<float, float>(nb) : step_fn<float, __nv_bfloat16>(nb)) : (a->w32 ? step_fn<__half, float>(nb) : step_fn<__half, __nv_bfloat16>(nb));
+    const size_t smem = (size_t)nb * a->dim * 4;
+    if (smem > 32 * 1024) return (int)cudaErrorNotSupported;
+    if ((n + nb - 1) / nb > 65535) return (int)cudaErrorInvalidValue;
+    return launch_rows(fn, dim3(a->n_heads * parts + 1, (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
+}
+
+B2_API int b2_latent_merge(const LatentMergeArgs* a, int n, int pdl, cudaStream_t st) {
+    if (n < 1 || a->n_heads < 1 || a->splits < 1 || a->splits > MAX_SPLITS || (!a->ml && a->splits != 1) || (a->cp & 15) || a->vdim < 1 || ((uintptr_t)a->uv & 15) || ((uintptr_t)a->acc & 15))
+        return (int)cudaErrorInvalidValue;
+    const int nb = n == 1 ? 1 : 4;
+    const size_t smem = (size_t)nb * a->cp * 4;
+    if (smem > 40 * 1024) return (int)cudaErrorNotSupported;
+    if ((n + nb - 1) / nb > 65535) return (int)cudaErrorInvalidValue;
+    LatentMergeArgs c = *a;
+    void* args[] = {&c, &n};
+    const void* fn = a->w32 ? (nb == 1 ? (const void*)latent_merge_kernel<float, 1> : (const void*)latent_merge_kernel<float, 4>)
+                            : (nb == 1 ? (const void*)latent_merge_kernel<__nv_bfloat16, 1> : (const void*)latent_merge_kernel<__nv_bfloat16, 4>);
+    return launch_rows(fn, dim3(a->n_heads, (a->vdim + VROWS - 1) / VROWS, (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
+}
+
+B2_API int b2_latent_gather(const LatentGatherArgs* a, int n_seqs, int max_len, cudaStream_t st) {
+    if (n_seqs < 1 || n_seqs > 65535 || max_len < 1 || (a->cp & 15) || (a->w & 7) || a->rp < a->rot) return (int)cudaErrorInvalidValue;
+    latent_gather_kernel<<<dim3((max_len + 7) / 8, n_seqs), 256, 0, st>>>(*a);
+    return (int)cudaGetLastError();
+}
+
+B2_API int b2_latent_query(const LatentQueryArgs* a, int rows, cudaStream_t st) {
+    if (rows < 1 || a->n_heads < 1 || a->dp < a->dim || a->rp < a->rot || (a->dp & 1) || (a->rp & 1) || (a->rot & 1) || a->rot > 4096) return (int)cudaErrorInvalidValue;
+    latent_query_kernel<<<rows, 256, (size_t)a->rot * 4, st>>>(*a);
+    return (int)cudaGetLastError();
+}

@@ -242,9 +242,9 @@ B2_API int b2_moe_gather(const void* h, const int* row_of_pair, int pairs, int k
     return (int)cudaGetLastError();
 }
 
-// out[t] (+)= sum_s wts[t][s] * ys[row_of_pair[t k + s]]   (pairs whose expert lives elsewhere contribute nothing)
+// out[t] (+)= mult * sum_s wts[t][s] * ys[row_of_pair[t k + s]]   (pairs whose expert lives elsewhere contribute nothing)
 __global__ void __launch_bounds__(256) moe_scatter_combine_kernel(const float* ys, const int* row_of_pair, const float* wts, int k, int d,
-                                                                  float* out, int accumulate) {
+                                                                  float* out, int ldo, int accumulate, float mult) {
     const int t = blockIdx.x;
     for (int c = threadIdx.x; c < (d >> 2); c += 256) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -255,7 +255,8 @@ __global__ void __launch_bounds__(256) moe_scatter_combine_kernel(const float* y
             const float4 v = *(const float4*)(ys + (size_t)r * d + 4 * c);
             acc.x += w * v.x; acc.y += w * v.y; acc.z += w * v.z; acc.w += w * v.w;
         }
-        float4* o = (float4*)(out + (size_t)t * d + 4 * c);
+        acc.x *= mult; acc.y *= mult; acc.z *= mult; acc.w *= mult;
+        float4* o = (float4*)(out + (size_t)t * ldo + 4 * c);
         if (accumulate) {
             const float4 x = *o;
             acc.x += x.x; acc.y += x.y; acc.z += x.z; acc.w += x.w;
@@ -264,9 +265,9 @@ __global__ void __launch_bounds__(256) moe_scatter_combine_kernel(const float* y
     }
 }
 
-B2_API int b2_moe_scatter_combine(const float* ys, const int* row_of_pair, const float* wts, int tokens, int k, int d, float* out,
-                                  int accumulate, cudaStream_t st) {
-    if (tokens < 1 || k < 1 || (d & 3)) return (int)cudaErrorInvalidValue;
-    moe_scatter_combine_kernel<<<tokens, 256, 0, st>>>(ys, row_of_pair, wts, k, d, out, accumulate);
+B2_API int b2_moe_scatter_combine(const float* ys, const int* row_of_pair, const float* wts, int tokens, int k, int d, float* out, int ldo,
+                                  int accumulate, float mult, cudaStream_t st) {
+    if (tokens < 1 || k < 1 || (d & 3) || ldo < d || (ldo & 3)) return (int)cudaErrorInvalidValue;
+    moe_scatter_combine_kernel<<<tokens, 256, 0, st>>>(ys, row_of_pair, wts, k, d, out, ldo, accumulate, mult);
     return (int)cudaGetLastError();
 }

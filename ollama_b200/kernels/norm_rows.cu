@@ -2,18 +2,46 @@
 // the same input with weights of their own read it once), two rows side by side, and a column window.  Results are bf16
 // (tensor-core operands) or fp32 (32-bit models); columns beyond the row length are written as zeros, so that products may run
 // over a padded row length.
+//
+// The norm is an RMS norm or a layer norm.  Before it, the row itself may be updated in place in the same pass: a branch's result
+// under an RMS norm of its own is added, and vectors that join a pass of a loop.
 #include "rows.cuh"
 
 struct NormRowsArgs {
-    const float* x;      // [rows][ldx]
+    float* x;            // [rows][ldx]; written only when one of y, x0, step is set
     int ldx, k, ldo;     // k values per row; outputs have pitch ldo >= k
     float eps;
     const float* w1;     // [k] weight of the first result
     const float* w2;     // [k] weight of the second result, or null
-    void* o1;
+    void* o1;            // null: only the update
     void* o2;
     int f32;             // element type of the results: 0 bf16, 1 fp32
+    const float* b1;     // [k] layer norm: bias of the first result; null: RMS norm
+    const float* b2;
+    // x += mult * rmsnorm(y) * wy + x0 + step, each term optional
+    const float* y;      // [rows][ldy]
+    const float* wy;     // [k]
+    const float* x0;     // [rows][ldx]
+    const float* step;   // [k]
+    int ldy;
+    float mult;
 };
+
+namespace {
+
+// Sum over the CTA of 256; `red` is free again after the call of the next one.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+    v = warp_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) t += red[i];
+    return t;
+}
+
+}  // namespace
 
 template <typename T>
 __global__ void __launch_bounds__(256) norm_rows_kernel(const __grid_constant__ NormRowsArgs a) {
@@ -21,29 +49,43 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const __grid_constant__ 
     const int row = blockIdx.x, tid = threadIdx.x;
     pdl_launch();
     pdl_wait();
-    const float* x = a.x + (size_t)row * a.ldx;
-    float ss = 0.f;
-    if ((a.k & 3) == 0) {
-        for (int i = 4 * tid; i < a.k; i += 1024) {
-            const float4 v = *(const float4*)(x + i);
-            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    float* x = a.x + (size_t)row * a.ldx;
+    if (a.y || a.x0 || a.step) {
+        const float* y = a.y ? a.y + (size_t)row * a.ldy : nullptr;
+        const float* x0 = a.x0 ? a.x0 + (size_t)row * a.ldx : nullptr;
+        float ry = 0.f;
+        if (y) {
+            float s = 0.f;
+            for (int i = tid; i < a.k; i += 256) s += y[i] * y[i];
+            ry = a.mult / sqrtf(block_sum(s, red) / (float)a.k + a.eps);
         }
-    } else {
-        for (int i = tid; i < a.k; i += 256) ss += x[i] * x[i];
+        for (int i = tid; i < a.k; i += 256) {      // a thread reads the same elements again below
+            float v = x[i];
+            if (y) v += ry * y[i] * a.wy[i];
+            if (x0) v += x0[i];
+            if (a.step) v += a.step[i];
+            x[i] = v;
+        }
     }
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float t = 0.f;
-#pragma unroll
-    for (int i = 0; i < 8; i++) t += red[i];
-    const float inv = 1.f / sqrtf(t / (float)a.k + a.eps);
+    if (!a.o1) return;
+    float mean = 0.f, ss = 0.f;
+    if (a.b1) {
+        float s = 0.f;
+        for (int i = tid; i < a.k; i += 256) s += x[i];
+        mean = block_sum(s, red) / (float)a.k;
+    }
+    for (int i = tid; i < a.k; i += 256) {
+        const float d = x[i] - mean;
+        ss += d * d;
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)a.k + a.eps);
     T* o1 = (T*)a.o1 + (size_t)row * a.ldo;
     T* o2 = a.o2 ? (T*)a.o2 + (size_t)row * a.ldo : nullptr;
     for (int i = tid; i < a.ldo; i += 256) {
-        const float v = i < a.k ? x[i] * inv : 0.f;
-        o1[i] = from_f<T>(i < a.k ? v * a.w1[i] : 0.f);
-        if (o2) o2[i] = from_f<T>(i < a.k ? v * a.w2[i] : 0.f);
+        const bool in = i < a.k;
+        const float v = in ? (x[i] - mean) * inv : 0.f;
+        o1[i] = from_f<T>(in ? v * a.w1[i] + (a.b1 ? a.b1[i] : 0.f) : 0.f);
+        if (o2) o2[i] = from_f<T>(in ? v * a.w2[i] + (a.b2 ? a.b2[i] : 0.f) : 0.f);
     }
 }
 
@@ -63,42 +105,79 @@ __global__ void __launch_bounds__(256) norm_rows4_kernel(const __grid_constant__
     constexpr int J = 4;
     __shared__ float red[8];
     const int row = blockIdx.x, tid = threadIdx.x, n4 = a.k >> 2;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     pdl_launch();
     pdl_wait();
-    const float* x = a.x + (size_t)row * a.ldx;
+    float* x = a.x + (size_t)row * a.ldx;
     float4 v[J], w[J];
-    float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < J; j++) {
         const int i = tid + 256 * j;
-        v[j] = i < n4 ? *(const float4*)(x + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        w[j] = i < n4 ? __ldg((const float4*)(a.w1 + 4 * i)) : v[j];
+        v[j] = i < n4 ? *(const float4*)(x + 4 * i) : zero;
+        w[j] = i < n4 && a.o1 ? __ldg((const float4*)(a.w1 + 4 * i)) : zero;
+    }
+    if (a.y || a.x0 || a.step) {
+        if (a.y) {
+            float4 y[J];
+            float s = 0.f;
+#pragma unroll
+            for (int j = 0; j < J; j++) {
+                const int i = tid + 256 * j;
+                y[j] = i < n4 ? *(const float4*)(a.y + (size_t)row * a.ldy + 4 * i) : zero;
+                s += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
+            }
+            const float ry = a.mult / sqrtf(block_sum(s, red) / (float)a.k + a.eps);
+#pragma unroll
+            for (int j = 0; j < J; j++) {
+                const int i = tid + 256 * j;
+                const float4 g = i < n4 ? __ldg((const float4*)(a.wy + 4 * i)) : zero;
+                v[j].x += ry * y[j].x * g.x; v[j].y += ry * y[j].y * g.y; v[j].z += ry * y[j].z * g.z; v[j].w += ry * y[j].w * g.w;
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < J; j++) {
+            const int i = tid + 256 * j;
+            if (i >= n4) continue;
+            if (a.x0) {
+                const float4 u = *(const float4*)(a.x0 + (size_t)row * a.ldx + 4 * i);
+                v[j].x += u.x; v[j].y += u.y; v[j].z += u.z; v[j].w += u.w;
+            }
+            if (a.step) {
+                const float4 u = __ldg((const float4*)(a.step + 4 * i));
+                v[j].x += u.x; v[j].y += u.y; v[j].z += u.z; v[j].w += u.w;
+            }
+            *(float4*)(x + 4 * i) = v[j];
+        }
+    }
+    if (!a.o1) return;
+    float ss = 0.f;
+    if (a.b1) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < J; j++) s += v[j].x + v[j].y + v[j].z + v[j].w;
+        const float mean = block_sum(s, red) / (float)a.k;
+#pragma unroll
+        for (int j = 0; j < J; j++) {
+            if (tid + 256 * j >= n4) continue;
+            v[j].x -= mean; v[j].y -= mean; v[j].z -= mean; v[j].w -= mean;
+        }
     }
 #pragma unroll
     for (int j = 0; j < J; j++) ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float t = 0.f;
-#pragma unroll
-    for (int i = 0; i < 8; i++) t += red[i];
-    const float inv = 1.f / sqrtf(t / (float)a.k + a.eps);
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)a.k + a.eps);
     T* o1 = (T*)a.o1 + (size_t)row * a.ldo;
     T* o2 = a.o2 ? (T*)a.o2 + (size_t)row * a.ldo : nullptr;
+    auto bias = [&](const float* b, int i) { return b ? __ldg((const float4*)(b + 4 * i)) : zero; };
 #pragma unroll
     for (int j = 0; j < J; j++) {
         const int i = tid + 256 * j;
         v[j].x *= inv; v[j].y *= inv; v[j].z *= inv; v[j].w *= inv;
-        if (i < n4) put4(o1 + 4 * i, v[j].x * w[j].x, v[j].y * w[j].y, v[j].z * w[j].z, v[j].w * w[j].w);
-    }
-    if (o2) {
-#pragma unroll
-        for (int j = 0; j < J; j++) {
-            const int i = tid + 256 * j;
-            if (i < n4) {
-                const float4 u = __ldg((const float4*)(a.w2 + 4 * i));
-                put4(o2 + 4 * i, v[j].x * u.x, v[j].y * u.y, v[j].z * u.z, v[j].w * u.w);
-            }
+        if (i >= n4) continue;
+        const float4 b = bias(a.b1, i);
+        put4(o1 + 4 * i, v[j].x * w[j].x + b.x, v[j].y * w[j].y + b.y, v[j].z * w[j].z + b.z, v[j].w * w[j].w + b.w);
+        if (o2) {
+            const float4 u = __ldg((const float4*)(a.w2 + 4 * i)), c = bias(a.b2, i);
+            put4(o2 + 4 * i, v[j].x * u.x + c.x, v[j].y * u.y + c.y, v[j].z * u.z + c.z, v[j].w * u.w + c.w);
         }
     }
     for (int i = a.k + tid; i < a.ldo; i += 256) {
@@ -108,11 +187,14 @@ __global__ void __launch_bounds__(256) norm_rows4_kernel(const __grid_constant__
 }
 
 B2_API int b2_norm_rows(const NormRowsArgs* a, int rows, int pdl, cudaStream_t st) {
-    if (rows < 1 || a->k < 1 || a->ldo < a->k || (a->ldx & 3) || !a->w1 || (a->o2 && !a->w2)) return (int)cudaErrorInvalidValue;
+    if (rows < 1 || a->k < 1 || !a->x || (a->ldx & 3) || (a->o1 && (!a->w1 || a->ldo < a->k)) || (a->o2 && (!a->w2 || !a->o1 || !a->b1 != !a->b2)) || (a->y && !a->wy) ||
+        (!a->o1 && !a->y && !a->x0 && !a->step))
+        return (int)cudaErrorInvalidValue;
     NormRowsArgs c = *a;
     void* args[] = {&c};
-    if ((a->k & 3) == 0 && a->k <= 4096 && (a->ldo & 3) == 0 &&
-        !(((uintptr_t)a->x | (uintptr_t)a->w1 | (uintptr_t)a->w2 | (uintptr_t)a->o1 | (uintptr_t)a->o2) & 15))
+    const uintptr_t all = (uintptr_t)a->x | (uintptr_t)a->w1 | (uintptr_t)a->w2 | (uintptr_t)a->o1 | (uintptr_t)a->o2 | (uintptr_t)a->b1 | (uintptr_t)a->b2 |
+                          (uintptr_t)a->y | (uintptr_t)a->wy | (uintptr_t)a->x0 | (uintptr_t)a->step;
+    if ((a->k & 3) == 0 && a->k <= 4096 && (a->ldo & 3) == 0 && (a->ldy & 3) == 0 && !(all & 15))
         return launch_rows(a->f32 ? (const void*)norm_rows4_kernel<float> : (const void*)norm_rows4_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, args, st, pdl);
     return launch_rows(a->f32 ? (const void*)norm_rows_kernel<float> : (const void*)norm_rows_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, args, st, pdl);
 }

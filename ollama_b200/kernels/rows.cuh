@@ -45,3 +45,25 @@ static inline int launch_rows(const void* fn, dim3 grid, dim3 block, size_t smem
     cfg.numAttrs = 1;
     return (int)cudaLaunchKernelExC(&cfg, fn, args);
 }
+
+// Matrix product of a step's rows: out[m][ldo] (+)= alpha * f(a[m][lda] . b[n][ldb]^T + bias).  Served by b2_gemm_rows (bf16 operands on the
+// tensor cores, gemm_tc.cu) and b2_gemm_rows_f32 (fp32 operands, gemm_f32.cu).
+struct GemmRowsArgs {
+    const void* a;
+    const void* b;
+    void* out;
+    const float* bias;        // [n] or null
+    // result times a table row: mul[mul_row[r] * ldm + column] in the operands' type, after the activation
+    const void* mul;
+    const int* mul_row;       // [m]
+    // grouped over experts: b holds `experts` stacked [n][k] matrices, the rows of a are sorted by expert and every tile of 128 rows
+    // belongs to expert tile_expert[row / 128] (-1: no rows)
+    const int* tile_expert;
+    float* ws;                // scratch for splitting k (bf16 products only), or null
+    long long ws_floats;
+    int m, n, k, lda, ldb, ldo;
+    int out_type;             // 0 fp32, 1 bf16, 2 f16
+    int act;                  // out_act's number, or GLU_BASE + glu_act's: rows 2i / 2i + 1 of b are gate / up of column i
+    int accumulate, experts, ldm;
+    float alpha, limit;       // limit: of the clamped gated unit
+};

@@ -673,22 +673,23 @@ def moe_plan(lids: torch.Tensor, n_experts: int) -> tuple[torch.Tensor, torch.Te
 
 
 def moe_gather(h: torch.Tensor, row_of_pair: torch.Tensor, k: int, rows: int) -> torch.Tensor:
-    """bf16 activation rows [T, d] -> [rows, d] sorted by expert (rows nobody owns are left as they are)."""
-    xs = torch.empty(rows, h.shape[1], dtype=torch.bfloat16, device=h.device)
+    """Activation rows [T, d] (bf16 or fp32) -> [rows, d] sorted by expert (rows nobody owns are left as they are)."""
+    xs = torch.empty(rows, h.shape[1], dtype=h.dtype, device=h.device)
     f = lib().b2_moe_gather
     f.argtypes = [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_void_p]
-    _check(f(ptr(h), ptr(row_of_pair), row_of_pair.numel(), k, h.shape[1], ptr(xs), stream()), "moe_gather")
+    _check(f(ptr(h), ptr(row_of_pair), row_of_pair.numel(), k, h.shape[1] * h.element_size() // 2, ptr(xs), stream()), "moe_gather")
     return xs
 
 
 def moe_scatter_combine(ys: torch.Tensor, row_of_pair: torch.Tensor, wts: torch.Tensor, tokens: int, k: int, out: torch.Tensor | None = None,
-                        accumulate: bool = False) -> torch.Tensor:
+                        accumulate: bool = False, mult: float = 1.0) -> torch.Tensor:
+    """out[t] (+)= mult * sum over t's slots of their weight times the sorted buffer's row."""
     d = ys.shape[1]
     if out is None:
         out = torch.empty(tokens, d, dtype=torch.float32, device=ys.device)
     f = lib().b2_moe_scatter_combine
-    f.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_void_p]
-    _check(f(ptr(ys), ptr(row_of_pair), ptr(wts), tokens, k, d, ptr(out), int(accumulate), stream()), "moe_scatter_combine")
+    f.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_int, C.c_float, C.c_void_p]
+    _check(f(ptr(ys), ptr(row_of_pair), ptr(wts), tokens, k, d, ptr(out), out.stride(0), int(accumulate), mult, stream()), "moe_scatter_combine")
     return out
 
 

@@ -1,16 +1,19 @@
-"""Bindings of the row kernels behind stack models: norms, fused decode products, 32-bit products, paged attention and the selective
-state-space mixer (kernels/norm_rows.cu, gemv_rows.cu, gemm_f32.cu, attn_paged.cu, ssm.cu)."""
+"""Bindings of the row kernels behind stack models: norms, fused decode products, products of many rows, paged attention and the selective
+state-space mixer (kernels/norm_rows.cu, gemv_rows.cu, gemm_tc.cu, gemm_f32.cu, attn_paged.cu, ssm.cu)."""
 from __future__ import annotations
 
 import ctypes as C
 import functools
+import math
 
 import torch
 
 from .cuda import AttnDecodeArgs, AttnPrefillArgs, AttnRopeArgs, _check, lib, ptr, stream
 
 P, I, F = C.c_void_p, C.c_int, C.c_float
-ACT = {"": 0, "relu2": 1}
+GLU_BASE = 16
+ACT = {"": 0, "relu2": 1, "gelu_tanh": 2, "glu:silu": GLU_BASE, "glu:gelu_tanh": GLU_BASE + 1, "glu:swiglu_oai": GLU_BASE + 2}
+OUT_TYPE = {torch.float32: 0, torch.bfloat16: 1, torch.float16: 2}
 SRC_ROWS, SRC_NORM, SRC_JOINED = range(3)
 GEMV_MAX_ROWS = 4
 
@@ -19,12 +22,18 @@ def _st(name: str, fields: list) -> type:
     return type(name, (C.Structure,), {"_fields_": fields})
 
 
-NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), ("eps", F), ("w1", P), ("w2", P), ("o1", P), ("o2", P), ("f32", I)])
+NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), ("eps", F), ("w1", P), ("w2", P), ("o1", P), ("o2", P), ("f32", I),
+                                    ("b1", P), ("b2", P), ("y", P), ("wy", P), ("x0", P), ("step", P), ("ldy", I), ("mult", F)])
 JoinRowsArgs = _st("JoinRowsArgs", [("a", P), ("b", P), ("lda", I), ("n_a", I), ("ldb", I), ("n_b", I), ("out", P), ("ldo", I), ("off_b", I), ("f32", I)])
-RowSeg = _st("RowSeg", [("w", P), ("g", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I)])
+RowSeg = _st("RowSeg", [("w", P), ("g", P), ("rs", P), ("rc", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I), ("alpha", F),
+                        ("limit", F)])
+GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P), ("mul", P), ("mul_row", P), ("tile_expert", P), ("ws", P),
+                                    ("ws_floats", C.c_longlong), ("m", I), ("n", I), ("k", I), ("lda", I), ("ldb", I), ("ldo", I), ("out_type", I), ("act", I),
+                                    ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
                                     ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
-                                    ("conv_b", P), ("conv_state", P), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P)])
+                                    ("conv_b", P), ("conv_state", P), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
+                                    ("layer", I), ("h", P), ("ldh", I), ("hb", P)])
 PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
                                           ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
                                           ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I)])
@@ -51,10 +60,15 @@ def _call(name: str, args, *more) -> None:
     _check(getattr(lib(), name)(C.byref(args), *more, stream()), name)
 
 
-def norm_rows(x: torch.Tensor, k: int, eps: float, w1: torch.Tensor, o1: torch.Tensor, w2: torch.Tensor | None = None, o2: torch.Tensor | None = None,
-              pdl: bool = False) -> None:
-    """o1 = rmsnorm(x) * w1 and, in the same pass, o2 = rmsnorm(x) * w2, for the first ``k`` columns; pad columns of the results are zeroed."""
-    a = NormRowsArgs(ptr(x), x.stride(0), k, o1.stride(0), eps, ptr(w1), ptr(w2), ptr(o1), ptr(o2), _is32(o1))
+def norm_rows(x: torch.Tensor, k: int, eps: float, w1: torch.Tensor | None, o1: torch.Tensor | None, w2: torch.Tensor | None = None,
+              o2: torch.Tensor | None = None, b1: torch.Tensor | None = None, b2: torch.Tensor | None = None, y: torch.Tensor | None = None,
+              wy: torch.Tensor | None = None, mult: float = 1.0, x0: torch.Tensor | None = None, step: torch.Tensor | None = None, pdl: bool = False) -> None:
+    """o1 = norm(x) * w1 and, in the same pass, o2 = norm(x) * w2, for the first ``k`` columns; pad columns of the results are zeroed.  With biases
+    a layer norm, else an RMS norm.  Before it x += mult * rmsnorm(y) * wy + x0 + step, in place, of the terms that are given; ``o1`` None: only that."""
+    if x0 is not None and x0.stride(0) != x.stride(0):
+        raise ValueError("norm_rows: row pitch of the joined rows")
+    a = NormRowsArgs(ptr(x), x.stride(0), k, o1.stride(0) if o1 is not None else 0, eps, ptr(w1), ptr(w2), ptr(o1), ptr(o2), _is32(o1) if o1 is not None else 0,
+                     ptr(b1), ptr(b2), ptr(y), ptr(wy), ptr(x0), ptr(step), y.stride(0) if y is not None else 0, mult)
     _call("b2_norm_rows", a, x.shape[0], int(pdl))
 
 
@@ -64,22 +78,28 @@ def join_rows(a: torch.Tensor, n_a: int, out: torch.Tensor, b: torch.Tensor | No
     _call("b2_join_rows", args, a.shape[0], int(pdl))
 
 
-def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = None, act: str = "", accumulate: bool = False) -> RowSeg:
-    """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``."""
-    s = RowSeg(ptr(w), ptr(g), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate))
-    s.keep = (w, g, out)             # the structure holds addresses only
+def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = None, act: str = "", accumulate: bool = False, alpha: float = 1.0,
+        limit: float = math.inf, rs: torch.Tensor | None = None, rc: torch.Tensor | None = None) -> RowSeg:
+    """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``, as out (+)= alpha * act(... + rc).  ``rs``: the rows' sums of
+    w * g (layer norm).  Gated activations ("glu:...") take rows 2i and 2i + 1 as gate and up of column i."""
+    s = RowSeg(ptr(w), ptr(g), ptr(rs), ptr(rc), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate), alpha, limit)
+    s.keep = (w, g, rs, rc, out)     # the structure holds addresses only
     return s
 
 
 def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,
          k1: int = 0, conv=None, conv_out: torch.Tensor | None = None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None,
-         pdl: bool = False) -> None:
+         layer: bool = False, h: torch.Tensor | None = None, hb: torch.Tensor | None = None, pdl: bool = False) -> None:
     """Products of up to four matrices with up to four source rows.  ``conv`` = (weights [taps, n], bias [n], state [slots, taps - 1, n]): the first n
-    results of the first matrix also run through that convolution and SiLU, into ``conv_out``."""
+    results of the first matrix also run through that convolution and SiLU, into ``conv_out``.  ``layer``: the norm source is a layer norm;
+    ``h``: its rows for the first matrix are stored too (``hb``: the norm's bias)."""
     a = GemvRowsArgs()
     for i, s in enumerate(segs):
         a.seg[i] = s
     a.nseg, a.nb, a.k, a.src, a.f32, a.x, a.ldx, a.eps, a.kn, a.conv_seg = len(segs), nb, k, src, int(f32), ptr(x), x.stride(0), eps, kn, -1
+    a.layer = int(layer)
+    if h is not None:
+        a.h, a.ldh, a.hb = ptr(h), h.stride(0), ptr(hb)
     if x2 is not None:
         a.x2, a.ldx2, a.k1 = ptr(x2), x2.stride(0), k1
     if conv is not None:
@@ -89,27 +109,28 @@ def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC
     _call("b2_gemv_rows", a, int(pdl))
 
 
-def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", accumulate: bool = False, k: int | None = None) -> None:
-    """out (+)= act(a[:, :k] @ w[:, :k]^T); bf16 operands on tcgen05 (result bf16 or fp32), fp32 operands in full 32 bits.  ``a`` and ``out`` may be
-    column windows of wider buffers."""
-    m, n, k = a.shape[0], w.shape[0], w.shape[1] if k is None else k
-    if a.dtype != w.dtype or out.shape[0] != m or out.shape[1] != n or a.shape[1] < k or a.stride(1) != 1 or out.stride(1) != 1:
+def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", accumulate: bool = False, k: int | None = None, alpha: float = 1.0,
+         limit: float = math.inf, bias: torch.Tensor | None = None, mul: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
+         experts: int = 0, tile_expert: torch.Tensor | None = None) -> None:
+    """out (+)= alpha * act(a[:, :k] @ w[:, :k]^T + bias) [* mul[mul_row]]; bf16 operands on tcgen05 (result bf16, f16 or fp32), fp32 operands in full
+    32 bits.  ``a``, ``out`` and ``mul`` may be column windows of wider buffers.  Gated activations ("glu:...") halve the columns.  ``experts``: w holds
+    that many stacked matrices and a's tiles of 128 rows belong to ``tile_expert``."""
+    n = w.shape[0] // max(experts, 1)
+    m, k = a.shape[0], w.shape[1] if k is None else k
+    cols = n // 2 if act.startswith("glu:") else n
+    if a.dtype != w.dtype or out.shape[0] != m or out.shape[1] != cols or a.shape[1] < k or a.stride(1) != 1 or out.stride(1) != 1:
         raise ValueError(f"gemm: {tuple(a.shape)} {a.dtype} x {tuple(w.shape)} {w.dtype} -> {tuple(out.shape)}")
-    if a.dtype == torch.float32:
-        f = lib().b2_gemm_f32
-        f.argtypes = [P, I, P, I, I, I, I, P, I, I, I, P]
-        _check(f(ptr(a), a.stride(0), ptr(w), w.stride(0), m, n, k, ptr(out), out.stride(0), ACT[act], int(accumulate), stream()), "gemm_f32")
-        return
-    size = _split_floats(m, n, k)
+    f32 = a.dtype == torch.float32
+    size = 0 if f32 or experts else _split_floats(m, n, k)
     ws = torch.empty(size, device=a.device) if size else None
-    f = lib().b2_gemm_bf16_act
-    f.argtypes = [P, I, P, I, I, I, P, I, I, I, I, P, C.c_longlong, P]
-    _check(f(ptr(a), a.stride(0), ptr(w), m, n, k, ptr(out), out.stride(0), 1 - _is32(out), ACT[act], int(accumulate), ptr(ws), size, stream()), "gemm_bf16_act")
+    g = GemmRowsArgs(ptr(a), ptr(w), ptr(out), ptr(bias), ptr(mul), ptr(mul_row), ptr(tile_expert), ptr(ws), size, m, n, k, a.stride(0), w.stride(0), out.stride(0),
+                     OUT_TYPE[out.dtype], ACT[act], int(accumulate), experts, mul.stride(0) if mul is not None else 0, alpha, limit)
+    _call("b2_gemm_rows_f32" if f32 else "b2_gemm_rows", g)
 
 
 @functools.lru_cache(maxsize=4096)
 def _split_floats(m: int, n: int, k: int) -> int:
-    f = lib().b2_gemm_bf16_act_scratch
+    f = lib().b2_gemm_rows_scratch
     f.restype, f.argtypes = C.c_longlong, [I, I, I]
     return int(f(m, n, k))
 

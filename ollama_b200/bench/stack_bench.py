@@ -1,10 +1,11 @@
-"""Throughput of stack models beside a dense model of equal size, both in bf16 with random weights on one GPU.
+"""Throughput of stack models beside a model of equal size, both in bf16 with random weights on one GPU.
 
-    python bench.py --stack [--model vazatar-1b|vazatar-8b|all] [--steps K] [--warmup W]
+    python bench.py --stack [--model NAME|all] [--steps K] [--warmup W]
 
 For each size: prompt evaluation of a 2048-token prompt, and decode steps of 1, 4 and 16 sequences at 1024 tokens of context.  Besides
 tokens per second every figure carries its fraction of the roofline: the matrix products' FLOPs over the bf16 GEMM peak for prompts, the
-weight and cache bytes of a step over the copy bandwidth for decoding.  Weights of a step exceed the L2, so that nothing has to be flushed.
+weight and cache bytes of a step over the copy bandwidth for decoding (of experts, the ones that a step of so many tokens picks on average).
+Weights of a step exceed the L2, so that nothing has to be flushed.
 """
 from __future__ import annotations
 
@@ -14,7 +15,7 @@ import statistics
 
 import torch
 
-PAIRS = {"vazatar-1b": "dense-1b", "vazatar-8b": "dense-8b"}
+PAIRS = {"vazatar-1b": "dense-1b", "vazatar-8b": "dense-8b", "kavenex-1b": "dense-1b", "kavenex-8b": "dense-8b", "kavenex-moe": "experts-2k"}
 PROMPT, CONTEXT, BATCHES, LOOP = 2048, 1024, (1, 4, 16), 32
 
 
@@ -30,24 +31,22 @@ def peaks() -> tuple[float, float]:
 
 
 def load(name: str, dev: str):
-    """(backend, matrix weights read by one pass over the layers and the head)."""
+    """(backend, matrix weights that a token is multiplied with, weights of the experts of one such pass, share of the experts a token picks)."""
     from ..models import synth
     if name in synth.STACK_SPECS:
         from ..engine.stack import StackBackend
         cfg = synth.stack_model_config(synth.STACK_SPECS[name])
         be = StackBackend(None, device=dev, cfg=cfg, tensors=synth.SyntheticStackTensors(synth.STACK_SPECS[name], device=dev))
-        n = be.head.numel()
-        for r in be.runs if be.stack.design.parallel else ():
-            L = be.layers[r.layer]
-            n += sum(t.numel() for t in (L.w_in, L.up, L.w_out, getattr(L, "w_x", None), getattr(L, "w_dt", None)) if t is not None)
-            n += be.loop_in.numel() if r.joins else 0
-        return be, n
+        dense, routed, share = be.product_weights()
+        return be, dense, routed, share
     from ..engine.b200 import B200Backend
     from ..models.config import config_from_gguf
     cfg = config_from_gguf(synth.synthetic_header(name, "BF16"))
     be = B200Backend(None, device=dev, cfg=cfg, tensors=synth.SyntheticTensors(name, "BF16", seed=0, device=dev), kv_type="f16")
-    n = cfg.n_layers * (cfg.d_model * (2 * cfg.q_dim + 2 * cfg.kv_dim) + 3 * cfg.d_model * cfg.d_ff) + cfg.vocab_size * cfg.d_model
-    return be, n
+    n = cfg.n_layers * cfg.d_model * (2 * cfg.q_dim + 2 * cfg.kv_dim) + cfg.vocab_size * cfg.d_model
+    if cfg.is_moe:
+        return be, n + cfg.n_layers * cfg.d_model * cfg.n_experts, cfg.n_layers * cfg.n_experts * 3 * cfg.d_model * cfg.d_ff_expert, cfg.n_experts_used / cfg.n_experts
+    return be, n + cfg.n_layers * 3 * cfg.d_model * cfg.d_ff, 0, 0.0
 
 
 def timed(fn, warmup: int, steps: int) -> float:
@@ -67,7 +66,8 @@ def timed(fn, warmup: int, steps: int) -> float:
 
 
 def measure(name: str, steps: int, warmup: int, dev: str = "cuda:0") -> dict:
-    be, n = load(name, dev)
+    be, dense, routed, share = load(name, dev)
+    n = int(dense + routed * share)
     cfg = be.cfg
     hbm, flops = peaks()
     be.alloc(max(BATCHES), PROMPT + 64)
@@ -81,7 +81,7 @@ def measure(name: str, steps: int, warmup: int, dev: str = "cuda:0") -> dict:
         for s in slots:
             be.prefill(s, toks[:CONTEXT], 0, need_logits=False)
         t = timed(lambda: be.decode_loop(slots, [1] * nb, [CONTEXT] * nb, LOOP), warmup, steps) / LOOP
-        byts = 2 * n + nb * cfg.kv_bytes_per_token() * CONTEXT
+        byts = 2 * (dense + routed * (1.0 - (1.0 - share) ** nb)) + nb * cfg.kv_bytes_per_token() * CONTEXT
         out[f"decode_{nb}"] = {"tok_s": round(nb / t, 1), "step_us": round(t * 1e6, 1), "roofline": round(byts / t / hbm, 3), "launches": be.launches_per_step}
     from ..ops import cuda as K
     out["status"] = K.gemm_status()
@@ -93,6 +93,6 @@ def measure(name: str, steps: int, warmup: int, dev: str = "cuda:0") -> dict:
 
 def run(model: str, steps: int, warmup: int) -> dict:
     names = list(PAIRS) if model in ("auto", "all") else [model]
-    rows = [measure(m, steps, max(warmup, 3)) for name in names for m in (name, PAIRS[name])]
+    rows = [measure(m, steps, max(warmup, 3)) for m in dict.fromkeys(m for name in names for m in (name, PAIRS[name]))]
     return {"metric": "stack_models", "unit": "tok/s", "dtype": "bf16", "data": "synthetic", "config": {"prompt": PROMPT, "context": CONTEXT, "batches": list(BATCHES),
             "l2": "weights of a step are larger than L2"}, "results": rows}

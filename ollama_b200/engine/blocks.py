@@ -72,7 +72,6 @@ class Norm:
 class Mat:
     """Matrix of a product; ``rs`` and ``rc`` fold a layer norm before it in (see kernels/gemv_rows.cu)."""
     w: torch.Tensor
-    n: int                            # rows that hold something
     bias: torch.Tensor | None = None
     rs: torch.Tensor | None = None
     rc: torch.Tensor | None = None
@@ -128,11 +127,11 @@ class Step:
             self.launched()
 
     def product(self, h: torch.Tensor, mat: Mat, out: torch.Tensor, **kw) -> None:
-        """out (+)= f(mat h + bias)."""
+        """out (+)= f(mat h + bias) [times the tokens' rows of a table ``mul``]."""
         if self.small:
-            O.gemv([O.seg(mat.w, mat.n, out, rc=mat.bias, **kw)], mat.w.shape[1], h, self.nb, self.be.f32, pdl=self.pdl)
+            O.gemv([O.seg(mat.w, mat.w.shape[0], out, rc=mat.bias, **kw)], mat.w.shape[1], h, self.nb, self.be.f32, mul_row=self.m.tokens, pdl=self.pdl)
         else:
-            O.gemm(h, mat.w, out, bias=mat.bias, **kw)
+            O.gemm(h, mat.w, out, bias=mat.bias, mul_row=self.m.tokens, **kw)
         self.launched()
 
     def add(self, h: torch.Tensor, mat: Mat) -> None:
@@ -145,7 +144,7 @@ class Step:
         h = self.buf("h", be.wp) if keep or not self.folded else None
         if self.folded:
             self.flush()
-            O.gemv([O.seg(mat.w, mat.n, out, norm.g, rs=mat.rs, rc=mat.rc, **kw)], be.wp, self.x, self.nb, False, O.SRC_NORM, st.eps, st.width, layer=True, h=h,
+            O.gemv([O.seg(mat.w, mat.w.shape[0], out, norm.g, rs=mat.rs, rc=mat.rc, **kw)], be.wp, self.x, self.nb, False, O.SRC_NORM, st.eps, st.width, layer=True, h=h,
                    hb=norm.b, pdl=self.pdl)
             self.launched()
             return h
@@ -162,8 +161,8 @@ class LatentAttention:
         self.m, self.norm, self.f32 = m, norm, f32
         nq = H * (m.dim + m.rot_dim)
         n_in = nq + m.kv_rank + m.rot_dim
-        self.w_in = Mat(src.pack([(0, 0, p + "attn_q.weight", (nq, w)), (nq, 0, p + "attn_kv_a_mqa.weight", (m.kv_rank + m.rot_dim, w))], up(n_in), src.wp), n_in)
-        self.w_o = Mat(src.pack([(0, 0, p + "attn_output.weight", (w, H * m.vdim))], src.wp, up(H * m.vdim)), w)
+        self.w_in = Mat(src.pack([(0, 0, p + "attn_q.weight", (nq, w)), (nq, 0, p + "attn_kv_a_mqa.weight", (m.kv_rank + m.rot_dim, w))], up(n_in), src.wp))
+        self.w_o = Mat(src.pack([(0, 0, p + "attn_output.weight", (w, H * m.vdim))], src.wp, up(H * m.vdim)))
         self.c_norm = src.vec(p + "attn_kv_a_norm.weight", m.kv_rank)
         self.cp = up(m.kv_rank, 16)
         self.row = up(self.cp + m.rot_dim, 32)           # values of a cache row
@@ -183,6 +182,9 @@ class LatentAttention:
             self.w_kv[H * self.dp:].view(H, self.vp, self.cp)[:, :m.vdim] = self.uv.view(H, m.vdim, self.cp)
         if not f32:
             self.w_in.fold(norm)
+
+    def product_weights(self) -> tuple[int, int, float]:
+        return sum(t.numel() for t in (self.w_in.w, self.uk, self.uv, self.w_o.w)), 0, 0.0
 
     def make_cache(self, cache) -> tuple[torch.Tensor]:
         return (cache.add_pages(1, self.row, self.cache_type),)
@@ -208,9 +210,9 @@ class LatentAttention:
                     positions=s.m.positions, slots=s.m.slots, table=s.be.cache.table, cp=self.cp, pdl=s.pdl)
 
     def splits(self, n: int, n_ctx: int, sms: int) -> int:
-        """Parts of the keys for ``n`` queries: about two CTAs per SM, none shorter than two pages."""
+        """Parts of the keys for ``n`` queries: as many CTAs as are resident (wide rows: one per SM), none shorter than two pages."""
         groups = -(-self.m.heads // (16 if self.m.heads <= 16 else 32))
-        return max(1, min(-(-n_ctx // 128), 2 * sms // (groups * n), MAX_SPLITS))
+        return max(1, min(-(-n_ctx // 128), (1 if self.row > 256 else 2) * sms // (groups * n), MAX_SPLITS))
 
     def _latent(self, s: Step, qkv, cache, out, n: int, rows, append: bool) -> None:
         """Attention of ``n`` rows in the latent space."""
@@ -247,10 +249,13 @@ class GatedFFN:
     def __init__(self, src: WeightSource, p: str, m: DenseMLP, norm: Norm, f32: bool, names=("ffn_gate", "ffn_up", "ffn_down")):
         gate, up_name, down = (p + n + ".weight" for n in names)
         self.norm, self.act, self.ffp = norm, "glu:" + m.act, up(m.ff)
-        self.w_gu = Mat(src.gate_up(gate, up_name, m.ff), 2 * m.ff)
-        self.w_down = Mat(src.pack([(0, 0, down, (src.width, m.ff))], src.wp, self.ffp), src.width)
+        self.w_gu = Mat(src.gate_up(gate, up_name, m.ff))
+        self.w_down = Mat(src.pack([(0, 0, down, (src.width, m.ff))], src.wp, self.ffp))
         if not f32:
             self.w_gu.fold(norm)
+
+    def product_weights(self) -> tuple[int, int, float]:
+        return self.w_gu.w.numel() + self.w_down.w.numel(), 0, 0.0
 
     def run(self, s: Step) -> None:
         f = s.buf("ff", self.ffp, zero=True)
@@ -272,17 +277,21 @@ class ExpertFFN:
     def __init__(self, src: WeightSource, p: str, m: ExpertMLP, norm: Norm, f32: bool):
         w, E = src.width, m.experts
         self.m, self.norm, self.ffp = m, norm, up(m.expert.ff)
-        self.router = Mat(src.pack([(0, 0, p + "ffn_gate_inp.weight", (E, w))], up(E), src.wp), E, bias=src.vec(p + "ffn_gate_inp.bias", E))
+        self.router = Mat(src.pack([(0, 0, p + "ffn_gate_inp.weight", (E, w))], up(E), src.wp), bias=src.vec(p + "ffn_gate_inp.bias", E))
         self.gu = src.gate_up(p + "ffn_gate_exps.weight", p + "ffn_up_exps.weight", m.expert.ff, (E,))
         self.down = src.zeros(E, src.wp, self.ffp)
         self.down[:, :w, :m.expert.ff] = src.tensor(p + "ffn_down_exps.weight", E, w, m.expert.ff)
         self.shared = None
         if m.shared is not None:
             ff = m.shared.ff
-            self.shared = _Shared(m.shared, Mat(src.gate_up(p + "ffn_gate_shexp.weight", p + "ffn_up_shexp.weight", ff), 2 * ff),
-                                  Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff)), w))
+            self.shared = _Shared(m.shared, Mat(src.gate_up(p + "ffn_gate_shexp.weight", p + "ffn_up_shexp.weight", ff)),
+                                  Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff))))
         if not f32:
             self.router.fold(norm)
+
+    def product_weights(self) -> tuple[int, int, float]:
+        sh = self.shared
+        return (self.router.w.numel() + (sh.gu.w.numel() + sh.down.w.numel() if sh else 0), self.gu.numel() + self.down.numel(), self.m.top / self.m.experts)
 
     def run(self, s: Step) -> None:
         m, sh = self.m, self.shared
@@ -317,25 +326,20 @@ class SideInput:
 
     def __init__(self, src: WeightSource, p: str, dim: int, table: torch.Tensor):
         self.dim, self.dimp, self.e = dim, up(dim), table      # table [vocab, dimp]: this layer's part of every token's row
-        self.gate = Mat(src.pack([(0, 0, p + "inp_gate.weight", (dim, src.width))], self.dimp, src.wp), dim)
-        self.proj = Mat(src.pack([(0, 0, p + "proj.weight", (src.width, dim))], src.wp, self.dimp), src.width)
+        self.gate = Mat(src.pack([(0, 0, p + "inp_gate.weight", (dim, src.width))], self.dimp, src.wp))
+        self.proj = Mat(src.pack([(0, 0, p + "proj.weight", (src.width, dim))], src.wp, self.dimp))
         self.w = src.vec(p + "post_norm.weight", src.width)
 
-    def run(self, s: Step, join: dict) -> dict:
-        """``join``: vectors that the next layer run adds first; returned where they are still to be added."""
-        st, mult = s.be.stack, s.be.stack.residual_mult
-        if s.small and A.side_rows(s.x, s.nb, st.width, self.gate.w, self.e, self.dim, s.m.tokens, self.proj.w, self.w, st.eps, mult, pdl=s.pdl, **join):
+    def product_weights(self) -> tuple[int, int, float]:
+        return self.gate.w.numel() + self.proj.w.numel(), 0, 0.0
+
+    def run(self, s: Step) -> None:
+        h = s.x
+        if h.dtype != s.act:
+            h = s.buf("side_x", s.be.wp)
+            O.join_rows(s.x, s.be.wp, h, pdl=s.pdl)
             s.launched()
-            return {}
-        act = s.be.act_dtype
-        xb = s.x
-        if act != torch.float32:
-            xb = s.buf("side_x", s.be.wp, act)
-            O.join_rows(s.x, s.be.wp, xb, pdl=s.pdl)
-            s.launched()
-        g, y = s.buf("side_g", self.dimp, act), s.buf("side_y", s.be.wp, torch.float32)
-        O.gemm(xb, self.gate.w, g, act="gelu_tanh", mul=self.e, mul_row=s.m.tokens)
-        O.gemm(g, self.proj.w, y)
-        s.launched(2)
-        s.pending = {"y": y, "wy": self.w, "mult": mult}
-        return join
+        g, y = s.buf("side_g", self.dimp), s.buf("side_y", s.be.wp, torch.float32)
+        s.product(h, self.gate, g, act="gelu_tanh", mul=self.e)
+        s.product(g, self.proj, y)
+        s.pending = {"y": y, "wy": self.w, "mult": s.be.stack.residual_mult}

@@ -20,6 +20,7 @@ from __future__ import annotations
 import logging
 from typing import Sequence
 
+import numpy as np
 import torch
 
 from .. import envconfig
@@ -180,7 +181,7 @@ class StackBackend(StepEngine):
         """Layers whose mixer and feed-forward follow one another, each behind a layer norm."""
         st, f32 = self.stack, self.f32
         self.out_norm = make_norm(src, "output_norm")
-        self.out_mat = Mat(self.head, st.vocab)
+        self.out_mat = Mat(self.head)
         if not f32:
             self.out_mat.fold(self.out_norm)
         if st.loop is not None:
@@ -222,6 +223,20 @@ class StackBackend(StepEngine):
 
     def weight_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in self._weights())
+
+    def product_weights(self) -> tuple[int, int, float]:
+        """Matrix weights over all layer runs and the head: (those every token is multiplied with, those of the routed experts, the share of
+        the routed ones that a token picks)."""
+        dense, routed, share = self.head.numel(), 0, 0.0
+        for r in self.runs:
+            L = self.layers[r.layer]
+            if self.stack.design.parallel:
+                dense += sum(t.numel() for t in (L.w_in, L.up, L.w_out, getattr(L, "w_x", None), getattr(L, "w_dt", None)) if t is not None)
+                dense += self.loop_in.numel() if r.joins else 0
+                continue
+            d, e, p = (sum(v) for v in zip(*(b.product_weights() for b in (L.mix, L.ff, L.side) if b is not None)))
+            dense, routed, share = dense + d, routed + e, max(share, p)
+        return dense, routed, share
 
     def kv_bytes(self) -> int:
         return self.cache.nbytes() if getattr(self, "cache", None) is not None else 0
@@ -415,15 +430,12 @@ class StackBackend(StepEngine):
             L.mix.run(s, self.mem[i])
             if L.ff is not None:
                 L.ff.run(s)
-            join = self._join(nxt, s)
+            if L.side is not None:
+                L.side.run(s)
             if tap is not None:                # the stream of this layer run, before anything is added for the next one
-                if L.side is not None:
-                    L.side.run(s, {})
                 s.flush()
                 tap(i, s.x[:, :self.stack.width])
-            elif L.side is not None:
-                join = L.side.run(s, join)
-            s.pending.update(join)
+            s.pending.update(self._join(nxt, s))
         s.flush()
         return s.x
 
@@ -433,7 +445,7 @@ class StackBackend(StepEngine):
         if isinstance(self.out_norm, Norm):
             if nb <= self.gemv_rows and not self.f32:
                 m = self.out_mat
-                O.gemv([O.seg(m.w, m.n, out, self.out_norm.g, rs=m.rs, rc=m.rc)], self.wp, x, nb, False, O.SRC_NORM, st.eps, st.width, layer=True, pdl=pdl)
+                O.gemv([O.seg(m.w, m.w.shape[0], out, self.out_norm.g, rs=m.rs, rc=m.rc)], self.wp, x, nb, False, O.SRC_NORM, st.eps, st.width, layer=True, pdl=pdl)
             else:
                 h = torch.empty(nb, self.wp, device=self.device, dtype=self.act_dtype)
                 O.norm_rows(x, st.width, st.eps, self.out_norm.g, h, b1=self.out_norm.b, pdl=pdl)
@@ -475,31 +487,33 @@ class StackBackend(StepEngine):
         """Rows of several sequences, each portion ``(slot, tokens, position of the first)``; returns the hidden rows in order."""
         dev = self.device
         self._reserve([s for s, _, _ in segs], [p0 + len(t) for _, t, p0 in segs])
-        cols: list[list[int]] = [[], [], [], []]
+        total = sum(len(t) for _, t, _ in segs)
+        cols = np.empty((4, total), np.int32)           # tokens | positions | slots | offset in the portion
         seg_rows, tiles, at = [], [], 0
         latent = any(isinstance(L.mixer, LatentMixer) for L in self.stack.layers)
-        long_tiles, seqs, rest, total = [], [], [], 0
+        long_tiles, seqs, rest, keys = [], [], [], 0
         for slot, toks, p0 in segs:
             n = len(toks)
-            cols[0] += [max(int(t), 0) for t in toks]
-            cols[1] += range(p0, p0 + n)
-            cols[2] += [slot] * n
-            cols[3] += range(n)
+            cols[0, at:at + n] = toks
+            cols[1, at:at + n] = np.arange(p0, p0 + n)
+            cols[2, at:at + n] = slot
+            cols[3, at:at + n] = np.arange(n)
             seg_rows.append((at, n, slot, p0))
             tiles += [(at + r, min(128, n - r), slot, p0 + r) for r in range(0, n, 128)]
             if latent and n >= LONG_PORTION:
-                long_tiles += [(at + r, min(128, n - r), total, p0 + r) for r in range(0, n, 128)]
-                seqs.append((total, p0 + n, slot, 0))
-                total += p0 + n
+                long_tiles += [(at + r, min(128, n - r), keys, p0 + r) for r in range(0, n, 128)]
+                seqs.append((keys, p0 + n, slot, 0))
+                keys += p0 + n
             else:
                 rest += range(at, at + n)
             at += n
-        meta = torch.tensor(cols, dtype=torch.int32).to(dev)
+        np.maximum(cols[0], 0, out=cols[0])
+        meta = torch.from_numpy(cols).to(dev)
         geom = torch.tensor(seg_rows + tiles + long_tiles + seqs, dtype=torch.int32).to(dev)
         self.h2d_bytes += 4 * (meta.numel() + geom.numel())
         long, n1, n2 = None, len(segs) + len(tiles), len(segs) + len(tiles) + len(long_tiles)
         if seqs:
-            long = LongPortions(geom[n1:n2], geom[n2:], total, max(q[1] for q in seqs), torch.tensor(rest, dtype=torch.int32).to(dev) if rest else None)
+            long = LongPortions(geom[n1:n2], geom[n2:], keys, max(q[1] for q in seqs), torch.tensor(rest, dtype=torch.int32).to(dev) if rest else None)
             self.h2d_bytes += 4 * len(rest)
         m = _Meta(meta[0], meta[1], meta[2], meta[3], geom[:len(segs)], geom[len(segs):n1], long)
         self._n = 0

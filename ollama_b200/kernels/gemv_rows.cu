@@ -24,6 +24,8 @@ struct RowSeg {
     int act;             // out_act's number, or GLU_BASE + glu_act's: rows 2i / 2i + 1 are gate / up of output i
     int accumulate;
     float alpha, limit;  // factor of the result; limit of the clamped gated unit
+    const void* mul;     // result times mul[mul_row[b] * ldm + row] in the weights' type, after the activation; or null
+    int ldm;
 };
 
 enum RowSrc : int { SRC_ROWS = 0, SRC_NORM = 1, SRC_JOINED = 2 };
@@ -52,6 +54,7 @@ struct GemvRowsArgs {
     float* h;                     // [nb][ldh], k columns
     int ldh;
     const float* hb;              // [k] layer norm's bias
+    const int* mul_row;           // [nb]
 };
 
 namespace {
@@ -231,6 +234,10 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
     }
     if (mine) {
         v = out_act(v, w.act);
+        if (w.mul) {
+            const size_t m = (size_t)a.mul_row[b] * w.ldm + row;
+            v *= F32 ? ((const float*)w.mul)[m] : __bfloat162float(((const __nv_bfloat16*)w.mul)[m]);
+        }
         float* o = w.out + (size_t)b * w.ldo + row;
         *o = w.accumulate ? *o + w.alpha * v : w.alpha * v;
         if (s == a.conv_seg && row < a.conv_n) {
@@ -281,14 +288,15 @@ B2_API int b2_gemv_rows(const GemvRowsArgs* a, int pdl, cudaStream_t st) {
     for (int s = 0; s < a->nseg; s++) {
         const RowSeg& w = a->seg[s];
         if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (a->src == SRC_NORM && (!w.g || ((uintptr_t)w.g & 15) || (a->layer && !w.rs))) ||
-            w.act < 0 || (w.act > 2 && w.act < GLU_BASE) || w.act > GLU_BASE + 2 || (w.act >= GLU_BASE && (w.n & 1)))
+            w.act < 0 || (w.act > 2 && w.act < GLU_BASE) || w.act > GLU_BASE + 2 || (w.act >= GLU_BASE && ((w.n & 1) || w.mul)) || (w.mul && !a->mul_row))
             return (int)cudaErrorInvalidValue;
         groups += (w.n + R - 1) / R;
     }
-    // split the row length over KS warps until there are several row groups per resident warp, or a lane has two pieces left
-    const long want = a->nb <= 2 ? 16000 : 8000;
+    // Split the row length over KS warps until there are warps enough for the loads in flight, as far as a lane keeps two pieces; and long
+    // rows further, down to eight pieces a lane (sweep over 2048 .. 11008 columns and 2048 .. 32768 rows).
+    const long want = a->nb == 2 ? 3600 : 1800;
     int ks = 1;
-    while (ks < 8 && groups * ks < want && (a->k >> 3) / (32 * ks * 2) >= 1) ks <<= 1;
+    while (ks < 8 && ((groups * ks < want && (a->k >> 3) / (64 * ks) >= 1) || (a->k >> 3) / (64 * ks) >= 8)) ks <<= 1;
     const int rgs = 8 / ks;
     GemvRowsArgs copy = *a;
     void* args[] = {&copy};

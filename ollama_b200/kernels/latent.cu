@@ -69,28 +69,42 @@ struct LatentQueryArgs {
 
 namespace {
 
-// Value i of a rotated part of n values.
-__device__ __forceinline__ float rotated_at(const float* v, int i, int n, int pos, const double* freqs, int interleaved) {
-    const int half = n >> 1;
-    const bool first = interleaved ? !(i & 1) : i < half;
-    const int pair = interleaved ? i >> 1 : (first ? i : i - half);
-    const float other = v[interleaved ? i ^ 1 : (first ? i + half : i - half)];
-    float sn, cs;
-    sincosf(rot_angle(pos, freqs[pair]), &sn, &cs);
-    return first ? v[i] * cs - other * sn : v[i] * cs + other * sn;
-}
-
-// One warp: cache row of step row r.
+// One CTA: cache row of step row r and, with q set, the rotated parts of its queries (rows of w values, cp behind their start) and the zeros
+// behind them.  `cs` holds rot floats.
 template <typename CT>
-__device__ __forceinline__ void append_row(const LatentStepArgs& a, int r, int lane) {
-    const int pos = a.positions[r], slot = a.slots[r];
-    const float* c = a.qkv + (size_t)r * a.ldq + (size_t)a.n_heads * (a.dim + a.rot);
+__device__ __forceinline__ void append_row(const LatentStepArgs& a, int r, CT* q, float* cs, float* red) {
+    const int tid = threadIdx.x, nt = blockDim.x, pos = a.positions[r], slot = a.slots[r], half = a.rot >> 1, pad = a.w - a.cp;
+    const float* row = a.qkv + (size_t)r * a.ldq;
+    const float* c = row + (size_t)a.n_heads * (a.dim + a.rot);
     float ss = 0.f;
-    for (int i = lane; i < a.rank; i += 32) ss += c[i] * c[i];
-    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)a.rank + a.eps);
-    CT* o = (CT*)a.cache + paged_row(a.page_table + (size_t)slot * a.max_pages, pos, 1, 0) * a.w;
-    for (int i = lane; i < a.cp; i += 32) o[i] = from_f<CT>(i < a.rank ? c[i] * inv * a.norm[i] : 0.f);
-    for (int i = lane; i < a.w - a.cp; i += 32) o[a.cp + i] = from_f<CT>(i < a.rot ? rotated_at(c + a.rank, i, a.rot, pos, a.freqs, a.interleaved) : 0.f);
+#pragma unroll 4
+    for (int i = tid; i < a.rank; i += nt) ss += c[i] * c[i];
+    ss = warp_sum(ss);
+    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    for (int i = tid; i < half; i += nt) sincosf(rot_angle(pos, a.freqs[i]), &cs[half + i], &cs[i]);
+    __syncthreads();
+    ss = 0.f;
+    for (int i = 0; i < nt >> 5; i++) ss += red[i];
+    const float inv = 1.f / sqrtf(ss / (float)a.rank + a.eps);
+    auto rotated = [&](const float* v, int i) {
+        const bool first = a.interleaved ? !(i & 1) : i < half;
+        const int p = a.interleaved ? i >> 1 : (first ? i : i - half);
+        const float other = v[a.interleaved ? i ^ 1 : (first ? i + half : i - half)];
+        return first ? v[i] * cs[p] - other * cs[half + p] : v[i] * cs[p] + other * cs[half + p];
+    };
+    if (a.append) {
+        CT* o = (CT*)a.cache + paged_row(a.page_table + (size_t)slot * a.max_pages, pos, 1, 0) * a.w;
+#pragma unroll 4
+        for (int i = tid; i < a.cp; i += nt) o[i] = from_f<CT>(i < a.rank ? c[i] * inv * a.norm[i] : 0.f);
+        for (int i = tid; i < pad; i += nt) o[a.cp + i] = from_f<CT>(i < a.rot ? rotated(c + a.rank, i) : 0.f);
+    }
+    if (q) {
+#pragma unroll 4
+        for (int j = tid; j < a.n_heads * pad; j += nt) {
+            const int h = j / pad, i = j - h * pad;
+            q[(size_t)h * a.w + a.cp + i] = from_f<CT>(i < a.rot ? rotated(row + (size_t)h * (a.dim + a.rot) + a.dim, i) : 0.f);
+        }
+    }
 }
 
 template <typename WT>
@@ -114,38 +128,29 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
 constexpr int COLS = 128;      // latent columns of a CTA of latent_step
 constexpr int DG = 16;         // groups of d values, one partial sum each
 
-// grid (heads * column parts + 1, row groups of NB): the last CTA of a row group appends, the others form U^T q
+// grid (heads * column parts + NB, row groups of NB): the last NB CTAs of a row group do what belongs to a row, the others form U^T q
 template <typename CT, typename WT, int NB>
 __global__ void __launch_bounds__(256) latent_step_kernel(const __grid_constant__ LatentStepArgs a, int n) {
-    extern __shared__ float sq[];                  // [NB][dim]
+    extern __shared__ float sq[];                  // [NB][dim], or the rotation's cosines and sines
     __shared__ float red[DG][COLS + 4];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, i0 = blockIdx.y * NB;
     const int parts = (a.cp + COLS - 1) / COLS;
     const int h = blockIdx.x / parts, part = blockIdx.x % parts;
-    const bool appends = blockIdx.x == gridDim.x - 1;
+    const int rb = (int)blockIdx.x - a.n_heads * parts;            // >= 0: row of the group
     const int cg = tid & 15, dg = tid >> 4, col = part * COLS + 8 * cg;
     const WT* u = (const WT*)a.uk + ((size_t)h * a.dim) * a.cp + col;
     pdl_launch();
-    if (!appends && col < a.cp && (cg & 7) == 0)
+    if (rb < 0 && col < a.cp && (cg & 7) == 0)
         for (int d = dg; d < a.dim; d += DG) asm volatile("prefetch.global.L2 [%0];" ::"l"(u + (size_t)d * a.cp));
     pdl_wait();
-    if (appends) {
-        if (a.append)
-            for (int b = warp; b < NB && i0 + b < n; b += 8) append_row<CT>(a, a.rows ? a.rows[i0 + b] : i0 + b, lane);
+    if (rb >= 0) {
+        if (i0 + rb < n) append_row<CT>(a, a.rows ? a.rows[i0 + rb] : i0 + rb, (CT*)a.q_out + (size_t)(i0 + rb) * a.n_heads * a.w, sq, &red[0][0]);
         return;
     }
     const int nb = min(NB, n - i0), dq = a.dim + a.rot;
     for (int j = tid; j < nb * a.dim; j += 256) {
         const int b = j / a.dim, d = j - b * a.dim, r = a.rows ? a.rows[i0 + b] : i0 + b;
         sq[b * a.dim + d] = a.qkv[(size_t)r * a.ldq + (size_t)h * dq + d];
-    }
-    if (part == 0) {                               // the rotated part and the zeros behind it
-        const int m = a.w - a.cp;
-        for (int j = tid; j < nb * m; j += 256) {
-            const int b = j / m, i = j - b * m, r = a.rows ? a.rows[i0 + b] : i0 + b;
-            const float* q = a.qkv + (size_t)r * a.ldq + (size_t)h * dq + a.dim;
-            ((CT*)a.q_out)[((size_t)(i0 + b) * a.n_heads + h) * a.w + a.cp + i] = from_f<CT>(i < a.rot ? rotated_at(q, i, a.rot, a.positions[r], a.freqs, a.interleaved) : 0.f);
-        }
     }
     __syncthreads();
     float acc[NB][8];
@@ -184,78 +189,167 @@ __global__ void __launch_bounds__(256) latent_step_kernel(const __grid_constant_
 }
 
 template <typename CT>
-__global__ void __launch_bounds__(128) latent_append_kernel(const __grid_constant__ LatentStepArgs a, int n) {
-    const int i = blockIdx.x * 4 + (threadIdx.x >> 5);
+__global__ void __launch_bounds__(128) latent_append_kernel(const __grid_constant__ LatentStepArgs a) {
+    extern __shared__ float sq[];
+    __shared__ float red[4];
     pdl_launch();
     pdl_wait();
-    if (i < n) append_row<CT>(a, a.rows ? a.rows[i] : i, threadIdx.x & 31);
+    append_row<CT>(a, a.rows ? a.rows[blockIdx.x] : blockIdx.x, nullptr, sq, red);
 }
 
-constexpr int MAX_SPLITS = 128, VROWS = 32;
+constexpr int MAX_SPLITS = 128;
 
-// grid (heads, value parts of VROWS, row groups of NB); a warp multiplies four value rows
-template <typename WT, int NB>
+// grid (heads, value parts of 8 VR, row groups of NB); a warp multiplies VR value rows.  The chain is latency: the value rows, which do not depend
+// on the producer kernel, are in registers before the wait (rows of up to 512 16-bit values), and the split sums are requested
+// together with their statistics.
+template <typename WT, int NB, int VR>
 __global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant__ LatentMergeArgs a, int n) {
+    constexpr bool PRE = sizeof(WT) == 2 && NB == 1;
+    constexpr int BATCH = 8;
     extern __shared__ __align__(16) float so[];    // [NB][cp]
+    __shared__ __align__(16) float half[PRE ? 512 : 4];
     __shared__ float sw[NB][MAX_SPLITS];
+    __shared__ int s_n[NB];                        // splits with keys: the first ones
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, i0 = blockIdx.z * NB, nb = min(NB, n - i0);
-    const int v0 = blockIdx.y * VROWS + warp * (VROWS / 8);
+    const int v0 = (blockIdx.y * 8 + warp) * VR;
+    const WT* uv = (const WT*)a.uv + ((size_t)h * a.vdim + v0) * a.cp;
+    const bool pre = PRE && a.cp <= 512;
+    uint4 wv[PRE ? VR : 1][2];
     pdl_launch();
-    for (int j = 0; j < VROWS / 8; j++)
-        if (v0 + j < a.vdim)
-            for (int c = lane * (128 / (int)sizeof(WT)); c < a.cp; c += 32 * (128 / (int)sizeof(WT)))
-                asm volatile("prefetch.global.L2 [%0];" ::"l"((const WT*)a.uv + ((size_t)h * a.vdim + v0 + j) * a.cp + c));
-    pdl_wait();
-    if (a.ml) {
-        if (warp < nb) {
-            const float2* ml = a.ml + ((size_t)(i0 + warp) * a.n_heads + h) * a.splits;
-            float m = -INFINITY, l = 0.f;
-            for (int s = lane; s < a.splits; s += 32)
-                if (ml[s].y > 0.f) m = fmaxf(m, ml[s].x);
-            m = warp_max(m);
-            for (int s = lane; s < a.splits; s += 32) {
-                const float w = ml[s].y > 0.f ? expf(ml[s].x - m) : 0.f;
-                sw[warp][s] = w;
-                l += w * ml[s].y;
+    if (pre) {
+#pragma unroll
+        for (int j = 0; j < VR; j++)
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const int c = 8 * lane + 256 * u;
+                wv[PRE ? j : 0][u] = v0 + j < a.vdim && c < a.cp ? ldg16(uv + (size_t)j * a.cp + c) : make_uint4(0, 0, 0, 0);
             }
-            l = warp_sum(l);
-            __syncwarp();
-            for (int s = lane; s < a.splits; s += 32) sw[warp][s] /= l;
+    } else {
+        for (int j = 0; j < VR; j++)
+            if (v0 + j < a.vdim)
+                for (int c = lane * (128 / (int)sizeof(WT)); c < a.cp; c += 32 * (128 / (int)sizeof(WT)))
+                    asm volatile("prefetch.global.L2 [%0];" ::"l"(uv + (size_t)j * a.cp + c));
+    }
+    pdl_wait();
+    const int q4 = a.cp >> 2;                      // float4 columns
+    if (a.ml && NB == 1 && q4 <= 128) {            // the two halves of the CTA take every other split
+        const float* p = a.acc + ((size_t)i0 * a.n_heads + h) * a.splits * a.cp;
+        const float2* ml = a.ml + ((size_t)i0 * a.n_heads + h) * a.splits;
+        const int col = tid & 127, part = tid >> 7;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        float m = -1e30f, l = 0.f;
+        for (int s0 = part; s0 < a.splits; s0 += 2 * BATCH) {
+            float2 st[BATCH];
+            float4 v[BATCH];
+#pragma unroll
+            for (int i = 0; i < BATCH; i++) {
+                const int s = s0 + 2 * i;
+                st[i] = s < a.splits ? ml[s] : make_float2(-1e30f, 0.f);
+                v[i] = s < a.splits && col < q4 ? *(const float4*)(p + (size_t)s * a.cp + 4 * col) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+            float mn = m;
+#pragma unroll
+            for (int i = 0; i < BATCH; i++) mn = st[i].y > 0.f ? fmaxf(mn, st[i].x) : mn;
+            const float c = expf(m - mn);
+            o.x *= c; o.y *= c; o.z *= c; o.w *= c;
+            l *= c;
+            m = mn;
+#pragma unroll
+            for (int i = 0; i < BATCH; i++) {
+                if (!(st[i].y > 0.f)) continue;    // splits without keys leave their sums unwritten
+                const float w = expf(st[i].x - mn);
+                l += w * st[i].y;
+                o.x += w * v[i].x; o.y += w * v[i].y; o.z += w * v[i].z; o.w += w * v[i].w;
+            }
+        }
+        float* stats = &sw[0][0];                  // (max, sum) of the second half
+        if (part == 1 && col < q4) *(float4*)(PRE ? half + 4 * col : so + 4 * col) = o;
+        if (tid == 128) {
+            stats[0] = m;
+            stats[1] = l;
         }
         __syncthreads();
-    }
-    for (int j = tid; j < nb * (a.cp >> 2); j += 256) {
-        const int b = j / (a.cp >> 2), c = 4 * (j - b * (a.cp >> 2));
-        const float* p = a.acc + ((size_t)(i0 + b) * a.n_heads + h) * a.splits * a.cp + c;
-        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (a.ml) {
-            for (int s = 0; s < a.splits; s++) {
-                const float w = sw[b][s];
-                if (w == 0.f) continue;            // splits without keys leave their sums unwritten
-                const float4 v = *(const float4*)(p + (size_t)s * a.cp);
-                o.x += w * v.x; o.y += w * v.y; o.z += w * v.z; o.w += w * v.w;
-            }
-        } else {
-            o = *(const float4*)p;
+        if (part == 0 && col < q4) {
+            const float4 o1 = *(const float4*)(PRE ? half + 4 * col : so + 4 * col);
+            const float mn = fmaxf(m, stats[0]), c0 = expf(m - mn), c1 = expf(stats[0] - mn), inv = 1.f / (c0 * l + c1 * stats[1]);
+            *(float4*)(so + 4 * col) = make_float4((c0 * o.x + c1 * o1.x) * inv, (c0 * o.y + c1 * o1.y) * inv, (c0 * o.z + c1 * o1.z) * inv, (c0 * o.w + c1 * o1.w) * inv);
         }
-        *(float4*)(so + b * a.cp + c) = o;
+    } else {
+        if (a.ml) {
+            if (warp < nb) {
+                const float2* ml = a.ml + ((size_t)(i0 + warp) * a.n_heads + h) * a.splits;
+                float m = -INFINITY, l = 0.f;
+                int used = 0;
+                for (int s = lane; s < a.splits; s += 32)
+                    if (ml[s].y > 0.f) m = fmaxf(m, ml[s].x);
+                m = warp_max(m);
+                for (int s = lane; s < a.splits; s += 32) {
+                    const float w = ml[s].y > 0.f ? expf(ml[s].x - m) : 0.f;
+                    sw[warp][s] = w;
+                    l += w * ml[s].y;
+                    if (ml[s].y > 0.f) used = s + 1;
+                }
+                l = warp_sum(l);
+                used = __reduce_max_sync(0xffffffffu, used);
+                if (lane == 0) s_n[warp] = used;
+                __syncwarp();
+                for (int s = lane; s < a.splits; s += 32) sw[warp][s] /= l;
+            }
+            __syncthreads();
+        }
+        for (int j = tid; j < nb * q4; j += 256) {
+            const int b = j / q4, c = 4 * (j - b * q4);
+            const float* p = a.acc + ((size_t)(i0 + b) * a.n_heads + h) * a.splits * a.cp + c;
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (a.ml) {
+                const int used = s_n[b];
+#pragma unroll 8
+                for (int s = 0; s < used; s++) {
+                    const float w = sw[b][s];
+                    const float4 v = *(const float4*)(p + (size_t)s * a.cp);
+                    o.x += w * v.x; o.y += w * v.y; o.z += w * v.z; o.w += w * v.w;
+                }
+            } else {
+                o = *(const float4*)p;
+            }
+            *(float4*)(so + b * a.cp + c) = o;
+        }
     }
     __syncthreads();
-    for (int j = 0; j < VROWS / 8; j++) {
+#pragma unroll
+    for (int j = 0; j < VR; j++) {
         const int v = v0 + j;
         if (v >= a.vdim) return;
-        const WT* w = (const WT*)a.uv + ((size_t)h * a.vdim + v) * a.cp;
         float acc[NB];
 #pragma unroll
         for (int b = 0; b < NB; b++) acc[b] = 0.f;
-        for (int c = 8 * lane; c < a.cp; c += 256) {
-            float f[8];
-            load8<WT>(w + c, f);
+        auto add = [&](const float (&f)[8], int c) {
 #pragma unroll
             for (int b = 0; b < NB; b++) {
                 if (b >= nb) break;
+                const float4 x = *(const float4*)(so + b * a.cp + c), y = *(const float4*)(so + b * a.cp + c + 4);
+                acc[b] += f[0] * x.x + f[1] * x.y + f[2] * x.z + f[3] * x.w + f[4] * y.x + f[5] * y.y + f[6] * y.z + f[7] * y.w;
+            }
+        };
+        if (pre) {
 #pragma unroll
-                for (int e = 0; e < 8; e++) acc[b] = fmaf(f[e], so[b * a.cp + c + e], acc[b]);
+            for (int u = 0; u < 2; u++) {
+                const int c = 8 * lane + 256 * u;
+                const uint4 w = wv[PRE ? j : 0][u];
+                const uint32_t q[4] = {w.x, w.y, w.z, w.w};
+                float f[8];
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    f[2 * i] = __uint_as_float(q[i] << 16);
+                    f[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
+                }
+                if (c < a.cp) add(f, c);
+            }
+        } else {
+            for (int c = 8 * lane; c < a.cp; c += 256) {
+                float f[8];
+                load8<WT>(uv + (size_t)j * a.cp + c, f);
+                add(f, c);
             }
         }
 #pragma unroll
@@ -336,28 +430,31 @@ B2_API int b2_latent_step(const LatentStepArgs* a, int n, int pdl, cudaStream_t 
         return (int)cudaErrorInvalidValue;
     LatentStepArgs c = *a;
     void* args[] = {&c, &n};
+    const size_t angles = (size_t)a->rot * 4;
+    if (angles > 32 * 1024) return (int)cudaErrorNotSupported;
     if (!a->uk)
-        return launch_rows(a->cache32 ? (const void*)latent_append_kernel<float> : (const void*)latent_append_kernel<__half>, dim3((n + 3) / 4), dim3(128), 0, args, st, pdl);
+        return launch_rows(a->cache32 ? (const void*)latent_append_kernel<float> : (const void*)latent_append_kernel<__half>, dim3(n), dim3(128), angles, args, st, pdl);
     const int nb = n == 1 ? 1 : 4, parts = (a->cp + COLS - 1) / COLS;
     const void* fn = a->cache32 ? (a->w32 ? step_fn<float, float>(nb) : step_fn<float, __nv_bfloat16>(nb)) : (a->w32 ? step_fn<__half, float>(nb) : step_fn<__half, __nv_bfloat16>(nb));
-    const size_t smem = (size_t)nb * a->dim * 4;
+    const size_t rows = (size_t)nb * a->dim * 4, smem = rows > angles ? rows : angles;
     if (smem > 32 * 1024) return (int)cudaErrorNotSupported;
     if ((n + nb - 1) / nb > 65535) return (int)cudaErrorInvalidValue;
-    return launch_rows(fn, dim3(a->n_heads * parts + 1, (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
+    return launch_rows(fn, dim3(a->n_heads * parts + nb, (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
 }
 
 B2_API int b2_latent_merge(const LatentMergeArgs* a, int n, int pdl, cudaStream_t st) {
     if (n < 1 || a->n_heads < 1 || a->splits < 1 || a->splits > MAX_SPLITS || (!a->ml && a->splits != 1) || (a->cp & 15) || a->vdim < 1 || ((uintptr_t)a->uv & 15) || ((uintptr_t)a->acc & 15))
         return (int)cudaErrorInvalidValue;
-    const int nb = n == 1 ? 1 : 4;
+    const int nb = n <= 32 ? 1 : 4;                // a decode step: latency counts, the value rows come from L2 for every row
     const size_t smem = (size_t)nb * a->cp * 4;
     if (smem > 40 * 1024) return (int)cudaErrorNotSupported;
     if ((n + nb - 1) / nb > 65535) return (int)cudaErrorInvalidValue;
     LatentMergeArgs c = *a;
     void* args[] = {&c, &n};
-    const void* fn = a->w32 ? (nb == 1 ? (const void*)latent_merge_kernel<float, 1> : (const void*)latent_merge_kernel<float, 4>)
-                            : (nb == 1 ? (const void*)latent_merge_kernel<__nv_bfloat16, 1> : (const void*)latent_merge_kernel<__nv_bfloat16, 4>);
-    return launch_rows(fn, dim3(a->n_heads, (a->vdim + VROWS - 1) / VROWS, (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
+    const int vr = nb == 1 ? 4 : 8;
+    const void* fn = a->w32 ? (nb == 1 ? (const void*)latent_merge_kernel<float, 1, 4> : (const void*)latent_merge_kernel<float, 4, 8>)
+                            : (nb == 1 ? (const void*)latent_merge_kernel<__nv_bfloat16, 1, 4> : (const void*)latent_merge_kernel<__nv_bfloat16, 4, 8>);
+    return launch_rows(fn, dim3(a->n_heads, (a->vdim + 8 * vr - 1) / (8 * vr), (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
 }
 
 B2_API int b2_latent_gather(const LatentGatherArgs* a, int n_seqs, int max_len, cudaStream_t st) {

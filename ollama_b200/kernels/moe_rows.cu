@@ -250,10 +250,10 @@ __global__ void __launch_bounds__(256) moe_down_rows_kernel(const __grid_constan
     }
 }
 
-// Warps that share a row group: until there are several groups per resident warp, or a lane has two pieces left.
-int split_of(long groups, int pieces) {
+// Warps that share a row group: until `want` warps carry loads, as far as a lane keeps two pieces.
+int split_of(long groups, int pieces, long want) {
     int ks = 1;
-    while (ks < 8 && groups * ks < 16000 && pieces / (64 * ks) >= 1) ks <<= 1;
+    while (ks < 8 && groups * ks < want && pieces / (64 * ks) >= 1) ks <<= 1;
     return ks;
 }
 
@@ -270,7 +270,7 @@ B2_API int b2_moe_up_rows(const MoeUpArgs* a, int nb, int f32, int pdl, cudaStre
         ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15))
         return (int)cudaErrorInvalidValue;
     const long groups = (long)a->top * ((a->n + R - 1) / R) + (a->ns + R - 1) / R;
-    const int ks = split_of(groups * nb, a->k >> 3), rgs = 8 / ks;
+    const int ks = split_of(groups * nb, a->k >> 3, 1800), rgs = 8 / ks;
     MoeUpArgs c = *a;
     void* args[] = {&c};
     return launch_rows(B2_PICK_KS(moe_up_rows_kernel, f32, ks), dim3((unsigned)((groups + rgs - 1) / rgs), nb), dim3(256), 0, args, st, pdl);
@@ -281,7 +281,7 @@ B2_API int b2_moe_down_rows(const MoeDownArgs* a, int nb, int f32, int pdl, cuda
         a->lda < a->top * a->ffp + a->sfp || ((uintptr_t)a->a & 15) || ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15))
         return (int)cudaErrorInvalidValue;
     const long groups = (a->n + R - 1) / R;
-    const int ks = split_of(groups * nb, (a->top * a->ffp + a->sfp) >> 3), rgs = 8 / ks;
+    const int ks = split_of(groups * nb, (a->top * a->ffp + a->sfp) >> 3, 16000), rgs = 8 / ks;
     MoeDownArgs c = *a;
     void* args[] = {&c};
     return launch_rows(B2_PICK_KS(moe_down_rows_kernel, f32, ks), dim3((unsigned)((groups + rgs - 1) / rgs), nb), dim3(256), 0, args, st, pdl);

@@ -54,6 +54,8 @@ SPECS: dict[str, ArchSpec] = {
     # dense models of the size of the stack models below, layer run by layer run (a gated FFN has three matrices for their two)
     "dense-1b": ArchSpec("llama", 20, 2048, 16, 4, 128, 5504, 32768, 500000.0),
     "dense-8b": ArchSpec("llama", 32, 4096, 32, 8, 128, 11008, 128256, 500000.0),
+    # a mixture-of-experts model of the size of kavenex-moe (whose shared expert counts as one more chosen expert)
+    "experts-2k": ArchSpec("qwen3moe", 20, 2048, 16, 4, 128, 5504, 32768, 500000.0, 1e-6, n_experts=64, n_experts_used=5, d_ff_expert=1408),
     # small stand-ins of every family for tests
     "tiny-tp": ArchSpec("llama", 2, 1024, 16, 8, 64, 4096, 4096, 500000.0, 1e-5, 4096),      # divides 2, 4 and 8 ways
     "tiny-qwen3": ArchSpec("qwen3", 2, 256, 4, 2, 64, 768, 4096, 1e6, 1e-6, 4096),
@@ -290,7 +292,24 @@ def stack_config(width: int, heads: int, kv_heads: int, dim: int, ff: int, inner
             "layers": [{**(att if c == "A" else mam), "mlp": {"kind": "dense", "ff": ff}} for c in layers]}
 
 
+def latent_config(width: int, heads: int, dim: int, rot: int, vdim: int, rank: int, ff: int, vocab: int, layers: str, loop: tuple[int, int, int] | None, side: int,
+                  experts: int = 0, top: int = 0, ff_expert: int = 0, ff_shared: int = 0) -> dict:
+    """``config.json`` of a Kavenex model; ``layers``: one letter per layer, D (dense feed-forward), E (experts) or N (none)."""
+    mix = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": (dim + rot) ** -0.5, "rot": {"base": 500000.0, "dims": rot}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff_expert, "limit": 7.0}}
+    if ff_shared:
+        moe["shared"] = {"ff": ff_shared, "limit": 7.0}
+    mlp = {"D": {"kind": "dense", "ff": ff}, "E": moe, "N": None}
+    return {"architecture": "Kavenex", "embedding": {"scale": math.sqrt(width)}, "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "token_side": {"dim": side} if side else None, "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]} if loop else None,
+            "layers": [{"type": "latent_attention", "mixer": mix, "mlp": mlp[c]} for c in layers]}
+
+
 STACK_SPECS: dict[str, dict] = {
+    "tiny-kavenex": latent_config(256, 4, 64, 32, 64, 128, 512, 4096, "DED", (0, 2, 2), 32, 8, 2, 128, 128),
+    "kavenex-1b": latent_config(2048, 16, 128, 64, 128, 512, 5504, 32768, "D" * 16, (0, 4, 2), 256),
+    "kavenex-8b": latent_config(4096, 32, 128, 64, 128, 512, 11008, 128256, "D" * 28, (0, 4, 2), 256),
+    "kavenex-moe": latent_config(2048, 16, 128, 64, 128, 512, 0, 32768, "E" * 16, (0, 4, 2), 256, 64, 4, 1408, 1408),
     "tiny-vazatar": stack_config(256, 4, 2, 64, 512, 512, 16, 16, 4096, "AMA", (0, 2, 2), 128),
     "vazatar-1b": stack_config(2048, 16, 4, 128, 8192, 4096, 16, 128, 32768, "AAMA" * 4, (0, 4, 2), 2048),
     "vazatar-8b": stack_config(4096, 32, 8, 128, 16384, 8192, 16, 256, 128256, "AAMA" * 7, (0, 4, 2), 8192),
@@ -304,21 +323,43 @@ class SyntheticStackTensors:
         from ..convert.stack import map_stack_name
         self.seed, self.device, w = seed, device, cfg["width"]
         names: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], w), "head": (cfg["vocab"], w), "final.norm": (w,)}
+        seq = cfg["architecture"] == "Kavenex"       # mixer and feed-forward one after the other, layer norms, gated feed-forwards
         if cfg.get("loop"):
-            names["loop.in"] = (w, 2 * w)
+            names.update({"loop.step": (cfg["loop"]["times"], w)} if seq else {"loop.in": (w, 2 * w)})
+        side = (cfg.get("token_side") or {}).get("dim")
+        if side:
+            names["side.embed"] = (cfg["vocab"], len(cfg["layers"]) * side)
+        stacked: dict[str, tuple[int, ...]] = {}
         for i, L in enumerate(cfg["layers"]):
             m, p = L["mixer"], f"l{i}."
             names[p + "norm1"] = (w,)
-            if L["type"] == "attention":
+            if L["type"] == "latent_attention":
+                H, d, r, dv, k = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+                names.update({p + "mix.q": (H * (d + r), w), p + "mix.dkv": (k + r, w), p + "mix.dkv.norm": (k,), p + "mix.uk": (H * d, k), p + "mix.uv": (H * dv, k),
+                              p + "mix.o": (w, H * dv)})
+            elif L["type"] == "attention":
                 nq, nk, nv, no = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
                 names.update({p + "mix.q": (nq, w), p + "mix.k": (nk, w), p + "mix.v": (nv, w), p + "mix.q.norm": (nq,), p + "mix.k.norm": (nk,), p + "mix.o": (w, no)})
             else:
                 c, n, r = m["inner"], m["state"], m["dt_rank"]
                 names.update({p + "mix.in": (2 * c, w), p + "mix.conv": (c, m["conv"]), p + "mix.conv.b": (c,), p + "mix.x": (r + 2 * n, c), p + "mix.dt": (c, r),
                               p + "mix.dt.b": (c,), p + "mix.A_log": (c, n), p + "mix.D": (c,), p + "mix.o": (w, c)})
-            if L.get("mlp"):
-                names.update({p + "norm2": (w,), p + "mlp.up": (L["mlp"]["ff"], w), p + "mlp.down": (w, L["mlp"]["ff"])})
-        self.table = {map_stack_name(n, cfg): s for n, s in names.items()}
+            f = L.get("mlp")
+            if f:
+                names[p + "norm2"] = (w,)
+            if f and f["kind"] == "dense":
+                names.update({p + "mlp.up": (f["ff"], w), p + "mlp.down": (w, f["ff"]), **({p + "mlp.gate": (f["ff"], w)} if seq else {})})
+            elif f:
+                E, fe, fs = f["router"]["experts"], f["expert"]["ff"], (f.get("shared") or {}).get("ff")
+                names.update({p + "mlp.router": (E, w), p + "mlp.router.b": (E,)})
+                for pre, fx in ((f"blk.{i}.ffn_%s_exps.weight", (E, fe)), (f"blk.{i}.ffn_%s_shexp.weight", (fs,))):
+                    if fx[-1]:
+                        stacked.update({pre % "gate": (*fx, w), pre % "up": (*fx, w), pre % "down": (*fx[:-1], w, fx[-1])})
+            if side:
+                names.update({p + "side.gate": (side, w), p + "side.proj": (w, side), p + "side.norm": (w,)})
+        if seq:
+            names.update({n + ".b": s for n, s in names.items() if n.endswith(("norm1", "norm2", "final.norm"))})
+        self.table = {**{map_stack_name(n, cfg): s for n, s in names.items()}, **stacked}
 
     def __contains__(self, name: str) -> bool:
         return name in self.table

@@ -1,5 +1,4 @@
-"""Bindings of latent attention, expert feed-forwards of decode rows and per-token layer inputs (kernels/latent.cu, attn_latent.cu,
-attn_prefill_tc.cu, moe_rows.cu, side_rows.cu)."""
+"""Bindings of latent attention and of expert feed-forwards (kernels/latent.cu, attn_latent.cu, attn_prefill_tc.cu, moe.cu, moe_rows.cu)."""
 from __future__ import annotations
 
 import ctypes as C
@@ -26,8 +25,6 @@ MoeUpArgs = _st("MoeUpArgs", [("z", P), ("ldz", I), ("n_experts", I), ("top", I)
                               ("ns", I), ("limit", F), ("limit_s", F), ("out", P), ("ldo", I), ("ffp", I), ("ids", P), ("wts", P)])
 MoeDownArgs = _st("MoeDownArgs", [("a", P), ("lda", I), ("top", I), ("ffp", I), ("sfp", I), ("ids", P), ("wts", P), ("w", P), ("ws", P), ("n", I), ("wrows", I),
                                   ("x", P), ("ldx", I), ("mult", F)])
-SideRowsArgs = _st("SideRowsArgs", [("x", P), ("ldx", I), ("width", I), ("k", I), ("gate", P), ("e", P), ("lde", I), ("dim", I), ("dimp", I), ("tokens", P),
-                                    ("proj", P), ("w", P), ("eps", F), ("mult", F), ("x0", P), ("step", P)])
 
 NOT_SUPPORTED = 801                # cudaErrorNotSupported: the launch does not take the shape, nothing ran
 
@@ -110,11 +107,3 @@ def moe_down_rows(a_rows: torch.Tensor, nb: int, ids, wts, w: torch.Tensor, x: t
     a = MoeDownArgs(ptr(a_rows), a_rows.stride(0), top, w.shape[2], ws.shape[1] if ws is not None else 0, ptr(ids), ptr(wts), ptr(w), ptr(ws), n, w.shape[1], ptr(x),
                     x.stride(0), mult)
     _call("b2_moe_down_rows", a, nb, _is32(w), int(pdl))
-
-
-def side_rows(x: torch.Tensor, nb: int, width: int, gate: torch.Tensor, e: torch.Tensor, dim: int, tokens, proj: torch.Tensor, w, eps: float, mult: float, x0=None,
-              step=None, cluster: int = 8, pdl: bool = False) -> bool:
-    """x += mult * rmsnorm(proj (gelu(gate x) * e[token])) * w [+ x0] [+ step] for up to four rows; False: shape not taken, nothing launched."""
-    a = SideRowsArgs(ptr(x), x.stride(0), width, gate.shape[1], ptr(gate), ptr(e), e.stride(0), dim, proj.shape[1], ptr(tokens), ptr(proj), ptr(w), eps, mult, ptr(x0),
-                     ptr(step))
-    return _taken("b2_side_rows", a, nb, _is32(gate), cluster, int(pdl))

@@ -26,14 +26,14 @@ NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), 
                                     ("b1", P), ("b2", P), ("y", P), ("wy", P), ("x0", P), ("step", P), ("ldy", I), ("mult", F)])
 JoinRowsArgs = _st("JoinRowsArgs", [("a", P), ("b", P), ("lda", I), ("n_a", I), ("ldb", I), ("n_b", I), ("out", P), ("ldo", I), ("off_b", I), ("f32", I)])
 RowSeg = _st("RowSeg", [("w", P), ("g", P), ("rs", P), ("rc", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I), ("alpha", F),
-                        ("limit", F)])
+                        ("limit", F), ("mul", P), ("ldm", I)])
 GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P), ("mul", P), ("mul_row", P), ("tile_expert", P), ("ws", P),
                                     ("ws_floats", C.c_longlong), ("m", I), ("n", I), ("k", I), ("lda", I), ("ldb", I), ("ldo", I), ("out_type", I), ("act", I),
                                     ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
                                     ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
                                     ("conv_b", P), ("conv_state", P), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
-                                    ("layer", I), ("h", P), ("ldh", I), ("hb", P)])
+                                    ("layer", I), ("h", P), ("ldh", I), ("hb", P), ("mul_row", P)])
 PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
                                           ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
                                           ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I)])
@@ -79,17 +79,19 @@ def join_rows(a: torch.Tensor, n_a: int, out: torch.Tensor, b: torch.Tensor | No
 
 
 def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = None, act: str = "", accumulate: bool = False, alpha: float = 1.0,
-        limit: float = math.inf, rs: torch.Tensor | None = None, rc: torch.Tensor | None = None) -> RowSeg:
-    """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``, as out (+)= alpha * act(... + rc).  ``rs``: the rows' sums of
+        limit: float = math.inf, rs: torch.Tensor | None = None, rc: torch.Tensor | None = None, mul: torch.Tensor | None = None) -> RowSeg:
+    """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``, as out (+)= alpha * act(... + rc) [* mul[mul_row]].  ``rs``: the rows' sums of
     w * g (layer norm).  Gated activations ("glu:...") take rows 2i and 2i + 1 as gate and up of column i."""
-    s = RowSeg(ptr(w), ptr(g), ptr(rs), ptr(rc), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate), alpha, limit)
-    s.keep = (w, g, rs, rc, out)     # the structure holds addresses only
+    s = RowSeg(ptr(w), ptr(g), ptr(rs), ptr(rc), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate), alpha, limit, ptr(mul),
+               mul.stride(0) if mul is not None else 0)
+    s.keep = (w, g, rs, rc, out, mul)     # the structure holds addresses only
     return s
 
 
 def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,
          k1: int = 0, conv=None, conv_out: torch.Tensor | None = None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None,
-         layer: bool = False, h: torch.Tensor | None = None, hb: torch.Tensor | None = None, pdl: bool = False) -> None:
+         layer: bool = False, h: torch.Tensor | None = None, hb: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
+         pdl: bool = False) -> None:
     """Products of up to four matrices with up to four source rows.  ``conv`` = (weights [taps, n], bias [n], state [slots, taps - 1, n]): the first n
     results of the first matrix also run through that convolution and SiLU, into ``conv_out``.  ``layer``: the norm source is a layer norm;
     ``h``: its rows for the first matrix are stored too (``hb``: the norm's bias)."""
@@ -97,7 +99,7 @@ def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC
     for i, s in enumerate(segs):
         a.seg[i] = s
     a.nseg, a.nb, a.k, a.src, a.f32, a.x, a.ldx, a.eps, a.kn, a.conv_seg = len(segs), nb, k, src, int(f32), ptr(x), x.stride(0), eps, kn, -1
-    a.layer = int(layer)
+    a.layer, a.mul_row = int(layer), ptr(mul_row)
     if h is not None:
         a.h, a.ldh, a.hb = ptr(h), h.stride(0), ptr(hb)
     if x2 is not None:

@@ -17,6 +17,7 @@ from ..ops import rows as O
 
 LONG_PORTION = 64                # prompt portions of this many tokens multiply keys and values out; shorter ones stay in the latent space
 MAX_SPLITS = 128
+MERGE_ROWS = 6                   # more rows than this merge their splits and multiply the values in two launches
 
 
 def up(n: int, m: int = 8) -> int:
@@ -228,8 +229,9 @@ class LatentAttention:
         else:
             splits, acc = 1, torch.empty(n, m.heads * self.cp, device=dev)
             O.paged_attn(q, cache, cache, dim=self.row, vdim=self.cp, scale=m.scale, out=acc, **at)
-        A.latent_merge(acc, ml, n, self.uv, out, heads=m.heads, splits=splits, cp=self.cp, vdim=m.vdim, rows=rows, pdl=s.pdl)
-        s.launched(3)
+        merged = torch.empty(n, m.heads, self.cp, device=dev, dtype=torch.bfloat16) if ml is not None and n > MERGE_ROWS and self.uv.dtype == torch.bfloat16 else None
+        A.latent_merge(acc, ml, n, self.uv, out, heads=m.heads, splits=splits, cp=self.cp, vdim=m.vdim, rows=rows, merged=merged, pdl=s.pdl)
+        s.launched(3 + (merged is not None))
 
     def _long(self, s: Step, qkv, cache, out, lp: LongPortions) -> None:
         """Attention of the query tiles of ``lp`` over keys and values multiplied out of the latents."""

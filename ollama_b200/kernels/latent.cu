@@ -7,7 +7,8 @@
 // out for the visible positions instead, which costs fewer products per score.
 //
 //   latent_step    a row's latent under its RMS norm and rotated key part into the cache; U_h^T q and the rotated query part
-//   latent_merge   the split results of the absorbed form added up and multiplied by V_h
+//   latent_merge   the split results of the absorbed form added up and multiplied by V_h (a few rows); latent_reduce and latent_values: the
+//                  same in two launches, the second on the tensor cores with 16 rows at a time
 //   latent_gather  cache rows of whole sequences side by side, for the products of the long form
 //   latent_query   query rows of the long form
 //
@@ -198,19 +199,49 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const __grid_constan
 }
 
 constexpr int MAX_SPLITS = 128;
+constexpr int VR = 4;          // value rows of a warp of latent_merge
+constexpr int BATCH = 8;       // splits whose sums are under way together
 
-// grid (heads, value parts of 8 VR, row groups of NB); a warp multiplies VR value rows.  The chain is latency: the value rows, which do not depend
-// on the producer kernel, are in registers before the wait (rows of up to 512 16-bit values), and the split sums are requested
-// together with their statistics.
-template <typename WT, int NB, int VR>
-__global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant__ LatentMergeArgs a, int n) {
-    constexpr bool PRE = sizeof(WT) == 2 && NB == 1;
-    constexpr int BATCH = 8;
-    extern __shared__ __align__(16) float so[];    // [NB][cp]
-    __shared__ __align__(16) float half[PRE ? 512 : 4];
-    __shared__ float sw[NB][MAX_SPLITS];
-    __shared__ int s_n[NB];                        // splits with keys: the first ones
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, i0 = blockIdx.z * NB, nb = min(NB, n - i0);
+// Column group `col` (four columns) of a head's split sums: those of splits first, first + step, ... added up under a common maximum.
+__device__ __forceinline__ void add_splits(const float* acc, const float2* ml, int splits, int cp, int col, int first, int step, float4& o, float& m, float& l) {
+    o = make_float4(0.f, 0.f, 0.f, 0.f);
+    m = -1e30f;
+    l = 0.f;
+    for (int s0 = first; s0 < splits; s0 += step * BATCH) {
+        float2 st[BATCH];
+        float4 v[BATCH];
+#pragma unroll
+        for (int i = 0; i < BATCH; i++) {
+            const int s = s0 + step * i;
+            st[i] = s < splits ? ml[s] : make_float2(-1e30f, 0.f);
+            v[i] = s < splits && 4 * col < cp ? *(const float4*)(acc + (size_t)s * cp + 4 * col) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        float mn = m;
+#pragma unroll
+        for (int i = 0; i < BATCH; i++) mn = st[i].y > 0.f ? fmaxf(mn, st[i].x) : mn;
+        const float c = expf(m - mn);
+        o.x *= c; o.y *= c; o.z *= c; o.w *= c;
+        l *= c;
+        m = mn;
+#pragma unroll
+        for (int i = 0; i < BATCH; i++) {
+            if (!(st[i].y > 0.f)) continue;        // splits without keys leave their sums unwritten
+            const float w = expf(st[i].x - mn);
+            l += w * st[i].y;
+            o.x += w * v[i].x; o.y += w * v[i].y; o.z += w * v[i].z; o.w += w * v[i].w;
+        }
+    }
+}
+
+// grid (heads, value parts of 8 VR, rows); a warp multiplies VR value rows.  The chain is latency: the value rows, which do not depend on
+// the producer kernel, are in registers before the wait (rows of up to 512 16-bit values), and the split sums are requested together with
+// their statistics, every other split by each half of the CTA.
+template <typename WT>
+__global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant__ LatentMergeArgs a) {
+    constexpr bool PRE = sizeof(WT) == 2;
+    extern __shared__ __align__(16) float so[];    // [cp], then the second half's sums [cp]
+    __shared__ float s_m[2], s_l[2];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, i = blockIdx.z;
     const int v0 = (blockIdx.y * 8 + warp) * VR;
     const WT* uv = (const WT*)a.uv + ((size_t)h * a.vdim + v0) * a.cp;
     const bool pre = PRE && a.cp <= 512;
@@ -231,105 +262,36 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant
                     asm volatile("prefetch.global.L2 [%0];" ::"l"(uv + (size_t)j * a.cp + c));
     }
     pdl_wait();
-    const int q4 = a.cp >> 2;                      // float4 columns
-    if (a.ml && NB == 1 && q4 <= 128) {            // the two halves of the CTA take every other split
-        const float* p = a.acc + ((size_t)i0 * a.n_heads + h) * a.splits * a.cp;
-        const float2* ml = a.ml + ((size_t)i0 * a.n_heads + h) * a.splits;
-        const int col = tid & 127, part = tid >> 7;
-        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-        float m = -1e30f, l = 0.f;
-        for (int s0 = part; s0 < a.splits; s0 += 2 * BATCH) {
-            float2 st[BATCH];
-            float4 v[BATCH];
-#pragma unroll
-            for (int i = 0; i < BATCH; i++) {
-                const int s = s0 + 2 * i;
-                st[i] = s < a.splits ? ml[s] : make_float2(-1e30f, 0.f);
-                v[i] = s < a.splits && col < q4 ? *(const float4*)(p + (size_t)s * a.cp + 4 * col) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float* acc = a.acc + ((size_t)i * a.n_heads + h) * a.splits * a.cp;
+    if (a.ml) {
+        const float2* ml = a.ml + ((size_t)i * a.n_heads + h) * a.splits;
+        const int part = tid >> 7;
+        float4 o;
+        float m, l;
+        for (int c0 = 0; c0 < a.cp; c0 += 512) {   // one turn for latents of up to 512 values
+            const int c = c0 + 4 * (tid & 127);
+            add_splits(acc, ml, a.splits, a.cp, c >> 2, part, 2, o, m, l);
+            if (c < a.cp) *(float4*)(so + part * a.cp + c) = o;
+            if ((tid & 127) == 0) {
+                s_m[part] = m;
+                s_l[part] = l;
             }
-            float mn = m;
-#pragma unroll
-            for (int i = 0; i < BATCH; i++) mn = st[i].y > 0.f ? fmaxf(mn, st[i].x) : mn;
-            const float c = expf(m - mn);
-            o.x *= c; o.y *= c; o.z *= c; o.w *= c;
-            l *= c;
-            m = mn;
-#pragma unroll
-            for (int i = 0; i < BATCH; i++) {
-                if (!(st[i].y > 0.f)) continue;    // splits without keys leave their sums unwritten
-                const float w = expf(st[i].x - mn);
-                l += w * st[i].y;
-                o.x += w * v[i].x; o.y += w * v[i].y; o.z += w * v[i].z; o.w += w * v[i].w;
-            }
-        }
-        float* stats = &sw[0][0];                  // (max, sum) of the second half
-        if (part == 1 && col < q4) *(float4*)(PRE ? half + 4 * col : so + 4 * col) = o;
-        if (tid == 128) {
-            stats[0] = m;
-            stats[1] = l;
         }
         __syncthreads();
-        if (part == 0 && col < q4) {
-            const float4 o1 = *(const float4*)(PRE ? half + 4 * col : so + 4 * col);
-            const float mn = fmaxf(m, stats[0]), c0 = expf(m - mn), c1 = expf(stats[0] - mn), inv = 1.f / (c0 * l + c1 * stats[1]);
-            *(float4*)(so + 4 * col) = make_float4((c0 * o.x + c1 * o1.x) * inv, (c0 * o.y + c1 * o1.y) * inv, (c0 * o.z + c1 * o1.z) * inv, (c0 * o.w + c1 * o1.w) * inv);
-        }
+        const float mn = fmaxf(s_m[0], s_m[1]), c0 = expf(s_m[0] - mn), c1 = expf(s_m[1] - mn), inv = 1.f / (c0 * s_l[0] + c1 * s_l[1]);
+        for (int c = tid; c < a.cp; c += 256) so[c] = (c0 * so[c] + c1 * so[a.cp + c]) * inv;
     } else {
-        if (a.ml) {
-            if (warp < nb) {
-                const float2* ml = a.ml + ((size_t)(i0 + warp) * a.n_heads + h) * a.splits;
-                float m = -INFINITY, l = 0.f;
-                int used = 0;
-                for (int s = lane; s < a.splits; s += 32)
-                    if (ml[s].y > 0.f) m = fmaxf(m, ml[s].x);
-                m = warp_max(m);
-                for (int s = lane; s < a.splits; s += 32) {
-                    const float w = ml[s].y > 0.f ? expf(ml[s].x - m) : 0.f;
-                    sw[warp][s] = w;
-                    l += w * ml[s].y;
-                    if (ml[s].y > 0.f) used = s + 1;
-                }
-                l = warp_sum(l);
-                used = __reduce_max_sync(0xffffffffu, used);
-                if (lane == 0) s_n[warp] = used;
-                __syncwarp();
-                for (int s = lane; s < a.splits; s += 32) sw[warp][s] /= l;
-            }
-            __syncthreads();
-        }
-        for (int j = tid; j < nb * q4; j += 256) {
-            const int b = j / q4, c = 4 * (j - b * q4);
-            const float* p = a.acc + ((size_t)(i0 + b) * a.n_heads + h) * a.splits * a.cp + c;
-            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (a.ml) {
-                const int used = s_n[b];
-#pragma unroll 8
-                for (int s = 0; s < used; s++) {
-                    const float w = sw[b][s];
-                    const float4 v = *(const float4*)(p + (size_t)s * a.cp);
-                    o.x += w * v.x; o.y += w * v.y; o.z += w * v.z; o.w += w * v.w;
-                }
-            } else {
-                o = *(const float4*)p;
-            }
-            *(float4*)(so + b * a.cp + c) = o;
-        }
+        for (int c = tid; c < a.cp; c += 256) so[c] = acc[c];
     }
     __syncthreads();
 #pragma unroll
     for (int j = 0; j < VR; j++) {
         const int v = v0 + j;
         if (v >= a.vdim) return;
-        float acc[NB];
-#pragma unroll
-        for (int b = 0; b < NB; b++) acc[b] = 0.f;
+        float sum = 0.f;
         auto add = [&](const float (&f)[8], int c) {
-#pragma unroll
-            for (int b = 0; b < NB; b++) {
-                if (b >= nb) break;
-                const float4 x = *(const float4*)(so + b * a.cp + c), y = *(const float4*)(so + b * a.cp + c + 4);
-                acc[b] += f[0] * x.x + f[1] * x.y + f[2] * x.z + f[3] * x.w + f[4] * y.x + f[5] * y.y + f[6] * y.z + f[7] * y.w;
-            }
+            const float4 x = *(const float4*)(so + c), y = *(const float4*)(so + c + 4);
+            sum += f[0] * x.x + f[1] * x.y + f[2] * x.z + f[3] * x.w + f[4] * y.x + f[5] * y.y + f[6] * y.z + f[7] * y.w;
         };
         if (pre) {
 #pragma unroll
@@ -339,9 +301,9 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant
                 const uint32_t q[4] = {w.x, w.y, w.z, w.w};
                 float f[8];
 #pragma unroll
-                for (int i = 0; i < 4; i++) {
-                    f[2 * i] = __uint_as_float(q[i] << 16);
-                    f[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
+                for (int e = 0; e < 4; e++) {
+                    f[2 * e] = __uint_as_float(q[e] << 16);
+                    f[2 * e + 1] = __uint_as_float(q[e] & 0xffff0000u);
                 }
                 if (c < a.cp) add(f, c);
             }
@@ -352,16 +314,64 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const __grid_constant
                 add(f, c);
             }
         }
-#pragma unroll
-        for (int b = 0; b < NB; b++) {
-            if (b >= nb) break;
-            const float s = warp_sum(acc[b]);
-            if (lane == 0) {
-                const size_t o = (size_t)(a.rows ? a.rows[i0 + b] : i0 + b) * a.ldo + (size_t)h * a.vdim + v;
-                if (a.out16) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(s);
-                else ((float*)a.out)[o] = s;
-            }
+        sum = warp_sum(sum);
+        if (lane == 0) {
+            const size_t o = (size_t)(a.rows ? a.rows[i] : i) * a.ldo + (size_t)h * a.vdim + v;
+            if (a.out16) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(sum);
+            else ((float*)a.out)[o] = sum;
         }
+    }
+}
+
+// grid (heads, rows): the split sums of a head added up, as bf16 rows [row][head][cp] of `merged`
+__global__ void __launch_bounds__(128) latent_reduce_kernel(const __grid_constant__ LatentMergeArgs a, __nv_bfloat16* merged) {
+    const int h = blockIdx.x, i = blockIdx.y;
+    pdl_launch();
+    pdl_wait();
+    const size_t at = (size_t)i * a.n_heads + h;
+    for (int c = 4 * threadIdx.x; c < a.cp; c += 512) {
+        float4 o;
+        float m, l;
+        add_splits(a.acc + at * a.splits * a.cp, a.ml + at * a.splits, a.splits, a.cp, c >> 2, 0, 1, o, m, l);
+        const float inv = 1.f / l;
+        const __nv_bfloat162 x = __floats2bfloat162_rn(o.x * inv, o.y * inv), y = __floats2bfloat162_rn(o.z * inv, o.w * inv);
+        *(uint2*)(merged + at * a.cp + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
+    }
+}
+
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+// grid (heads, value parts of 32, row groups of 16), 4 warps; a warp multiplies 8 value rows with 16 merged rows.  Both operands run along cp, so a
+// thread loads eight consecutive values of each and uses them as the fragments of two products: the order of the terms is the same on both sides.
+__global__ void __launch_bounds__(128) latent_values_kernel(const __grid_constant__ LatentMergeArgs a, const __nv_bfloat16* merged, int n) {
+    const int lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3, h = blockIdx.x, i0 = blockIdx.z * 16;
+    const int v0 = blockIdx.y * 32 + 8 * (threadIdx.x >> 5);
+    if (v0 >= a.vdim) return;
+    const __nv_bfloat16* w = (const __nv_bfloat16*)a.uv + ((size_t)h * a.vdim + min(v0 + g, a.vdim - 1)) * a.cp + 8 * tq;
+    const __nv_bfloat16* r0 = merged + ((size_t)min(i0 + g, n - 1) * a.n_heads + h) * a.cp + 8 * tq;
+    const __nv_bfloat16* r1 = merged + ((size_t)min(i0 + g + 8, n - 1) * a.n_heads + h) * a.cp + 8 * tq;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    float c[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f};
+    pdl_launch();
+    for (int k = 0; k < a.cp; k += 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + k));
+    pdl_wait();
+#pragma unroll 4
+    for (int k = 0; k < a.cp; k += 32) {
+        const bool in = k + 8 * tq < a.cp;         // cp is a multiple of 16
+        const uint4 b = in ? ldg16(w + k) : zero, x = in ? *(const uint4*)(r0 + k) : zero, y = in ? *(const uint4*)(r1 + k) : zero;
+        mma_bf16(c, x.x, y.x, x.y, y.y, b.x, b.y);
+        mma_bf16(d, x.z, y.z, x.w, y.w, b.z, b.w);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        const int i = i0 + g + 8 * (e >> 1), v = v0 + 2 * tq + (e & 1);
+        if (i >= n || v >= a.vdim) continue;
+        const size_t o = (size_t)(a.rows ? a.rows[i] : i) * a.ldo + (size_t)h * a.vdim + v;
+        if (a.out16) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(c[e] + d[e]);
+        else ((float*)a.out)[o] = c[e] + d[e];
     }
 }
 
@@ -442,19 +452,23 @@ B2_API int b2_latent_step(const LatentStepArgs* a, int n, int pdl, cudaStream_t 
     return launch_rows(fn, dim3(a->n_heads * parts + nb, (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
 }
 
-B2_API int b2_latent_merge(const LatentMergeArgs* a, int n, int pdl, cudaStream_t st) {
-    if (n < 1 || a->n_heads < 1 || a->splits < 1 || a->splits > MAX_SPLITS || (!a->ml && a->splits != 1) || (a->cp & 15) || a->vdim < 1 || ((uintptr_t)a->uv & 15) || ((uintptr_t)a->acc & 15))
+// With `merged` (bf16 [n][heads][cp] of scratch) the two-launch form: 16-bit values and splits with statistics only.
+B2_API int b2_latent_merge(const LatentMergeArgs* a, int n, void* merged, int pdl, cudaStream_t st) {
+    if (n < 1 || n > 65535 || a->n_heads < 1 || a->splits < 1 || a->splits > MAX_SPLITS || (!a->ml && a->splits != 1) || (a->cp & 15) || a->vdim < 1 || ((uintptr_t)a->uv & 15) ||
+        ((uintptr_t)a->acc & 15) || (merged && (a->w32 || !a->ml || ((uintptr_t)merged & 15))))
         return (int)cudaErrorInvalidValue;
-    const int nb = n <= 32 ? 1 : 4;                // a decode step: latency counts, the value rows come from L2 for every row
-    const size_t smem = (size_t)nb * a->cp * 4;
-    if (smem > 40 * 1024) return (int)cudaErrorNotSupported;
-    if ((n + nb - 1) / nb > 65535) return (int)cudaErrorInvalidValue;
     LatentMergeArgs c = *a;
-    void* args[] = {&c, &n};
-    const int vr = nb == 1 ? 4 : 8;
-    const void* fn = a->w32 ? (nb == 1 ? (const void*)latent_merge_kernel<float, 1, 4> : (const void*)latent_merge_kernel<float, 4, 8>)
-                            : (nb == 1 ? (const void*)latent_merge_kernel<__nv_bfloat16, 1, 4> : (const void*)latent_merge_kernel<__nv_bfloat16, 4, 8>);
-    return launch_rows(fn, dim3(a->n_heads, (a->vdim + 8 * vr - 1) / (8 * vr), (n + nb - 1) / nb), dim3(256), smem, args, st, pdl);
+    if (merged) {
+        void* args[] = {&c, &merged, &n};
+        const int rc = launch_rows((const void*)latent_reduce_kernel, dim3(a->n_heads, n), dim3(128), 0, args, st, pdl);
+        if (rc) return rc;
+        return launch_rows((const void*)latent_values_kernel, dim3(a->n_heads, (a->vdim + 31) / 32, (n + 15) / 16), dim3(128), 0, args, st, pdl);
+    }
+    const size_t smem = (size_t)2 * a->cp * 4;
+    if (smem > 40 * 1024) return (int)cudaErrorNotSupported;
+    void* args[] = {&c};
+    return launch_rows(a->w32 ? (const void*)latent_merge_kernel<float> : (const void*)latent_merge_kernel<__nv_bfloat16>, dim3(a->n_heads, (a->vdim + 8 * VR - 1) / (8 * VR), n),
+                       dim3(256), smem, args, st, pdl);
 }
 
 B2_API int b2_latent_gather(const LatentGatherArgs* a, int n_seqs, int max_len, cudaStream_t st) {

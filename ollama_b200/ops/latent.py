@@ -48,10 +48,11 @@ def latent_step(qkv: torch.Tensor, n: int, *, heads: int, dim: int, rot: int, ra
 
 
 def latent_merge(acc: torch.Tensor, ml: torch.Tensor | None, n: int, uv: torch.Tensor, out: torch.Tensor, *, heads: int, splits: int, cp: int, vdim: int, rows=None,
-                 pdl: bool = False) -> None:
-    """Split results [n, heads, splits, cp] merged and multiplied by ``uv`` [heads * vdim, cp] into rows of ``out``."""
+                 merged: torch.Tensor | None = None, pdl: bool = False) -> None:
+    """Split results [n, heads, splits, cp] merged and multiplied by ``uv`` [heads * vdim, cp] into rows of ``out``.  ``merged``: bf16 scratch [n, heads, cp] for
+    the two-launch form, whose product runs on the tensor cores."""
     a = LatentMergeArgs(ptr(acc), ptr(ml), heads, splits, cp, vdim, ptr(uv), _is32(uv), ptr(rows), ptr(out), out.stride(0), 1 - _is32(out))
-    _call("b2_latent_merge", a, n, int(pdl))
+    _call("b2_latent_merge", a, n, C.c_void_p(ptr(merged)), int(pdl))
 
 
 def attn_latent(q: torch.Tensor, n: int, cache: torch.Tensor, acc, ml, *, heads: int, cp: int, scale: float, splits: int, positions, slots, table, rows=None,

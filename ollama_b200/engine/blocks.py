@@ -14,6 +14,7 @@ from ..models.stack import DenseMLP, Expert, ExpertMLP, LatentMixer
 from ..ops import cuda as K
 from ..ops import latent as A
 from ..ops import rows as O
+from .cache import PAGE
 
 LONG_PORTION = 64                # prompt portions of this many tokens multiply keys and values out; shorter ones stay in the latent space
 MAX_SPLITS = 128
@@ -211,9 +212,9 @@ class LatentAttention:
                     positions=s.m.positions, slots=s.m.slots, table=s.be.cache.table, cp=self.cp, pdl=s.pdl)
 
     def splits(self, n: int, n_ctx: int, sms: int) -> int:
-        """Parts of the keys for ``n`` queries: as many CTAs as are resident (wide rows: one per SM), none shorter than two pages."""
+        """Parts of the keys for ``n`` queries: as many CTAs as are resident (wide rows: one per SM), none shorter than a page."""
         groups = -(-self.m.heads // (16 if self.m.heads <= 16 else 32))
-        return max(1, min(-(-n_ctx // 128), (1 if self.row > 256 else 2) * sms // (groups * n), MAX_SPLITS))
+        return max(1, min(-(-n_ctx // PAGE), (1 if self.row > 256 else 2) * sms // (groups * n), MAX_SPLITS))
 
     def _latent(self, s: Step, qkv, cache, out, n: int, rows, append: bool) -> None:
         """Attention of ``n`` rows in the latent space."""

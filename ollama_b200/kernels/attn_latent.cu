@@ -2,8 +2,9 @@
 //
 // All heads of a row score the same cache rows, so the heads are the rows of m16n8k16 tiles and a cache row is read once for up to 32
 // heads: score = q . (latent | rotated part), result = sum of p times the latent part of the same row.  grid = (splits, groups of heads,
-// query rows), 8 warps.  Tiles of 64 positions (a page) arrive by cp.async in NS stages.  Per tile each warp scores 8 positions, the
-// soft-max statistics of a head are kept by a few neighbouring threads, and each warp owns 16-column units of the result.
+// query rows), 8 warps.  Tiles of a page arrive by cp.async in two stages.  The query fragments stay in registers: a warp scores half of a
+// tile's positions over a quarter of the row, the quarters are added by the threads that keep a head's soft-max statistics, and each
+// warp owns 16-column units of the result.
 #include "rows.cuh"
 
 struct LatentAttnArgs {
@@ -22,7 +23,7 @@ struct LatentAttnArgs {
 
 namespace {
 
-constexpr int BN = 64, PAD = 8, LDS = BN + 4, LDP = BN + 8;
+constexpr int BN = PAGE, PAD = 8, QUARTERS = 4;
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -35,54 +36,68 @@ __device__ __forceinline__ void mma_f16(float (&c)[4], const uint32_t (&a)[4], u
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
-}
+template <int MT>
+struct Lay {
+    static constexpr int HR = 16 * MT, LDS = BN + 4, LDP = BN + 8;
+    static size_t bytes(int w) { return (size_t)2 * BN * (w + PAD) * 2 + (size_t)HR * (QUARTERS * LDS * 4 + LDP * 2); }
+};
 
-// MT: tiles of 16 heads per CTA; NU: 16-column units of the result per warp
-template <int MT, int NU, int NS>
-__global__ void __launch_bounds__(256) attn_latent_kernel(const __grid_constant__ LatentAttnArgs a) {
-    constexpr int HR = 16 * MT, TPR = 256 / HR, KPT = BN / TPR;
+// MT: tiles of 16 heads per CTA; NU: 16-column units of the result per warp; KQ: 16-column steps of a quarter of the row, at most
+template <int MT, int NU, int KQ>
+__global__ void __launch_bounds__(256, MT == 1 ? 2 : 1) attn_latent_kernel(const __grid_constant__ LatentAttnArgs a) {
+    using L = Lay<MT>;
+    constexpr int HR = L::HR, LDS = L::LDS, LDP = L::LDP, TPR = 256 / HR, KPT = BN / TPR, NT = BN / 16;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ float s_corr[HR];
     const int ld = a.w + PAD;
-    __half* sQ = reinterpret_cast<__half*>(smem_raw);            // [HR][ld]
-    __half* sKV = sQ + HR * ld;                                  // [NS][BN][ld]
-    float* sS = reinterpret_cast<float*>(sKV + NS * BN * ld);    // [HR][LDS]
-    __half* sP = reinterpret_cast<__half*>(sS + HR * LDS);       // [HR][LDP]
+    __half* sKV = reinterpret_cast<__half*>(smem_raw);           // [2][BN][ld]
+    float* sS = reinterpret_cast<float*>(sKV + 2 * BN * ld);     // [QUARTERS][HR][LDS]
+    __half* sP = reinterpret_cast<__half*>(sS + QUARTERS * HR * LDS);      // [HR][LDP]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int split = blockIdx.x, head0 = blockIdx.y * HR, i = blockIdx.z;
-    const int heads = min(HR, a.n_heads - head0), chunks = a.w >> 3;
+    const int heads = min(HR, a.n_heads - head0);
 
     pdl_launch();
     pdl_wait();
     const int row = a.rows ? a.rows[i] : i;
     const int kv_len = a.positions[row] + 1;
     const int* table = a.page_table + (size_t)a.slots[row] * a.max_pages;
-    const int pages = (kv_len + BN - 1) / BN, per = (pages + a.splits - 1) / a.splits;
-    const int t0 = split * per, n_tiles = min(per, pages - t0);
-    if (n_tiles <= 0) {
+    const int pages = (kv_len + PAGE - 1) / PAGE, per = (pages + a.splits - 1) / a.splits;
+    const int p0 = split * per * PAGE, n_tiles = (min(kv_len - p0, per * PAGE) + BN - 1) / BN;
+    if (kv_len <= p0) {
         for (int h = tid; h < heads; h += 256) a.ml[((size_t)i * a.n_heads + head0 + h) * a.splits + split] = make_float2(-1e30f, 0.f);
         return;
     }
     auto load_tile = [&](int tile) {
-        const __half* src = a.cache + paged_row(table, (t0 + tile) * BN, 1, 0) * a.w;
-        __half* dst = sKV + (tile % NS) * BN * ld;
-        for (int c = tid; c < BN * chunks; c += 256) {
-            const int r = c / chunks, col = (c - r * chunks) * 8;
-            cp_async16(dst + r * ld + col, src + (size_t)r * a.w + col);
-        }
-    };
+        const __half* src = a.cache + paged_row(table, p0 + tile * BN + warp, 1, 0) * a.w + 8 * lane;
+        const __half* end = src + a.w - 8 * lane;
+        uint32_t dst = smem_addr(sKV + ((tile & 1) * BN + warp) * ld + 8 * lane);
 #pragma unroll
-    for (int t = 0; t < NS - 1; t++) {
-        if (t < n_tiles) load_tile(t);
+        for (int r = 0; r < BN / 8; r++, src += 8 * a.w, end += 8 * a.w, dst += 16 * ld) {      // a warp per row
+#pragma unroll
+            for (int c = 0; c < (KQ * QUARTERS * 16 + 255) / 256; c++)
+                if (src + 256 * c < end) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + 512 * c), "l"(src + 256 * c) : "memory");
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
-    }
-    for (int c = tid; c < HR * chunks; c += 256) {
-        const int r = c / chunks, col = (c - r * chunks) * 8;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (r < heads) v = *(const uint4*)(a.q + ((size_t)i * a.n_heads + head0 + r) * a.w + col);
-        *(uint4*)(sQ + r * ld + col) = v;
+    };
+    load_tile(0);
+    // this warp's part of the scores: positions [BN / 2 * half, + BN / 2) of a tile, columns [16 k0, 16 k1) of the row
+    const int quarter = warp & 3, half = warp >> 2, steps = a.w >> 4, kq = (steps + QUARTERS - 1) / QUARTERS;
+    const int k0 = quarter * kq, k1 = min(k0 + kq, steps);
+    uint32_t qf[MT][KQ][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++) {
+        const __half* q0 = a.q + ((size_t)i * a.n_heads + head0 + 16 * m + g) * a.w + 2 * tq;
+        const bool in0 = 16 * m + g < heads, in1 = 16 * m + g + 8 < heads;
+#pragma unroll
+        for (int k = 0; k < KQ; k++) {
+            const bool in = k0 + k < k1;
+            const __half* q = q0 + 16 * (k0 + k);
+            qf[m][k][0] = in && in0 ? *(const uint32_t*)q : 0u;
+            qf[m][k][1] = in && in1 ? *(const uint32_t*)(q + (size_t)8 * a.w) : 0u;
+            qf[m][k][2] = in && in0 ? *(const uint32_t*)(q + 8) : 0u;
+            qf[m][k][3] = in && in1 ? *(const uint32_t*)(q + (size_t)8 * a.w + 8) : 0u;
+        }
     }
     float o[MT][NU][2][4];
 #pragma unroll
@@ -94,52 +109,58 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(const __grid_constant_
     const int srow = tid / TPR, sub = tid % TPR;                 // soft-max phase: head row and first position of this thread
     float m_run = -1e30f, l_run = 0.f;
     const int units = a.cp >> 4;
-    const uint32_t qa = smem_addr(sQ + ((lane & 7) + 8 * ((lane >> 3) & 1)) * ld + 8 * (lane >> 4));
 
     for (int tile = 0; tile < n_tiles; tile++) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(NS - 2) : "memory");
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                         // the tile is there; everyone has left the stage of tile - 1
-        if (tile + NS - 1 < n_tiles) load_tile(tile + NS - 1);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        const __half* kv = sKV + (tile % NS) * BN * ld;
-        float s[MT][2][4];
+        if (tile + 1 < n_tiles) load_tile(tile + 1);
+        const __half* kv = sKV + (tile & 1) * BN * ld;
+        float s[MT][NT][4];
 #pragma unroll
         for (int m = 0; m < MT; m++)
 #pragma unroll
-            for (int j = 0; j < 2; j++) s[m][j][0] = s[m][j][1] = s[m][j][2] = s[m][j][3] = 0.f;
-        const uint32_t ka = smem_addr(kv + (8 * warp + (lane & 7)) * ld + 8 * (lane >> 3));
-#pragma unroll 3
-        for (int kk = 0; kk < a.w; kk += 32) {
-            uint32_t kb[4];
-            ldmatrix_x4(kb, ka + 2 * kk);
+            for (int j = 0; j < NT; j++) s[m][j][0] = s[m][j][1] = s[m][j][2] = s[m][j][3] = 0.f;
+        const uint32_t ka = smem_addr(kv + (BN / 2 * half + (lane & 7) + 8 * (lane >> 4)) * ld + 16 * k0 + 8 * ((lane >> 3) & 1));
 #pragma unroll
-            for (int m = 0; m < MT; m++) {
-                uint32_t q0[4], q1[4];
-                ldmatrix_x4(q0, qa + 2 * (16 * m * ld + kk));
-                ldmatrix_x4(q1, qa + 2 * (16 * m * ld + kk + 16));
-                mma_f16(s[m][0], q0, kb[0], kb[1]);
-                mma_f16(s[m][1], q1, kb[2], kb[3]);
+        for (int k = 0; k < KQ; k++) {
+            if (k0 + k >= k1) break;                             // warp-uniform
+#pragma unroll
+            for (int j = 0; j < NT / 2; j++) {                   // 16 positions
+                uint32_t kb[4];
+                ldmatrix_x4(kb, ka + 2 * (16 * j * ld + 16 * k));
+#pragma unroll
+                for (int m = 0; m < MT; m++) {
+                    mma_f16(s[m][2 * j], qf[m][k], kb[0], kb[1]);
+                    mma_f16(s[m][2 * j + 1], qf[m][k], kb[2], kb[3]);
+                }
             }
         }
 #pragma unroll
-        for (int m = 0; m < MT; m++) {
-            float* d = sS + (16 * m + g) * LDS + 8 * warp + 2 * tq;
-            *(float2*)d = make_float2(s[m][0][0] + s[m][1][0], s[m][0][1] + s[m][1][1]);
-            *(float2*)(d + 8 * LDS) = make_float2(s[m][0][2] + s[m][1][2], s[m][0][3] + s[m][1][3]);
-        }
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+            for (int j = 0; j < NT; j++) {
+                float* d = sS + (quarter * HR + 16 * m + g) * LDS + BN / 2 * half + 8 * j + 2 * tq;
+                *(float2*)d = make_float2(s[m][j][0], s[m][j][1]);
+                *(float2*)(d + 8 * LDS) = make_float2(s[m][j][2], s[m][j][3]);
+            }
         __syncthreads();
         {
             float v[KPT];
             float mx = -1e30f;
-            const int k0 = (t0 + tile) * BN + sub * KPT;
+            const int kp = p0 + tile * BN + sub * KPT;
 #pragma unroll
-            for (int j = 0; j < KPT; j += 4) {
-                const float4 f = *(const float4*)(sS + srow * LDS + sub * KPT + j);
-                v[j] = f.x; v[j + 1] = f.y; v[j + 2] = f.z; v[j + 3] = f.w;
+            for (int j = 0; j < KPT; j += 2) {
+                float2 f = make_float2(0.f, 0.f);
+#pragma unroll
+                for (int x = 0; x < QUARTERS; x++) {
+                    const float2 t = *(const float2*)(sS + (x * HR + srow) * LDS + sub * KPT + j);
+                    f.x += t.x; f.y += t.y;
+                }
+                v[j] = f.x; v[j + 1] = f.y;
             }
 #pragma unroll
             for (int j = 0; j < KPT; j++) {
-                v[j] = k0 + j < kv_len ? v[j] * a.scale : -INFINITY;
+                v[j] = kp + j < kv_len ? v[j] * a.scale : -INFINITY;
                 mx = fmaxf(mx, v[j]);
             }
 #pragma unroll
@@ -148,9 +169,9 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(const __grid_constant_
             float ls = 0.f;
 #pragma unroll
             for (int j = 0; j < KPT; j += 2) {
-                const float p0 = __expf(v[j] - m_new), p1 = __expf(v[j + 1] - m_new);
-                ls += p0 + p1;
-                *(__half2*)(sP + srow * LDP + sub * KPT + j) = __floats2half2_rn(p0, p1);
+                const float e0 = __expf(v[j] - m_new), e1 = __expf(v[j + 1] - m_new);
+                ls += e0 + e1;
+                *(__half2*)(sP + srow * LDP + sub * KPT + j) = __floats2half2_rn(e0, e1);
             }
             l_run = l_run * corr + ls;
             m_run = m_new;
@@ -210,37 +231,31 @@ __global__ void __launch_bounds__(256) attn_latent_kernel(const __grid_constant_
 
 constexpr size_t SMEM_MAX = 226 * 1024;
 
-size_t smem_bytes(int mt, int ns, int w) { return (size_t)(16 * mt + ns * BN) * (w + PAD) * 2 + (size_t)16 * mt * (LDS * 4 + LDP * 2); }
-
-template <int MT, int NU, int NS>
+template <int MT, int NU, int KQ>
 int launch(const LatentAttnArgs& a, int n, int pdl, cudaStream_t st) {
+    const size_t smem = Lay<MT>::bytes(a.w);
+    if (smem > SMEM_MAX) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(attn_latent_kernel<MT, NU, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_MAX);
+    if (once.first()) cudaFuncSetAttribute(attn_latent_kernel<MT, NU, KQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_MAX);
     LatentAttnArgs c = a;
     void* args[] = {&c};
-    return launch_rows((const void*)attn_latent_kernel<MT, NU, NS>, dim3(a.splits, (a.n_heads + 16 * MT - 1) / (16 * MT), n), dim3(256), smem_bytes(MT, NS, a.w), args, st, pdl);
-}
-
-template <int MT, int NU>
-int launch_ns(const LatentAttnArgs& a, int n, int pdl, cudaStream_t st) {
-    if (smem_bytes(MT, 3, a.w) <= SMEM_MAX / 2) return launch<MT, NU, 3>(a, n, pdl, st);      // two CTAs per SM
-    if (smem_bytes(MT, 2, a.w) <= SMEM_MAX) return launch<MT, NU, 2>(a, n, pdl, st);
-    return (int)cudaErrorNotSupported;
+    return launch_rows((const void*)attn_latent_kernel<MT, NU, KQ>, dim3(a.splits, (a.n_heads + 16 * MT - 1) / (16 * MT), n), dim3(256), smem, args, st, pdl);
 }
 
 template <int MT>
-int launch_nu(const LatentAttnArgs& a, int n, int pdl, cudaStream_t st) {
-    if (a.cp <= 128) return launch_ns<MT, 1>(a, n, pdl, st);
-    if (a.cp <= 256) return launch_ns<MT, 2>(a, n, pdl, st);
-    return launch_ns<MT, 4>(a, n, pdl, st);
+int launch_w(const LatentAttnArgs& a, int n, int pdl, cudaStream_t st) {
+    if (a.cp <= 128 && a.w <= 256) return launch<MT, 1, 4>(a, n, pdl, st);
+    if (a.cp <= 256 && a.w <= 448) return launch<MT, 2, 7>(a, n, pdl, st);
+    if (a.w <= 576) return launch<MT, 4, 9>(a, n, pdl, st);
+    return launch<MT, 4, 10>(a, n, pdl, st);
 }
 
 }  // namespace
 
-// f16 cache with w % 32 == 0 and a latent of up to 512 (padded) values; other shapes: cudaErrorNotSupported, nothing launched.
+// f16 cache with rows of up to 640 values, a multiple of 32, and a latent of up to 512; other shapes: cudaErrorNotSupported, nothing launched.
 B2_API int b2_attn_latent(const LatentAttnArgs* a, int n, int pdl, cudaStream_t st) {
     if (n < 1 || a->n_heads < 1 || a->splits < 1 || a->splits > 128 || a->cp < 16 || (a->cp & 15) || a->w < a->cp || a->max_pages < 1 || ((uintptr_t)a->q & 15) || ((uintptr_t)a->cache & 15))
         return (int)cudaErrorInvalidValue;
-    if ((a->w & 31) || a->cp > 512 || n > 65535) return (int)cudaErrorNotSupported;
-    return a->n_heads <= 16 ? launch_nu<1>(*a, n, pdl, st) : launch_nu<2>(*a, n, pdl, st);
+    if ((a->w & 31) || a->cp > 512 || a->w > 640 || n > 65535) return (int)cudaErrorNotSupported;
+    return a->n_heads <= 16 ? launch_w<1>(*a, n, pdl, st) : launch_w<2>(*a, n, pdl, st);
 }

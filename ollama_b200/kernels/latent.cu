@@ -134,7 +134,7 @@ template <typename CT, typename WT, int NB>
 __global__ void __launch_bounds__(256) latent_step_kernel(const __grid_constant__ LatentStepArgs a, int n) {
     extern __shared__ float sq[];                  // [NB][dim], or the rotation's cosines and sines
     __shared__ float red[DG][COLS + 4];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, i0 = blockIdx.y * NB;
+    const int tid = threadIdx.x, i0 = blockIdx.y * NB;
     const int parts = (a.cp + COLS - 1) / COLS;
     const int h = blockIdx.x / parts, part = blockIdx.x % parts;
     const int rb = (int)blockIdx.x - a.n_heads * parts;            // >= 0: row of the group

@@ -115,6 +115,8 @@ class Step:
         self.act = torch.float32 if self.small else be.act_dtype
         self.pdl = be.pdl and decode
         self.pending: dict = {}
+        self.copy = None                               # bf16 copy of the rows, made by the last product before a per-token input
+        self.last = False                              # the block that runs is a layer's last before its per-token input
 
     def buf(self, name: str, cols: int, dtype=None, zero: bool = False) -> torch.Tensor:
         return self.B.get(name, cols, dtype or self.act, self.nb, zero)
@@ -138,7 +140,10 @@ class Step:
 
     def add(self, h: torch.Tensor, mat: Mat) -> None:
         """x += residual multiplier * mat h."""
-        self.product(h, mat, self.x, accumulate=True, alpha=self.be.stack.residual_mult)
+        kw = {}
+        if self.last and not self.small and self.act == torch.bfloat16:
+            kw["copy"] = self.copy = self.buf("copy", self.be.wp)
+        self.product(h, mat, self.x, accumulate=True, alpha=self.be.stack.residual_mult, **kw)
 
     def normed(self, norm: Norm, mat: Mat, out: torch.Tensor, keep: bool = False, **kw) -> torch.Tensor | None:
         """out = f(mat norm(x) + bias); returns the normalised rows where they exist (always with ``keep``)."""
@@ -199,8 +204,6 @@ class LatentAttention:
         if lp is None or self.w_kv is None or s.decode:
             self._latent(s, qkv, cache, out, s.nb, None, True)
         else:
-            A.latent_step(qkv, s.nb, cache=cache, **self._step_args(s))
-            s.launched()
             self._long(s, qkv, cache, out, lp)
             if lp.rest is not None:
                 self._latent(s, qkv, cache, out, lp.rest.numel(), lp.rest, False)
@@ -235,10 +238,10 @@ class LatentAttention:
         s.launched(3 + (merged is not None))
 
     def _long(self, s: Step, qkv, cache, out, lp: LongPortions) -> None:
-        """Attention of the query tiles of ``lp`` over keys and values multiplied out of the latents."""
+        """Attention of the query tiles of ``lp`` over keys and values multiplied out of the latents; cache rows of the whole step."""
         m, dev, H = self.m, qkv.device, self.m.heads
         q = torch.empty(s.nb, H, self.dp + self.rp, device=dev, dtype=torch.float16)
-        A.latent_query(qkv, q, heads=H, dim=m.dim, rot=m.rot_dim, freqs=self.freqs, interleaved=self.interleaved, positions=s.m.positions, dp=self.dp, rp=self.rp)
+        A.latent_step(qkv, s.nb, cache=cache, q_out=q, dp=self.dp, rp=self.rp, **self._step_args(s))
         c = torch.empty(lp.total, self.cp, device=dev, dtype=torch.bfloat16)
         r = torch.empty(lp.total, max(self.rp, 8), device=dev, dtype=torch.float16)
         A.latent_gather(cache, self.cp, m.rot_dim, lp.seqs, lp.longest, s.be.cache.table, c, r)
@@ -337,9 +340,9 @@ class SideInput:
         return self.gate.w.numel() + self.proj.w.numel(), 0, 0.0
 
     def run(self, s: Step) -> None:
-        h = s.x
+        h, s.copy = s.copy if s.copy is not None else s.x, None
         if h.dtype != s.act:
-            h = s.buf("side_x", s.be.wp)
+            h = s.buf("copy", s.be.wp)
             O.join_rows(s.x, s.be.wp, h, pdl=s.pdl)
             s.launched()
         g, y = s.buf("side_g", self.dimp), s.buf("side_y", s.be.wp, torch.float32)

@@ -427,8 +427,10 @@ class StackBackend(StepEngine):
         s.pending = self._join(self.runs[0], s)
         for i, run in enumerate(self.runs):
             L, nxt = self.layers[run.layer], self.runs[i + 1] if i + 1 < len(self.runs) else None
+            s.last = L.side is not None and L.ff is None
             L.mix.run(s, self.mem[i])
             if L.ff is not None:
+                s.last = L.side is not None
                 L.ff.run(s)
             if L.side is not None:
                 L.side.run(s)

@@ -52,6 +52,7 @@ struct GemmParams {
     const __nv_bfloat16* mul;      // factor per element: mul[mul_row[row] * ldm + column], or null
     const int* mul_row;
     int ldm;
+    __nv_bfloat16* copy;    // fp32 results also go here as bf16, rows of pitch ldo
     int lda;                // row pitch of a, 0: k
     // split-K (splits > 1): part s of a tile covers its own range of k blocks and stores plain fp32 sums at part + s * part_stride
     // ([m][part_ld]); a second kernel adds the parts in order and applies the epilogue
@@ -92,14 +93,21 @@ __device__ __forceinline__ uint32_t pack2_f16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-// Four consecutive sums of a row, as the product's caller wants them: activation or gated pairs, factors, type, accumulation.
-__device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, int col) {
-    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
+// What the result's four elements at (row, col) are combined with: the sums they are added to, or the factors of a table.  Fetched ahead of
+// store4, so that the loads of several rows are under way together.
+__device__ __forceinline__ float4 fetch4(const GemmParams& p, int row, int col) {
+    if (p.accumulate) return *(const float4*)((const float*)p.out + (size_t)row * p.ldo + col);
     if (p.mul) {
         const uint2 u = *(const uint2*)(p.mul + (size_t)p.mul_row[row] * p.ldm + col);
-        r.x *= __uint_as_float(u.x << 16); r.y *= __uint_as_float(u.x & 0xffff0000u);
-        r.z *= __uint_as_float(u.y << 16); r.w *= __uint_as_float(u.y & 0xffff0000u);
+        return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
     }
+    return make_float4(0.f, 0.f, 0.f, 0.f);
+}
+
+// Four consecutive sums of a row, as the product's caller wants them: activation or gated pairs, factors, type, accumulation.
+__device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, int col, const float4& with) {
+    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
+    if (p.mul) { r.x *= with.x; r.y *= with.y; r.z *= with.z; r.w *= with.w; }
     if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
         const float h0 = glu_act(r.x, r.y, p.glu - 1, p.glu_alpha, p.glu_limit), h1 = glu_act(r.z, r.w, p.glu - 1, p.glu_alpha, p.glu_limit);
         *(uint32_t*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + (col >> 1)) = pack2_bf16(h0, h1);
@@ -116,11 +124,9 @@ __device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, i
         *(uint2*)((__half*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_f16(r.x, r.y), pack2_f16(r.z, r.w));
     } else {
         float* o = (float*)p.out + (size_t)row * p.ldo + col;
-        if (p.accumulate) {
-            const float4 old = *(const float4*)o;
-            r.x += old.x; r.y += old.y; r.z += old.z; r.w += old.w;
-        }
+        if (p.accumulate) { r.x += with.x; r.y += with.y; r.z += with.z; r.w += with.w; }
         *(float4*)o = r;
+        if (p.copy) *(uint2*)(p.copy + (size_t)row * p.ldo + col) = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
     }
 }
 
@@ -244,13 +250,21 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
             for (int c0 = 0; c0 < BN; c0 += 32) {
                 uint32_t v[32];
                 const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(buf * L::ACC_STRIDE + c0);
+                const int col = n0 + c0 + cq;
+                float4 with[8];
+                if (!SPLIT && (p.accumulate || p.mul)) {
+#pragma unroll
+                    for (int rr = 0; rr < 8; rr++) {
+                        const int row = mt * BM + q * 32 + rr * 4 + sub;
+                        if (row < p.m && col < p.n) with[rr] = fetch4(p, row, col);
+                    }
+                }
                 tmem_ld32(taddr, v);
                 if (n0 + c0 >= p.n) continue;       // warp-uniform
 #pragma unroll
                 for (int j = 0; j < 32; j += 4)
                     *(uint4*)(st + lane * L::EPI_LD + j) = make_uint4(v[j], v[j + 1], v[j + 2], v[j + 3]);
                 __syncwarp();
-                const int col = n0 + c0 + cq;
                 float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (p.bias && col < p.n) bias = *(const float4*)(p.bias + (size_t)e * p.n + col);
 #pragma unroll
@@ -264,7 +278,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                         continue;
                     }
                     r.x += bias.x; r.y += bias.y; r.z += bias.z; r.w += bias.w;
-                    store4(p, r, row, col);
+                    store4(p, r, row, col, with[rr]);
                 }
                 __syncwarp();
             }
@@ -335,11 +349,18 @@ __global__ void __launch_bounds__(256) gemm_parts_kernel(const __grid_constant__
         const float4 b = *(const float4*)(p.bias + col);
         r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
     }
-    store4(p, r, row, col);
+    store4(p, r, row, col, fetch4(p, row, col));
+}
+
+// Products of moderate row length whose narrowest tiles occupy a good part of the machine in one round: quicker whole than split.
+bool narrow(int m, int n, int k) {
+    const long tiles = (long)((m + BM - 1) / BM) * ((n + 63) / 64);
+    return m > 32 && n >= 64 && k <= 2560 && tiles <= sm_count() && 3 * tiles >= sm_count() && 2L * ((m + BM - 1) / BM) * ((n + 127) / 128) <= sm_count();
 }
 
 // How many parts to cut the row length into: a product whose tiles leave most SMs idle, as far as each part keeps some length.
 int split_count(int m, int n, int k) {
+    if (narrow(m, n, k)) return 1;
     const int bn = m <= 32 && n >= 64 && (n + 127) / 128 < sm_count() ? 64 : n >= 128 ? 128 : 64;      // dispatch()'s tile at such sizes
     const long tiles = (long)((m + BM - 1) / BM) * ((n + bn - 1) / bn);
     if (tiles * 2 > sm_count() || k < 1024) return 1;
@@ -378,11 +399,13 @@ B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
         g->out_type > 2 || (g->out_type && g->accumulate) || ((uintptr_t)g->out & (g->out_type ? 7 : 15)) || ((uintptr_t)g->ws & 15) || ((uintptr_t)g->bias & 15))
         return (int)cudaErrorInvalidValue;
     if (glu && (g->out_type != 1 || (n & 7) || g->mul)) return (int)cudaErrorInvalidValue;
-    if (g->mul && (!g->mul_row || (g->ldm & 3) || ((uintptr_t)g->mul & 7))) return (int)cudaErrorInvalidValue;
+    if (g->mul && (!g->mul_row || g->accumulate || (g->ldm & 3) || ((uintptr_t)g->mul & 7))) return (int)cudaErrorInvalidValue;
     if (g->tile_expert && (g->experts < 1 || (m & 127))) return (int)cudaErrorInvalidValue;
+    if (g->copy && (g->out_type || ((uintptr_t)g->copy & 7))) return (int)cudaErrorInvalidValue;
     GemmParams p{m, n, k, g->out, g->ldo, g->bias, g->accumulate, g->out_type, {}, 0, g->tile_expert, glu, SWIGLU_ALPHA, g->limit, glu ? 0 : g->act, g->alpha == 1.f ? 0.f : g->alpha,
-                 (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, g->lda};
+                 (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, (__nv_bfloat16*)g->copy, g->lda};
     if (g->tile_expert) return dispatch(g->a, g->b, p, st, g->experts * n);
+    if (narrow(m, n, k)) return launch<64>(g->a, g->b, p, st);
     const int splits = g->ws ? split_count(m, n, k) : 1;
     if (splits > 1 && (long long)splits * m * n <= g->ws_floats && m <= 65535) {
         p.splits = splits;

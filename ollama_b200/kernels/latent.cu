@@ -10,7 +10,7 @@
 //   latent_merge   the split results of the absorbed form added up and multiplied by V_h (a few rows); latent_reduce and latent_values: the
 //                  same in two launches, the second on the tensor cores with 16 rows at a time
 //   latent_gather  cache rows of whole sequences side by side, for the products of the long form
-//   latent_query   query rows of the long form
+//   latent_rows    cache rows and query rows of the long form
 //
 // Rows: `rows` lists the rows of a step that a launch is for (null: all); results are stored in the order of that list, except
 // where noted.
@@ -33,7 +33,8 @@ struct LatentStepArgs {
     int append;              // write the cache rows
     const void* uk;          // [heads][dim][cp], bf16 or (w32) fp32; null: no queries
     int w32;
-    void* q_out;             // [n][heads][w] in the cache's type
+    void* q_out;             // [n][heads][w] in the cache's type; long form: [n][heads][dp + rp] f16, unrotated part, zeros, rotated part, zeros
+    int dp, rp;              // long form (uk null)
 };
 
 struct LatentMergeArgs {
@@ -56,16 +57,6 @@ struct LatentGatherArgs {
     __nv_bfloat16* c;        // [.][cp]
     __half* r;               // [.][rp] rotated key part, zero-padded
     int rp;
-};
-
-struct LatentQueryArgs {
-    const float* qkv;
-    int ldq, n_heads, dim, rot;
-    const double* freqs;
-    int interleaved;
-    const int* positions;
-    __half* q;               // [rows][heads][dp + rp]: unrotated part, zeros, rotated part, zeros
-    int dp, rp;
 };
 
 namespace {
@@ -189,13 +180,35 @@ __global__ void __launch_bounds__(256) latent_step_kernel(const __grid_constant_
     }
 }
 
-template <typename CT>
-__global__ void __launch_bounds__(128) latent_append_kernel(const __grid_constant__ LatentStepArgs a) {
-    extern __shared__ float sq[];
-    __shared__ float red[4];
+// One CTA per row.
+__global__ void __launch_bounds__(256) latent_rows_kernel(const __grid_constant__ LatentStepArgs a) {
+    extern __shared__ float cs[];
+    __shared__ float red[8];
+    const int i = blockIdx.x, r = a.rows ? a.rows[i] : i, half = a.rot >> 1, dk = a.dp + a.rp, dk2 = dk >> 1;
     pdl_launch();
     pdl_wait();
-    append_row<CT>(a, a.rows ? a.rows[blockIdx.x] : blockIdx.x, nullptr, sq, red);
+    append_row<__half>(a, r, nullptr, cs, red);
+    const float* q = a.qkv + (size_t)r * a.ldq;
+    __half* o = (__half*)a.q_out + (size_t)i * a.n_heads * dk;
+    for (int j = threadIdx.x; j < a.n_heads * dk2; j += 256) {      // two neighbouring values
+        const int h = j / dk2, c = 2 * (j - h * dk2);
+        const float* qh = q + (size_t)h * (a.dim + a.rot);
+        float v[2];
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int d = c + e - a.dp;
+            if (c + e < a.dim) v[e] = qh[c + e];
+            else if (d < 0 || d >= a.rot) v[e] = 0.f;
+            else {
+                const float* t = qh + a.dim;
+                const bool first = a.interleaved ? !(d & 1) : d < half;
+                const int p = a.interleaved ? d >> 1 : (first ? d : d - half);
+                const float y = t[a.interleaved ? d ^ 1 : (first ? d + half : d - half)];
+                v[e] = first ? t[d] * cs[p] - y * cs[half + p] : t[d] * cs[p] + y * cs[half + p];
+            }
+        }
+        *(__half2*)(o + (size_t)h * dk + c) = __floats2half2_rn(v[0], v[1]);
+    }
 }
 
 constexpr int MAX_SPLITS = 128;
@@ -397,35 +410,6 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const __grid_constan
     for (int i = lane; i < a.rp; i += 32) r[i] = i < a.rot ? src[a.cp + i] : __float2half_rn(0.f);
 }
 
-// one CTA per row
-__global__ void __launch_bounds__(256) latent_query_kernel(const __grid_constant__ LatentQueryArgs a) {
-    extern __shared__ float cs[];                  // [rot / 2] cosines, then sines
-    const int r = blockIdx.x, half = a.rot >> 1, pos = a.positions[r], dk = a.dp + a.rp;
-    for (int i = threadIdx.x; i < half; i += 256) sincosf(rot_angle(pos, a.freqs[i]), &cs[half + i], &cs[i]);
-    __syncthreads();
-    const float* q = a.qkv + (size_t)r * a.ldq;
-    __half* o = a.q + (size_t)r * a.n_heads * dk;
-    for (int j = threadIdx.x; j < a.n_heads * (dk >> 1); j += 256) {      // two neighbouring values
-        const int h = j / (dk >> 1), c = 2 * (j - h * (dk >> 1));
-        const float* qh = q + (size_t)h * (a.dim + a.rot);
-        float v[2];
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-            const int i = c + e - a.dp;
-            if (c + e < a.dim) v[e] = qh[c + e];
-            else if (i < 0 || i >= a.rot) v[e] = 0.f;
-            else {
-                const float* t = qh + a.dim;
-                const bool first = a.interleaved ? !(i & 1) : i < half;
-                const int p = a.interleaved ? i >> 1 : (first ? i : i - half);
-                const float y = t[a.interleaved ? i ^ 1 : (first ? i + half : i - half)];
-                v[e] = first ? t[i] * cs[p] - y * cs[half + p] : t[i] * cs[p] + y * cs[half + p];
-            }
-        }
-        *(__half2*)(o + (size_t)h * dk + c) = __floats2half2_rn(v[0], v[1]);
-    }
-}
-
 template <typename CT, typename WT>
 const void* step_fn(int nb) {
     return nb == 1 ? (const void*)latent_step_kernel<CT, WT, 1> : (const void*)latent_step_kernel<CT, WT, 4>;
@@ -433,17 +417,16 @@ const void* step_fn(int nb) {
 
 }  // namespace
 
-// Cache rows (append) and absorbed queries (uk set) of n rows.  Returns a cudaError_t value, as do the entry points below.
+// Cache rows (append) and absorbed queries of n rows; without uk the query rows of the long form (f16 caches).  Returns a cudaError_t value, as do the entry points below.
 B2_API int b2_latent_step(const LatentStepArgs* a, int n, int pdl, cudaStream_t st) {
     if (n < 1 || a->n_heads < 1 || a->dim < 1 || a->rot < 0 || (a->rot & 1) || a->rank < 1 || a->cp < a->rank || (a->cp & 15) || a->w < a->cp + a->rot || (a->rot && !a->freqs) ||
-        (!a->uk && !a->append) || (a->uk && (!a->q_out || ((uintptr_t)a->uk & 15))) || a->dim > 8192 || a->max_pages < 1)
+        !a->q_out || ((uintptr_t)a->uk & 15) || (!a->uk && (a->cache32 || a->dp < a->dim || a->rp < a->rot || (a->dp & 1) || (a->rp & 1))) || a->dim > 8192 || a->max_pages < 1)
         return (int)cudaErrorInvalidValue;
     LatentStepArgs c = *a;
     void* args[] = {&c, &n};
     const size_t angles = (size_t)a->rot * 4;
     if (angles > 32 * 1024) return (int)cudaErrorNotSupported;
-    if (!a->uk)
-        return launch_rows(a->cache32 ? (const void*)latent_append_kernel<float> : (const void*)latent_append_kernel<__half>, dim3(n), dim3(128), angles, args, st, pdl);
+    if (!a->uk) return launch_rows((const void*)latent_rows_kernel, dim3(n), dim3(256), angles, args, st, pdl);
     const int nb = n == 1 ? 1 : 4, parts = (a->cp + COLS - 1) / COLS;
     const void* fn = a->cache32 ? (a->w32 ? step_fn<float, float>(nb) : step_fn<float, __nv_bfloat16>(nb)) : (a->w32 ? step_fn<__half, float>(nb) : step_fn<__half, __nv_bfloat16>(nb));
     const size_t rows = (size_t)nb * a->dim * 4, smem = rows > angles ? rows : angles;
@@ -474,11 +457,5 @@ B2_API int b2_latent_merge(const LatentMergeArgs* a, int n, void* merged, int pd
 B2_API int b2_latent_gather(const LatentGatherArgs* a, int n_seqs, int max_len, cudaStream_t st) {
     if (n_seqs < 1 || n_seqs > 65535 || max_len < 1 || (a->cp & 15) || (a->w & 7) || a->rp < a->rot) return (int)cudaErrorInvalidValue;
     latent_gather_kernel<<<dim3((max_len + 7) / 8, n_seqs), 256, 0, st>>>(*a);
-    return (int)cudaGetLastError();
-}
-
-B2_API int b2_latent_query(const LatentQueryArgs* a, int rows, cudaStream_t st) {
-    if (rows < 1 || a->n_heads < 1 || a->dp < a->dim || a->rp < a->rot || (a->dp & 1) || (a->rp & 1) || (a->rot & 1) || a->rot > 4096) return (int)cudaErrorInvalidValue;
-    latent_query_kernel<<<rows, 256, (size_t)a->rot * 4, st>>>(*a);
     return (int)cudaGetLastError();
 }

@@ -21,9 +21,9 @@ __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log
 // Rotation angle of `pos` at frequency `f`, reduced to one turn: the product is formed in double, so that the angle keeps its
 // 24 bits at any position.
 __device__ __forceinline__ float rot_angle(int pos, double f) {
-    constexpr double TURN = 6.283185307179586476925;
+    constexpr double TURN = 6.283185307179586476925, PER_RADIAN = 1.0 / TURN;
     const double a = (double)pos * f;
-    return (float)(a - TURN * rint(a / TURN));
+    return (float)(a - TURN * rint(a * PER_RADIAN));
 }
 
 // Cache position -> row of a paged cache [page][kv head][64 positions][row length].
@@ -59,6 +59,7 @@ struct GemmRowsArgs {
     // grouped over experts: b holds `experts` stacked [n][k] matrices, the rows of a are sorted by expert and every tile of 128 rows
     // belongs to expert tile_expert[row / 128] (-1: no rows)
     const int* tile_expert;
+    void* copy;               // fp32 results are also stored as bf16 rows of pitch ldo here (bf16 products only), or null
     float* ws;                // scratch for splitting k (bf16 products only), or null
     long long ws_floats;
     int m, n, k, lda, ldb, ldo;

@@ -10,13 +10,11 @@ from .rows import F, I, P, _call, _is32, _st
 
 LatentStepArgs = _st("LatentStepArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("dim", I), ("rot", I), ("rank", I), ("norm", P), ("eps", F), ("freqs", P),
                                         ("interleaved", I), ("rows", P), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I), ("cache", P),
-                                        ("cp", I), ("w", I), ("cache32", I), ("append", I), ("uk", P), ("w32", I), ("q_out", P)])
+                                        ("cp", I), ("w", I), ("cache32", I), ("append", I), ("uk", P), ("w32", I), ("q_out", P), ("dp", I), ("rp", I)])
 LatentMergeArgs = _st("LatentMergeArgs", [("acc", P), ("ml", P), ("n_heads", I), ("splits", I), ("cp", I), ("vdim", I), ("uv", P), ("w32", I), ("rows", P),
                                           ("out", P), ("ldo", I), ("out16", I)])
 LatentGatherArgs = _st("LatentGatherArgs", [("cache", P), ("cp", I), ("w", I), ("rot", I), ("seqs", P), ("page_table", P), ("max_pages", I), ("c", P), ("r", P),
                                             ("rp", I)])
-LatentQueryArgs = _st("LatentQueryArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("dim", I), ("rot", I), ("freqs", P), ("interleaved", I), ("positions", P),
-                                          ("q", P), ("dp", I), ("rp", I)])
 LatentAttnArgs = _st("LatentAttnArgs", [("q", P), ("cache", P), ("rows", P), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I), ("n_heads", I),
                                         ("cp", I), ("w", I), ("splits", I), ("scale", F), ("acc", P), ("ml", P)])
 AttnPartsArgs = _st("AttnPartsArgs", [("q", P), ("kv", P), ("shared", P), ("n_rows", I), ("dp", I), ("vp", I), ("rp", I), ("tiles", P), ("H", I), ("vdim", I),
@@ -38,12 +36,12 @@ def _taken(name: str, args, *more) -> bool:
 
 
 def latent_step(qkv: torch.Tensor, n: int, *, heads: int, dim: int, rot: int, rank: int, norm, eps: float, freqs, interleaved: bool, positions, slots, table,
-                cache: torch.Tensor, cp: int, rows=None, append: bool = True, uk: torch.Tensor | None = None, q_out: torch.Tensor | None = None,
+                cache: torch.Tensor, cp: int, q_out: torch.Tensor, rows=None, append: bool = True, uk: torch.Tensor | None = None, dp: int = 0, rp: int = 0,
                 pdl: bool = False) -> None:
     """Of ``n`` rows: latent and rotated key part into the cache (``append``), and the queries taken into the latent space by ``uk`` [heads, dim, cp] ->
-    ``q_out`` [n, heads, w] in the cache's type."""
+    ``q_out`` [n, heads, w] in the cache's type; without ``uk`` the queries as they are, rotated, each part padded: [n, heads, dp + rp] f16."""
     a = LatentStepArgs(ptr(qkv), qkv.stride(0), heads, dim, rot, rank, ptr(norm), eps, ptr(freqs), int(interleaved), ptr(rows), ptr(positions), ptr(slots), ptr(table),
-                       table.shape[1], ptr(cache), cp, cache.shape[-1], _is32(cache), int(append), ptr(uk), _is32(uk) if uk is not None else 0, ptr(q_out))
+                       table.shape[1], ptr(cache), cp, cache.shape[-1], _is32(cache), int(append), ptr(uk), _is32(uk) if uk is not None else 0, ptr(q_out), dp, rp)
     _call("b2_latent_step", a, n, int(pdl))
 
 
@@ -66,11 +64,6 @@ def latent_gather(cache: torch.Tensor, cp: int, rot: int, seqs: torch.Tensor, ma
     """Positions of whole sequences side by side: latents to bf16 rows ``c``, rotated key parts to ``r``.  ``seqs`` [n, 4] int32: first row, positions, slot, -."""
     a = LatentGatherArgs(ptr(cache), cp, cache.shape[-1], rot, ptr(seqs), ptr(table), table.shape[1], ptr(c), ptr(r), r.shape[1])
     _call("b2_latent_gather", a, seqs.shape[0], max_len)
-
-
-def latent_query(qkv: torch.Tensor, q: torch.Tensor, *, heads: int, dim: int, rot: int, freqs, interleaved: bool, positions, dp: int, rp: int) -> None:
-    a = LatentQueryArgs(ptr(qkv), qkv.stride(0), heads, dim, rot, ptr(freqs), int(interleaved), ptr(positions), ptr(q), dp, rp)
-    _call("b2_latent_query", a, qkv.shape[0])
 
 
 def parts_supported(dp: int, rp: int, vp: int) -> bool:

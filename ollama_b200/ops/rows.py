@@ -27,7 +27,7 @@ NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), 
 JoinRowsArgs = _st("JoinRowsArgs", [("a", P), ("b", P), ("lda", I), ("n_a", I), ("ldb", I), ("n_b", I), ("out", P), ("ldo", I), ("off_b", I), ("f32", I)])
 RowSeg = _st("RowSeg", [("w", P), ("g", P), ("rs", P), ("rc", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I), ("alpha", F),
                         ("limit", F), ("mul", P), ("ldm", I)])
-GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P), ("mul", P), ("mul_row", P), ("tile_expert", P), ("ws", P),
+GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P), ("mul", P), ("mul_row", P), ("tile_expert", P), ("copy", P), ("ws", P),
                                     ("ws_floats", C.c_longlong), ("m", I), ("n", I), ("k", I), ("lda", I), ("ldb", I), ("ldo", I), ("out_type", I), ("act", I),
                                     ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
@@ -113,19 +113,22 @@ def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC
 
 def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", accumulate: bool = False, k: int | None = None, alpha: float = 1.0,
          limit: float = math.inf, bias: torch.Tensor | None = None, mul: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
-         experts: int = 0, tile_expert: torch.Tensor | None = None) -> None:
+         experts: int = 0, tile_expert: torch.Tensor | None = None, copy: torch.Tensor | None = None) -> None:
     """out (+)= alpha * act(a[:, :k] @ w[:, :k]^T + bias) [* mul[mul_row]]; bf16 operands on tcgen05 (result bf16, f16 or fp32), fp32 operands in full
-    32 bits.  ``a``, ``out`` and ``mul`` may be column windows of wider buffers.  Gated activations ("glu:...") halve the columns.  ``experts``: w holds
+    32 bits.  ``copy``: bf16 rows of out's pitch that receive an fp32 result too.
+    ``a``, ``out`` and ``mul`` may be column windows of wider buffers.  Gated activations ("glu:...") halve the columns.  ``experts``: w holds
     that many stacked matrices and a's tiles of 128 rows belong to ``tile_expert``."""
     n = w.shape[0] // max(experts, 1)
     m, k = a.shape[0], w.shape[1] if k is None else k
     cols = n // 2 if act.startswith("glu:") else n
     if a.dtype != w.dtype or out.shape[0] != m or out.shape[1] != cols or a.shape[1] < k or a.stride(1) != 1 or out.stride(1) != 1:
         raise ValueError(f"gemm: {tuple(a.shape)} {a.dtype} x {tuple(w.shape)} {w.dtype} -> {tuple(out.shape)}")
+    if copy is not None and (copy.stride(0) != out.stride(0) or copy.shape != out.shape or copy.dtype != torch.bfloat16):
+        raise ValueError(f"gemm: copy {tuple(copy.shape)} {copy.dtype}")
     f32 = a.dtype == torch.float32
     size = 0 if f32 or experts else _split_floats(m, n, k)
     ws = torch.empty(size, device=a.device) if size else None
-    g = GemmRowsArgs(ptr(a), ptr(w), ptr(out), ptr(bias), ptr(mul), ptr(mul_row), ptr(tile_expert), ptr(ws), size, m, n, k, a.stride(0), w.stride(0), out.stride(0),
+    g = GemmRowsArgs(ptr(a), ptr(w), ptr(out), ptr(bias), ptr(mul), ptr(mul_row), ptr(tile_expert), ptr(copy), ptr(ws), size, m, n, k, a.stride(0), w.stride(0), out.stride(0),
                      OUT_TYPE[out.dtype], ACT[act], int(accumulate), experts, mul.stride(0) if mul is not None else 0, alpha, limit)
     _call("b2_gemm_rows_f32" if f32 else "b2_gemm_rows", g)
 

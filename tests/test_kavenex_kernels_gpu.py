@@ -115,8 +115,10 @@ def test_products_of_many_rows(ops, m, n, k, f32):
         close(out, 1.7 * O.gelu_tanh(p) * table[tok.long()].double(), tol if t != torch.float32 else 2e-5)
     acc = rnd(m, n, seed=9)
     want = acc.double() + 0.4 * p
-    R.gemm(a, w, acc, bias=bias, accumulate=True, alpha=0.4)
+    copy = None if f32 else torch.zeros(m, n, device="cuda", dtype=dt)
+    R.gemm(a, w, acc, bias=bias, accumulate=True, alpha=0.4, copy=copy)
     close(acc, want, 2e-5)
+    assert f32 or torch.equal(copy, acc.to(dt))
     if n % 8 == 0:
         h = torch.zeros(m, n // 2, device="cuda", dtype=dt)
         R.gemm(a, w, h, bias=bias, act="glu:gelu_tanh")
@@ -273,6 +275,15 @@ def test_absorbed_queries_and_cache_rows(ops, rank, cache32):
             close(got[:, cp:cp + rot], turn(k)[:, 0], tol)
             assert (got[:, rank:cp] == 0).all() and (got[:, cp + rot:] == 0).all() and (q[..., cp + rot:] == 0).all()
             assert int((cache != 7.0).any(-1).sum()) == n                       # nothing else was written
+            if not cache32:                                                     # the long form: queries as they are, the same cache rows
+                again, dp, rp = torch.full_like(cache, 7.0), 24, 10
+                q = torch.full((n, H, dp + rp), 9.0, device="cuda", dtype=torch.float16)
+                A.latent_step(qkv, n, heads=H, dim=d, rot=rot, rank=rank, norm=norm, eps=eps, freqs=freqs, interleaved=inter, positions=pos, slots=slots, table=table,
+                              cache=again, cp=cp, q_out=q, dp=dp, rp=rp)
+                assert torch.equal(again, cache)
+                close(q[..., :d], qs[..., :d], tol)
+                close(q[..., dp:dp + rot], turn(qs[..., d:]), tol)
+                assert (q[..., d:dp] == 0).all() and (q[..., dp + rot:] == 0).all()
 
 
 @pytest.mark.parametrize("heads,dim,rot,vdim", [(2, 20, 8, 28), (3, 128, 64, 128), (1, 64, 64, 100), (4, 100, 40, 64), (2, 64, 0, 64)])

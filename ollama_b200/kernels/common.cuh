@@ -86,36 +86,41 @@ __device__ __forceinline__ float e8m0_to_float(uint32_t e) {
 // tanh through one exponential and one quotient of the special-function unit; absolute error about 2^-22 (soft caps of attention scores).
 __device__ __forceinline__ float tanh_exp(float x) { return 1.f - __fdividef(2.f, __expf(2.f * x) + 1.f); }
 
+// Tanh form of gelu: v (1 + tanh z) / 2 = v / (1 + exp(-2 z)).  EXACT: with the math library's exponential (32-bit models).
+template <bool EXACT = false>
 __device__ __forceinline__ float gelu_tanh_f(float v) {
-    return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+    const float z2 = -1.5957691216057308f * (v + 0.044715f * v * v * v);
+    return EXACT ? v / (1.f + expf(z2)) : __fdividef(v, 1.f + __expf(z2));
 }
 
 // Activation of single values in a matrix product's epilogue: 0 none, 1 square of relu, 2 tanh form of gelu.
+template <bool EXACT = false>
 __device__ __forceinline__ float out_act(float v, int act) {
     if (act == 1) {
         const float r = fmaxf(v, 0.f);
         return r * r;
     }
-    return act == 2 ? gelu_tanh_f(v) : v;
+    return act == 2 ? gelu_tanh_f<EXACT>(v) : v;
 }
 
 // Epilogue activations of products whose rows 2i / 2i + 1 are gate / up of output i: GLU_BASE + the number glu_act takes.
 constexpr int GLU_BASE = 16;
 constexpr float SWIGLU_ALPHA = 1.702f;
 
+// The quotients below are the special-function unit's: an IEEE division there made epilogues of wide products twice as long as their matrix part.
 // Gated FFN activation: 0 = SiLU(g) * u, 1 = tanh-GELU(g) * u, 2 = clamped SwiGLU with alpha and limit (gpt-oss).
 __device__ __forceinline__ float glu_act(float g, float u, int act, float alpha, float limit) {
-    if (act == 0) return g / (1.f + __expf(-g)) * u;
+    if (act == 0) return __fdividef(g, 1.f + __expf(-g)) * u;
     if (act == 1) return gelu_tanh_f(g) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
-    return g / (1.f + __expf(-alpha * g)) * (u + 1.f);
+    return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
 }
 
 // The same with the exponentials of the math library: 32-bit models.
 __device__ __forceinline__ float glu_act_exact(float g, float u, int act, float alpha, float limit) {
     if (act == 0) return g / (1.f + expf(-g)) * u;
-    if (act == 1) return gelu_tanh_f(g) * u;
+    if (act == 1) return gelu_tanh_f<true>(g) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + expf(-alpha * g)) * (u + 1.f);

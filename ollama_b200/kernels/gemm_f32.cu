@@ -73,7 +73,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
             const int col = n0 + 4 * tx + j;
             if (col >= p.n) continue;
             float* o = (float*)p.out + (size_t)row * p.ldo + col;
-            float r = out_act(v[j], p.act);
+            float r = out_act<true>(v[j], p.act);
             if (p.mul) r *= ((const float*)p.mul)[(size_t)p.mul_row[row] * p.ldm + col];
             r *= p.alpha;
             *o = p.accumulate ? *o + r : r;

@@ -239,6 +239,10 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
             if (e < 0) continue;
             const int buf = i & 1, use = i >> 1;
             i++;
+            if (!SPLIT && p.mul && mt * BM + q * 32 + lane < p.m) {      // the table's rows are anywhere in memory: asked for while the products run
+                const __nv_bfloat16* r = p.mul + (size_t)p.mul_row[mt * BM + q * 32 + lane] * p.ldm;
+                for (int c = nt * BN; c < min(nt * BN + BN, p.n); c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(r + c));
+            }
             if (!mbar_wait(&acc_full[buf], use & 1)) { ok = false; break; }
             tc_fence_after();
             // Each thread reads 32 columns of its own accumulator row; a 32 x 32 transpose through shared memory turns that into

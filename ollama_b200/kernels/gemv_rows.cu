@@ -233,7 +233,7 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
         return;
     }
     if (mine) {
-        v = out_act(v, w.act);
+        v = out_act<F32>(v, w.act);
         if (w.mul) {
             const size_t m = (size_t)a.mul_row[b] * w.ldm + row;
             v *= F32 ? ((const float*)w.mul)[m] : __bfloat162float(((const __nv_bfloat16*)w.mul)[m]);

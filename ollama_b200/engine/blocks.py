@@ -151,7 +151,7 @@ class Step:
         h = self.buf("h", be.wp) if keep or not self.folded else None
         if self.folded:
             self.flush()
-            O.gemv([O.seg(mat.w, mat.w.shape[0], out, norm.g, rs=mat.rs, rc=mat.rc, **kw)], be.wp, self.x, self.nb, False, O.SRC_NORM, st.eps, st.width, layer=True, h=h,
+            O.gemv([O.seg(mat.w, mat.w.shape[0], out, norm.g, rs=mat.rs, rc=mat.rc, **kw)], be.wp, self.x, self.nb, False, O.SRC_LAYER, st.eps, st.width, h=h,
                    hb=norm.b, pdl=self.pdl)
             self.launched()
             return h

@@ -447,7 +447,7 @@ class StackBackend(StepEngine):
         if isinstance(self.out_norm, Norm):
             if nb <= self.gemv_rows and not self.f32:
                 m = self.out_mat
-                O.gemv([O.seg(m.w, m.w.shape[0], out, self.out_norm.g, rs=m.rs, rc=m.rc)], self.wp, x, nb, False, O.SRC_NORM, st.eps, st.width, layer=True, pdl=pdl)
+                O.gemv([O.seg(m.w, m.w.shape[0], out, self.out_norm.g, rs=m.rs, rc=m.rc)], self.wp, x, nb, False, O.SRC_LAYER, st.eps, st.width, pdl=pdl)
             else:
                 h = torch.empty(nb, self.wp, device=self.device, dtype=self.act_dtype)
                 O.norm_rows(x, st.width, st.eps, self.out_norm.g, h, b1=self.out_norm.b, pdl=pdl)

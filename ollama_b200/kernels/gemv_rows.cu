@@ -1,11 +1,12 @@
 // Matrix-vector products of decode steps over unquantised weights (bf16, or fp32 for 32-bit models), 1..4 rows, with what
 // surrounds them in a layer fused in, sm_100a.
 //
-// Up to four matrices share one launch and one source row.  The source is read in one of three ways:
+// Up to four matrices share one launch and one source row.  The source is read in one of four ways:
 //   rows     fp32 activations as they are;
 //   norm     RMS-normalised: every segment has a norm weight of its own (branches of a parallel block), the weight is multiplied
-//            into the row while the dot products run and the row's 1 / rms, which every CTA computes, into the results.  A layer norm
-//            also subtracts mean times the matrix row's weighted sum and adds the row's product with the bias, both made at load;
+//            into the row while the dot products run and the row's 1 / rms, which every CTA computes, into the results;
+//   layer    layer-normalised: the same, and the results less mean times the matrix row's weighted sum, plus the row's product with the
+//            bias, both made at load;
 //   joined   two rows side by side;
 // The epilogue applies an activation (of single rows, or of gate / up pairs), a factor, and stores or accumulates (the residual add).  The first rows of one matrix may also run
 // through a causal depthwise convolution + SiLU with the slot's last inputs (the state is only read here: the kernel that advances the
@@ -28,7 +29,9 @@ struct RowSeg {
     int ldm;
 };
 
-enum RowSrc : int { SRC_ROWS = 0, SRC_NORM = 1, SRC_JOINED = 2 };
+enum RowSrc : int { SRC_ROWS = 0, SRC_NORM = 1, SRC_JOINED = 2, SRC_LAYER = 3 };
+
+__host__ __device__ constexpr bool norm_source(int src) { return src == SRC_NORM || src == SRC_LAYER; }
 
 struct GemvRowsArgs {
     RowSeg seg[4];
@@ -49,8 +52,7 @@ struct GemvRowsArgs {
     int ldu;
     const int* slots;
     const int* positions;         // 0: the state counts as zeros
-    // norm source: layer norm instead of RMS norm, and the normalised row of matrix 0 as a result of its own (h = null: none)
-    int layer;
+    // norm sources: the normalised row of matrix 0 as a result of its own (h = null: none)
     float* h;                     // [nb][ldh], k columns
     int ldh;
     const float* hb;              // [k] layer norm's bias
@@ -64,7 +66,7 @@ constexpr int R = 4;
 template <int NB, int SRC>
 __device__ __forceinline__ void source8(const GemvRowsArgs& a, const float* g, int col, float (&x)[NB][8]) {
     float gv[8];
-    if (SRC == SRC_NORM) {
+    if (norm_source(SRC)) {
         *(float4*)gv = __ldg((const float4*)(g + col));
         *(float4*)(gv + 4) = __ldg((const float4*)(g + col + 4));
     }
@@ -75,7 +77,7 @@ __device__ __forceinline__ void source8(const GemvRowsArgs& a, const float* g, i
         if (SRC == SRC_JOINED && col >= a.k1) p = a.x2 + (size_t)bb * a.ldx2 + col - a.k1;
         *(float4*)x[b] = *(const float4*)p;
         *(float4*)(x[b] + 4) = *(const float4*)(p + 4);
-        if (SRC == SRC_NORM) {
+        if (norm_source(SRC)) {
 #pragma unroll
             for (int i = 0; i < 8; i++) x[b][i] *= gv[i];
         }
@@ -111,7 +113,7 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
         }
     }
     pdl_wait();
-    if (SRC == SRC_NORM) {
+    if (norm_source(SRC)) {
 #pragma unroll
         for (int b = 0; b < NB; b++) {
             const float* x = a.x + (size_t)(b < a.nb ? b : 0) * a.ldx;
@@ -119,13 +121,13 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
             for (int i = 4 * threadIdx.x; i < a.k; i += 1024) {      // columns beyond the true length are zero
                 const float4 v = *(const float4*)(x + i);
                 ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-                sm += v.x + v.y + v.z + v.w;
+                if (SRC == SRC_LAYER) sm += v.x + v.y + v.z + v.w;
             }
             ss = warp_sum(ss);
-            if (a.layer) sm = warp_sum(sm);
+            if (SRC == SRC_LAYER) sm = warp_sum(sm);
             if (lane == 0) {
                 s_ss[warp][b] = ss;
-                s_sm[warp][b] = sm;
+                if (SRC == SRC_LAYER) s_sm[warp][b] = sm;
             }
         }
     }
@@ -197,12 +199,12 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
 #pragma unroll
         for (int i = 0; i < 8; i++) {
             ss += s_ss[i][b];
-            sm += s_sm[i][b];
+            if (SRC == SRC_LAYER) sm += s_sm[i][b];
         }
-        mean = a.layer ? sm / (float)a.kn : 0.f;
-        inv = 1.f / sqrtf(fmaxf(ss / (float)a.kn - mean * mean, 0.f) + a.eps);
+        mean = SRC == SRC_LAYER ? sm / (float)a.kn : 0.f;
+        inv = 1.f / sqrtf((SRC == SRC_LAYER ? fmaxf(ss / (float)a.kn - mean * mean, 0.f) : ss / (float)a.kn) + a.eps);
     };
-    if (SRC == SRC_NORM && a.h) {          // a slice of the normalised rows per CTA
+    if (norm_source(SRC) && a.h) {          // a slice of the normalised rows per CTA
         for (int i = blockIdx.x * 256 + threadIdx.x; i < a.nb * a.k; i += gridDim.x * 256) {
             const int b = i / a.k, c = i - b * a.k;
             float mean, inv;
@@ -217,10 +219,10 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
     if (mine) {
 #pragma unroll
         for (int k2 = 0; k2 < KS; k2++) v += red[rg * KS + k2][lane];
-        if (SRC == SRC_NORM) {
+        if (norm_source(SRC)) {
             float mean, inv;
             row_stats(b, mean, inv);
-            v = a.layer ? (v - mean * w.rs[row]) * inv : v * inv;
+            v = SRC == SRC_LAYER ? (v - mean * w.rs[row]) * inv : v * inv;
         }
         if (w.rc) v += w.rc[row];
     }
@@ -268,6 +270,7 @@ template <bool F32>
 const void* pick_src(int src, int nb, int ks) {
     switch (src) {
         case SRC_NORM: return pick_nb<SRC_NORM, F32>(nb, ks);
+        case SRC_LAYER: return pick_nb<SRC_LAYER, F32>(nb, ks);
         case SRC_JOINED: return pick_nb<SRC_JOINED, F32>(nb, ks);
         default: return pick_nb<SRC_ROWS, F32>(nb, ks);
     }
@@ -277,26 +280,27 @@ const void* pick_src(int src, int nb, int ks) {
 
 // Returns a cudaError_t value.
 B2_API int b2_gemv_rows(const GemvRowsArgs* a, int pdl, cudaStream_t st) {
-    if (a->nb < 1 || a->nb > 4 || a->nseg < 1 || a->nseg > 4 || a->k < 8 || (a->k & 7) || !a->x || (a->ldx & 3) || ((uintptr_t)a->x & 15) || a->src < 0 || a->src > 2)
+    if (a->nb < 1 || a->nb > 4 || a->nseg < 1 || a->nseg > 4 || a->k < 8 || (a->k & 7) || !a->x || (a->ldx & 3) || ((uintptr_t)a->x & 15) || a->src < 0 || a->src > SRC_LAYER)
         return (int)cudaErrorInvalidValue;
     if (a->src == SRC_JOINED && (!a->x2 || (a->ldx2 & 3) || ((uintptr_t)a->x2 & 15) || (a->k1 & 7))) return (int)cudaErrorInvalidValue;
     if (a->conv_seg >= 0 && (a->conv_seg >= a->nseg || a->conv_n < 1 || a->conv_n > a->seg[a->conv_seg].n || a->taps < 1 || !a->conv_w || !a->conv_b || !a->conv_state ||
                              !a->conv_out || !a->slots || !a->positions))
         return (int)cudaErrorInvalidValue;
-    if (a->h && a->src != SRC_NORM) return (int)cudaErrorInvalidValue;
+    if (a->h && !norm_source(a->src)) return (int)cudaErrorInvalidValue;
     long groups = 0;
     for (int s = 0; s < a->nseg; s++) {
         const RowSeg& w = a->seg[s];
-        if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (a->src == SRC_NORM && (!w.g || ((uintptr_t)w.g & 15) || (a->layer && !w.rs))) ||
+        if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (norm_source(a->src) && (!w.g || ((uintptr_t)w.g & 15) || (a->src == SRC_LAYER && !w.rs))) ||
             w.act < 0 || (w.act > 2 && w.act < GLU_BASE) || w.act > GLU_BASE + 2 || (w.act >= GLU_BASE && ((w.n & 1) || w.mul)) || (w.mul && !a->mul_row))
             return (int)cudaErrorInvalidValue;
         groups += (w.n + R - 1) / R;
     }
     // Split the row length over KS warps until there are warps enough for the loads in flight, as far as a lane keeps two pieces; and long
-    // rows further, down to eight pieces a lane (sweep over 2048 .. 11008 columns and 2048 .. 32768 rows).
+    // rows further, down to four to eight pieces a lane (sweep over 2048 .. 11008 columns and 2048 .. 32768 rows).
+    const int pieces = a->k >> 3, enough = a->nb <= 2 && pieces >= 512 ? 4 : 8;
     const long want = a->nb == 2 ? 3600 : 1800;
     int ks = 1;
-    while (ks < 8 && ((groups * ks < want && (a->k >> 3) / (64 * ks) >= 1) || (a->k >> 3) / (64 * ks) >= 8)) ks <<= 1;
+    while (ks < 8 && ((groups * ks < want && pieces / (64 * ks) >= 1) || pieces / (64 * ks) >= enough)) ks <<= 1;
     const int rgs = 8 / ks;
     GemvRowsArgs copy = *a;
     void* args[] = {&copy};

@@ -14,7 +14,7 @@ P, I, F = C.c_void_p, C.c_int, C.c_float
 GLU_BASE = 16
 ACT = {"": 0, "relu2": 1, "gelu_tanh": 2, "glu:silu": GLU_BASE, "glu:gelu_tanh": GLU_BASE + 1, "glu:swiglu_oai": GLU_BASE + 2}
 OUT_TYPE = {torch.float32: 0, torch.bfloat16: 1, torch.float16: 2}
-SRC_ROWS, SRC_NORM, SRC_JOINED = range(3)
+SRC_ROWS, SRC_NORM, SRC_JOINED, SRC_LAYER = range(4)
 GEMV_MAX_ROWS = 4
 
 
@@ -33,7 +33,7 @@ GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P),
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
                                     ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
                                     ("conv_b", P), ("conv_state", P), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
-                                    ("layer", I), ("h", P), ("ldh", I), ("hb", P), ("mul_row", P)])
+                                    ("h", P), ("ldh", I), ("hb", P), ("mul_row", P)])
 PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
                                           ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
                                           ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I)])
@@ -90,16 +90,16 @@ def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = Non
 
 def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,
          k1: int = 0, conv=None, conv_out: torch.Tensor | None = None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None,
-         layer: bool = False, h: torch.Tensor | None = None, hb: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
+         h: torch.Tensor | None = None, hb: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
          pdl: bool = False) -> None:
     """Products of up to four matrices with up to four source rows.  ``conv`` = (weights [taps, n], bias [n], state [slots, taps - 1, n]): the first n
-    results of the first matrix also run through that convolution and SiLU, into ``conv_out``.  ``layer``: the norm source is a layer norm;
-    ``h``: its rows for the first matrix are stored too (``hb``: the norm's bias)."""
+    results of the first matrix also run through that convolution and SiLU, into ``conv_out``.  ``h``: the normalised
+    rows for the first matrix are stored too (``hb``: a layer norm's bias)."""
     a = GemvRowsArgs()
     for i, s in enumerate(segs):
         a.seg[i] = s
     a.nseg, a.nb, a.k, a.src, a.f32, a.x, a.ldx, a.eps, a.kn, a.conv_seg = len(segs), nb, k, src, int(f32), ptr(x), x.stride(0), eps, kn, -1
-    a.layer, a.mul_row = int(layer), ptr(mul_row)
+    a.mul_row = ptr(mul_row)
     if h is not None:
         a.h, a.ldh, a.hb = ptr(h), h.stride(0), ptr(hb)
     if x2 is not None:

@@ -71,12 +71,12 @@ def test_decode_product_with_folded_layer_norm(ops, nb, k, n):
     h64 = O.layer_norm(x[:, :k].double(), g[:k].double(), b[:k].double(), eps)
     want = h64 @ w[:, :k].double().t() + bias.double()
     out, h = torch.zeros(nb, n).cuda(), torch.full((nb, kp), 9.0, device="cuda")
-    R.gemv([R.seg(w, n, out, g, rs=rs, rc=rc)], kp, x, nb, False, R.SRC_NORM, eps, k, layer=True, h=h, hb=b)
+    R.gemv([R.seg(w, n, out, g, rs=rs, rc=rc)], kp, x, nb, False, R.SRC_LAYER, eps, k, h=h, hb=b)
     close(out, want, 2e-5)
     close(h[:, :k], h64, 1e-5)
     assert (h[:, k:] == 0).all()
     gu = torch.zeros(nb, n // 2).cuda()
-    R.gemv([R.seg(w, n, gu, g, act="glu:gelu_tanh", rs=rs, rc=rc)], kp, x, nb, False, R.SRC_NORM, eps, k, layer=True)
+    R.gemv([R.seg(w, n, gu, g, act="glu:gelu_tanh", rs=rs, rc=rc)], kp, x, nb, False, R.SRC_LAYER, eps, k)
     close(gu, O.gelu_tanh(want[:, 0::2]) * want[:, 1::2], 3e-5)
 
 

@@ -306,7 +306,7 @@ def latent_config(width: int, heads: int, dim: int, rot: int, vdim: int, rank: i
 
 
 STACK_SPECS: dict[str, dict] = {
-    "tiny-kavenex": latent_config(256, 4, 64, 32, 64, 128, 512, 4096, "DED", (0, 2, 2), 32, 8, 2, 128, 128),
+    "tiny-kavenex": latent_config(192, 6, 40, 24, 48, 80, 384, 4096, "DED", (1, 3, 2), 24, 6, 2, 96, 64),
     "kavenex-1b": latent_config(2048, 16, 128, 64, 128, 512, 5504, 32768, "D" * 16, (0, 4, 2), 256),
     "kavenex-8b": latent_config(4096, 32, 128, 64, 128, 512, 11008, 128256, "D" * 28, (0, 4, 2), 256),
     "kavenex-moe": latent_config(2048, 16, 128, 64, 128, 512, 0, 32768, "E" * 16, (0, 4, 2), 256, 64, 4, 1408, 1408),

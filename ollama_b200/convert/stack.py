@@ -29,10 +29,13 @@ _LAYER = {
     "mlp.router": "ffn_gate_inp.weight", "mlp.router.b": "ffn_gate_inp.bias",
     "mlp.shared.gate": "ffn_gate_shexp.weight", "mlp.shared.up": "ffn_up_shexp.weight", "mlp.shared.down": "ffn_down_shexp.weight",
     "side.gate": "inp_gate.weight", "side.proj": "proj.weight", "side.norm": "post_norm.weight",
+    "norm1b": "post_attention_norm.weight", "norm2b": "post_ffw_norm.weight", "mix.g": "attn_gate.weight", "mix.q.b": "attn_q.bias", "mix.k.b": "attn_k.bias",
+    "mix.q.conv": "attn_q_conv1d.weight", "mix.k.conv": "attn_k_conv1d.weight", "mix.v.conv": "attn_v_conv1d.weight",
+    "mix.dt_bias": "ssm_dt.bias", "mix.norm": "ssm_norm.weight", "mlp.correction": "exp_probs_b.bias", "mlp.shared.sg": "ffn_gate_inp_shexp.weight",
 }
 _EXPERT = re.compile(r"l(\d+)\.mlp\.e(\d+)\.(gate|up|down)")
-_ONE_PLUS = ("attn_norm.weight", "ffn_norm.weight", "output_norm.weight")
-_F32 = ("ssm_a", "ssm_d", "ssm_conv1d.weight", "ssm_conv1d.bias", "ssm_dt.bias")
+_ONE_PLUS = ("attn_norm.weight", "ffn_norm.weight", "output_norm.weight", "post_attention_norm.weight", "post_ffw_norm.weight")
+_F32 = ("ssm_a", "ssm_d", "conv1d.weight", "ssm_conv1d.bias", "ssm_dt.bias")
 
 
 def is_stack_config(cfg: dict[str, Any]) -> bool:
@@ -77,7 +80,7 @@ def map_stack_name(name: str, cfg: dict[str, Any]) -> str | None:
         return None
     rest = m.group(2)
     if rest == "mix.o":
-        return f"blk.{m.group(1)}.{'ssm_out' if cfg['layers'][int(m.group(1))]['type'] == 'mamba1' else 'attn_output'}.weight"
+        return f"blk.{m.group(1)}.{'ssm_out' if cfg['layers'][int(m.group(1))]['type'].startswith('mamba') else 'attn_output'}.weight"
     e = _EXPERT.fullmatch(name)
     if e:
         router = (cfg["layers"][int(e.group(1))].get("mlp") or {}).get("router") or {}

@@ -1,5 +1,5 @@
-"""Mixers and feed-forwards of stack models that run one after the other inside a layer (engine/stack.py): latent attention, gated and
-mixture-of-experts feed-forwards, inputs of a layer's own per token.
+"""Parts of stack models' layers that run one after the other (engine/stack.py): latent attention, gated and mixture-of-experts feed-forwards,
+inputs of a layer's own per token.  Further mixers are in engine/mixers.py.
 
 Each class holds a layer's weights, laid out for the kernels, and adds its result to the residual rows of a :class:`Step`.
 """
@@ -65,9 +65,9 @@ class WeightSource:
 
 @dataclass
 class Norm:
-    """Layer norm."""
+    """Layer norm, or without a bias an RMS norm."""
     g: torch.Tensor
-    b: torch.Tensor
+    b: torch.Tensor | None
 
 
 @dataclass
@@ -86,8 +86,8 @@ class Mat:
         return self
 
 
-def make_norm(src: WeightSource, name: str) -> Norm:
-    return Norm(src.vec(name + ".weight", src.width), src.vec(name + ".bias", src.width))
+def make_norm(src: WeightSource, name: str, kind: str = "layer") -> Norm:
+    return Norm(src.vec(name + ".weight", src.width), src.vec(name + ".bias", src.width) if kind == "layer" else None)
 
 
 @dataclass
@@ -145,19 +145,37 @@ class Step:
             kw["copy"] = self.copy = self.buf("copy", self.be.wp)
         self.product(h, mat, self.x, accumulate=True, alpha=self.be.stack.residual_mult, **kw)
 
+    def rows(self, norm: Norm) -> torch.Tensor:
+        """norm(x), after what is pending."""
+        h = self.buf("h", self.be.wp)
+        O.norm_rows(self.x, self.be.stack.width, self.be.stack.eps, norm.g, h, b1=norm.b, pdl=self.pdl, **self.pending)
+        self.pending = {}
+        self.launched()
+        return h
+
+    def result(self, h: torch.Tensor, mat: Mat, post: Norm | None) -> None:
+        """Adds mat h to the stream, under the norm ``post`` where there is one."""
+        if post is None:
+            self.add(h, mat)
+            return
+        y = self.buf("y", self.be.wp, torch.float32)
+        self.product(h, mat, y)
+        self.leave(y, post)
+
+    def leave(self, y: torch.Tensor, post: Norm) -> None:
+        self.pending = {"y": y, "wy": post.g, "mult": self.be.stack.residual_mult}
+
     def normed(self, norm: Norm, mat: Mat, out: torch.Tensor, keep: bool = False, **kw) -> torch.Tensor | None:
         """out = f(mat norm(x) + bias); returns the normalised rows where they exist (always with ``keep``)."""
         be, st = self.be, self.be.stack
-        h = self.buf("h", be.wp) if keep or not self.folded else None
-        if self.folded:
+        if self.folded and norm.b is not None:
+            h = self.buf("h", be.wp) if keep else None
             self.flush()
             O.gemv([O.seg(mat.w, mat.w.shape[0], out, norm.g, rs=mat.rs, rc=mat.rc, **kw)], be.wp, self.x, self.nb, False, O.SRC_LAYER, st.eps, st.width, h=h,
                    hb=norm.b, pdl=self.pdl)
             self.launched()
             return h
-        O.norm_rows(self.x, st.width, st.eps, norm.g, h, b1=norm.b, pdl=self.pdl, **self.pending)
-        self.pending = {}
-        self.launched()
+        h = self.rows(norm)
         self.product(h, mat, out, **kw)
         return h
 
@@ -277,13 +295,16 @@ class _Shared:
 
 
 class ExpertFFN:
-    """Mixture of experts; the experts stand stacked in one matrix each for gate / up and down."""
-    ACT = "glu:swiglu_oai"
+    """Mixture of experts; the experts stand stacked in one matrix each for gate / up and down.  The router's last row is the shared expert's gate where it has one."""
 
-    def __init__(self, src: WeightSource, p: str, m: ExpertMLP, norm: Norm, f32: bool):
-        w, E = src.width, m.experts
-        self.m, self.norm, self.ffp = m, norm, up(m.expert.ff)
-        self.router = Mat(src.pack([(0, 0, p + "ffn_gate_inp.weight", (E, w))], up(E), src.wp), bias=src.vec(p + "ffn_gate_inp.bias", E))
+    def __init__(self, src: WeightSource, p: str, m: ExpertMLP, norm: Norm, f32: bool, post: Norm | None = None):
+        w, E, n = src.width, m.experts, m.outputs
+        self.m, self.norm, self.post, self.ffp, self.act = m, norm, post, up(m.expert.ff), "glu:" + m.act
+        parts = [(0, 0, p + "ffn_gate_inp.weight", (n, w))]
+        if m.shared is not None and m.shared_gate:
+            parts.append((n, 0, p + "ffn_gate_inp_shexp.weight", (1, w)))
+        self.router = Mat(src.pack(parts, up(n + len(parts) - 1), src.wp), bias=src.vec(p + "ffn_gate_inp.bias", E) if m.router_bias else None)
+        self.correction = src.vec(p + "exp_probs_b.bias", n) if m.correction else None
         self.gu = src.gate_up(p + "ffn_gate_exps.weight", p + "ffn_up_exps.weight", m.expert.ff, (E,))
         self.down = src.zeros(E, src.wp, self.ffp)
         self.down[:, :w, :m.expert.ff] = src.tensor(p + "ffn_down_exps.weight", E, w, m.expert.ff)
@@ -292,39 +313,51 @@ class ExpertFFN:
             ff = m.shared.ff
             self.shared = _Shared(m.shared, Mat(src.gate_up(p + "ffn_gate_shexp.weight", p + "ffn_up_shexp.weight", ff)),
                                   Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff))))
-        if not f32:
+        if not f32 and norm.b is not None:
             self.router.fold(norm)
 
     def product_weights(self) -> tuple[int, int, float]:
         sh = self.shared
-        return (self.router.w.numel() + (sh.gu.w.numel() + sh.down.w.numel() if sh else 0), self.gu.numel() + self.down.numel(), self.m.top / self.m.experts)
+        return (self.router.w.numel() + (sh.gu.w.numel() + sh.down.w.numel() if sh else 0), self.gu.numel() + self.down.numel(), self.m.top / self.m.outputs)
 
     def run(self, s: Step) -> None:
-        m, sh = self.m, self.shared
+        m, sh, post, mult = self.m, self.shared, self.post, s.be.stack.residual_mult
         z = s.buf("router", self.router.w.shape[0], torch.float32)
         h = s.normed(self.norm, self.router, z, keep=True)
+        gate = z[:, m.outputs:m.outputs + 1] if sh and m.shared_gate else None
+        out = s.x if post is None else s.buf("y", s.be.wp, torch.float32)
+        if post is not None:
+            mult = 1.0
         if s.small:
             sfp = up(sh.e.ff) if sh else 0
             a = s.buf("experts", m.top * self.ffp + sfp, zero=True)
             ids, wts = s.buf("ids", m.top, torch.int32), s.buf("weights", m.top)
-            A.moe_up_rows(z, h, s.nb, self.gu, 2 * m.expert.ff, a, ids, wts, experts=m.experts, top=m.top, ffp=self.ffp, limit=m.expert.limit,
-                          ws=sh.gu.w if sh else None, ns=2 * sh.e.ff if sh else 0, limit_s=sh.e.limit if sh else math.inf, pdl=s.pdl)
-            A.moe_down_rows(a, s.nb, ids, wts, self.down, s.x, top=m.top, n=s.be.stack.width, mult=s.be.stack.residual_mult, ws=sh.down.w if sh else None, pdl=s.pdl)
+            A.moe_up_rows(z, h, s.nb, self.gu, 2 * m.expert.ff, a, ids, wts, experts=m.experts, top=m.top, ffp=self.ffp, limit=m.expert.limit, act=self.act, outputs=m.outputs,
+                          correction=self.correction, ws=sh.gu.w if sh else None, ns=2 * sh.e.ff if sh else 0, limit_s=sh.e.limit if sh else math.inf, pdl=s.pdl)
+            A.moe_down_rows(a, s.nb, ids, wts, self.down, out, top=m.top, n=s.be.stack.width, mult=mult, ws=sh.down.w if sh else None, store=post is not None, h=h, gate=gate,
+                            pdl=s.pdl)
             s.launched(2)
-            return
-        ids, wts = A.moe_route(z, m.experts, m.top)
-        row, tile_expert, rows = K.moe_plan(ids, m.experts)
-        xs = K.moe_gather(h, row, m.top, rows)
-        f = torch.empty(rows, self.ffp, device=h.device, dtype=s.act)
-        O.gemm(xs, self.gu.view(-1, self.gu.shape[2]), f, act=self.ACT, limit=m.expert.limit, experts=m.experts, tile_expert=tile_expert)
-        y = torch.empty(rows, s.be.wp, device=h.device)
-        O.gemm(f, self.down.view(-1, self.ffp), y, experts=m.experts, tile_expert=tile_expert)
-        K.moe_scatter_combine(y, row, wts, s.nb, m.top, out=s.x, accumulate=True, mult=s.be.stack.residual_mult)
-        s.launched(6)
-        if sh:
-            f = s.buf("shared", up(sh.e.ff), zero=True)
-            s.product(h, sh.gu, f, act=self.ACT, limit=sh.e.limit)
-            s.add(f, sh.down)
+        else:
+            ids, lids, wts = A.moe_route(z, m.outputs, m.top, m.experts, self.correction)
+            row, tile_expert, rows = K.moe_plan(lids, m.experts)
+            xs = K.moe_gather(h, row, m.top, rows)
+            f = torch.empty(rows, self.ffp, device=h.device, dtype=s.act)
+            O.gemm(xs, self.gu.view(-1, self.gu.shape[2]), f, act=self.act, limit=m.expert.limit, experts=m.experts, tile_expert=tile_expert)
+            y = torch.empty(rows, s.be.wp, device=h.device)
+            O.gemm(f, self.down.view(-1, self.ffp), y, experts=m.experts, tile_expert=tile_expert)
+            more, late = {"ids": ids, "n_experts": m.experts, "h": h} if m.identity else {}, post is None and gate is None
+            if sh:
+                f = s.buf("shared", up(sh.e.ff), zero=True)
+                s.product(h, sh.gu, f, act=self.act, limit=sh.e.limit)
+                if not late:
+                    more["shared"], more["gate"] = s.buf("shared_y", s.be.wp, torch.float32), gate
+                    s.product(f, sh.down, more["shared"])
+            K.moe_scatter_combine(y, row, wts, s.nb, m.top, out=out, accumulate=post is None, mult=mult, **more)
+            s.launched(6)
+            if sh and late:
+                s.add(f, sh.down)
+        if post is not None:
+            s.leave(out, post)
 
 
 class SideInput:

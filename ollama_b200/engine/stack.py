@@ -26,13 +26,14 @@ import torch
 from .. import envconfig
 from ..gguf.reader import GGUFFile
 from ..models.config import ModelConfig, config_from_gguf
-from ..models.stack import AttentionMixer, DenseMLP, ExpertMLP, LatentMixer, LayerRun, MambaMixer
+from ..models.stack import AttentionMixer, DenseMLP, ExpertMLP, LatentMixer, LayerRun, Mamba2Mixer, MambaMixer
 from ..models.weights import QWeight, load_tensor
 from ..ops import cuda as K
 from ..ops import reference as R
 from ..ops import rows as O
 from .blocks import LONG_PORTION, ExpertFFN, GatedFFN, LatentAttention, LongPortions, Mat, Norm, SideInput, Step, WeightSource, make_norm, up
 from .cache import CacheFull, PagedCache
+from .mixers import HeadAttention, StateSpaceHeads
 from .steps import StepEngine
 
 MAX_DECODE_ROWS = 32
@@ -178,11 +179,12 @@ class StackBackend(StepEngine):
         torch.cuda.synchronize(dev)
 
     def _load_sequential(self, src: WeightSource) -> None:
-        """Layers whose mixer and feed-forward follow one another, each behind a layer norm."""
+        """Layers whose mixer and feed-forward follow one another, each behind a norm and, in some designs, under another one."""
         st, f32 = self.stack, self.f32
-        self.out_norm = make_norm(src, "output_norm")
+        norm = st.design.norm
+        self.out_norm = make_norm(src, "output_norm", norm)
         self.out_mat = Mat(self.head)
-        if not f32:
+        if not f32 and norm == "layer":
             self.out_mat.fold(self.out_norm)
         if st.loop is not None:
             self.loop_step = torch.zeros(st.loop[2], src.wp, device=src.device)
@@ -193,14 +195,24 @@ class StackBackend(StepEngine):
             self.side_table[..., :d] = src.tensor("per_layer_token_embd.weight", st.vocab, n * d).view(st.vocab, n, d)
         for i, sl in enumerate(st.layers):
             L, p = _Layer(), f"blk.{i}."
-            if not isinstance(sl.mixer, LatentMixer):
+            pre = make_norm(src, p + "attn_norm", norm)
+            post = make_norm(src, p + "post_attention_norm", norm) if st.design.post_norm else None
+            if isinstance(sl.mixer, LatentMixer):
+                L.mix = LatentAttention(src, p, sl.mixer, pre, f32)
+            elif isinstance(sl.mixer, (AttentionMixer, Mamba2Mixer)):
+                L.mix = (HeadAttention if isinstance(sl.mixer, AttentionMixer) else StateSpaceHeads)(src, p, sl.mixer, pre, f32, post)
+            else:
                 raise NotImplementedError(f"{type(sl.mixer).__name__} in a sequential layer")
-            L.mix = LatentAttention(src, p, sl.mixer, make_norm(src, p + "attn_norm"), f32)
             L.ff = L.side = None
-            if isinstance(sl.mlp, ExpertMLP):
-                L.ff = ExpertFFN(src, p, sl.mlp, make_norm(src, p + "ffn_norm"), f32)
-            elif isinstance(sl.mlp, DenseMLP):
-                L.ff = GatedFFN(src, p, sl.mlp, make_norm(src, p + "ffn_norm"), f32)
+            if sl.mlp is not None:
+                pre = make_norm(src, p + "ffn_norm", norm)
+                post = make_norm(src, p + "post_ffw_norm", norm) if st.design.post_norm else None
+                if isinstance(sl.mlp, ExpertMLP):
+                    L.ff = ExpertFFN(src, p, sl.mlp, pre, f32, post)
+                elif post is None:
+                    L.ff = GatedFFN(src, p, sl.mlp, pre, f32)
+                else:
+                    raise NotImplementedError("a dense feed-forward under a norm of its own")
             if st.side_dim:
                 L.side = SideInput(src, p, st.side_dim, self.side_table[:, i])
             self.layers.append(L)
@@ -444,20 +456,23 @@ class StackBackend(StepEngine):
     def _head_rows(self, x: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
         """Logits (before the soft cap) of hidden rows ``x`` into the rows of ``out`` [rows, padded vocabulary]."""
         nb, st = x.shape[0], self.stack
+        scale = st.logit_scale
         if isinstance(self.out_norm, Norm):
-            if nb <= self.gemv_rows and not self.f32:
+            if nb <= self.gemv_rows and self.out_norm.b is None:
+                O.gemv([O.seg(self.head, st.vocab, out, self.out_norm.g, alpha=scale)], self.wp, x, nb, self.f32, O.SRC_NORM, st.eps, st.width, pdl=pdl)
+            elif nb <= self.gemv_rows and not self.f32:
                 m = self.out_mat
-                O.gemv([O.seg(m.w, m.w.shape[0], out, self.out_norm.g, rs=m.rs, rc=m.rc)], self.wp, x, nb, False, O.SRC_LAYER, st.eps, st.width, pdl=pdl)
+                O.gemv([O.seg(m.w, m.w.shape[0], out, self.out_norm.g, rs=m.rs, rc=m.rc, alpha=scale)], self.wp, x, nb, False, O.SRC_LAYER, st.eps, st.width, pdl=pdl)
             else:
                 h = torch.empty(nb, self.wp, device=self.device, dtype=self.act_dtype)
                 O.norm_rows(x, st.width, st.eps, self.out_norm.g, h, b1=self.out_norm.b, pdl=pdl)
-                self._mm(h, self.head, out)
+                self._mm(h, self.head, out, alpha=scale)
         elif nb <= self.gemv_rows:
-            O.gemv([O.seg(self.head, st.vocab, out, self.out_norm)], self.wp, x, nb, self.f32, O.SRC_NORM, st.eps, st.width, pdl=pdl)
+            O.gemv([O.seg(self.head, st.vocab, out, self.out_norm, alpha=scale)], self.wp, x, nb, self.f32, O.SRC_NORM, st.eps, st.width, pdl=pdl)
         else:
             h = torch.empty(nb, self.wp, device=self.device, dtype=self.act_dtype)
             O.norm_rows(x, st.width, st.eps, self.out_norm, h, pdl=pdl)
-            self._mm(h, self.head, out)
+            self._mm(h, self.head, out, alpha=scale)
         self._n += 1
 
     # -- decode ---------------------------------------------------------------------------------------
@@ -526,6 +541,8 @@ class StackBackend(StepEngine):
     def _final_norm(self, x: torch.Tensor) -> torch.Tensor:
         w = self.stack.width
         if isinstance(self.out_norm, Norm):
+            if self.out_norm.b is None:
+                return R.rmsnorm(x[:, :w], self.out_norm.g[:w], self.stack.eps)
             return torch.nn.functional.layer_norm(x[:, :w], (w,), self.out_norm.g[:w], self.out_norm.b[:w], self.stack.eps)
         return R.rmsnorm(x[:, :w], self.out_norm[:w], self.stack.eps)
 

@@ -1,6 +1,6 @@
 // Argument block shared by the decode-attention kernels (scalar split-K kernel and tensor-core split-K kernel).
 #pragma once
-#include "common.cuh"
+#include "rows.cuh"
 
 struct AttnDecodeArgs {
     const float* q;          // [nb][H][HD]
@@ -19,6 +19,7 @@ struct AttnDecodeArgs {
     const int* page_table;   // [slots][max_pages]
     int max_pages;
     int chunk;               // > 0: position p sees the keys from floor(p / chunk) * chunk on
+    int keep;                // with window > 0: the first `keep` keys are seen too
 };
 
 // Optional second argument of the tensor-core kernel: with `qkv` set the kernel takes the query rows straight from the
@@ -31,19 +32,21 @@ struct AttnRopeArgs {
     float mscale;
     int n_rot, neox;
     // paged form: heads of dim / vdim columns inside rows of pitch ldq (the cache rows are padded to HD), RMS norms over the whole
-    // q and k projections (or null), rotation in the half-split order with frequencies in double
-    const float* q_norm;     // [H * dim]
-    const float* k_norm;     // [Hkv * dim]
+    // q and k projections or over each head (or null), rotation in the half-split order with frequencies in double
+    const float* q_norm;     // [H * dim], head_norm: [dim]
+    const float* k_norm;     // [Hkv * dim], head_norm: [dim]
     float eps;
     int ldq, dim, vdim;
     const double* freqs;     // [n_rot / 2]
+    int head_norm;
+    int v_off;               // column of the first value head
 };
 
 // Rows of a step over a paged cache: see attn_paged.cu.
 struct PagedAppendArgs {
-    const float* qkv;        // [rows][ldq]: q heads | k heads | v heads
+    const float* qkv;        // [rows][ldq]: q heads | k heads | ..., value heads from column v_off on
     int ldq, n_heads, n_kv_heads, dim, vdim;
-    const float* q_norm;     // [H * dim], or null with k_norm
+    const float* q_norm;     // [H * dim], or null with k_norm; head_norm: [dim]
     const float* k_norm;     // [Hkv * dim]
     float eps;
     const double* freqs;     // [n_rot / 2]
@@ -57,6 +60,8 @@ struct PagedAppendArgs {
     void* k_cache;           // [pages][Hkv][64][dk]
     void* v_cache;           // [pages][Hkv][64][dv]
     int dk, dv, cache32;     // cache32: fp32 caches, else f16
+    int head_norm, v_off;
+    float mscale;            // factor of the rotated dimensions
 };
 
 struct PagedAttnArgs {
@@ -72,6 +77,8 @@ struct PagedAttnArgs {
     float scale, softcap;
     void* out;               // [rows][ldo], head h at column h * vdim
     int ldo, out16;
+    int window, keep;
+    HeadGate gate;
 };
 
 // Tensor-core variant (attn_decode_mma.cu): same partial outputs, so the same combine kernel follows.

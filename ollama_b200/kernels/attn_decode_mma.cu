@@ -11,7 +11,7 @@
 // through shared memory at the end.  The scalar kernel stays the choice for short contexts and for head
 // sizes without an instantiation here.
 // The paged form (PAGED) reads its tiles through a page table (a tile of 64 positions is a page), starts at the query's chunk
-// instead of a sliding window, and normalises q and k over their whole projections before the rotation.
+// or window (keys that are kept in front of a window come first), and normalises q and k over their whole projections or heads before the rotation.
 #include "attn_args.cuh"
 #include "rows.cuh"
 
@@ -57,17 +57,19 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
     pdl_wait();
     const int qpos = a.positions[b], slot = a.slots[b];
     const int kv_len = qpos + 1;
-    const int start = a.chunk > 0 ? qpos - qpos % a.chunk : (a.window > 0 && kv_len > a.window) ? kv_len - a.window : 0;
+    const int start = first_key(qpos, a.chunk, a.window);
     const int base = PAGED ? start & ~(BN - 1) : start;         // paged: tiles begin at page borders
-    const int span = kv_len - base;
+    // the keys to visit, numbered from 0: `front` of them at the sequence's start (whole tiles with kept keys), the rest `shift` positions further on
+    const int front = PAGED && a.window > 0 ? BN * kept_tiles(a.keep, base, BN) : 0, shift = base - front, keep = PAGED ? a.keep : 0;
+    const int span = kv_len - shift;
     int chunk = (span + a.n_splits - 1) / a.n_splits;
     chunk = ((chunk + BN - 1) / BN) * BN;
-    const int p0 = base + split * chunk, p1 = min(p0 + chunk, kv_len);
+    const int p0 = split * chunk, p1 = min(p0 + chunk, span);
     const int n_tiles = p1 > p0 ? (p1 - p0 + BN - 1) / BN : 0;
     const size_t row0 = ((size_t)slot * a.n_kv_heads + kvh) * a.n_ctx;      // first cache row of this (slot, kv head)
 
     auto load_kv = [&](int tile, int stage) {
-        const int n0 = p0 + tile * BN;
+        const int v0 = p0 + tile * BN, n0 = v0 < front ? v0 : v0 + shift;
         __half* dk = sK + stage * BN * LD;
         __half* dv = sV + stage * BN * LD;
         if (PAGED) {
@@ -124,7 +126,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         else asm volatile("cp.async.commit_group;" ::: "memory");
     }
     const bool fresh = r.qkv != nullptr;
-    const bool owner = fresh && n_tiles > 0 && qpos >= p0 && qpos < p1;      // this split holds the query token's own position
+    const bool owner = fresh && n_tiles > 0 && qpos - shift >= p0 && qpos - shift < p1;      // this split holds the query token's own position
     // element i of a raw head row after the rotary embedding (pairs (2p, 2p+1), or (p, p + n_rot/2) in the neox order)
     auto rotated = [&](const float* row, int i) -> float {
         const float x = row[i];
@@ -143,9 +145,14 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         if (PAGED) {
             const float* tok = r.qkv + (size_t)b * r.ldq;
             const int nq = a.n_heads * r.dim, nk = a.n_kv_heads * r.dim;
-            for (int p = tid; p < (r.n_rot >> 1); p += 128) sincosf(rot_angle(qpos, r.freqs[p]), &s_sn[p], &s_cs[p]);
+            for (int p = tid; p < (r.n_rot >> 1); p += 128) {
+                float sn, cs;
+                sincosf(rot_angle(qpos, r.freqs[p]), &sn, &cs);
+                s_sn[p] = sn * r.mscale;
+                s_cs[p] = cs * r.mscale;
+            }
             float iq = 1.f, ik = 1.f;
-            if (r.q_norm) {
+            if (r.q_norm && !r.head_norm) {
                 float s0 = 0.f, s1 = 0.f;
                 const int total = owner ? nq + nk : nq;
                 if (((nq | nk | r.ldq) & 3) == 0) {
@@ -181,12 +188,28 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
                     if (col < r.dim) {
                         const int i = rr < group ? (head0 + rr) * r.dim + col : kvh * r.dim + col;
                         v = tok[rr < group ? i : nq + i];
-                        if (r.q_norm) v *= rr < group ? iq * r.q_norm[i] : ik * r.k_norm[i];
+                        if (r.q_norm && !r.head_norm) v *= rr < group ? iq * r.q_norm[i] : ik * r.k_norm[i];
                     }
                 } else if (col < r.vdim) {
-                    v = tok[nq + nk + kvh * r.vdim + col];
+                    v = tok[r.v_off + kvh * r.vdim + col];
                 }
                 raw[c] = v;
+            }
+            if (r.q_norm && r.head_norm) {          // a warp per head
+                __syncthreads();
+                for (int rr = warp; rr < group + (owner ? 1 : 0); rr += 4) {
+                    const float* w = rr < group ? r.q_norm : r.k_norm;
+                    float x[D / 32], s = 0.f;
+#pragma unroll
+                    for (int i = 0; i < D / 32; i++) {
+                        x[i] = raw[rr * D + lane + 32 * i];      // columns beyond dim are zero
+                        s += x[i] * x[i];
+                    }
+                    const float inv = 1.f / sqrtf(warp_sum(s) / (float)r.dim + r.eps);
+#pragma unroll
+                    for (int i = 0; i < D / 32; i++)
+                        if (lane + 32 * i < r.dim) raw[rr * D + lane + 32 * i] = x[i] * inv * w[lane + 32 * i];
+                }
             }
         } else {
         const float* tok = r.qkv + (size_t)b * (a.n_heads + 2 * a.n_kv_heads) * D;
@@ -255,7 +278,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         asm volatile("cp.async.wait_group %0;" ::"n"(NS - 1) : "memory");               // tile's own group is complete
         __syncthreads();
         if (owner && tile == n_tiles - 1) {      // the query's own row did not come from the cache: put it into the tile
-            const int rr = qpos - (p0 + tile * BN);
+            const int rr = qpos - shift - (p0 + tile * BN);
             for (int i = tid; i < D; i += 128) {
                 sK[stage * BN * LD + rr * LD + i] = s_newk[i];
                 sV[stage * BN * LD + rr * LD + i] = s_newv[i];
@@ -264,7 +287,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         }
         const __half* tk = sK + stage * BN * LD + 16 * warp * LD;       // this warp's 16 positions of the tile
         const __half* tv = sV + stage * BN * LD + 16 * warp * LD;
-        const int n0 = p0 + tile * BN + 16 * warp;
+        const int v0 = p0 + tile * BN, n0 = (v0 < front ? v0 : v0 + shift) + 16 * warp, end = v0 < front ? n0 + BN : p1 + shift;
 
         float s[2][4];
         s[0][0] = s[0][1] = s[0][2] = s[0][3] = s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.f;
@@ -283,7 +306,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int kp = n0 + 8 * j + 2 * tq + e;
-                ok[j][e] = kp < p1 && (!PAGED || kp >= start);
+                ok[j][e] = kp < end && (!PAGED || kp >= start || kp < keep);
             }
 #pragma unroll
             for (int e = 0; e < 4; e++) {
@@ -423,7 +446,8 @@ int launch_d(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int pdl, cu
 int attn_decode_mma_rope_launch(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int hd, int pdl, cudaStream_t st) {
     if (a.n_kv_heads < 1 || a.n_heads % a.n_kv_heads || a.n_heads / a.n_kv_heads > ROWS) return (int)cudaErrorNotSupported;
     if (r.qkv && (a.k_scale || a.v_scale || r.n_rot > 256 || r.n_rot > hd || (r.n_rot & 1) || (a.page_table ? r.n_rot && !r.freqs : !r.inv_freq))) return (int)cudaErrorNotSupported;
-    if (a.page_table && (!r.qkv || !r.neox || r.dim < 1 || r.dim > hd || r.vdim < 1 || r.vdim > hd || r.n_rot > r.dim || a.max_pages < 1)) return (int)cudaErrorInvalidValue;
+    if (a.page_table && (!r.qkv || !r.neox || r.dim < 1 || r.dim > hd || r.vdim < 1 || r.vdim > hd || r.n_rot > r.dim || a.max_pages < 1 || a.window < 0 || a.keep < 0 || r.v_off < 0 ||
+                         r.v_off + a.n_kv_heads * r.vdim > r.ldq)) return (int)cudaErrorInvalidValue;
     if (hd == 128) return launch_d<128>(a, r, nb, pdl, st);
     if (hd == 64) return launch_d<64>(a, r, nb, pdl, st);
     return (int)cudaErrorNotSupported;

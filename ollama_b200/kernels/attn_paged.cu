@@ -4,14 +4,14 @@
 // Cache layout per layer run: K [page][kv head][64 positions][dk], V [page][kv head][64 positions][dv]; page_table[slot][i]
 // is the page that holds positions 64 i .. 64 i + 63 of the slot.  dk and dv are the padded row lengths (pad columns are zero).
 //
-// Chunked masks: with chunk > 0 the query at position p sees the keys floor(p / chunk) * chunk .. p.
+// Masks: see first_key in rows.cuh.
 #include "attn_args.cuh"
 #include "rows.cuh"
 
 namespace {
 
 // ---------------------------------------------------------------------------------------------------------------------
-// RMS norm of q and k over their whole projections, rotary embedding, q to padded fp32 rows, k and v into the cache.
+// RMS norm of q and k over their whole projections or over each head, rotary embedding, q to padded fp32 rows, k and v into the cache.
 // One CTA per row.
 // ---------------------------------------------------------------------------------------------------------------------
 template <typename CT>
@@ -44,7 +44,12 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
             else s1 += v * v;
         }
     }
-    for (int p = tid; p < half; p += 256) sincosf(rot_angle(pos, a.freqs[p]), &sn[p], &cs[p]);
+    for (int p = tid; p < half; p += 256) {
+        float s, c;
+        sincosf(rot_angle(pos, a.freqs[p]), &s, &c);
+        sn[p] = s * a.mscale;
+        cs[p] = c * a.mscale;
+    }
     s0 = warp_sum(s0);
     s1 = warp_sum(s1);
     if (lane == 0) {
@@ -52,7 +57,17 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
         red[1][warp] = s1;
     }
     __syncthreads();
-    if (a.q_norm) {
+    if (a.q_norm && a.head_norm) {
+        for (int h = warp; h < a.n_heads + a.n_kv_heads; h += 8) {
+            float* head = sq + h * a.dim;
+            const float* w = h < a.n_heads ? a.q_norm : a.k_norm;
+            float s = 0.f;
+            for (int d = lane; d < a.dim; d += 32) s += head[d] * head[d];
+            const float inv = 1.f / sqrtf(warp_sum(s) / (float)a.dim + a.eps);
+            for (int d = lane; d < a.dim; d += 32) head[d] *= inv * __ldg(w + d);
+        }
+        __syncthreads();
+    } else if (a.q_norm) {
         s0 = s1 = 0.f;
 #pragma unroll
         for (int i = 0; i < 8; i++) {
@@ -82,7 +97,7 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
             for (int d = lane; d < a.dk; d += 32) k[d] = from_f<CT>(d < a.dim ? rotated(head, d) : 0.f);
         } else {
             const int g = h - a.n_heads - a.n_kv_heads;
-            const float* head = row + nq + nk + g * a.vdim;
+            const float* head = row + a.v_off + g * a.vdim;
             CT* v = (CT*)a.v_cache + paged_row(table, pos, a.n_kv_heads, g) * a.dv;
             for (int d = lane; d < a.dv; d += 32) v[d] = from_f<CT>(d < a.vdim ? head[d] : 0.f);
         }
@@ -109,12 +124,12 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__
     const float* q = a.q + ((size_t)t * a.n_heads + h) * a.dq;
     for (int i = tid; i < a.dim; i += 128) sq[i] = q[i];
     __syncthreads();
-    const int lo = a.chunk > 0 ? pos - pos % a.chunk : 0;
+    const int lo = first_key(pos, a.chunk, a.window), kept = min(a.window > 0 ? a.keep : 0, lo);      // kept keys first, then the ones from lo on
     float acc[VCOLS] = {}, m = -INFINITY, l = 0.f;
-    for (int k0 = lo; k0 <= pos; k0 += 128) {
-        const int kp = k0 + tid;
+    for (int k0 = kept > 0 ? 0 : lo; k0 <= pos; k0 = k0 < kept && k0 + 128 >= kept ? lo : k0 + 128) {
+        const int kp = k0 + tid, last = k0 < kept ? kept - 1 : pos;
         float s = -INFINITY;
-        if (kp <= pos) {
+        if (kp <= last) {
             const CT* kr = (const CT*)a.k_cache + paged_row(table, kp, a.n_kv_heads, g) * a.dk;
             float d = 0.f;
             for (int i = 0; i < a.dim; i++) d = fmaf(sq[i], to_f(kr[i]), d);
@@ -134,7 +149,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__
         __syncthreads();
         l = l * corr + red[1][0] + red[1][1] + red[1][2] + red[1][3];
         m = mn;
-        const int n = min(128, pos - k0 + 1);
+        const int n = min(128, last - k0 + 1);
 #pragma unroll
         for (int j = 0; j < VCOLS; j++) acc[j] *= corr;
         for (int i = 0; i < n; i++) {
@@ -152,7 +167,10 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(const __grid_constant__
 #pragma unroll
     for (int j = 0; j < VCOLS; j++) {
         const int d = v0 + tid + 128 * j;
-        if (d < a.vdim) o[d] = from_f<OT>(acc[j] / l);
+        if (d >= a.vdim) continue;
+        float v = acc[j] / l;
+        if (a.gate.kind) v *= sigmoid_exact(a.gate.g[(size_t)t * a.gate.ld + (a.gate.kind == 1 ? h * a.vdim + d : h)]);
+        o[d] = from_f<OT>(v);
     }
 }
 
@@ -163,6 +181,7 @@ struct PagedCombineArgs {
     int n_heads, n_splits, hd, vdim;
     void* out;
     int ldo, out16;
+    HeadGate gate;
 };
 
 __global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constant__ PagedCombineArgs a) {
@@ -180,11 +199,14 @@ __global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constan
         o += a.part_acc[(p0 + s) * a.hd + d] * c;
         l += ml.y * c;
     }
-    const float v = l > 0.f ? o / l : 0.f;
+    float v = l > 0.f ? o / l : 0.f;
+    if (a.gate.kind) v *= sigmoid_f(a.gate.g[(size_t)b * a.gate.ld + (a.gate.kind == 1 ? h * a.vdim + d : h)]);
     const size_t oi = (size_t)b * a.ldo + (size_t)h * a.vdim + d;
     if (a.out16) ((__nv_bfloat16*)a.out)[oi] = __float2bfloat16_rn(v);
     else ((float*)a.out)[oi] = v;
 }
+
+bool bad_gate(const HeadGate& g) { return g.kind < 0 || g.kind > 2 || (g.kind && !g.g); }
 
 bool bad_shape(int H, int G, int dim, int vdim) { return H < 1 || G < 1 || H % G || dim < 1 || vdim < 1; }
 
@@ -193,7 +215,7 @@ bool bad_shape(int H, int G, int dim, int vdim) { return H < 1 || G < 1 || H % G
 // Returns a cudaError_t value (as do the entry points below).
 B2_API int b2_paged_append(const PagedAppendArgs* a, int rows, int pdl, cudaStream_t st) {
     if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dq < a->dim || a->dk < a->dim || a->dv < a->vdim || a->n_rot < 0 || a->n_rot > a->dim ||
-        (a->n_rot & 1) || (a->n_rot && !a->freqs) || (!a->q_norm != !a->k_norm))
+        (a->n_rot & 1) || (a->n_rot && !a->freqs) || (!a->q_norm != !a->k_norm) || a->v_off < 0 || a->v_off + a->n_kv_heads * a->vdim > a->ldq)
         return (int)cudaErrorInvalidValue;
     const size_t smem = ((size_t)(a->n_heads + a->n_kv_heads) * a->dim + a->n_rot) * 4;
     if (smem > 200 * 1024) return (int)cudaErrorNotSupported;
@@ -208,7 +230,7 @@ B2_API int b2_paged_append(const PagedAppendArgs* a, int rows, int pdl, cudaStre
 }
 
 B2_API int b2_paged_attn(const PagedAttnArgs* a, int rows, int pdl, cudaStream_t st) {
-    if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dim > 8192 || a->n_heads > 65535) return (int)cudaErrorInvalidValue;
+    if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dim > 8192 || a->n_heads > 65535 || a->window < 0 || a->keep < 0 || bad_gate(a->gate)) return (int)cudaErrorInvalidValue;
     PagedAttnArgs c = *a;
     void* args[] = {&c};
     const void* fn = a->cache32 ? (a->out16 ? (const void*)paged_attn_kernel<float, __nv_bfloat16> : (const void*)paged_attn_kernel<float, float>)
@@ -218,12 +240,12 @@ B2_API int b2_paged_attn(const PagedAttnArgs* a, int rows, int pdl, cudaStream_t
 
 // Decode step over a paged f16 cache: norm and rotation of the new query and key, cache append and split-K attention in one launch,
 // then the merge of the splits.  cudaErrorNotSupported (nothing launched): the caller runs b2_paged_append + b2_paged_attn.
-B2_API int b2_attn_decode_paged(const AttnDecodeArgs* a, const AttnRopeArgs* r, int nb, int hd, void* out, int ldo, int out16, int pdl, cudaStream_t st) {
-    if (!r || !r->qkv || !a->page_table || bad_shape(a->n_heads, a->n_kv_heads, r->dim, r->vdim) || r->dim > hd || r->vdim > hd || nb < 1 || a->n_splits < 1)
+B2_API int b2_attn_decode_paged(const AttnDecodeArgs* a, const AttnRopeArgs* r, int nb, int hd, void* out, int ldo, int out16, const HeadGate* gate, int pdl, cudaStream_t st) {
+    if (!r || bad_gate(*gate) || !r->qkv || !a->page_table || bad_shape(a->n_heads, a->n_kv_heads, r->dim, r->vdim) || r->dim > hd || r->vdim > hd || nb < 1 || a->n_splits < 1)
         return (int)cudaErrorInvalidValue;
     const cudaError_t e = (cudaError_t)attn_decode_mma_rope_launch(*a, *r, nb, hd, pdl, st);
     if (e != cudaSuccess) return (int)e;
-    PagedCombineArgs c{a->part_acc, a->part_ml, a->n_heads, a->n_splits, hd, r->vdim, out, ldo, out16};
+    PagedCombineArgs c{a->part_acc, a->part_ml, a->n_heads, a->n_splits, hd, r->vdim, out, ldo, out16, *gate};
     void* args[] = {&c};
     return launch_rows((const void*)paged_combine_kernel, dim3(a->n_heads, nb), dim3(128), 0, args, st, pdl);
 }

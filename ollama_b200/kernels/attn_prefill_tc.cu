@@ -19,6 +19,7 @@
 // Attention sinks, logit soft-capping and sliding windows follow attn_prefill.cu, which stays the kernel for int8 caches
 // and head sizes other than 64 / 128.  In the reference stack this is ggml-cuda's fattn family (mma / tile / vec).
 #include "tc_common.cuh"
+#include "rows.cuh"
 
 struct AttnPrefillArgs {      // the same block as in attn_prefill.cu
     const float* q;          // [T][H][D] fp32, rotary embedding already applied
@@ -37,12 +38,14 @@ struct AttnPrefillArgs {      // the same block as in attn_prefill.cu
 };
 
 // Paged form of the pipelined kernel: the query tiles of a step (portions of several sequences) come as a list, K / V tiles are
-// read through a page table (two 64-position pages per tile; caches [page][Hkv][64][D], pad columns zero), the mask may be chunked
-// (position p sees the keys from floor(p / chunk) * chunk on), and heads of vdim <= D columns go to output rows of pitch ldo.
+// read through a page table (two 64-position pages per tile; caches [page][Hkv][64][D], pad columns zero), the mask may be chunked or a window
+// with kept first keys (first_key in rows.cuh), and heads of vdim <= D columns, times their gates, go to output rows of pitch ldo.
 struct AttnPagedArgs {
     const int4* tiles;       // [tiles] (first row, rows <= 128, slot, position of the first row)
     const int* page_table;   // [slots][max_pages]
     int max_pages, chunk, vdim, ldo;
+    int window, keep;
+    HeadGate gate;
 };
 
 // Form for keys in two parts (latent attention, latent.cu): rows of one buffer hold every head's own key part and value, rows of another the
@@ -506,8 +509,11 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     const int kv_len = PAGED ? q_hi + 1 : a.kv_len;
     const int k_end = a.causal ? min(kv_len, q_hi + 1) : kv_len;
     const int chunk = FORM == PAGED_CACHE ? pg.chunk : 0;
-    const int k_begin = (chunk > 0 ? q_lo - q_lo % chunk : a.window > 0 ? max(0, q_lo - a.window + 1) : 0) & ~(BKV - 1);
-    const int n_tiles = k_end > k_begin ? (k_end - k_begin + BKV - 1) / BKV : 0;
+    const int window = FORM == PAGED_CACHE ? pg.window : a.window, keep = FORM == PAGED_CACHE && window > 0 ? pg.keep : 0;
+    const int k_begin = first_key(q_lo, chunk, window) & ~(BKV - 1);
+    const int front = kept_tiles(keep, k_begin, BKV);      // tiles at the sequence's start, for its kept keys
+    const int n_tiles = front + (k_end > k_begin ? (k_end - k_begin + BKV - 1) / BKV : 0);
+    auto first_of = [&](int t) { return t < front ? t * BKV : k_begin + (t - front) * BKV; };
 
     if (threadIdx.x == 0) {
         *failed = 0;
@@ -583,7 +589,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                         else if (at < own) tma_load_2d(dst, &map_k, h * pt.dp + 64 * at, y, &full[b]);
                         else tma_load_2d(dst, &map_v, 64 * (at - own), y, &full[b]);
                     } else if (PAGED) {   // a tile may reach past the sequence's last page: any page will do there, its keys are masked
-                        const int p0 = (k_begin + t * BKV) >> 6, last = (kv_len - 1) >> 6;
+                        const int p0 = first_of(t) >> 6, last = (kv_len - 1) >> 6;
                         tma_load_2d(dst, map, 64 * at, (table[min(p0, last)] * a.Hkv + hkv) * 64, &full[b]);
                         tma_load_2d(dst + ATOM_BYTES / 2, map, 64 * at, (table[min(p0 + 1, last)] * a.Hkv + hkv) * 64, &full[b]);
                     } else {
@@ -630,7 +636,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
         const int q = warp & 3, c = warp >> 2;
         const int r = 32 * q + lane;
         const int qp = q_lo + r;
-        const int chunk_lo = chunk > 0 ? qp - qp % chunk : 0, chunk_hi = chunk > 0 ? q_hi - q_hi % chunk : 0;      // this row's first key; the last row's
+        const int row_lo = first_key(qp, chunk, window), last_lo = first_key(q_hi, chunk, window);      // this row's first key (but for kept ones); the last row's
         const float LOG2E = 1.4426950408889634f;
         const float sl2 = a.scale * LOG2E;
         const uint32_t lane_base = (uint32_t)(32 * q) << 16;
@@ -654,13 +660,13 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
         };
         for (int t = 0; t < n_tiles && ok; t++) {
             const int b = t & 1;
-            const int n0 = k_begin + t * BKV;
+            const int n0 = first_of(t);
             if (!mbar_wait(&s_full[b], (t >> 1) & 1)) { ok = false; break; }
             tc_fence_after();
             uint32_t v[2][32];
             tmem_ld32(tmem + lane_base + (uint32_t)(128 * b + 64 * c), v[0]);
             tmem_ld32(tmem + lane_base + (uint32_t)(128 * b + 64 * c + 32), v[1]);
-            const bool masked = (a.causal && n0 + BKV - 1 > q_lo) || n0 + BKV > kv_len || a.window > 0 || n0 < chunk_hi;
+            const bool masked = (a.causal && n0 + BKV - 1 > q_lo) || n0 + BKV > kv_len || n0 < last_lo;
             float mx = -INFINITY;
             if (a.softcap > 0.f) {
                 const float cap2 = a.softcap * LOG2E, inv_cap = a.scale / a.softcap;
@@ -676,13 +682,13 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             }
             if (masked) {
                 const int kp0 = n0 + 64 * c;
-                const int hi = min(a.causal ? qp : kv_len - 1, kv_len - 1), lo = FORM == PAGED_CACHE ? chunk_lo : a.window > 0 ? qp - a.window + 1 : 0;
+                const int hi = min(a.causal ? qp : kv_len - 1, kv_len - 1), lo = row_lo;
 #pragma unroll
                 for (int i = 0; i < 2; i++)
 #pragma unroll
                     for (int j = 0; j < 32; j++) {
                         const int kp = kp0 + 32 * i + j;
-                        if (kp > hi || kp < lo) v[i][j] = 0xff800000u;
+                        if (kp > hi || (kp < lo && (FORM != PAGED_CACHE || kp >= keep))) v[i][j] = 0xff800000u;
                     }
             }
 #pragma unroll
@@ -739,6 +745,28 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                 const int vdim = FORM == PARTS ? pt.vdim : pg.vdim, ldo = FORM == PARTS ? pt.ldo : pg.ldo;
                 __nv_bfloat16* op = a.out + (size_t)(m0 + r) * ldo + (size_t)h * vdim + OH * c;
                 const bool whole = (vdim & 7) == 0 && (ldo & 7) == 0;
+                if (FORM == PAGED_CACHE && pg.gate.kind) {
+                    const float* gp = pg.gate.g + (size_t)(m0 + r) * pg.gate.ld;
+                    if (pg.gate.kind == 2) {
+                        const float gv = sigmoid_f(gp[h]);
+#pragma unroll
+                        for (int j = 0; j < OH; j++) o[j] *= gv;
+                    } else {
+                        gp += (size_t)h * vdim + OH * c;
+                        const bool vec = whole && ((uintptr_t)gp & 15) == 0;
+#pragma unroll
+                        for (int j = 0; j < OH; j += 4) {
+                            if (vec && OH * c + j + 4 <= vdim) {
+                                const float4 gv = *(const float4*)(gp + j);
+                                o[j] *= sigmoid_f(gv.x); o[j + 1] *= sigmoid_f(gv.y); o[j + 2] *= sigmoid_f(gv.z); o[j + 3] *= sigmoid_f(gv.w);
+                            } else {
+#pragma unroll
+                                for (int e = 0; e < 4; e++)
+                                    if (OH * c + j + e < vdim) o[j + e] *= sigmoid_f(gp[j + e]);
+                            }
+                        }
+                    }
+                }
 #pragma unroll
                 for (int j = 0; j < OH; j += 8) {
                     if (OH * c + j >= vdim) continue;
@@ -856,7 +884,8 @@ B2_API int b2_attn_prefill_parts(const AttnPartsArgs* p, int n_tiles, cudaStream
 // nothing launched).  a: q [rows][H][head_dim], caches, out, H, Hkv, scale, softcap; the other fields are not used.
 B2_API int b2_attn_prefill_paged(const AttnPrefillArgs* a, const AttnPagedArgs* pg, int head_dim, int n_tiles, int n_pages, cudaStream_t st) {
     if (!a || !pg || !pg->tiles || !pg->page_table || n_tiles < 1 || n_pages < 1 || pg->max_pages < 1 || a->H < 1 || a->H > 65535 || a->Hkv < 1 || a->H % a->Hkv ||
-        pg->vdim < 1 || pg->vdim > head_dim || pg->ldo < a->H * pg->vdim)
+        pg->vdim < 1 || pg->vdim > head_dim || pg->ldo < a->H * pg->vdim || pg->window < 0 || pg->keep < 0 || pg->gate.kind < 0 || pg->gate.kind > 2 ||
+        (pg->gate.kind && !pg->gate.g))
         return (int)cudaErrorInvalidValue;
     if (((uintptr_t)a->k_cache & 15) || ((uintptr_t)a->v_cache & 15) || ((uintptr_t)a->q & 15) || ((uintptr_t)a->out & 15)) return (int)cudaErrorNotSupported;
     if ((size_t)n_pages * a->Hkv * 64 >= ((size_t)1 << 31)) return (int)cudaErrorNotSupported;

@@ -9,8 +9,8 @@
 //            bias, both made at load;
 //   joined   two rows side by side;
 // The epilogue applies an activation (of single rows, or of gate / up pairs), a factor, and stores or accumulates (the residual add).  The first rows of one matrix may also run
-// through a causal depthwise convolution + SiLU with the slot's last inputs (the state is only read here: the kernel that advances the
-// recurrence shifts it).  A warp owns four consecutive rows of a matrix and strides over their 16-byte pieces; short problems split the row
+// through a causal depthwise convolution, with or without SiLU, with the slot's last inputs, which are shifted here or by the kernel that advances the
+// recurrence.  A warp owns four consecutive rows of a matrix and strides over their 16-byte pieces; short problems split the row
 // length over KS warps of the CTA.  Weight rows are requested from L2 before the grid-dependency wait (they do not depend on the producer
 // kernel).  One group of rows per warp measured faster than resident CTAs that walk over groups (5.5 against 4.7 TB/s on 184 MB).
 #include "rows.cuh"
@@ -46,8 +46,9 @@ struct GemvRowsArgs {
     // convolution of the rows 0 .. conv_n - 1 of matrix conv_seg (conv_seg < 0: none)
     int conv_seg, conv_n, taps;
     const float* conv_w;          // [taps][conv_n], last tap = current token
-    const float* conv_b;          // [conv_n]
-    const float* conv_state;      // [slots][taps - 1][conv_n], oldest first
+    const float* conv_b;          // [conv_n] or null
+    float* conv_state;            // [slots][taps - 1][conv_n], oldest first
+    int conv_silu, conv_shift;    // conv_shift: the state is moved on here
     float* conv_out;              // [nb][ldu]
     int ldu;
     const int* slots;
@@ -243,12 +244,16 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
         float* o = w.out + (size_t)b * w.ldo + row;
         *o = w.accumulate ? *o + w.alpha * v : w.alpha * v;
         if (s == a.conv_seg && row < a.conv_n) {
-            float u = a.conv_b[row] + a.conv_w[(size_t)(a.taps - 1) * a.conv_n + row] * v;
-            if (a.positions[b] > 0) {
-                const float* st = a.conv_state + (size_t)a.slots[b] * (a.taps - 1) * a.conv_n + row;
-                for (int j = 0; j < a.taps - 1; j++) u += st[(size_t)j * a.conv_n] * a.conv_w[(size_t)j * a.conv_n + row];
+            float u = (a.conv_b ? a.conv_b[row] : 0.f) + a.conv_w[(size_t)(a.taps - 1) * a.conv_n + row] * v;
+            const bool old = a.positions[b] > 0;
+            float* st = a.conv_state + (size_t)a.slots[b] * (a.taps - 1) * a.conv_n + row;
+            for (int j = 0; j < a.taps - 1; j++) {
+                const float in = old ? st[(size_t)j * a.conv_n] : 0.f;
+                u += in * a.conv_w[(size_t)j * a.conv_n + row];
+                if (a.conv_shift && j > 0) st[(size_t)(j - 1) * a.conv_n] = in;
             }
-            a.conv_out[(size_t)b * a.ldu + row] = silu_f(u);
+            if (a.conv_shift && a.taps > 1) st[(size_t)(a.taps - 2) * a.conv_n] = v;
+            a.conv_out[(size_t)b * a.ldu + row] = a.conv_silu ? silu_f(u) : u;
         }
     }
 }
@@ -283,7 +288,7 @@ B2_API int b2_gemv_rows(const GemvRowsArgs* a, int pdl, cudaStream_t st) {
     if (a->nb < 1 || a->nb > 4 || a->nseg < 1 || a->nseg > 4 || a->k < 8 || (a->k & 7) || !a->x || (a->ldx & 3) || ((uintptr_t)a->x & 15) || a->src < 0 || a->src > SRC_LAYER)
         return (int)cudaErrorInvalidValue;
     if (a->src == SRC_JOINED && (!a->x2 || (a->ldx2 & 3) || ((uintptr_t)a->x2 & 15) || (a->k1 & 7))) return (int)cudaErrorInvalidValue;
-    if (a->conv_seg >= 0 && (a->conv_seg >= a->nseg || a->conv_n < 1 || a->conv_n > a->seg[a->conv_seg].n || a->taps < 1 || !a->conv_w || !a->conv_b || !a->conv_state ||
+    if (a->conv_seg >= 0 && (a->conv_seg >= a->nseg || a->conv_n < 1 || a->conv_n > a->seg[a->conv_seg].n || a->taps < 1 || !a->conv_w || !a->conv_state ||
                              !a->conv_out || !a->slots || !a->positions))
         return (int)cudaErrorInvalidValue;
     if (a->h && !norm_source(a->src)) return (int)cudaErrorInvalidValue;

@@ -11,12 +11,14 @@ struct MoeRouteArgs {
     int ld;
     int n_experts;         // <= 512
     int k;                 // experts per token, <= 16
-    int mode;              // 0: softmax over all experts, then top-k (optionally renormalised); 1: top-k, then softmax over the selected
+    int mode;              // 0: softmax over all experts, then top-k (optionally renormalised); 1: top-k, then softmax over the selected;
+                           // 2: softmax over all, top-k of that plus `correction`, weights without it
     int norm_topk;
     int e_lo, e_cnt;       // experts resident on this GPU: [e_lo, e_lo + e_cnt)
     int* ids;              // [tokens][k] global expert ids
     int* lids;             // [tokens][k] id relative to e_lo, or -1 when the expert lives elsewhere
     float* wts;            // [tokens][k]
+    const float* correction;      // [n_experts], mode 2
 };
 
 // one warp per token
@@ -42,6 +44,18 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ 
 #pragma unroll
         for (int j = 0; j < MAXJ; j++) denom += (lane + 32 * j < a.n_experts) ? __expf(v[j] - mx) : 0.f;
         denom = warp_sum(denom);
+    }
+    if (a.mode == 2) {
+        float e[MAXJ];
+#pragma unroll
+        for (int j = 0; j < MAXJ; j++) {
+            e[j] = lane + 32 * j < a.n_experts ? expf(v[j] - mx) : 0.f;
+            denom += e[j];
+        }
+        denom = warp_sum(denom);
+#pragma unroll
+        for (int j = 0; j < MAXJ; j++)
+            if (lane + 32 * j < a.n_experts) v[j] = e[j] / denom + a.correction[lane + 32 * j];
     }
     float sel_v = 0.f;     // lane s keeps the value of the s-th selected expert
     int sel_e = 0;
@@ -69,6 +83,8 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ 
     if (a.mode == 0) {
         w = mine ? __expf(sel_v - mx) / denom : 0.f;
         if (a.norm_topk) w /= warp_sum(w);
+    } else if (a.mode == 2) {
+        w = mine ? expf(lg[sel_e] - mx) / denom : 0.f;
     } else {
         const float top = __shfl_sync(0xffffffffu, sel_v, 0);          // the first selected is the largest
         const float ex = mine ? __expf(sel_v - top) : 0.f;
@@ -84,7 +100,8 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ 
 }
 
 B2_API int b2_moe_route(const MoeRouteArgs* a, int tokens, int pdl, cudaStream_t st) {
-    if (tokens < 1 || a->n_experts < 1 || a->n_experts > 512 || a->k < 1 || a->k > 16 || a->k > a->n_experts) return (int)cudaErrorInvalidValue;
+    if (tokens < 1 || a->n_experts < 1 || a->n_experts > 512 || a->k < 1 || a->k > 16 || a->k > a->n_experts || (a->mode == 2 && !a->correction))
+        return (int)cudaErrorInvalidValue;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3((tokens + 3) / 4);
     cfg.blockDim = dim3(128);
@@ -242,22 +259,57 @@ B2_API int b2_moe_gather(const void* h, const int* row_of_pair, int pairs, int k
     return (int)cudaGetLastError();
 }
 
-// out[t] (+)= mult * sum_s wts[t][s] * ys[row_of_pair[t k + s]]   (pairs whose expert lives elsewhere contribute nothing)
-__global__ void __launch_bounds__(256) moe_scatter_combine_kernel(const float* ys, const int* row_of_pair, const float* wts, int k, int d,
-                                                                  float* out, int ldo, int accumulate, float mult) {
+// out[t] (+)= mult * sum_s wts[t][s] * ys[row_of_pair[t k + s]]   (pairs whose expert lives elsewhere contribute nothing), and of a layer with more than routed
+// experts: + h[t] times the weights of the pairs whose choice is n_experts or above (the input itself), + sigmoid(gate[t]) * shared[t]
+struct MoeScatterArgs {
+    const float* ys;          // [rows][d]
+    const int* row_of_pair;
+    const float* wts;         // [tokens][k]
+    int k, d;                 // d: a multiple of 4
+    float* out;               // [tokens][ldo]
+    int ldo, accumulate;
+    float mult;
+    const int* ids;           // [tokens][k] chosen router outputs, or null
+    int n_experts;
+    const void* h;            // [tokens][ldh] bf16 or (f32) fp32
+    int ldh, f32;
+    const float* shared;      // [tokens][lds] or null
+    int lds;
+    const float* gate;        // one value per token, rows of ldg
+    int ldg;
+};
+
+template <bool MORE>
+__global__ void __launch_bounds__(256) moe_scatter_combine_kernel(const __grid_constant__ MoeScatterArgs a) {
     const int t = blockIdx.x;
-    for (int c = threadIdx.x; c < (d >> 2); c += 256) {
+    float same = 0.f, sg = 0.f;
+    if (MORE) {
+        if (a.ids)
+            for (int s = 0; s < a.k; s++) same += a.ids[(size_t)t * a.k + s] >= a.n_experts ? a.wts[(size_t)t * a.k + s] : 0.f;
+        if (a.shared) sg = a.gate ? 1.f / (1.f + expf(-a.gate[(size_t)t * a.ldg])) : 1.f;
+    }
+    for (int c = threadIdx.x; c < (a.d >> 2); c += 256) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int s = 0; s < k; s++) {
-            const int r = row_of_pair[(size_t)t * k + s];
+        auto add = [&](float w, const float4& v) { acc.x += w * v.x; acc.y += w * v.y; acc.z += w * v.z; acc.w += w * v.w; };
+        for (int s = 0; s < a.k; s++) {
+            const int r = a.row_of_pair[(size_t)t * a.k + s];
             if (r < 0) continue;
-            const float w = wts[(size_t)t * k + s];
-            const float4 v = *(const float4*)(ys + (size_t)r * d + 4 * c);
-            acc.x += w * v.x; acc.y += w * v.y; acc.z += w * v.z; acc.w += w * v.w;
+            add(a.wts[(size_t)t * a.k + s], *(const float4*)(a.ys + (size_t)r * a.d + 4 * c));
         }
-        acc.x *= mult; acc.y *= mult; acc.z *= mult; acc.w *= mult;
-        float4* o = (float4*)(out + (size_t)t * ldo + 4 * c);
-        if (accumulate) {
+        if (MORE) {
+            if (same != 0.f) {
+                if (a.f32) {
+                    add(same, *(const float4*)((const float*)a.h + (size_t)t * a.ldh + 4 * c));
+                } else {
+                    const uint2 q = *(const uint2*)((const __nv_bfloat16*)a.h + (size_t)t * a.ldh + 4 * c);
+                    add(same, make_float4(__uint_as_float(q.x << 16), __uint_as_float(q.x & 0xffff0000u), __uint_as_float(q.y << 16), __uint_as_float(q.y & 0xffff0000u)));
+                }
+            }
+            if (a.shared) add(sg, *(const float4*)(a.shared + (size_t)t * a.lds + 4 * c));
+        }
+        acc.x *= a.mult; acc.y *= a.mult; acc.z *= a.mult; acc.w *= a.mult;
+        float4* o = (float4*)(a.out + (size_t)t * a.ldo + 4 * c);
+        if (a.accumulate) {
             const float4 x = *o;
             acc.x += x.x; acc.y += x.y; acc.z += x.z; acc.w += x.w;
         }
@@ -265,9 +317,9 @@ __global__ void __launch_bounds__(256) moe_scatter_combine_kernel(const float* y
     }
 }
 
-B2_API int b2_moe_scatter_combine(const float* ys, const int* row_of_pair, const float* wts, int tokens, int k, int d, float* out, int ldo,
-                                  int accumulate, float mult, cudaStream_t st) {
-    if (tokens < 1 || k < 1 || (d & 3) || ldo < d || (ldo & 3)) return (int)cudaErrorInvalidValue;
-    moe_scatter_combine_kernel<<<tokens, 256, 0, st>>>(ys, row_of_pair, wts, k, d, out, ldo, accumulate, mult);
+B2_API int b2_moe_scatter_combine(const MoeScatterArgs* a, int tokens, cudaStream_t st) {
+    if (tokens < 1 || a->k < 1 || (a->d & 3) || a->ldo < a->d || (a->ldo & 3) || (a->ids && (!a->h || (a->ldh & 3))) || (a->shared && (a->lds & 3))) return (int)cudaErrorInvalidValue;
+    if (a->ids || a->shared) moe_scatter_combine_kernel<true><<<tokens, 256, 0, st>>>(*a);
+    else moe_scatter_combine_kernel<false><<<tokens, 256, 0, st>>>(*a);
     return (int)cudaGetLastError();
 }

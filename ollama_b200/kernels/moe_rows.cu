@@ -11,7 +11,7 @@
 
 struct MoeUpArgs {
     const float* z;          // [nb][ldz] router logits
-    int ldz, n_experts, top; // top-k, then the softmax over the chosen ones
+    int ldz, n_experts, top; // n_experts: router outputs; scoring: see choose
     const float* h;          // [nb][ldh]
     int ldh, k;              // k: padded row length, a multiple of 8
     const void* w;           // [experts][wrows][k], rows 2i / 2i + 1 = gate / up of hidden column i
@@ -23,6 +23,8 @@ struct MoeUpArgs {
     int ldo, ffp;
     int* ids;                // [nb][top]
     float* wts;              // [nb][top]
+    const float* correction; // [n_experts] or null
+    int real, act;           // router outputs from `real` on stand for the input itself and have no matrices; act: glu_act's number
 };
 
 struct MoeDownArgs {
@@ -33,22 +35,44 @@ struct MoeDownArgs {
     const void* w;           // [experts][wrows][ffp]
     const void* ws;          // [.][sfp]
     int n, wrows;            // result columns, rows stored of an expert
-    float* x;                // [nb][ldx] += mult * result
+    float* x;                // [nb][ldx] (+)= mult * result
     int ldx;
     float mult;
+    int store, real;         // store: the result replaces x; real: choices from this one on are the input itself
+    const float* h;          // [nb][ldh] that input
+    int ldh;
+    const float* gate;       // [nb] rows of ldg: the shared expert is multiplied by the sigmoid, or null
+    int ldg;
 };
 
 namespace {
 
 constexpr int R = 4, MAXJ = 16, MAX_TOP = 16;
 
-// Experts of a row in order of their logits (ties: the lower index) and the softmax over their logits; by one warp.
-__device__ __forceinline__ void choose(const float* z, int n, int top, int lane, int* ids, float* wts) {
-    float v[MAXJ];
+// Experts of a row in order of their scores (ties: the lower index) and their weights; by one warp.  Without a correction the scores are the logits and the
+// weights the softmax over the chosen ones; with it the softmax over all plus the correction, and that softmax.
+__device__ __forceinline__ void choose(const float* z, const float* correction, int n, int top, int lane, int* ids, float* wts) {
+    float v[MAXJ], mz = -INFINITY, total = 0.f;
 #pragma unroll
     for (int j = 0; j < MAXJ; j++) {
         const int e = lane + 32 * j;
         v[j] = e < n ? z[e] : -INFINITY;
+        mz = fmaxf(mz, v[j]);
+    }
+    if (correction) {
+        mz = warp_max(mz);
+#pragma unroll
+        for (int j = 0; j < MAXJ; j++) {
+            if (32 * j >= n) break;
+            v[j] = expf(v[j] - mz);
+            total += v[j];
+        }
+        total = warp_sum(total);
+#pragma unroll
+        for (int j = 0; j < MAXJ; j++) {
+            if (32 * j >= n) break;
+            v[j] = lane + 32 * j < n ? v[j] / total + correction[lane + 32 * j] : -INFINITY;
+        }
     }
     float val = -INFINITY;
     int idx = 0;
@@ -79,6 +103,13 @@ __device__ __forceinline__ void choose(const float* z, int n, int top, int lane,
 #pragma unroll
         for (int j = 0; j < MAXJ; j++)
             if (lane + 32 * j == be) v[j] = -INFINITY;
+    }
+    if (correction) {
+        if (lane < top) {
+            ids[lane] = idx;
+            wts[lane] = expf(z[idx] - mz) / total;
+        }
+        return;
     }
     const float mx = __shfl_sync(0xffffffffu, val, 0);
     const float e = lane < top ? expf(val - mx) : 0.f;
@@ -130,7 +161,7 @@ __global__ void __launch_bounds__(256) moe_up_rows_kernel(const __grid_constant_
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, rg = warp / KS, ks = warp % KS, b = blockIdx.y;
     pdl_launch();
     pdl_wait();
-    if (warp == 0) choose(a.z + (size_t)b * a.ldz, a.n_experts, a.top, lane, s_id, s_w);
+    if (warp == 0) choose(a.z + (size_t)b * a.ldz, a.correction, a.n_experts, a.top, lane, s_id, s_w);
     __syncthreads();
     if (blockIdx.x == 0 && threadIdx.x < a.top) {
         a.ids[b * a.top + threadIdx.x] = s_id[threadIdx.x];
@@ -146,7 +177,7 @@ __global__ void __launch_bounds__(256) moe_up_rows_kernel(const __grid_constant_
     const void* base = shared || !active ? a.ws : a.w;
     const size_t first = shared || !active ? 0 : (size_t)s_id[slot] * a.wrows;
     float acc[R] = {};
-    if (active) {
+    if (active && (shared || s_id[slot] < a.real)) {
         const float* x = a.h + (size_t)b * a.ldh;
         const int pieces = a.k >> 3, step = KS * 32;
         for (int p0 = ks * 32 + lane; p0 < pieces; p0 += U * step) {
@@ -183,7 +214,7 @@ __global__ void __launch_bounds__(256) moe_up_rows_kernel(const __grid_constant_
             v1 += red[rg * KS + j][2 * lane + 1];
         }
         const float limit = shared ? a.limit_s : a.limit;
-        const float y = F32 ? glu_act_exact(v0, v1, 2, SWIGLU_ALPHA, limit) : glu_act(v0, v1, 2, SWIGLU_ALPHA, limit);
+        const float y = F32 ? glu_act_exact(v0, v1, a.act, SWIGLU_ALPHA, limit) : glu_act(v0, v1, a.act, SWIGLU_ALPHA, limit);
         a.out[(size_t)b * a.ldo + (size_t)slot * a.ffp + (row0 >> 1) + lane] = y;
     }
 }
@@ -194,6 +225,7 @@ __global__ void __launch_bounds__(256) moe_down_rows_kernel(const __grid_constan
     __shared__ int s_id[MAX_TOP];
     __shared__ float s_w[MAX_TOP];
     __shared__ float red[8][R];
+    float same = 0.f;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, rg = warp / KS, ks = warp % KS, b = blockIdx.y;
     const int row0 = (blockIdx.x * RGS + rg) * R;
     const bool active = row0 < a.n;
@@ -207,6 +239,9 @@ __global__ void __launch_bounds__(256) moe_down_rows_kernel(const __grid_constan
     float acc[R] = {};
     if (active) {
         const float* x = a.a + (size_t)b * a.lda;
+        const float sw = a.gate && a.sfp ? (F32 ? sigmoid_exact(a.gate[(size_t)b * a.ldg]) : sigmoid_f(a.gate[(size_t)b * a.ldg])) : 1.f;
+        for (int s = 0; s < a.top; s++)
+            if (s_id[s] >= a.real) same += s_w[s];
         const int f8 = a.ffp >> 3, routed = a.top * f8, pieces = routed + (a.sfp >> 3), step = KS * 32;
         for (int p0 = ks * 32 + lane; p0 < pieces; p0 += U * step) {
             Piece<F32> w[U][R];
@@ -215,19 +250,19 @@ __global__ void __launch_bounds__(256) moe_down_rows_kernel(const __grid_constan
             for (int u = 0; u < U; u++) {
                 const int p = p0 + u * step;
                 f[u] = 0.f;
-                if (p >= pieces) continue;
+                if (p >= pieces || (p < routed && s_id[p / f8] >= a.real)) continue;
                 const bool shared = p >= routed;
                 const int slot = shared ? 0 : p / f8, c = 8 * (shared ? p - routed : p - slot * f8), ld = shared ? a.sfp : a.ffp;
                 const void* base = shared ? a.ws : a.w;
                 const size_t first = shared ? 0 : (size_t)s_id[slot] * a.wrows;
-                f[u] = shared ? 1.f : s_w[slot];
+                f[u] = shared ? sw : s_w[slot];
 #pragma unroll
                 for (int r = 0; r < R; r++) w[u][r].load(base, (first + min(row0 + r, a.n - 1)) * ld + c);
             }
 #pragma unroll
             for (int u = 0; u < U; u++) {
                 const int p = p0 + u * step;
-                if (p >= pieces) continue;
+                if (p >= pieces || f[u] == 0.f) continue;
                 float xv[8];
                 *(float4*)xv = *(const float4*)(x + 8 * p);
                 *(float4*)(xv + 4) = *(const float4*)(x + 8 * p + 4);
@@ -246,7 +281,9 @@ __global__ void __launch_bounds__(256) moe_down_rows_kernel(const __grid_constan
         float v = 0.f;
 #pragma unroll
         for (int j = 0; j < KS; j++) v += red[rg * KS + j][lane];
-        a.x[(size_t)b * a.ldx + row0 + lane] += a.mult * v;
+        if (same != 0.f) v = fmaf(same, a.h[(size_t)b * a.ldh + row0 + lane], v);
+        float* o = a.x + (size_t)b * a.ldx + row0 + lane;
+        *o = a.store ? a.mult * v : *o + a.mult * v;
     }
 }
 
@@ -267,7 +304,7 @@ int split_of(long groups, int pieces, long want) {
 B2_API int b2_moe_up_rows(const MoeUpArgs* a, int nb, int f32, int pdl, cudaStream_t st) {
     if (nb < 1 || nb > 65535 || a->n_experts < 1 || a->n_experts > 32 * MAXJ || a->top < 1 || a->top > MAX_TOP || a->top > a->n_experts || a->k < 8 || (a->k & 7) || (a->ldh & 3) ||
         a->n < 2 || (a->n & 1) || a->wrows < a->n || (a->ns & 1) || (a->ns && !a->ws) || a->ffp < a->n / 2 || a->ldo < a->top * a->ffp + a->ns / 2 || ((uintptr_t)a->h & 15) ||
-        ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15))
+        ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15) || a->real < 1 || a->real > a->n_experts || a->act < 0 || a->act > 2)
         return (int)cudaErrorInvalidValue;
     const long groups = (long)a->top * ((a->n + R - 1) / R) + (a->ns + R - 1) / R;
     const int ks = split_of(groups * nb, a->k >> 3, 1800), rgs = 8 / ks;
@@ -278,7 +315,7 @@ B2_API int b2_moe_up_rows(const MoeUpArgs* a, int nb, int f32, int pdl, cudaStre
 
 B2_API int b2_moe_down_rows(const MoeDownArgs* a, int nb, int f32, int pdl, cudaStream_t st) {
     if (nb < 1 || nb > 65535 || a->top < 1 || a->top > MAX_TOP || a->ffp < 8 || (a->ffp & 7) || (a->sfp & 7) || (a->sfp && !a->ws) || a->n < 1 || a->wrows < a->n || (a->lda & 3) ||
-        a->lda < a->top * a->ffp + a->sfp || ((uintptr_t)a->a & 15) || ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15))
+        a->lda < a->top * a->ffp + a->sfp || ((uintptr_t)a->a & 15) || ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15) || a->real < 1)
         return (int)cudaErrorInvalidValue;
     const long groups = (a->n + R - 1) / R;
     const int ks = split_of(groups * nb, (a->top * a->ffp + a->sfp) >> 3, 16000), rgs = 8 / ks;

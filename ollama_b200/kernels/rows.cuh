@@ -32,6 +32,20 @@ __device__ __forceinline__ size_t paged_row(const int* table, int pos, int n_kv_
     return ((size_t)table[pos >> PAGE_SHIFT] * n_kv_heads + kvh) * PAGE + (pos & (PAGE - 1));
 }
 
+// Keys that the query at a position sees: not later ones, and with chunk > 0 those of its chunk of positions, with window > 0 the last `window` up to itself
+// and the first `keep` of the sequence.
+__device__ __forceinline__ int first_key(int pos, int chunk, int window) { return chunk > 0 ? pos - pos % chunk : window > 0 ? max(0, pos - window + 1) : 0; }
+// Tiles of `tile` keys ahead of the one that holds position `first` which contain kept keys.
+__device__ __forceinline__ int kept_tiles(int keep, int first, int tile) { return min((keep + tile - 1) / tile, first / tile); }
+
+// Sigmoid gate of attention results: kind 1 one number per element, 2 one per head; before the sigmoid.
+struct HeadGate {
+    const float* g;          // [rows][ld]
+    int ld, kind;
+};
+__device__ __forceinline__ float sigmoid_f(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+__device__ __forceinline__ float sigmoid_exact(float v) { return 1.f / (1.f + expf(-v)); }
+
 static inline int launch_rows(const void* fn, dim3 grid, dim3 block, size_t smem, void** args, cudaStream_t st, int pdl) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;

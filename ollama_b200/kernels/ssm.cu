@@ -26,13 +26,15 @@ struct SsmConvArgs {
     const void* xz;          // [rows][ldx], x in the first `inner` columns
     int ldx, inner, taps;    // inner: padded to a multiple of 8
     const float* w;          // [taps][inner]
-    const float* b;          // [inner]
-    const float* state;      // [slots][taps - 1][inner], oldest first
+    const float* b;          // [inner] or null
+    float* state;            // [slots][taps - 1][inner], oldest first
     const int* slots;        // [rows]
     const int* positions;    // [rows]
     const int* offs;         // [rows] index of the row within its sequence's portion
     void* u;                 // [rows][ldu]
     int ldu;
+    int silu;                // activation of the results
+    int shift;               // decode rows (one per slot): the state is moved on by the row's input
 };
 
 // Gates of the 16-bit form: the exponential, quotient and logarithm of the special-function unit; log(1 + e) of a small e by its series,
@@ -75,7 +77,7 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ S
     const int c = 4 * (blockIdx.x * 128 + threadIdx.x);
     pdl_launch();
     if (c >= a.inner) return;
-    const float4 bias = *(const float4*)(a.b + c);
+    const float4 bias = a.b ? *(const float4*)(a.b + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     constexpr int W = TAPS > 0 ? TAPS : 1;
     float w[W][4], win[W][4];
     if (TAPS > 0) {
@@ -87,7 +89,7 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ S
     auto finish = [&](int r, float (&acc)[4]) {
         T* o = (T*)a.u + (size_t)r * a.ldu + c;
 #pragma unroll
-        for (int i = 0; i < 4; i++) acc[i] = silu_of<T>(acc[i]);
+        for (int i = 0; i < 4; i++) acc[i] = a.silu ? silu_of<T>(acc[i]) : acc[i];
         if (sizeof(T) == 2) {
             const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1]), hi = __floats2bfloat162_rn(acc[2], acc[3]);
             *(uint2*)o = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
@@ -103,6 +105,7 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ S
                 conv_input<T>(a, r, a.taps - 1 - j, c, v);
                 const float4 wj = *(const float4*)(a.w + (size_t)j * a.inner + c);
                 acc[0] += wj.x * v[0]; acc[1] += wj.y * v[1]; acc[2] += wj.z * v[2]; acc[3] += wj.w * v[3];
+                if (a.shift && j > 0) *(float4*)(a.state + ((size_t)a.slots[r] * (a.taps - 1) + j - 1) * a.inner + c) = make_float4(v[0], v[1], v[2], v[3]);
             }
             finish(r, acc);
         }
@@ -142,6 +145,10 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const __grid_constant__ S
 #pragma unroll
                 for (int j = 0; j < W - 1; j++) win[j][i] = win[j + 1][i];
             }
+            if (a.shift) {
+#pragma unroll
+                for (int j = 0; j < W - 1; j++) *(float4*)(a.state + ((size_t)a.slots[r] * (W - 1) + j) * a.inner + c) = *(const float4*)win[j];
+            }
             finish(r, acc);
         }
     }
@@ -165,6 +172,35 @@ B2_API int b2_ssm_conv(const SsmConvArgs* a, int rows, int f32, int pdl, cudaStr
     void* args[] = {&c, &rows, &per};
     const dim3 grid((a->inner + 511) / 512, (rows + per - 1) / per);
     return launch_rows(f32 ? pick_conv<float>(a->taps) : pick_conv<__nv_bfloat16>(a->taps), grid, dim3(128), 0, args, st, pdl);
+}
+
+// The last taps - 1 inputs of every portion become its slot's state.  grid (channels / 256, portions)
+struct ConvKeepArgs {
+    const void* xz;          // [rows][ldx]
+    int ldx, inner, taps;
+    float* state;            // [slots][taps - 1][inner], oldest first
+    const int4* seg;         // [n_seg] (first row, rows, slot, position of the first row)
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) conv_keep_kernel(const __grid_constant__ ConvKeepArgs a) {
+    const int c = blockIdx.x * 256 + threadIdx.x;
+    pdl_launch();
+    pdl_wait();
+    if (c >= a.inner) return;
+    const int4 sg = a.seg[blockIdx.y];
+    float* cs = a.state + (size_t)sg.z * (a.taps - 1) * a.inner + c;
+    for (int i = 0; i < a.taps - 1; i++) {
+        const int src = sg.y - (a.taps - 1) + i;      // ascending: an entry is read before it is overwritten
+        cs[(size_t)i * a.inner] = src >= 0 ? to_f(((const T*)a.xz)[(size_t)(sg.x + src) * a.ldx + c]) : sg.w > 0 ? cs[(size_t)(i + sg.y) * a.inner] : 0.f;
+    }
+}
+
+B2_API int b2_conv_keep(const ConvKeepArgs* a, int n_seg, int f32, int pdl, cudaStream_t st) {
+    if (n_seg < 1 || n_seg > 65535 || a->inner < 1 || a->taps < 2 || a->ldx < a->inner) return (int)cudaErrorInvalidValue;
+    ConvKeepArgs c = *a;
+    void* args[] = {&c};
+    return launch_rows(f32 ? (const void*)conv_keep_kernel<float> : (const void*)conv_keep_kernel<__nv_bfloat16>, dim3((a->inner + 255) / 256, n_seg), dim3(256), 0, args, st, pdl);
 }
 
 struct SsmScanArgs {

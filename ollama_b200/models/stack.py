@@ -8,11 +8,11 @@ from __future__ import annotations
 
 import json
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Any
 
 # checkpoint "architecture" -> GGUF architecture of the designs described this way
-STACK_ARCHS = {"Vazatar": "vazatar", "Kavenex": "kavenex"}
+STACK_ARCHS = {"Vazatar": "vazatar", "Kavenex": "kavenex", "Tirudra": "tirudra"}
 
 
 @dataclass(frozen=True)
@@ -23,10 +23,17 @@ class Design:
     loop_join: str                    # "product": a pass begins with a matrix over [stream | embedding output]; "add": with sums of vectors
     ff_act: str                       # activation of dense feed-forwards
     interleaved: bool                 # rotary pairs are (2i, 2i + 1), otherwise (i, i + dims / 2)
+    post_norm: bool = False           # the result of a mixer or feed-forward is normalised before it is added to the stream
+    mixers: dict[str, dict] = field(default_factory=dict)     # mixer name -> fields of its class that its configuration does not give
+    experts: dict[str, Any] = field(default_factory=dict)     # the same of ExpertMLP
 
 
-DESIGNS = {"Vazatar": Design(True, "rms_one_plus", "product", "relu2", False),
-           "Kavenex": Design(False, "layer", "add", "gelu_tanh", True)}
+DESIGNS = {"Vazatar": Design(True, "rms_one_plus", "product", "relu2", False, mixers={"attention": {"qk_norm": "row", "mask": "chunk"}}),
+           "Kavenex": Design(False, "layer", "add", "gelu_tanh", True, experts={"act": "swiglu_oai", "scoring": "chosen", "router_bias": True}),
+           "Tirudra": Design(False, "rms_one_plus", "", "", False, post_norm=True,
+                             mixers={"attention": {"qk_norm": "head", "mask": "window", "gate": "element"},
+                                     "attention_2": {"qk_norm": "head", "mask": "window", "gate": "head", "bias": True, "keys_as_values": True}},
+                             experts={"act": "silu", "scoring": "all", "correction": True, "shared_gate": True})}
 GATED_ACTS = ("gelu_tanh", "swiglu_oai")
 SWIGLU_ALPHA = 1.702                  # sigmoid slope of the clamped gated unit
 
@@ -34,16 +41,35 @@ SWIGLU_ALPHA = 1.702                  # sigmoid slope of the clamped gated unit
 @dataclass(frozen=True)
 class Rotation:
     """Rotary embedding of the first ``dims`` dimensions, in the half-split order or interleaved.  ``scaling`` (factor, low, high, original): frequencies
-    of wavelengths beyond original / low are divided by factor, those below original / high kept, blended in between."""
+    of wavelengths beyond original / low are divided by factor, those below original / high kept, blended in between.  ``yarn`` (factor, original, fast,
+    slow): pairs that turn at least ``fast`` times within ``original`` positions keep their frequency, those that turn at most ``slow`` times have it divided by
+    factor, with a ramp over the pair's index in between, and the rotated vectors grow by ``magnitude``."""
     dims: int
     base: float
     scaling: tuple[float, float, float, float] | None = None
     interleaved: bool = False
+    yarn: tuple[float, float, float, float] | None = None
+
+    @property
+    def magnitude(self) -> float:
+        return 1.0 if self.yarn is None else 0.1 * math.log(self.yarn[0]) + 1.0
+
+    def _ramp(self) -> tuple[float, float]:
+        """First and last pair index of the ramp."""
+        _, original, fast, slow = self.yarn
+
+        def index(turns: float) -> float:
+            return self.dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+        return max(math.floor(index(fast)), 0), min(math.ceil(index(slow)), self.dims - 1)
 
     def freqs(self) -> list[float]:
         out = []
+        lo, hi = self._ramp() if self.yarn is not None else (0, 0)
         for i in range(self.dims // 2):
             f = self.base ** (-2.0 * i / self.dims)
+            if self.yarn is not None:
+                r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+                f = f / self.yarn[0] * r + f * (1.0 - r)
             if self.scaling is not None:
                 factor, low, high, original = self.scaling
                 wave = 2.0 * math.pi / f
@@ -66,6 +92,29 @@ class AttentionMixer:
     softcap: float = 0.0
     chunk: int = 0                    # > 0: position p sees the keys from floor(p / chunk) * chunk on
     rot: Rotation | None = None
+    qk_norm: str = "row"              # RMS norm of queries and keys: "row" over the whole projection, "head" over each head with one weight vector for all
+    window: int = 0                   # > 0: position p sees the keys from p - window + 1 on,
+    keep: int = 0                     # and the first ``keep`` keys of the sequence
+    conv: int = 0                     # > 0: taps of a causal convolution over time on every channel of q, k and v
+    gate: str = ""                    # sigmoid gate of the heads' results: "element", "head" (one number each) or none
+    bias: bool = False                # of the q and k projections
+    keys_as_values: bool = False      # the values are the projected keys, before norm and rotation
+
+    @property
+    def n_q(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def n_k(self) -> int:
+        return self.kv_heads * self.dim
+
+    @property
+    def n_v(self) -> int:
+        return 0 if self.keys_as_values else self.kv_heads * self.vdim
+
+    @property
+    def n_gate(self) -> int:
+        return {"element": self.heads * self.vdim, "head": self.heads, "": 0}[self.gate]
 
 
 @dataclass(frozen=True)
@@ -89,7 +138,28 @@ class MambaMixer:
     conv: int                         # taps of the causal convolution
 
 
-Mixer = AttentionMixer | LatentMixer | MambaMixer
+@dataclass(frozen=True)
+class Mamba2Mixer:
+    """State-space mixer with one decay per head: a state of [vdim, state] per head, B and C shared by the heads of a group; the gated result is
+    normalised in ``norm_groups`` equal parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        """Of the convolution."""
+        return self.inner + 2 * self.groups * self.state
+
+
+Mixer = AttentionMixer | LatentMixer | MambaMixer | Mamba2Mixer
 
 
 @dataclass(frozen=True)
@@ -104,18 +174,31 @@ class DenseMLP:
 
 @dataclass(frozen=True)
 class Expert:
-    """Gated feed-forward min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1)."""
+    """One expert's hidden size, and the limit of gate and up where its activation has one."""
     ff: int
     limit: float = math.inf
 
 
 @dataclass(frozen=True)
 class ExpertMLP:
-    """``top`` of ``experts`` feed-forwards per token, weighted by the softmax over the chosen router logits; ``shared`` runs for every token."""
+    """``top`` of ``experts`` feed-forwards per token; ``shared`` runs for every token.  Activations: "swiglu_oai" is min(g, limit) sigmoid(1.702 min(g, limit))
+    (clamp(u, -limit, limit) + 1), "silu" g sigmoid(g) u.  Scoring "chosen": the largest router logits, weighted by the softmax over those alone; "all": the largest of
+    softmax plus ``correction``, weighted by the softmax over all outputs as it is."""
     experts: int
     top: int
     expert: Expert
     shared: Expert | None = None
+    act: str = "swiglu_oai"
+    scoring: str = "chosen"
+    router_bias: bool = False
+    correction: bool = False          # a vector that is added for the choice only
+    shared_gate: bool = False         # the shared expert is multiplied by the sigmoid of a number per token
+    identity: int = 0                 # router outputs behind the experts' that stand for the input itself
+
+    @property
+    def outputs(self) -> int:
+        """Of the router."""
+        return self.experts + self.identity
 
 
 @dataclass(frozen=True)
@@ -143,6 +226,7 @@ class Stack:
     design: Design = DESIGNS["Vazatar"]
     residual_mult: float = 1.0
     side_dim: int = 0                 # > 0: every layer adds an input of its own per token, a vector of this size
+    logit_scale: float = 1.0
 
     def runs(self) -> list[LayerRun]:
         """Layer runs in order; each has a cache or state of its own."""
@@ -161,11 +245,14 @@ class Stack:
     def state_bytes(self) -> int:
         """Recurrent state of one sequence over all layer runs (fp32)."""
         ms = [self.layers[r.layer].mixer for r in self.runs()]
-        return sum(4 * m.inner * (m.state + m.conv - 1) for m in ms if isinstance(m, MambaMixer))
+        return 4 * (sum(m.inner * (m.state + m.conv - 1) for m in ms if isinstance(m, MambaMixer))
+                    + sum(m.inner * m.state + m.channels * (m.conv - 1) for m in ms if isinstance(m, Mamba2Mixer))
+                    + sum((m.n_q + m.n_k + m.n_v) * (m.conv - 1) for m in ms if isinstance(m, AttentionMixer) and m.conv))
 
     @property
     def recurrent(self) -> bool:
-        return any(isinstance(L.mixer, MambaMixer) for L in self.layers)
+        """Whether a sequence has state besides its cached keys and values: a prefix of it cannot be taken up again in the middle."""
+        return any(isinstance(L.mixer, (MambaMixer, Mamba2Mixer)) or (isinstance(L.mixer, AttentionMixer) and L.mixer.conv > 1) for L in self.layers)
 
 
 def _rotation(r: dict[str, Any] | None, dim: int, interleaved: bool = False) -> Rotation | None:
@@ -175,22 +262,34 @@ def _rotation(r: dict[str, Any] | None, dim: int, interleaved: bool = False) -> 
     if dims % 2 or not 0 < dims <= dim:
         raise ValueError(f"rotary embedding of {dims} of {dim} dimensions")
     s = r.get("scaling")
+    if s and "fast" in s:
+        return Rotation(dims, float(r["base"]), None, interleaved, tuple(float(s[k]) for k in ("factor", "original", "fast", "slow")))
     return Rotation(dims, float(r["base"]), tuple(float(s[k]) for k in ("factor", "low", "high", "original")) if s else None, interleaved)
 
 
 def _mixer(kind: str, m: dict[str, Any], design: Design) -> Mixer:
-    if kind == "attention":
+    if kind in design.mixers and kind.startswith("attention"):
         H, G, d = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
         if G < 1 or H % G:
             raise ValueError(f"{H} query heads on {G} key/value heads")
-        return AttentionMixer(H, G, d, int(m.get("vdim") or d), float(m["scale"]), float(m.get("softcap") or 0.0),
-                              int((m.get("mask") or {}).get("size") or 0), _rotation(m.get("rot"), d, design.interleaved))
+        fixed = dict(design.mixers[kind])
+        mask, keys = m.get("mask") or {}, fixed.get("keys_as_values", False)
+        vdim, span = int(m.get("vdim") or d), {fixed.pop("mask"): int(mask.get("size") or 0)}
+        if keys and vdim != d:
+            raise ValueError(f"values of {vdim} dimensions that are keys of {d}")
+        return AttentionMixer(H, G, d, vdim, float(m["scale"]), float(m.get("softcap") or 0.0), rot=_rotation(m.get("rot"), d, design.interleaved),
+                              keep=int(mask.get("keep_first") or 0), conv=int(m.get("conv") or 0), **span, **fixed)
     if kind == "latent_attention":
         r = int(m.get("rot_dim") or 0)
         rot = _rotation({**(m.get("rot") or {}), "dims": r}, r, design.interleaved) if r else None
         return LatentMixer(int(m["heads"]), int(m["dim"]), r, int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]), rot)
     if kind == "mamba1":
         return MambaMixer(int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"]))
+    if kind == "mamba2":
+        mix = Mamba2Mixer(int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"]), int(m["conv"]), int(m.get("norm_groups") or 1))
+        if mix.heads % mix.groups or mix.inner % mix.norm_groups:
+            raise ValueError(f"{mix.heads} heads in {mix.groups} groups, {mix.inner} channels in {mix.norm_groups} norm groups")
+        return mix
     raise NotImplementedError(f"unknown mixer {kind!r}")
 
 
@@ -206,10 +305,10 @@ def _mlp(m: dict[str, Any] | None, design: Design) -> DenseMLP | ExpertMLP | Non
     if kind == "dense":
         return DenseMLP(int(m["ff"]), design.ff_act)
     if kind == "moe":
-        n, top = int(m["router"]["experts"]), int(m["router"]["top"])
-        if not 0 < top <= n:
-            raise ValueError(f"{top} of {n} experts")
-        return ExpertMLP(n, top, _expert(m["expert"]), _expert(m["shared"]) if m.get("shared") else None)
+        n, top, same = int(m["router"]["experts"]), int(m["router"]["top"]), int(m["router"].get("identity") or 0)
+        if not 0 < top <= n + same:
+            raise ValueError(f"{top} of {n + same} experts")
+        return ExpertMLP(n, top, _expert(m["expert"]), _expert(m["shared"]) if m.get("shared") else None, identity=same, **design.experts)
     raise NotImplementedError(f"unknown feed-forward {kind!r}")
 
 
@@ -224,6 +323,7 @@ def parse_stack(cfg: dict[str, Any] | str) -> Stack:
         loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
         if not 0 <= loop[0] < loop[1] <= len(layers) or loop[2] < 1:
             raise ValueError(f"loop {loop} over {len(layers)} layers")
-    scale, mult = (cfg.get("embedding") or {}).get("scale"), cfg.get("residual_mult")
+    scale, mult, out = (cfg.get("embedding") or {}).get("scale"), cfg.get("residual_mult"), cfg.get("logit_scale")
     return Stack(layers, loop or None, 1.0 if scale is None else float(scale), float(cfg["norm"]["eps"]), int(cfg["width"]), int(cfg["vocab"]),
-                 float(cfg.get("logit_softcap") or 0.0), design, 1.0 if mult is None else float(mult), int((cfg.get("token_side") or {}).get("dim") or 0))
+                 float(cfg.get("logit_softcap") or 0.0), design, 1.0 if mult is None else float(mult), int((cfg.get("token_side") or {}).get("dim") or 0),
+                 1.0 if out is None else float(out))

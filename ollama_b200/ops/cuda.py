@@ -120,7 +120,7 @@ class GluArgs(C.Structure):
 
 class MoeRouteArgs(C.Structure):
     _fields_ = [("logits", C.c_void_p), ("ld", C.c_int), ("n_experts", C.c_int), ("k", C.c_int), ("mode", C.c_int), ("norm_topk", C.c_int),
-                ("e_lo", C.c_int), ("e_cnt", C.c_int), ("ids", C.c_void_p), ("lids", C.c_void_p), ("wts", C.c_void_p)]
+                ("e_lo", C.c_int), ("e_cnt", C.c_int), ("ids", C.c_void_p), ("lids", C.c_void_p), ("wts", C.c_void_p), ("correction", C.c_void_p)]
 
 
 class MoeCombineArgs(C.Structure):
@@ -158,12 +158,14 @@ class AttnDecodeArgs(C.Structure):
     _fields_ = [("q", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("positions", C.c_void_p),
                 ("slots", C.c_void_p), ("n_heads", C.c_int), ("n_kv_heads", C.c_int), ("n_ctx", C.c_int), ("n_splits", C.c_int),
                 ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int), ("part_acc", C.c_void_p), ("part_ml", C.c_void_p),
-                ("k_scale", C.c_void_p), ("v_scale", C.c_void_p), ("page_table", C.c_void_p), ("max_pages", C.c_int), ("chunk", C.c_int)]
+                ("k_scale", C.c_void_p), ("v_scale", C.c_void_p), ("page_table", C.c_void_p), ("max_pages", C.c_int), ("chunk", C.c_int),
+                ("keep", C.c_int)]
 
 
 class AttnRopeArgs(C.Structure):
     _fields_ = [("qkv", C.c_void_p), ("inv_freq", C.c_void_p), ("mscale", C.c_float), ("n_rot", C.c_int), ("neox", C.c_int),
-                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float), ("ldq", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("freqs", C.c_void_p)]
+                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float), ("ldq", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("freqs", C.c_void_p),
+                ("head_norm", C.c_int), ("v_off", C.c_int)]
 
 
 class AttnCombineArgs(C.Structure):
@@ -681,15 +683,26 @@ def moe_gather(h: torch.Tensor, row_of_pair: torch.Tensor, k: int, rows: int) ->
     return xs
 
 
+class MoeScatterArgs(C.Structure):
+    _fields_ = [("ys", C.c_void_p), ("row_of_pair", C.c_void_p), ("wts", C.c_void_p), ("k", C.c_int), ("d", C.c_int), ("out", C.c_void_p), ("ldo", C.c_int),
+                ("accumulate", C.c_int), ("mult", C.c_float), ("ids", C.c_void_p), ("n_experts", C.c_int), ("h", C.c_void_p), ("ldh", C.c_int), ("f32", C.c_int),
+                ("shared", C.c_void_p), ("lds", C.c_int), ("gate", C.c_void_p), ("ldg", C.c_int)]
+
+
 def moe_scatter_combine(ys: torch.Tensor, row_of_pair: torch.Tensor, wts: torch.Tensor, tokens: int, k: int, out: torch.Tensor | None = None,
-                        accumulate: bool = False, mult: float = 1.0) -> torch.Tensor:
-    """out[t] (+)= mult * sum over t's slots of their weight times the sorted buffer's row."""
+                        accumulate: bool = False, mult: float = 1.0, ids: torch.Tensor | None = None, n_experts: int = 0, h: torch.Tensor | None = None,
+                        shared: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """out[t] (+)= mult * (sum over t's slots of their weight times the sorted buffer's row).  ``ids``: slots whose choice is ``n_experts`` or above add their weight times
+    h[t].  ``shared``: rows that are added too, times the sigmoid of ``gate`` [tokens, 1] where that is given."""
     d = ys.shape[1]
     if out is None:
         out = torch.empty(tokens, d, dtype=torch.float32, device=ys.device)
+    a = MoeScatterArgs(ptr(ys), ptr(row_of_pair), ptr(wts), k, d, ptr(out), out.stride(0), int(accumulate), mult, ptr(ids), n_experts, ptr(h),
+                       h.stride(0) if h is not None else 0, int(h is not None and h.dtype == torch.float32), ptr(shared), shared.stride(0) if shared is not None else 0,
+                       ptr(gate), gate.stride(0) if gate is not None else 0)
     f = lib().b2_moe_scatter_combine
-    f.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_int, C.c_float, C.c_void_p]
-    _check(f(ptr(ys), ptr(row_of_pair), ptr(wts), tokens, k, d, ptr(out), out.stride(0), int(accumulate), mult, stream()), "moe_scatter_combine")
+    f.argtypes = [C.c_void_p, C.c_int, C.c_void_p]
+    _check(f(C.addressof(a), tokens, stream()), "moe_scatter_combine")
     return out
 
 

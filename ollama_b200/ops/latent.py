@@ -6,7 +6,7 @@ import ctypes as C
 import torch
 
 from .cuda import MoeRouteArgs, _check, lib, ptr, stream
-from .rows import F, I, P, _call, _is32, _st
+from .rows import ACT, GLU_BASE, F, I, P, _call, _is32, _st
 
 LatentStepArgs = _st("LatentStepArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("dim", I), ("rot", I), ("rank", I), ("norm", P), ("eps", F), ("freqs", P),
                                         ("interleaved", I), ("rows", P), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I), ("cache", P),
@@ -20,9 +20,10 @@ LatentAttnArgs = _st("LatentAttnArgs", [("q", P), ("cache", P), ("rows", P), ("p
 AttnPartsArgs = _st("AttnPartsArgs", [("q", P), ("kv", P), ("shared", P), ("n_rows", I), ("dp", I), ("vp", I), ("rp", I), ("tiles", P), ("H", I), ("vdim", I),
                                       ("ldo", I), ("scale", F), ("out", P)])
 MoeUpArgs = _st("MoeUpArgs", [("z", P), ("ldz", I), ("n_experts", I), ("top", I), ("h", P), ("ldh", I), ("k", I), ("w", P), ("n", I), ("wrows", I), ("ws", P),
-                              ("ns", I), ("limit", F), ("limit_s", F), ("out", P), ("ldo", I), ("ffp", I), ("ids", P), ("wts", P)])
+                              ("ns", I), ("limit", F), ("limit_s", F), ("out", P), ("ldo", I), ("ffp", I), ("ids", P), ("wts", P),
+                              ("correction", P), ("real", I), ("act", I)])
 MoeDownArgs = _st("MoeDownArgs", [("a", P), ("lda", I), ("top", I), ("ffp", I), ("sfp", I), ("ids", P), ("wts", P), ("w", P), ("ws", P), ("n", I), ("wrows", I),
-                                  ("x", P), ("ldx", I), ("mult", F)])
+                                  ("x", P), ("ldx", I), ("mult", F), ("store", I), ("real", I), ("h", P), ("ldh", I), ("gate", P), ("ldg", I)])
 
 NOT_SUPPORTED = 801                # cudaErrorNotSupported: the launch does not take the shape, nothing ran
 
@@ -77,27 +78,31 @@ def attn_prefill_parts(q: torch.Tensor, kv: torch.Tensor, shared: torch.Tensor, 
     _call("b2_attn_prefill_parts", a, tiles.shape[0])
 
 
-def moe_route(z: torch.Tensor, experts: int, top: int) -> tuple[torch.Tensor, torch.Tensor]:
-    """Experts [rows, top] of router logits and their weights: the largest logits, softmax over those."""
+def moe_route(z: torch.Tensor, outputs: int, top: int, experts: int | None = None, correction: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+    """Router outputs [rows, top] chosen by logits ``z``, the same with -1 for those that are no experts, and their weights: the largest logits and the softmax over those,
+    or with a ``correction`` the largest of softmax + correction and that softmax."""
     n = z.shape[0]
     ids, lids = torch.empty(2, n, top, device=z.device, dtype=torch.int32)
     wts = torch.empty(n, top, device=z.device)
-    a = MoeRouteArgs(ptr(z), z.stride(0), experts, top, 1, 0, 0, experts, ptr(ids), ptr(lids), ptr(wts))
+    a = MoeRouteArgs(ptr(z), z.stride(0), outputs, top, 1 if correction is None else 2, 0, 0, outputs if experts is None else experts, ptr(ids), ptr(lids), ptr(wts), ptr(correction))
     _call("b2_moe_route", a, n, 0)
-    return lids, wts
+    return ids, lids, wts
 
 
 def moe_up_rows(z: torch.Tensor, h: torch.Tensor, nb: int, w: torch.Tensor, n: int, out: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, *, experts: int, top: int,
-                ffp: int, limit: float, ws: torch.Tensor | None = None, ns: int = 0, limit_s: float = 0.0, pdl: bool = False) -> None:
-    """Hidden columns of the chosen experts (and of the shared one, ``ws``) of up to four rows; ``w`` [experts, rows, k] with gate / up interleaved."""
-    a = MoeUpArgs(ptr(z), z.stride(0), experts, top, ptr(h), h.stride(0), w.shape[2], ptr(w), n, w.shape[1], ptr(ws), ns, limit, limit_s, ptr(out), out.stride(0), ffp,
-                  ptr(ids), ptr(wts))
+                ffp: int, limit: float, ws: torch.Tensor | None = None, ns: int = 0, limit_s: float = 0.0, act: str = "glu:swiglu_oai", outputs: int | None = None,
+                correction: torch.Tensor | None = None, pdl: bool = False) -> None:
+    """Hidden columns of the chosen experts (and of the shared one, ``ws``) of up to four rows; ``w`` [experts, rows, k] with gate / up interleaved.  The choice is
+    that of :func:`moe_route` among ``outputs`` router outputs."""
+    a = MoeUpArgs(ptr(z), z.stride(0), experts if outputs is None else outputs, top, ptr(h), h.stride(0), w.shape[2], ptr(w), n, w.shape[1], ptr(ws), ns, limit, limit_s, ptr(out),
+                  out.stride(0), ffp, ptr(ids), ptr(wts), ptr(correction), experts, ACT[act] - GLU_BASE)
     _call("b2_moe_up_rows", a, nb, _is32(w), int(pdl))
 
 
 def moe_down_rows(a_rows: torch.Tensor, nb: int, ids, wts, w: torch.Tensor, x: torch.Tensor, *, top: int, n: int, mult: float, ws: torch.Tensor | None = None,
-                  pdl: bool = False) -> None:
-    """x += mult * (sum of weight * w[id] a over the chosen experts, plus the shared expert's product); ``w`` [experts, rows, ffp]."""
+                  store: bool = False, h: torch.Tensor | None = None, gate: torch.Tensor | None = None, pdl: bool = False) -> None:
+    """x += mult * (sum of weight * w[id] a over the chosen experts, plus the shared expert's product); ``w`` [experts, rows, ffp].  Choices beyond the experts are the
+    input ``h`` itself; ``gate`` [rows, 1]: the shared expert's product is multiplied by its sigmoid; ``store``: the result replaces x."""
     a = MoeDownArgs(ptr(a_rows), a_rows.stride(0), top, w.shape[2], ws.shape[1] if ws is not None else 0, ptr(ids), ptr(wts), ptr(w), ptr(ws), n, w.shape[1], ptr(x),
-                    x.stride(0), mult)
+                    x.stride(0), mult, int(store), w.shape[0], ptr(h), h.stride(0) if h is not None else 0, ptr(gate), gate.stride(0) if gate is not None else 0)
     _call("b2_moe_down_rows", a, nb, _is32(w), int(pdl))

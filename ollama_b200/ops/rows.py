@@ -32,17 +32,20 @@ GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P),
                                     ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
                                     ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
-                                    ("conv_b", P), ("conv_state", P), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
+                                    ("conv_b", P), ("conv_state", P), ("conv_silu", I), ("conv_shift", I), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
                                     ("h", P), ("ldh", I), ("hb", P), ("mul_row", P)])
 PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
                                           ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
-                                          ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I)])
+                                          ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I),
+                                          ("head_norm", I), ("v_off", I), ("mscale", F)])
+HeadGate = _st("HeadGate", [("g", P), ("ld", I), ("kind", I)])
 PagedAttnArgs = _st("PagedAttnArgs", [("q", P), ("dq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("k_cache", P), ("v_cache", P),
                                       ("dk", I), ("dv", I), ("cache32", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
-                                      ("chunk", I), ("scale", F), ("softcap", F), ("out", P), ("ldo", I), ("out16", I)])
-AttnPagedArgs = _st("AttnPagedArgs", [("tiles", P), ("page_table", P), ("max_pages", I), ("chunk", I), ("vdim", I), ("ldo", I)])
+                                      ("chunk", I), ("scale", F), ("softcap", F), ("out", P), ("ldo", I), ("out16", I), ("window", I), ("keep", I), ("gate", HeadGate)])
+AttnPagedArgs = _st("AttnPagedArgs", [("tiles", P), ("page_table", P), ("max_pages", I), ("chunk", I), ("vdim", I), ("ldo", I), ("window", I), ("keep", I), ("gate", HeadGate)])
 SsmConvArgs = _st("SsmConvArgs", [("xz", P), ("ldx", I), ("inner", I), ("taps", I), ("w", P), ("b", P), ("state", P), ("slots", P), ("positions", P),
-                                  ("offs", P), ("u", P), ("ldu", I)])
+                                  ("offs", P), ("u", P), ("ldu", I), ("silu", I), ("shift", I)])
+ConvKeepArgs = _st("ConvKeepArgs", [("xz", P), ("ldx", I), ("inner", I), ("taps", I), ("state", P), ("seg", P)])
 SsmScanArgs = _st("SsmScanArgs", [("xz", P), ("ldx", I), ("off_z", I), ("u", P), ("ldu", I), ("dt", P), ("lddt", I), ("bc", P), ("ldbc", I), ("off_b", I),
                                   ("dt_bias", P), ("a2", P), ("d", P), ("inner", I), ("n_state", I), ("taps", I), ("state", P), ("conv_state", P), ("seg", P),
                                   ("out", P), ("ldo", I)])
@@ -91,9 +94,9 @@ def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = Non
 def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC_ROWS, eps: float = 0.0, kn: int = 0, x2: torch.Tensor | None = None,
          k1: int = 0, conv=None, conv_out: torch.Tensor | None = None, slots: torch.Tensor | None = None, positions: torch.Tensor | None = None,
          h: torch.Tensor | None = None, hb: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
-         pdl: bool = False) -> None:
-    """Products of up to four matrices with up to four source rows.  ``conv`` = (weights [taps, n], bias [n], state [slots, taps - 1, n]): the first n
-    results of the first matrix also run through that convolution and SiLU, into ``conv_out``.  ``h``: the normalised
+         conv_silu: bool = True, conv_shift: bool = False, pdl: bool = False) -> None:
+    """Products of up to four matrices with up to four source rows.  ``conv`` = (weights [taps, n], bias [n] or None, state [slots, taps - 1, n]): the first n
+    results of the first matrix also run through that convolution, and with ``conv_silu`` SiLU, into ``conv_out``; ``conv_shift``: they enter the state.  ``h``: the normalised
     rows for the first matrix are stored too (``hb``: a layer norm's bias)."""
     a = GemvRowsArgs()
     for i, s in enumerate(segs):
@@ -107,7 +110,7 @@ def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC
     if conv is not None:
         a.conv_seg, a.conv_n, a.taps = 0, conv[0].shape[1], conv[0].shape[0]
         a.conv_w, a.conv_b, a.conv_state, a.conv_out, a.ldu = ptr(conv[0]), ptr(conv[1]), ptr(conv[2]), ptr(conv_out), conv_out.stride(0)
-        a.slots, a.positions = ptr(slots), ptr(positions)
+        a.slots, a.positions, a.conv_silu, a.conv_shift = ptr(slots), ptr(positions), int(conv_silu), int(conv_shift)
     _call("b2_gemv_rows", a, int(pdl))
 
 
@@ -140,46 +143,67 @@ def _split_floats(m: int, n: int, k: int) -> int:
     return int(f(m, n, k))
 
 
-def paged_append(qkv, *, heads, kv_heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, positions, slots, table, q_out, k_cache, v_cache, pdl=False) -> None:
-    """Norm over the whole q / k projections, rotation, q to padded fp32 rows [rows, H, dq], k and v into the paged caches."""
+NO_GATE = HeadGate(None, 0, 0)
+
+
+def head_gate(g: torch.Tensor, kind: str) -> HeadGate:
+    """Rows ``g`` of gate values, before the sigmoid: "element" one for each result column, "head" one for each head."""
+    return HeadGate(ptr(g), g.stride(0), {"element": 1, "head": 2}[kind])
+
+
+def paged_append(qkv, *, heads, kv_heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, positions, slots, table, q_out, k_cache, v_cache, head_norm=False, v_off=None,
+                 mscale=1.0, pdl=False) -> None:
+    """Norm over the whole q / k projections (``head_norm``: over each head), rotation, q to padded fp32 rows [rows, H, dq], k and v (columns from ``v_off`` on) into
+    the paged caches."""
+    v_off = (heads + kv_heads) * dim if v_off is None else v_off
     a = PagedAppendArgs(ptr(qkv), qkv.stride(0), heads, kv_heads, dim, vdim, ptr(q_norm), ptr(k_norm), eps, ptr(freqs), n_rot, ptr(positions), ptr(slots),
-                        ptr(table), table.shape[1], ptr(q_out), q_out.shape[2], ptr(k_cache), ptr(v_cache), k_cache.shape[3], v_cache.shape[3], _is32(k_cache))
+                        ptr(table), table.shape[1], ptr(q_out), q_out.shape[2], ptr(k_cache), ptr(v_cache), k_cache.shape[3], v_cache.shape[3], _is32(k_cache),
+                        int(head_norm), v_off, mscale)
     _call("b2_paged_append", a, qkv.shape[0], int(pdl))
 
 
-def paged_attn(q, k_cache, v_cache, positions, slots, table, out, *, dim, vdim, scale, softcap=0.0, chunk=0, pdl=False) -> None:
+def paged_attn(q, k_cache, v_cache, positions, slots, table, out, *, dim, vdim, scale, softcap=0.0, chunk=0, window=0, keep=0, gate=NO_GATE, pdl=False) -> None:
     """Attention of any head size over a paged cache: q [rows, H, dq] fp32 -> out[row, h * vdim ...]."""
     a = PagedAttnArgs(ptr(q), q.shape[2], q.shape[1], k_cache.shape[1], dim, vdim, ptr(k_cache), ptr(v_cache), k_cache.shape[3], v_cache.shape[3], _is32(k_cache),
-                      ptr(positions), ptr(slots), ptr(table), table.shape[1], chunk, scale, softcap, ptr(out), out.stride(0), 1 - _is32(out))
+                      ptr(positions), ptr(slots), ptr(table), table.shape[1], chunk, scale, softcap, ptr(out), out.stride(0), 1 - _is32(out), window, keep, gate)
     _call("b2_paged_attn", a, q.shape[0], int(pdl))
 
 
-def attn_prefill_paged(q, k_cache, v_cache, tiles, table, out, *, vdim, scale, softcap=0.0, chunk=0) -> None:
+def attn_prefill_paged(q, k_cache, v_cache, tiles, table, out, *, vdim, scale, softcap=0.0, chunk=0, window=0, keep=0, gate=NO_GATE) -> None:
     """tcgen05 attention of query tiles ([n, 4] int32: first row, rows, slot, position) over a paged f16 cache of row length 64 or 128."""
     a = AttnPrefillArgs(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), None, q.shape[0], q.shape[1], k_cache.shape[1], 0, 0, 0, 0, 1, 0, scale, softcap, None, None)
-    pg = AttnPagedArgs(ptr(tiles), ptr(table), table.shape[1], chunk, vdim, out.stride(0))
+    pg = AttnPagedArgs(ptr(tiles), ptr(table), table.shape[1], chunk, vdim, out.stride(0), window, keep, gate)
     _check(lib().b2_attn_prefill_paged(C.byref(a), C.byref(pg), q.shape[2], tiles.shape[0], k_cache.shape[0], stream()), "attn_prefill_paged")
 
 
 def attn_decode_paged(qkv, k_cache, v_cache, positions, slots, table, out, nb, *, heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, scale, softcap,
-                      chunk, n_splits, n_ctx, part_acc, part_ml, pdl=False) -> bool:
-    """Decode attention on raw projections: norms, rotation, cache append, split-K attention, merge.  False: shape not taken, nothing launched."""
-    hd = k_cache.shape[3]
-    a = AttnDecodeArgs(None, ptr(k_cache), ptr(v_cache), ptr(positions), ptr(slots), heads, k_cache.shape[1], n_ctx, n_splits, scale, softcap, 0,
-                       ptr(part_acc), ptr(part_ml), None, None, ptr(table), table.shape[1], chunk)
-    r = AttnRopeArgs(ptr(qkv), None, 1.0, n_rot, 1, ptr(q_norm), ptr(k_norm), eps, qkv.stride(0), dim, vdim, ptr(freqs))
+                      chunk, n_splits, n_ctx, part_acc, part_ml, window=0, keep=0, head_norm=False, v_off=None, mscale=1.0, gate=NO_GATE, pdl=False) -> bool:
+    """Decode attention on raw projections: norms, rotation, cache append, split-K attention, merge and gate.  False: shape not taken, nothing launched."""
+    hd, G = k_cache.shape[3], k_cache.shape[1]
+    v_off = (heads + G) * dim if v_off is None else v_off
+    a = AttnDecodeArgs(None, ptr(k_cache), ptr(v_cache), ptr(positions), ptr(slots), heads, G, n_ctx, n_splits, scale, softcap, window,
+                       ptr(part_acc), ptr(part_ml), None, None, ptr(table), table.shape[1], chunk, keep)
+    r = AttnRopeArgs(ptr(qkv), None, mscale, n_rot, 1, ptr(q_norm), ptr(k_norm), eps, qkv.stride(0), dim, vdim, ptr(freqs), int(head_norm), v_off)
     f = lib().b2_attn_decode_paged
-    f.argtypes = [P, P, I, I, P, I, I, I, P]
-    rc = f(C.addressof(a), C.addressof(r), nb, hd, ptr(out), out.stride(0), 1 - _is32(out), int(pdl), stream())
+    f.argtypes = [P, P, I, I, P, I, I, P, I, P]
+    rc = f(C.addressof(a), C.addressof(r), nb, hd, ptr(out), out.stride(0), 1 - _is32(out), C.addressof(gate), int(pdl), stream())
     if rc == 801:
         return False
     _check(rc, "attn_decode_paged")
     return True
 
 
-def ssm_conv(xz, inner, w, b, state, slots, positions, offs, u, pdl=False) -> None:
-    a = SsmConvArgs(ptr(xz), xz.stride(0), inner, w.shape[0], ptr(w), ptr(b), ptr(state), ptr(slots), ptr(positions), ptr(offs), ptr(u), u.stride(0))
+def ssm_conv(xz, inner, w, b, state, slots, positions, offs, u, silu=True, shift=False, pdl=False) -> None:
+    """Causal convolution over time of the first ``inner`` columns, each with ``w`` [taps, inner]; ``shift``: rows of one token per slot, which enter the state."""
+    a = SsmConvArgs(ptr(xz), xz.stride(0), inner, w.shape[0], ptr(w), ptr(b), ptr(state), ptr(slots), ptr(positions), ptr(offs), ptr(u), u.stride(0), int(silu), int(shift))
     _call("b2_ssm_conv", a, xz.shape[0], _is32(xz), int(pdl))
+
+
+def conv_keep(xz, inner, taps, state, segs, pdl=False) -> None:
+    """The last taps - 1 rows of every portion (``segs`` [n, 4] int32: first row, rows, slot, position) become its slot's convolution state."""
+    if taps > 1:
+        a = ConvKeepArgs(ptr(xz), xz.stride(0), inner, taps, ptr(state), ptr(segs))
+        _call("b2_conv_keep", a, segs.shape[0], _is32(xz), int(pdl))
 
 
 def ssm_scan(xz, off_z, u, dt, bc, off_b, dt_bias, a2, d, taps, state, conv_state, segs, out, pdl=False) -> None:

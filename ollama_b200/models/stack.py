@@ -29,11 +29,11 @@ class Design:
 
 
 DESIGNS = {"Vazatar": Design(True, "rms_one_plus", "product", "relu2", False, mixers={"attention": {"qk_norm": "row", "mask": "chunk"}}),
-           "Kavenex": Design(False, "layer", "add", "gelu_tanh", True, experts={"act": "swiglu_oai", "scoring": "chosen", "router_bias": True}),
+           "Kavenex": Design(False, "layer", "add", "gelu_tanh", True, experts={"act": "swiglu_oai", "scoring": "chosen"}),
            "Tirudra": Design(False, "rms_one_plus", "", "", False, post_norm=True,
                              mixers={"attention": {"qk_norm": "head", "mask": "window", "gate": "element"},
                                      "attention_2": {"qk_norm": "head", "mask": "window", "gate": "head", "bias": True, "keys_as_values": True}},
-                             experts={"act": "silu", "scoring": "all", "correction": True, "shared_gate": True})}
+                             experts={"act": "silu", "scoring": "all", "router_bias": False, "correction": True, "shared_gate": True})}
 GATED_ACTS = ("gelu_tanh", "swiglu_oai")
 SWIGLU_ALPHA = 1.702                  # sigmoid slope of the clamped gated unit
 
@@ -190,7 +190,7 @@ class ExpertMLP:
     shared: Expert | None = None
     act: str = "swiglu_oai"
     scoring: str = "chosen"
-    router_bias: bool = False
+    router_bias: bool = True
     correction: bool = False          # a vector that is added for the choice only
     shared_gate: bool = False         # the shared expert is multiplied by the sigmoid of a number per token
     identity: int = 0                 # router outputs behind the experts' that stand for the input itself

@@ -54,8 +54,9 @@ SPECS: dict[str, ArchSpec] = {
     # dense models of the size of the stack models below, layer run by layer run (a gated FFN has three matrices for their two)
     "dense-1b": ArchSpec("llama", 20, 2048, 16, 4, 128, 5504, 32768, 500000.0),
     "dense-8b": ArchSpec("llama", 32, 4096, 32, 8, 128, 11008, 128256, 500000.0),
-    # a mixture-of-experts model of the size of kavenex-moe (whose shared expert counts as one more chosen expert)
+    # mixture-of-experts models of the size of kavenex-moe and tirudra-2k / 4k (whose shared expert counts as one more chosen expert)
     "experts-2k": ArchSpec("qwen3moe", 20, 2048, 16, 4, 128, 5504, 32768, 500000.0, 1e-6, n_experts=64, n_experts_used=5, d_ff_expert=1408),
+    "experts-4k": ArchSpec("qwen3moe", 12, 4096, 32, 8, 128, 8192, 65536, 500000.0, 1e-6, n_experts=32, n_experts_used=5, d_ff_expert=2048),
     # small stand-ins of every family for tests
     "tiny-tp": ArchSpec("llama", 2, 1024, 16, 8, 64, 4096, 4096, 500000.0, 1e-5, 4096),      # divides 2, 4 and 8 ways
     "tiny-qwen3": ArchSpec("qwen3", 2, 256, 4, 2, 64, 768, 4096, 1e6, 1e-6, 4096),
@@ -305,7 +306,23 @@ def latent_config(width: int, heads: int, dim: int, rot: int, vdim: int, rank: i
             "layers": [{"type": "latent_attention", "mixer": mix, "mlp": mlp[c]} for c in layers]}
 
 
+def heads_config(width: int, heads: int, kv_heads: int, dim: int, window: int, full_kv: int, ssm_heads: int, ssm_dim: int, state: int, groups: int, vocab: int, layers: str,
+                 experts: int, top: int, identity: int, ff_expert: int, ff_shared: int) -> dict:
+    """``config.json`` of a Tirudra model; ``layers``: one letter per layer, W (windowed attention), F (full attention), M (Mamba-2), in lower case without a feed-forward."""
+    mix = {"W": {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": 4, "mask": {"size": window, "keep_first": 4}, "scale": dim ** -0.5,
+                                               "rot": {"base": 10000.0, "dims": dim, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}},
+           "F": {"type": "attention_2", "mixer": {"heads": heads, "kv_heads": full_kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                 "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}},
+           "M": {"type": "mamba2", "mixer": {"heads": ssm_heads, "vdim": ssm_dim, "state": state, "groups": groups, "conv": 4, "norm_groups": groups}}}
+    moe = {"kind": "moe", "router": {"experts": experts, "identity": identity, "top": top}, "expert": {"ff": ff_expert}, "shared": {"ff": ff_shared}}
+    return {"architecture": "Tirudra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{**mix[c.upper()], "mlp": moe if c.isupper() else None} for c in layers]}
+
+
 STACK_SPECS: dict[str, dict] = {
+    "tiny-tirudra": heads_config(192, 6, 2, 48, 40, 3, 6, 32, 48, 2, 4096, "MWFm", 6, 2, 2, 96, 64),
+    "tirudra-2k": heads_config(2048, 16, 4, 128, 1024, 4, 64, 64, 128, 2, 32768, "MWMF" * 5, 64, 4, 4, 1408, 1408),
+    "tirudra-4k": heads_config(4096, 32, 8, 128, 1024, 8, 128, 64, 128, 8, 65536, "MWMF" * 3, 32, 4, 2, 2048, 2048),
     "tiny-kavenex": latent_config(192, 6, 40, 24, 48, 80, 384, 4096, "DED", (1, 3, 2), 24, 6, 2, 96, 64),
     "kavenex-1b": latent_config(2048, 16, 128, 64, 128, 512, 5504, 32768, "D" * 16, (0, 4, 2), 256),
     "kavenex-8b": latent_config(4096, 32, 128, 64, 128, 512, 11008, 128256, "D" * 28, (0, 4, 2), 256),
@@ -323,7 +340,8 @@ class SyntheticStackTensors:
         from ..convert.stack import map_stack_name
         self.seed, self.device, w = seed, device, cfg["width"]
         names: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], w), "head": (cfg["vocab"], w), "final.norm": (w,)}
-        seq = cfg["architecture"] == "Kavenex"       # mixer and feed-forward one after the other, layer norms, gated feed-forwards
+        seq = cfg["architecture"] == "Kavenex"       # layer norms, gated feed-forwards, a loop that begins with sums
+        post = cfg["architecture"] == "Tirudra"      # norms behind every part, a correction of the router and a gate of the shared expert instead of a bias
         if cfg.get("loop"):
             names.update({"loop.step": (cfg["loop"]["times"], w)} if seq else {"loop.in": (w, 2 * w)})
         side = (cfg.get("token_side") or {}).get("dim")
@@ -332,11 +350,22 @@ class SyntheticStackTensors:
         stacked: dict[str, tuple[int, ...]] = {}
         for i, L in enumerate(cfg["layers"]):
             m, p = L["mixer"], f"l{i}."
-            names[p + "norm1"] = (w,)
+            names.update({p + "norm1": (w,), **({p + "norm1b": (w,)} if post else {})})
             if L["type"] == "latent_attention":
                 H, d, r, dv, k = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
                 names.update({p + "mix.q": (H * (d + r), w), p + "mix.dkv": (k + r, w), p + "mix.dkv.norm": (k,), p + "mix.uk": (H * d, k), p + "mix.uv": (H * dv, k),
                               p + "mix.o": (w, H * dv)})
+            elif L["type"] == "mamba2":
+                H, c, bc = m["heads"], m["heads"] * m["vdim"], 2 * m["groups"] * m["state"]
+                names.update({p + "mix.in": (2 * c + bc + H, w), p + "mix.conv": (c + bc, m["conv"]), p + "mix.conv.b": (c + bc,), p + "mix.dt_bias": (H,), p + "mix.A_log": (H,),
+                              p + "mix.D": (H,), p + "mix.norm": (c,), p + "mix.o": (w, c)})
+            elif post:
+                H, nq, nk, nv = m["heads"], m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+                names.update({p + "mix.q": (nq, w), p + "mix.k": (nk, w), p + "mix.q.norm": (m["dim"],), p + "mix.k.norm": (m["dim"],), p + "mix.o": (w, H * m["vdim"])})
+                if L["type"] == "attention":
+                    names.update({p + "mix.v": (nv, w), p + "mix.g": (H * m["vdim"], w), **{p + f"mix.{n}.conv": (k, m["conv"]) for n, k in (("q", nq), ("k", nk), ("v", nv))}})
+                else:
+                    names.update({p + "mix.q.b": (nq,), p + "mix.k.b": (nk,), p + "mix.g": (H, w)})
             elif L["type"] == "attention":
                 nq, nk, nv, no = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
                 names.update({p + "mix.q": (nq, w), p + "mix.k": (nk, w), p + "mix.v": (nv, w), p + "mix.q.norm": (nq,), p + "mix.k.norm": (nk,), p + "mix.o": (w, no)})
@@ -346,12 +375,13 @@ class SyntheticStackTensors:
                               p + "mix.dt.b": (c,), p + "mix.A_log": (c, n), p + "mix.D": (c,), p + "mix.o": (w, c)})
             f = L.get("mlp")
             if f:
-                names[p + "norm2"] = (w,)
+                names.update({p + "norm2": (w,), **({p + "norm2b": (w,)} if post else {})})
             if f and f["kind"] == "dense":
                 names.update({p + "mlp.up": (f["ff"], w), p + "mlp.down": (w, f["ff"]), **({p + "mlp.gate": (f["ff"], w)} if seq else {})})
             elif f:
                 E, fe, fs = f["router"]["experts"], f["expert"]["ff"], (f.get("shared") or {}).get("ff")
-                names.update({p + "mlp.router": (E, w), p + "mlp.router.b": (E,)})
+                n = E + f["router"].get("identity", 0)
+                names.update({p + "mlp.router": (n, w), **({p + "mlp.correction": (n,), p + "mlp.shared.sg": (1, w)} if post else {p + "mlp.router.b": (n,)})})
                 for pre, fx in ((f"blk.{i}.ffn_%s_exps.weight", (E, fe)), (f"blk.{i}.ffn_%s_shexp.weight", (fs,))):
                     if fx[-1]:
                         stacked.update({pre % "gate": (*fx, w), pre % "up": (*fx, w), pre % "down": (*fx[:-1], w, fx[-1])})
@@ -372,8 +402,8 @@ class SyntheticStackTensors:
         s = self.table[name]
         x = random_tensor(name, s, self.seed, self.device)
         if name.endswith("ssm_a"):
-            x = -(1.0 + torch.arange(s[1], device=x.device, dtype=torch.float32)).expand(s).contiguous()
-        f32 = len(s) < 2 or name.endswith(("ssm_a", "ssm_conv1d.weight"))
+            x = -(1.0 + torch.arange(s[-1], device=x.device, dtype=torch.float32)).expand(s).contiguous()
+        f32 = len(s) < 2 or name.endswith(("ssm_a", "conv1d.weight"))
         raw = (x if f32 else x.to(torch.bfloat16)).contiguous().view(-1).view(torch.uint8)
         return QWeight(name, GGMLType.F32 if f32 else GGMLType.BF16, tuple(s), raw)
 

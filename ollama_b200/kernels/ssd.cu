@@ -2,38 +2,19 @@
 //
 //   dt = softplus(dt' + b),  S[p][n] <- exp(a dt) S[p][n] + dt x[p] B[n],  y[p] = sum_n S[p][n] C[n] + D x[p],  result y silu(z)
 //
-// A scan over prompt rows that carries the state through portions of any length, a decode step of one token per sequence, and the
-// RMS norm of the gated result in equal parts of a row.  x, B and C come convolved and activated (ssm.cu).  Step sizes, decays, state and norm are fp32;
+// A scan over prompt rows that carries the state through portions of any length (32-bit models; the 16-bit form is in ssd_chunk.cu), a decode step of one token
+// per sequence, and the RMS norm of the gated result in equal parts of a row.  x, B and C come convolved and activated (ssm.cu).  Step sizes, decays, state and norm are fp32;
 // the state advances as S + S expm1(a dt), which keeps the distance of a slow decay from 1 to full precision.
 //
 // Heads stand `vdim` columns apart (padded to a multiple of 8, pad columns zero), B and C have rows of n_state padded to a multiple of 16 per group.
 // A slot's state is [head][vdim][n_state]; a sequence at position 0 takes it as zeros.
-#include "rows.cuh"
-
-struct SsdArgs {
-    const void* u;           // [rows][ldu]: x from column 0, B of group g at off_b + g n_state, C at off_c + g n_state
-    int ldu, off_b, off_c;
-    const void* z;           // [rows][ldz]
-    int ldz;
-    const float* dt;         // [rows][lddt], before bias and softplus
-    int lddt;
-    const float* dt_bias;    // [heads]
-    const float* a;          // [heads], negative
-    const float* d;          // [heads]
-    int heads, groups, vdim, n_state;
-    float* state;            // [slots][heads][vdim][n_state]
-    const int4* seg;         // scan: [n_seg] (first row, rows, slot, position of the first row)
-    const int* slots;        // step: [rows]
-    const int* positions;    // step: [rows]
-    void* out;               // [rows][ldo]
-    int ldo;
-};
+#include "ssd.cuh"
 
 namespace {
 
 // LPC lanes share a channel and hold SPL state dimensions each.  Time runs in tiles of TT rows staged in shared memory; eight rows are advanced before
 // their partial sums over the state are reduced.
-template <typename T, int LPC, int SPL>
+template <int LPC, int SPL>
 __global__ void __launch_bounds__(128) ssd_scan_kernel(const __grid_constant__ SsdArgs a) {
     constexpr int CH = 128 / LPC, NP = LPC * SPL, TT = NP <= 128 ? 32 : 16, U = 8;
     constexpr int PER = TT * CH / 128;
@@ -52,10 +33,10 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const __grid_constant__ S
 #pragma unroll
     for (int i = 0; i < SPL; i++) S[i] = live && l * SPL + i < a.n_state && pos0 > 0 ? st[l * SPL + i] : 0.f;
     const float A = a.a[h], bias = a.dt_bias[h], dd = a.d[h];
-    const T* u = (const T*)a.u + (size_t)row0 * a.ldu;
-    const T* z = (const T*)a.z + (size_t)row0 * a.ldz + h * a.vdim;
+    const float* u = (const float*)a.u + (size_t)row0 * a.ldu;
+    const float* z = (const float*)a.z + (size_t)row0 * a.ldz + h * a.vdim;
     const float* pdt = a.dt + (size_t)row0 * a.lddt + h;
-    T* out = (T*)a.out + (size_t)row0 * a.ldo + h * a.vdim;
+    float* out = (float*)a.out + (size_t)row0 * a.ldo + h * a.vdim;
     const int lc = tid % CH, lt = tid / CH;      // element (lt + LPC * i, lc) of a tile is this thread's to move
     const bool lok = c0 + lc < a.vdim;
     for (int t0 = 0; t0 < rows; t0 += TT) {
@@ -67,16 +48,16 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const __grid_constant__ S
         for (int e = tid; e < TT * NP; e += 128) {
             const int t = e / NP, n = e % NP;
             const bool ok = t0 + t < rows && n < a.n_state;
-            const T* r = u + (size_t)(t0 + t) * a.ldu + g * a.n_state + n;
-            s_b[t][n] = ok ? to_f(r[a.off_b]) : 0.f;
-            s_c[t][n] = ok ? to_f(r[a.off_c]) : 0.f;
+            const float* r = u + (size_t)(t0 + t) * a.ldu + g * a.n_state + n;
+            s_b[t][n] = ok ? r[a.off_b] : 0.f;
+            s_c[t][n] = ok ? r[a.off_c] : 0.f;
         }
         float x[PER];
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < PER; i++) {
             const int t = lt + LPC * i;
-            x[i] = lok && t0 + t < rows ? to_f(u[(size_t)(t0 + t) * a.ldu + h * a.vdim + c0 + lc]) : 0.f;
+            x[i] = lok && t0 + t < rows ? u[(size_t)(t0 + t) * a.ldu + h * a.vdim + c0 + lc] : 0.f;
             s_dx[t][lc] = s_dt[t] * x[i];
         }
         __syncthreads();
@@ -118,7 +99,7 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const __grid_constant__ S
 #pragma unroll
         for (int i = 0; i < PER; i++) {
             const int t = lt + LPC * i;
-            if (lok && t0 + t < rows) out[(size_t)(t0 + t) * a.ldo + c0 + lc] = from_f<T>((s_y[t][lc] + dd * x[i]) * silu_f(to_f(z[(size_t)(t0 + t) * a.ldz + c0 + lc])));
+            if (lok && t0 + t < rows) out[(size_t)(t0 + t) * a.ldo + c0 + lc] = (s_y[t][lc] + dd * x[i]) * silu_f(z[(size_t)(t0 + t) * a.ldz + c0 + lc]);
         }
     }
     if (!live) return;
@@ -193,13 +174,12 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
     }
 }
 
-template <typename T>
 const void* pick_scan(int n, int& ch) {
-    if (n <= 16) { ch = 16; return (const void*)ssd_scan_kernel<T, 8, 2>; }
-    if (n <= 32) { ch = 16; return (const void*)ssd_scan_kernel<T, 8, 4>; }
-    if (n <= 64) { ch = 8; return (const void*)ssd_scan_kernel<T, 16, 4>; }
-    if (n <= 128) { ch = 8; return (const void*)ssd_scan_kernel<T, 16, 8>; }
-    if (n <= 256) { ch = 8; return (const void*)ssd_scan_kernel<T, 16, 16>; }
+    if (n <= 16) { ch = 16; return (const void*)ssd_scan_kernel<8, 2>; }
+    if (n <= 32) { ch = 16; return (const void*)ssd_scan_kernel<8, 4>; }
+    if (n <= 64) { ch = 8; return (const void*)ssd_scan_kernel<16, 4>; }
+    if (n <= 128) { ch = 8; return (const void*)ssd_scan_kernel<16, 8>; }
+    if (n <= 256) { ch = 8; return (const void*)ssd_scan_kernel<16, 16>; }
     return nullptr;
 }
 template <typename T>
@@ -221,8 +201,9 @@ bool bad_ssd(const SsdArgs* a) {
 // At most 256 state dimensions (more: cudaErrorNotSupported).  Both return a cudaError_t value.
 B2_API int b2_ssd_scan(const SsdArgs* a, int n_seg, int f32, int pdl, cudaStream_t st) {
     if (n_seg < 1 || n_seg > 65535 || bad_ssd(a) || !a->seg) return (int)cudaErrorInvalidValue;
+    if (!f32) return ssd_chunk_launch(*a, n_seg, pdl, st);
     int ch = 0;
-    const void* fn = f32 ? pick_scan<float>(a->n_state, ch) : pick_scan<__nv_bfloat16>(a->n_state, ch);
+    const void* fn = pick_scan(a->n_state, ch);
     if (!fn) return (int)cudaErrorNotSupported;
     SsdArgs c = *a;
     void* args[] = {&c};

@@ -5,9 +5,9 @@
 //   y_t = exp(l_t) S C_t + sum_{s <= t} (C_t . B_s) exp(l_t - l_s) dt_s x_s + D x_t,   S <- exp(l_63) S + sum_s exp(l_63 - l_s) dt_s x_s B_s^T
 //
 // One CTA walks over the chunks of one head (or of a part of its columns) of one portion.  The state stays in the accumulators of its warps, fp32: warp
-// (p, half) holds 16 columns times one half of the state dimensions, and feeds it to the products with C straight from there.  x, B and C are the 16-bit values that the
+// (p, part) holds 16 columns times a quarter of the state dimensions, and feeds it to the products with C straight from there.  x, B and C are the 16-bit values that the
 // convolution left; the fp32 factors of the products (the state, the decayed scores and the decayed steps) enter as the sum of two 16-bit numbers each, which
-// keeps 16 bits of them.  The results of the two halves meet in shared memory, where the gate is applied.  The next chunk's rows arrive by cp.async meanwhile.
+// keeps 16 bits of them.  The results of the parts meet in shared memory, where the gate is applied.  The next chunk's rows arrive by cp.async meanwhile.
 #include "ssd.cuh"
 
 namespace {
@@ -22,7 +22,7 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
 }
 __device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
@@ -39,21 +39,22 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
 // MT tiles of 16 columns, NP state dimensions (padded)
 template <int MT, int NP>
 struct Lay {
+    static constexpr int SP = NP >= 64 ? 4 : 2;                             // parts of the state dimensions
     static constexpr int LX = 16 * MT + PAD, LN = NP + PAD, LM = Q + PAD, LY = 16 * MT + 4;
     static constexpr int X = Q * LX * 2, BC = Q * LN * 2;                   // bytes of one stage
     static constexpr int OFF_B = 2 * X, OFF_C = OFF_B + 2 * BC, OFF_XH = OFF_C + 2 * BC, OFF_XL = OFF_XH + X, OFF_MH = OFF_XL + X, OFF_ML = OFF_MH + Q * LM * 2,
-                         OFF_Y = OFF_ML + Q * LM * 2, OFF_T = OFF_Y + 2 * Q * LY * 4, TOTAL = OFF_T + 2 * 4 * Q * 4;
+                         OFF_Y = OFF_ML + Q * LM * 2, OFF_T = OFF_Y + SP * Q * LY * 4, TOTAL = OFF_T + 2 * 4 * Q * 4;
 };
 
 template <int MT, int NP>
-__global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_constant__ SsdArgs a) {
+__global__ void __launch_bounds__(32 * MT * Lay<MT, NP>::SP, 1) ssd_chunk_kernel(const __grid_constant__ SsdArgs a) {
     using L = Lay<MT, NP>;
-    constexpr int THREADS = 64 * MT, PT = 16 * MT, NT = NP / 16;             // NT: accumulator tiles of 8 state dimensions per warp
+    constexpr int SP = L::SP, WARPS = MT * SP, THREADS = 32 * WARPS, PT = 16 * MT, NT = NP / 8 / SP;      // NT: accumulator tiles of 8 state dimensions per warp
     constexpr int ITEMS = Q * PT / 8 / THREADS;                               // 16-byte pieces of a column tile per thread
     typedef __nv_bfloat16 bf;
     extern __shared__ __align__(16) uint8_t sm[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-    const int pt = warp % MT, half = warp / MT, h = blockIdx.y, grp = h / (a.heads / a.groups), p0 = blockIdx.x * PT, np = min(PT, a.vdim - p0);
+    const int pt = warp % MT, part = warp / MT, h = blockIdx.y, grp = h / (a.heads / a.groups), p0 = blockIdx.x * PT, np = min(PT, a.vdim - p0);
     bf *sXh = (bf*)(sm + L::OFF_XH), *sXl = (bf*)(sm + L::OFF_XL), *sMh = (bf*)(sm + L::OFF_MH), *sMl = (bf*)(sm + L::OFF_ML);
     float *sY = (float*)(sm + L::OFF_Y), *sT = (float*)(sm + L::OFF_T);
     pdl_launch();
@@ -86,14 +87,22 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    // per row of chunk c: l, dt, exp(l), exp(l_63 - l) dt; by one warp, two rows a lane
+    // per row of chunk c: l, dt, exp(l), exp(l_63 - l) dt; by one warp, two rows a lane, whose inputs it has fetched a chunk ahead
+    constexpr int STEP_WARP = WARPS == 16 ? 12 : WARPS - 1;              // of 16 warps one that has no block of scores
+    float raw[2];
+    auto fetch_steps = [&](int c) {
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int r = min(c * Q + 2 * lane + i, rows - 1);
+            raw[i] = a.dt[(size_t)(row0 + r) * a.lddt + h];
+        }
+    };
     auto steps = [&](int c) {
         float* t = sT + (c & 1) * 4 * Q;
         float dt[2], l[2];
 #pragma unroll
         for (int i = 0; i < 2; i++) {
-            const int r = c * Q + 2 * lane + i;
-            dt[i] = r < rows ? softplus_f(a.dt[(size_t)(row0 + r) * a.lddt + h] + bias) : 0.f;
+            dt[i] = c * Q + 2 * lane + i < rows ? softplus_f(raw[i] + bias) : 0.f;
             l[i] = A * dt[i];
         }
         float s = l[0] + l[1];
@@ -115,11 +124,15 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
     };
 
     request(0);
-    if (warp == 0) steps(0);
-    // this warp's part of the state: columns p0 + 16 pt + (g, g + 8), dimensions half * NP / 2 + 8 j + 2 tq + (0, 1)
+    if (warp == STEP_WARP) {
+        fetch_steps(0);
+        steps(0);
+        fetch_steps(1);
+    }
+    // this warp's part of the state: columns p0 + 16 pt + (g, g + 8), dimensions part * NP / SP + 8 j + 2 tq + (0, 1)
     float S[NT][4];
     float* st = a.state + (((size_t)sg.z * a.heads + h) * a.vdim + p0) * a.n_state;
-    const int pr = 16 * pt + g, nc = half * (NP / 2) + 2 * tq;
+    const int pr = 16 * pt + g, nc = part * (NP / SP) + 2 * tq;
 #pragma unroll
     for (int j = 0; j < NT; j++)
 #pragma unroll
@@ -147,15 +160,16 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
         __syncthreads();                     // chunk c has arrived, its predecessor is done with
         if (c + 1 < n_chunks) {
             request(c + 1);
-            if (warp == 2 * MT - 1) steps(c + 1);
+            if (warp == STEP_WARP) {
+                steps(c + 1);
+                fetch_steps(c + 2);
+            }
         }
-        // decayed scores of 16 rows t and the blocks of 16 s of one half
-        for (int w = warp; w < 8; w += 2 * MT) {
-            const int tt = w & 3, hh = w >> 2;
+        // decayed scores of blocks of 16 rows t and 16 rows s
 #pragma unroll
-            for (int i = 0; i < 2; i++) {
-                const int b = hh ? 1 + i : 3 * i;
-                if (b > tt) continue;
+        for (int w = warp; w < 16; w += WARPS) {
+            const int tt = w & 3, b = w >> 2;
+            if (b <= tt) {
                 float m[2][4] = {};
 #pragma unroll
                 for (int kk = 0; kk < NP / 16; kk++) {
@@ -192,7 +206,7 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
             *(uint4*)(sXh + r * L::LX + k) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
             *(uint4*)(sXl + r * L::LX + k) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
-        // y^T of all rows, over this half's state dimensions
+        // y^T of all rows, over this part of the state dimensions
         float y[Q / 8][4] = {};
 #pragma unroll
         for (int kk = 0; kk < NT / 2; kk++) {
@@ -204,7 +218,7 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
 #pragma unroll
             for (int j = 0; j < Q / 8; j += 2) {
                 uint32_t cb[4];
-                ldsm4(cb, sC + (8 * j + rK) * L::LN + half * (NP / 2) + 16 * kk + cK);
+                ldsm4(cb, sC + (8 * j + rK) * L::LN + part * (NP / SP) + 16 * kk + cK);
                 mma(y[j], hi, cb[0], cb[1]);
                 mma(y[j + 1], hi, cb[2], cb[3]);
                 mma(y[j], lo, cb[0], cb[1]);
@@ -218,8 +232,8 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
         }
         __syncthreads();                     // scores and decayed steps are there
 #pragma unroll
-        for (int i = 0; i < 2; i++) {
-            const int b = half ? 1 + i : 3 * i;
+        for (int i = 0; i < 4 / SP; i++) {
+            const int b = SP == 4 ? part : part ? 1 + i : 3 * i;
             uint32_t xa[4];
             ldsm4t(xa, sX + (16 * b + rK) * L::LX + 16 * pt + cK);
 #pragma unroll
@@ -234,7 +248,7 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
                 mma(y[j + 1], xa, ml[2], ml[3]);
             }
         }
-        float* yo = sY + half * Q * L::LY + 16 * pt;
+        float* yo = sY + part * Q * L::LY + 16 * pt;
 #pragma unroll
         for (int j = 0; j < Q / 8; j++) {
             const int t = 8 * j + 2 * tq;
@@ -255,28 +269,33 @@ __global__ void __launch_bounds__(64 * MT, 1) ssd_chunk_kernel(const __grid_cons
 #pragma unroll
             for (int j = 0; j < NT; j += 2) {
                 uint32_t bb[4];
-                ldsm4t(bb, sB + (16 * kk + rV) * L::LN + half * (NP / 2) + 8 * j + cV);
+                ldsm4t(bb, sB + (16 * kk + rV) * L::LN + part * (NP / SP) + 8 * j + cV);
                 mma(S[j], xh, bb[0], bb[1]);
                 mma(S[j + 1], xh, bb[2], bb[3]);
                 mma(S[j], xl, bb[0], bb[1]);
                 mma(S[j + 1], xl, bb[2], bb[3]);
             }
         }
-        __syncthreads();                     // both halves of y
+        __syncthreads();                     // all parts of y
 #pragma unroll
         for (int i = 0; i < ITEMS; i++) {
             const int e = tid + THREADS * i, t = e / (PT / 8), k = 8 * (e % (PT / 8)), r = c * Q + t;
             if (r >= rows || k >= np) continue;
             const float* y0 = sY + t * L::LY + k;
-            const float* y1 = y0 + Q * L::LY;
             const uint4 v = *(const uint4*)(sX + t * L::LX + k);
             const uint32_t xq[4] = {v.x, v.y, v.z, v.w}, zq[4] = {zv[i].x, zv[i].y, zv[i].z, zv[i].w};
             uint32_t o[4];
 #pragma unroll
             for (int j = 0; j < 4; j++) {
-                const float2 p = *(const float2*)(y0 + 2 * j), q = *(const float2*)(y1 + 2 * j);
+                float2 y = *(const float2*)(y0 + 2 * j);
+#pragma unroll
+                for (int k2 = 1; k2 < SP; k2++) {
+                    const float2 q = *(const float2*)(y0 + k2 * Q * L::LY + 2 * j);
+                    y.x += q.x;
+                    y.y += q.y;
+                }
                 const float z0 = __uint_as_float(zq[j] << 16), z1 = __uint_as_float(zq[j] & 0xffff0000u);
-                const float v0 = (p.x + q.x + dd * __uint_as_float(xq[j] << 16)) * z0 * sigmoid_f(z0), v1 = (p.y + q.y + dd * __uint_as_float(xq[j] & 0xffff0000u)) * z1 * sigmoid_f(z1);
+                const float v0 = (y.x + dd * __uint_as_float(xq[j] << 16)) * z0 * sigmoid_f(z0), v1 = (y.y + dd * __uint_as_float(xq[j] & 0xffff0000u)) * z1 * sigmoid_f(z1);
                 const __nv_bfloat162 b2 = __floats2bfloat162_rn(v0, v1);
                 o[j] = *reinterpret_cast<const uint32_t*>(&b2);
             }
@@ -297,7 +316,7 @@ int launch(const SsdArgs& a, int n_seg, int pdl, cudaStream_t st) {
     if (once.first()) cudaFuncSetAttribute(ssd_chunk_kernel<MT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
     SsdArgs c = a;
     void* args[] = {&c};
-    return launch_rows((const void*)ssd_chunk_kernel<MT, NP>, dim3((a.vdim + 16 * MT - 1) / (16 * MT), a.heads, n_seg), dim3(64 * MT), L::TOTAL, args, st, pdl);
+    return launch_rows((const void*)ssd_chunk_kernel<MT, NP>, dim3((a.vdim + 16 * MT - 1) / (16 * MT), a.heads, n_seg), dim3(32 * MT * L::SP), L::TOTAL, args, st, pdl);
 }
 
 template <int MT>

@@ -79,9 +79,10 @@ def measure(name: str, steps: int, warmup: int, dev: str = "cuda:0") -> dict:
     out = {"model": name, "weights_per_pass": n, "prompt": {"tokens": PROMPT, "tok_s": round(PROMPT / t, 1), "roofline": round(2 * (n - head) * PROMPT / t / flops, 3)}}
     for nb in BATCHES:
         slots = list(range(nb))
-        for s in slots:
-            be.prefill(s, toks[:CONTEXT], 0, need_logits=False)
-        t = timed(lambda: be.decode_loop(slots, [1] * nb, [CONTEXT] * nb, LOOP), warmup, steps) / LOOP
+        for s in slots:               # sequences of their own, which choose experts of their own
+            be.prefill(s, torch.randint(0, cfg.vocab_size, (CONTEXT,), generator=gen).tolist(), 0, need_logits=False)
+        first = torch.randint(0, cfg.vocab_size, (nb,), generator=gen).tolist()
+        t = timed(lambda: be.decode_loop(slots, first, [CONTEXT] * nb, LOOP), warmup, steps) / LOOP
         byts = 2 * (dense + routed * (1.0 - (1.0 - share) ** nb)) + nb * cfg.kv_bytes_per_token() * CONTEXT
         out[f"decode_{nb}"] = {"tok_s": round(nb / t, 1), "step_us": round(t * 1e6, 1), "roofline": round(byts / t / hbm, 3), "launches": be.launches_per_step}
     from ..ops import cuda as K

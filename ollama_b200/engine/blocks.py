@@ -6,7 +6,7 @@ Each class holds a layer's weights, laid out for the kernels, and adds its resul
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass, field
+from dataclasses import dataclass
 
 import torch
 
@@ -290,8 +290,9 @@ class GatedFFN:
 @dataclass
 class _Shared:
     e: Expert
-    gu: Mat = field(default=None)
-    down: Mat = field(default=None)
+    gu: Mat
+    down: Mat
+    gu_router: Mat
 
 
 class ExpertFFN:
@@ -303,16 +304,20 @@ class ExpertFFN:
         parts = [(0, 0, p + "ffn_gate_inp.weight", (n, w))]
         if m.shared is not None and m.shared_gate:
             parts.append((n, 0, p + "ffn_gate_inp_shexp.weight", (1, w)))
-        self.router = Mat(src.pack(parts, up(n + len(parts) - 1), src.wp), bias=src.vec(p + "ffn_gate_inp.bias", E) if m.router_bias else None)
+        router, bias = src.pack(parts, up(n + len(parts) - 1), src.wp), src.vec(p + "ffn_gate_inp.bias", E) if m.router_bias else None
         self.correction = src.vec(p + "exp_probs_b.bias", n) if m.correction else None
         self.gu = src.gate_up(p + "ffn_gate_exps.weight", p + "ffn_up_exps.weight", m.expert.ff, (E,))
         self.down = src.zeros(E, src.wp, self.ffp)
         self.down[:, :w, :m.expert.ff] = src.tensor(p + "ffn_down_exps.weight", E, w, m.expert.ff)
         self.shared = None
-        if m.shared is not None:
+        if m.shared is not None:              # its gate / up and the router stand below one another: one product of many rows gives both
             ff = m.shared.ff
-            self.shared = _Shared(m.shared, Mat(src.gate_up(p + "ffn_gate_shexp.weight", p + "ffn_up_shexp.weight", ff)),
-                                  Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff))))
+            gu = torch.cat([src.gate_up(p + "ffn_gate_shexp.weight", p + "ffn_up_shexp.weight", ff), router])
+            n_gu = 2 * up(ff)
+            router = gu[n_gu:]
+            both = Mat(gu, torch.cat([torch.zeros(n_gu, device=src.device), bias]) if bias is not None else None)
+            self.shared = _Shared(m.shared, Mat(gu[:n_gu]), Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff))), both)
+        self.router = Mat(router, bias)
         if not f32 and norm.b is not None:
             self.router.fold(norm)
 
@@ -323,7 +328,13 @@ class ExpertFFN:
     def run(self, s: Step) -> None:
         m, sh, post, mult = self.m, self.shared, self.post, s.be.stack.residual_mult
         z = s.buf("router", self.router.w.shape[0], torch.float32)
-        h = s.normed(self.norm, self.router, z, keep=True)
+        both = sh is not None and not s.small and s.act == torch.bfloat16
+        if both:
+            h, fs = s.rows(self.norm), s.buf("shared", up(sh.e.ff), zero=True)
+            O.gemm(h, sh.gu_router.w, fs, act=self.act, limit=sh.e.limit, bias=sh.gu_router.bias, tail=z)
+            s.launched()
+        else:
+            h = s.normed(self.norm, self.router, z, keep=True)
         gate = z[:, m.outputs:m.outputs + 1] if sh and m.shared_gate else None
         out = s.x if post is None else s.buf("y", s.be.wp, torch.float32)
         if post is not None:
@@ -347,15 +358,16 @@ class ExpertFFN:
             O.gemm(f, self.down.view(-1, self.ffp), y, experts=m.experts, tile_expert=tile_expert)
             more, late = {"ids": ids, "n_experts": m.experts, "h": h} if m.identity else {}, post is None and gate is None
             if sh:
-                f = s.buf("shared", up(sh.e.ff), zero=True)
-                s.product(h, sh.gu, f, act=self.act, limit=sh.e.limit)
+                if not both:
+                    fs = s.buf("shared", up(sh.e.ff), zero=True)
+                    s.product(h, sh.gu, fs, act=self.act, limit=sh.e.limit)
                 if not late:
                     more["shared"], more["gate"] = s.buf("shared_y", s.be.wp, torch.float32), gate
-                    s.product(f, sh.down, more["shared"])
+                    s.product(fs, sh.down, more["shared"])
             K.moe_scatter_combine(y, row, wts, s.nb, m.top, out=out, accumulate=post is None, mult=mult, **more)
             s.launched(6)
             if sh and late:
-                s.add(f, sh.down)
+                s.add(fs, sh.down)
         if post is not None:
             s.leave(out, post)
 

@@ -130,7 +130,7 @@ class StateSpaceHeads:
         n_in = self.inner + self.ch
         w_in = src.zeros(n_in + up(H), src.wp)                           # z | x B C | step sizes
         w_in[:self.inner, :w], w_in[self.inner:n_in, :w], w_in[n_in:n_in + H, :w] = heads(z, H, P, self.vp), channels(xbc), dt
-        self.w_in, self.w_dt = Mat(w_in[:n_in]), Mat(w_in[n_in:])
+        self.w_all, self.w_in, self.w_dt = w_in, Mat(w_in[:n_in]), Mat(w_in[n_in:])
         self.conv_w = channels(src.tensor(p + "ssm_conv1d.weight", m.channels, m.conv).float()).t().contiguous()
         self.conv_b = channels(src.tensor(p + "ssm_conv1d.bias", m.channels).float())
         self.dt_bias, self.a, self.d = src.vec(p + "ssm_dt.bias", H), src.vec(p + "ssm_a", H), src.vec(p + "ssm_d", H)
@@ -156,8 +156,12 @@ class StateSpaceHeads:
                    conv_shift=True, slots=s.m.slots, positions=s.m.positions, pdl=s.pdl)
             s.launched()
         else:
-            s.product(h, self.w_in, zx)
-            s.product(h, self.w_dt, dt)
+            if be.f32:
+                s.product(h, self.w_in, zx)
+                s.product(h, self.w_dt, dt)
+            else:
+                O.gemm(h, self.w_all, zx, tail=dt)
+                s.launched()
             O.ssm_conv(xbc, self.ch, *conv, s.m.slots, s.m.positions, s.m.offs, u, shift=s.decode, pdl=s.pdl)
             if not s.decode:
                 O.conv_keep(xbc, self.ch, m.conv, conv_state, s.m.segs)
@@ -168,6 +172,12 @@ class StateSpaceHeads:
             D.ssd_step(*args, s.m.slots, s.m.positions, out, pdl=s.pdl)
         else:
             D.ssd_scan(*args, s.m.segs, out, pdl=s.pdl)
-        D.group_norm(out, m.heads, m.vdim, self.vp, m.norm_groups, self.g, be.stack.eps, pdl=s.pdl)
-        s.launched(2)
-        s.result(out, self.w_o, self.post)
+        s.launched()
+        if s.small and m.norm_groups == 1 and self.post is not None:        # one root mean square per row: the product applies it to its results
+            y = s.buf("y", be.wp, f32)
+            O.gemv([O.seg(self.w_o.w, be.wp, y, self.g)], self.inner, out, s.nb, be.f32, O.SRC_NORM, be.stack.eps, m.inner, pdl=s.pdl)
+            s.leave(y, self.post)
+        else:
+            D.group_norm(out, m.heads, m.vdim, self.vp, m.norm_groups, self.g, be.stack.eps, pdl=s.pdl)
+            s.result(out, self.w_o, self.post)
+        s.launched()

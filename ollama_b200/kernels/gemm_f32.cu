@@ -86,7 +86,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
 // k, lda and ldb multiples of four, n even for gated products, bases 16-byte aligned.  Returns a cudaError_t value.
 B2_API int b2_gemm_rows_f32(const GemmRowsArgs* g, cudaStream_t st) {
     const int glu = g->act >= GLU_BASE ? 1 : 0;
-    if (g->m < 1 || g->n < 1 || g->k < 4 || (g->k & 3) || (g->lda & 3) || (g->ldb & 3) || ((uintptr_t)g->a & 15) || ((uintptr_t)g->b & 15) || g->out_type || g->copy || g->act < 0 ||
+    if (g->m < 1 || g->n < 1 || g->k < 4 || (g->k & 3) || (g->lda & 3) || (g->ldb & 3) || ((uintptr_t)g->a & 15) || ((uintptr_t)g->b & 15) || g->out_type || g->copy || g->tail || g->act < 0 ||
         (!glu && g->act > 2) || g->act > GLU_BASE + 2 || (glu && ((g->n & 1) || g->accumulate || g->mul)) || (g->mul && !g->mul_row) ||
         (g->tile_expert && (g->experts < 1 || (g->m & 127))))
         return (int)cudaErrorInvalidValue;

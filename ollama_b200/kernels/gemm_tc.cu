@@ -54,6 +54,8 @@ struct GemmParams {
     int ldm;
     __nv_bfloat16* copy;    // fp32 results also go here as bf16, rows of pitch ldo
     int lda;                // row pitch of a, 0: k
+    float* tail;            // sums of the columns from tail_col on go here, rows of ld_tail
+    int tail_col, ld_tail;
     // split-K (splits > 1): part s of a tile covers its own range of k blocks and stores plain fp32 sums at part + s * part_stride
     // ([m][part_ld]); a second kernel adds the parts in order and applies the epilogue
     int splits;
@@ -130,7 +132,8 @@ __device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, i
     }
 }
 
-template <int BN, bool SPLIT>
+// TAIL: some columns are p.tail's.  A form of its own, since a test per stored element made all products 8 % longer.
+template <int BN, bool SPLIT, bool TAIL>
 __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                                                               const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -271,6 +274,19 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                 __syncwarp();
                 float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (p.bias && col < p.n) bias = *(const float4*)(p.bias + (size_t)e * p.n + col);
+                if (TAIL && n0 + c0 + 32 > p.tail_col) {      // warp-uniform
+#pragma unroll 1
+                    for (int rr = 0; rr < 8; rr++) {
+                        const int lr = rr * 4 + sub, row = mt * BM + q * 32 + lr;
+                        if (row >= p.m || col >= p.n) continue;
+                        float4 r = *(const float4*)(st + lr * L::EPI_LD + cq);
+                        r.x += bias.x; r.y += bias.y; r.z += bias.z; r.w += bias.w;
+                        if (col >= p.tail_col) *(float4*)(p.tail + (size_t)row * p.ld_tail + col - p.tail_col) = r;
+                        else store4(p, r, row, col, make_float4(0.f, 0.f, 0.f, 0.f));
+                    }
+                    __syncwarp();
+                    continue;
+                }
 #pragma unroll
                 for (int rr = 0; rr < 8; rr++) {
                     const int lr = rr * 4 + sub;
@@ -313,31 +329,32 @@ int sm_count() {
     return n;
 }
 
-template <int BN, bool SPLIT = false>
+template <int BN, bool SPLIT = false, bool TAIL = false>
 int launch(const void* a, const void* b, const GemmParams& p, cudaStream_t st, int b_rows = 0) {
     CUtensorMap ma, mb;
     if (!make_map(&ma, a, p.m, p.k, BM, p.lda) || !make_map(&mb, b, b_rows ? b_rows : p.n, p.k, BN)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
+    if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN, SPLIT, TAIL>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
     const int total = ((p.m + BM - 1) / BM) * ((p.n + BN - 1) / BN) * (SPLIT ? p.splits : 1);
     const int grid = total < sm_count() ? total : sm_count();
-    gemm_bf16_tc_kernel<BN, SPLIT><<<grid, 192, Cfg<BN>::TOTAL, st>>>(ma, mb, p);
+    gemm_bf16_tc_kernel<BN, SPLIT, TAIL><<<grid, 192, Cfg<BN>::TOTAL, st>>>(ma, mb, p);
     return (int)cudaGetLastError();
 }
 
+template <bool TAIL = false>
 int dispatch(const void* a, const void* b, const GemmParams& p, cudaStream_t st, int b_rows = 0) {
     // wide tiles once they fill the machine; narrower ones keep more SMs busy on small problems
     const long tiles_m = (p.m + BM - 1) / BM;
     // a handful of rows (a decode step of several sequences): the product streams b once, so the narrowest tile that spreads
     // b over the most SMs wins
     if (p.m <= 32 && (p.lda || (!p.out_bf16 && !p.glu)) && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
-        return p.splits > 1 ? launch<64, true>(a, b, p, st, b_rows) : launch<64>(a, b, p, st, b_rows);
+        return p.splits > 1 ? launch<64, true>(a, b, p, st, b_rows) : launch<64, false, TAIL>(a, b, p, st, b_rows);
     if (p.splits > 1) return p.n >= 128 ? launch<128, true>(a, b, p, st, b_rows) : launch<64, true>(a, b, p, st, b_rows);
-    if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256>(a, b, p, st, b_rows);
+    if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256, false, TAIL>(a, b, p, st, b_rows);
     // one round either way: the widest tile that still gives every SM at most one tile
-    if (p.n >= 192 && tiles_m * ((p.n + 191) / 192) <= sm_count() && tiles_m * ((p.n + 127) / 128) > sm_count()) return launch<192>(a, b, p, st, b_rows);
-    if (p.n >= 128) return launch<128>(a, b, p, st, b_rows);
-    return launch<64>(a, b, p, st, b_rows);
+    if (p.n >= 192 && tiles_m * ((p.n + 191) / 192) <= sm_count() && tiles_m * ((p.n + 127) / 128) > sm_count()) return launch<192, false, TAIL>(a, b, p, st, b_rows);
+    if (p.n >= 128) return launch<128, false, TAIL>(a, b, p, st, b_rows);
+    return launch<64, false, TAIL>(a, b, p, st, b_rows);
 }
 
 // Parts of a split product, added in order; bias, activation, factors, accumulation and output type of the whole.
@@ -353,7 +370,8 @@ __global__ void __launch_bounds__(256) gemm_parts_kernel(const __grid_constant__
         const float4 b = *(const float4*)(p.bias + col);
         r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
     }
-    store4(p, r, row, col, fetch4(p, row, col));
+    if (p.tail && col >= p.tail_col) *(float4*)(p.tail + (size_t)row * p.ld_tail + col - p.tail_col) = r;
+    else store4(p, r, row, col, fetch4(p, row, col));
 }
 
 // Products of moderate row length whose narrowest tiles occupy a good part of the machine in one round: quicker whole than split.
@@ -406,10 +424,13 @@ B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
     if (g->mul && (!g->mul_row || g->accumulate || (g->ldm & 3) || ((uintptr_t)g->mul & 7))) return (int)cudaErrorInvalidValue;
     if (g->tile_expert && (g->experts < 1 || (m & 127))) return (int)cudaErrorInvalidValue;
     if (g->copy && (g->out_type || ((uintptr_t)g->copy & 7))) return (int)cudaErrorInvalidValue;
+    if (g->tail && (g->tail_col < 8 || (g->tail_col & 7) || g->tail_col >= n || g->ld_tail < n - g->tail_col || (g->ld_tail & 3) || ((uintptr_t)g->tail & 15) || g->accumulate ||
+                    g->mul || g->tile_expert))
+        return (int)cudaErrorInvalidValue;
     GemmParams p{m, n, k, g->out, g->ldo, g->bias, g->accumulate, g->out_type, {}, 0, g->tile_expert, glu, SWIGLU_ALPHA, g->limit, glu ? 0 : g->act, g->alpha == 1.f ? 0.f : g->alpha,
-                 (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, (__nv_bfloat16*)g->copy, g->lda};
+                 (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, (__nv_bfloat16*)g->copy, g->lda, g->tail, g->tail_col, g->ld_tail};
     if (g->tile_expert) return dispatch(g->a, g->b, p, st, g->experts * n);
-    if (narrow(m, n, k)) return launch<64>(g->a, g->b, p, st);
+    if (narrow(m, n, k)) return g->tail ? launch<64, false, true>(g->a, g->b, p, st) : launch<64>(g->a, g->b, p, st);
     const int splits = g->ws ? split_count(m, n, k) : 1;
     if (splits > 1 && (long long)splits * m * n <= g->ws_floats && m <= 65535) {
         p.splits = splits;
@@ -421,7 +442,7 @@ B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
         gemm_parts_kernel<<<dim3((n + 1023) / 1024, m), 256, 0, st>>>(p);
         return (int)cudaGetLastError();
     }
-    return dispatch(g->a, g->b, p, st);
+    return g->tail ? dispatch<true>(g->a, g->b, p, st) : dispatch(g->a, g->b, p, st);
 }
 
 // Floats of scratch with which b2_gemm_rows would split a product of this size (0: it would not).

@@ -81,4 +81,7 @@ struct GemmRowsArgs {
     int act;                  // out_act's number, or GLU_BASE + glu_act's: rows 2i / 2i + 1 of b are gate / up of column i
     int accumulate, experts, ldm;
     float alpha, limit;       // limit: of the clamped gated unit
+    // results from column tail_col on (bias added, nothing else) go to fp32 rows of their own instead (bf16 products only), or null
+    float* tail;              // [m][ld_tail]
+    int tail_col, ld_tail;
 };

@@ -29,7 +29,7 @@ RowSeg = _st("RowSeg", [("w", P), ("g", P), ("rs", P), ("rc", P), ("out", P), ("
                         ("limit", F), ("mul", P), ("ldm", I)])
 GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P), ("mul", P), ("mul_row", P), ("tile_expert", P), ("copy", P), ("ws", P),
                                     ("ws_floats", C.c_longlong), ("m", I), ("n", I), ("k", I), ("lda", I), ("ldb", I), ("ldo", I), ("out_type", I), ("act", I),
-                                    ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F)])
+                                    ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F), ("tail", P), ("tail_col", I), ("ld_tail", I)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
                                     ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
                                     ("conv_b", P), ("conv_state", P), ("conv_silu", I), ("conv_shift", I), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
@@ -116,23 +116,27 @@ def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC
 
 def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", accumulate: bool = False, k: int | None = None, alpha: float = 1.0,
          limit: float = math.inf, bias: torch.Tensor | None = None, mul: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
-         experts: int = 0, tile_expert: torch.Tensor | None = None, copy: torch.Tensor | None = None) -> None:
+         experts: int = 0, tile_expert: torch.Tensor | None = None, copy: torch.Tensor | None = None, tail: torch.Tensor | None = None) -> None:
     """out (+)= alpha * act(a[:, :k] @ w[:, :k]^T + bias) [* mul[mul_row]]; bf16 operands on tcgen05 (result bf16, f16 or fp32), fp32 operands in full
     32 bits.  ``copy``: bf16 rows of out's pitch that receive an fp32 result too.
     ``a``, ``out`` and ``mul`` may be column windows of wider buffers.  Gated activations ("glu:...") halve the columns.  ``experts``: w holds
-    that many stacked matrices and a's tiles of 128 rows belong to ``tile_expert``."""
+    that many stacked matrices and a's tiles of 128 rows belong to ``tile_expert``.  ``tail``: fp32 rows that receive the last columns' sums, as they are, instead of
+    ``out`` (bf16 operands)."""
     n = w.shape[0] // max(experts, 1)
-    m, k = a.shape[0], w.shape[1] if k is None else k
-    cols = n // 2 if act.startswith("glu:") else n
+    m, k, nt = a.shape[0], w.shape[1] if k is None else k, tail.shape[1] if tail is not None else 0
+    cols = (n - nt) // 2 if act.startswith("glu:") else n - nt
     if a.dtype != w.dtype or out.shape[0] != m or out.shape[1] != cols or a.shape[1] < k or a.stride(1) != 1 or out.stride(1) != 1:
         raise ValueError(f"gemm: {tuple(a.shape)} {a.dtype} x {tuple(w.shape)} {w.dtype} -> {tuple(out.shape)}")
+    if nt and (tail.shape[0] != m or tail.dtype != torch.float32 or tail.stride(1) != 1):
+        raise ValueError(f"gemm: tail {tuple(tail.shape)} {tail.dtype}")
     if copy is not None and (copy.stride(0) != out.stride(0) or copy.shape != out.shape or copy.dtype != torch.bfloat16):
         raise ValueError(f"gemm: copy {tuple(copy.shape)} {copy.dtype}")
     f32 = a.dtype == torch.float32
     size = 0 if f32 or experts else _split_floats(m, n, k)
     ws = torch.empty(size, device=a.device) if size else None
     g = GemmRowsArgs(ptr(a), ptr(w), ptr(out), ptr(bias), ptr(mul), ptr(mul_row), ptr(tile_expert), ptr(copy), ptr(ws), size, m, n, k, a.stride(0), w.stride(0), out.stride(0),
-                     OUT_TYPE[out.dtype], ACT[act], int(accumulate), experts, mul.stride(0) if mul is not None else 0, alpha, limit)
+                     OUT_TYPE[out.dtype], ACT[act], int(accumulate), experts, mul.stride(0) if mul is not None else 0, alpha, limit, ptr(tail), n - nt,
+                     tail.stride(0) if nt else 0)
     _call("b2_gemm_rows_f32" if f32 else "b2_gemm_rows", g)
 
 

@@ -52,7 +52,7 @@ def test_convolution_and_group_norm():
     x, z = torch.randn(3, 12, dtype=O.F64), torch.randn(3, 12, dtype=O.F64)
     n = O.gated_group_norm(x, z, torch.ones(12), 3, 0.0)
     assert torch.allclose((n.view(3, 3, 4) ** 2).mean(-1), torch.ones(3, 3, dtype=O.F64))
-    assert torch.allclose(n / n[:, :1], (x * O.silu(z)) / (x * O.silu(z))[:, :1]) is False      # parts have scales of their own
+    assert not torch.allclose(n / n[:, :1], (x * O.silu(z)) / (x * O.silu(z))[:, :1])      # parts have scales of their own
     assert torch.allclose(n[:, :4] / n[:, :1], (x * O.silu(z))[:, :4] / (x * O.silu(z))[:, :1])
 
 

@@ -11,6 +11,9 @@ from ..ops import ssd as D
 from .blocks import Mat, Norm, Step, WeightSource, up
 
 
+MIN_SPLIT = 128                  # keys
+
+
 class HeadAttention:
     """The projections of queries, keys, values and gate are one product; with a convolution the first three go through it, and the slot keeps their last inputs."""
 
@@ -57,7 +60,8 @@ class HeadAttention:
     def splits(self, nb: int, n_ctx: int, sms: int) -> tuple[int, int]:
         """(parts of the keys for a decode step of ``nb`` sequences, most keys a query sees)."""
         keys = min(n_ctx, self.m.chunk or (self.m.window + self.m.keep + 128 if self.m.window else n_ctx))
-        return max(1, min(envconfig.attn_splits(), keys // envconfig.attn_split_len())), keys
+        room = sms // (self.m.kv_heads * nb)          # shorter parts than usual as long as SMs would stand idle
+        return max(1, min(envconfig.attn_splits(), max(keys // envconfig.attn_split_len(), min(keys // MIN_SPLIT, room)))), keys
 
     def run(self, s: Step, mem: tuple[torch.Tensor, ...]) -> None:
         m, be, f32 = self.m, s.be, torch.float32

@@ -298,7 +298,7 @@ class Ssd:
         return self._call(D.ssd_step, rows, None, i32(*slots), i32(*ts))[..., :self.P]
 
 
-SSD = [(1, 1, 1, 1), (4, 16, 16, 2), (3, 20, 9, 1), (6, 12, 20, 3), (8, 64, 128, 2), (5, 72, 40, 5), (2, 130, 100, 1), (2, 40, 200, 2), (100, 64, 64, 4)]
+SSD = [(1, 1, 1, 1), (4, 16, 16, 2), (3, 20, 9, 1), (6, 12, 20, 3), (8, 64, 128, 2), (5, 72, 40, 5), (2, 130, 100, 1), (2, 40, 200, 2), (100, 64, 64, 4), (96, 40, 128, 1), (96, 64, 128, 8), (96, 48, 20, 3)]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -320,7 +320,7 @@ def heads_config(width: int, heads: int, kv_heads: int, dim: int, window: int, f
 
 
 STACK_SPECS: dict[str, dict] = {
-    "tiny-tirudra": heads_config(192, 6, 2, 48, 40, 3, 6, 32, 48, 2, 4096, "MWFm", 6, 2, 2, 96, 64),
+    "tiny-tirudra": heads_config(192, 6, 2, 48, 40, 3, 12, 16, 40, 3, 4096, "MWFm", 6, 3, 1, 96, 80),
     "tirudra-2k": heads_config(2048, 16, 4, 128, 1024, 4, 64, 64, 128, 2, 32768, "MWMF" * 5, 64, 4, 4, 1408, 1408),
     "tirudra-4k": heads_config(4096, 32, 8, 128, 1024, 8, 128, 64, 128, 8, 65536, "MWMF" * 3, 32, 4, 2, 2048, 2048),
     "tiny-kavenex": latent_config(192, 6, 40, 24, 48, 80, 384, 4096, "DED", (1, 3, 2), 24, 6, 2, 96, 64),

@@ -31,8 +31,11 @@ _LAYER = {
     "side.gate": "inp_gate.weight", "side.proj": "proj.weight", "side.norm": "post_norm.weight",
     "norm1b": "post_attention_norm.weight", "norm2b": "post_ffw_norm.weight", "mix.g": "attn_gate.weight", "mix.q.b": "attn_q.bias", "mix.k.b": "attn_k.bias",
     "mix.q.conv": "attn_q_conv1d.weight", "mix.k.conv": "attn_k_conv1d.weight", "mix.v.conv": "attn_v_conv1d.weight",
+    "mix.v.b": "attn_v.bias", "mix.lq1": "attn_lambda_q1.weight", "mix.lk1": "attn_lambda_k1.weight", "mix.lq2": "attn_lambda_q2.weight", "mix.lk2": "attn_lambda_k2.weight",
+    "mix.dq": "attn_q_a.weight", "mix.dq.norm": "attn_q_a_norm.weight", "mix.uq": "attn_q_b.weight", "mlp.act": "ffn_act.weight", "dwa": "depth_average.weight",
     "mix.dt_bias": "ssm_dt.bias", "mix.norm": "ssm_norm.weight", "mlp.correction": "exp_probs_b.bias", "mlp.shared.sg": "ffn_gate_inp_shexp.weight",
 }
+_GRU = {"mix.z": "gru_z.weight", "mix.z.b": "gru_z.bias", "mix.x": "gru_x.weight", "mix.x.b": "gru_x.bias", "mix.g": "gru_gate.weight", "mix.o": "gru_out.weight"}
 _EXPERT = re.compile(r"l(\d+)\.mlp\.e(\d+)\.(gate|up|down)")
 _ONE_PLUS = ("attn_norm.weight", "ffn_norm.weight", "output_norm.weight", "post_attention_norm.weight", "post_ffw_norm.weight")
 _F32 = ("ssm_a", "ssm_d", "conv1d.weight", "ssm_conv1d.bias", "ssm_dt.bias")
@@ -78,9 +81,11 @@ def map_stack_name(name: str, cfg: dict[str, Any]) -> str | None:
     m = re.fullmatch(r"l(\d+)\.(.+)", name)
     if not m or int(m.group(1)) >= len(cfg["layers"]):
         return None
-    rest = m.group(2)
+    rest, kind = m.group(2), cfg["layers"][int(m.group(1))]["type"]
+    if kind == "mingru" and rest in _GRU:
+        return f"blk.{m.group(1)}.{_GRU[rest]}"
     if rest == "mix.o":
-        return f"blk.{m.group(1)}.{'ssm_out' if cfg['layers'][int(m.group(1))]['type'].startswith('mamba') else 'attn_output'}.weight"
+        return f"blk.{m.group(1)}.{'ssm_out' if kind.startswith('mamba') else 'attn_output'}.weight"
     e = _EXPERT.fullmatch(name)
     if e:
         router = (cfg["layers"][int(e.group(1))].get("mlp") or {}).get("router") or {}

@@ -40,6 +40,10 @@ struct AttnRopeArgs {
     const double* freqs;     // [n_rot / 2]
     int head_norm;
     int v_off;               // column of the first value head
+    // differential attention (maps = 2): n_heads counts maps.  A cache row holds the keys of a head's maps side by side, and the query of a map stands in the
+    // map's columns of an otherwise empty row, so that both maps of a head score the same cache rows
+    int maps;
+    int no_append;           // key and value of this position are in the cache already (another layer's); the rows of qkv hold queries only
 };
 
 // Rows of a step over a paged cache: see attn_paged.cu.
@@ -62,6 +66,8 @@ struct PagedAppendArgs {
     int dk, dv, cache32;     // cache32: fp32 caches, else f16
     int head_norm, v_off;
     float mscale;            // factor of the rotated dimensions
+    int maps;                // see AttnRopeArgs
+    int no_append;
 };
 
 struct PagedAttnArgs {

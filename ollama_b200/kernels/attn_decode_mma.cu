@@ -126,10 +126,16 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         else asm volatile("cp.async.commit_group;" ::: "memory");
     }
     const bool fresh = r.qkv != nullptr;
-    const bool owner = fresh && n_tiles > 0 && qpos - shift >= p0 && qpos - shift < p1;      // this split holds the query token's own position
+    const bool owner = fresh && !(PAGED && r.no_append) && n_tiles > 0 && qpos - shift >= p0 && qpos - shift < p1;      // this split holds the query token's own position
     // element i of a raw head row after the rotary embedding (pairs (2p, 2p+1), or (p, p + n_rot/2) in the neox order)
+    // the second map's columns of a row of two (differential attention) turn like the first's
     auto rotated = [&](const float* row, int i) -> float {
         const float x = row[i];
+        if (PAGED && r.maps > 1 && i >= r.dim) {
+            i -= r.dim;
+            row += r.dim;
+            if (i >= r.dim) return x;
+        }
         if (i >= r.n_rot) return x;
         const int half_rot = r.n_rot >> 1;
         const bool first = r.neox ? i < half_rot : !(i & 1);
@@ -144,7 +150,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
         const int nrows = group + (owner ? 2 : 0);
         if (PAGED) {
             const float* tok = r.qkv + (size_t)b * r.ldq;
-            const int nq = a.n_heads * r.dim, nk = a.n_kv_heads * r.dim;
+            const int kdim = r.maps * r.dim, nq = a.n_heads * r.dim, nk = a.n_kv_heads * kdim;
             for (int p = tid; p < (r.n_rot >> 1); p += 128) {
                 float sn, cs;
                 sincosf(rot_angle(qpos, r.freqs[p]), &sn, &cs);
@@ -185,8 +191,9 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const __grid_const
                 const int rr = c / D, col = c % D;
                 float v = 0.f;
                 if (rr <= group) {
-                    if (col < r.dim) {
-                        const int i = rr < group ? (head0 + rr) * r.dim + col : kvh * r.dim + col;
+                    const int off = rr < group ? (head0 + rr) % r.maps * r.dim : 0;
+                    if (col >= off && col < (rr < group ? off + r.dim : kdim)) {
+                        const int i = rr < group ? (head0 + rr) * r.dim + col - off : kvh * kdim + col;
                         v = tok[rr < group ? i : nq + i];
                         if (r.q_norm && !r.head_norm) v *= rr < group ? iq * r.q_norm[i] : ik * r.k_norm[i];
                     }
@@ -446,8 +453,9 @@ int launch_d(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int pdl, cu
 int attn_decode_mma_rope_launch(const AttnDecodeArgs& a, const AttnRopeArgs& r, int nb, int hd, int pdl, cudaStream_t st) {
     if (a.n_kv_heads < 1 || a.n_heads % a.n_kv_heads || a.n_heads / a.n_kv_heads > ROWS) return (int)cudaErrorNotSupported;
     if (r.qkv && (a.k_scale || a.v_scale || r.n_rot > 256 || r.n_rot > hd || (r.n_rot & 1) || (a.page_table ? r.n_rot && !r.freqs : !r.inv_freq))) return (int)cudaErrorNotSupported;
-    if (a.page_table && (!r.qkv || !r.neox || r.dim < 1 || r.dim > hd || r.vdim < 1 || r.vdim > hd || r.n_rot > r.dim || a.max_pages < 1 || a.window < 0 || a.keep < 0 || r.v_off < 0 ||
-                         r.v_off + a.n_kv_heads * r.vdim > r.ldq)) return (int)cudaErrorInvalidValue;
+    if (a.page_table && (r.maps < 1 || r.maps > 2 || a.n_heads / a.n_kv_heads % r.maps || (r.maps > 1 && r.q_norm) || (r.no_append && r.q_norm))) return (int)cudaErrorInvalidValue;
+    if (a.page_table && (!r.qkv || !r.neox || r.dim < 1 || r.maps * r.dim > hd || r.vdim < 1 || r.vdim > hd || r.n_rot > r.dim || a.max_pages < 1 || a.window < 0 || a.keep < 0 || r.v_off < 0 ||
+                         (!r.no_append && r.v_off + a.n_kv_heads * r.vdim > r.ldq))) return (int)cudaErrorInvalidValue;
     if (hd == 128) return launch_d<128>(a, r, nb, pdl, st);
     if (hd == 64) return launch_d<64>(a, r, nb, pdl, st);
     return (int)cudaErrorNotSupported;

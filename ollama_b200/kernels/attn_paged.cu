@@ -19,7 +19,8 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[2][8];
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int nq = a.n_heads * a.dim, nk = a.n_kv_heads * a.dim, half = a.n_rot >> 1;
+    const int kvs = a.no_append ? 0 : a.n_kv_heads, kdim = a.maps * a.dim;      // columns of a key head
+    const int nq = a.n_heads * a.dim, nk = kvs * kdim, half = a.n_rot >> 1;
     float* sq = sm;                // [nq + nk]
     float* cs = sm + nq + nk;      // [half], then sines
     float* sn = cs + half;
@@ -85,18 +86,22 @@ __global__ void __launch_bounds__(256) paged_append_kernel(const __grid_constant
         return d < half ? x * cs[d] - head[d + half] * sn[d] : x * cs[d - half] + head[d - half] * sn[d - half];
     };
     const int* table = a.page_table + (size_t)slot * a.max_pages;
-    for (int h = warp; h < a.n_heads + 2 * a.n_kv_heads; h += 8) {          // a warp per head
+    for (int h = warp; h < a.n_heads + 2 * kvs; h += 8) {          // a warp per head
         if (h < a.n_heads) {
             const float* head = sq + h * a.dim;
             float* q = a.q_out + ((size_t)t * a.n_heads + h) * a.dq;
-            for (int d = lane; d < a.dq; d += 32) q[d] = d < a.dim ? rotated(head, d) : 0.f;
-        } else if (h < a.n_heads + a.n_kv_heads) {
+            const int off = h % a.maps * a.dim;
+            for (int d = lane; d < a.dq; d += 32) q[d] = d >= off && d < off + a.dim ? rotated(head, d - off) : 0.f;
+        } else if (h < a.n_heads + kvs) {
             const int g = h - a.n_heads;
-            const float* head = sq + nq + g * a.dim;
+            const float* head = sq + nq + g * kdim;
             CT* k = (CT*)a.k_cache + paged_row(table, pos, a.n_kv_heads, g) * a.dk;
-            for (int d = lane; d < a.dk; d += 32) k[d] = from_f<CT>(d < a.dim ? rotated(head, d) : 0.f);
+            for (int d = lane; d < a.dk; d += 32) {
+                const int off = d < a.dim ? 0 : a.dim;      // the map's first column
+                k[d] = from_f<CT>(d < kdim ? rotated(head + off, d - off) : 0.f);
+            }
         } else {
-            const int g = h - a.n_heads - a.n_kv_heads;
+            const int g = h - a.n_heads - kvs;
             const float* head = row + a.v_off + g * a.vdim;
             CT* v = (CT*)a.v_cache + paged_row(table, pos, a.n_kv_heads, g) * a.dv;
             for (int d = lane; d < a.dv; d += 32) v[d] = from_f<CT>(d < a.vdim ? head[d] : 0.f);
@@ -182,13 +187,11 @@ struct PagedCombineArgs {
     void* out;
     int ldo, out16;
     HeadGate gate;
+    DiffHeads diff;
 };
 
-__global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constant__ PagedCombineArgs a) {
-    const int h = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
-    pdl_launch();
-    pdl_wait();
-    if (d >= a.vdim) return;
+// Split sums of head h of batch row b at column d.
+__device__ __forceinline__ float merged_split(const PagedCombineArgs& a, int b, int h, int d) {
     const size_t p0 = ((size_t)b * a.n_heads + h) * a.n_splits;
     float mn = -1e30f;
     for (int s = 0; s < a.n_splits; s++) mn = fmaxf(mn, a.part_ml[p0 + s].x);
@@ -199,11 +202,48 @@ __global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constan
         o += a.part_acc[(p0 + s) * a.hd + d] * c;
         l += ml.y * c;
     }
-    float v = l > 0.f ? o / l : 0.f;
+    return l > 0.f ? o / l : 0.f;
+}
+
+__global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constant__ PagedCombineArgs a) {
+    const int h = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
+    pdl_launch();
+    pdl_wait();
+    float v;
+    if (a.diff.on) {                 // two maps of a head
+        __shared__ float red[4];
+        v = d < a.vdim ? merged_split(a, b, 2 * h, d) - a.diff.lambda * merged_split(a, b, 2 * h + 1, d) : 0.f;
+        const float s = warp_sum(v * v);
+        if ((d & 31) == 0) red[d >> 5] = s;
+        __syncthreads();
+        v *= a.diff.scale / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)a.vdim + a.diff.eps);
+        if (d >= a.vdim) return;
+    } else {
+        if (d >= a.vdim) return;
+        v = merged_split(a, b, h, d);
+    }
     if (a.gate.kind) v *= sigmoid_f(a.gate.g[(size_t)b * a.gate.ld + (a.gate.kind == 1 ? h * a.vdim + d : h)]);
     const size_t oi = (size_t)b * a.ldo + (size_t)h * a.vdim + d;
     if (a.out16) ((__nv_bfloat16*)a.out)[oi] = __float2bfloat16_rn(v);
     else ((float*)a.out)[oi] = v;
+}
+
+// Results of both maps of every head, [rows][H][2][vdim] fp32 -> the heads' results.  A warp per (row, head).
+template <typename OT>
+__global__ void __launch_bounds__(128) diff_rows_kernel(const float* x, int n, int H, int vdim, const __grid_constant__ DiffHeads f, OT* out, int ldo) {
+    const int i = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    pdl_launch();
+    pdl_wait();
+    if (i >= n * H) return;
+    const float* a = x + (size_t)i * 2 * vdim;
+    OT* o = out + (size_t)(i / H) * ldo + (size_t)(i % H) * vdim;
+    float s = 0.f;
+    for (int d = lane; d < vdim; d += 32) {
+        const float v = a[d] - f.lambda * a[vdim + d];
+        s += v * v;
+    }
+    const float r = f.scale / sqrtf(warp_sum(s) / (float)vdim + f.eps);
+    for (int d = lane; d < vdim; d += 32) o[d] = from_f<OT>((a[d] - f.lambda * a[vdim + d]) * r);
 }
 
 bool bad_gate(const HeadGate& g) { return g.kind < 0 || g.kind > 2 || (g.kind && !g.g); }
@@ -214,10 +254,12 @@ bool bad_shape(int H, int G, int dim, int vdim) { return H < 1 || G < 1 || H % G
 
 // Returns a cudaError_t value (as do the entry points below).
 B2_API int b2_paged_append(const PagedAppendArgs* a, int rows, int pdl, cudaStream_t st) {
-    if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dq < a->dim || a->dk < a->dim || a->dv < a->vdim || a->n_rot < 0 || a->n_rot > a->dim ||
-        (a->n_rot & 1) || (a->n_rot && !a->freqs) || (!a->q_norm != !a->k_norm) || a->v_off < 0 || a->v_off + a->n_kv_heads * a->vdim > a->ldq)
+    if (a->maps < 1 || a->maps > 2 || a->n_heads % a->maps || (a->maps > 1 && a->q_norm) || (a->no_append && a->q_norm)) return (int)cudaErrorInvalidValue;
+    const int kdim = a->maps * a->dim;
+    if (rows < 1 || bad_shape(a->n_heads, a->n_kv_heads, a->dim, a->vdim) || a->dq < kdim || a->dk < kdim || a->dv < a->vdim || a->n_rot < 0 || a->n_rot > a->dim ||
+        (a->n_rot & 1) || (a->n_rot && !a->freqs) || (!a->q_norm != !a->k_norm) || a->v_off < 0 || (!a->no_append && a->v_off + a->n_kv_heads * a->vdim > a->ldq))
         return (int)cudaErrorInvalidValue;
-    const size_t smem = ((size_t)(a->n_heads + a->n_kv_heads) * a->dim + a->n_rot) * 4;
+    const size_t smem = ((size_t)a->n_heads * a->dim + (a->no_append ? 0 : (size_t)a->n_kv_heads * kdim) + a->n_rot) * 4;
     if (smem > 200 * 1024) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
     if (once.first()) {
@@ -240,12 +282,23 @@ B2_API int b2_paged_attn(const PagedAttnArgs* a, int rows, int pdl, cudaStream_t
 
 // Decode step over a paged f16 cache: norm and rotation of the new query and key, cache append and split-K attention in one launch,
 // then the merge of the splits.  cudaErrorNotSupported (nothing launched): the caller runs b2_paged_append + b2_paged_attn.
-B2_API int b2_attn_decode_paged(const AttnDecodeArgs* a, const AttnRopeArgs* r, int nb, int hd, void* out, int ldo, int out16, const HeadGate* gate, int pdl, cudaStream_t st) {
+B2_API int b2_attn_decode_paged(const AttnDecodeArgs* a, const AttnRopeArgs* r, int nb, int hd, void* out, int ldo, int out16, const HeadGate* gate, const DiffHeads* diff, int pdl,
+                                cudaStream_t st) {
+    if (diff->on && (r->maps != 2 || r->vdim > 128)) return (int)cudaErrorInvalidValue;
     if (!r || bad_gate(*gate) || !r->qkv || !a->page_table || bad_shape(a->n_heads, a->n_kv_heads, r->dim, r->vdim) || r->dim > hd || r->vdim > hd || nb < 1 || a->n_splits < 1)
         return (int)cudaErrorInvalidValue;
     const cudaError_t e = (cudaError_t)attn_decode_mma_rope_launch(*a, *r, nb, hd, pdl, st);
     if (e != cudaSuccess) return (int)e;
-    PagedCombineArgs c{a->part_acc, a->part_ml, a->n_heads, a->n_splits, hd, r->vdim, out, ldo, out16, *gate};
+    PagedCombineArgs c{a->part_acc, a->part_ml, a->n_heads, a->n_splits, hd, r->vdim, out, ldo, out16, *gate, *diff};
     void* args[] = {&c};
-    return launch_rows((const void*)paged_combine_kernel, dim3(a->n_heads, nb), dim3(128), 0, args, st, pdl);
+    return launch_rows((const void*)paged_combine_kernel, dim3(diff->on ? a->n_heads / 2 : a->n_heads, nb), dim3(128), 0, args, st, pdl);
+}
+
+// The heads' results of differential attention from those of both maps, x [rows][H][2][vdim].
+B2_API int b2_diff_rows(const float* x, int rows, int H, int vdim, const DiffHeads* f, void* out, int ldo, int out16, int pdl, cudaStream_t st) {
+    if (rows < 1 || H < 1 || vdim < 1 || ldo < H * vdim || !x || !out || (long long)rows * H > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
+    DiffHeads d = *f;
+    void* args[] = {&x, &rows, &H, &vdim, &d, &out, &ldo};
+    return launch_rows(out16 ? (const void*)diff_rows_kernel<__nv_bfloat16> : (const void*)diff_rows_kernel<float>, dim3((unsigned)(((long long)rows * H + 3) / 4)), dim3(128), 0,
+                       args, st, pdl);
 }

@@ -73,7 +73,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
             const int col = n0 + 4 * tx + j;
             if (col >= p.n) continue;
             float* o = (float*)p.out + (size_t)row * p.ldo + col;
-            float r = out_act<true>(v[j], p.act);
+            float r = out_act<true>(v[j], p.act, p.act_p, p.act_q);
             if (p.mul) r *= ((const float*)p.mul)[(size_t)p.mul_row[row] * p.ldm + col];
             r *= p.alpha;
             *o = p.accumulate ? *o + r : r;
@@ -87,7 +87,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
 B2_API int b2_gemm_rows_f32(const GemmRowsArgs* g, cudaStream_t st) {
     const int glu = g->act >= GLU_BASE ? 1 : 0;
     if (g->m < 1 || g->n < 1 || g->k < 4 || (g->k & 3) || (g->lda & 3) || (g->ldb & 3) || ((uintptr_t)g->a & 15) || ((uintptr_t)g->b & 15) || g->out_type || g->copy || g->tail || g->act < 0 ||
-        (!glu && g->act > 2) || g->act > GLU_BASE + 2 || (glu && ((g->n & 1) || g->accumulate || g->mul)) || (g->mul && !g->mul_row) ||
+        (!glu && g->act > ACT_LAST) || g->act > GLU_BASE + 2 || (glu && ((g->n & 1) || g->accumulate || g->mul)) || (g->mul && !g->mul_row) ||
         (g->tile_expert && (g->experts < 1 || (g->m & 127))))
         return (int)cudaErrorInvalidValue;
     const dim3 grid((g->n + TN - 1) / TN, (g->m + TM - 1) / TM);

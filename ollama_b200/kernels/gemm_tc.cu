@@ -62,6 +62,7 @@ struct GemmParams {
     float* part;
     long long part_stride;
     int part_ld;
+    float act_p, act_q;     // numbers of the activation
 };
 
 template <int BN>
@@ -108,7 +109,10 @@ __device__ __forceinline__ float4 fetch4(const GemmParams& p, int row, int col) 
 
 // Four consecutive sums of a row, as the product's caller wants them: activation or gated pairs, factors, type, accumulation.
 __device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, int col, const float4& with) {
-    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
+    if (p.act) {
+        r.x = out_act(r.x, p.act, p.act_p, p.act_q); r.y = out_act(r.y, p.act, p.act_p, p.act_q);
+        r.z = out_act(r.z, p.act, p.act_p, p.act_q); r.w = out_act(r.w, p.act, p.act_p, p.act_q);
+    }
     if (p.mul) { r.x *= with.x; r.y *= with.y; r.z *= with.z; r.w *= with.w; }
     if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
         const float h0 = glu_act(r.x, r.y, p.glu - 1, p.glu_alpha, p.glu_limit), h1 = glu_act(r.z, r.w, p.glu - 1, p.glu_alpha, p.glu_limit);
@@ -417,7 +421,7 @@ B2_API int b2_gemm_bf16_out16(const void* a, const void* b, int m, int n, int k,
 // gated: n a multiple of 8, bf16 results).  With scratch (b2_gemm_rows_scratch floats) products of few tiles are split along k.
 B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
     const int glu = g->act >= GLU_BASE ? 1 + g->act - GLU_BASE : 0, m = g->m, n = g->n, k = g->k;
-    if (bad_operands(g->a, g->b, m, n, k, g->ldo) || g->lda < k || (g->lda & 7) || g->ldb != k || g->act < 0 || (!glu && g->act > 2) || glu > 3 || g->out_type < 0 ||
+    if (bad_operands(g->a, g->b, m, n, k, g->ldo) || g->lda < k || (g->lda & 7) || g->ldb != k || g->act < 0 || (!glu && g->act > ACT_LAST) || glu > 3 || g->out_type < 0 ||
         g->out_type > 2 || (g->out_type && g->accumulate) || ((uintptr_t)g->out & (g->out_type ? 7 : 15)) || ((uintptr_t)g->ws & 15) || ((uintptr_t)g->bias & 15))
         return (int)cudaErrorInvalidValue;
     if (glu && (g->out_type != 1 || (n & 7) || g->mul)) return (int)cudaErrorInvalidValue;
@@ -429,6 +433,8 @@ B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
         return (int)cudaErrorInvalidValue;
     GemmParams p{m, n, k, g->out, g->ldo, g->bias, g->accumulate, g->out_type, {}, 0, g->tile_expert, glu, SWIGLU_ALPHA, g->limit, glu ? 0 : g->act, g->alpha == 1.f ? 0.f : g->alpha,
                  (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, (__nv_bfloat16*)g->copy, g->lda, g->tail, g->tail_col, g->ld_tail};
+    p.act_p = g->act_p;
+    p.act_q = g->act_q;
     if (g->tile_expert) return dispatch(g->a, g->b, p, st, g->experts * n);
     if (narrow(m, n, k)) return g->tail ? launch<64, false, true>(g->a, g->b, p, st) : launch<64>(g->a, g->b, p, st);
     const int splits = g->ws ? split_count(m, n, k) : 1;

@@ -27,6 +27,7 @@ struct RowSeg {
     float alpha, limit;  // factor of the result; limit of the clamped gated unit
     const void* mul;     // result times mul[mul_row[b] * ldm + row] in the weights' type, after the activation; or null
     int ldm;
+    float act_p, act_q;  // numbers of the activation, where it has some
 };
 
 enum RowSrc : int { SRC_ROWS = 0, SRC_NORM = 1, SRC_JOINED = 2, SRC_LAYER = 3 };
@@ -236,7 +237,7 @@ __global__ void __launch_bounds__(256, NB == 1 ? 3 : NB == 2 ? 4 : 2) gemv_rows_
         return;
     }
     if (mine) {
-        v = out_act<F32>(v, w.act);
+        v = out_act<F32>(v, w.act, w.act_p, w.act_q);
         if (w.mul) {
             const size_t m = (size_t)a.mul_row[b] * w.ldm + row;
             v *= F32 ? ((const float*)w.mul)[m] : __bfloat162float(((const __nv_bfloat16*)w.mul)[m]);
@@ -296,7 +297,7 @@ B2_API int b2_gemv_rows(const GemvRowsArgs* a, int pdl, cudaStream_t st) {
     for (int s = 0; s < a->nseg; s++) {
         const RowSeg& w = a->seg[s];
         if (!w.w || !w.out || w.n < 1 || w.ldw < a->k || (w.ldw & 7) || ((uintptr_t)w.w & 15) || (norm_source(a->src) && (!w.g || ((uintptr_t)w.g & 15) || (a->src == SRC_LAYER && !w.rs))) ||
-            w.act < 0 || (w.act > 2 && w.act < GLU_BASE) || w.act > GLU_BASE + 2 || (w.act >= GLU_BASE && ((w.n & 1) || w.mul)) || (w.mul && !a->mul_row))
+            w.act < 0 || (w.act > ACT_LAST && w.act < GLU_BASE) || w.act > GLU_BASE + 2 || (w.act >= GLU_BASE && ((w.n & 1) || w.mul)) || (w.mul && !a->mul_row))
             return (int)cudaErrorInvalidValue;
         groups += (w.n + R - 1) / R;
     }

@@ -43,6 +43,11 @@ struct HeadGate {
     const float* g;          // [rows][ld]
     int ld, kind;
 };
+// Differential attention: a head's result is a1 - lambda a2 of its two maps, divided by its root mean square, times `scale`.
+struct DiffHeads {
+    float lambda, scale, eps;
+    int on;
+};
 __device__ __forceinline__ float sigmoid_f(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
 __device__ __forceinline__ float sigmoid_exact(float v) { return 1.f / (1.f + expf(-v)); }
 
@@ -84,4 +89,5 @@ struct GemmRowsArgs {
     // results from column tail_col on (bias added, nothing else) go to fp32 rows of their own instead (bf16 products only), or null
     float* tail;              // [m][ld_tail]
     int tail_col, ld_tail;
+    float act_p, act_q;       // numbers of the activation, where it has some
 };

@@ -16,6 +16,7 @@ struct LatentAttnArgs {
     const int* page_table;   // [slots][max_pages]
     int max_pages;
     int n_heads, cp, w, splits;
+    int window;              // > 0: a query sees the last `window` positions up to its own
     float scale;
     float* acc;              // [n][heads][splits][cp]; not written for splits without positions
     float2* ml;              // [n][heads][splits]
@@ -62,8 +63,9 @@ __global__ void __launch_bounds__(256, MT == 1 ? 2 : 1) attn_latent_kernel(const
     const int row = a.rows ? a.rows[i] : i;
     const int kv_len = a.positions[row] + 1;
     const int* table = a.page_table + (size_t)a.slots[row] * a.max_pages;
-    const int pages = (kv_len + PAGE - 1) / PAGE, per = (pages + a.splits - 1) / a.splits;
-    const int p0 = split * per * PAGE, n_tiles = (min(kv_len - p0, per * PAGE) + BN - 1) / BN;
+    const int lo = a.window > 0 ? max(0, kv_len - a.window) : 0, page0 = lo / PAGE;      // first visible position and its page
+    const int pages = (kv_len + PAGE - 1) / PAGE - page0, per = (pages + a.splits - 1) / a.splits;
+    const int p0 = (page0 + split * per) * PAGE, n_tiles = (min(kv_len - p0, per * PAGE) + BN - 1) / BN;
     if (kv_len <= p0) {
         for (int h = tid; h < heads; h += 256) a.ml[((size_t)i * a.n_heads + head0 + h) * a.splits + split] = make_float2(-1e30f, 0.f);
         return;
@@ -160,7 +162,7 @@ __global__ void __launch_bounds__(256, MT == 1 ? 2 : 1) attn_latent_kernel(const
             }
 #pragma unroll
             for (int j = 0; j < KPT; j++) {
-                v[j] = kp + j < kv_len ? v[j] * a.scale : -INFINITY;
+                v[j] = kp + j < kv_len && kp + j >= lo ? v[j] * a.scale : -INFINITY;
                 mx = fmaxf(mx, v[j]);
             }
 #pragma unroll
@@ -254,7 +256,7 @@ int launch_w(const LatentAttnArgs& a, int n, int pdl, cudaStream_t st) {
 
 // f16 cache with rows of up to 640 values, a multiple of 32, and a latent of up to 512; other shapes: cudaErrorNotSupported, nothing launched.
 B2_API int b2_attn_latent(const LatentAttnArgs* a, int n, int pdl, cudaStream_t st) {
-    if (n < 1 || a->n_heads < 1 || a->splits < 1 || a->splits > 128 || a->cp < 16 || (a->cp & 15) || a->w < a->cp || a->max_pages < 1 || ((uintptr_t)a->q & 15) || ((uintptr_t)a->cache & 15))
+    if (n < 1 || a->n_heads < 1 || a->splits < 1 || a->splits > 128 || a->cp < 16 || (a->cp & 15) || a->w < a->cp || a->max_pages < 1 || a->window < 0 || ((uintptr_t)a->q & 15) || ((uintptr_t)a->cache & 15))
         return (int)cudaErrorInvalidValue;
     if ((a->w & 31) || a->cp > 512 || a->w > 640 || n > 65535) return (int)cudaErrorNotSupported;
     return a->n_heads <= 16 ? launch_w<1>(*a, n, pdl, st) : launch_w<2>(*a, n, pdl, st);

@@ -46,6 +46,7 @@ struct AttnPagedArgs {
     int max_pages, chunk, vdim, ldo;
     int window, keep;
     HeadGate gate;
+    DiffHeads diff;          // on: differential attention, H counts maps; query tiles of up to 64 rows
 };
 
 // Form for keys in two parts (latent attention, latent.cu): rows of one buffer hold every head's own key part and value, rows of another the
@@ -59,6 +60,7 @@ struct AttnPartsArgs {
     int H, vdim, ldo;
     float scale;
     __nv_bfloat16* out;      // [rows][ldo], head h at column h * vdim
+    int window;              // 0 = none
 };
 
 __device__ int g_attn_tc_status = 0;
@@ -476,8 +478,9 @@ struct Lay2 {
     static constexpr int TOTAL = OFF_BAR + 256 + 2 * 2 * 128 * 4 + 1024;
 };
 
-// D: value columns, DK: query / key columns (D unless the form is PARTS)
-template <int D, int DK, int FORM>
+// D: value columns, DK: query / key columns (D unless the form is PARTS).  DIFF: a CTA takes 64 queries of a head of differential attention, rows 0 .. 63 of its tile
+// with the first map, rows 64 .. 127 with the second; the key rows hold both maps' keys, of which a query row has zeros against the other map's.
+template <int D, int DK, int FORM, bool DIFF = false>
 __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                                                                        const __grid_constant__ AttnPrefillArgs a, const __grid_constant__ AttnPagedArgs pg,
                                                                        const __grid_constant__ AttnPartsArgs pt) {
@@ -504,7 +507,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int mt = gridDim.x - 1 - blockIdx.x;
     const int4 tile = FORM == PARTS ? pt.tiles[mt] : PAGED ? pg.tiles[mt] : make_int4(mt * BQ, min(BQ, a.T - mt * BQ), a.slot, a.pos0 + mt * BQ);
-    const int m0 = tile.x, rows = tile.y, h = blockIdx.y, hkv = FORM == PARTS ? h : h / (a.H / a.Hkv);
+    const int m0 = tile.x, rows = tile.y, h = blockIdx.y, hkv = FORM == PARTS ? h : h / (a.H / (DIFF ? 2 : 1) / a.Hkv);
     const int q_lo = tile.w, q_hi = q_lo + rows - 1;
     const int kv_len = PAGED ? q_hi + 1 : a.kv_len;
     const int k_end = a.causal ? min(kv_len, q_hi + 1) : kv_len;
@@ -534,8 +537,8 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     if (warp < SOFTMAX_WARPS) {
-        const int r = 32 * (warp & 3) + lane, c = warp >> 2;
-        const bool live = r < rows;
+        const int r = 32 * (warp & 3) + lane, c = warp >> 2, qi = DIFF ? r & 63 : r;
+        const bool live = qi < rows;
         if (FORM == PARTS) {
             const __half* qp = pt.q + ((size_t)(m0 + r) * a.H + h) * DK + QH * c;
 #pragma unroll
@@ -544,7 +547,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
                 *(uint4*)(sQ + atom * ATOM_BYTES + r * 128 + ((chunk ^ (r & 7)) << 4)) = live ? *(const uint4*)(qp + 8 * j) : make_uint4(0, 0, 0, 0);
             }
         } else {
-        const float* qp = a.q + ((size_t)(m0 + r) * a.H + h) * D + OH * c;
+        const float* qp = a.q + ((size_t)(m0 + qi) * a.H + (DIFF ? 2 * h + (r >> 6) : h)) * D + OH * c;
 #pragma unroll
         for (int j = 0; j < OH / 8; j++) {
             float4 v0 = make_float4(0.f, 0.f, 0.f, 0.f), v1 = v0;
@@ -635,7 +638,7 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
     } else {
         const int q = warp & 3, c = warp >> 2;
         const int r = 32 * q + lane;
-        const int qp = q_lo + r;
+        const int qp = q_lo + (DIFF ? r & 63 : r);
         const int row_lo = first_key(qp, chunk, window), last_lo = first_key(q_hi, chunk, window);      // this row's first key (but for kept ones); the last row's
         const float LOG2E = 1.4426950408889634f;
         const float sl2 = a.scale * LOG2E;
@@ -731,7 +734,51 @@ __global__ void __launch_bounds__(THREADS2, 1) attn_prefill_tc2_kernel(const __g
             ok = false;
             atomicExch(failed, 1);
         }
-        if (ok) {
+        if constexpr (DIFF) {      // the second map's rows meet the first's in the key buffers, which no product reads any more; every softmax thread passes the barriers
+            constexpr int LDX = D + 4;
+            float* other = reinterpret_cast<float*>(sm + L::OFF_K);      // [64][LDX]
+            const float l = l_run + x_sum[(c ^ 1) * 128 + r], inv = l > 0.f ? 1.f / l : 0.f;
+            if (r >= 64) {
+#pragma unroll
+                for (int j = 0; j < OH; j += 4)
+                    *(float4*)(other + (r - 64) * LDX + OH * c + j) = make_float4(o[j] * inv, o[j + 1] * inv, o[j + 2] * inv, o[j + 3] * inv);
+            }
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            float ss = 0.f;
+            if (r < 64) {
+#pragma unroll
+                for (int j = 0; j < OH; j += 4) {
+                    const float4 y = *(const float4*)(other + r * LDX + OH * c + j);
+                    o[j] = o[j] * inv - pg.diff.lambda * y.x; o[j + 1] = o[j + 1] * inv - pg.diff.lambda * y.y;
+                    o[j + 2] = o[j + 2] * inv - pg.diff.lambda * y.z; o[j + 3] = o[j + 3] * inv - pg.diff.lambda * y.w;
+                    ss += o[j] * o[j] + o[j + 1] * o[j + 1] + o[j + 2] * o[j + 2] + o[j + 3] * o[j + 3];
+                }
+                x_max[c * 128 + r] = ss;
+            }
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            if (ok && r < rows) {
+                const float f = pg.diff.scale / sqrtf((ss + x_max[(c ^ 1) * 128 + r]) / (float)pg.vdim + pg.diff.eps);
+                __nv_bfloat16* op = a.out + (size_t)(m0 + r) * pg.ldo + (size_t)h * pg.vdim + OH * c;
+                const bool whole = (pg.vdim & 7) == 0 && (pg.ldo & 7) == 0;
+#pragma unroll
+                for (int j = 0; j < OH; j += 8) {
+                    if (OH * c + j >= pg.vdim) continue;
+                    if (whole) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const __nv_bfloat162 bb = __floats2bfloat162_rn(o[j + 2 * e] * f, o[j + 2 * e + 1] * f);
+                            w[e] = *reinterpret_cast<const uint32_t*>(&bb);
+                        }
+                        *(uint4*)(op + j) = make_uint4(w[0], w[1], w[2], w[3]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; e++)
+                            if (OH * c + j + e < pg.vdim) op[j + e] = __float2bfloat16_rn(o[j + e] * f);
+                    }
+                }
+            }
+        } else if (ok) {
             float l = l_run + x_sum[(c ^ 1) * 128 + r];
             float oc = 1.f;
             if (a.sinks) {
@@ -835,14 +882,14 @@ int launch2(const AttnPrefillArgs& a, int n_slots, cudaStream_t st) {
     return (int)cudaGetLastError();
 }
 
-template <int D>
+template <int D, bool DIFF>
 int launch_paged(const AttnPrefillArgs& a, const AttnPagedArgs& pg, int n_tiles, int n_pages, cudaStream_t st) {
     CUtensorMap mk, mv;
     const size_t rows = (size_t)n_pages * a.Hkv * 64;
     if (!cached_kv_map(&mk, a.k_cache, rows, D, 64) || !cached_kv_map(&mv, a.v_cache, rows, D, 64)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, D, PAGED_CACHE>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D, D>::TOTAL);
-    attn_prefill_tc2_kernel<D, D, PAGED_CACHE><<<dim3(n_tiles, a.H), THREADS2, Lay2<D, D>::TOTAL, st>>>(mk, mv, a, pg, AttnPartsArgs{});
+    if (once.first()) cudaFuncSetAttribute(attn_prefill_tc2_kernel<D, D, PAGED_CACHE, DIFF>, cudaFuncAttributeMaxDynamicSharedMemorySize, Lay2<D, D>::TOTAL);
+    attn_prefill_tc2_kernel<D, D, PAGED_CACHE, DIFF><<<dim3(n_tiles, DIFF ? a.H / 2 : a.H), THREADS2, Lay2<D, D>::TOTAL, st>>>(mk, mv, a, pg, AttnPartsArgs{});
     return (int)cudaGetLastError();
 }
 
@@ -857,6 +904,7 @@ int launch_parts(const AttnPartsArgs& p, int n_tiles, cudaStream_t st) {
     a.H = a.Hkv = p.H;
     a.causal = 1;
     a.scale = p.scale;
+    a.window = p.window;
     a.out = p.out;
     attn_prefill_tc2_kernel<D, DK, PARTS><<<dim3(n_tiles, p.H), THREADS2, Lay2<D, DK>::TOTAL, st>>>(mk, ms, a, AttnPagedArgs{}, p);
     return (int)cudaGetLastError();
@@ -868,7 +916,7 @@ int launch_parts(const AttnPartsArgs& p, int n_tiles, cudaStream_t st) {
 // cudaErrorNotSupported, nothing launched.
 B2_API int b2_attn_prefill_parts(const AttnPartsArgs* p, int n_tiles, cudaStream_t st) {
     if (!p || !p->tiles || n_tiles < 1 || p->n_rows < 1 || p->H < 1 || p->H > 65535 || p->dp < 64 || (p->dp & 63) || (p->vp & 63) || p->rp < 0 || (p->rp & 63) ||
-        (p->rp && !p->shared) || p->vdim < 1 || p->vdim > p->vp || p->ldo < p->H * p->vdim)
+        (p->rp && !p->shared) || p->window < 0 || p->vdim < 1 || p->vdim > p->vp || p->ldo < p->H * p->vdim)
         return (int)cudaErrorInvalidValue;
     if (((uintptr_t)p->kv & 15) || ((uintptr_t)p->shared & 15) || ((uintptr_t)p->q & 15) || ((uintptr_t)p->out & 15)) return (int)cudaErrorNotSupported;
     const int dk = p->dp + p->rp;
@@ -884,7 +932,7 @@ B2_API int b2_attn_prefill_parts(const AttnPartsArgs* p, int n_tiles, cudaStream
 // nothing launched).  a: q [rows][H][head_dim], caches, out, H, Hkv, scale, softcap; the other fields are not used.
 B2_API int b2_attn_prefill_paged(const AttnPrefillArgs* a, const AttnPagedArgs* pg, int head_dim, int n_tiles, int n_pages, cudaStream_t st) {
     if (!a || !pg || !pg->tiles || !pg->page_table || n_tiles < 1 || n_pages < 1 || pg->max_pages < 1 || a->H < 1 || a->H > 65535 || a->Hkv < 1 || a->H % a->Hkv ||
-        pg->vdim < 1 || pg->vdim > head_dim || pg->ldo < a->H * pg->vdim || pg->window < 0 || pg->keep < 0 || pg->gate.kind < 0 || pg->gate.kind > 2 ||
+        pg->vdim < 1 || pg->vdim > head_dim || pg->ldo < (pg->diff.on ? a->H / 2 : a->H) * pg->vdim || (pg->diff.on && (a->H / a->Hkv & 1)) || pg->window < 0 || pg->keep < 0 || pg->gate.kind < 0 || pg->gate.kind > 2 ||
         (pg->gate.kind && !pg->gate.g))
         return (int)cudaErrorInvalidValue;
     if (((uintptr_t)a->k_cache & 15) || ((uintptr_t)a->v_cache & 15) || ((uintptr_t)a->q & 15) || ((uintptr_t)a->out & 15)) return (int)cudaErrorNotSupported;
@@ -893,8 +941,14 @@ B2_API int b2_attn_prefill_paged(const AttnPrefillArgs* a, const AttnPagedArgs* 
     c.causal = 1;
     c.window = 0;
     c.sinks = nullptr;
-    if (head_dim == 128) return launch_paged<128>(c, *pg, n_tiles, n_pages, st);
-    if (head_dim == 64) return launch_paged<64>(c, *pg, n_tiles, n_pages, st);
+    if (pg->diff.on) {
+        if (pg->gate.kind) return (int)cudaErrorNotSupported;
+        if (head_dim == 128) return launch_paged<128, true>(c, *pg, n_tiles, n_pages, st);
+        if (head_dim == 64) return launch_paged<64, true>(c, *pg, n_tiles, n_pages, st);
+        return (int)cudaErrorNotSupported;
+    }
+    if (head_dim == 128) return launch_paged<128, false>(c, *pg, n_tiles, n_pages, st);
+    if (head_dim == 64) return launch_paged<64, false>(c, *pg, n_tiles, n_pages, st);
     return (int)cudaErrorNotSupported;
 }
 

@@ -17,8 +17,9 @@
 #include "rows.cuh"
 
 struct LatentStepArgs {
-    const float* qkv;        // [.][ldq]: per head dim unrotated | rot rotated values, then the latent, then the rotated key part
-    int ldq, n_heads, dim, rot, rank;
+    const float* q;          // [.][ldq]: per head dim unrotated | rot rotated values
+    const float* c;          // [.][ldc]: the latent, then the rotated key part
+    int ldq, ldc, n_heads, dim, rot, rank;
     const float* norm;       // [rank] weight of the latent's norm
     float eps;
     const double* freqs;     // [rot / 2]
@@ -35,6 +36,7 @@ struct LatentStepArgs {
     int w32;
     void* q_out;             // [n][heads][w] in the cache's type; long form: [n][heads][dp + rp] f16, unrotated part, zeros, rotated part, zeros
     int dp, rp;              // long form (uk null)
+    float mscale;            // factor of cosines and sines
 };
 
 struct LatentMergeArgs {
@@ -51,7 +53,7 @@ struct LatentMergeArgs {
 struct LatentGatherArgs {
     const __half* cache;
     int cp, w, rot;
-    const int4* seqs;        // (first result row, positions, slot, -)
+    const int4* seqs;        // (result row of position 0, end of the positions, slot, first position)
     const int* page_table;
     int max_pages;
     __nv_bfloat16* c;        // [.][cp]
@@ -66,14 +68,19 @@ namespace {
 template <typename CT>
 __device__ __forceinline__ void append_row(const LatentStepArgs& a, int r, CT* q, float* cs, float* red) {
     const int tid = threadIdx.x, nt = blockDim.x, pos = a.positions[r], slot = a.slots[r], half = a.rot >> 1, pad = a.w - a.cp;
-    const float* row = a.qkv + (size_t)r * a.ldq;
-    const float* c = row + (size_t)a.n_heads * (a.dim + a.rot);
+    const float* row = a.q + (size_t)r * a.ldq;
+    const float* c = a.c + (size_t)r * a.ldc;
     float ss = 0.f;
 #pragma unroll 4
     for (int i = tid; i < a.rank; i += nt) ss += c[i] * c[i];
     ss = warp_sum(ss);
     if ((tid & 31) == 0) red[tid >> 5] = ss;
-    for (int i = tid; i < half; i += nt) sincosf(rot_angle(pos, a.freqs[i]), &cs[half + i], &cs[i]);
+    for (int i = tid; i < half; i += nt) {
+        float sn, co;
+        sincosf(rot_angle(pos, a.freqs[i]), &sn, &co);
+        cs[i] = co * a.mscale;
+        cs[half + i] = sn * a.mscale;
+    }
     __syncthreads();
     ss = 0.f;
     for (int i = 0; i < nt >> 5; i++) ss += red[i];
@@ -142,7 +149,7 @@ __global__ void __launch_bounds__(256) latent_step_kernel(const __grid_constant_
     const int nb = min(NB, n - i0), dq = a.dim + a.rot;
     for (int j = tid; j < nb * a.dim; j += 256) {
         const int b = j / a.dim, d = j - b * a.dim, r = a.rows ? a.rows[i0 + b] : i0 + b;
-        sq[b * a.dim + d] = a.qkv[(size_t)r * a.ldq + (size_t)h * dq + d];
+        sq[b * a.dim + d] = a.q[(size_t)r * a.ldq + (size_t)h * dq + d];
     }
     __syncthreads();
     float acc[NB][8];
@@ -188,7 +195,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const __grid_constant_
     pdl_launch();
     pdl_wait();
     append_row<__half>(a, r, nullptr, cs, red);
-    const float* q = a.qkv + (size_t)r * a.ldq;
+    const float* q = a.q + (size_t)r * a.ldq;
     __half* o = (__half*)a.q_out + (size_t)i * a.n_heads * dk;
     for (int j = threadIdx.x; j < a.n_heads * dk2; j += 256) {      // two neighbouring values
         const int h = j / dk2, c = 2 * (j - h * dk2);
@@ -390,7 +397,7 @@ __global__ void __launch_bounds__(128) latent_values_kernel(const __grid_constan
 
 __global__ void __launch_bounds__(256) latent_gather_kernel(const __grid_constant__ LatentGatherArgs a) {
     const int4 q = a.seqs[blockIdx.y];
-    const int pos = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int pos = q.w + blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (pos >= q.y) return;
     const __half* src = a.cache + paged_row(a.page_table + (size_t)q.z * a.max_pages, pos, 1, 0) * a.w;
     __nv_bfloat16* c = a.c + (size_t)(q.x + pos) * a.cp;
@@ -420,7 +427,7 @@ const void* step_fn(int nb) {
 // Cache rows (append) and absorbed queries of n rows; without uk the query rows of the long form (f16 caches).  Returns a cudaError_t value, as do the entry points below.
 B2_API int b2_latent_step(const LatentStepArgs* a, int n, int pdl, cudaStream_t st) {
     if (n < 1 || a->n_heads < 1 || a->dim < 1 || a->rot < 0 || (a->rot & 1) || a->rank < 1 || a->cp < a->rank || (a->cp & 15) || a->w < a->cp + a->rot || (a->rot && !a->freqs) ||
-        !a->q_out || ((uintptr_t)a->uk & 15) || (!a->uk && (a->cache32 || a->dp < a->dim || a->rp < a->rot || (a->dp & 1) || (a->rp & 1))) || a->dim > 8192 || a->max_pages < 1)
+        !a->q_out || !a->q || !a->c || a->ldq < a->n_heads * (a->dim + a->rot) || a->ldc < a->rank + a->rot || ((uintptr_t)a->uk & 15) || (!a->uk && (a->cache32 || a->dp < a->dim || a->rp < a->rot || (a->dp & 1) || (a->rp & 1))) || a->dim > 8192 || a->max_pages < 1)
         return (int)cudaErrorInvalidValue;
     LatentStepArgs c = *a;
     void* args[] = {&c, &n};

@@ -36,8 +36,8 @@ def _stale(target: str, deps: list[str]) -> bool:
 
 
 # sources of a part of the library, for a first start that should compile what one kind of model needs and no more
-GROUPS = {"stack": ("attn_decode_mma.cu", "attn_latent.cu", "attn_paged.cu", "attn_prefill_tc.cu", "elementwise.cu", "gemm_f32.cu", "gemm_tc.cu", "gemv_rows.cu",
-                    "latent.cu", "moe.cu", "moe_rows.cu", "norm_rows.cu", "sample.cu", "ssd.cu", "ssd_chunk.cu", "ssm.cu")}
+GROUPS = {"stack": ("attn_decode_mma.cu", "attn_latent.cu", "attn_paged.cu", "attn_prefill_tc.cu", "depth.cu", "elementwise.cu", "gemm_f32.cu", "gemm_tc.cu", "gemv_rows.cu",
+                    "gru.cu", "latent.cu", "moe.cu", "moe_rows.cu", "norm_rows.cu", "sample.cu", "ssd.cu", "ssd_chunk.cu", "ssm.cu")}
 
 
 def build_group(group: str, verbose: bool = False, force: bool = False) -> str:

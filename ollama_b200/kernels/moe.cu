@@ -4,7 +4,9 @@
 //
 // In the reference stack these are ggml-cuda's topk-moe / argsort / softmax kernels and the ids paths of
 // mul_mat_id and add_id.
+#include "choose.cuh"
 #include "comm.cuh"
+#include "rows.cuh"
 
 struct MoeRouteArgs {
     const float* logits;   // [tokens][ld]
@@ -12,13 +14,15 @@ struct MoeRouteArgs {
     int n_experts;         // <= 512
     int k;                 // experts per token, <= 16
     int mode;              // 0: softmax over all experts, then top-k (optionally renormalised); 1: top-k, then softmax over the selected;
-                           // 2: softmax over all, top-k of that plus `correction`, weights without it
+                           // 2: softmax over all, top-k of that plus `correction`, weights without it; 3: sigmoids, top-k of those plus
+                           // `correction` in the best groups, weights: the chosen sigmoids over their sum, times a factor
     int norm_topk;
     int e_lo, e_cnt;       // experts resident on this GPU: [e_lo, e_lo + e_cnt)
     int* ids;              // [tokens][k] global expert ids
     int* lids;             // [tokens][k] id relative to e_lo, or -1 when the expert lives elsewhere
     float* wts;            // [tokens][k]
-    const float* correction;      // [n_experts], mode 2
+    const float* correction;      // [n_experts], modes 2 and 3
+    ExpertGroups groups;          // mode 3
 };
 
 // one warp per token
@@ -30,12 +34,19 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ 
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
     if (t >= tokens) return;
     const float* lg = a.logits + (size_t)t * a.ld;
+    extern __shared__ float scratch_all[];         // mode 3: [4][2 n_experts]
+    float* scratch = scratch_all + (threadIdx.x >> 5) * 2 * a.n_experts;
+    if (a.mode == 3) {
+        for (int e = lane; e < a.n_experts; e += 32) scratch[e] = sigmoid_exact(lg[e]) + (a.correction ? a.correction[e] : 0.f);
+        __syncwarp();
+        keep_groups(scratch, scratch + a.n_experts, a.n_experts, a.groups, lane);
+    }
     float v[MAXJ];
     float mx = -INFINITY;
 #pragma unroll
     for (int j = 0; j < MAXJ; j++) {
         const int e = lane + 32 * j;
-        v[j] = e < a.n_experts ? lg[e] : -INFINITY;
+        v[j] = e < a.n_experts ? (a.mode == 3 ? scratch[e] : lg[e]) : -INFINITY;
         mx = fmaxf(mx, v[j]);
     }
     mx = warp_max(mx);
@@ -85,6 +96,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ 
         if (a.norm_topk) w /= warp_sum(w);
     } else if (a.mode == 2) {
         w = mine ? expf(lg[sel_e] - mx) / denom : 0.f;
+    } else if (a.mode == 3) {
+        w = mine ? sigmoid_exact(lg[min(sel_e, a.n_experts - 1)]) : 0.f;
+        w = w / (warp_sum(w) + 1e-20f) * a.groups.scale;
     } else {
         const float top = __shfl_sync(0xffffffffu, sel_v, 0);          // the first selected is the largest
         const float ex = mine ? __expf(sel_v - top) : 0.f;
@@ -100,11 +114,13 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const __grid_constant__ 
 }
 
 B2_API int b2_moe_route(const MoeRouteArgs* a, int tokens, int pdl, cudaStream_t st) {
-    if (tokens < 1 || a->n_experts < 1 || a->n_experts > 512 || a->k < 1 || a->k > 16 || a->k > a->n_experts || (a->mode == 2 && !a->correction))
+    if (tokens < 1 || a->n_experts < 1 || a->n_experts > 512 || a->k < 1 || a->k > 16 || a->k > a->n_experts || (a->mode == 2 && !a->correction) ||
+        (a->mode == 3 && (a->groups.count < 1 || a->n_experts % a->groups.count || a->groups.keep < 1 || a->k > a->n_experts / a->groups.count * a->groups.keep)))
         return (int)cudaErrorInvalidValue;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3((tokens + 3) / 4);
     cfg.blockDim = dim3(128);
+    cfg.dynamicSmemBytes = a->mode == 3 ? (size_t)a->n_experts * 32 : 0;
     cfg.stream = st;
     cudaLaunchAttribute at[1];
     at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;

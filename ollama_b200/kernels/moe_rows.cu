@@ -7,6 +7,7 @@
 //                   to the residual
 //
 // A warp owns four consecutive matrix rows; short problems split the row length over KS warps, as in gemv_rows.cu.
+#include "choose.cuh"
 #include "rows.cuh"
 
 struct MoeUpArgs {
@@ -25,6 +26,7 @@ struct MoeUpArgs {
     float* wts;              // [nb][top]
     const float* correction; // [n_experts] or null
     int real, act;           // router outputs from `real` on stand for the input itself and have no matrices; act: glu_act's number
+    ExpertGroups groups;     // count > 0: scores are sigmoids, see choose
 };
 
 struct MoeDownArgs {
@@ -50,16 +52,23 @@ namespace {
 constexpr int R = 4, MAXJ = 16, MAX_TOP = 16;
 
 // Experts of a row in order of their scores (ties: the lower index) and their weights; by one warp.  Without a correction the scores are the logits and the
-// weights the softmax over the chosen ones; with it the softmax over all plus the correction, and that softmax.
-__device__ __forceinline__ void choose(const float* z, const float* correction, int n, int top, int lane, int* ids, float* wts) {
+// weights the softmax over the chosen ones; with it the softmax over all plus the correction, and that softmax.  With groups the scores are the sigmoids plus the
+// correction, inside the groups that are kept, and the weights the chosen sigmoids over their sum, times a factor; `scratch`: 2 n floats of shared memory.
+__device__ __forceinline__ void choose(const float* z, const float* correction, int n, int top, int lane, int* ids, float* wts, const ExpertGroups& groups, float* scratch) {
     float v[MAXJ], mz = -INFINITY, total = 0.f;
+    const bool sigmoid = groups.count > 0;
+    if (sigmoid) {
+        for (int e = lane; e < n; e += 32) scratch[e] = sigmoid_exact(z[e]) + (correction ? correction[e] : 0.f);
+        __syncwarp();
+        keep_groups(scratch, scratch + n, n, groups, lane);
+    }
 #pragma unroll
     for (int j = 0; j < MAXJ; j++) {
         const int e = lane + 32 * j;
-        v[j] = e < n ? z[e] : -INFINITY;
+        v[j] = e < n ? (sigmoid ? scratch[e] : z[e]) : -INFINITY;
         mz = fmaxf(mz, v[j]);
     }
-    if (correction) {
+    if (correction && !sigmoid) {
         mz = warp_max(mz);
 #pragma unroll
         for (int j = 0; j < MAXJ; j++) {
@@ -103,6 +112,14 @@ __device__ __forceinline__ void choose(const float* z, const float* correction, 
 #pragma unroll
         for (int j = 0; j < MAXJ; j++)
             if (lane + 32 * j == be) v[j] = -INFINITY;
+    }
+    if (sigmoid) {
+        const float w = lane < top ? sigmoid_exact(z[idx]) : 0.f, sum = warp_sum(w) + 1e-20f;
+        if (lane < top) {
+            ids[lane] = idx;
+            wts[lane] = w / sum * groups.scale;
+        }
+        return;
     }
     if (correction) {
         if (lane < top) {
@@ -158,10 +175,11 @@ __global__ void __launch_bounds__(256) moe_up_rows_kernel(const __grid_constant_
     __shared__ int s_id[MAX_TOP];
     __shared__ float s_w[MAX_TOP];
     __shared__ float red[8][R];
+    extern __shared__ float scratch[];             // [2 n_experts] with groups
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, rg = warp / KS, ks = warp % KS, b = blockIdx.y;
     pdl_launch();
     pdl_wait();
-    if (warp == 0) choose(a.z + (size_t)b * a.ldz, a.correction, a.n_experts, a.top, lane, s_id, s_w);
+    if (warp == 0) choose(a.z + (size_t)b * a.ldz, a.correction, a.n_experts, a.top, lane, s_id, s_w, a.groups, scratch);
     __syncthreads();
     if (blockIdx.x == 0 && threadIdx.x < a.top) {
         a.ids[b * a.top + threadIdx.x] = s_id[threadIdx.x];
@@ -304,13 +322,15 @@ int split_of(long groups, int pieces, long want) {
 B2_API int b2_moe_up_rows(const MoeUpArgs* a, int nb, int f32, int pdl, cudaStream_t st) {
     if (nb < 1 || nb > 65535 || a->n_experts < 1 || a->n_experts > 32 * MAXJ || a->top < 1 || a->top > MAX_TOP || a->top > a->n_experts || a->k < 8 || (a->k & 7) || (a->ldh & 3) ||
         a->n < 2 || (a->n & 1) || a->wrows < a->n || (a->ns & 1) || (a->ns && !a->ws) || a->ffp < a->n / 2 || a->ldo < a->top * a->ffp + a->ns / 2 || ((uintptr_t)a->h & 15) ||
-        ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15) || a->real < 1 || a->real > a->n_experts || a->act < 0 || a->act > 2)
+        ((uintptr_t)a->w & 15) || ((uintptr_t)a->ws & 15) || a->real < 1 || a->real > a->n_experts || a->act < 0 || a->act > 2 || a->groups.count < 0 ||
+        (a->groups.count && (a->n_experts % a->groups.count || a->groups.keep < 1 || a->top > a->n_experts / a->groups.count * a->groups.keep)))
         return (int)cudaErrorInvalidValue;
     const long groups = (long)a->top * ((a->n + R - 1) / R) + (a->ns + R - 1) / R;
     const int ks = split_of(groups * nb, a->k >> 3, 1800), rgs = 8 / ks;
     MoeUpArgs c = *a;
     void* args[] = {&c};
-    return launch_rows(B2_PICK_KS(moe_up_rows_kernel, f32, ks), dim3((unsigned)((groups + rgs - 1) / rgs), nb), dim3(256), 0, args, st, pdl);
+    return launch_rows(B2_PICK_KS(moe_up_rows_kernel, f32, ks), dim3((unsigned)((groups + rgs - 1) / rgs), nb), dim3(256), a->groups.count ? (size_t)a->n_experts * 8 : 0, args, st,
+                       pdl);
 }
 
 B2_API int b2_moe_down_rows(const MoeDownArgs* a, int nb, int f32, int pdl, cudaStream_t st) {

@@ -118,9 +118,15 @@ class GluArgs(C.Structure):
                 ("hf", C.c_void_p), ("ids", C.c_void_p), ("x_div", C.c_int), ("n_pairs", C.c_int)]
 
 
+class ExpertGroups(C.Structure):
+    """Equal groups of experts, of which the best ``keep`` can be chosen (router scores are sigmoids then); ``scale``: factor of the weights."""
+    _fields_ = [("count", C.c_int), ("keep", C.c_int), ("scale", C.c_float)]
+
+
 class MoeRouteArgs(C.Structure):
     _fields_ = [("logits", C.c_void_p), ("ld", C.c_int), ("n_experts", C.c_int), ("k", C.c_int), ("mode", C.c_int), ("norm_topk", C.c_int),
-                ("e_lo", C.c_int), ("e_cnt", C.c_int), ("ids", C.c_void_p), ("lids", C.c_void_p), ("wts", C.c_void_p), ("correction", C.c_void_p)]
+                ("e_lo", C.c_int), ("e_cnt", C.c_int), ("ids", C.c_void_p), ("lids", C.c_void_p), ("wts", C.c_void_p), ("correction", C.c_void_p),
+                ("groups", ExpertGroups)]
 
 
 class MoeCombineArgs(C.Structure):
@@ -165,7 +171,7 @@ class AttnDecodeArgs(C.Structure):
 class AttnRopeArgs(C.Structure):
     _fields_ = [("qkv", C.c_void_p), ("inv_freq", C.c_void_p), ("mscale", C.c_float), ("n_rot", C.c_int), ("neox", C.c_int),
                 ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float), ("ldq", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("freqs", C.c_void_p),
-                ("head_norm", C.c_int), ("v_off", C.c_int)]
+                ("head_norm", C.c_int), ("v_off", C.c_int), ("maps", C.c_int), ("no_append", C.c_int)]
 
 
 class AttnCombineArgs(C.Structure):

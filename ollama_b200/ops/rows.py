@@ -1,5 +1,5 @@
 """Bindings of the row kernels behind stack models: norms, fused decode products, products of many rows, paged attention and the selective
-state-space mixer (kernels/norm_rows.cu, gemv_rows.cu, gemm_tc.cu, gemm_f32.cu, attn_paged.cu, ssm.cu)."""
+state-space mixer (kernels/norm_rows.cu, gemv_rows.cu, gemm_tc.cu, gemm_f32.cu, attn_paged.cu, ssm.cu, depth.cu, gru.cu)."""
 from __future__ import annotations
 
 import ctypes as C
@@ -12,10 +12,11 @@ from .cuda import AttnDecodeArgs, AttnPrefillArgs, AttnRopeArgs, _check, lib, pt
 
 P, I, F = C.c_void_p, C.c_int, C.c_float
 GLU_BASE = 16
-ACT = {"": 0, "relu2": 1, "gelu_tanh": 2, "glu:silu": GLU_BASE, "glu:gelu_tanh": GLU_BASE + 1, "glu:swiglu_oai": GLU_BASE + 2}
+ACT = {"": 0, "relu2": 1, "gelu_tanh": 2, "xielu": 3, "glu:silu": GLU_BASE, "glu:gelu_tanh": GLU_BASE + 1, "glu:swiglu_oai": GLU_BASE + 2}
 OUT_TYPE = {torch.float32: 0, torch.bfloat16: 1, torch.float16: 2}
 SRC_ROWS, SRC_NORM, SRC_JOINED, SRC_LAYER = range(4)
 GEMV_MAX_ROWS = 4
+NO_NUMS = (0.0, 0.0)
 
 
 def _st(name: str, fields: list) -> type:
@@ -26,10 +27,11 @@ NormRowsArgs = _st("NormRowsArgs", [("x", P), ("ldx", I), ("k", I), ("ldo", I), 
                                     ("b1", P), ("b2", P), ("y", P), ("wy", P), ("x0", P), ("step", P), ("ldy", I), ("mult", F)])
 JoinRowsArgs = _st("JoinRowsArgs", [("a", P), ("b", P), ("lda", I), ("n_a", I), ("ldb", I), ("n_b", I), ("out", P), ("ldo", I), ("off_b", I), ("f32", I)])
 RowSeg = _st("RowSeg", [("w", P), ("g", P), ("rs", P), ("rc", P), ("out", P), ("n", I), ("ldw", I), ("ldo", I), ("act", I), ("accumulate", I), ("alpha", F),
-                        ("limit", F), ("mul", P), ("ldm", I)])
+                        ("limit", F), ("mul", P), ("ldm", I), ("act_p", F), ("act_q", F)])
 GemmRowsArgs = _st("GemmRowsArgs", [("a", P), ("b", P), ("out", P), ("bias", P), ("mul", P), ("mul_row", P), ("tile_expert", P), ("copy", P), ("ws", P),
                                     ("ws_floats", C.c_longlong), ("m", I), ("n", I), ("k", I), ("lda", I), ("ldb", I), ("ldo", I), ("out_type", I), ("act", I),
-                                    ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F), ("tail", P), ("tail_col", I), ("ld_tail", I)])
+                                    ("accumulate", I), ("experts", I), ("ldm", I), ("alpha", F), ("limit", F), ("tail", P), ("tail_col", I), ("ld_tail", I),
+                                    ("act_p", F), ("act_q", F)])
 GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I), ("k", I), ("src", I), ("f32", I), ("x", P), ("ldx", I), ("x2", P),
                                     ("ldx2", I), ("k1", I), ("eps", F), ("kn", I), ("conv_seg", I), ("conv_n", I), ("taps", I), ("conv_w", P),
                                     ("conv_b", P), ("conv_state", P), ("conv_silu", I), ("conv_shift", I), ("conv_out", P), ("ldu", I), ("slots", P), ("positions", P),
@@ -37,12 +39,14 @@ GemvRowsArgs = _st("GemvRowsArgs", [("seg", RowSeg * 4), ("nseg", I), ("nb", I),
 PagedAppendArgs = _st("PagedAppendArgs", [("qkv", P), ("ldq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("q_norm", P), ("k_norm", P),
                                           ("eps", F), ("freqs", P), ("n_rot", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
                                           ("q_out", P), ("dq", I), ("k_cache", P), ("v_cache", P), ("dk", I), ("dv", I), ("cache32", I),
-                                          ("head_norm", I), ("v_off", I), ("mscale", F)])
+                                          ("head_norm", I), ("v_off", I), ("mscale", F), ("maps", I), ("no_append", I)])
 HeadGate = _st("HeadGate", [("g", P), ("ld", I), ("kind", I)])
+DiffHeads = _st("DiffHeads", [("lam", F), ("scale", F), ("eps", F), ("on", I)])
 PagedAttnArgs = _st("PagedAttnArgs", [("q", P), ("dq", I), ("n_heads", I), ("n_kv_heads", I), ("dim", I), ("vdim", I), ("k_cache", P), ("v_cache", P),
                                       ("dk", I), ("dv", I), ("cache32", I), ("positions", P), ("slots", P), ("page_table", P), ("max_pages", I),
                                       ("chunk", I), ("scale", F), ("softcap", F), ("out", P), ("ldo", I), ("out16", I), ("window", I), ("keep", I), ("gate", HeadGate)])
-AttnPagedArgs = _st("AttnPagedArgs", [("tiles", P), ("page_table", P), ("max_pages", I), ("chunk", I), ("vdim", I), ("ldo", I), ("window", I), ("keep", I), ("gate", HeadGate)])
+AttnPagedArgs = _st("AttnPagedArgs", [("tiles", P), ("page_table", P), ("max_pages", I), ("chunk", I), ("vdim", I), ("ldo", I), ("window", I), ("keep", I), ("gate", HeadGate),
+                                      ("diff", DiffHeads)])
 SsmConvArgs = _st("SsmConvArgs", [("xz", P), ("ldx", I), ("inner", I), ("taps", I), ("w", P), ("b", P), ("state", P), ("slots", P), ("positions", P),
                                   ("offs", P), ("u", P), ("ldu", I), ("silu", I), ("shift", I)])
 ConvKeepArgs = _st("ConvKeepArgs", [("xz", P), ("ldx", I), ("inner", I), ("taps", I), ("state", P), ("seg", P)])
@@ -53,6 +57,9 @@ SsmStepArgs = _st("SsmStepArgs", [("xz", P), ("ldx", I), ("off_z", I), ("xz16", 
                                   ("inner", I), ("n_state", I), ("p", P), ("ldp", I), ("off_b", I), ("w_dt", P), ("rank", I), ("w32", I), ("dt", P),
                                   ("lddt", I), ("dt_bias", P), ("a2", P), ("d", P), ("state", P), ("slots", P), ("positions", P), ("out", P), ("ldo", I),
                                   ("out16", I), ("exact", I), ("u", P), ("ldu", I)])
+DepthRowsArgs = _st("DepthRowsArgs", [("hist", P), ("stride", C.c_longlong), ("w", P), ("n", I), ("k", I), ("ldx", I), ("x", P), ("g", P), ("b", P), ("h", P), ("ldo", I),
+                                      ("f32", I), ("eps", F)])
+GruArgs = _st("GruArgs", [("x", P), ("ldx", I), ("off_u", I), ("off_g", I), ("width", I), ("state", P), ("seg", P), ("slots", P), ("positions", P), ("out", P), ("ldo", I)])
 
 
 def _is32(t: torch.Tensor) -> int:
@@ -82,11 +89,12 @@ def join_rows(a: torch.Tensor, n_a: int, out: torch.Tensor, b: torch.Tensor | No
 
 
 def seg(w: torch.Tensor, n: int, out: torch.Tensor, g: torch.Tensor | None = None, act: str = "", accumulate: bool = False, alpha: float = 1.0,
-        limit: float = math.inf, rs: torch.Tensor | None = None, rc: torch.Tensor | None = None, mul: torch.Tensor | None = None) -> RowSeg:
+        limit: float = math.inf, nums: tuple[float, float] = NO_NUMS, rs: torch.Tensor | None = None, rc: torch.Tensor | None = None,
+        mul: torch.Tensor | None = None) -> RowSeg:
     """One matrix of :func:`gemv`: the first ``n`` rows of ``w`` into the rows of ``out``, as out (+)= alpha * act(... + rc) [* mul[mul_row]].  ``rs``: the rows' sums of
-    w * g (layer norm).  Gated activations ("glu:...") take rows 2i and 2i + 1 as gate and up of column i."""
+    w * g (layer norm).  ``nums``: the two numbers of the "xielu" activation.  Gated activations ("glu:...") take rows 2i and 2i + 1 as gate and up of column i."""
     s = RowSeg(ptr(w), ptr(g), ptr(rs), ptr(rc), ptr(out), n, w.stride(0), out.stride(0), ACT[act], int(accumulate), alpha, limit, ptr(mul),
-               mul.stride(0) if mul is not None else 0)
+               mul.stride(0) if mul is not None else 0, *nums)
     s.keep = (w, g, rs, rc, out, mul)     # the structure holds addresses only
     return s
 
@@ -115,7 +123,7 @@ def gemv(segs: list, k: int, x: torch.Tensor, nb: int, f32: bool, src: int = SRC
 
 
 def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", accumulate: bool = False, k: int | None = None, alpha: float = 1.0,
-         limit: float = math.inf, bias: torch.Tensor | None = None, mul: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
+         limit: float = math.inf, nums: tuple[float, float] = NO_NUMS, bias: torch.Tensor | None = None, mul: torch.Tensor | None = None, mul_row: torch.Tensor | None = None,
          experts: int = 0, tile_expert: torch.Tensor | None = None, copy: torch.Tensor | None = None, tail: torch.Tensor | None = None) -> None:
     """out (+)= alpha * act(a[:, :k] @ w[:, :k]^T + bias) [* mul[mul_row]]; bf16 operands on tcgen05 (result bf16, f16 or fp32), fp32 operands in full
     32 bits.  ``copy``: bf16 rows of out's pitch that receive an fp32 result too.
@@ -136,7 +144,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str = "", acc
     ws = torch.empty(size, device=a.device) if size else None
     g = GemmRowsArgs(ptr(a), ptr(w), ptr(out), ptr(bias), ptr(mul), ptr(mul_row), ptr(tile_expert), ptr(copy), ptr(ws), size, m, n, k, a.stride(0), w.stride(0), out.stride(0),
                      OUT_TYPE[out.dtype], ACT[act], int(accumulate), experts, mul.stride(0) if mul is not None else 0, alpha, limit, ptr(tail), n - nt,
-                     tail.stride(0) if nt else 0)
+                     tail.stride(0) if nt else 0, *nums)
     _call("b2_gemm_rows_f32" if f32 else "b2_gemm_rows", g)
 
 
@@ -148,6 +156,7 @@ def _split_floats(m: int, n: int, k: int) -> int:
 
 
 NO_GATE = HeadGate(None, 0, 0)
+NO_DIFF = DiffHeads(0.0, 0.0, 0.0, 0)
 
 
 def head_gate(g: torch.Tensor, kind: str) -> HeadGate:
@@ -156,13 +165,14 @@ def head_gate(g: torch.Tensor, kind: str) -> HeadGate:
 
 
 def paged_append(qkv, *, heads, kv_heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, positions, slots, table, q_out, k_cache, v_cache, head_norm=False, v_off=None,
-                 mscale=1.0, pdl=False) -> None:
+                 mscale=1.0, maps=1, append=True, pdl=False) -> None:
     """Norm over the whole q / k projections (``head_norm``: over each head), rotation, q to padded fp32 rows [rows, H, dq], k and v (columns from ``v_off`` on) into
-    the paged caches."""
-    v_off = (heads + kv_heads) * dim if v_off is None else v_off
+    the paged caches.  ``maps`` 2: differential attention, ``heads`` counts maps, a key head is two keys side by side and a query row has zeros beside its map's
+    columns.  ``append`` False: queries only."""
+    v_off = (heads + maps * kv_heads) * dim if v_off is None else v_off
     a = PagedAppendArgs(ptr(qkv), qkv.stride(0), heads, kv_heads, dim, vdim, ptr(q_norm), ptr(k_norm), eps, ptr(freqs), n_rot, ptr(positions), ptr(slots),
                         ptr(table), table.shape[1], ptr(q_out), q_out.shape[2], ptr(k_cache), ptr(v_cache), k_cache.shape[3], v_cache.shape[3], _is32(k_cache),
-                        int(head_norm), v_off, mscale)
+                        int(head_norm), v_off, mscale, maps, int(not append))
     _call("b2_paged_append", a, qkv.shape[0], int(pdl))
 
 
@@ -173,28 +183,60 @@ def paged_attn(q, k_cache, v_cache, positions, slots, table, out, *, dim, vdim, 
     _call("b2_paged_attn", a, q.shape[0], int(pdl))
 
 
-def attn_prefill_paged(q, k_cache, v_cache, tiles, table, out, *, vdim, scale, softcap=0.0, chunk=0, window=0, keep=0, gate=NO_GATE) -> None:
-    """tcgen05 attention of query tiles ([n, 4] int32: first row, rows, slot, position) over a paged f16 cache of row length 64 or 128."""
+def attn_prefill_paged(q, k_cache, v_cache, tiles, table, out, *, vdim, scale, softcap=0.0, chunk=0, window=0, keep=0, gate=NO_GATE, diff=NO_DIFF) -> None:
+    """tcgen05 attention of query tiles ([n, 4] int32: first row, rows, slot, position) over a paged f16 cache of row length 64 or 128.  ``diff``: differential
+    attention, the heads of ``q`` are maps and the tiles have up to 64 rows."""
     a = AttnPrefillArgs(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), None, q.shape[0], q.shape[1], k_cache.shape[1], 0, 0, 0, 0, 1, 0, scale, softcap, None, None)
-    pg = AttnPagedArgs(ptr(tiles), ptr(table), table.shape[1], chunk, vdim, out.stride(0), window, keep, gate)
+    pg = AttnPagedArgs(ptr(tiles), ptr(table), table.shape[1], chunk, vdim, out.stride(0), window, keep, gate, diff)
     _check(lib().b2_attn_prefill_paged(C.byref(a), C.byref(pg), q.shape[2], tiles.shape[0], k_cache.shape[0], stream()), "attn_prefill_paged")
 
 
 def attn_decode_paged(qkv, k_cache, v_cache, positions, slots, table, out, nb, *, heads, dim, vdim, q_norm, k_norm, eps, freqs, n_rot, scale, softcap,
-                      chunk, n_splits, n_ctx, part_acc, part_ml, window=0, keep=0, head_norm=False, v_off=None, mscale=1.0, gate=NO_GATE, pdl=False) -> bool:
-    """Decode attention on raw projections: norms, rotation, cache append, split-K attention, merge and gate.  False: shape not taken, nothing launched."""
+                      chunk, n_splits, n_ctx, part_acc, part_ml, window=0, keep=0, head_norm=False, v_off=None, mscale=1.0, gate=NO_GATE, maps=1,
+                      append=True, diff=NO_DIFF, pdl=False) -> bool:
+    """Decode attention on raw projections: norms, rotation, cache append, split-K attention, merge, difference of maps and gate (``maps`` and ``append``:
+    :func:`paged_append`).  False: shape not taken, nothing launched."""
     hd, G = k_cache.shape[3], k_cache.shape[1]
-    v_off = (heads + G) * dim if v_off is None else v_off
+    v_off = (heads + maps * G) * dim if v_off is None else v_off
     a = AttnDecodeArgs(None, ptr(k_cache), ptr(v_cache), ptr(positions), ptr(slots), heads, G, n_ctx, n_splits, scale, softcap, window,
                        ptr(part_acc), ptr(part_ml), None, None, ptr(table), table.shape[1], chunk, keep)
-    r = AttnRopeArgs(ptr(qkv), None, mscale, n_rot, 1, ptr(q_norm), ptr(k_norm), eps, qkv.stride(0), dim, vdim, ptr(freqs), int(head_norm), v_off)
+    r = AttnRopeArgs(ptr(qkv), None, mscale, n_rot, 1, ptr(q_norm), ptr(k_norm), eps, qkv.stride(0), dim, vdim, ptr(freqs), int(head_norm), v_off, maps, int(not append))
     f = lib().b2_attn_decode_paged
-    f.argtypes = [P, P, I, I, P, I, I, P, I, P]
-    rc = f(C.addressof(a), C.addressof(r), nb, hd, ptr(out), out.stride(0), 1 - _is32(out), C.addressof(gate), int(pdl), stream())
+    f.argtypes = [P, P, I, I, P, I, I, P, P, I, P]
+    rc = f(C.addressof(a), C.addressof(r), nb, hd, ptr(out), out.stride(0), 1 - _is32(out), C.addressof(gate), C.addressof(diff), int(pdl), stream())
     if rc == 801:
         return False
     _check(rc, "attn_decode_paged")
     return True
+
+
+def diff_rows(x: torch.Tensor, heads: int, vdim: int, diff, out: torch.Tensor, pdl: bool = False) -> None:
+    """Results of both maps, ``x`` [rows, heads * 2 * vdim] fp32 -> the heads' results of differential attention."""
+    f = lib().b2_diff_rows
+    f.argtypes = [P, I, I, I, P, P, I, I, I, P]
+    _check(f(ptr(x), x.shape[0], heads, vdim, C.addressof(diff), ptr(out), out.stride(0), 1 - _is32(out), int(pdl), stream()), "diff_rows")
+
+
+def depth_rows(hist: torch.Tensor, n: int, w: torch.Tensor, k: int, eps: float, g: torch.Tensor | None = None, b: torch.Tensor | None = None,
+               h: torch.Tensor | None = None, pdl: bool = False) -> torch.Tensor:
+    """x = the sum of the first ``n`` blocks of ``hist`` [blocks, rows, columns] with weights ``w``, written to block ``n`` and returned; ``h`` = its layer norm."""
+    x = hist[n]
+    a = DepthRowsArgs(ptr(hist), hist.stride(0), ptr(w), n, k, hist.shape[2], ptr(x), ptr(g), ptr(b), ptr(h), h.stride(0) if h is not None else 0,
+                      _is32(h) if h is not None else 0, eps)
+    _call("b2_depth_rows", a, x.shape[0], int(pdl))
+    return x
+
+
+def gru_scan(x: torch.Tensor, off: int, state: torch.Tensor, segs: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
+    """Rows [z | u | gate], ``off`` columns apart, of prompt portions ``segs`` ([n, 4] int32: first row, rows, slot, position) through the gated recurrence."""
+    a = GruArgs(ptr(x), x.stride(0), off, 2 * off, state.shape[1], ptr(state), ptr(segs), None, None, ptr(out), out.stride(0))
+    _call("b2_gru_scan", a, segs.shape[0], _is32(x), int(pdl))
+
+
+def gru_step(x: torch.Tensor, off: int, state: torch.Tensor, slots, positions, out: torch.Tensor, exact: bool = False, pdl: bool = False) -> None:
+    """One token per sequence."""
+    a = GruArgs(ptr(x), x.stride(0), off, 2 * off, state.shape[1], ptr(state), None, ptr(slots), ptr(positions), ptr(out), out.stride(0))
+    _call("b2_gru_step", a, x.shape[0], _is32(x), int(exact), int(pdl))
 
 
 def ssm_conv(xz, inner, w, b, state, slots, positions, offs, u, silu=True, shift=False, pdl=False) -> None:

@@ -10,9 +10,10 @@ from dataclasses import dataclass
 
 import torch
 
-from ..models.stack import DenseMLP, Expert, ExpertMLP, LatentMixer
+from ..models.stack import DenseMLP, Expert, ExpertMLP, GruMixer, LatentMixer
 from ..ops import cuda as K
 from ..ops import latent as A
+from ..ops.cuda import ExpertGroups
 from ..ops import rows as O
 from .cache import PAGE
 
@@ -28,8 +29,8 @@ def up(n: int, m: int = 8) -> int:
 class WeightSource:
     """Named tensors of a model as zero-padded matrices and vectors on the device."""
 
-    def __init__(self, get, device, act_dtype, width: int):
-        self._get, self.device, self.act_dtype, self.width, self.wp = get, device, act_dtype, width, up(width)
+    def __init__(self, get, device, act_dtype, width: int, eps: float):
+        self._get, self.device, self.act_dtype, self.width, self.wp, self.eps = get, device, act_dtype, width, up(width), eps
 
     def tensor(self, name: str, *shape: int) -> torch.Tensor:
         t = self._get(name)
@@ -92,11 +93,12 @@ def make_norm(src: WeightSource, name: str, kind: str = "layer") -> Norm:
 
 @dataclass
 class LongPortions:
-    """Rows of a step whose keys and values are multiplied out: query tiles, the sequences' places in the scratch buffer, and the other rows."""
+    """Rows of a step whose keys and values are multiplied out: query tiles, the sequences' places in the scratch buffer, and the other rows.  Under a window the
+    buffer begins with a sequence's first visible position, so that the row of position 0 may be negative."""
     tiles: torch.Tensor               # [n, 4]: first row, rows, buffer row of the sequence's position 0, position
-    seqs: torch.Tensor                # [n, 4]: first buffer row, positions, slot, -
+    seqs: torch.Tensor                # [n, 4]: buffer row of position 0, end of the positions, slot, first position
     total: int
-    longest: int
+    longest: int                      # positions of one sequence in the buffer
     rest: torch.Tensor | None         # step rows that stay in the latent space
 
 
@@ -107,8 +109,9 @@ class Step:
     applies it in its own pass over the rows.
     """
 
-    def __init__(self, be, B, m, x: torch.Tensor, x0: torch.Tensor | None, decode: bool):
+    def __init__(self, be, B, m, x: torch.Tensor, x0: torch.Tensor | None, decode: bool, hist: torch.Tensor | None = None):
         self.be, self.B, self.m, self.x, self.x0, self.decode = be, B, m, x, x0, decode
+        self.hist = hist                               # [blocks, rows, columns]: embedding output and layer results, where layers read an average of them
         self.nb = x.shape[0]
         self.small = decode and self.nb <= be.gemv_rows
         self.folded = self.small and not be.f32        # norms inside the products; 32-bit models form them first
@@ -129,6 +132,25 @@ class Step:
             O.norm_rows(self.x, self.be.stack.width, self.be.stack.eps, None, None, pdl=self.pdl, **self.pending)
             self.pending = {}
             self.launched()
+
+    def average(self, n: int, w: torch.Tensor, norm: Norm | None) -> torch.Tensor | None:
+        """The stream becomes the sum of the first ``n`` blocks of the history with weights ``w`` (and block ``n``, which the layer adds to); returns its norm."""
+        h = self.buf("h", self.be.wp) if norm is not None else None
+        g, b = (norm.g, norm.b) if norm is not None else (None, None)
+        self.x = O.depth_rows(self.hist, n, w, self.be.stack.width, self.be.stack.eps, g, b, h, pdl=self.pdl)
+        self.launched()
+        return h
+
+    def enter(self, h: torch.Tensor, mat: Mat, out: torch.Tensor, segs=(), joined: Mat | None = None, tail: torch.Tensor | None = None, **conv) -> None:
+        """out = mat h + bias.  Beside it, in the same launch: the products ``segs`` for a few rows, for many rows the last columns of ``joined``, which begins with
+        ``mat``, as fp32 rows ``tail``."""
+        if self.small:
+            O.gemv([O.seg(mat.w, out.shape[1], out, rc=mat.bias), *segs], mat.w.shape[1], h, self.nb, self.be.f32, slots=self.m.slots, positions=self.m.positions,
+                   pdl=self.pdl, **conv)
+        else:
+            m = joined or mat
+            O.gemm(h, m.w, out, bias=m.bias, tail=tail)
+        self.launched()
 
     def product(self, h: torch.Tensor, mat: Mat, out: torch.Tensor, **kw) -> None:
         """out (+)= f(mat h + bias) [times the tokens' rows of a table ``mul``]."""
@@ -181,12 +203,22 @@ class Step:
 
 
 class LatentAttention:
-    def __init__(self, src: WeightSource, p: str, m: LatentMixer, norm: Norm, f32: bool):
+    """The input product gives queries, latent and rotated key part; with a latent of the queries' own the queries follow in a product of their own.  ``norm`` None: the
+    layer's parts share one, and the layer calls :meth:`project` and :meth:`mix`."""
+
+    def __init__(self, src: WeightSource, p: str, m: LatentMixer, norm: Norm | None, f32: bool):
         H, w = m.heads, src.width
         self.m, self.norm, self.f32 = m, norm, f32
         nq = H * (m.dim + m.rot_dim)
-        n_in = nq + m.kv_rank + m.rot_dim
-        self.w_in = Mat(src.pack([(0, 0, p + "attn_q.weight", (nq, w)), (nq, 0, p + "attn_kv_a_mqa.weight", (m.kv_rank + m.rot_dim, w))], up(n_in), src.wp))
+        self.w_uq = self.q_norm = None
+        if m.q_rank:
+            self.off_c, name = up(m.q_rank), "attn_q_a"
+            self.q_norm = src.vec(p + "attn_q_a_norm.weight", m.q_rank)
+            self.w_uq = Mat(src.pack([(0, 0, p + "attn_q_b.weight", (nq, m.q_rank))], up(nq), self.off_c))
+        else:
+            self.off_c, name = nq, "attn_q"
+        n_in = self.off_c + m.kv_rank + m.rot_dim
+        self.w_in = Mat(src.pack([(0, 0, f"{p}{name}.weight", (m.q_rank or nq, w)), (self.off_c, 0, p + "attn_kv_a_mqa.weight", (m.kv_rank + m.rot_dim, w))], up(n_in), src.wp))
         self.w_o = Mat(src.pack([(0, 0, p + "attn_output.weight", (w, H * m.vdim))], src.wp, up(H * m.vdim)))
         self.c_norm = src.vec(p + "attn_kv_a_norm.weight", m.kv_rank)
         self.cp = up(m.kv_rank, 16)
@@ -198,51 +230,77 @@ class LatentAttention:
         self.uk[..., :m.kv_rank] = uk.view(H, m.dim, m.kv_rank)
         self.uv[:, :m.kv_rank] = uv
         self.freqs = torch.tensor(m.rot.freqs() if m.rot else [0.0], dtype=torch.float64, device=src.device)
-        self.interleaved = bool(m.rot and m.rot.interleaved)
+        self.interleaved, self.magnitude = (m.rot.interleaved, m.rot.magnitude) if m.rot else (False, 1.0)
         self.dp, self.rp, self.vp = up(m.dim, 64), up(m.rot_dim, 64), up(m.vdim, 64)
         self.w_kv = None
         if self.cache_type == torch.float16 and A.parts_supported(self.dp, self.rp, self.vp):
             self.w_kv = src.zeros(H * (self.dp + self.vp), self.cp)      # rows: every head's keys, then every head's values
             self.w_kv[:H * self.dp].view(H, self.dp, self.cp)[:, :m.dim] = self.uk
             self.w_kv[H * self.dp:].view(H, self.vp, self.cp)[:, :m.vdim] = self.uv.view(H, m.vdim, self.cp)
-        if not f32:
+        if not f32 and norm is not None:
             self.w_in.fold(norm)
 
     def product_weights(self) -> tuple[int, int, float]:
-        return sum(t.numel() for t in (self.w_in.w, self.uk, self.uv, self.w_o.w)), 0, 0.0
+        return sum(t.numel() for t in (self.w_in.w, self.uk, self.uv, self.w_o.w, *((self.w_uq.w,) if self.w_uq else ()))), 0, 0.0
 
     def make_cache(self, cache) -> tuple[torch.Tensor]:
         return (cache.add_pages(1, self.row, self.cache_type),)
 
     def run(self, s: Step, mem: tuple[torch.Tensor]) -> None:
-        m, (cache,), lp = self.m, mem, s.m.long
         qkv = s.buf("in", self.w_in.w.shape[0], torch.float32)
         s.normed(self.norm, self.w_in, qkv)
         out = s.buf("mix", self.w_o.w.shape[1], zero=True)
-        if lp is None or self.w_kv is None or s.decode:
-            self._latent(s, qkv, cache, out, s.nb, None, True)
-        else:
-            self._long(s, qkv, cache, out, lp)
-            if lp.rest is not None:
-                self._latent(s, qkv, cache, out, lp.rest.numel(), lp.rest, False)
+        self.mix(s, qkv, mem, out)
         s.add(out, self.w_o)
+
+    def project(self, s: Step, h: torch.Tensor, mem, **beside) -> torch.Tensor:
+        proj = s.buf("in", self.w_in.w.shape[0], torch.float32)
+        s.enter(h, self.w_in, proj, **beside)
+        return proj
+
+    def mix(self, s: Step, proj: torch.Tensor, mem: tuple[torch.Tensor], out: torch.Tensor) -> None:
+        (cache,), lp = mem, (s.m.long or {}).get(self.m.window)
+        qc = (self._queries(s, proj), proj[:, self.off_c:])
+        if lp is None or self.w_kv is None or s.decode:
+            self._latent(s, qc, cache, out, s.nb, None, True)
+        else:
+            self._long(s, qc, cache, out, lp)
+            if lp.rest is not None:
+                self._latent(s, qc, cache, out, lp.rest.numel(), lp.rest, False)
+
+    def _queries(self, s: Step, proj: torch.Tensor) -> torch.Tensor:
+        m, eps = self.m, s.be.stack.eps
+        if self.w_uq is None:
+            return proj
+        n, w = self.off_c, self.w_uq.w
+        q = s.buf("latent_q", w.shape[0], torch.float32)
+        if s.small:
+            O.gemv([O.seg(w, q.shape[1], q, self.q_norm)], n, proj, s.nb, s.be.f32, O.SRC_NORM, eps, m.q_rank, pdl=s.pdl)
+        else:
+            c = s.buf("latent_cq", n)
+            O.norm_rows(proj, m.q_rank, eps, self.q_norm, c, pdl=s.pdl)
+            O.gemm(c, w, q)
+            s.launched()
+        s.launched()
+        return q
 
     def _step_args(self, s: Step) -> dict:
         m = self.m
         return dict(heads=m.heads, dim=m.dim, rot=m.rot_dim, rank=m.kv_rank, norm=self.c_norm, eps=s.be.stack.eps, freqs=self.freqs, interleaved=self.interleaved,
-                    positions=s.m.positions, slots=s.m.slots, table=s.be.cache.table, cp=self.cp, pdl=s.pdl)
+                    positions=s.m.positions, slots=s.m.slots, table=s.be.cache.table, cp=self.cp, mscale=self.magnitude, pdl=s.pdl)
 
     def splits(self, n: int, n_ctx: int, sms: int) -> int:
         """Parts of the keys for ``n`` queries: as many CTAs as are resident (wide rows: one per SM), none shorter than a page."""
         groups = -(-self.m.heads // (16 if self.m.heads <= 16 else 32))
-        return max(1, min(-(-n_ctx // PAGE), (1 if self.row > 256 else 2) * sms // (groups * n), MAX_SPLITS))
+        keys = min(n_ctx, self.m.window + PAGE - 1) if self.m.window else n_ctx
+        return max(1, min(-(-keys // PAGE), (1 if self.row > 256 else 2) * sms // (groups * n), MAX_SPLITS))
 
-    def _latent(self, s: Step, qkv, cache, out, n: int, rows, append: bool) -> None:
+    def _latent(self, s: Step, qc, cache, out, n: int, rows, append: bool) -> None:
         """Attention of ``n`` rows in the latent space."""
-        m, dev, table = self.m, qkv.device, s.be.cache.table
+        m, dev, table = self.m, out.device, s.be.cache.table
         q = torch.empty(n, m.heads, self.row, device=dev, dtype=cache.dtype)
-        A.latent_step(qkv, n, cache=cache, rows=rows, append=append, uk=self.uk, q_out=q, **self._step_args(s))
-        at = dict(positions=s.m.positions, slots=s.m.slots, table=table, pdl=s.pdl)
+        A.latent_step(*qc, n, cache=cache, rows=rows, append=append, uk=self.uk, q_out=q, **self._step_args(s))
+        at = dict(positions=s.m.positions, slots=s.m.slots, table=table, window=m.window, pdl=s.pdl)
         splits, ml = self.splits(n, s.be.n_ctx, s.be.sms), None
         if cache.dtype == torch.float16:
             acc, ml = torch.empty(n, m.heads, splits, self.cp, device=dev), torch.empty(n, m.heads, splits, 2, device=dev)
@@ -255,18 +313,63 @@ class LatentAttention:
         A.latent_merge(acc, ml, n, self.uv, out, heads=m.heads, splits=splits, cp=self.cp, vdim=m.vdim, rows=rows, merged=merged, pdl=s.pdl)
         s.launched(3 + (merged is not None))
 
-    def _long(self, s: Step, qkv, cache, out, lp: LongPortions) -> None:
+    def _long(self, s: Step, qc, cache, out, lp: LongPortions) -> None:
         """Attention of the query tiles of ``lp`` over keys and values multiplied out of the latents; cache rows of the whole step."""
-        m, dev, H = self.m, qkv.device, self.m.heads
+        m, dev, H = self.m, out.device, self.m.heads
         q = torch.empty(s.nb, H, self.dp + self.rp, device=dev, dtype=torch.float16)
-        A.latent_step(qkv, s.nb, cache=cache, q_out=q, dp=self.dp, rp=self.rp, **self._step_args(s))
+        A.latent_step(*qc, s.nb, cache=cache, q_out=q, dp=self.dp, rp=self.rp, **self._step_args(s))
         c = torch.empty(lp.total, self.cp, device=dev, dtype=torch.bfloat16)
         r = torch.empty(lp.total, max(self.rp, 8), device=dev, dtype=torch.float16)
         A.latent_gather(cache, self.cp, m.rot_dim, lp.seqs, lp.longest, s.be.cache.table, c, r)
         kv = torch.empty(lp.total, self.w_kv.shape[0], device=dev, dtype=torch.float16)
         O.gemm(c, self.w_kv, kv)
-        A.attn_prefill_parts(q, kv, r, lp.tiles, out, heads=H, dp=self.dp, vp=self.vp, rp=self.rp, vdim=m.vdim, scale=m.scale)
+        A.attn_prefill_parts(q, kv, r, lp.tiles, out, heads=H, dp=self.dp, vp=self.vp, rp=self.rp, vdim=m.vdim, scale=m.scale, window=m.window)
         s.launched(4)
+
+
+class GatedRecurrence:
+    """Channels padded to whole vectors; the input product's rows are update gate, candidate and output gate."""
+
+    def __init__(self, src: WeightSource, p: str, m: GruMixer, f32: bool):
+        n, w, wp = m.width, src.width, up(m.width)
+        self.m, self.wp, self.f32 = m, wp, f32
+        bias = torch.zeros(3 * wp, device=src.device)
+        bias[:n], bias[wp:wp + n] = src.vec(p + "gru_z.bias", n)[:n], src.vec(p + "gru_x.bias", n)[:n]
+        self.w_in = Mat(src.pack([(i * wp, 0, f"{p}gru_{name}.weight", (n, w)) for i, name in enumerate(("z", "x", "gate"))], 3 * wp, src.wp), bias)
+        self.w_o = Mat(src.pack([(0, 0, p + "gru_out.weight", (w, n))], src.wp, wp))
+
+    def product_weights(self) -> tuple[int, int, float]:
+        return self.w_in.w.numel() + self.w_o.w.numel(), 0, 0.0
+
+    def make_cache(self, cache) -> tuple[torch.Tensor]:
+        return (cache.add_state(self.wp),)
+
+    def project(self, s: Step, h: torch.Tensor, mem, **beside) -> torch.Tensor:
+        proj = s.buf("gru", 3 * self.wp)
+        s.enter(h, self.w_in, proj, **beside)
+        return proj
+
+    def mix(self, s: Step, proj: torch.Tensor, mem: tuple[torch.Tensor], out: torch.Tensor) -> None:
+        if s.decode:
+            O.gru_step(proj, self.wp, mem[0], s.m.slots, s.m.positions, out, self.f32, pdl=s.pdl)
+        else:
+            O.gru_scan(proj, self.wp, mem[0], s.m.segs, out)
+        s.launched()
+
+
+class DenseFFN:
+    """Two matrices with an activation of single values between them, which may have two numbers of the layer's own."""
+
+    def __init__(self, src: WeightSource, p: str, m: DenseMLP):
+        self.act, self.ffp, self.nums = m.act, up(m.ff), O.NO_NUMS
+        if m.act == "xielu":
+            a, b = torch.nn.functional.softplus(src.tensor(p + "ffn_act.weight", 2).double()).tolist()
+            self.nums = (a, 0.5 + b)
+        self.up = Mat(src.pack([(0, 0, p + "ffn_up.weight", (m.ff, src.width))], self.ffp, src.wp))
+        self.down = Mat(src.pack([(0, 0, p + "ffn_down.weight", (src.width, m.ff))], src.wp, self.ffp))
+
+    def product_weights(self) -> tuple[int, int, float]:
+        return self.up.w.numel() + self.down.w.numel(), 0, 0.0
 
 
 class GatedFFN:
@@ -298,8 +401,9 @@ class _Shared:
 class ExpertFFN:
     """Mixture of experts; the experts stand stacked in one matrix each for gate / up and down.  The router's last row is the shared expert's gate where it has one."""
 
-    def __init__(self, src: WeightSource, p: str, m: ExpertMLP, norm: Norm, f32: bool, post: Norm | None = None):
+    def __init__(self, src: WeightSource, p: str, m: ExpertMLP, norm: Norm | None, f32: bool, post: Norm | None = None):
         w, E, n = src.width, m.experts, m.outputs
+        self.groups = ExpertGroups(m.groups, m.keep, m.scale) if m.scoring == "sigmoid" else A.NO_GROUPS
         self.m, self.norm, self.post, self.ffp, self.act = m, norm, post, up(m.expert.ff), "glu:" + m.act
         parts = [(0, 0, p + "ffn_gate_inp.weight", (n, w))]
         if m.shared is not None and m.shared_gate:
@@ -318,7 +422,7 @@ class ExpertFFN:
             both = Mat(gu, torch.cat([torch.zeros(n_gu, device=src.device), bias]) if bias is not None else None)
             self.shared = _Shared(m.shared, Mat(gu[:n_gu]), Mat(src.pack([(0, 0, p + "ffn_down_shexp.weight", (w, ff))], src.wp, up(ff))), both)
         self.router = Mat(router, bias)
-        if not f32 and norm.b is not None:
+        if not f32 and norm is not None and norm.b is not None:
             self.router.fold(norm)
 
     def product_weights(self) -> tuple[int, int, float]:
@@ -326,7 +430,7 @@ class ExpertFFN:
         return (self.router.w.numel() + (sh.gu.w.numel() + sh.down.w.numel() if sh else 0), self.gu.numel() + self.down.numel(), self.m.top / self.m.outputs)
 
     def run(self, s: Step) -> None:
-        m, sh, post, mult = self.m, self.shared, self.post, s.be.stack.residual_mult
+        m, sh, fs = self.m, self.shared, None
         z = s.buf("router", self.router.w.shape[0], torch.float32)
         both = sh is not None and not s.small and s.act == torch.bfloat16
         if both:
@@ -335,21 +439,31 @@ class ExpertFFN:
             s.launched()
         else:
             h = s.normed(self.norm, self.router, z, keep=True)
+        self.mix(s, h, z, fs)
+
+    def mix(self, s: Step, h: torch.Tensor, z: torch.Tensor, fs: torch.Tensor | None = None, beside: Mat | None = None, fill=None) -> None:
+        """The experts' part behind the router's product ``z``.  ``fs``: the shared expert's hidden columns where they exist already.  ``beside``: another part of the layer whose
+        last product is added in the same launch (a few rows; layers without a shared expert), ``fill(out)`` forms the columns it is multiplied with."""
+        m, sh, post, mult = self.m, self.shared, self.post, s.be.stack.residual_mult
+        both = fs is not None
         gate = z[:, m.outputs:m.outputs + 1] if sh and m.shared_gate else None
         out = s.x if post is None else s.buf("y", s.be.wp, torch.float32)
         if post is not None:
             mult = 1.0
         if s.small:
-            sfp = up(sh.e.ff) if sh else 0
+            tail = sh.down if sh else beside
+            sfp = tail.w.shape[1] if tail else 0
             a = s.buf("experts", m.top * self.ffp + sfp, zero=True)
             ids, wts = s.buf("ids", m.top, torch.int32), s.buf("weights", m.top)
+            if fill is not None:
+                fill(a[:, m.top * self.ffp:])
             A.moe_up_rows(z, h, s.nb, self.gu, 2 * m.expert.ff, a, ids, wts, experts=m.experts, top=m.top, ffp=self.ffp, limit=m.expert.limit, act=self.act, outputs=m.outputs,
-                          correction=self.correction, ws=sh.gu.w if sh else None, ns=2 * sh.e.ff if sh else 0, limit_s=sh.e.limit if sh else math.inf, pdl=s.pdl)
-            A.moe_down_rows(a, s.nb, ids, wts, self.down, out, top=m.top, n=s.be.stack.width, mult=mult, ws=sh.down.w if sh else None, store=post is not None, h=h, gate=gate,
+                          correction=self.correction, groups=self.groups, ws=sh.gu.w if sh else None, ns=2 * sh.e.ff if sh else 0, limit_s=sh.e.limit if sh else math.inf, pdl=s.pdl)
+            A.moe_down_rows(a, s.nb, ids, wts, self.down, out, top=m.top, n=s.be.stack.width, mult=mult, ws=tail.w if tail else None, store=post is not None, h=h, gate=gate,
                             pdl=s.pdl)
             s.launched(2)
         else:
-            ids, lids, wts = A.moe_route(z, m.outputs, m.top, m.experts, self.correction)
+            ids, lids, wts = A.moe_route(z, m.outputs, m.top, m.experts, self.correction, self.groups)
             row, tile_expert, rows = K.moe_plan(lids, m.experts)
             xs = K.moe_gather(h, row, m.top, rows)
             f = torch.empty(rows, self.ffp, device=h.device, dtype=s.act)

@@ -34,6 +34,7 @@ from ..ops import rows as O
 from .blocks import LONG_PORTION, ExpertFFN, GatedFFN, LatentAttention, LongPortions, Mat, Norm, SideInput, Step, WeightSource, make_norm, up
 from .cache import CacheFull, PagedCache
 from .mixers import HeadAttention, StateSpaceHeads
+from .shared import DepthAverage, SharedNormLayer
 from .steps import StepEngine
 
 MAX_DECODE_ROWS = 32
@@ -65,8 +66,9 @@ class _Rows:
 class _Meta:
     """Device arrays that describe the rows of a step."""
 
-    def __init__(self, tokens, positions, slots, offs=None, segs=None, tiles=None, long: LongPortions | None = None):
-        self.tokens, self.positions, self.slots, self.offs, self.segs, self.tiles, self.long = tokens, positions, slots, offs, segs, tiles, long
+    def __init__(self, tokens, positions, slots, offs=None, segs=None, tiles=None, half_tiles=None, long: dict[int, LongPortions] | None = None):
+        self.tokens, self.positions, self.slots, self.offs, self.segs, self.tiles, self.half_tiles = tokens, positions, slots, offs, segs, tiles, half_tiles
+        self.long = long              # by window (0: none)
 
 
 class StackBackend(StepEngine):
@@ -104,14 +106,14 @@ class StackBackend(StepEngine):
         def get(name: str) -> torch.Tensor:
             return (tensors[name] if tensors is not None else load_tensor(g, name)).dequant().to(dev)
 
-        src = WeightSource(get, dev, self.act_dtype, width)
+        src = WeightSource(get, dev, self.act_dtype, width, st.eps)
         vec, pack = src.vec, src.pack
         wp = self.wp
         self.embd = K.DevWeight(K.WT_F32 if self.f32 else K.WT_BF16, st.vocab, wp, [pack([(0, 0, "token_embd.weight", (st.vocab, width))], st.vocab, wp)])
         self.head = pack([(0, 0, "output.weight", (st.vocab, width))], _up8(st.vocab), wp)
-        self.loop_in = self.loop_step = self.side_table = None
+        self.loop_in = self.loop_step = self.side_table = self.depth = None
         self.layers: list[_Layer] = []
-        if not st.design.parallel:
+        if not st.design.paired:
             self._load_sequential(src)
             torch.cuda.synchronize(dev)
             return
@@ -179,7 +181,8 @@ class StackBackend(StepEngine):
         torch.cuda.synchronize(dev)
 
     def _load_sequential(self, src: WeightSource) -> None:
-        """Layers whose mixer and feed-forward follow one another, each behind a norm and, in some designs, under another one."""
+        """Layers made of the parts in blocks.py and mixers.py: mixer and feed-forward follow one another, each behind a norm and, in some designs, under another
+        one, or read one norm."""
         st, f32 = self.stack, self.f32
         norm = st.design.norm
         self.out_norm = make_norm(src, "output_norm", norm)
@@ -193,8 +196,12 @@ class StackBackend(StepEngine):
             n, d = len(st.layers), st.side_dim
             self.side_table = src.zeros(st.vocab, n, _up8(d))
             self.side_table[..., :d] = src.tensor("per_layer_token_embd.weight", st.vocab, n * d).view(st.vocab, n, d)
+        self.depth = DepthAverage(src, len(st.layers)) if st.design.depth_average else None
         for i, sl in enumerate(st.layers):
             L, p = _Layer(), f"blk.{i}."
+            if st.design.shared_norm:
+                self.layers.append(SharedNormLayer(src, p, sl, norm, f32))
+                continue
             pre = make_norm(src, p + "attn_norm", norm)
             post = make_norm(src, p + "post_attention_norm", norm) if st.design.post_norm else None
             if isinstance(sl.mixer, LatentMixer):
@@ -223,18 +230,18 @@ class StackBackend(StepEngine):
 
         def walk(o):
             if isinstance(o, torch.Tensor):
-                if o.data_ptr() not in seen:
-                    seen.add(o.data_ptr())
+                if o.untyped_storage().data_ptr() not in seen:           # matrices of several parts may be windows of one
+                    seen.add(o.untyped_storage().data_ptr())
                     yield o
             elif isinstance(o, (list, tuple)):
                 for v in o:
                     yield from walk(v)
             elif hasattr(o, "__dict__") and type(o).__module__.startswith(__package__):
                 yield from walk(list(vars(o).values()))
-        yield from walk([self.embd.planes[0], self.head, self.loop_in, self.loop_step, self.side_table, self.out_norm, self.layers])
+        yield from walk([self.embd.planes[0], self.head, self.loop_in, self.loop_step, self.side_table, self.out_norm, self.layers, self.depth])
 
     def weight_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self._weights())
+        return sum(t.untyped_storage().nbytes() for t in self._weights())
 
     def product_weights(self) -> tuple[int, int, float]:
         """Matrix weights over all layer runs and the head: (those every token is multiplied with, those of the routed experts, the share of
@@ -242,7 +249,7 @@ class StackBackend(StepEngine):
         dense, routed, share = self.head.numel(), 0, 0.0
         for r in self.runs:
             L = self.layers[r.layer]
-            if self.stack.design.parallel:
+            if self.stack.design.paired:
                 dense += sum(t.numel() for t in (L.w_in, L.up, L.w_out, getattr(L, "w_x", None), getattr(L, "w_dt", None)) if t is not None)
                 dense += self.loop_in.numel() if r.joins else 0
                 continue
@@ -263,8 +270,10 @@ class StackBackend(StepEngine):
         self.mem: list[tuple[torch.Tensor, torch.Tensor]] = []        # per layer run: (keys, values) or (state, convolution inputs)
         for r in self.runs:
             L = self.layers[r.layer]
-            if not self.stack.design.parallel:
-                self.mem.append(L.mix.make_cache(self.cache))
+            if not self.stack.design.paired:
+                j = getattr(L.mix.m, "kv_from", None)
+                kv = {} if j is None else {"kv": next(self.mem[k] for k in reversed(range(len(self.mem))) if self.runs[k].layer == j)}
+                self.mem.append(L.mix.make_cache(self.cache, **kv))
             elif isinstance(L.mixer, AttentionMixer):
                 self.mem.append((self.cache.add_pages(L.mixer.kv_heads, L.dk, kv_dt), self.cache.add_pages(L.mixer.kv_heads, L.dv, kv_dt)))
             else:
@@ -280,7 +289,7 @@ class StackBackend(StepEngine):
         b.sampled = torch.zeros(MB, device=dev, dtype=i32)
         b.host_in, b.host_out = torch.zeros(3, MB, dtype=i32).pin_memory(), torch.zeros(MB, dtype=i32).pin_memory()
         b.host_np, b.host_out_np = b.host_in.numpy(), b.host_out.numpy()
-        att = [L for L in self.layers if self.stack.design.parallel and isinstance(L.mixer, AttentionMixer) and L.hd]
+        att = [L for L in self.layers if self.stack.design.paired and isinstance(L.mixer, AttentionMixer) and L.hd]
         for L in att:       # split-K width of decode attention, by the most keys a query of the layer can see
             L.keys = min(n_ctx, L.mixer.chunk or n_ctx)
             L.n_splits = max(1, min(envconfig.attn_splits(), L.keys // envconfig.attn_split_len()))
@@ -413,14 +422,20 @@ class StackBackend(StepEngine):
 
     def _run_rows(self, B: _Rows, m: _Meta, nb: int, decode: bool, tap=None) -> torch.Tensor:
         """All layer runs on ``nb`` rows; ``tap(i, x)``: called after every run (inspection)."""
-        x = B.get("x", self.wp, torch.float32, nb, True)
+        hist = None
+        if self.depth is not None:
+            n = len(self.runs) + 2
+            hist = B.get("hist", n * self.wp, torch.float32, nb).view(n, nb, self.wp)
+        x = B.get("x", self.wp, torch.float32, nb, True) if hist is None else hist[0]
         K.embed(self.embd, m.tokens[:nb], self.stack.embed_scale, out=x)
         self._n += 1
         x0 = x
         if self.stack.loop is not None:
             x0 = B.get("x0", self.wp, torch.float32, nb, True)
             x0.copy_(x)
-        if not self.stack.design.parallel:
+        if hist is not None:
+            return self._run_depth(Step(self, B, m, x, x0, decode, hist), tap)
+        if not self.stack.design.paired:
             return self._run_sequential(Step(self, B, m, x, x0, decode), tap)
         for i in range(len(self.runs)):
             x = self._layer(i, x, x0, B, m, decode)
@@ -451,6 +466,17 @@ class StackBackend(StepEngine):
                 tap(i, s.x[:, :self.stack.width])
             s.pending.update(self._join(nxt, s))
         s.flush()
+        return s.x
+
+    def _run_depth(self, s: Step, tap=None) -> torch.Tensor:
+        """Layers that read a weighted sum of the embedding output and all earlier results; the output reads one too."""
+        w, n = self.depth.w, len(self.runs)
+        for i in range(n + 1):
+            h = s.average(i + 1, w[i], self.layers[self.runs[i].layer].norm if i < n else None)
+            if tap is not None and i > 0:
+                tap(i - 1, s.x[:, :self.stack.width])
+            if i < n:
+                self.layers[self.runs[i].layer].run(s, self.mem[i], h)
         return s.x
 
     def _head_rows(self, x: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
@@ -507,8 +533,10 @@ class StackBackend(StepEngine):
         total = sum(len(t) for _, t, _ in segs)
         cols = np.empty((4, total), np.int32)           # tokens | positions | slots | offset in the portion
         seg_rows, tiles, at = [], [], 0
-        latent = any(isinstance(L.mixer, LatentMixer) for L in self.stack.layers)
-        long_tiles, seqs, rest, keys = [], [], [], 0
+        windows = sorted({L.mixer.window for L in self.stack.layers if isinstance(L.mixer, LatentMixer)})
+        longs = {w: ([], [], []) for w in windows}          # tiles, sequences, positions of each
+        halves, rest = any(isinstance(L.mixer, AttentionMixer) and L.mixer.maps > 1 for L in self.stack.layers), []
+        half_tiles = []
         for slot, toks, p0 in segs:
             n = len(toks)
             cols[0, at:at + n] = toks
@@ -517,22 +545,30 @@ class StackBackend(StepEngine):
             cols[3, at:at + n] = np.arange(n)
             seg_rows.append((at, n, slot, p0))
             tiles += [(at + r, min(128, n - r), slot, p0 + r) for r in range(0, n, 128)]
-            if latent and n >= LONG_PORTION:
-                long_tiles += [(at + r, min(128, n - r), keys, p0 + r) for r in range(0, n, 128)]
-                seqs.append((keys, p0 + n, slot, 0))
-                keys += p0 + n
-            else:
+            if halves:
+                half_tiles += [(at + r, min(64, n - r), slot, p0 + r) for r in range(0, n, 64)]
+            if n < LONG_PORTION:
                 rest += range(at, at + n)
+            else:
+                for w, (lt, seqs, count) in longs.items():
+                    first = max(0, p0 - w + 1) & ~127 if w else 0       # keys are visited in tiles of 128 positions
+                    row0 = sum(count) - first
+                    lt += [(at + r, min(128, n - r), row0, p0 + r) for r in range(0, n, 128)]
+                    seqs.append((row0, p0 + n, slot, first))
+                    count.append(p0 + n - first)
             at += n
         np.maximum(cols[0], 0, out=cols[0])
         meta = torch.from_numpy(cols).to(dev)
-        geom = torch.tensor(seg_rows + tiles + long_tiles + seqs, dtype=torch.int32).to(dev)
+        lists = [seg_rows, tiles, half_tiles, *(t for lt, seqs, _ in longs.values() for t in (lt, seqs))]
+        geom = torch.tensor([r for t in lists for r in t], dtype=torch.int32).to(dev)
         self.h2d_bytes += 4 * (meta.numel() + geom.numel())
-        long, n1, n2 = None, len(segs) + len(tiles), len(segs) + len(tiles) + len(long_tiles)
-        if seqs:
-            long = LongPortions(geom[n1:n2], geom[n2:], keys, max(q[1] for q in seqs), torch.tensor(rest, dtype=torch.int32).to(dev) if rest else None)
+        parts = list(torch.split(geom, [len(t) for t in lists]))
+        long = None
+        if windows and len(rest) < total:
+            rows = torch.tensor(rest, dtype=torch.int32).to(dev) if rest else None
             self.h2d_bytes += 4 * len(rest)
-        m = _Meta(meta[0], meta[1], meta[2], meta[3], geom[:len(segs)], geom[len(segs):n1], long)
+            long = {w: LongPortions(parts[3 + 2 * i], parts[4 + 2 * i], sum(count), max(count), rows) for i, (w, (_, _, count)) in enumerate(longs.items())}
+        m = _Meta(meta[0], meta[1], meta[2], meta[3], *parts[:2], parts[2] if halves else None, long)
         self._n = 0
         out = self._run_rows(_Rows(at, dev), m, at, decode=False, tap=tap)
         self.kernel_launches += self._n

@@ -254,7 +254,7 @@ def test_absorbed_queries_and_cache_rows(ops, rank, cache32):
         for inter in (True, False):
             cache = torch.full((5, 1, 64, w), 7.0, device="cuda", dtype=torch.float32 if cache32 else torch.float16)
             q = torch.zeros(n, H, w, device="cuda", dtype=cache.dtype)
-            A.latent_step(qkv, n, heads=H, dim=d, rot=rot, rank=rank, norm=norm, eps=eps, freqs=freqs, interleaved=inter, positions=pos, slots=slots, table=table,
+            A.latent_step(qkv, qkv[:, H * (d + rot):], n, heads=H, dim=d, rot=rot, rank=rank, norm=norm, eps=eps, freqs=freqs, interleaved=inter, positions=pos, slots=slots, table=table,
                           cache=cache, cp=cp, uk=uk, q_out=q)
             tol = 1e-5 if cache32 else 1e-3
             x = qkv.double().cpu()
@@ -278,7 +278,7 @@ def test_absorbed_queries_and_cache_rows(ops, rank, cache32):
             if not cache32:                                                     # the long form: queries as they are, the same cache rows
                 again, dp, rp = torch.full_like(cache, 7.0), 24, 10
                 q = torch.full((n, H, dp + rp), 9.0, device="cuda", dtype=torch.float16)
-                A.latent_step(qkv, n, heads=H, dim=d, rot=rot, rank=rank, norm=norm, eps=eps, freqs=freqs, interleaved=inter, positions=pos, slots=slots, table=table,
+                A.latent_step(qkv, qkv[:, H * (d + rot):], n, heads=H, dim=d, rot=rot, rank=rank, norm=norm, eps=eps, freqs=freqs, interleaved=inter, positions=pos, slots=slots, table=table,
                               cache=again, cp=cp, q_out=q, dp=dp, rp=rp)
                 assert torch.equal(again, cache)
                 close(q[..., :d], qs[..., :d], tol)

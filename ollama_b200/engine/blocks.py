@@ -29,7 +29,7 @@ def up(n: int, m: int = 8) -> int:
 class WeightSource:
     """Named tensors of a model as zero-padded matrices and vectors on the device."""
 
-    def __init__(self, get, device, act_dtype, width: int, eps: float):
+    def __init__(self, get, device, act_dtype, width: int, eps: float = 0.0):
         self._get, self.device, self.act_dtype, self.width, self.wp, self.eps = get, device, act_dtype, width, up(width), eps
 
     def tensor(self, name: str, *shape: int) -> torch.Tensor:

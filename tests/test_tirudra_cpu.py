@@ -93,8 +93,8 @@ def test_configuration():
     assert [type(L.mixer) for L in st.layers] == [AttentionMixer, Mamba2Mixer, AttentionMixer, Mamba2Mixer, AttentionMixer, AttentionMixer]
     assert [type(L.mlp) for L in st.layers] == [ExpertMLP, type(None), ExpertMLP, ExpertMLP, type(None), type(None)]
     a, f = st.layers[0].mixer, st.layers[2].mixer
-    assert (a.window, a.keep, a.chunk, a.conv, a.gate, a.qk_norm, a.bias, a.keys_as_values, a.n_gate, a.n_v) == (37, 3, 0, 4, "element", "head", False, False, 4 * 28, 2 * 28)
-    assert (f.window, f.keep, f.conv, f.gate, f.bias, f.keys_as_values, f.n_gate, f.n_v) == (0, 0, 0, "head", True, True, 6, 0)
+    assert (a.window, a.keep, a.chunk, a.conv, a.gate, a.qk_norm, a.bias, a.keys_as_values, a.n_gate, a.n_v) == (37, 3, 0, 4, "element", "head", "", False, 4 * 28, 2 * 28)
+    assert (f.window, f.keep, f.conv, f.gate, f.bias, f.keys_as_values, f.n_gate, f.n_v) == (0, 0, 0, "head", "qk", True, 6, 0)
     assert a.rot.yarn == (3.0, 90.0, 9.0, 0.7) and a.rot.scaling is None and f.rot.scaling == (5.0, 1.0, 3.5, 70.0) and f.rot.magnitude == 1.0
     e = st.layers[0].mlp
     assert (e.experts, e.top, e.identity, e.outputs, e.act, e.scoring, e.router_bias, e.correction, e.shared_gate) == (6, 3, 2, 8, "silu", "all", False, True, True)

@@ -209,7 +209,7 @@ def main() -> None:
                     help="N > 1: tp = tensor/expert parallel ranks (default), pp = layer pipeline driven by rank 0 (the reference's multi-GPU mode)")
     ap.add_argument("--kv-type", default="f16", choices=["f16", "q8_0"], help="K/V cache encoding (OLLAMA_KV_CACHE_TYPE)")
     ap.add_argument("--layers", type=int, default=0, help="truncate the model to this many layers (profiling only; not a benchmark number)")
-    ap.add_argument("--stack", action="store_true", help="another workload: stack models (vazatar-1b / 8b, kavenex-1b / 8b / moe, tirudra-2k / 4k) beside models of equal size, bf16, one GPU")
+    ap.add_argument("--stack", action="store_true", help="another workload: stack models (vazatar-1b / 8b, kavenex-1b / 8b / moe, tirudra-2k / 4k, rinirax-1b / 8b / 2k) beside models of equal size, bf16, one GPU")
     args = ap.parse_args()
     if args.stack and args.impl != "reference":
         from ollama_b200.bench.stack_bench import run

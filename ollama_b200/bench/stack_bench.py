@@ -16,7 +16,7 @@ import statistics
 import torch
 
 PAIRS = {"vazatar-1b": "dense-1b", "vazatar-8b": "dense-8b", "kavenex-1b": "dense-1b", "kavenex-8b": "dense-8b", "kavenex-moe": "experts-2k", "tirudra-2k": "experts-2k",
-         "tirudra-4k": "experts-4k"}
+         "tirudra-4k": "experts-4k", "rinirax-1b": "dense-1b", "rinirax-8b": "dense-8b", "rinirax-2k": "experts-2k"}
 PROMPT, CONTEXT, BATCHES, LOOP = 2048, 1024, (1, 4, 16), 32
 
 

@@ -319,7 +319,30 @@ def heads_config(width: int, heads: int, kv_heads: int, dim: int, window: int, f
             "layers": [{**mix[c.upper()], "mlp": moe if c.isupper() else None} for c in layers]}
 
 
+def shared_norm_config(width: int, heads: int, kv_heads: int, dim: int, gru: int, rank: int, q_rank: int, window: int, ff: int, vocab: int, layers: str, experts: int = 0, top: int = 0,
+                       ff_expert: int = 0, groups: int = 1, keep: int = 1) -> dict:
+    """``config.json`` of a Rinirax model; ``layers``: one letter per layer, A (differential attention), S (the same on the keys and values of the last A), G (gated recurrence), L (latent
+    attention), followed by d for a dense feed-forward, e for experts or - for none."""
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "conv": 4, "diff": 0.5, "scale": (dim // 2) ** -0.5, "rot": {"base": 500000.0, "dims": dim // 2}}
+    lat = {"heads": heads, "dim": dim, "rot_dim": 64, "vdim": dim, "kv_rank": rank, "q_rank": q_rank, "mask": {"size": window}, "scale": (dim + 64) ** -0.5,
+           "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mix = {"A": ("attention", att), "G": ("mingru", {"width": gru}), "L": ("latent_attention", lat)}
+    mlp = {"d": {"kind": "dense", "ff": ff}, "-": None,
+           "e": {"kind": "moe", "expert": {"ff": ff_expert}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}, "scale": 2.0}}}
+    out: list[dict] = []
+    for i in range(0, len(layers), 2):
+        c, f = layers[i:i + 2]
+        source = layers[:i:2].rfind("A")
+        kind, m = ("attention", {**att, "kv_from": source}) if c == "S" else mix[c]
+        out.append({"type": kind, "mixer": m, "mlp": mlp[f]})
+    return {"architecture": "Rinirax", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": out}
+
+
 STACK_SPECS: dict[str, dict] = {
+    "tiny-rinirax": shared_norm_config(192, 6, 2, 64, 136, 80, 64, 40, 384, 4096, "AdGeLeSe", 6, 2, 96, 3, 2),
+    "rinirax-1b": shared_norm_config(2048, 16, 4, 128, 2048, 512, 768, 1024, 8192, 32768, "AdGdLdSd" * 4),
+    "rinirax-8b": shared_norm_config(4096, 32, 8, 128, 4096, 512, 1536, 1024, 16384, 128256, "AdGdLdSd" * 8),
+    "rinirax-2k": shared_norm_config(2048, 16, 4, 128, 2048, 512, 768, 1024, 8192, 32768, "AeGeLeSe" * 5, 64, 4, 1408, 8, 4),
     "tiny-tirudra": heads_config(192, 6, 2, 48, 40, 3, 12, 16, 40, 3, 4096, "MWFm", 6, 3, 1, 96, 80),
     "tirudra-2k": heads_config(2048, 16, 4, 128, 1024, 4, 64, 64, 128, 2, 32768, "MWMF" * 5, 64, 4, 4, 1408, 1408),
     "tirudra-4k": heads_config(4096, 32, 8, 128, 1024, 8, 128, 64, 128, 8, 65536, "MWMF" * 3, 32, 4, 2, 2048, 2048),
@@ -339,6 +362,7 @@ class SyntheticStackTensors:
     def __init__(self, cfg: dict, seed: int = 0, device="cpu"):
         from ..convert.stack import map_stack_name
         self.seed, self.device, w = seed, device, cfg["width"]
+        shared = cfg["architecture"] == "Rinirax"    # one norm per layer, averages over depth
         names: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], w), "head": (cfg["vocab"], w), "final.norm": (w,)}
         seq = cfg["architecture"] == "Kavenex"       # layer norms, gated feed-forwards, a loop that begins with sums
         post = cfg["architecture"] == "Tirudra"      # norms behind every part, a correction of the router and a gate of the shared expert instead of a bias
@@ -352,13 +376,22 @@ class SyntheticStackTensors:
             m, p = L["mixer"], f"l{i}."
             names.update({p + "norm1": (w,), **({p + "norm1b": (w,)} if post else {})})
             if L["type"] == "latent_attention":
-                H, d, r, dv, k = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-                names.update({p + "mix.q": (H * (d + r), w), p + "mix.dkv": (k + r, w), p + "mix.dkv.norm": (k,), p + "mix.uk": (H * d, k), p + "mix.uv": (H * dv, k),
+                H, d, r, dv, k, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m.get("q_rank")
+                names.update({p + "mix.dq": (rank, w), p + "mix.dq.norm": (rank,), p + "mix.uq": (H * (d + r), rank)} if rank else {p + "mix.q": (H * (d + r), w)})
+                names.update({p + "mix.dkv": (k + r, w), p + "mix.dkv.norm": (k,), p + "mix.uk": (H * d, k), p + "mix.uv": (H * dv, k),
                               p + "mix.o": (w, H * dv)})
             elif L["type"] == "mamba2":
                 H, c, bc = m["heads"], m["heads"] * m["vdim"], 2 * m["groups"] * m["state"]
                 names.update({p + "mix.in": (2 * c + bc + H, w), p + "mix.conv": (c + bc, m["conv"]), p + "mix.conv.b": (c + bc,), p + "mix.dt_bias": (H,), p + "mix.A_log": (H,),
                               p + "mix.D": (H,), p + "mix.norm": (c,), p + "mix.o": (w, c)})
+            elif L["type"] == "mingru":
+                n = m["width"]
+                names.update({p + "mix.z": (n, w), p + "mix.z.b": (n,), p + "mix.x": (n, w), p + "mix.x.b": (n,), p + "mix.g": (n, w), p + "mix.o": (w, n)})
+            elif shared:
+                n = {"q": 2 * m["heads"] * m["dim"], "k": 2 * m["kv_heads"] * m["dim"], "v": m["kv_heads"] * m["vdim"]}
+                for x in "q" if "kv_from" in m else "qkv":
+                    names.update({p + "mix." + x: (n[x], w), f"{p}mix.{x}.b": (n[x],), f"{p}mix.{x}.conv": (n[x], m["conv"])})
+                names.update({p + "mix.o": (w, m["heads"] * m["vdim"]), **{p + "mix." + x: (m["dim"],) for x in ("lq1", "lk1", "lq2", "lk2")}})
             elif post:
                 H, nq, nk, nv = m["heads"], m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
                 names.update({p + "mix.q": (nq, w), p + "mix.k": (nk, w), p + "mix.q.norm": (m["dim"],), p + "mix.k.norm": (m["dim"],), p + "mix.o": (w, H * m["vdim"])})
@@ -374,20 +407,22 @@ class SyntheticStackTensors:
                 names.update({p + "mix.in": (2 * c, w), p + "mix.conv": (c, m["conv"]), p + "mix.conv.b": (c,), p + "mix.x": (r + 2 * n, c), p + "mix.dt": (c, r),
                               p + "mix.dt.b": (c,), p + "mix.A_log": (c, n), p + "mix.D": (c,), p + "mix.o": (w, c)})
             f = L.get("mlp")
-            if f:
+            if shared:
+                names[p + "dwa"] = (i + 2,)
+            if f and not shared:
                 names.update({p + "norm2": (w,), **({p + "norm2b": (w,)} if post else {})})
             if f and f["kind"] == "dense":
-                names.update({p + "mlp.up": (f["ff"], w), p + "mlp.down": (w, f["ff"]), **({p + "mlp.gate": (f["ff"], w)} if seq else {})})
+                names.update({p + "mlp.up": (f["ff"], w), p + "mlp.down": (w, f["ff"]), **({p + "mlp.gate": (f["ff"], w)} if seq else {p + "mlp.act": (2,)} if shared else {})})
             elif f:
                 E, fe, fs = f["router"]["experts"], f["expert"]["ff"], (f.get("shared") or {}).get("ff")
                 n = E + f["router"].get("identity", 0)
-                names.update({p + "mlp.router": (n, w), **({p + "mlp.correction": (n,), p + "mlp.shared.sg": (1, w)} if post else {p + "mlp.router.b": (n,)})})
+                names.update({p + "mlp.router": (n, w), **({p + "mlp.correction": (n,)} if post or shared else {p + "mlp.router.b": (n,)}), **({p + "mlp.shared.sg": (1, w)} if post else {})})
                 for pre, fx in ((f"blk.{i}.ffn_%s_exps.weight", (E, fe)), (f"blk.{i}.ffn_%s_shexp.weight", (fs,))):
                     if fx[-1]:
                         stacked.update({pre % "gate": (*fx, w), pre % "up": (*fx, w), pre % "down": (*fx[:-1], w, fx[-1])})
             if side:
                 names.update({p + "side.gate": (side, w), p + "side.proj": (w, side), p + "side.norm": (w,)})
-        if seq:
+        if seq or shared:
             names.update({n + ".b": s for n, s in names.items() if n.endswith(("norm1", "norm2", "final.norm"))})
         self.table = {**{map_stack_name(n, cfg): s for n, s in names.items()}, **stacked}
 
@@ -403,6 +438,9 @@ class SyntheticStackTensors:
         x = random_tensor(name, s, self.seed, self.device)
         if name.endswith("ssm_a"):
             x = -(1.0 + torch.arange(s[-1], device=x.device, dtype=torch.float32)).expand(s).contiguous()
+        if name.endswith("depth_average.weight"):
+            x = 0.1 * torch.sin(torch.arange(s[0], device=x.device, dtype=torch.float32))
+            x[-1] = 1.0
         f32 = len(s) < 2 or name.endswith(("ssm_a", "conv1d.weight"))
         raw = (x if f32 else x.to(torch.bfloat16)).contiguous().view(-1).view(torch.uint8)
         return QWeight(name, GGMLType.F32 if f32 else GGMLType.BF16, tuple(s), raw)

@@ -121,10 +121,11 @@ def expert(h, gate, up, down, product=exact):
     return product(silu(product(h, gate)) * product(h, up), down)
 
 
-def moe_ff(h, w, m, product=exact):
+def moe_ff(h, w, m, product=exact, coarse=False):
+    """``coarse``: the router reads the input's bf16 rounding."""
     r = m["router"]
     gr = r.get("groups") or {"count": 1, "keep": 1}
-    idx, wt = route(h, w("router"), w("correction"), r["top"], gr["count"], gr["keep"], r.get("scale", 1.0))
+    idx, wt = route(h.bfloat16().to(h.dtype) if coarse else h, w("router"), w("correction"), r["top"], gr["count"], gr["keep"], r.get("scale", 1.0))
     out = torch.zeros_like(h)
     for e in range(r["experts"]):
         rows, place = (idx == e).nonzero(as_tuple=True)
@@ -138,8 +139,8 @@ def depth_average(history, weights):
 
 
 @torch.no_grad()
-def forward(cfg, weights, tokens, dtype=F64, residuals=None, product=exact):
-    """Logits [T, vocab] of a whole sequence; ``residuals``: a list that receives the stream after every layer."""
+def forward(cfg, weights, tokens, dtype=F64, residuals=None, product=exact, coarse=False):
+    """Logits [T, vocab] of a whole sequence; ``coarse``: see moe_ff; ``residuals``: a list that receives the stream after every layer."""
     W = {k: v.to(dtype) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     x = W["embed"][torch.as_tensor(list(tokens))]
@@ -154,7 +155,7 @@ def forward(cfg, weights, tokens, dtype=F64, residuals=None, product=exact):
         else:
             y = gru_mixer(h, w, product) if L["type"] == "mingru" else latent_mixer(h, w, m, eps, product)
         if L.get("mlp"):
-            y = y + (moe_ff(h, f, L["mlp"], product) if L["mlp"]["kind"] == "moe" else dense_ff(h, f, product))
+            y = y + (moe_ff(h, f, L["mlp"], product, coarse) if L["mlp"]["kind"] == "moe" else dense_ff(h, f, product))
         history.append(x + y)
         x = depth_average(history, W[p + "dwa"])
         if residuals is not None:

@@ -225,7 +225,7 @@ def greedy(cfg, w, prompt, n):
 
 @pytest.fixture(scope="module")
 def tiny():
-    cfg = M.config([M.diff(M.moe(4, 2, 8, 2, 1), heads=2, kv_heads=1, dim=8, vdim=12), M.gru(M.dense(12), width=10), M.latent(None, heads=2, dim=6, rot_dim=4, vdim=8, kv_rank=12, q_rank=8, size=9)], width=24, vocab=61)
+    cfg = M.config([M.diff(M.moe(4, 2, 8, 2, 1), heads=2, kv_heads=1, dim=8, vdim=12, rot={"base": 50.0, "dims": 6}), M.gru(M.dense(12), width=10), M.latent(None, heads=2, dim=6, rot_dim=4, vdim=8, kv_rank=12, q_rank=8, size=9)], width=24, vocab=61)
     return cfg, M.weights(cfg, 5)
 
 

@@ -208,7 +208,7 @@ class LatentAttention:
 
     def __init__(self, src: WeightSource, p: str, m: LatentMixer, norm: Norm | None, f32: bool):
         H, w = m.heads, src.width
-        self.m, self.norm, self.f32 = m, norm, f32
+        self.m, self.norm, self.f32, self.n_out = m, norm, f32, H * m.vdim
         nq = H * (m.dim + m.rot_dim)
         self.w_uq = self.q_norm = None
         if m.q_rank:
@@ -332,7 +332,7 @@ class GatedRecurrence:
 
     def __init__(self, src: WeightSource, p: str, m: GruMixer, f32: bool):
         n, w, wp = m.width, src.width, up(m.width)
-        self.m, self.wp, self.f32 = m, wp, f32
+        self.m, self.wp, self.f32, self.n_out = m, wp, f32, wp
         bias = torch.zeros(3 * wp, device=src.device)
         bias[:n], bias[wp:wp + n] = src.vec(p + "gru_z.bias", n)[:n], src.vec(p + "gru_x.bias", n)[:n]
         self.w_in = Mat(src.pack([(i * wp, 0, f"{p}gru_{name}.weight", (n, w)) for i, name in enumerate(("z", "x", "gate"))], 3 * wp, src.wp), bias)
@@ -353,7 +353,7 @@ class GatedRecurrence:
         if s.decode:
             O.gru_step(proj, self.wp, mem[0], s.m.slots, s.m.positions, out, self.f32, pdl=s.pdl)
         else:
-            O.gru_scan(proj, self.wp, mem[0], s.m.segs, out)
+            O.gru_scan(proj, self.wp, mem[0], s.m.segs, s.m.longest, out)
         s.launched()
 
 

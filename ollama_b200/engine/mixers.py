@@ -21,7 +21,7 @@ class HeadAttention:
 
     def __init__(self, src: WeightSource, p: str, m: AttentionMixer, norm: Norm | None, f32: bool, post: Norm | None):
         w, nq, nk, nv = src.width, m.n_q, m.n_k, m.n_v
-        self.m, self.norm, self.post, self.f32 = m, norm, post, f32
+        self.m, self.norm, self.post, self.f32, self.n_out = m, norm, post, f32, m.heads * m.vdim
         self.n8 = up(nq + nk + nv)                                       # the gate starts here
         n_in = self.n8 + up(m.n_gate)
         w_in, bias, self.conv_w = src.zeros(n_in, src.wp), torch.zeros(n_in, device=src.device) if m.bias else None, None

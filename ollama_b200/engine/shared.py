@@ -29,6 +29,7 @@ class SharedNormLayer:
         self.mix, self.ff, self.side, self.w_first, self.w_last = _mixer(src, p, layer.mixer, f32), None, None, None, None
         w_in, w_o = self.mix.w_in, self.mix.w_o
         self.mixp = w_o.w.shape[1]
+        self.pads = self.mixp != self.mix.n_out          # columns that nobody writes
         if isinstance(layer.mlp, DenseMLP):
             ff = self.ff = DenseFFN(src, p, layer.mlp)
             self.w_last = Mat(torch.cat([w_o.w, ff.down.w], 1))          # the parts' matrices become windows of it
@@ -62,12 +63,12 @@ class SharedNormLayer:
             else:
                 proj = mix.project(s, h, mem)
                 s.product(h, ff.router, z)
-            out = s.buf("mix", self.mixp, zero=True)
+            out = s.buf("mix", self.mixp, zero=self.pads)
             mix.mix(s, proj, mem, out)
             s.add(out, mix.w_o)
             ff.mix(s, h, z)
             return
-        cat = s.buf("cat", self.mixp + (ff.ffp if ff else 0), zero=True)
+        cat = s.buf("cat", self.mixp + (ff.ffp if ff else 0), zero=self.pads)
         segs = ()
         if ff is not None:
             f = cat[:, self.mixp:]

@@ -66,9 +66,10 @@ class _Rows:
 class _Meta:
     """Device arrays that describe the rows of a step."""
 
-    def __init__(self, tokens, positions, slots, offs=None, segs=None, tiles=None, half_tiles=None, long: dict[int, LongPortions] | None = None):
+    def __init__(self, tokens, positions, slots, offs=None, segs=None, tiles=None, half_tiles=None, long: dict[int, LongPortions] | None = None,
+                 longest: int = 1):
         self.tokens, self.positions, self.slots, self.offs, self.segs, self.tiles, self.half_tiles = tokens, positions, slots, offs, segs, tiles, half_tiles
-        self.long = long              # by window (0: none)
+        self.long, self.longest = long, longest      # by window (0: none); rows of the longest portion
 
 
 class StackBackend(StepEngine):
@@ -568,7 +569,7 @@ class StackBackend(StepEngine):
             rows = torch.tensor(rest, dtype=torch.int32).to(dev) if rest else None
             self.h2d_bytes += 4 * len(rest)
             long = {w: LongPortions(parts[3 + 2 * i], parts[4 + 2 * i], sum(count), max(count), rows) for i, (w, (_, _, count)) in enumerate(longs.items())}
-        m = _Meta(meta[0], meta[1], meta[2], meta[3], *parts[:2], parts[2] if halves else None, long)
+        m = _Meta(meta[0], meta[1], meta[2], meta[3], *parts[:2], parts[2] if halves else None, long, max(len(t) for _, t, _ in segs))
         self._n = 0
         out = self._run_rows(_Rows(at, dev), m, at, decode=False, tap=tap)
         self.kernel_launches += self._n

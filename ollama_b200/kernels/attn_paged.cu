@@ -190,32 +190,54 @@ struct PagedCombineArgs {
     DiffHeads diff;
 };
 
-// Split sums of head h of batch row b at column d.
+// Split sums of head h of batch row b at column d; the statistics and sums of several splits are requested together.
 __device__ __forceinline__ float merged_split(const PagedCombineArgs& a, int b, int h, int d) {
+    constexpr int BATCH = 8;
     const size_t p0 = ((size_t)b * a.n_heads + h) * a.n_splits;
-    float mn = -1e30f;
-    for (int s = 0; s < a.n_splits; s++) mn = fmaxf(mn, a.part_ml[p0 + s].x);
-    float o = 0.f, l = 0.f;
-    for (int s = 0; s < a.n_splits; s++) {
-        const float2 ml = a.part_ml[p0 + s];
-        const float c = __expf(ml.x - mn);
-        o += a.part_acc[(p0 + s) * a.hd + d] * c;
-        l += ml.y * c;
+    float mn = -1e30f, o = 0.f, l = 0.f;
+    for (int s0 = 0; s0 < a.n_splits; s0 += BATCH) {
+        float2 ml[BATCH];
+        float v[BATCH], top = mn;
+#pragma unroll
+        for (int i = 0; i < BATCH; i++) {
+            const bool in = s0 + i < a.n_splits;
+            ml[i] = in ? a.part_ml[p0 + s0 + i] : make_float2(-1e30f, 0.f);
+            v[i] = in ? a.part_acc[(p0 + s0 + i) * a.hd + d] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < BATCH; i++) top = fmaxf(top, ml[i].x);
+        const float c = __expf(mn - top);
+        o *= c;
+        l *= c;
+        mn = top;
+#pragma unroll
+        for (int i = 0; i < BATCH; i++) {
+            const float w = __expf(ml[i].x - mn);
+            o = fmaf(v[i], w, o);
+            l = fmaf(ml[i].y, w, l);
+        }
     }
     return l > 0.f ? o / l : 0.f;
 }
 
-__global__ void __launch_bounds__(128) paged_combine_kernel(const __grid_constant__ PagedCombineArgs a) {
-    const int h = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
+// 128 threads, with two maps of a head 256: a half each
+__global__ void __launch_bounds__(256) paged_combine_kernel(const __grid_constant__ PagedCombineArgs a) {
+    const int h = blockIdx.x, b = blockIdx.y, d = threadIdx.x & 127;
     pdl_launch();
     pdl_wait();
     float v;
-    if (a.diff.on) {                 // two maps of a head
-        __shared__ float red[4];
-        v = d < a.vdim ? merged_split(a, b, 2 * h, d) - a.diff.lambda * merged_split(a, b, 2 * h + 1, d) : 0.f;
-        const float s = warp_sum(v * v);
-        if ((d & 31) == 0) red[d >> 5] = s;
+    if (a.diff.on) {
+        __shared__ float red[4], second[128];
+        const int map = threadIdx.x >> 7;
+        v = d < a.vdim ? merged_split(a, b, 2 * h + map, d) : 0.f;
+        if (map) second[d] = v;
         __syncthreads();
+        v -= a.diff.lambda * second[d];
+        if (map) v = 0.f;
+        const float s = warp_sum(v * v);
+        if (!map && (d & 31) == 0) red[d >> 5] = s;
+        __syncthreads();
+        if (map) return;
         v *= a.diff.scale / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)a.vdim + a.diff.eps);
         if (d >= a.vdim) return;
     } else {
@@ -291,7 +313,7 @@ B2_API int b2_attn_decode_paged(const AttnDecodeArgs* a, const AttnRopeArgs* r, 
     if (e != cudaSuccess) return (int)e;
     PagedCombineArgs c{a->part_acc, a->part_ml, a->n_heads, a->n_splits, hd, r->vdim, out, ldo, out16, *gate, *diff};
     void* args[] = {&c};
-    return launch_rows((const void*)paged_combine_kernel, dim3(diff->on ? a->n_heads / 2 : a->n_heads, nb), dim3(128), 0, args, st, pdl);
+    return launch_rows((const void*)paged_combine_kernel, dim3(diff->on ? a->n_heads / 2 : a->n_heads, nb), dim3(diff->on ? 256 : 128), 0, args, st, pdl);
 }
 
 // The heads' results of differential attention from those of both maps, x [rows][H][2][vdim].

@@ -93,21 +93,26 @@ __device__ __forceinline__ float gelu_tanh_f(float v) {
     return EXACT ? v / (1.f + expf(z2)) : __fdividef(v, 1.f + __expf(z2));
 }
 
-// Activation of single values in a matrix product's epilogue: 0 none, 1 square of relu, 2 tanh form of gelu, 3 the expanded integral of elu with the layer's
-// two numbers: p v^2 + v / 2 above zero, q (exp(v) - 1 - v) + v / 2 below (without EXACT the difference keeps 2^-23 of 1, which vanishes beside v / 2).
-constexpr int ACT_LAST = 3;
+// Expanded integral of elu with two numbers of the layer: p v^2 + v / 2 above zero, q (exp(v) - 1 - v) + v / 2 below.  Without EXACT the difference keeps 2^-23 of
+// 1, which vanishes beside v / 2.
 template <bool EXACT = false>
-__device__ __forceinline__ float out_act(float v, int act, float p, float q) {
-    if (act == 3) {
-        const float n = fminf(v, 0.f);
-        return (v > 0.f ? p * v * v : q * ((EXACT ? expm1f(n) : __expf(n) - 1.f) - n)) + 0.5f * v;
-    }
+__device__ __forceinline__ float xielu_f(float v, float p, float q) {
+    const float n = fminf(v, 0.f);
+    return (v > 0.f ? p * v * v : q * ((EXACT ? expm1f(n) : __expf(n) - 1.f) - n)) + 0.5f * v;
+}
+
+// Activation of single values in a matrix product's epilogue: 0 none, 1 square of relu, 2 tanh form of gelu, ACT_XIELU with two numbers.
+constexpr int ACT_XIELU = 3, ACT_LAST = ACT_XIELU;
+template <bool EXACT = false>
+__device__ __forceinline__ float out_act(float v, int act) {
     if (act == 1) {
         const float r = fmaxf(v, 0.f);
         return r * r;
     }
     return act == 2 ? gelu_tanh_f<EXACT>(v) : v;
 }
+template <bool EXACT = false>
+__device__ __forceinline__ float out_act(float v, int act, float p, float q) { return act == ACT_XIELU ? xielu_f<EXACT>(v, p, q) : out_act<EXACT>(v, act); }
 
 // Epilogue activations of products whose rows 2i / 2i + 1 are gate / up of output i: GLU_BASE + the number glu_act takes.
 constexpr int GLU_BASE = 16;

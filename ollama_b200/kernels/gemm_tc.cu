@@ -107,12 +107,17 @@ __device__ __forceinline__ float4 fetch4(const GemmParams& p, int row, int col) 
     return make_float4(0.f, 0.f, 0.f, 0.f);
 }
 
-// Four consecutive sums of a row, as the product's caller wants them: activation or gated pairs, factors, type, accumulation.
+// Four consecutive sums of a row, as the product's caller wants them: activation or gated pairs, factors, type, accumulation.  XIELU: that activation and the
+// result's type, nothing else; without a branch the elements of several rows are under way together (with one the epilogue took longer than the products).
+template <bool XIELU = false>
 __device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, int col, const float4& with) {
-    if (p.act) {
-        r.x = out_act(r.x, p.act, p.act_p, p.act_q); r.y = out_act(r.y, p.act, p.act_p, p.act_q);
-        r.z = out_act(r.z, p.act, p.act_p, p.act_q); r.w = out_act(r.w, p.act, p.act_p, p.act_q);
+    if (XIELU) {
+        r.x = xielu_f(r.x, p.act_p, p.act_q); r.y = xielu_f(r.y, p.act_p, p.act_q); r.z = xielu_f(r.z, p.act_p, p.act_q); r.w = xielu_f(r.w, p.act_p, p.act_q);
+        if (p.out_bf16) *(uint2*)((__nv_bfloat16*)p.out + (size_t)row * p.ldo + col) = make_uint2(pack2_bf16(r.x, r.y), pack2_bf16(r.z, r.w));
+        else *(float4*)((float*)p.out + (size_t)row * p.ldo + col) = r;
+        return;
     }
+    if (p.act) { r.x = out_act(r.x, p.act); r.y = out_act(r.y, p.act); r.z = out_act(r.z, p.act); r.w = out_act(r.w, p.act); }
     if (p.mul) { r.x *= with.x; r.y *= with.y; r.z *= with.z; r.w *= with.w; }
     if (p.glu) {               // (gate, up, gate, up) -> two activated outputs
         const float h0 = glu_act(r.x, r.y, p.glu - 1, p.glu_alpha, p.glu_limit), h1 = glu_act(r.z, r.w, p.glu - 1, p.glu_alpha, p.glu_limit);
@@ -137,7 +142,7 @@ __device__ __forceinline__ void store4(const GemmParams& p, float4 r, int row, i
 }
 
 // TAIL: some columns are p.tail's.  A form of its own, since a test per stored element made all products 8 % longer.
-template <int BN, bool SPLIT, bool TAIL>
+template <int BN, bool SPLIT, bool TAIL, bool XIELU>
 __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                                                               const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -263,7 +268,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                 const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(buf * L::ACC_STRIDE + c0);
                 const int col = n0 + c0 + cq;
                 float4 with[8];
-                if (!SPLIT && (p.accumulate || p.mul)) {
+                if (!SPLIT && !XIELU && (p.accumulate || p.mul)) {
 #pragma unroll
                     for (int rr = 0; rr < 8; rr++) {
                         const int row = mt * BM + q * 32 + rr * 4 + sub;
@@ -302,7 +307,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tc_kernel(const __grid_const
                         continue;
                     }
                     r.x += bias.x; r.y += bias.y; r.z += bias.z; r.w += bias.w;
-                    store4(p, r, row, col, with[rr]);
+                    store4<XIELU>(p, r, row, col, with[rr]);
                 }
                 __syncwarp();
             }
@@ -333,32 +338,32 @@ int sm_count() {
     return n;
 }
 
-template <int BN, bool SPLIT = false, bool TAIL = false>
+template <int BN, bool SPLIT = false, bool TAIL = false, bool XIELU = false>
 int launch(const void* a, const void* b, const GemmParams& p, cudaStream_t st, int b_rows = 0) {
     CUtensorMap ma, mb;
     if (!make_map(&ma, a, p.m, p.k, BM, p.lda) || !make_map(&mb, b, b_rows ? b_rows : p.n, p.k, BN)) return (int)cudaErrorNotSupported;
     static PerDeviceOnce once;
-    if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN, SPLIT, TAIL>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
+    if (once.first()) cudaFuncSetAttribute(gemm_bf16_tc_kernel<BN, SPLIT, TAIL, XIELU>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<BN>::TOTAL);
     const int total = ((p.m + BM - 1) / BM) * ((p.n + BN - 1) / BN) * (SPLIT ? p.splits : 1);
     const int grid = total < sm_count() ? total : sm_count();
-    gemm_bf16_tc_kernel<BN, SPLIT, TAIL><<<grid, 192, Cfg<BN>::TOTAL, st>>>(ma, mb, p);
+    gemm_bf16_tc_kernel<BN, SPLIT, TAIL, XIELU><<<grid, 192, Cfg<BN>::TOTAL, st>>>(ma, mb, p);
     return (int)cudaGetLastError();
 }
 
-template <bool TAIL = false>
+template <bool TAIL = false, bool XIELU = false>
 int dispatch(const void* a, const void* b, const GemmParams& p, cudaStream_t st, int b_rows = 0) {
     // wide tiles once they fill the machine; narrower ones keep more SMs busy on small problems
     const long tiles_m = (p.m + BM - 1) / BM;
     // a handful of rows (a decode step of several sequences): the product streams b once, so the narrowest tile that spreads
     // b over the most SMs wins
     if (p.m <= 32 && (p.lda || (!p.out_bf16 && !p.glu)) && p.cm.n_dst == 0 && !b_rows && p.n >= 64 && (p.n + 127) / 128 < sm_count())
-        return p.splits > 1 ? launch<64, true>(a, b, p, st, b_rows) : launch<64, false, TAIL>(a, b, p, st, b_rows);
+        return p.splits > 1 ? launch<64, true>(a, b, p, st, b_rows) : launch<64, false, TAIL, XIELU>(a, b, p, st, b_rows);
     if (p.splits > 1) return p.n >= 128 ? launch<128, true>(a, b, p, st, b_rows) : launch<64, true>(a, b, p, st, b_rows);
-    if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256, false, TAIL>(a, b, p, st, b_rows);
+    if (p.n >= 256 && tiles_m * ((p.n + 255) / 256) >= sm_count()) return launch<256, false, TAIL, XIELU>(a, b, p, st, b_rows);
     // one round either way: the widest tile that still gives every SM at most one tile
-    if (p.n >= 192 && tiles_m * ((p.n + 191) / 192) <= sm_count() && tiles_m * ((p.n + 127) / 128) > sm_count()) return launch<192, false, TAIL>(a, b, p, st, b_rows);
-    if (p.n >= 128) return launch<128, false, TAIL>(a, b, p, st, b_rows);
-    return launch<64, false, TAIL>(a, b, p, st, b_rows);
+    if (p.n >= 192 && tiles_m * ((p.n + 191) / 192) <= sm_count() && tiles_m * ((p.n + 127) / 128) > sm_count()) return launch<192, false, TAIL, XIELU>(a, b, p, st, b_rows);
+    if (p.n >= 128) return launch<128, false, TAIL, XIELU>(a, b, p, st, b_rows);
+    return launch<64, false, TAIL, XIELU>(a, b, p, st, b_rows);
 }
 
 // Parts of a split product, added in order; bias, activation, factors, accumulation and output type of the whole.
@@ -375,6 +380,7 @@ __global__ void __launch_bounds__(256) gemm_parts_kernel(const __grid_constant__
         r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
     }
     if (p.tail && col >= p.tail_col) *(float4*)(p.tail + (size_t)row * p.ld_tail + col - p.tail_col) = r;
+    else if (p.act == ACT_XIELU) store4<true>(p, r, row, col, r);
     else store4(p, r, row, col, fetch4(p, row, col));
 }
 
@@ -435,8 +441,10 @@ B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
                  (const __nv_bfloat16*)g->mul, g->mul_row, g->ldm, (__nv_bfloat16*)g->copy, g->lda, g->tail, g->tail_col, g->ld_tail};
     p.act_p = g->act_p;
     p.act_q = g->act_q;
+    const bool xielu = p.act == ACT_XIELU;
+    if (xielu && (g->tile_expert || g->tail || g->mul || g->accumulate || g->copy || g->out_type > 1 || g->alpha != 1.f)) return (int)cudaErrorNotSupported;
     if (g->tile_expert) return dispatch(g->a, g->b, p, st, g->experts * n);
-    if (narrow(m, n, k)) return g->tail ? launch<64, false, true>(g->a, g->b, p, st) : launch<64>(g->a, g->b, p, st);
+    if (narrow(m, n, k)) return xielu ? launch<64, false, false, true>(g->a, g->b, p, st) : g->tail ? launch<64, false, true>(g->a, g->b, p, st) : launch<64>(g->a, g->b, p, st);
     const int splits = g->ws ? split_count(m, n, k) : 1;
     if (splits > 1 && (long long)splits * m * n <= g->ws_floats && m <= 65535) {
         p.splits = splits;
@@ -448,6 +456,7 @@ B2_API int b2_gemm_rows(const GemmRowsArgs* g, cudaStream_t st) {
         gemm_parts_kernel<<<dim3((n + 1023) / 1024, m), 256, 0, st>>>(p);
         return (int)cudaGetLastError();
     }
+    if (xielu) return dispatch<false, true>(g->a, g->b, p, st);
     return g->tail ? dispatch<true>(g->a, g->b, p, st) : dispatch(g->a, g->b, p, st);
 }
 

@@ -227,10 +227,10 @@ def depth_rows(hist: torch.Tensor, n: int, w: torch.Tensor, k: int, eps: float, 
     return x
 
 
-def gru_scan(x: torch.Tensor, off: int, state: torch.Tensor, segs: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
-    """Rows [z | u | gate], ``off`` columns apart, of prompt portions ``segs`` ([n, 4] int32: first row, rows, slot, position) through the gated recurrence."""
+def gru_scan(x: torch.Tensor, off: int, state: torch.Tensor, segs: torch.Tensor, longest: int, out: torch.Tensor, pdl: bool = False) -> None:
+    """Rows [z | u | gate], ``off`` columns apart, of prompt portions ``segs`` ([n, 4] int32: first row, rows, slot, position; ``longest``: the most rows of one) through the gated recurrence."""
     a = GruArgs(ptr(x), x.stride(0), off, 2 * off, state.shape[1], ptr(state), ptr(segs), None, None, ptr(out), out.stride(0))
-    _call("b2_gru_scan", a, segs.shape[0], _is32(x), int(pdl))
+    _call("b2_gru_scan", a, segs.shape[0], longest, _is32(x), int(pdl))
 
 
 def gru_step(x: torch.Tensor, off: int, state: torch.Tensor, slots, positions, out: torch.Tensor, exact: bool = False, pdl: bool = False) -> None:

@@ -187,7 +187,7 @@ def test_differential_attention_of_portions_and_decoded_tokens(shape, kind, rota
     a = Diff(H, G, dim, vdim, n, kind, dims if rotated else 0)
     a.aim(pairs_for(n))
     want = a.expected()
-    lo, tol = 0, TOL[kind] * (4 if vdim == 1 else 1)
+    lo, tol = 0, TOL[kind] * (20 if vdim == 1 else 1)      # a head of one value is little more than a sign
     for size in (200, 1, 2, 64, 63, 1):
         close(a.rows(lo, lo + size), want[lo:lo + size], tol)
         lo += size

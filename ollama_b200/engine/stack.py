@@ -7,7 +7,8 @@ matrix products; attention reads each sequence's pages, the state-space scan eac
               -> one product over [attention output | feed-forward hidden] with the residual add in its epilogue
 
 because W_o a + W_down f is one product over joined columns.  Layers whose mixer and feed-forward follow one another (engine/blocks.py, engine/mixers.py)
-take each norm into the product behind it, or into one pass with what is still to be added to the stream.  Decode steps of up to four sequences fuse the norms into a
+take each norm into the product behind it, or into one pass with what is still to be added to the stream.  Layers whose parts read one norm (engine/shared.py) share
+their first and last products.  Decode steps of up to four sequences fuse the norms into a
 multi-matrix GEMV (kernels/gemv_rows.cu), norm + rotation + cache append into the attention kernel, and the convolution and step-size
 projection into the products around the recurrence: four launches per layer plus the merge of the attention splits.  Larger steps and
 prompts multiply on the tcgen05 GEMM.  ``dtype`` "float32" runs weights, activations, cache and products in 32 bits.
